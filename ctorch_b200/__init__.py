@@ -4,6 +4,7 @@ another implementation: a missing library or a failing call raises."""
 from __future__ import annotations
 
 import ctypes as C
+import json
 import os
 
 import numpy as np
@@ -42,12 +43,42 @@ class QkvArgs(C.Structure):
                 ("q_up", C.c_void_p), ("v_up", C.c_void_p)]
 
 
+class ElementwiseNorm(C.Structure):
+    """Dynamic Tanh: tanh(alpha * x) * weight + bias, f32 device vectors."""
+    _fields_ = [("alpha", C.c_float), ("weight", C.c_void_p), ("bias", C.c_void_p)]
+
+
 class ShadowLinearArgs(C.Structure):
     _fields_ = [("x_hi", C.c_void_p), ("x_lo", C.c_void_p), ("rows", C.c_int64), ("inner", C.c_int64), ("weight", C.c_void_p),
                 ("out", C.c_int64), ("sumsq_in", C.c_void_p), ("parts_in", C.c_int32), ("eps", C.c_double), ("epilogue", C.c_int),
                 ("residual", C.c_void_p), ("qkv", C.POINTER(QkvArgs)), ("y", C.c_void_p), ("out_hi", C.c_void_p),
                 ("out_lo", C.c_void_p), ("out_norm_weight", C.c_void_p), ("out_norm_dtype", C.c_int32), ("sumsq_out", C.c_void_p),
-                ("best_value", C.c_void_p), ("best_index", C.c_void_p), ("y_copies", C.POINTER(C.c_void_p)), ("copies", C.c_int32)]
+                ("best_value", C.c_void_p), ("best_index", C.c_void_p), ("y_copies", C.POINTER(C.c_void_p)), ("copies", C.c_int32),
+                ("out_norm", C.POINTER(ElementwiseNorm))]
+
+
+class Rows(C.Structure):
+    """A packed pass: b200_rows."""
+    _fields_ = [("rows", C.c_int64), ("sequences", C.c_int32), ("max_count", C.c_int32), ("slot", C.c_void_p), ("first", C.c_void_p),
+                ("sequence", C.c_void_p), ("lengths", C.c_void_p)]
+
+
+class SsmArgs(C.Structure):
+    _fields_ = [("heads", C.c_int32), ("vdim", C.c_int32), ("state", C.c_int32), ("groups", C.c_int32), ("taps", C.c_int32),
+                ("conv_weight", C.c_void_p), ("conv_bias", C.c_void_p), ("dt_bias", C.c_void_p), ("a_log", C.c_void_p), ("d", C.c_void_p),
+                ("conv_state", C.c_void_p), ("ssm_state", C.c_void_p), ("projected", C.c_void_p), ("mixed", C.c_void_p), ("y", C.c_void_p)]
+
+
+class LatentArgs(C.Structure):
+    _fields_ = [("heads", C.c_int32), ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32), ("kv_rank", C.c_int32),
+                ("q_rank", C.c_int32), ("rot_dims", C.c_int32), ("scale", C.c_float), ("eps", C.c_double), ("cosine", C.c_void_p),
+                ("sine", C.c_void_p), ("positions", C.c_int32), ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("cache", C.c_void_p),
+                ("weight_dtype", C.c_int32), ("w_key", C.c_void_p), ("w_value", C.c_void_p)]
+
+
+class PassEntry(C.Structure):
+    _fields_ = [("slot", C.c_int64), ("tokens", C.POINTER(C.c_int64)), ("token_count", C.c_size_t), ("want", C.POINTER(C.c_int64)),
+                ("want_count", C.c_size_t)]
 
 
 class B200Error(RuntimeError):
@@ -121,6 +152,15 @@ def _declare(l: C.CDLL) -> None:
         "dl_onnx_save_decoder": (C.c_int, [C.c_char_p, vp, vp, vp]),
         "dl_decoder_generate": (C.c_int, [vp, vp, vp, vp, i64, vp, pp]),
         "dl_generation_profile_step": (C.c_int, [vp, C.POINTER(C.c_double)]),
+        "dl_model_architectures": (C.c_char_p, []), "dl_model_create": (C.c_int, [C.c_char_p, TensorOptions, pp]),
+        "dl_model_load": (C.c_int, [C.c_char_p, TensorOptions, pp]), "dl_state_load_safetensors": (C.c_int, [C.c_char_p, pp]),
+        "dl_model_cache_create": (C.c_int, [vp, i64, i64, pp]), "dl_model_cache_release_slot": (C.c_int, [vp, i64]),
+        "dl_model_cache_slot_length": (C.c_int, [vp, i64, C.POINTER(i64)]),
+        "dl_model_pass": (C.c_int, [vp, vp, C.POINTER(PassEntry), sz, vp]),
+        "dl_model_trail": (C.c_int, [vp, vp, C.POINTER(PassEntry), vp, sz]),
+        "dl_model_set_activation_dtype": (C.c_int, [vp, C.c_int]),
+        "dl_model_generation_create": (C.c_int, [vp, vp, i64, i64, pp]),
+        "dl_generation_prefill_lengths": (C.c_int, [vp, vp, C.POINTER(i64)]),
         "dl_b200_tp_unique_id": (C.c_int, [vp]), "dl_b200_tp_init": (C.c_int, [Device, i32, i32, vp]),
         "dl_b200_tp_finalize": (C.c_int, [Device]), "dl_b200_tp_set_push": (C.c_int, [Device, i32]),
         "dl_b200_tp_symmetric_handle": (C.c_int, [Device, sz, vp]), "dl_b200_tp_symmetric_open": (C.c_int, [Device, vp, i32]), "dl_transformer_decoder_set_tensor_parallel": (C.c_int, [vp, i32, i32]),
@@ -161,6 +201,19 @@ def _declare(l: C.CDLL) -> None:
         "b200_tp_reduce_shadow": (C.c_int, [pp, i32, i32, i32, sz, i32, i64, i64, vp, i32, vp, vp, vp, vp, vp]),
         "b200_argmax_finish": (C.c_int, [vp, vp, i32, i64, vp, vp, vp, i64, vp, pp, i32, vp]),
         "b200_scaled_add": (C.c_int, [vp, vp, C.c_float, i64, vp]),
+        "b200_gather_rows": (C.c_int, [vp, vp, i64, i64, vp, vp]),
+        "b200_rows_advance": (C.c_int, [C.POINTER(Rows), vp]),
+        "b200_embedding_scaled": (C.c_int, [vp, i32, vp, i64, i64, i64, C.c_float, vp, vp]),
+        "b200_dynamic_tanh": (C.c_int, [vp, vp, vp, i64, i64, C.POINTER(ElementwiseNorm), vp, vp, vp, vp, vp]),
+        "b200_ssm_forward": (C.c_int, [C.POINTER(SsmArgs), C.POINTER(Rows), vp]),
+        "b200_gated_group_norm": (C.c_int, [vp, vp, i64, vp, i64, i64, i32, C.c_double, vp, vp, vp, vp]),
+        "b200_latent_cache_create": (C.c_int, [i32, i32, i32, i32, i32, i32, vp, pp]),
+        "b200_latent_prepare": (C.c_int, [C.POINTER(LatentArgs), C.POINTER(Rows), vp, vp, vp, vp, vp]),
+        "b200_latent_query": (C.c_int, [C.POINTER(LatentArgs), C.POINTER(Rows), vp, vp, vp]),
+        "b200_latent_scratch_bytes": (sz, [C.POINTER(LatentArgs), i64, i32, i32, i32]),
+        "b200_latent_attention": (C.c_int, [C.POINTER(LatentArgs), C.POINTER(Rows), vp, i32, vp, sz, vp, vp]),
+        "b200_latent_value": (C.c_int, [C.POINTER(LatentArgs), i64, vp, vp, i64, vp, vp, vp, vp]),
+        "b200_latent_attention_kernel": (C.c_char_p, [C.POINTER(LatentArgs)]),
         "b200_take_device_status": (C.c_int, [i32, vp, C.POINTER(i32)]),
     }
     for name, (restype, argtypes) in sig.items():
@@ -239,6 +292,11 @@ class Tensor:
     def to(self, device: Device) -> "Tensor":
         out = C.c_void_p()
         check(lib().dl_to(self.h, device, C.byref(out)))
+        return Tensor(out)
+
+    def astype(self, dtype: int) -> "Tensor":
+        out = C.c_void_p()
+        check(lib().dl_astype(self.h, dtype, C.byref(out)))
         return Tensor(out)
 
     def select(self, axis: int, index: int) -> "Tensor":
@@ -467,12 +525,145 @@ class DecoderModel:
         return Tensor(out).numpy()
 
 
+class SlotCache:
+    """Sequence slots of a language model (or the caches of a grouped-query one)."""
+
+    def __init__(self, model: "LanguageModel", slots: int, capacity: int):
+        self.h = C.c_void_p()
+        check(lib().dl_model_cache_create(model.module.h, slots, capacity, C.byref(self.h)))
+
+    def release(self, slot: int) -> None:
+        check(lib().dl_model_cache_release_slot(self.h, slot))
+
+    def clear(self) -> None:
+        check(lib().dl_decoder_cache_clear(self.h))
+
+    def length(self, slot: int) -> int:
+        n = C.c_int64()
+        check(lib().dl_model_cache_slot_length(self.h, slot, C.byref(n)))
+        return n.value
+
+    def __del__(self):
+        try:
+            if self.h:
+                lib().dl_decoder_cache_release(self.h)
+                self.h = None
+        except Exception:
+            pass
+
+
+class LanguageModel:
+    """A model made from a configuration through the registry: `LanguageModel.load(folder)` reads config.json and
+    model.safetensors, `LanguageModel(config, weights)` takes them from memory."""
+
+    def __init__(self, config: dict, weights: dict[str, np.ndarray] | None = None, dtype: str = "bf16", device: int | None = 0):
+        module = C.c_void_p()
+        check(lib().dl_model_create(json.dumps(config).encode(), options(_code(dtype), cpu()), C.byref(module)))
+        self._adopt(Module(module), config, device)
+        if weights is not None:
+            state = {}
+            for name, tensor in self.module.state().items():
+                if name in weights:
+                    array = np.ascontiguousarray(weights[name])
+                    state[name] = Tensor.from_numpy(array, dtype=BF16 if array.dtype == np.uint16 else None)
+                    if state[name].dtype != tensor.dtype:
+                        state[name] = state[name].astype(tensor.dtype)
+                elif "rotary." in name:
+                    state[name] = tensor
+                else:
+                    raise KeyError(f"weight {name} is missing")
+            self.module.load_state(state)
+        if device is not None:
+            self.module.to(cuda(device))
+
+    @classmethod
+    def load(cls, folder: str, dtype: str = "bf16", device: int | None = 0) -> "LanguageModel":
+        with open(os.path.join(folder, "config.json")) as f:
+            config = json.load(f)
+        module = C.c_void_p()
+        where = cuda(device) if device is not None else cpu()
+        check(lib().dl_model_load(os.fsencode(folder), options(_code(dtype), where), C.byref(module)))
+        self = cls.__new__(cls)
+        self._adopt(Module(module), config, device)
+        return self
+
+    def _adopt(self, module: Module, config: dict, device: int | None) -> None:
+        self.module, self.config, self.device = module, config, device
+        self.dev = cuda(device) if device is not None else cpu()
+        self.vocab = config["vocab"]
+        self.cache: SlotCache | None = None
+
+    def new_cache(self, slots: int, capacity: int) -> SlotCache:
+        self.cache = SlotCache(self, slots, capacity)
+        return self.cache
+
+    def set_activation_dtype(self, dtype: str) -> None:
+        check(lib().dl_model_set_activation_dtype(self.module.h, _code(dtype)))
+
+    @staticmethod
+    def _entries(entries):
+        keep, array = [], (PassEntry * len(entries))()
+        ip = C.POINTER(C.c_int64)
+        for i, (slot, tokens, want) in enumerate(entries):
+            t, w = np.ascontiguousarray(tokens, dtype=np.int64), np.ascontiguousarray(want, dtype=np.int64)
+            keep += [t, w]
+            array[i] = PassEntry(slot, t.ctypes.data_as(ip), t.size, w.ctypes.data_as(ip), w.size)
+        return array, keep
+
+    def run(self, entries, cache: SlotCache | None = None) -> np.ndarray:
+        """One batched pass: entries of (slot, next tokens, wanted places); logits [wanted, vocabulary]."""
+        cache = cache or self.cache
+        array, keep = self._entries(entries)
+        out = np.empty((sum(len(w) for _, _, w in entries), self.vocab), dtype=np.float32)
+        check(lib().dl_model_pass(self.module.h, cache.h, array, len(entries), out.ctypes.data))
+        return out
+
+    def trail(self, slot: int, tokens, cache: SlotCache | None = None) -> np.ndarray:
+        """Residual stream [runs, tokens, width] after every layer run of one pass (hybrid decoders)."""
+        loop = self.config.get("loop") or {"start": 0, "stop": 0, "times": 1}
+        runs = len(self.config["layers"]) + (loop["times"] - 1) * (loop["stop"] - loop["start"])
+        out = np.empty((runs, len(tokens), self.config["width"]), dtype=np.float32)
+        array, keep = self._entries([(slot, tokens, [])])
+        check(lib().dl_model_trail(self.module.h, (cache or self.cache).h, array, out.ctypes.data, out.size))
+        return out
+
+    def generate(self, prompts, steps: int, temperature: float | None = None, seed: int = 0) -> np.ndarray:
+        """Continuations [batch, steps] of token-id prompts of any lengths: greedy, or sampled at a temperature."""
+        lengths = [len(p) for p in prompts]
+        longest = max(lengths)
+        self.new_cache(len(prompts), longest + steps)
+        padded = np.zeros((len(prompts), longest), dtype=np.int64)
+        for row, prompt in zip(padded, prompts):
+            row[:len(prompt)] = prompt
+        generation = Generation(self, len(prompts), steps)
+        generation.prefill(padded, lengths=None if len(set(lengths)) == 1 else lengths)
+        if temperature is None:
+            generation.step(steps - 1)
+        else:
+            draw = np.random.default_rng(seed)
+            for _ in range(steps - 1):
+                generation.step_sampled(temperature, draw.random(len(prompts)))
+        return generation.tokens()
+
+
+def architectures() -> list[str]:
+    return lib().dl_model_architectures().decode().split(",")
+
+
+def _code(dtype: str) -> int:
+    return {"bf16": BF16, "bfloat16": BF16, "f32": F32, "float32": F32}[dtype]
+
+
 class Generation:
-    def __init__(self, model: DecoderModel, batch: int, max_steps: int):
+    def __init__(self, model: "DecoderModel | LanguageModel", batch: int, max_steps: int):
         self.model = model
         g = C.c_void_p()
-        check(lib().dl_generation_create(model.decoder.h, model.embedding.h, model.output.h, model.cache, batch, max_steps,
-                                         C.byref(g)))
+        if isinstance(model, LanguageModel):
+            self._cache = model.cache   # borrowed by the library: kept alive here
+            check(lib().dl_model_generation_create(model.module.h, model.cache.h, batch, max_steps, C.byref(g)))
+        else:
+            check(lib().dl_generation_create(model.decoder.h, model.embedding.h, model.output.h, model.cache, batch, max_steps,
+                                             C.byref(g)))
         self.h = g
         self.batch = batch
 
@@ -484,9 +675,15 @@ class Generation:
         except Exception:
             pass
 
-    def prefill(self, prompt: np.ndarray, on_device: bool = False) -> None:
+    def prefill(self, prompt: np.ndarray, on_device: bool = False, lengths=None) -> None:
+        """Prompt ids [batch, length]; with `lengths` row b counts for its first lengths[b] ids and the rest is padding."""
         p = Tensor.from_numpy(np.asarray(prompt, dtype=np.int64), device=self.model.dev if on_device else cpu())
-        check(lib().dl_generation_prefill(self.h, p.h))
+        if lengths is None:
+            check(lib().dl_generation_prefill(self.h, p.h))
+        else:
+            counts = np.ascontiguousarray(lengths, dtype=np.int64)
+            assert counts.shape == (self.batch,)
+            check(lib().dl_generation_prefill_lengths(self.h, p.h, counts.ctypes.data_as(C.POINTER(C.c_int64))))
 
     def step(self, steps: int = 1) -> None:
         check(lib().dl_generation_step(self.h, steps))

@@ -12,6 +12,8 @@ with `-lctorch` and the headers under include/dl/ links against this directory u
 """
 from __future__ import annotations
 
+import contextlib
+import fcntl
 import os
 import subprocess
 import sys
@@ -48,6 +50,15 @@ def headers_mtime() -> float:
                 if name.endswith((".h", ".cuh", ".hpp")):
                     newest = max(newest, os.path.getmtime(os.path.join(base, name)))
     return newest
+
+
+@contextlib.contextmanager
+def lock():
+    """Serialises builds of one checkout by several processes."""
+    os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
 
 
 def build(force: bool = False, verbose: bool = False) -> str:

@@ -2,6 +2,7 @@
 // (the contract of the reference's src/api/common.h:53-69 and src/api/decoder.cpp:10-70).
 #include "ctorch_b200_c_api.h"
 #include "dl/dl.h"
+#include "dl/hybrid.h"
 #include "dl/internal.h"
 #include "dl/plan.h"
 
@@ -14,7 +15,11 @@
 struct dl_tensor { dl::Tensor value; };
 struct dl_module { std::shared_ptr<dl::nn::UnaryModule> value; };
 struct dl_state { dl::StateDict value; };
-struct dl_decoder_cache { std::vector<dl::nn::KVCache> value; };
+// Either the grouped-query decoder's caches (one per layer) or the slots of a hybrid decoder.
+struct dl_decoder_cache {
+    std::vector<dl::nn::KVCache> value;
+    std::shared_ptr<dl::nn::HybridCache> slots;
+};
 struct dl_generation { std::unique_ptr<dl::nn::Generation> value; };
 
 namespace {
@@ -281,11 +286,18 @@ dl_status dl_decoder_cache_create(const dl_module* decoder, dl_decoder_cache** o
 }
 void dl_decoder_cache_release(dl_decoder_cache* cache) { delete cache; }
 dl_status dl_decoder_cache_clear(dl_decoder_cache* cache) {
-    return invoke([&] { for (auto& layer : need(cache, "cache").value) layer.clear(); });
+    return invoke([&] {
+        if (need(cache, "cache").slots) cache->slots->clear();
+        for (auto& layer : cache->value) layer.clear();
+    });
 }
 dl_status dl_decoder_cache_truncate(dl_decoder_cache* cache, int64_t length) {
     return invoke([&] {
-        auto& layers = need(cache, "cache").value;
+        if (need(cache, "cache").slots) {
+            if (length != 0) throw std::invalid_argument("a recurrent state cannot be cut back: only truncation to 0 is possible");
+            return cache->slots->clear();
+        }
+        auto& layers = cache->value;
         for (const auto& layer : layers)
             if (length < 0 || length > layer.length()) throw std::out_of_range("KV cache truncation must keep an existing prefix");
         for (auto& layer : layers) layer.truncate(length);
@@ -294,7 +306,11 @@ dl_status dl_decoder_cache_truncate(dl_decoder_cache* cache, int64_t length) {
 dl_status dl_decoder_cache_length(const dl_decoder_cache* cache, int64_t* length) {
     return invoke([&] {
         if (!length) throw std::invalid_argument("length slot is NULL");
-        const auto& layers = need(cache, "cache").value;
+        if (need(cache, "cache").slots) {
+            *length = cache->slots->longest();
+            return;
+        }
+        const auto& layers = cache->value;
         *length = layers.empty() ? 0 : layers.front().length();
     });
 }
@@ -396,6 +412,98 @@ dl_status dl_decoder_generate(dl_module* decoder, dl_module* embedding, dl_modul
         generation.prefill(ids);
         generation.step(steps - 1);
         return generation.tokens().to(ids.device());
+    });
+}
+
+// ---- models from configurations -----------------------------------------------------------------------------------
+dl_status dl_model_create(const char* config_json, dl_tensor_options options, dl_module** output) {
+    return make_handle(output, [&] {
+        if (!config_json) throw std::invalid_argument("configuration is NULL");
+        return dl::models::create(dl::Json::parse(config_json), convert(options));
+    });
+}
+dl_status dl_model_load(const char* folder, dl_tensor_options options, dl_module** output) {
+    return make_handle(output, [&] {
+        if (!folder) throw std::invalid_argument("folder is NULL");
+        return dl::models::load(folder, static_cast<dl::DType>(options.dtype), convert(options.device));
+    });
+}
+const char* dl_model_architectures(void) {
+    static const std::string names = [] {
+        std::string joined;
+        for (const auto& name : dl::models::architectures()) joined += (joined.empty() ? "" : ",") + name;
+        return joined;
+    }();
+    return names.c_str();
+}
+dl_status dl_state_load_safetensors(const char* path, dl_state** output) {
+    return make_handle(output, [&] {
+        if (!path) throw std::invalid_argument("path is NULL");
+        return dl::io::load_safetensors(path);
+    });
+}
+dl_status dl_model_cache_create(const dl_module* model, int64_t slots, int64_t capacity, dl_decoder_cache** output) {
+    return make_handle(output, [&] {
+        const auto& module = need(model, "module").value;
+        if (auto hybrid = std::dynamic_pointer_cast<dl::nn::HybridDecoder>(module))
+            return dl_decoder_cache{{}, std::make_shared<dl::nn::HybridCache>(*hybrid, slots, capacity)};
+        if (auto lm = std::dynamic_pointer_cast<dl::nn::DecoderLanguageModel>(module)) return dl_decoder_cache{lm->decoder()->make_cache(), nullptr};
+        throw std::invalid_argument("module is not a language model");
+    });
+}
+dl_status dl_model_cache_release_slot(dl_decoder_cache* cache, int64_t slot) {
+    return invoke([&] {
+        if (!need(cache, "cache").slots) throw std::invalid_argument("the cache has no slots");
+        cache->slots->release(slot);
+    });
+}
+dl_status dl_model_cache_slot_length(const dl_decoder_cache* cache, int64_t slot, int64_t* length) {
+    return invoke([&] {
+        if (!need(cache, "cache").slots || !length) throw std::invalid_argument("the cache has no slots");
+        *length = cache->slots->length(slot);
+    });
+}
+dl_status dl_model_pass(dl_module* model, dl_decoder_cache* cache, const dl_pass_entry* entries, size_t count, float* logits) {
+    return invoke([&] {
+        auto& hybrid = as<dl::nn::HybridDecoder>(model, "HybridDecoder");
+        if (!need(cache, "cache").slots) throw std::invalid_argument("the cache has no slots");
+        if (count > 0 && !entries) throw std::invalid_argument("entries are NULL");
+        std::vector<dl::nn::PassEntry> list;
+        for (size_t i = 0; i < count; ++i)
+            list.push_back({entries[i].slot, {entries[i].tokens, entries[i].token_count}, {entries[i].want, entries[i].want_count}});
+        hybrid.pass(*cache->slots, list, logits);
+    });
+}
+dl_status dl_model_trail(dl_module* model, dl_decoder_cache* cache, const dl_pass_entry* entry, float* trail, size_t trail_floats) {
+    return invoke([&] {
+        auto& hybrid = as<dl::nn::HybridDecoder>(model, "HybridDecoder");
+        if (!need(cache, "cache").slots || !entry || !trail) throw std::invalid_argument("cache, entry or result is NULL");
+        const dl::nn::PassEntry one{entry->slot, {entry->tokens, entry->token_count}, {}};
+        std::vector<float> rows;
+        hybrid.pass(*cache->slots, {&one, 1}, nullptr, &rows);
+        if (rows.size() != trail_floats) throw std::invalid_argument("the result buffer needs " + std::to_string(rows.size()) + " floats");
+        std::copy(rows.begin(), rows.end(), trail);
+    });
+}
+dl_status dl_model_set_activation_dtype(dl_module* model, dl_dtype dtype) {
+    return invoke([&] { as<dl::nn::HybridDecoder>(model, "HybridDecoder").set_activation_dtype(static_cast<dl::DType>(dtype)); });
+}
+dl_status dl_model_generation_create(dl_module* model, dl_decoder_cache* cache, int64_t batch, int64_t max_steps, dl_generation** result) {
+    return make_handle(result, [&] {
+        const auto& module = need(model, "module").value;
+        auto& storage = need(cache, "cache");
+        if (auto hybrid = std::dynamic_pointer_cast<dl::nn::HybridDecoder>(module))
+            return std::make_unique<dl::nn::Generation>(dl::nn::make_token_model(hybrid, storage.slots), batch, max_steps);
+        if (auto lm = std::dynamic_pointer_cast<dl::nn::DecoderLanguageModel>(module))
+            return std::make_unique<dl::nn::Generation>(lm->decoder(), lm->tokens(), lm->output(), &storage.value, batch, max_steps);
+        throw std::invalid_argument("module is not a language model");
+    });
+}
+dl_status dl_generation_prefill_lengths(dl_generation* generation, const dl_tensor* prompt, const int64_t* lengths) {
+    return invoke([&] {
+        const auto& ids = need(prompt, "tensor").value;
+        if (!lengths) throw std::invalid_argument("lengths are NULL");
+        need(generation, "generation").value->prefill(ids, {lengths, static_cast<size_t>(ids.ndim() == 2 ? ids.size(0) : 0)});
     });
 }
 

@@ -366,12 +366,31 @@ private:
     std::unique_ptr<DecodePlan> plan_;
 };
 
+// Embedding, decoder and output layer as one module, under the names of the reference's example model
+// (examples/decoder_model.h:15-18): "tokens.weight", "decoder.*", and "output.weight" unless the table is tied.
+class DecoderLanguageModel : public UnaryModule {
+public:
+    DecoderLanguageModel(Index vocabulary, Index layers, Index dimensions, Index heads, Index kv_heads, Index hidden, Index context, bool tied,
+                         TensorOptions options = {});
+    Tensor forward(const Tensor& ids) override;   // [batch, length] -> logits [batch, length, vocabulary]
+    const std::shared_ptr<Embedding>& tokens() const { return tokens_; }
+    const std::shared_ptr<TransformerDecoder>& decoder() const { return decoder_; }
+    std::shared_ptr<Linear> output();
+private:
+    std::shared_ptr<Embedding> tokens_;
+    std::shared_ptr<TransformerDecoder> decoder_;
+    std::shared_ptr<Linear> output_;              // tied: a view of the table, remade when the table moves
+    bool tied_;
+    std::uint64_t tied_version_ = ~0ull;
+};
+
 }  // namespace nn
 
 // ---- include/dl/io.h of the reference: weight archives (".ct"), see checkpoint.cpp for the layout --------------
 namespace io {
 void save(const std::filesystem::path& path, std::span<const NamedTensor> state);
 StateDict load(const std::filesystem::path& path);   // tensors in host memory
+StateDict load_safetensors(const std::filesystem::path& path);   // tensors in host memory, in name order (safetensors.cpp)
 }  // namespace io
 
 // ---- extensions/onnx/include/dl/onnx.h:30-35 of the reference: the decoder with its KV cache as graph ports ----

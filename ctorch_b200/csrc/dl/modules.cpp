@@ -400,4 +400,20 @@ DecodePlan& TransformerDecoder::plan() {
 }
 Tensor TransformerDecoder::decode(const Tensor& input, std::span<KVCache> cache) { return plan().decode(input, cache); }
 
+DecoderLanguageModel::DecoderLanguageModel(Index vocabulary, Index layers, Index dimensions, Index heads, Index kv_heads, Index hidden,
+                                           Index context, bool tied, TensorOptions options)
+    : tied_(tied) {
+    tokens_ = add_module<Embedding>("tokens", vocabulary, dimensions, options);
+    decoder_ = add_module<TransformerDecoder>("decoder", layers, dimensions, heads, kv_heads, hidden, context, options);
+    if (!tied) output_ = add_module<Linear>("output", dimensions, vocabulary, false, options);
+}
+std::shared_ptr<Linear> DecoderLanguageModel::output() {
+    if (tied_ && (!output_ || tied_version_ != tokens_->version())) {
+        output_ = std::make_shared<Linear>(tokens_->weight());
+        tied_version_ = tokens_->version();
+    }
+    return output_;
+}
+Tensor DecoderLanguageModel::forward(const Tensor& ids) { return output()->forward(decoder_->forward(tokens_->forward(ids))); }
+
 }  // namespace dl::nn

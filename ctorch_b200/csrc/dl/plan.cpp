@@ -25,7 +25,6 @@ struct StepProbe {
     }
 };
 thread_local StepProbe* step_probe = nullptr;
-void probe(int kind) { if (step_probe) step_probe->mark(kind); }
 
 int code_of(DType dtype) { return dtype == DType::bf16 ? B200_BF16 : B200_F32; }
 
@@ -44,6 +43,8 @@ void copy_rows(void* dst, std::size_t dst_pitch, const Tensor& src, int device) 
 }
 
 }  // namespace
+
+void probe(int kind) { if (step_probe) step_probe->mark(kind); }
 
 Tensor interleave_rows(const Tensor& even_rows, const Tensor& odd_rows) {
     require_cuda(even_rows, "interleave_rows");
@@ -560,25 +561,126 @@ Tensor DecodePlan::decode(const Tensor& input, std::span<KVCache> cache) {
     return result;
 }
 
-// ---- Generation -----------------------------------------------------------------------------------------
-Generation::Generation(std::shared_ptr<TransformerDecoder> decoder, std::shared_ptr<Embedding> tokens, std::shared_ptr<Linear> output,
-                       std::vector<KVCache>* cache, Index batch, Index max_steps)
-    : decoder_(std::move(decoder)), tokens_(std::move(tokens)), output_(std::move(output)), cache_(cache), batch_(batch),
-      max_steps_(max_steps) {
+// ---- DecoderTokenModel ------------------------------------------------------------------------------------
+DecoderTokenModel::DecoderTokenModel(std::shared_ptr<TransformerDecoder> decoder, std::shared_ptr<Embedding> tokens,
+                                     std::shared_ptr<Linear> output, std::vector<KVCache>* cache)
+    : decoder_(std::move(decoder)), tokens_(std::move(tokens)), output_(std::move(output)), cache_(cache) {
     if (!decoder_ || !tokens_ || !output_ || !cache_) throw std::invalid_argument("generation needs a decoder, an embedding, an output layer and a cache");
-    if (batch <= 0 || max_steps <= 0) throw std::invalid_argument("generation needs a positive batch and step budget");
     require_cuda(tokens_->weight(), "generation");
     if (tokens_->weight().size(1) != decoder_->dimensions() || output_->weight().size(1) != decoder_->dimensions())
         throw std::invalid_argument("embedding and output widths must equal the decoder's dimensions");
     device_ = tokens_->weight().device().index;
+}
+
+std::vector<b200_kv_cache*> DecoderTokenModel::handles() const {
+    std::vector<b200_kv_cache*> result;
+    for (auto& layer : *cache_) result.push_back(layer.handle());
+    return result;
+}
+
+void DecoderTokenModel::reserve_rows(Index batch) {
+    if (x_.defined() && x_.size(0) == batch) return;
+    x_ = empty({batch, decoder_->dimensions()}, {DType::f32, Device::cuda(device_)});
+    ++x_epoch_;
+}
+
+void DecoderTokenModel::prefill(const Tensor& prompt, std::span<const Index> lengths, float* logits) {
+    const Index batch = prompt.size(0), P = prompt.size(1), D = decoder_->dimensions();
+    void* stream = runtime::stream(device_);
+    auto& plan = decoder_->plan();
+    reserve_rows(batch);
+    const Index before = cache_->front().length();
+    // Chunked prefill: at most ~8192 rows per pass; chunked decode equals one pass (tests/state.cpp:54-63 of the reference).
+    const Index chunk = std::max<Index>(1, std::min<Index>(P, 8192 / batch > 0 ? 8192 / batch : 1));
+    Tensor features = empty({batch * chunk, D}, {DType::f32, Device::cuda(device_)});
+    const auto caches = handles();
+    Index done = 0;
+    while (done < P) {
+        const Index count = std::min(chunk, P - done);
+        const Tensor part = count == P ? prompt : prompt.narrow(1, done, count);
+        runtime::check(b200_embedding(tokens_->weight().raw_data(), code_of(tokens_->weight().dtype()), part.data<Index>(), batch * count,
+                                      tokens_->weight().size(0), D, static_cast<float*>(features.mutable_data()), stream), "embedding");
+        const Index max_length = cache_->front().length() + count;
+        plan.reserve(batch * count, max_length, device_);
+        plan.run_layers(features.data<float>(), batch, count, *cache_, max_length, stream);
+        runtime::check(b200_kv_cache_advance(caches.data(), static_cast<int32_t>(caches.size()), static_cast<int32_t>(count), stream), "KV advance");
+        for (auto& layer : *cache_) layer.commit(count);
+        if (lengths.empty()) {
+            if (done + count == P)
+                runtime::check(b200_select_rows(plan.hidden(), count - 1, count, batch, D, static_cast<float*>(x_.mutable_data()), stream), "select");
+        } else {   // the last token of a shorter prompt may lie in any chunk
+            for (Index b = 0; b < batch; ++b) {
+                const Index last = lengths[static_cast<std::size_t>(b)] - 1 - done;
+                if (last >= 0 && last < count)
+                    runtime::check_cuda(cudaMemcpyAsync(static_cast<float*>(x_.mutable_data()) + b * D, plan.hidden() + (b * count + last) * D,
+                                                        static_cast<std::size_t>(D) * sizeof(float), cudaMemcpyDeviceToDevice,
+                                                        static_cast<cudaStream_t>(stream)), "cudaMemcpyAsync");
+            }
+        }
+        done += count;
+        synchronize(Device::cuda(device_));  // `part` and the chunk buffers are reused
+    }
+    if (!lengths.empty()) {
+        // Padding went into the cache behind the shorter prompts; their lengths end before it, so it is overwritten by the tokens
+        // that follow and never seen.
+        std::vector<std::int32_t> valid;
+        for (const Index n : lengths) valid.push_back(static_cast<std::int32_t>(before + n));
+        for (auto* cache : caches) runtime::check(b200_kv_cache_set_lengths(cache, valid.data(), stream), "KV lengths");
+    }
+    // final norm fused into the projection
+    const Tensor* norm = decoder_->normalization().weight();
+    runtime::check(b200_linear(x_.data<float>(), batch, D, output_->weight().raw_data(), code_of(output_->weight().dtype()), outputs(), norm->raw_data(),
+                               code_of(norm->dtype()), decoder_->normalization().epsilon(), B200_EPI_STORE, nullptr, nullptr, logits, stream),
+                   "logits");
+    probe(0);
+}
+
+bool DecoderTokenModel::prepare_step(Index batch) {
+    auto& plan = decoder_->plan();
+    reserve_rows(batch);
+    plan.reserve(batch, cache_->front().capacity(), device_);
+    return plan.prepare_choice(*output_, batch, device_);
+}
+
+void DecoderTokenModel::step(const Index* ids, Index batch, void* stream) {
+    auto& plan = decoder_->plan();
+    plan.embed(*tokens_, ids, batch, static_cast<float*>(x_.mutable_data()), stream);
+    plan.run_layers(x_.data<float>(), batch, 1, *cache_, cache_->front().capacity(), stream, plan.shadows_for(batch));
+}
+
+void DecoderTokenModel::advance(Index, void* stream) {
+    const auto caches = handles();
+    runtime::check(b200_kv_cache_advance(caches.data(), static_cast<int32_t>(caches.size()), 1, stream), "KV advance");
+    probe(2);
+}
+
+void DecoderTokenModel::choose(Index batch, const TokenFeedback& f, void* stream) {
+    auto caches = handles();
+    if (caches.size() > 64) {   // the merge kernel of the fused choice advances up to 64 caches itself
+        advance(batch, stream);
+        caches.clear();
+    }
+    decoder_->plan().choose(*output_, batch, f.next, f.ids, f.history, f.history_rows, f.counter, caches, stream);
+}
+
+void DecoderTokenModel::commit(Index steps) { for (auto& layer : *cache_) layer.commit(steps); }
+
+// ---- Generation -----------------------------------------------------------------------------------------
+Generation::Generation(std::shared_ptr<TransformerDecoder> decoder, std::shared_ptr<Embedding> tokens, std::shared_ptr<Linear> output,
+                       std::vector<KVCache>* cache, Index batch, Index max_steps)
+    : Generation(std::make_unique<DecoderTokenModel>(std::move(decoder), std::move(tokens), std::move(output), cache), batch, max_steps) {}
+
+Generation::Generation(std::unique_ptr<TokenModel> model, Index batch, Index max_steps)
+    : model_(std::move(model)), batch_(batch), max_steps_(max_steps) {
+    if (batch <= 0 || max_steps <= 0) throw std::invalid_argument("generation needs a positive batch and step budget");
+    device_ = model_->device();
     runtime::set_device(device_);
     const Device where = Device::cuda(device_);
     ids_ = zeros({batch}, {DType::i64, where});
     next_ = zeros({batch}, {DType::i64, where});
-    logits_ = empty({batch, output_->weight().size(0)}, {DType::f32, where});
+    logits_ = empty({batch, model_->outputs()}, {DType::f32, where});
     history_ = zeros({max_steps, batch}, {DType::i64, where});
     counter_ = zeros({1}, {DType::i64, where});  // the kernel uses the first 32 bits
-    x_ = empty({batch, decoder_->dimensions()}, {DType::f32, where});
     uniform_ = zeros({batch}, {DType::f64, where});
     // pinned staging: ids in, ids out, uniform variates
     pinned_ = std::make_shared<runtime::Storage>(sizeof(Index) * static_cast<std::size_t>(batch) * 3, Device::cpu(), true);
@@ -588,115 +690,70 @@ Generation::~Generation() {
     if (graph_) cudaGraphExecDestroy(graph_);
 }
 
-// logits of `rows` hidden rows (final RMSNorm fused into the projection), argmax, token feedback
-static void enqueue_head(TransformerDecoder& decoder, const Linear& output, const float* hidden, Index batch, float* logits,
-                         Index* next, Index* ids, Index* history, Index history_rows, int32_t* counter, void* stream) {
-    const Tensor* norm = decoder.normalization().weight();
-    const Index V = output.weight().size(0), D = decoder.dimensions();
-    runtime::check(b200_linear(hidden, batch, D, output.weight().raw_data(), code_of(output.weight().dtype()), V, norm->raw_data(),
-                               code_of(norm->dtype()), decoder.normalization().epsilon(), B200_EPI_STORE, nullptr, nullptr, logits, stream),
-                   "logits");
-    probe(0);
-    runtime::check(b200_argmax(logits, batch, V, next, stream), "argmax");
-    runtime::check(b200_token_feedback(next, batch, ids, history, history_rows, counter, stream), "token feedback");
-    probe(2);
+TokenFeedback Generation::feedback() const {
+    return {static_cast<Index*>(next_.mutable_data()), static_cast<Index*>(ids_.mutable_data()), static_cast<Index*>(history_.mutable_data()),
+            max_steps_, static_cast<int32_t*>(counter_.mutable_data())};
 }
 
-void Generation::prefill(const Tensor& prompt) {
+void Generation::prefill(const Tensor& prompt, std::span<const Index> lengths) {
     if (prompt.ndim() != 2 || prompt.size(0) != batch_ || prompt.dtype() != DType::i64 || prompt.size(1) <= 0)
         throw std::invalid_argument("prompt must be int64 [batch, length] with a positive length");
-    const Index P = prompt.size(1), D = decoder_->dimensions();
+    const Index P = prompt.size(1);
+    if (!lengths.empty() && static_cast<Index>(lengths.size()) != batch_) throw std::invalid_argument("one prompt length per sequence is needed");
+    for (const Index n : lengths)
+        if (n <= 0 || n > P) throw std::invalid_argument("prompt lengths must lie in [1, length]");
     runtime::set_device(device_);
     void* stream = runtime::stream(device_);
     if (prompt.device().type == DeviceType::cpu) {
-        const Index V = tokens_->weight().size(0);
+        const Index V = model_->vocabulary();
         for (Index i = 0; i < prompt.numel(); ++i)
             if (prompt.data<Index>()[i] < 0 || prompt.data<Index>()[i] >= V) throw std::out_of_range("embedding index out of range");
     }
     const Tensor device_prompt = prompt.to(Device::cuda(device_));
-    auto& plan = decoder_->plan();
-    plan.refresh();
-    plan.validate(batch_, P, *cache_, device_);
+    model_->refresh();
+    model_->validate(batch_, P);
     if (generated_ >= max_steps_) throw std::out_of_range("generation step budget exhausted");
-    // Chunked prefill: at most ~8192 rows per pass; chunked decode equals one pass (tests/state.cpp:54-63 of the reference).
-    const Index chunk = std::max<Index>(1, std::min<Index>(P, 8192 / batch_ > 0 ? 8192 / batch_ : 1));
-    Tensor features = empty({batch_ * chunk, D}, {DType::f32, Device::cuda(device_)});
-    Index done = 0;
-    while (done < P) {
-        const Index count = std::min(chunk, P - done);
-        const Tensor part = count == P ? device_prompt : device_prompt.narrow(1, done, count);
-        runtime::check(b200_embedding(tokens_->weight().raw_data(), code_of(tokens_->weight().dtype()), part.data<Index>(), batch_ * count,
-                                      tokens_->weight().size(0), D, static_cast<float*>(features.mutable_data()), stream), "embedding");
-        const Index max_length = cache_->front().length() + count;
-        plan.reserve(batch_ * count, max_length, device_);
-        plan.run_layers(features.data<float>(), batch_, count, *cache_, max_length, stream);
-        std::vector<b200_kv_cache*> handles;
-        for (auto& layer : *cache_) handles.push_back(layer.handle());
-        runtime::check(b200_kv_cache_advance(handles.data(), static_cast<int32_t>(handles.size()), static_cast<int32_t>(count), stream), "KV advance");
-        for (auto& layer : *cache_) layer.commit(count);
-        done += count;
-        if (done == P) {
-            // last position of every sequence -> first generated token
-            runtime::check(b200_select_rows(plan.hidden(), count - 1, count, batch_, D, static_cast<float*>(x_.mutable_data()), stream), "select");
-            enqueue_head(*decoder_, *output_, x_.data<float>(), batch_, static_cast<float*>(logits_.mutable_data()),
-                         static_cast<Index*>(next_.mutable_data()), static_cast<Index*>(ids_.mutable_data()),
-                         static_cast<Index*>(history_.mutable_data()), max_steps_, static_cast<int32_t*>(counter_.mutable_data()), stream);
-        }
-        synchronize(Device::cuda(device_));  // `part` and the chunk buffers are reused
-    }
-    plan.set_user(this);
+    // the last position of every sequence -> first generated token
+    model_->prefill(device_prompt, lengths, static_cast<float*>(logits_.mutable_data()));
+    const TokenFeedback f = feedback();
+    runtime::check(b200_argmax(logits_.data<float>(), batch_, model_->outputs(), f.next, stream), "argmax");
+    runtime::check(b200_token_feedback(f.next, batch_, f.ids, f.history, f.history_rows, f.counter, stream), "token feedback");
+    probe(2);
+    synchronize(Device::cuda(device_));
+    model_->set_user(this);
     logits_current_ = true;   // the prompt's last position went through the materialised head
     ++generated_;
 }
 
-void Generation::enqueue_step(void* stream, Index max_length) {
-    auto& plan = decoder_->plan();
-    const Index D = decoder_->dimensions();
-    plan.embed(*tokens_, ids_.data<Index>(), batch_, static_cast<float*>(x_.mutable_data()), stream);
-    plan.run_layers(x_.data<float>(), batch_, 1, *cache_, max_length, stream, plan.shadows_for(batch_));
-    std::vector<b200_kv_cache*> handles;
-    for (auto& layer : *cache_) handles.push_back(layer.handle());
-    if (fused_choice_ && handles.size() <= 64) {   // the merge kernel of the fused choice also advances the caches
-        plan.choose(*output_, batch_, static_cast<Index*>(next_.mutable_data()), static_cast<Index*>(ids_.mutable_data()),
-                    static_cast<Index*>(history_.mutable_data()), max_steps_, static_cast<int32_t*>(counter_.mutable_data()), handles, stream);
-        return;
-    }
-    runtime::check(b200_kv_cache_advance(handles.data(), static_cast<int32_t>(handles.size()), 1, stream), "KV advance");
-    probe(2);
+void Generation::enqueue_step(void* stream) {
+    const TokenFeedback f = feedback();
+    model_->step(ids_.data<Index>(), batch_, stream);
     if (fused_choice_) {
-        plan.choose(*output_, batch_, static_cast<Index*>(next_.mutable_data()), static_cast<Index*>(ids_.mutable_data()),
-                    static_cast<Index*>(history_.mutable_data()), max_steps_, static_cast<int32_t*>(counter_.mutable_data()), {}, stream);
+        model_->choose(batch_, f, stream);
         return;
     }
-    plan.logits(*output_, batch_, static_cast<float*>(logits_.mutable_data()), stream);
-    runtime::check(b200_argmax(logits_.data<float>(), batch_, output_->weight().size(0), static_cast<Index*>(next_.mutable_data()), stream), "argmax");
-    runtime::check(b200_token_feedback(next_.data<Index>(), batch_, static_cast<Index*>(ids_.mutable_data()),
-                                       static_cast<Index*>(history_.mutable_data()), max_steps_,
-                                       static_cast<int32_t*>(counter_.mutable_data()), stream), "token feedback");
+    model_->advance(batch_, stream);
+    model_->logits(batch_, static_cast<float*>(logits_.mutable_data()), stream);
+    runtime::check(b200_argmax(logits_.data<float>(), batch_, model_->outputs(), f.next, stream), "argmax");
+    runtime::check(b200_token_feedback(f.next, batch_, f.ids, f.history, f.history_rows, f.counter, stream), "token feedback");
     probe(2);
 }
 
-void Generation::prepare() {
-    auto& plan = decoder_->plan();
-    plan.reserve(batch_, cache_->front().capacity(), device_);
-    fused_choice_ = plan.prepare_choice(*output_, batch_, device_);
-}
+void Generation::prepare() { fused_choice_ = model_->prepare_step(batch_); }
 
 void Generation::capture() {
-    auto& plan = decoder_->plan();
-    plan.refresh();
-    const std::uint64_t version = decoder_->version() + tokens_->version() + output_->version();
+    model_->refresh();
+    const std::uint64_t version = model_->version();
     runtime::set_device(device_);
-    const Index capacity = cache_->front().capacity();
     prepare();
-    if (graph_ && graph_version_ == version && graph_epoch_ == plan.buffer_epoch()) return;
+    if (graph_ && graph_version_ == version && graph_epoch_ == model_->buffer_epoch()) return;
     if (graph_) { cudaGraphExecDestroy(graph_); graph_ = nullptr; }
     cudaStream_t stream = cuda_stream(device_);
     runtime::check_cuda(cudaStreamSynchronize(stream), "cudaStreamSynchronize");
     runtime::check_cuda(cudaStreamBeginCapture(stream, cudaStreamCaptureModeThreadLocal), "cudaStreamBeginCapture");
     cudaGraph_t graph = nullptr;
     try {
-        enqueue_step(stream, capacity);
+        enqueue_step(stream);
     } catch (...) {
         cudaStreamEndCapture(stream, &graph);
         if (graph) cudaGraphDestroy(graph);
@@ -710,7 +767,7 @@ void Generation::capture() {
     cudaGraphDestroy(graph);
     runtime::check_cuda(status, "cudaGraphInstantiate");
     graph_version_ = version;
-    graph_epoch_ = plan.buffer_epoch();
+    graph_epoch_ = model_->buffer_epoch();
 }
 
 void Generation::step(Index steps) {
@@ -718,16 +775,16 @@ void Generation::step(Index steps) {
     if (generated_ == 0) throw std::logic_error("prefill a prompt before stepping");
     if (generated_ + steps > max_steps_) throw std::out_of_range("generation step budget exhausted");
     runtime::set_device(device_);
-    decoder_->plan().refresh();
-    decoder_->plan().validate(batch_, steps, *cache_, device_);  // capacity for all `steps` single-token appends
+    model_->refresh();
+    model_->validate(batch_, steps);  // capacity for all `steps` single-token appends
     capture();
     if (steps > 0) {
-        decoder_->plan().set_user(this);
+        model_->set_user(this);
         logits_current_ = !fused_choice_;
     }
     cudaStream_t stream = cuda_stream(device_);
     for (Index i = 0; i < steps; ++i) runtime::check_cuda(cudaGraphLaunch(graph_, stream), "cudaGraphLaunch");
-    for (auto& layer : *cache_) layer.commit(steps);
+    model_->commit(steps);
     generated_ += steps;
 }
 
@@ -736,7 +793,7 @@ void Generation::step_host(const Index* ids_in, Index* ids_out) {
     cudaStream_t stream = cuda_stream(device_);
     auto* staging = static_cast<Index*>(pinned_->data);
     if (ids_in) {
-        const Index V = tokens_->weight().size(0);
+        const Index V = model_->vocabulary();
         for (Index b = 0; b < batch_; ++b) {
             if (ids_in[b] < 0 || ids_in[b] >= V) throw std::out_of_range("embedding index out of range");
             staging[b] = ids_in[b];
@@ -760,30 +817,23 @@ void Generation::step_sampled(double temperature, const double* uniforms, Index*
     for (Index b = 0; b < batch_; ++b)
         if (!(uniforms[b] >= 0.0 && uniforms[b] < 1.0)) throw std::invalid_argument("uniform variates must lie in [0, 1)");
     runtime::set_device(device_);
-    auto& plan = decoder_->plan();
-    plan.refresh();
-    plan.validate(batch_, 1, *cache_, device_);
-    const Index capacity = cache_->front().capacity();
-    plan.reserve(batch_, capacity, device_);
-    plan.set_user(this);
+    model_->refresh();
+    model_->validate(batch_, 1);
+    model_->prepare_step(batch_);
+    model_->set_user(this);
     cudaStream_t stream = cuda_stream(device_);
     auto* staging = static_cast<Index*>(pinned_->data);
     auto* variates = reinterpret_cast<double*>(staging + 2 * batch_);
     std::copy(uniforms, uniforms + batch_, variates);
     runtime::check_cuda(cudaMemcpyAsync(uniform_.mutable_data(), variates, sizeof(double) * static_cast<std::size_t>(batch_),
                                         cudaMemcpyHostToDevice, stream), "cudaMemcpyAsync");
-    plan.embed(*tokens_, ids_.data<Index>(), batch_, static_cast<float*>(x_.mutable_data()), stream);
-    plan.run_layers(x_.data<float>(), batch_, 1, *cache_, capacity, stream, plan.shadows_for(batch_));
-    std::vector<b200_kv_cache*> handles;
-    for (auto& layer : *cache_) handles.push_back(layer.handle());
-    runtime::check(b200_kv_cache_advance(handles.data(), static_cast<int32_t>(handles.size()), 1, stream), "KV advance");
-    plan.logits(*output_, batch_, static_cast<float*>(logits_.mutable_data()), stream);
-    runtime::check(b200_sample(logits_.data<float>(), batch_, output_->weight().size(0), temperature, uniform_.data<double>(),
-                               static_cast<Index*>(next_.mutable_data()), stream), "sampling");
-    runtime::check(b200_token_feedback(next_.data<Index>(), batch_, static_cast<Index*>(ids_.mutable_data()),
-                                       static_cast<Index*>(history_.mutable_data()), max_steps_,
-                                       static_cast<int32_t*>(counter_.mutable_data()), stream), "token feedback");
-    for (auto& layer : *cache_) layer.commit(1);
+    const TokenFeedback f = feedback();
+    model_->step(ids_.data<Index>(), batch_, stream);
+    model_->advance(batch_, stream);
+    model_->logits(batch_, static_cast<float*>(logits_.mutable_data()), stream);
+    runtime::check(b200_sample(logits_.data<float>(), batch_, model_->outputs(), temperature, uniform_.data<double>(), f.next, stream), "sampling");
+    runtime::check(b200_token_feedback(f.next, batch_, f.ids, f.history, f.history_rows, f.counter, stream), "token feedback");
+    model_->commit(1);
     ++generated_;
     logits_current_ = true;
     runtime::check_cuda(cudaMemcpyAsync(staging + batch_, next_.raw_data(), sizeof(Index) * static_cast<std::size_t>(batch_),
@@ -796,11 +846,10 @@ Generation::StepProfile Generation::profile_step() {
     if (generated_ == 0) throw std::logic_error("prefill a prompt before stepping");
     if (generated_ + 1 > max_steps_) throw std::out_of_range("generation step budget exhausted");
     runtime::set_device(device_);
-    auto& plan = decoder_->plan();
-    plan.refresh();
-    plan.validate(batch_, 1, *cache_, device_);
+    model_->refresh();
+    model_->validate(batch_, 1);
     prepare();
-    plan.set_user(this);
+    model_->set_user(this);
     logits_current_ = !fused_choice_;
     cudaStream_t stream = cuda_stream(device_);
     runtime::check_cuda(cudaStreamSynchronize(stream), "cudaStreamSynchronize");
@@ -808,14 +857,14 @@ Generation::StepProfile Generation::profile_step() {
     trail.mark(2);
     step_probe = &trail;
     try {
-        enqueue_step(stream, cache_->front().capacity());
+        enqueue_step(stream);
     } catch (...) {
         step_probe = nullptr;
         throw;
     }
     step_probe = nullptr;
     runtime::check_cuda(cudaStreamSynchronize(stream), "cudaStreamSynchronize");
-    for (auto& layer : *cache_) layer.commit(1);
+    model_->commit(1);
     ++generated_;
     StepProfile result{0.0, 0.0, 0.0, static_cast<Index>(trail.events.size()) - 1};
     for (std::size_t i = 1; i < trail.events.size(); ++i) {
@@ -840,10 +889,9 @@ Tensor Generation::tokens() const {
 Tensor Generation::last_logits() {
     if (logits_current_) return logits_;
     if (generated_ == 0) throw std::logic_error("nothing has been generated yet");
-    auto& plan = decoder_->plan();
-    if (plan.user() != this) throw std::logic_error("the decoder has run something else since this generation's last step");
+    if (model_->user() != this) throw std::logic_error("the decoder has run something else since this generation's last step");
     runtime::set_device(device_);
-    plan.logits(*output_, batch_, static_cast<float*>(logits_.mutable_data()), runtime::stream(device_));
+    model_->logits(batch_, static_cast<float*>(logits_.mutable_data()), runtime::stream(device_));
     logits_current_ = true;
     return logits_;
 }

@@ -10,6 +10,7 @@
 #pragma once
 
 #include "dl/dl.h"
+#include "dl/token_model.h"
 
 #include <cuda_runtime.h>
 
@@ -84,14 +85,50 @@ private:
     const void* user_ = nullptr;
 };
 
+// The grouped-query decoder with its embedding and output layers over one cache per layer.
+class DecoderTokenModel : public TokenModel {
+public:
+    DecoderTokenModel(std::shared_ptr<TransformerDecoder> decoder, std::shared_ptr<Embedding> tokens, std::shared_ptr<Linear> output,
+                      std::vector<KVCache>* cache);
+    int device() const override { return device_; }
+    Index vocabulary() const override { return tokens_->weight().size(0); }
+    Index outputs() const override { return output_->weight().size(0); }
+    std::uint64_t version() const override { return decoder_->version() + tokens_->version() + output_->version(); }
+    void refresh() override { decoder_->plan().refresh(); }
+    void validate(Index batch, Index length) override { decoder_->plan().validate(batch, length, *cache_, device_); }
+    std::uint64_t buffer_epoch() const override { return decoder_->plan().buffer_epoch() + x_epoch_; }
+    void prefill(const Tensor& prompt, std::span<const Index> lengths, float* logits) override;
+    bool prepare_step(Index batch) override;
+    void step(const Index* ids, Index batch, void* stream) override;
+    void advance(Index batch, void* stream) override;
+    void logits(Index batch, float* out, void* stream) override { decoder_->plan().logits(*output_, batch, out, stream); }
+    void choose(Index batch, const TokenFeedback& feedback, void* stream) override;
+    void commit(Index steps) override;
+    void set_user(const void* user) override { decoder_->plan().set_user(user); }
+    const void* user() const override { return decoder_->plan().user(); }
+
+private:
+    std::vector<b200_kv_cache*> handles() const;
+    void reserve_rows(Index batch);   // x_: first hidden rows of a step
+    std::shared_ptr<TransformerDecoder> decoder_;
+    std::shared_ptr<Embedding> tokens_;
+    std::shared_ptr<Linear> output_;
+    std::vector<KVCache>* cache_;
+    int device_ = 0;
+    std::uint64_t x_epoch_ = 0;
+    Tensor x_;
+};
+
 // Greedy generation with the token loop resident on the device (the loop of examples/decoder_generate.cpp:20-31).
 class Generation {
 public:
     Generation(std::shared_ptr<TransformerDecoder> decoder, std::shared_ptr<Embedding> tokens, std::shared_ptr<Linear> output,
                std::vector<KVCache>* cache, Index batch, Index max_steps);
+    Generation(std::unique_ptr<TokenModel> model, Index batch, Index max_steps);
     ~Generation();
-    // Prefill the prompt [batch, P] (int64, host or device) in chunks and choose the first token.
-    void prefill(const Tensor& prompt);
+    // Prefill the prompt [batch, P] (int64, host or device) in chunks and choose the first token.  With `lengths` the prompts are
+    // of unequal length: sequence s takes its first lengths[s] tokens, the rest of its row is padding.
+    void prefill(const Tensor& prompt, std::span<const Index> lengths = {});
     // Enqueue `steps` single-token steps (graph replays); no host synchronisation.
     void step(Index steps);
     // One step driven from the host: ids_in [batch] host -> H2D, step, D2H -> ids_out [batch] host (the reference's
@@ -115,17 +152,15 @@ public:
     StepProfile profile_step();
 
 private:
-    void enqueue_step(void* stream, Index max_length);
+    void enqueue_step(void* stream);
+    TokenFeedback feedback() const;
     void prepare();   // workspaces of a single-token step, before anything is enqueued or captured
     void capture();
-    std::shared_ptr<TransformerDecoder> decoder_;
-    std::shared_ptr<Embedding> tokens_;
-    std::shared_ptr<Linear> output_;
-    std::vector<KVCache>* cache_;
+    std::unique_ptr<TokenModel> model_;
     Index batch_, max_steps_, generated_ = 0, launches_per_step_ = 0;
     bool fused_choice_ = false, logits_current_ = false;
     int device_ = 0;
-    Tensor ids_, next_, logits_, history_, counter_, x_, uniform_;
+    Tensor ids_, next_, logits_, history_, counter_, uniform_;
     std::shared_ptr<runtime::Storage> pinned_;
     cudaGraphExec_t graph_ = nullptr;
     std::uint64_t graph_version_ = ~0ull, graph_epoch_ = ~0ull;

@@ -1,0 +1,73 @@
+// Registry of model designs and loading of a model folder (config.json + model.safetensors).
+#include "dl/hybrid.h"
+#include "dl/internal.h"
+
+#include <fstream>
+#include <sstream>
+#include <stdexcept>
+
+namespace dl::models {
+
+namespace {
+
+using Factory = std::shared_ptr<nn::UnaryModule> (*)(const Json&, TensorOptions);
+
+std::shared_ptr<nn::UnaryModule> hybrid(const Json& config, TensorOptions options) { return std::make_shared<nn::HybridDecoder>(config, options); }
+
+// Grouped-query decoder with its embedding and output layers, under the names of the reference's example model.
+std::shared_ptr<nn::UnaryModule> transformer(const Json& c, TensorOptions options) {
+    const bool tied = !c.has("tied") || c.at("tied").integer() != 0;
+    return std::make_shared<nn::DecoderLanguageModel>(c.at("vocab").positive(), c.at("layers").positive(), c.at("width").positive(),
+                                                      c.at("heads").positive(), c.at("kv_heads").positive(), c.at("ff").positive(),
+                                                      c.at("context").positive(), tied, options);
+}
+
+struct Entry { const char* name; Factory make; };
+constexpr Entry kRegistry[] = {
+    {"Ripitar", hybrid},
+    {"TransformerDecoder", transformer},
+};
+
+std::string read_text(const std::filesystem::path& path) {
+    std::ifstream in(path, std::ios::binary);
+    if (!in) throw std::runtime_error("cannot read " + path.string());
+    std::ostringstream text;
+    text << in.rdbuf();
+    return text.str();
+}
+
+}  // namespace
+
+std::vector<std::string> architectures() {
+    std::vector<std::string> names;
+    for (const auto& entry : kRegistry) names.emplace_back(entry.name);
+    return names;
+}
+
+std::shared_ptr<nn::UnaryModule> create(const Json& config, TensorOptions options) {
+    const std::string& name = config.at("architecture").text();
+    for (const auto& entry : kRegistry)
+        if (name == entry.name) return entry.make(config, options);
+    throw std::invalid_argument("configuration: unknown architecture '" + name + "'");
+}
+
+std::shared_ptr<nn::UnaryModule> load(const std::filesystem::path& folder, DType dtype, Device device) {
+    auto model = create(Json::parse(read_text(folder / "config.json")), {dtype, Device::cpu()});
+    StateDict converted;
+    for (auto& [name, tensor] : io::load_safetensors(folder / "model.safetensors")) {
+        const bool floating = tensor.dtype() == DType::bf16 || tensor.dtype() == DType::f32 || tensor.dtype() == DType::f64;
+        converted.emplace_back(name, floating ? tensor.astype(dtype) : tensor);
+    }
+    // buffers (position tables) are computed, not loaded
+    for (const auto& [name, tensor] : model->state_dict()) {
+        if (name.find("rotary.") == std::string::npos) continue;
+        bool found = false;
+        for (const auto& entry : converted) found = found || entry.first == name;
+        if (!found) converted.emplace_back(name, tensor);
+    }
+    model->load_state_dict(converted);
+    model->to(device);
+    return model;
+}
+
+}  // namespace dl::models

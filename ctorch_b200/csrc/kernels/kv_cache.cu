@@ -89,11 +89,11 @@ using namespace b200;
 
 extern "C" {
 
-int b200_kv_cache_create(int32_t device, int32_t dtype, int32_t sequences, int32_t kv_heads, int32_t head_dim,
-                         int32_t capacity, int32_t page_size, b200_kv_cache** out) {
+static int create_cache(int32_t device, int32_t dtype, int32_t sequences, int32_t kv_heads, int32_t head_dim, int32_t capacity,
+                        int32_t page_size, int pools, int32_t* lengths, b200_kv_cache** out) {
     if (!out) return B200_BAD_ARGUMENT;
     *out = nullptr;
-    if ((dtype != B200_F32 && dtype != B200_BF16) || sequences <= 0 || kv_heads <= 0 || head_dim <= 0 || (head_dim & 1)
+    if ((dtype != B200_F32 && dtype != B200_BF16) || sequences <= 0 || kv_heads <= 0 || head_dim <= 0 || (pools == 2 && (head_dim & 1))
         || capacity <= 0 || page_size <= 0) {
         set_error("b200_kv_cache_create: bad shape or dtype");
         return B200_BAD_ARGUMENT;
@@ -108,7 +108,7 @@ int b200_kv_cache_create(int32_t device, int32_t dtype, int32_t sequences, int32
     c->num_pages = c->pages_per_seq * sequences;
     c->pool_bytes = static_cast<size_t>(c->num_pages) * kv_heads * page_size * head_dim * (dtype == B200_BF16 ? 2 : 4);
     auto fail = [&](int status) { b200_kv_cache_release(c); return status; };
-    for (int which = 0; which < 2; ++which) {
+    for (int which = 0; which < pools; ++which) {
         cudaError_t e = cudaMalloc(&c->pool[which], c->pool_bytes);
         if (e != cudaSuccess) return fail(cuda_status(e, "cudaMalloc(KV pool)"));
         // Pages start as zeros so that masked positions of a partly filled page are finite.
@@ -117,8 +117,12 @@ int b200_kv_cache_create(int32_t device, int32_t dtype, int32_t sequences, int32
     }
     cudaError_t e = cudaMalloc(reinterpret_cast<void**>(&c->page_table), sizeof(int32_t) * c->num_pages);
     if (e != cudaSuccess) return fail(cuda_status(e, "cudaMalloc(page table)"));
-    e = cudaMalloc(reinterpret_cast<void**>(&c->lengths), sizeof(int32_t) * sequences);
-    if (e != cudaSuccess) return fail(cuda_status(e, "cudaMalloc(lengths)"));
+    c->lengths = lengths;
+    c->owns_lengths = !lengths;
+    if (!lengths) {
+        e = cudaMalloc(reinterpret_cast<void**>(&c->lengths), sizeof(int32_t) * sequences);
+        if (e != cudaSuccess) return fail(cuda_status(e, "cudaMalloc(lengths)"));
+    }
     // Default assignment: logical page p of sequence s lives in physical page p * sequences + s, so that the
     // pages the batch touches in one step are neighbours in memory.
     std::vector<int32_t> table(static_cast<size_t>(c->num_pages));
@@ -126,19 +130,32 @@ int b200_kv_cache_create(int32_t device, int32_t dtype, int32_t sequences, int32
         for (int p = 0; p < c->pages_per_seq; ++p) table[static_cast<size_t>(s) * c->pages_per_seq + p] = p * sequences + s;
     e = cudaMemcpy(c->page_table, table.data(), sizeof(int32_t) * table.size(), cudaMemcpyHostToDevice);
     if (e != cudaSuccess) return fail(cuda_status(e, "cudaMemcpy(page table)"));
-    e = cudaMemset(c->lengths, 0, sizeof(int32_t) * sequences);
-    if (e != cudaSuccess) return fail(cuda_status(e, "cudaMemset(lengths)"));
+    if (c->owns_lengths) {
+        e = cudaMemset(c->lengths, 0, sizeof(int32_t) * sequences);
+        if (e != cudaSuccess) return fail(cuda_status(e, "cudaMemset(lengths)"));
+    }
     c->even_lengths = true;
-    const int status = make_maps(c);
+    const int status = pools == 2 ? make_maps(c) : B200_OK;
     if (status != B200_OK) return fail(status);
     *out = c;
     return B200_OK;
 }
 
+int b200_kv_cache_create(int32_t device, int32_t dtype, int32_t sequences, int32_t kv_heads, int32_t head_dim,
+                         int32_t capacity, int32_t page_size, b200_kv_cache** out) {
+    return create_cache(device, dtype, sequences, kv_heads, head_dim, capacity, page_size, 2, nullptr, out);
+}
+int b200_latent_cache_create(int32_t device, int32_t dtype, int32_t slots, int32_t width, int32_t capacity, int32_t page_size, int32_t* lengths,
+                             b200_kv_cache** out) {
+    if (!lengths) { set_error("b200_latent_cache_create: lengths missing"); return B200_BAD_ARGUMENT; }
+    return create_cache(device, dtype, slots, 1, width, capacity, page_size, 1, lengths, out);
+}
+
 void b200_kv_cache_release(b200_kv_cache* c) {
     if (!c) return;
     cudaSetDevice(c->device);
-    cudaFree(c->pool[0]); cudaFree(c->pool[1]); cudaFree(c->page_table); cudaFree(c->lengths);
+    cudaFree(c->pool[0]); cudaFree(c->pool[1]); cudaFree(c->page_table);
+    if (c->owns_lengths) cudaFree(c->lengths);
     delete c;
 }
 

@@ -56,9 +56,10 @@ const CUtensorMap* kv_tensor_map(const b200_kv_cache* cache, int which);
 struct b200_kv_cache {
     int32_t device, dtype, sequences, kv_heads, head_dim, capacity, page_size, pages_per_seq, num_pages;
     size_t pool_bytes;
-    void* pool[2];
+    void* pool[2];       // a latent cache has one pool: what it holds serves as key and as value
     int32_t* page_table;
     int32_t* lengths;
+    bool owns_lengths;   // a latent cache uses the lengths of the model's slots
     bool has_maps;
     bool even_lengths;   // host-side knowledge: every sequence has the same length (set_lengths with unequal entries clears it)
     alignas(64) CUtensorMap map[2];

@@ -1,0 +1,732 @@
+// Latent attention over a paged cache of latents: per token one latent vector (kv_rank values) and one rotated key part shared by
+// all heads.  The key and value up-projections are absorbed: a query is taken through its head's key up-projection once
+// (b200_latent_query), attends to the latents themselves, and the weighted latent goes through the value up-projection
+// (b200_latent_value).  Every cached byte serves all heads as key and as value.
+//
+//   * latent_mma_kernel: bf16 caches.  A producer warp copies pages row by row (bulk copies into padded rows, mbarrier ring);
+//     eight consumer warps hold the queries as tensor-core fragments in registers, the query-key product split 4 ways over the
+//     width and 2 ways over the keys of a page; the partial scores meet in shared memory, a warp finishes whole rows of the
+//     online softmax in f32; then every warp multiplies the weights (as hi + lo planes) with its columns of the same page.
+//     Decode: 16 rows (heads of one token), the queries as hi + lo planes.  Longer passes and wide head counts: 32 rows.
+//   * latent_generic_kernel: f32 caches and odd sizes, f32 FMAs, one (row, head) per CTA.
+#include "kv_cache.cuh"
+#include "mma.cuh"
+#include "rows.cuh"
+
+#include <algorithm>
+
+namespace b200 {
+namespace {
+
+struct LatentParams {
+    int heads, dim, rot_dim, vdim, rank, q_rank, rot_dims, width;   // width = rank + rot_dim
+    float scale, eps;
+    const float *cosine, *sine;
+    int positions;
+    const float *q_norm, *kv_norm;
+    KvView kv;
+    int weight_dtype;
+    const void *w_key, *w_value;
+};
+
+bool latent_params(const b200_latent_args* a, LatentParams& p, bool needs_cache) {
+    if (!a || a->heads <= 0 || a->dim <= 0 || a->rot_dim < 0 || a->vdim <= 0 || a->kv_rank <= 0 || a->q_rank <= 0 || a->rot_dims < 0
+        || (a->rot_dims & 1) || a->rot_dims > a->rot_dim || (a->rot_dims > 0 && (!a->cosine || !a->sine)) || !a->q_norm || !a->kv_norm
+        || !a->w_key || !a->w_value || (a->weight_dtype != B200_F32 && a->weight_dtype != B200_BF16)) {
+        set_error("latent attention: bad pointer or size");
+        return false;
+    }
+    p = LatentParams{};
+    p.heads = a->heads; p.dim = a->dim; p.rot_dim = a->rot_dim; p.vdim = a->vdim; p.rank = a->kv_rank; p.q_rank = a->q_rank;
+    p.rot_dims = a->rot_dims; p.width = a->kv_rank + a->rot_dim;
+    p.scale = a->scale; p.eps = static_cast<float>(a->eps);
+    p.cosine = a->cosine; p.sine = a->sine; p.positions = a->positions; p.q_norm = a->q_norm; p.kv_norm = a->kv_norm;
+    p.weight_dtype = a->weight_dtype; p.w_key = a->w_key; p.w_value = a->w_value;
+    if (needs_cache) {
+        if (!a->cache) { set_error("latent attention: no cache"); return false; }
+        p.kv = kv_view(a->cache);
+        if (p.kv.kv_heads != 1 || p.kv.head_dim != p.width) { set_error("latent attention: the cache has another width"); return false; }
+    }
+    return true;
+}
+
+// Entry i of a rotated part: interleaved pairs (2j, 2j + 1) turned by the angle of pair j at `position`; the rest passes.
+__device__ __forceinline__ float rotated(const LatentParams& p, const float* part, int i, int position) {
+    const float v = part[i];
+    if (i >= p.rot_dims || static_cast<unsigned>(position) >= static_cast<unsigned>(p.positions)) return v;
+    const int64_t at = static_cast<int64_t>(position) * (p.rot_dims >> 1) + (i >> 1);
+    const float c = __ldg(p.cosine + at), s = __ldg(p.sine + at);
+    return i & 1 ? __fadd_rn(__fmul_rn(v, c), __fmul_rn(part[i - 1], s)) : __fsub_rn(__fmul_rn(v, c), __fmul_rn(part[i + 1], s));
+}
+
+__device__ __forceinline__ void cache_store(const KvView& kv, int64_t at, float v) {
+    if (kv.dtype == B200_BF16) static_cast<__nv_bfloat16*>(kv.pool[0])[at] = __float2bfloat16_rn(v);
+    else static_cast<float*>(kv.pool[0])[at] = v;
+}
+
+// One CTA per row.
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentParams p, const RowsView rows, const float* projected, int64_t stride,
+                                                             float* q_latent, __nv_bfloat16* q_hi, __nv_bfloat16* q_lo) {
+    __shared__ float scratch[32];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row = blockIdx.x;
+    const RowPlace place = row_place(rows, row);
+    const float* query = projected + row * stride;
+    const float* latent = query + p.q_rank;
+    const float* key = latent + p.rank;
+    float qs = 0.0f, ks = 0.0f;
+    for (int c = threadIdx.x; c < p.q_rank; c += blockDim.x) qs = fmaf(query[c], query[c], qs);
+    for (int c = threadIdx.x; c < p.rank; c += blockDim.x) ks = fmaf(latent[c], latent[c], ks);
+    qs = block_sum(qs, scratch);
+    ks = block_sum(ks, scratch);
+    const float q_inverse = 1.0f / sqrtf(qs / static_cast<float>(p.q_rank) + p.eps);
+    const float k_inverse = 1.0f / sqrtf(ks / static_cast<float>(p.rank) + p.eps);
+    for (int c = threadIdx.x; c < p.q_rank; c += blockDim.x)
+        store_forms(query[c] * q_inverse * p.q_norm[c], static_cast<int64_t>(row) * p.q_rank + c, q_latent, q_hi, q_lo);
+    if (place.position >= p.kv.pages_per_seq * p.kv.page_size) return;   // the host refuses passes that do not fit
+    const int64_t at = kv_offset(p.kv, place.slot, place.position, 0);
+    for (int c = threadIdx.x; c < p.rank; c += blockDim.x) cache_store(p.kv, at + c, latent[c] * k_inverse * p.kv_norm[c]);
+    for (int c = threadIdx.x; c < p.rot_dim; c += blockDim.x) cache_store(p.kv, at + p.rank + c, rotated(p, key, c, place.position));
+}
+
+// ---- per-head projections ---------------------------------------------------------------------------------------
+// y[row, head, o] = sum_k x[row, head, k] w[head][o][k] for two callers: the absorbed query (results stored at the head's slice of
+// the wide query, plus its rotated part) and the value up-projection (results gated, stored as f32 or planes).
+struct HeadLinear {
+    LatentParams latent;
+    RowsView rows;           // query form only
+    const float* x;
+    int64_t x_row, x_head;   // strides of x
+    int row_count, in, out;
+    const void* w;
+    bool query;
+    float* y;                // query form: [rows, heads, width]
+    const float* gate;       // value form
+    int64_t gate_stride;
+    __nv_bfloat16 *out_hi, *out_lo;
+};
+
+__device__ __forceinline__ void head_result(const HeadLinear& h, int row, int head, int o, float v) {
+    if (h.query) {
+        h.y[(static_cast<int64_t>(row) * h.latent.heads + head) * h.latent.width + o] = v;
+    } else {
+        const int64_t column = static_cast<int64_t>(head) * h.out + o;
+        const float g = h.gate[row * h.gate_stride + column];
+        store_forms(v * (1.0f / (1.0f + expf(-g))), row * static_cast<int64_t>(h.latent.heads) * h.out + column, h.y, h.out_hi, h.out_lo);
+    }
+}
+__device__ __forceinline__ void head_rotated(const HeadLinear& h, int row, int head, int i) {
+    const LatentParams& p = h.latent;
+    const float* part = h.x + row * h.x_row + head * h.x_head + p.dim;
+    h.y[(static_cast<int64_t>(row) * p.heads + head) * p.width + p.rank + i] = rotated(p, part, i, row_place(h.rows, row).position);
+}
+
+// One warp per output; grid (output blocks, rows, heads).
+template <class W> __global__ void __launch_bounds__(256) head_linear_generic_kernel(const __grid_constant__ HeadLinear h) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.y, head = blockIdx.z;
+    const float* x = h.x + row * h.x_row + head * h.x_head;
+    for (int o = blockIdx.x * 64 + warp; o < min(h.out, static_cast<int>(blockIdx.x + 1) * 64); o += 8) {
+        const W* w = static_cast<const W*>(h.w) + (static_cast<int64_t>(head) * h.out + o) * h.in;
+        float acc = 0.0f;
+        for (int k = lane; k < h.in; k += 32) acc = fmaf(x[k], load_as_f32(w, k), acc);
+        acc = warp_sum(acc);
+        if (lane == 0) head_result(h, row, head, o, acc);
+    }
+    if (h.query && blockIdx.x == 0)
+        for (int i = threadIdx.x; i < h.latent.rot_dim; i += blockDim.x) head_rotated(h, row, head, i);
+}
+
+// bf16 weights on the tensor cores; the f32 inputs are split into planes while they are staged.  16 * WM rows x 64 outputs per CTA,
+// 64 input columns at a time.  WM = 4: a warp per 16 rows; WM = 1: the four warps share the 16 rows and split the outputs.
+constexpr int kHeadThreads = 128, kHeadTile = 64, kHeadPitch = 72;
+template <int WM> constexpr int head_linear_smem() { return 2 * (2 * 16 * WM + kHeadTile) * kHeadPitch * 2; }
+
+template <int WM> __global__ void __launch_bounds__(kHeadThreads) head_linear_mma_kernel(const __grid_constant__ HeadLinear h) {
+    constexpr int M = 16 * WM, kTiles = WM == 4 ? 8 : 2, kQuads = M * kHeadTile / 4 / kHeadThreads;
+    extern __shared__ __align__(16) uint8_t smem[];
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem);            // [2 buffers][2 planes][M][pitch]
+    __nv_bfloat16* ws = xs + 4 * M * kHeadPitch;                           // [2 buffers][64][pitch]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int o0 = blockIdx.x * kHeadTile, row0 = blockIdx.y * M, head = blockIdx.z;
+    const __nv_bfloat16* weight = static_cast<const __nv_bfloat16*>(h.w) + static_cast<int64_t>(head) * h.out * h.in;
+    auto stage_weights = [&](int chunk) {
+        __nv_bfloat16* dst = ws + (chunk & 1) * kHeadTile * kHeadPitch;
+        for (int i = threadIdx.x; i < kHeadTile * 8; i += kHeadThreads) {
+            const int o = i >> 3, k = chunk * kHeadTile + (i & 7) * 8;
+            const bool live = o0 + o < h.out && k < h.in;
+            copy_async_16(smem_u32(dst + o * kHeadPitch + (i & 7) * 8), live ? weight + static_cast<int64_t>(o0 + o) * h.in + k : weight, live);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    float4 ahead[kQuads];
+    auto fetch_rows = [&](int chunk) {
+#pragma unroll
+        for (int j = 0; j < kQuads; ++j) {
+            const int i = threadIdx.x + j * kHeadThreads, r = i >> 4, k = chunk * kHeadTile + (i & 15) * 4;
+            ahead[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (row0 + r < h.row_count && k < h.in)
+                ahead[j] = *reinterpret_cast<const float4*>(h.x + (row0 + r) * h.x_row + head * h.x_head + k);
+        }
+    };
+    auto put_rows = [&](int chunk) {
+        __nv_bfloat16* hi = xs + (chunk & 1) * 2 * M * kHeadPitch;
+        __nv_bfloat16* lo = hi + M * kHeadPitch;
+#pragma unroll
+        for (int j = 0; j < kQuads; ++j) {
+            const int i = threadIdx.x + j * kHeadThreads, r = i >> 4, c = (i & 15) * 4;
+            uint32_t h0, l0, h1, l1;
+            pack_planes(ahead[j].x, ahead[j].y, h0, l0);
+            pack_planes(ahead[j].z, ahead[j].w, h1, l1);
+            *reinterpret_cast<uint2*>(hi + r * kHeadPitch + c) = make_uint2(h0, h1);
+            *reinterpret_cast<uint2*>(lo + r * kHeadPitch + c) = make_uint2(l0, l1);
+        }
+    };
+    float acc[kTiles][4];
+#pragma unroll
+    for (int n = 0; n < kTiles; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[n][i] = 0.0f;
+
+    const int chunks = (h.in + kHeadTile - 1) / kHeadTile;
+    stage_weights(0);          // weights are constants: requested before the producer of x is waited for
+    grid_dependency_wait();
+    grid_launch_dependents();
+    fetch_rows(0);
+    put_rows(0);
+    for (int chunk = 0; chunk < chunks; ++chunk) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (chunk + 1 < chunks) { stage_weights(chunk + 1); fetch_rows(chunk + 1); }
+        const __nv_bfloat16* hi = xs + (chunk & 1) * 2 * M * kHeadPitch;
+        const int m0 = WM == 4 ? warp * 16 : 0, n0 = WM == 4 ? 0 : warp * 16;
+        const uint32_t a_hi = smem_u32(hi + (m0 + (lane & 15)) * kHeadPitch + (lane >> 4) * 8);
+        const uint32_t a_lo = a_hi + M * kHeadPitch * 2;
+        const uint32_t b = smem_u32(ws + (chunk & 1) * kHeadTile * kHeadPitch + (n0 + (lane >> 4) * 8 + (lane & 7)) * kHeadPitch + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int k = 0; k < kHeadTile / 16; ++k) {
+            uint32_t ah[4], al[4];
+            ldsm_x4(ah, a_hi + k * 32);
+            ldsm_x4(al, a_lo + k * 32);
+#pragma unroll
+            for (int n = 0; n < kTiles; n += 2) {
+                uint32_t w[4];
+                ldsm_x4(w, b + n * 8 * kHeadPitch * 2 + k * 32);
+                mma_16816(acc[n], ah, w[0], w[1]);
+                mma_16816(acc[n], al, w[0], w[1]);
+                mma_16816(acc[n + 1], ah, w[2], w[3]);
+                mma_16816(acc[n + 1], al, w[2], w[3]);
+            }
+        }
+        if (chunk + 1 < chunks) put_rows(chunk + 1);
+    }
+    const int m = row0 + (WM == 4 ? warp * 16 : 0) + (lane >> 2), c = o0 + (WM == 4 ? 0 : warp * 16) + (lane & 3) * 2;
+#pragma unroll
+    for (int n = 0; n < kTiles; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int row = m + (i >> 1) * 8, o = c + n * 8 + (i & 1);
+            if (row < h.row_count && o < h.out) head_result(h, row, head, o, acc[n][i]);
+        }
+    if (h.query && blockIdx.x == 0)
+        for (int i = threadIdx.x; i < M * h.latent.rot_dim; i += kHeadThreads) {
+            const int r = i / h.latent.rot_dim;
+            if (row0 + r < h.row_count) head_rotated(h, row0 + r, head, i - r * h.latent.rot_dim);
+        }
+}
+
+int launch_head_linear(const HeadLinear& h, cudaStream_t stream) {
+    const LatentParams& p = h.latent;
+    if (h.row_count > 65535 || p.heads > 65535) { set_error("latent attention: at most 65535 rows and heads in one pass"); return B200_UNSUPPORTED; }
+    const unsigned tiles = static_cast<unsigned>((h.out + kHeadTile - 1) / kHeadTile);
+    const bool mma = p.weight_dtype == B200_BF16 && h.in % 8 == 0 && h.x_row % 4 == 0 && h.x_head % 4 == 0
+        && ((reinterpret_cast<uintptr_t>(h.x) | reinterpret_cast<uintptr_t>(h.w)) & 15) == 0;
+    if (!mma) {
+        const dim3 grid(tiles, static_cast<unsigned>(h.row_count), static_cast<unsigned>(p.heads));
+        return cuda_status(p.weight_dtype == B200_BF16 ? launch_dependent(head_linear_generic_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, h)
+                                                       : launch_dependent(head_linear_generic_kernel<float>, grid, dim3(256), 0, stream, h),
+                           "head_linear_generic_kernel launch");
+    }
+    if (h.row_count <= 16) {
+        B200_CUDA(cudaFuncSetAttribute(head_linear_mma_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, head_linear_smem<1>()));
+        return cuda_status(launch_dependent(head_linear_mma_kernel<1>, dim3(tiles, 1, static_cast<unsigned>(p.heads)), dim3(kHeadThreads),
+                                            head_linear_smem<1>(), stream, h), "head_linear_mma_kernel launch");
+    }
+    B200_CUDA(cudaFuncSetAttribute(head_linear_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, head_linear_smem<4>()));
+    return cuda_status(launch_dependent(head_linear_mma_kernel<4>, dim3(tiles, static_cast<unsigned>((h.row_count + 63) / 64), static_cast<unsigned>(p.heads)),
+                                        dim3(kHeadThreads), head_linear_smem<4>(), stream, h), "head_linear_mma_kernel launch");
+}
+
+// ---- attention ----------------------------------------------------------------------------------------------------
+struct LatentAttention {
+    LatentParams latent;
+    RowsView rows;
+    const float* query;        // [rows, heads, width]
+    float* out;                // [rows, heads, rank]
+    int positions_per_item, head_chunk, head_chunks, splits;
+    float *partial, *partial_ml;   // splits > 1: [rows, heads, splits, rank], [rows, heads, splits, 2]
+    int stages;
+    int32_t* status;
+};
+
+constexpr int kPage = 64, kConsumerWarps = 8, kConsumerThreads = kConsumerWarps * 32, kLatentThreads = kConsumerThreads + 32;
+constexpr int kScorePitch = 68, kWeightPitch = 72;
+constexpr float kLog2e = 1.4426950408889634f;
+
+int latent_row_bytes(int width) { return (((width + 15) & ~15) + 8) * 2; }   // odd multiple of 16 bytes: conflict-free ldmatrix
+int latent_fixed_bytes(int m) { return 4 * m * kScorePitch * 4 + 2 * m * kWeightPitch * 2 + 4 * m * 4 + 256; }
+
+__device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kConsumerThreads) : "memory"); }
+
+// KS: 16-wide steps of the width per quarter; VT: 8-column tiles of the latent per warp; MT: 16-row tiles.  MT = 1 multiplies the
+// queries as hi + lo planes.
+template <int KS, int VT, int MT>
+__global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __grid_constant__ LatentAttention a) {
+    constexpr int M = 16 * MT, kPlanes = 2;   // fragments per step: planes (MT = 1) or row tiles (MT = 2)
+    extern __shared__ __align__(16) uint8_t smem[];
+    const LatentParams& p = a.latent;
+    const int row_elements = ((p.width + 15) & ~15) + 8, stage_elements = kPage * row_elements;
+    __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem);
+    float* scores = reinterpret_cast<float*>(ring + a.stages * stage_elements);      // [4][M][kScorePitch]
+    __nv_bfloat16* weights = reinterpret_cast<__nv_bfloat16*>(scores + 4 * M * kScorePitch);   // [2 planes][M][kWeightPitch]
+    float* shrink = reinterpret_cast<float*>(weights + 2 * M * kWeightPitch);       // [M] factor of the accumulators
+    float* row_m = shrink + M;
+    float* row_l = row_m + M;
+    int* visible = reinterpret_cast<int*>(row_l + M);                               // [M] keys the row sees
+    uint64_t* full = reinterpret_cast<uint64_t*>(visible + M);
+    uint64_t* empty = full + 8;
+    int* gave_up = reinterpret_cast<int*>(empty + 8);
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int split = blockIdx.z % a.splits, chunk = blockIdx.z / a.splits, sequence = blockIdx.y;
+    // columns past the width are read by the products (times zero): they must be finite
+    for (int i = threadIdx.x; i < a.stages * kPage; i += kLatentThreads)
+        for (int c = p.width; c < row_elements; ++c) ring[i * row_elements + c] = __float2bfloat16_rn(0.0f);
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < a.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], kConsumerWarps); }
+        mbar_fence_init();
+        *gave_up = 0;
+    }
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int first = __ldg(a.rows.first + sequence), count = __ldg(a.rows.first + sequence + 1) - first;
+    const int slot = __ldg(a.rows.slot + sequence), length = a.rows.lengths[slot];
+    // the items with the most keys start first
+    const int offset = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * a.positions_per_item;
+    if (offset >= count) return;
+    const int last = min(offset + a.positions_per_item, count);
+    const int keys = length + last;
+    const int pages = (keys + kPage - 1) / kPage, per_split = (pages + a.splits - 1) / a.splits;
+    const int page0 = split * per_split, page1 = min(pages, page0 + per_split);
+    if (threadIdx.x < M) {
+        const int position = threadIdx.x / a.head_chunk, head = chunk * M + threadIdx.x % a.head_chunk;
+        const bool live = position < a.positions_per_item && offset + position < last && head < p.heads;
+        visible[threadIdx.x] = live ? length + offset + position + 1 : 0;
+        shrink[threadIdx.x] = 1.0f;
+    }
+    __syncthreads();
+
+    if (warp == kConsumerWarps) {   // producer
+        const int32_t* table = p.kv.page_table + static_cast<int64_t>(slot) * p.kv.pages_per_seq;
+        const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(p.kv.pool[0]);
+        const uint32_t bytes = static_cast<uint32_t>(p.width) * 2;
+        for (int t = page0; t < page1; ++t) {
+            const int i = t - page0, s = i % a.stages;
+            if (i >= a.stages && !mbar_wait(&empty[s], ((i / a.stages) - 1) & 1)) {
+                if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
+                break;
+            }
+            if (lane == 0) mbar_expect_tx(&full[s], bytes * kPage);
+            __syncwarp();
+            const __nv_bfloat16* page = pool + static_cast<int64_t>(__ldg(table + t)) * kPage * p.width;
+            for (int r = lane; r < kPage; r += 32) bulk_load(ring + s * stage_elements + r * row_elements, page + r * p.width, bytes, &full[s]);
+        }
+        return;
+    }
+
+    // queries as A fragments: quarter `quarter` of the width
+    const int quarter = warp & 3, half = warp >> 2, steps = (p.width + 15) >> 4;
+    uint32_t q[KS][kPlanes][4];
+    {
+        const float* source[2 * MT];
+#pragma unroll
+        for (int i = 0; i < 2 * MT; ++i) {
+            const int m = (i >> 1) * 16 + (i & 1) * 8 + (lane >> 2);
+            const int64_t row = first + offset + m / a.head_chunk;
+            source[i] = visible[m] > 0 ? a.query + (row * p.heads + chunk * M + m % a.head_chunk) * p.width : nullptr;
+        }
+#pragma unroll
+        for (int i = 0; i < KS; ++i) {
+            const int k = (quarter * KS + i) * 16 + (lane & 3) * 2;
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+                for (int part = 0; part < 4; ++part) {
+                    const float* from = source[mt * 2 + (part & 1)];
+                    const int at = k + (part >> 1) * 8;
+                    float2 v = make_float2(0.0f, 0.0f);
+                    if (from && at < p.width) v = *reinterpret_cast<const float2*>(from + at);
+                    if constexpr (MT == 1) pack_planes(v.x, v.y, q[i][0][part], q[i][1][part]);
+                    else q[i][mt][part] = pack_bf16(v.x, v.y);
+                }
+        }
+    }
+    float o[MT][VT][4];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int v = 0; v < VT; ++v)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) o[mt][v][i] = 0.0f;
+    constexpr int kOwn = M / kConsumerWarps;   // rows whose softmax this warp keeps
+    float m_own[kOwn], l_own[kOwn];
+#pragma unroll
+    for (int r = 0; r < kOwn; ++r) { m_own[r] = -INFINITY; l_own[r] = 0.0f; }
+    const float scale2 = p.scale * kLog2e;
+    const uint32_t key_lane = static_cast<uint32_t>(((half * 32 + (lane >> 4) * 8 + (lane & 7)) * row_elements + ((lane >> 3) & 1) * 8) * 2);
+    const int value_columns = ((p.width + 15) & ~15);
+    bool alive = true;
+
+    for (int t = page0; t < page1; ++t) {
+        const int i = t - page0, s = i % a.stages;
+        if (!mbar_wait(&full[s], (i / a.stages) & 1)) {
+            if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
+            *static_cast<volatile int*>(gave_up) = 1;
+        }
+        const uint32_t page = smem_u32(ring + s * stage_elements);
+        float sc[MT][4][4];
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+            for (int n = 0; n < 4; ++n)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) sc[mt][n][j] = 0.0f;
+#pragma unroll
+        for (int k = 0; k < KS; ++k) {
+            const int step = quarter * KS + k;
+            if (step < steps) {
+#pragma unroll
+                for (int n = 0; n < 4; n += 2) {
+                    uint32_t b[4];
+                    ldsm_x4(b, page + key_lane + static_cast<uint32_t>(n * 8 * row_elements * 2 + step * 32));
+                    if constexpr (MT == 1) {
+                        mma_16816(sc[0][n], q[k][0], b[0], b[1]);
+                        mma_16816(sc[0][n + 1], q[k][0], b[2], b[3]);
+                        mma_16816(sc[0][n], q[k][1], b[0], b[1]);
+                        mma_16816(sc[0][n + 1], q[k][1], b[2], b[3]);
+                    } else {
+#pragma unroll
+                        for (int mt = 0; mt < MT; ++mt) {
+                            mma_16816(sc[mt][n], q[k][mt], b[0], b[1]);
+                            mma_16816(sc[mt][n + 1], q[k][mt], b[2], b[3]);
+                        }
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+                float* at = scores + (quarter * M + mt * 16 + (lane >> 2)) * kScorePitch + half * 32 + n * 8 + (lane & 3) * 2;
+                *reinterpret_cast<float2*>(at) = make_float2(sc[mt][n][0], sc[mt][n][1]);
+                *reinterpret_cast<float2*>(at + 8 * kScorePitch) = make_float2(sc[mt][n][2], sc[mt][n][3]);
+            }
+        consumers_sync();
+        if (*static_cast<volatile int*>(gave_up)) { alive = false; break; }   // a page never arrived: every consumer leaves here
+#pragma unroll
+        for (int r = 0; r < kOwn; ++r) {
+            const int m = warp * kOwn + r, sees = visible[m] - t * kPage;
+            float v0 = 0.0f, v1 = 0.0f;
+#pragma unroll
+            for (int w = 0; w < 4; ++w) {
+                v0 += scores[(w * M + m) * kScorePitch + lane];
+                v1 += scores[(w * M + m) * kScorePitch + lane + 32];
+            }
+            v0 = lane < sees ? v0 * scale2 : -INFINITY;
+            v1 = lane + 32 < sees ? v1 * scale2 : -INFINITY;
+            const float top = fmaxf(m_own[r], warp_max(fmaxf(v0, v1)));
+            const float base = top == -INFINITY ? 0.0f : top;
+            const float p0 = exp2f(v0 - base), p1 = exp2f(v1 - base), factor = exp2f(m_own[r] - base);
+            l_own[r] = l_own[r] * factor + warp_sum(p0 + p1);
+            m_own[r] = top;
+            if (lane == 0) shrink[m] = factor;
+            __nv_bfloat16 hi, lo;
+            split_planes(p0, hi, lo);
+            weights[m * kWeightPitch + lane] = hi;
+            weights[(M + m) * kWeightPitch + lane] = lo;
+            split_planes(p1, hi, lo);
+            weights[m * kWeightPitch + lane + 32] = hi;
+            weights[(M + m) * kWeightPitch + lane + 32] = lo;
+        }
+        consumers_sync();
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+            const float f0 = shrink[mt * 16 + (lane >> 2)], f1 = shrink[mt * 16 + (lane >> 2) + 8];
+#pragma unroll
+            for (int v = 0; v < VT; ++v) { o[mt][v][0] *= f0; o[mt][v][1] *= f0; o[mt][v][2] *= f1; o[mt][v][3] *= f1; }
+        }
+#pragma unroll
+        for (int k = 0; k < kPage / 16; ++k) {
+            uint32_t w[MT][2][4];
+#pragma unroll
+            for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+                for (int plane = 0; plane < 2; ++plane)
+                    ldsm_x4(w[mt][plane], smem_u32(weights + (plane * M + mt * 16 + (lane & 15)) * kWeightPitch + k * 16 + (lane >> 4) * 8));
+#pragma unroll
+            for (int v = 0; v < VT; v += 2) {
+                // tiles past the latent's columns are never stored; their reads stay inside the row
+                const int column = min((warp * VT + v) * 8, value_columns - 16);
+                uint32_t b[4];
+                ldsm_x4_trans(b, page + static_cast<uint32_t>(((k * 16 + (lane & 15)) * row_elements + column + (lane >> 4) * 8) * 2));
+#pragma unroll
+                for (int mt = 0; mt < MT; ++mt) {
+                    mma_16816(o[mt][v], w[mt][0], b[0], b[1]);
+                    mma_16816(o[mt][v + 1], w[mt][0], b[2], b[3]);
+                    mma_16816(o[mt][v], w[mt][1], b[0], b[1]);
+                    mma_16816(o[mt][v + 1], w[mt][1], b[2], b[3]);
+                }
+            }
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&empty[s]);
+    }
+    if (!alive) return;
+    if (lane == 0) {
+#pragma unroll
+        for (int r = 0; r < kOwn; ++r) { row_m[warp * kOwn + r] = m_own[r]; row_l[warp * kOwn + r] = l_own[r]; }
+    }
+    consumers_sync();
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int side = 0; side < 2; ++side) {
+            const int m = mt * 16 + side * 8 + (lane >> 2);
+            if (visible[m] == 0) continue;
+            const int64_t row_head = static_cast<int64_t>(first + offset + m / a.head_chunk) * p.heads + chunk * M + m % a.head_chunk;
+            const bool whole = a.splits == 1;
+            const float factor = whole ? 1.0f / row_l[m] : 1.0f;
+            float* target = whole ? a.out + row_head * p.rank : a.partial + (row_head * a.splits + split) * p.rank;
+#pragma unroll
+            for (int v = 0; v < VT; ++v) {
+                const int column = (warp * VT + v) * 8 + (lane & 3) * 2;
+                if (column < p.rank)
+                    *reinterpret_cast<float2*>(target + column) = make_float2(o[mt][v][side * 2] * factor, o[mt][v][side * 2 + 1] * factor);
+            }
+            if (!whole && warp == 0 && (lane & 3) == 0) {
+                a.partial_ml[(row_head * a.splits + split) * 2] = row_m[m];
+                a.partial_ml[(row_head * a.splits + split) * 2 + 1] = row_l[m];
+            }
+        }
+}
+
+// out[row_head, :] from the splits' (max, sum, unscaled accumulator); one CTA per (row, head)
+__global__ void __launch_bounds__(128) latent_combine_kernel(const float* partial, const float* ml, int splits, int rank, float* out) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t at = blockIdx.x;
+    float top = -INFINITY;
+    for (int s = 0; s < splits; ++s) top = fmaxf(top, ml[(at * splits + s) * 2]);
+    float total = 0.0f;
+    for (int s = 0; s < splits; ++s) total += ml[(at * splits + s) * 2 + 1] * exp2f(ml[(at * splits + s) * 2] - top);
+    const float inverse = 1.0f / total;
+    for (int c = threadIdx.x; c < rank; c += blockDim.x) {
+        float v = 0.0f;
+        for (int s = 0; s < splits; ++s) {
+            const float factor = exp2f(ml[(at * splits + s) * 2] - top);
+            if (factor > 0.0f) v = fmaf(partial[(at * splits + s) * rank + c], factor, v);
+        }
+        out[at * rank + c] = v * inverse;
+    }
+}
+
+constexpr int kGenericThreads = 128, kGenericKeys = 128;
+// grid (heads, rows): f32 FMAs over the cached values of either dtype
+__global__ void __launch_bounds__(kGenericThreads) latent_generic_kernel(const __grid_constant__ LatentAttention a) {
+    extern __shared__ __align__(16) float sm[];   // query [width], accumulator [rank], weights [keys], scratch
+    const LatentParams& p = a.latent;
+    float* query = sm;
+    float* acc = query + p.width;
+    float* w = acc + p.rank;
+    float* scratch = w + kGenericKeys;
+    int64_t* where = reinterpret_cast<int64_t*>(scratch + 32 + ((p.width + p.rank) & 1));   // [keys] 8-byte aligned
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int head = blockIdx.x, row = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const RowPlace place = row_place(a.rows, row);
+    const int64_t row_head = static_cast<int64_t>(row) * p.heads + head;
+    for (int c = threadIdx.x; c < p.width; c += kGenericThreads) query[c] = a.query[row_head * p.width + c];
+    for (int c = threadIdx.x; c < p.rank; c += kGenericThreads) acc[c] = 0.0f;
+    float top = -INFINITY, total = 0.0f;
+    const int keys = place.position + 1;
+    for (int k0 = 0; k0 < keys; k0 += kGenericKeys) {
+        const int n = min(kGenericKeys, keys - k0);
+        __syncthreads();
+        if (threadIdx.x < n) where[threadIdx.x] = kv_offset(p.kv, place.slot, k0 + threadIdx.x, 0);
+        __syncthreads();
+        for (int j = warp; j < n; j += kGenericThreads / 32) {
+            float dot = 0.0f;
+            for (int c = lane; c < p.width; c += 32) dot = fmaf(query[c], kv_load(p.kv, 0, where[j] + c), dot);
+            dot = warp_sum(dot);
+            if (lane == 0) w[j] = dot * p.scale;
+        }
+        __syncthreads();
+        float local = -INFINITY;
+        for (int j = 0; j < n; ++j) local = fmaxf(local, w[j]);
+        const float next = fmaxf(top, local), factor = expf(top - next);
+        __syncthreads();
+        if (threadIdx.x < n) w[threadIdx.x] = expf(w[threadIdx.x] - next);
+        const float sum = block_sum(threadIdx.x < n ? w[threadIdx.x] : 0.0f, scratch);
+        total = total * factor + sum;
+        top = next;
+        for (int c = threadIdx.x; c < p.rank; c += kGenericThreads) {
+            float v = acc[c] * factor;
+            for (int j = 0; j < n; ++j) v = fmaf(w[j], kv_load(p.kv, 0, where[j] + c), v);
+            acc[c] = v;
+        }
+    }
+    const float inverse = 1.0f / total;
+    for (int c = threadIdx.x; c < p.rank; c += kGenericThreads) a.out[row_head * p.rank + c] = acc[c] * inverse;
+}
+
+bool latent_takes_mma(const LatentParams& p) {
+    return p.kv.dtype == B200_BF16 && p.kv.page_size == kPage && p.width % 8 == 0 && p.rank % 8 == 0 && p.rank <= 512 && p.width <= 576;
+}
+// Rows of an item: 16 for decode steps of up to 16 heads, 32 otherwise.
+int latent_tile(const LatentParams& p, int max_count) { return max_count == 1 && p.heads <= 16 ? 16 : 32; }
+
+int latent_splits(const LatentParams& p, int sequences, int max_count, int max_length) {
+    if (max_count > 1) return 1;
+    int device = 0;
+    if (cudaGetDevice(&device) != cudaSuccess) { cudaGetLastError(); device = -1; }
+    const int sms = sm_count(device), tile = latent_tile(p, max_count);
+    const int64_t items = static_cast<int64_t>(sequences) * ((p.heads + tile - 1) / tile);
+    const int pages = std::max(1, (max_length + kPage - 1) / kPage);
+    // rounds of CTAs x (pages of one + its fixed cost in pages), plus the merge
+    int best = 1;
+    double best_cost = 1e30;
+    for (int s = 1; s <= std::min(64, pages); ++s) {
+        const double rounds = static_cast<double>((items * s + sms - 1) / sms);
+        const double cost = rounds * ((pages + s - 1) / s + 1.5) + (s > 1 ? 2.0 + 0.05 * s : 0.0);
+        if (cost < best_cost - 1e-9) { best_cost = cost; best = s; }
+    }
+    return best;
+}
+
+template <int KS, int VT, int MT> int launch_latent_mma(LatentAttention& a, int sequences, int max_count, cudaStream_t stream) {
+    constexpr int M = 16 * MT;
+    const LatentParams& p = a.latent;
+    const int stage = kPage * latent_row_bytes(p.width), fixed = latent_fixed_bytes(M);
+    a.stages = std::min(6, (227 * 1024 - fixed) / stage);
+    if (a.stages < 2) { set_error("latent attention: two pages of width %d do not fit shared memory", p.width); return B200_UNSUPPORTED; }
+    const int smem = fixed + a.stages * stage;
+    a.head_chunk = std::min(p.heads, M);
+    a.head_chunks = (p.heads + M - 1) / M;
+    a.positions_per_item = max_count == 1 ? 1 : std::max(1, M / a.head_chunk);
+    auto kernel = latent_mma_kernel<KS, VT, MT>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    const dim3 grid(static_cast<unsigned>((max_count + a.positions_per_item - 1) / a.positions_per_item), static_cast<unsigned>(sequences),
+                    static_cast<unsigned>(a.head_chunks * a.splits));
+    return cuda_status(launch_dependent(kernel, grid, dim3(kLatentThreads), smem, stream, a), "latent_mma_kernel launch");
+}
+template <int MT> int pick_latent_mma(LatentAttention& a, int sequences, int max_count, cudaStream_t stream) {
+    const LatentParams& p = a.latent;
+    if (p.rank <= 128 && p.width <= 192) return launch_latent_mma<3, 2, MT>(a, sequences, max_count, stream);
+    if (p.rank <= 256 && p.width <= 320) return launch_latent_mma<5, 4, MT>(a, sequences, max_count, stream);
+    return launch_latent_mma<9, 8, MT>(a, sequences, max_count, stream);
+}
+
+}  // namespace
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" {
+
+int b200_latent_prepare(const b200_latent_args* args, const b200_rows* pass, const float* projected, float* q_latent, void* q_hi, void* q_lo,
+                        void* stream) {
+    LatentParams p;
+    RowsView rows;
+    if (!latent_params(args, p, true) || !rows_view(pass, rows)) return B200_BAD_ARGUMENT;
+    if (!projected || (!q_latent && !q_hi)) { set_error("b200_latent_prepare: operands missing"); return B200_BAD_ARGUMENT; }
+    const int64_t stride = static_cast<int64_t>(p.q_rank) + p.width + static_cast<int64_t>(p.heads) * p.vdim;
+    return cuda_status(launch_dependent(latent_prepare_kernel, dim3(static_cast<unsigned>(rows.rows)), dim3(256), 0, as_stream(stream), p, rows,
+                                        projected, stride, q_latent, static_cast<__nv_bfloat16*>(q_hi), static_cast<__nv_bfloat16*>(q_lo)),
+                       "latent_prepare_kernel launch");
+}
+
+int b200_latent_query(const b200_latent_args* args, const b200_rows* pass, const float* query, float* absorbed, void* stream) {
+    HeadLinear h{};
+    if (!latent_params(args, h.latent, false) || !rows_view(pass, h.rows)) return B200_BAD_ARGUMENT;
+    if (!query || !absorbed) { set_error("b200_latent_query: operands missing"); return B200_BAD_ARGUMENT; }
+    const LatentParams& p = h.latent;
+    h.x = query; h.x_head = p.dim + p.rot_dim; h.x_row = h.x_head * p.heads;
+    h.row_count = h.rows.rows; h.in = p.dim; h.out = p.rank; h.w = p.w_key; h.query = true; h.y = absorbed;
+    return launch_head_linear(h, as_stream(stream));
+}
+
+int b200_latent_value(const b200_latent_args* args, int64_t rows, const float* latent, const float* gate, int64_t gate_stride, float* out,
+                      void* out_hi, void* out_lo, void* stream) {
+    HeadLinear h{};
+    if (!latent_params(args, h.latent, false)) return B200_BAD_ARGUMENT;
+    if (!latent || !gate || rows < 0 || rows > INT32_MAX || (!out && !out_hi)) { set_error("b200_latent_value: operands missing"); return B200_BAD_ARGUMENT; }
+    if (rows == 0) return B200_OK;
+    const LatentParams& p = h.latent;
+    h.x = latent; h.x_head = p.rank; h.x_row = static_cast<int64_t>(p.rank) * p.heads;
+    h.row_count = static_cast<int>(rows); h.in = p.rank; h.out = p.vdim; h.w = p.w_value;
+    h.y = out; h.gate = gate; h.gate_stride = gate_stride;
+    h.out_hi = static_cast<__nv_bfloat16*>(out_hi); h.out_lo = static_cast<__nv_bfloat16*>(out_lo);
+    return launch_head_linear(h, as_stream(stream));
+}
+
+size_t b200_latent_scratch_bytes(const b200_latent_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length) {
+    LatentParams p;
+    if (!latent_params(args, p, true) || rows <= 0 || !latent_takes_mma(p)) return 0;
+    const int splits = latent_splits(p, sequences, max_count, max_length);
+    return splits > 1 ? static_cast<size_t>(rows) * p.heads * splits * (p.rank + 2) * sizeof(float) : 0;
+}
+
+const char* b200_latent_attention_kernel(const b200_latent_args* args) {
+    LatentParams p;
+    return latent_params(args, p, true) ? (latent_takes_mma(p) ? "latent_mma_kernel" : "latent_generic_kernel") : "";
+}
+
+int b200_latent_attention(const b200_latent_args* args, const b200_rows* pass, const float* absorbed, int32_t max_length, void* scratch,
+                          size_t scratch_bytes, float* latent_out, void* stream) {
+    LatentAttention a{};
+    if (!latent_params(args, a.latent, true) || !rows_view(pass, a.rows)) return B200_BAD_ARGUMENT;
+    if (!absorbed || !latent_out || max_length <= 0) { set_error("b200_latent_attention: operands missing"); return B200_BAD_ARGUMENT; }
+    const LatentParams& p = a.latent;
+    a.query = absorbed; a.out = latent_out;
+    if (!latent_takes_mma(p)) {
+        const size_t smem = sizeof(float) * (p.width + p.rank + kGenericKeys + 32 + 2) + sizeof(int64_t) * kGenericKeys;
+        if (smem > 200 * 1024 || a.rows.rows > 65535) { set_error("latent attention: sizes outside the generic kernel"); return B200_UNSUPPORTED; }
+        if (smem > 48 * 1024) B200_CUDA(cudaFuncSetAttribute(latent_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+        return cuda_status(launch_dependent(latent_generic_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)),
+                                            dim3(kGenericThreads), smem, as_stream(stream), a), "latent_generic_kernel launch");
+    }
+    int device = 0;
+    B200_CUDA(cudaGetDevice(&device));
+    a.status = device_status_word(device);
+    if (!a.status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
+    a.splits = latent_splits(p, a.rows.sequences, a.rows.max_count, max_length);
+    if (a.rows.sequences > 65535) { set_error("latent attention: too many sequences in one pass"); return B200_UNSUPPORTED; }
+    if (a.splits > 1) {
+        const size_t pairs = static_cast<size_t>(a.rows.rows) * p.heads * a.splits;
+        if (!scratch || scratch_bytes < pairs * (p.rank + 2) * sizeof(float)) { set_error("latent attention: scratch too small"); return B200_BAD_ARGUMENT; }
+        a.partial = static_cast<float*>(scratch);
+        a.partial_ml = a.partial + pairs * p.rank;
+    }
+    const int sequences = a.rows.sequences, max_count = a.rows.max_count;
+    const int status = latent_tile(p, max_count) == 16 ? pick_latent_mma<1>(a, sequences, max_count, as_stream(stream))
+                                                       : pick_latent_mma<2>(a, sequences, max_count, as_stream(stream));
+    if (status != B200_OK || a.splits == 1) return status;
+    return cuda_status(launch_dependent(latent_combine_kernel, dim3(static_cast<unsigned>(a.rows.rows * p.heads)), dim3(128), 0, as_stream(stream),
+                                        static_cast<const float*>(a.partial), static_cast<const float*>(a.partial_ml), a.splits, p.rank, a.out),
+                       "latent_combine_kernel launch");
+}
+
+}  // extern "C"

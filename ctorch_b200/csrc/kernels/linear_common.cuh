@@ -33,6 +33,8 @@ struct LinearParams {
     __nv_bfloat16 *out_hi, *out_lo;    // output shadow (residual: [rows, out]; SwiGLU: [rows, out/2])
     const void* out_norm_weight;       // weight of the RMSNorm that follows, folded into the output shadow
     int out_norm_dtype;
+    const float* out_norm_bias;        // set: the norm that follows is Dynamic Tanh (f32 weight and bias), which needs no row
+    float out_norm_alpha;              //   statistic; the output shadow holds tanh(alpha * row) * weight + bias
     float* sumsq_out;                  // [tiles][rows] per-tile sums of squares of the (un-weighted) result rows
     // B200_EPI_ARGMAX: per feature tile and row, the preferred value and its feature index
     float* best_value;                 // [tiles][rows]
@@ -43,6 +45,12 @@ struct LinearParams {
     float* y_copy[7];
     int copies;
 };
+
+// What the output shadow of a residual epilogue holds for the new residual value v: v * w (an RMSNorm follows, whose scale the
+// consumer applies) or the finished Dynamic Tanh norm.
+__device__ __forceinline__ float out_norm_value(const LinearParams& p, float v, float w, float bias) {
+    return p.out_norm_bias ? fmaf(tanhf(p.out_norm_alpha * v), w, bias) : __fmul_rn(v, w);
+}
 
 // The result pair of (row, feature0) to every extra destination (see LinearParams::y_copy).  The destinations are named
 // one by one: a loop over the array would index the kernel's parameters with a register, which costs a copy of the whole

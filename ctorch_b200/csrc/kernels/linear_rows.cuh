@@ -53,7 +53,8 @@ __device__ __forceinline__ void finish_pair(const LinearParams& p, int row, int 
                     wb = second ? w[1] : 0.0f;
                 }
             }
-            const float va = __fmul_rn(a, wa), vb = __fmul_rn(b, wb);
+            const float va = out_norm_value(p, a, wa, p.out_norm_bias ? p.out_norm_bias[feature0] : 0.0f);
+            const float vb = out_norm_value(p, b, wb, p.out_norm_bias && second ? p.out_norm_bias[feature0 + 1] : 0.0f);
             const __nv_bfloat162 hi = __floats2bfloat162_rn(va, vb);
             const __nv_bfloat162 lo = __floats2bfloat162_rn(va - __low2float(hi), vb - __high2float(hi));
             const int64_t at = static_cast<int64_t>(row) * p.out + feature0;
@@ -90,6 +91,7 @@ __host__ __device__ __forceinline__ bool rows_take_quads(const LinearParams& p) 
     }
     if constexpr (EPI == B200_EPI_RESIDUAL) {
         bits |= reinterpret_cast<uintptr_t>(p.residual) | (reinterpret_cast<uintptr_t>(p.out_hi) << 1) | (reinterpret_cast<uintptr_t>(p.out_lo) << 1)
+              | reinterpret_cast<uintptr_t>(p.out_norm_bias)
               | (p.out_norm_dtype == B200_BF16 ? reinterpret_cast<uintptr_t>(p.out_norm_weight) << 1 : reinterpret_cast<uintptr_t>(p.out_norm_weight));
     }
     if constexpr (EPI == B200_EPI_SWIGLU)
@@ -146,14 +148,16 @@ __device__ __forceinline__ void finish_rows_quads(const LinearParams& p, const f
     constexpr int kBatch = 4, kPasses = kTileN / 128;
     if (last > p.rows - m0) last = p.rows - m0;
     if (first >= last) return;
-    float4 norm[kPasses];
+    float4 norm[kPasses], bias[kPasses];
     bool live[kPasses];   // this lane's four features exist and the accumulators are valid
 #pragma unroll
     for (int pass = 0; pass < kPasses; ++pass) {
         const int feature0 = n0 + pass * 128 + lane * 4;
         live[pass] = ready && feature0 < p.out;
         norm[pass] = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+        bias[pass] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if constexpr (EPI == B200_EPI_RESIDUAL) {
+            if (p.out_hi && p.out_norm_bias && feature0 < p.out) bias[pass] = __ldg(reinterpret_cast<const float4*>(p.out_norm_bias + feature0));
             if (p.out_hi && p.out_norm_weight && feature0 < p.out) {
                 if (p.out_norm_dtype == B200_BF16) {
                     const uint2 w = __ldg(reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(p.out_norm_weight) + feature0));
@@ -232,8 +236,8 @@ __device__ __forceinline__ void finish_rows_quads(const LinearParams& p, const f
                     sum[r][pass] = t;
                     squares[r] += t.x * t.x + t.y * t.y;
                     squares[r] += t.z * t.z + t.w * t.w;
-                    const float a = __fmul_rn(t.x, norm[pass].x), b = __fmul_rn(t.y, norm[pass].y), c2 = __fmul_rn(t.z, norm[pass].z),
-                                d = __fmul_rn(t.w, norm[pass].w);
+                    const float a = out_norm_value(p, t.x, norm[pass].x, bias[pass].x), b = out_norm_value(p, t.y, norm[pass].y, bias[pass].y),
+                                c2 = out_norm_value(p, t.z, norm[pass].z, bias[pass].z), d = out_norm_value(p, t.w, norm[pass].w, bias[pass].w);
                     const __nv_bfloat162 hi0 = __floats2bfloat162_rn(a, b), hi1 = __floats2bfloat162_rn(c2, d);
                     const __nv_bfloat162 lo0 = __floats2bfloat162_rn(a - __low2float(hi0), b - __high2float(hi0));
                     const __nv_bfloat162 lo1 = __floats2bfloat162_rn(c2 - __low2float(hi1), d - __high2float(hi1));

@@ -288,6 +288,14 @@ extern "C" int b200_linear_shadow(const b200_shadow_linear_args* args, void* str
     p.sumsq_in = args->sumsq_in; p.parts_in = args->parts_in;
     p.out_hi = static_cast<__nv_bfloat16*>(args->out_hi); p.out_lo = static_cast<__nv_bfloat16*>(args->out_lo);
     p.out_norm_weight = args->out_norm_weight; p.out_norm_dtype = args->out_norm_dtype; p.sumsq_out = args->sumsq_out;
+    if (args->out_norm) {
+        if (epilogue != B200_EPI_RESIDUAL || !args->out_hi || !args->out_norm->weight || !args->out_norm->bias) {
+            set_error("b200_linear_shadow: an elementwise norm needs the residual epilogue, output planes, weight and bias");
+            return B200_BAD_ARGUMENT;
+        }
+        p.out_norm_weight = args->out_norm->weight; p.out_norm_dtype = B200_F32;
+        p.out_norm_bias = args->out_norm->bias; p.out_norm_alpha = args->out_norm->alpha;
+    }
     p.best_value = args->best_value; p.best_index = args->best_index;
     if (args->copies < 0 || args->copies > 7 || (args->copies > 0 && (!args->y_copies || (epilogue != B200_EPI_STORE && epilogue != B200_EPI_RESIDUAL)))) {
         set_error("b200_linear_shadow: at most 7 result copies, for store and residual epilogues only");

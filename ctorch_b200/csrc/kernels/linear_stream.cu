@@ -399,7 +399,8 @@ __global__ void __launch_bounds__(kThreads, 2) linear_stream_kernel(const Stream
                             wb = second ? w[1] : 0.0f;
                         }
                     }
-                    const float va = __fmul_rn(a, wa), vb = __fmul_rn(b, wb);
+                    const float va = out_norm_value(p, a, wa, p.out_norm_bias ? p.out_norm_bias[feature0] : 0.0f);
+                    const float vb = out_norm_value(p, b, wb, p.out_norm_bias ? p.out_norm_bias[feature0 + 1] : 0.0f);
                     const __nv_bfloat162 hi = __floats2bfloat162_rn(va, vb);
                     const __nv_bfloat162 lo = __floats2bfloat162_rn(va - __low2float(hi), vb - __high2float(hi));
                     const int64_t at = static_cast<int64_t>(row) * p.out + feature0;  // out is even on this path

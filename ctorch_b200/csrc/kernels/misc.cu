@@ -63,6 +63,14 @@ encode_tiled_fn tensor_map_encoder() {
 
 namespace {
 
+// out[r, :] = x[index[r], :]
+__global__ void gather_rows_kernel(const float* x, const int32_t* index, int64_t width, float* out) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x, from = index[row];
+    for (int64_t c = threadIdx.x; c < width; c += blockDim.x) out[row * width + c] = x[from * width + c];
+}
+
 template <class T>
 __global__ void embedding_kernel(const T* table, const int64_t* ids, int64_t rows, int64_t vocab, int64_t width, float* out,
                                  int32_t* status) {
@@ -470,6 +478,13 @@ int b200_permute(const float* in, const int64_t* sizes, const int64_t* order, in
     if (count == 0) return B200_OK;
     b200::permute_kernel<<<b200::blocks_for(count), 256, 0, as_stream(stream)>>>(in, shape, count, out);
     return cuda_status(cudaGetLastError(), "permute_kernel launch");
+}
+
+int b200_gather_rows(const float* x, const int32_t* index, int64_t rows, int64_t width, float* out, void* stream) {
+    if (!x || !index || !out || rows < 0 || width <= 0) { set_error("b200_gather_rows: bad pointer or size"); return B200_BAD_ARGUMENT; }
+    if (rows == 0) return B200_OK;
+    return cuda_status(launch_dependent(b200::gather_rows_kernel, dim3(static_cast<unsigned>(rows)), dim3(256), 0, as_stream(stream), x, index, width,
+                                        out), "gather_rows_kernel launch");
 }
 
 int b200_token_feedback(const int64_t* next, int64_t batch, int64_t* ids, int64_t* history, int64_t history_rows,

@@ -1,0 +1,510 @@
+// State-space layers (Mamba-2): short causal convolution, selective recurrence, gated group norm; and the small kernels of
+// packed passes.  Everything here is f32: decays, step sizes, states and norms.
+//
+//   * Decode (one row per sequence): ssm_step_kernel, one CTA per (head, sequence).  It convolves the channels its head needs
+//     from the slot's ring of recent inputs, then streams the head's [state][vdim] matrix through registers once: load,
+//     decay, add dt B x^T, store, and the partial sums of S^T C on the way.  The layer is bound by that traffic
+//     (8 bytes per state value and token).
+//   * Longer passes: short_conv_kernel over all rows, conv_ring_kernel (the last inputs into the slot's ring), and
+//     ssm_scan_kernel: the state lives in registers across the whole pass, spread over a warp as state-dimension slices
+//     x 4 value columns per lane; tokens are staged through a double-buffered shared-memory chunk; products go two at a
+//     time through the packed f32 pipe.
+// The ring has `taps` entries although a token needs only taps - 1 old inputs: the entry a step writes is never one that the
+// same step reads, so the CTAs of a head group need no ordering among themselves.
+#include "rows.cuh"
+
+#include <cmath>
+
+namespace b200 {
+
+bool rows_view(const b200_rows* pass, RowsView& view) {
+    if (!pass || pass->rows <= 0 || pass->rows > INT32_MAX || pass->sequences <= 0 || pass->sequences > pass->rows || pass->max_count <= 0
+        || pass->max_count > pass->rows || !pass->slot || !pass->first || !pass->sequence || !pass->lengths) {
+        set_error("inconsistent packed pass (b200_rows)");
+        return false;
+    }
+    view = RowsView{static_cast<int>(pass->rows), pass->sequences, pass->max_count, pass->slot, pass->first, pass->sequence, pass->lengths};
+    return true;
+}
+
+namespace {
+
+struct SsmParams {
+    int heads, vdim, state, groups, taps, channels, stride;
+    const float *conv_weight, *conv_bias, *dt_bias, *a_log, *d;
+    float *conv_state, *ssm_state;
+    const float* projected;
+    float *mixed, *y;
+};
+
+__device__ __forceinline__ float softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
+__device__ __forceinline__ float sigmoid_exact(float v) { return 1.0f / (1.0f + expf(-v)); }
+
+// Input of the convolution at `position` of a slot, from the ring of earlier passes (zero before the sequence's start).
+__device__ __forceinline__ float ring_input(const SsmParams& p, int slot, int position, int channel) {
+    if (position < 0) return 0.0f;
+    return p.conv_state[(static_cast<int64_t>(slot) * p.taps + position % p.taps) * p.channels + channel];
+}
+
+constexpr int kStepThreads = 256;
+
+template <int V> struct Lanes { float v[V]; };
+template <int V> __device__ __forceinline__ Lanes<V> load_lanes(const float* p) {
+    Lanes<V> r;
+    if constexpr (V == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(p);
+        r.v[0] = q.x; r.v[1] = q.y; r.v[2] = q.z; r.v[3] = q.w;
+    } else {
+        r.v[0] = p[0];
+    }
+    return r;
+}
+template <int V> __device__ __forceinline__ void store_lanes(float* p, const Lanes<V>& r) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else p[0] = r.v[0];
+}
+
+// grid (heads, sequences); one row per sequence.  V = 4 when vdim is a multiple of 4.
+template <int V>
+__global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams p, const RowsView rows) {
+    extern __shared__ __align__(16) float sm[];   // [vdim + 2 state] convolved channels, then [threads * V] partial outputs
+    const int P = p.vdim, N = p.state, head = blockIdx.x, row = blockIdx.y;
+    const int group = head / (p.heads / p.groups), inner = p.heads * P;
+    float* mixed = sm;
+    float* partial = sm + ((P + 2 * N + 3) & ~3);
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const RowPlace place = row_place(rows, row);
+    const float* in = p.projected + static_cast<int64_t>(row) * p.stride;
+    const bool fresh = place.position == 0;
+    float* state = p.ssm_state + (static_cast<int64_t>(place.slot) * p.heads + head) * N * P;
+
+    // this thread's part of the state: value columns p0.., every `slices`-th state row; the first batch is requested before
+    // the convolution so that its latency is covered
+    const int columns = P / V, slices = kStepThreads / columns > 0 ? kStepThreads / columns : 1;
+    constexpr int kAhead = 8;
+
+    const bool shared_writer = head % (p.heads / p.groups) == 0;
+    for (int i = threadIdx.x; i < P + 2 * N; i += kStepThreads) {
+        const int c = i < P ? head * P + i : i < P + N ? inner + group * N + (i - P) : inner + (p.groups + group) * N + (i - P - N);
+        const float now = in[inner + c];
+        float acc = p.conv_bias[c];
+        for (int j = 0; j < p.taps - 1; ++j)
+            acc = fmaf(p.conv_weight[static_cast<int64_t>(c) * p.taps + j], ring_input(p, place.slot, place.position - (p.taps - 1 - j), c), acc);
+        acc = fmaf(p.conv_weight[static_cast<int64_t>(c) * p.taps + p.taps - 1], now, acc);
+        mixed[i] = acc * sigmoid_exact(acc);
+        if (i < P || shared_writer)
+            p.conv_state[(static_cast<int64_t>(place.slot) * p.taps + place.position % p.taps) * p.channels + c] = now;
+    }
+    const float dt = softplus(in[inner + p.channels + head] + p.dt_bias[head]);
+    const float decay = expf(-expf(p.a_log[head]) * dt);
+    __syncthreads();
+    const float *x = mixed, *B = mixed + P, *C = mixed + P + N;
+
+    for (int base = 0; base < columns; base += kStepThreads) {
+        const int column = base + (columns <= kStepThreads ? static_cast<int>(threadIdx.x) % columns : static_cast<int>(threadIdx.x));
+        const int slice = columns <= kStepThreads ? static_cast<int>(threadIdx.x) / columns : 0;
+        const bool active = column < columns && slice < slices;
+        Lanes<V> sum;
+#pragma unroll
+        for (int k = 0; k < V; ++k) sum.v[k] = 0.0f;
+        if (active) {
+            Lanes<V> xd;
+#pragma unroll
+            for (int k = 0; k < V; ++k) xd.v[k] = x[column * V + k] * dt;
+            for (int n0 = slice; n0 < N; n0 += slices * kAhead) {
+                Lanes<V> s[kAhead];
+#pragma unroll
+                for (int i = 0; i < kAhead; ++i) {
+                    const int n = n0 + i * slices;
+#pragma unroll
+                    for (int k = 0; k < V; ++k) s[i].v[k] = 0.0f;
+                    if (!fresh && n < N) s[i] = load_lanes<V>(state + static_cast<int64_t>(n) * P + column * V);
+                }
+#pragma unroll
+                for (int i = 0; i < kAhead; ++i) {
+                    const int n = n0 + i * slices;
+                    if (n >= N) continue;
+                    const float b = B[n], c = C[n];
+#pragma unroll
+                    for (int k = 0; k < V; ++k) {
+                        s[i].v[k] = fmaf(s[i].v[k], decay, xd.v[k] * b);
+                        sum.v[k] = fmaf(s[i].v[k], c, sum.v[k]);
+                    }
+                    store_lanes<V>(state + static_cast<int64_t>(n) * P + column * V, s[i]);
+                }
+            }
+        }
+        __syncthreads();
+        store_lanes<V>(partial + threadIdx.x * V, sum);
+        __syncthreads();
+        const int width = columns <= kStepThreads ? columns : min(kStepThreads, columns - base);
+        for (int i = threadIdx.x; i < width * V; i += kStepThreads) {
+            float total = 0.0f;
+            for (int s = 0; s < slices; ++s) total += partial[(s * (columns <= kStepThreads ? columns : 0)) * V + i];
+            const int at = base * V + i;
+            p.y[static_cast<int64_t>(row) * inner + head * P + at] = fmaf(p.d[head], x[at], total);
+        }
+    }
+}
+
+// mixed[row, c] = silu(conv(x | B | C)), grid (channel blocks, rows)
+__global__ void __launch_bounds__(256) short_conv_kernel(const SsmParams p, const RowsView rows) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, row = blockIdx.y;
+    if (c >= p.channels) return;
+    const RowPlace place = row_place(rows, row);
+    const int offset = row - __ldg(rows.first + place.sequence), inner = p.heads * p.vdim;
+    const float* in = p.projected + static_cast<int64_t>(row) * p.stride + inner + c;
+    const float* weight = p.conv_weight + static_cast<int64_t>(c) * p.taps;
+    float acc = p.conv_bias[c];
+    for (int j = 0; j < p.taps; ++j) {
+        const int back = p.taps - 1 - j;   // how many tokens before this one
+        const float v = back <= offset ? in[-static_cast<int64_t>(back) * p.stride] : ring_input(p, place.slot, place.position - back, c);
+        acc = fmaf(weight[j], v, acc);
+    }
+    p.mixed[static_cast<int64_t>(row) * p.channels + c] = acc * sigmoid_exact(acc);
+}
+
+// The last inputs of every sequence into its slot's ring, grid (channel blocks, sequences)
+__global__ void __launch_bounds__(256) conv_ring_kernel(const SsmParams p, const RowsView rows) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, s = blockIdx.y;
+    if (c >= p.channels) return;
+    const int first = __ldg(rows.first + s), count = __ldg(rows.first + s + 1) - first, slot = __ldg(rows.slot + s);
+    const int length = rows.lengths[slot], inner = p.heads * p.vdim;
+    for (int t = max(0, count - p.taps); t < count; ++t)
+        p.conv_state[(static_cast<int64_t>(slot) * p.taps + (length + t) % p.taps) * p.channels + c] =
+            p.projected[static_cast<int64_t>(first + t) * p.stride + inner + c];
+}
+
+// ---- scan -----------------------------------------------------------------------------------------------------
+// Packed f32 pairs: two independent IEEE operations per instruction.
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ void copy_async_4(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+
+constexpr int kScanWarps = 4;
+
+// LN lanes of a warp share the state dimension (4 * Q values each, in quads LN * 4 apart), the other 32 / LN lane groups hold
+// four value columns each.  grid (column tiles, heads, sequences).
+template <int LN, int Q>
+__global__ void __launch_bounds__(kScanWarps * 32) ssm_scan_kernel(const SsmParams p, const RowsView rows) {
+    constexpr int kNp = LN * 4 * Q;                      // padded state size
+    constexpr int kScanTokens = kNp <= 128 ? 16 : 4;     // tokens staged at a time
+    constexpr int kGroups = 32 / LN;
+    constexpr int kColumns = kScanWarps * kGroups * 4;   // value columns of the CTA
+    __shared__ __align__(16) float sB[2][kScanTokens][kNp], sC[2][kScanTokens][kNp], sx[2][kScanTokens][kColumns];
+    __shared__ float sdt[2][kScanTokens];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int P = p.vdim, N = p.state, head = blockIdx.y, s = blockIdx.z, column0 = blockIdx.x * kColumns;
+    const int group = head / (p.heads / p.groups), inner = p.heads * P;
+    const int first = __ldg(rows.first + s), count = __ldg(rows.first + s + 1) - first, slot = __ldg(rows.slot + s);
+    const bool fresh = rows.lengths[slot] == 0;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, ln = lane % LN, lg = lane / LN;
+    const int local = (warp * kGroups + lg) * 4;         // first of this lane's four value columns inside the tile
+    const int column = column0 + local;
+    float* state = p.ssm_state + (static_cast<int64_t>(slot) * p.heads + head) * N * P;
+
+    for (int i = threadIdx.x; i < 2 * kScanTokens * kNp; i += blockDim.x) { (&sB[0][0][0])[i] = 0.0f; (&sC[0][0][0])[i] = 0.0f; }
+    for (int i = threadIdx.x; i < 2 * kScanTokens * kColumns; i += blockDim.x) (&sx[0][0][0])[i] = 0.0f;
+    __syncthreads();
+
+    uint64_t S[4][2 * Q];
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int q = 0; q < 2 * Q; ++q) {
+            const int n = (q >> 1) * LN * 4 + ln * 4 + (q & 1) * 2;
+            float a = 0.0f, b = 0.0f;
+            if (!fresh && column + k < P) {
+                if (n < N) a = state[static_cast<int64_t>(n) * P + column + k];
+                if (n + 1 < N) b = state[static_cast<int64_t>(n + 1) * P + column + k];
+            }
+            S[k][q] = pack2(a, b);
+        }
+    const float rate = -expf(p.a_log[head]), dt_bias = p.dt_bias[head], skip = p.d[head];
+    const int live_columns = min(kColumns, P - column0);
+
+    auto stage = [&](int chunk) {
+        const int buffer = chunk & 1, t0 = chunk * kScanTokens, tokens = min(kScanTokens, count - t0);
+        const int width = live_columns + 2 * N;
+        for (int i = threadIdx.x; i < tokens * width; i += blockDim.x) {
+            const int t = i / width, c = i - t * width;
+            const float* row = p.mixed + static_cast<int64_t>(first + t0 + t) * p.channels;
+            if (c < live_columns) copy_async_4(&sx[buffer][t][c], row + head * P + column0 + c);
+            else if (c < live_columns + N) copy_async_4(&sB[buffer][t][c - live_columns], row + inner + group * N + (c - live_columns));
+            else copy_async_4(&sC[buffer][t][c - live_columns - N], row + inner + (p.groups + group) * N + (c - live_columns - N));
+        }
+        if (threadIdx.x < tokens)
+            copy_async_4(&sdt[buffer][threadIdx.x], p.projected + static_cast<int64_t>(first + t0 + threadIdx.x) * p.stride + inner + p.channels + head);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+
+    const int chunks = (count + kScanTokens - 1) / kScanTokens;
+    stage(0);
+    for (int chunk = 0; chunk < chunks; ++chunk) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                  // the chunk has landed; the other buffer is free
+        if (chunk + 1 < chunks) stage(chunk + 1);
+        const int buffer = chunk & 1, t0 = chunk * kScanTokens, tokens = min(kScanTokens, count - t0);
+        // step size and decay of token `lane` of the chunk, handed round by shuffles
+        float dt_mine = 0.0f, decay_mine = 1.0f;
+        if (lane < tokens) {
+            dt_mine = softplus(sdt[buffer][lane] + dt_bias);
+            decay_mine = expf(rate * dt_mine);
+        }
+        for (int t = 0; t < tokens; ++t) {
+            const float dt = __shfl_sync(0xffffffffu, dt_mine, t), decay = __shfl_sync(0xffffffffu, decay_mine, t);
+            const float4 xv = *reinterpret_cast<const float4*>(&sx[buffer][t][local]);
+            const float x[4] = {xv.x, xv.y, xv.z, xv.w};
+            const uint64_t decay2 = pack2(decay, decay);
+            uint64_t xd[4], acc[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { xd[k] = pack2(x[k] * dt, x[k] * dt); acc[k] = pack2(0.0f, 0.0f); }
+#pragma unroll
+            for (int q = 0; q < Q; ++q) {
+                const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(&sB[buffer][t][q * LN * 4 + ln * 4]);
+                const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(&sC[buffer][t][q * LN * 4 + ln * 4]);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    S[k][2 * q] = fma2(S[k][2 * q], decay2, mul2(xd[k], b.x));
+                    acc[k] = fma2(S[k][2 * q], c.x, acc[k]);
+                    S[k][2 * q + 1] = fma2(S[k][2 * q + 1], decay2, mul2(xd[k], b.y));
+                    acc[k] = fma2(S[k][2 * q + 1], c.y, acc[k]);
+                }
+            }
+            float part[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) { const float2 v = unpack2(acc[k]); part[k] = v.x + v.y; }
+            // sum over the LN lanes: two exchanges halve the four columns, the rest are plain butterflies
+            const bool odd = lane & 1, second = lane & 2;
+            const float keep0 = odd ? part[2] : part[0], give0 = odd ? part[0] : part[2];
+            const float keep1 = odd ? part[3] : part[1], give1 = odd ? part[1] : part[3];
+            const float two0 = keep0 + __shfl_xor_sync(0xffffffffu, give0, 1), two1 = keep1 + __shfl_xor_sync(0xffffffffu, give1, 1);
+            float one = (second ? two1 : two0) + __shfl_xor_sync(0xffffffffu, second ? two0 : two1, 2);
+#pragma unroll
+            for (int o = 4; o < LN; o <<= 1) one += __shfl_xor_sync(0xffffffffu, one, o);
+            const int k = (odd ? 2 : 0) + (second ? 1 : 0);
+            if (ln < 4 && column + k < P) {
+                const float mine = k == 0 ? x[0] : k == 1 ? x[1] : k == 2 ? x[2] : x[3];
+                p.y[static_cast<int64_t>(first + t0 + t) * inner + head * P + column + k] = fmaf(skip, mine, one);
+            }
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+#pragma unroll
+        for (int q = 0; q < 2 * Q; ++q) {
+            const int n = (q >> 1) * LN * 4 + ln * 4 + (q & 1) * 2;
+            const float2 v = unpack2(S[k][q]);
+            if (column + k < P) {
+                if (n < N) state[static_cast<int64_t>(n) * P + column + k] = v.x;
+                if (n + 1 < N) state[static_cast<int64_t>(n + 1) * P + column + k] = v.y;
+            }
+        }
+}
+
+template <int LN, int Q> int launch_scan(const SsmParams& p, const RowsView& rows, cudaStream_t stream) {
+    constexpr int kColumns = kScanWarps * (32 / LN) * 4;
+    const dim3 grid(static_cast<unsigned>((p.vdim + kColumns - 1) / kColumns), static_cast<unsigned>(p.heads), static_cast<unsigned>(rows.sequences));
+    return cuda_status(launch_dependent(ssm_scan_kernel<LN, Q>, grid, dim3(kScanWarps * 32), 0, stream, p, rows), "ssm_scan_kernel launch");
+}
+
+// grid (rows, parts)
+__global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* y, const float* z, int64_t z_stride, const float* weight, int width,
+                                                               int parts, float eps, float* out, __nv_bfloat16* out_hi, __nv_bfloat16* out_lo) {
+    __shared__ float scratch[32];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    const int size = width / parts, c0 = blockIdx.y * size;
+    constexpr int kKeep = 8;   // values a thread keeps in registers; longer parts are computed again
+    float kept[kKeep];
+    float squares = 0.0f;
+    auto value = [&](int c) {
+        const float g = z[row * z_stride + c0 + c];
+        return y[row * width + c0 + c] * (g * sigmoid_exact(g));
+    };
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+        const int c = threadIdx.x + i * 256;
+        kept[i] = c < size ? value(c) : 0.0f;
+        squares = fmaf(kept[i], kept[i], squares);
+    }
+    for (int c = threadIdx.x + kKeep * 256; c < size; c += 256) {
+        const float v = value(c);
+        squares = fmaf(v, v, squares);
+    }
+    squares = block_sum(squares, scratch);
+    const float inverse = 1.0f / sqrtf(squares / static_cast<float>(size) + eps);
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < size) store_forms(kept[i] * inverse * weight[c0 + c], row * width + c0 + c, out, out_hi, out_lo);
+    }
+    for (int c = threadIdx.x + kKeep * 256; c < size; c += 256)
+        store_forms(value(c) * inverse * weight[c0 + c], row * width + c0 + c, out, out_hi, out_lo);
+}
+
+__global__ void rows_advance_kernel(const RowsView rows) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int s = blockIdx.x * blockDim.x + threadIdx.x;
+    if (s < rows.sequences) rows.lengths[rows.slot[s]] += rows.first[s + 1] - rows.first[s];
+}
+
+__global__ void __launch_bounds__(256) dynamic_tanh_kernel(const float* x, const float* add_rows, const float* add_vector, int width,
+                                                           b200_elementwise_norm norm, float* sum, float* out, __nv_bfloat16* out_hi,
+                                                           __nv_bfloat16* out_lo) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
+        const int64_t at = row * width + c;
+        float v = x[at];
+        if (add_rows) v += add_rows[at];
+        if (add_vector) v += add_vector[c];
+        if (sum) sum[at] = v;
+        store_forms(fmaf(tanhf(norm.alpha * v), norm.weight[c], norm.bias[c]), at, out, out_hi, out_lo);
+    }
+}
+
+template <class T>
+__global__ void __launch_bounds__(256) embedding_scaled_kernel(const T* table, const int64_t* ids, int64_t vocab, int64_t width, float scale,
+                                                               float* out, int32_t* status) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t row = blockIdx.x;
+    int64_t id = ids[row];
+    if (id < 0 || id >= vocab) {   // the host API validates ids it can see; device-resident ids are clamped and flagged
+        if (threadIdx.x == 0) atomicExch(status, B200_BAD_ARGUMENT);
+        id = id < 0 ? 0 : vocab - 1;
+    }
+    for (int64_t c = threadIdx.x; c < width; c += blockDim.x) out[row * width + c] = load_as_f32(table, id * width + c) * scale;
+}
+
+}  // namespace
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" {
+
+int b200_rows_advance(const b200_rows* pass, void* stream) {
+    RowsView rows;
+    if (!rows_view(pass, rows)) return B200_BAD_ARGUMENT;
+    return cuda_status(launch_dependent(rows_advance_kernel, dim3((rows.sequences + 127) / 128), dim3(128), 0, as_stream(stream), rows),
+                       "rows_advance_kernel launch");
+}
+
+int b200_embedding_scaled(const void* table, int32_t table_dtype, const int64_t* ids, int64_t rows, int64_t vocab, int64_t width, float scale,
+                          float* out, void* stream) {
+    if (!table || !ids || !out || rows < 0 || vocab <= 0 || width <= 0) { set_error("b200_embedding_scaled: bad pointer or size"); return B200_BAD_ARGUMENT; }
+    if (rows == 0) return B200_OK;
+    int device = 0;
+    B200_CUDA(cudaGetDevice(&device));
+    int32_t* status = device_status_word(device);
+    if (!status) { set_error("b200_embedding_scaled: the device status word could not be allocated"); return B200_NO_DEVICE; }
+    const dim3 grid(static_cast<unsigned>(rows));
+    if (table_dtype == B200_BF16)
+        return cuda_status(launch_dependent(embedding_scaled_kernel<__nv_bfloat16>, grid, dim3(256), 0, as_stream(stream),
+                                            static_cast<const __nv_bfloat16*>(table), ids, vocab, width, scale, out, status), "embedding_scaled_kernel launch");
+    if (table_dtype == B200_F32)
+        return cuda_status(launch_dependent(embedding_scaled_kernel<float>, grid, dim3(256), 0, as_stream(stream), static_cast<const float*>(table),
+                                            ids, vocab, width, scale, out, status), "embedding_scaled_kernel launch");
+    set_error("b200_embedding_scaled: table dtype %d is not f32 or bf16", table_dtype);
+    return B200_UNSUPPORTED;
+}
+
+int b200_dynamic_tanh(const float* x, const float* add_rows, const float* add_vector, int64_t rows, int64_t width,
+                      const b200_elementwise_norm* norm, float* sum, float* out, void* out_hi, void* out_lo, void* stream) {
+    if (!x || !norm || !norm->weight || !norm->bias || rows < 0 || width <= 0 || width > INT32_MAX || (!out && !out_hi)) {
+        set_error("b200_dynamic_tanh: bad pointer or size");
+        return B200_BAD_ARGUMENT;
+    }
+    if (rows == 0) return B200_OK;
+    const unsigned slices = static_cast<unsigned>(rows >= 512 ? 1 : (width + 1023) / 1024);
+    return cuda_status(launch_dependent(dynamic_tanh_kernel, dim3(static_cast<unsigned>(rows), slices), dim3(256), 0, as_stream(stream), x, add_rows,
+                                        add_vector, static_cast<int>(width), *norm, sum, out, static_cast<__nv_bfloat16*>(out_hi),
+                                        static_cast<__nv_bfloat16*>(out_lo)), "dynamic_tanh_kernel launch");
+}
+
+int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream) {
+    RowsView rows;
+    if (!rows_view(pass, rows)) return B200_BAD_ARGUMENT;
+    if (!a || a->heads <= 0 || a->vdim <= 0 || a->state <= 0 || a->groups <= 0 || a->heads % a->groups || a->taps <= 0 || !a->conv_weight
+        || !a->conv_bias || !a->dt_bias || !a->a_log || !a->d || !a->conv_state || !a->ssm_state || !a->projected || !a->y) {
+        set_error("b200_ssm_forward: bad pointer or size");
+        return B200_BAD_ARGUMENT;
+    }
+    SsmParams p{};
+    p.heads = a->heads; p.vdim = a->vdim; p.state = a->state; p.groups = a->groups; p.taps = a->taps;
+    p.channels = a->heads * a->vdim + 2 * a->groups * a->state;
+    p.stride = a->heads * a->vdim + p.channels + a->heads;
+    p.conv_weight = a->conv_weight; p.conv_bias = a->conv_bias; p.dt_bias = a->dt_bias; p.a_log = a->a_log; p.d = a->d;
+    p.conv_state = a->conv_state; p.ssm_state = a->ssm_state; p.projected = a->projected; p.mixed = a->mixed; p.y = a->y;
+    cudaStream_t s = as_stream(stream);
+    if (rows.max_count == 1) {
+        const bool quads = a->vdim % 4 == 0 && (reinterpret_cast<uintptr_t>(a->ssm_state) & 15) == 0;
+        const size_t smem = sizeof(float) * (((a->vdim + 2 * a->state + 3) & ~3) + kStepThreads * (quads ? 4 : 1));
+        if (smem > 200 * 1024) { set_error("b200_ssm_forward: a head of %d x %d values does not fit shared memory", a->state, a->vdim); return B200_UNSUPPORTED; }
+        auto kernel = quads ? ssm_step_kernel<4> : ssm_step_kernel<1>;
+        if (smem > 48 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+        return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(a->heads), static_cast<unsigned>(rows.sequences)), dim3(kStepThreads),
+                                            smem, s, p, rows), "ssm_step_kernel launch");
+    }
+    if (!a->mixed) { set_error("b200_ssm_forward: workspace missing"); return B200_BAD_ARGUMENT; }
+    if (a->state > B200_SSM_MAX_STATE) { set_error("b200_ssm_forward: state sizes above %d are not supported", B200_SSM_MAX_STATE); return B200_UNSUPPORTED; }
+    if (rows.sequences > 65535) { set_error("b200_ssm_forward: too many sequences in one pass"); return B200_UNSUPPORTED; }
+    const unsigned blocks = static_cast<unsigned>((p.channels + 255) / 256);
+    if (rows.rows > 65535) { set_error("b200_ssm_forward: at most 65535 rows in one pass"); return B200_UNSUPPORTED; }
+    int status = cuda_status(launch_dependent(short_conv_kernel, dim3(blocks, static_cast<unsigned>(rows.rows)), dim3(256), 0, s, p, rows), "short_conv_kernel launch");
+    if (status != B200_OK) return status;
+    status = cuda_status(launch_dependent(conv_ring_kernel, dim3(blocks, static_cast<unsigned>(rows.sequences)), dim3(256), 0, s, p, rows), "conv_ring_kernel launch");
+    if (status != B200_OK) return status;
+    if (a->state <= 32) return launch_scan<8, 1>(p, rows, s);
+    if (a->state <= 64) return launch_scan<8, 2>(p, rows, s);
+    if (a->state <= 96) return launch_scan<8, 3>(p, rows, s);
+    if (a->state <= 128) return launch_scan<8, 4>(p, rows, s);
+    if (a->state <= 256) return launch_scan<32, 2>(p, rows, s);
+    return launch_scan<32, 4>(p, rows, s);
+}
+
+int b200_gated_group_norm(const float* y, const float* z, int64_t z_stride, const float* weight, int64_t rows, int64_t width, int32_t parts,
+                          double eps, float* out, void* out_hi, void* out_lo, void* stream) {
+    if (!y || !z || !weight || rows < 0 || width <= 0 || width > INT32_MAX || parts <= 0 || width % parts || parts > 65535 || (!out && !out_hi)) {
+        set_error("b200_gated_group_norm: bad pointer or size");
+        return B200_BAD_ARGUMENT;
+    }
+    if (rows == 0) return B200_OK;
+    return cuda_status(launch_dependent(gated_group_norm_kernel, dim3(static_cast<unsigned>(rows), static_cast<unsigned>(parts)), dim3(256), 0,
+                                        as_stream(stream), y, z, z_stride, weight, static_cast<int>(width), static_cast<int>(parts),
+                                        static_cast<float>(eps), out, static_cast<__nv_bfloat16*>(out_hi), static_cast<__nv_bfloat16*>(out_lo)),
+                       "gated_group_norm_kernel launch");
+}
+
+}  // extern "C"

@@ -212,6 +212,38 @@ DL_API dl_status dl_generation_profile_step(dl_generation* generation, double mi
 DL_API dl_status dl_decoder_generate(dl_module* decoder, dl_module* embedding, dl_module* output,
     const dl_tensor* prompt, int64_t steps, dl_decoder_cache* cache, dl_tensor** tokens);
 
+/* ---- models from configurations (no counterpart in the reference) -----------------------------------------
+ * A model design is chosen by "architecture" of a JSON configuration: "Ripitar" (hybrid decoder: state-space and latent-attention
+ * layers, Dynamic Tanh norms, looped layers) or "TransformerDecoder" (the grouped-query decoder above with its embedding and
+ * output layers; keys vocab, layers, width, heads, kv_heads, ff, context, tied). */
+DL_API const char* dl_model_architectures(void);   /* comma-separated */
+DL_API dl_status dl_model_create(const char* config_json, dl_tensor_options options, dl_module** output);
+/* config.json and model.safetensors of a folder; weights are converted to options.dtype (DL_BF16 or DL_F32). */
+DL_API dl_status dl_model_load(const char* folder, dl_tensor_options options, dl_module** output);
+DL_API dl_status dl_state_load_safetensors(const char* path, dl_state** output);
+/* Hybrid decoders: `slots` sequences of up to `capacity` tokens.  Grouped-query decoders: their own caches (both numbers unused). */
+DL_API dl_status dl_model_cache_create(const dl_module* model, int64_t slots, int64_t capacity, dl_decoder_cache** output);
+DL_API dl_status dl_model_cache_release_slot(dl_decoder_cache* cache, int64_t slot);
+DL_API dl_status dl_model_cache_slot_length(const dl_decoder_cache* cache, int64_t slot, int64_t* length);
+/* One sequence's share of a pass: its next tokens, and the places among them whose logits are wanted. */
+typedef struct dl_pass_entry {
+    int64_t slot;
+    const int64_t* tokens;
+    size_t token_count;
+    const int64_t* want;
+    size_t want_count;
+} dl_pass_entry;
+/* Runs the entries as one batch (any lengths, each from what earlier passes left in its slot); logits: host, [wanted, vocabulary] in
+ * the order of the entries and of their wants. */
+DL_API dl_status dl_model_pass(dl_module* model, dl_decoder_cache* cache, const dl_pass_entry* entries, size_t count, float* logits);
+/* The same for one entry, returning the residual stream after every layer run instead of logits: host, [runs, tokens, width]. */
+DL_API dl_status dl_model_trail(dl_module* model, dl_decoder_cache* cache, const dl_pass_entry* entry, float* trail, size_t trail_floats);
+DL_API dl_status dl_model_set_activation_dtype(dl_module* model, dl_dtype dtype);
+/* The generation loop for a model made here; sequence b of the batch lives in slot b. */
+DL_API dl_status dl_model_generation_create(dl_module* model, dl_decoder_cache* cache, int64_t batch, int64_t max_steps, dl_generation** result);
+/* dl_generation_prefill for prompts of unequal length: row b of prompt [batch, length] counts for its first lengths[b] ids. */
+DL_API dl_status dl_generation_prefill_lengths(dl_generation* generation, const dl_tensor* prompt, const int64_t* lengths);
+
 /* KV-head tensor parallelism (one process per GPU).  A group is one NCCL communicator per device: one rank asks for
  * a 128-byte id, every rank receives it by whatever transport the application has and joins.  A decoder then computes
  * slice `rank` of `world`: query heads, KV heads and SwiGLU features are split evenly; norms, the residual stream, the

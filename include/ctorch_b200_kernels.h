@@ -128,6 +128,13 @@ B200_API int b200_linear(const float* x, int64_t rows, int64_t in, const void* w
  * An RMSNorm between producer and consumer is split: the producer folds the norm weight into the shadow and leaves
  * per-row partial sums of squares of the un-weighted values; the consumer multiplies its results by
  * 1/sqrt(sum/width + eps).  The f32 arithmetic differs from the reference's f64 norm by rounding only. */
+/* Dynamic Tanh, a norm without mean or variance: tanh(alpha * x) * weight + bias.  f32 vectors [width] on the device. */
+typedef struct b200_elementwise_norm {
+    float alpha;
+    const float* weight;
+    const float* bias;
+} b200_elementwise_norm;
+
 typedef struct b200_shadow_linear_args {
     const void* x_hi;              /* bf16 [rows, in] */
     const void* x_lo;              /* may be NULL for calls the dense kernel serves (more than 16 rows or in > 2048): the
@@ -151,6 +158,8 @@ typedef struct b200_shadow_linear_args {
     int32_t* best_index;           /* B200_EPI_ARGMAX: same shape, feature index of best_value */
     float* const* y_copies;        /* store / residual epilogues: `copies` (0..7) further [rows, out] f32 matrices that receive the */
     int32_t copies;                /*   same rows as y - a tensor-parallel rank's slot in each peer's memory (plain peer stores) */
+    const b200_elementwise_norm* out_norm; /* residual epilogue: the norm that follows needs no row statistic; the output shadow holds the
+                                      normed rows themselves (out_norm_weight and sumsq_out are then unused) */
 } b200_shadow_linear_args;
 /* Up to 16 rows with in <= 2048: streaming kernel (bulk-TMA weight ring, mma.sync).  More rows or a wider input:
  * dense tcgen05 kernel (TMA operand tiles, accumulator in tensor memory; K split over a thread-block cluster when the
@@ -248,6 +257,9 @@ B200_API int b200_sample(const float* x, int64_t rows, int64_t width, double tem
 B200_API int b200_select_rows(const float* x, int64_t first, int64_t stride, int64_t rows_out, int64_t width,
                               float* out, void* stream);
 
+/* out[r, :] = x[index[r], :] for row numbers in device memory (the rows of a packed pass whose logits are wanted). */
+B200_API int b200_gather_rows(const float* x, const int32_t* index, int64_t rows, int64_t width, float* out, void* stream);
+
 /* dl::rotary_embedding (src/ops/contraction.cpp:44-49): x [outer, length, head_dim] f32, tables [length, head_dim/2];
  * adjacent pairs, each product rounded before the subtraction / addition. */
 B200_API int b200_rotary(const float* x, int64_t outer, int64_t length, int64_t head_dim, const float* cosine,
@@ -302,6 +314,102 @@ B200_API int b200_tp_argmax_finish(void* const* regions, int32_t rank, int32_t w
                                    const float* best_value, const int32_t* best_index, int32_t parts, int64_t rows, int64_t* next,
                                    int64_t* ids, int64_t* history, int64_t history_rows, int32_t* counter,
                                    b200_kv_cache* const* caches, int32_t cache_count, void* stream);
+
+/* ---- hybrid decoders: packed passes, elementwise norms, state-space layers, latent attention --------------------------
+ * (no counterpart in the reference, whose one decoder is grouped-query attention + SwiGLU)
+ *
+ * A pass runs `rows` activation rows of `sequences` sequences, packed: sequence s owns the rows first[s] .. first[s+1]-1
+ * in order of position, whatever the other sequences bring, and lives in cache slot slot[s].  Row r of sequence s is the
+ * token at position lengths[slot[s]] + r - first[s]; lengths counts what earlier passes left in the slot.  A slot whose
+ * length is 0 starts afresh: nothing it held before is read.  All arrays are int32 in device memory. */
+typedef struct b200_rows {
+    int64_t rows;
+    int32_t sequences;
+    int32_t max_count;             /* host: the largest number of rows of one sequence */
+    const int32_t* slot;           /* [sequences] */
+    const int32_t* first;          /* [sequences + 1] */
+    const int32_t* sequence;       /* [rows] the sequence of each row */
+    int32_t* lengths;              /* [slots] */
+} b200_rows;
+
+/* lengths[slot[s]] += rows of s, for every sequence of the pass. */
+B200_API int b200_rows_advance(const b200_rows* pass, void* stream);
+
+/* out[r, :] = f32(table[ids[r], :]) * scale */
+B200_API int b200_embedding_scaled(const void* table, int32_t table_dtype, const int64_t* ids, int64_t rows, int64_t vocab,
+                                   int64_t width, float scale, float* out, void* stream);
+
+/* Residual stream at a point where no projection ends: x[r, :] (+ add_rows[r, :]) (+ add_vector[:]) -> sum (may be NULL or
+ * equal x), and Dynamic Tanh of it -> out (f32, may be NULL) and / or the shadow planes out_hi / out_lo (may be NULL). */
+B200_API int b200_dynamic_tanh(const float* x, const float* add_rows, const float* add_vector, int64_t rows, int64_t width,
+                               const b200_elementwise_norm* norm, float* sum, float* out, void* out_hi, void* out_lo, void* stream);
+
+/* State-space layer (Mamba-2): sizes, parameters (f32), and the per-slot state.
+ * The projected row is [z: heads*vdim | x: heads*vdim | B: groups*state | C: groups*state | dt: heads]; x, B and C pass the
+ * causal convolution per channel and SiLU.  Per head h of group g = h / (heads / groups):
+ *   dt = softplus(dt + dt_bias), S = exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + d x.
+ * conv_state [slots][taps][channels]: the input of position p in entry p mod taps; ssm_state [slots][heads][state][vdim]. */
+typedef struct b200_ssm_args {
+    int32_t heads, vdim, state, groups, taps;
+    const float* conv_weight;      /* [channels, taps], last column = current token */
+    const float* conv_bias;        /* [channels] */
+    const float* dt_bias;          /* [heads] */
+    const float* a_log;            /* [heads] */
+    const float* d;                /* [heads] */
+    float* conv_state;
+    float* ssm_state;
+    const float* projected;        /* [rows, 2*heads*vdim + 2*groups*state + heads] */
+    float* mixed;                  /* workspace [rows, heads*vdim + 2*groups*state], unused by passes of one row per sequence */
+    float* y;                      /* [rows, heads*vdim] */
+} b200_ssm_args;
+/* Convolution, step sizes, recurrence and its output for every row; the slots' states move on.  Passes with one row per
+ * sequence run as one kernel bound by the state's traffic, longer ones as convolution + scan. */
+B200_API int b200_ssm_forward(const b200_ssm_args* args, const b200_rows* pass, void* stream);
+/* Largest state size (N) the scan keeps in registers. */
+#define B200_SSM_MAX_STATE 512
+
+/* v = y * silu(z), then an RMS norm of each of `parts` equal parts of the row, times weight [width].  z has z_stride floats
+ * between rows.  Result as f32 (out) and / or shadow planes. */
+B200_API int b200_gated_group_norm(const float* y, const float* z, int64_t z_stride, const float* weight, int64_t rows, int64_t width,
+                                   int32_t parts, double eps, float* out, void* out_hi, void* out_lo, void* stream);
+
+/* One-pool cache of a latent-attention layer: per token kv_rank latent values and the shared rotated key part, width values
+ * in all, paged like the other caches with one head.  `lengths` [slots] is the caller's. */
+B200_API int b200_latent_cache_create(int32_t device, int32_t dtype, int32_t slots, int32_t width, int32_t capacity, int32_t page_size,
+                                      int32_t* lengths, b200_kv_cache** out);
+
+typedef struct b200_latent_args {
+    int32_t heads, dim, rot_dim, vdim, kv_rank, q_rank, rot_dims;   /* rot_dims: leading entries of the rot_dim part that rotate */
+    float scale;
+    double eps;
+    const float* cosine;           /* [positions, rot_dims / 2] */
+    const float* sine;
+    int32_t positions;
+    const float* q_norm;           /* [q_rank] f32 */
+    const float* kv_norm;          /* [kv_rank] f32 */
+    b200_kv_cache* cache;          /* width kv_rank + rot_dim */
+    int32_t weight_dtype;
+    const void* w_key;             /* per head transposed key up-projection [heads][kv_rank][dim] */
+    const void* w_value;           /* value up-projection [heads][vdim][kv_rank] */
+} b200_latent_args;
+/* projected [rows, q_rank + kv_rank + rot_dim + heads*vdim] = [query latent | latent | rotated key part | gate].  RMS-norms the
+ * query latent (-> q_latent f32 or planes), RMS-norms the latent, rotates the key part and appends both to the cache. */
+B200_API int b200_latent_prepare(const b200_latent_args* args, const b200_rows* pass, const float* projected, float* q_latent,
+                                 void* q_hi, void* q_lo, void* stream);
+/* query [rows, heads, dim + rot_dim] -> absorbed [rows, heads, kv_rank + rot_dim]: the unrotated part through the head's key
+ * up-projection, the rotated part turned by its position. */
+B200_API int b200_latent_query(const b200_latent_args* args, const b200_rows* pass, const float* query, float* absorbed, void* stream);
+/* Causal softmax attention of the absorbed queries over the cached latents; latent_out [rows, heads, kv_rank] f32 is the
+ * weighted sum of latents.  max_length bounds lengths[slot] + rows of any sequence. */
+B200_API size_t b200_latent_scratch_bytes(const b200_latent_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length);
+B200_API int b200_latent_attention(const b200_latent_args* args, const b200_rows* pass, const float* absorbed, int32_t max_length,
+                                   void* scratch, size_t scratch_bytes, float* latent_out, void* stream);
+/* Value up-projection of every head times sigmoid(gate): [rows, heads*vdim] as f32 (out) or planes.  gate has gate_stride
+ * floats between rows. */
+B200_API int b200_latent_value(const b200_latent_args* args, int64_t rows, const float* latent, const float* gate, int64_t gate_stride,
+                               float* out, void* out_hi, void* out_lo, void* stream);
+/* Name of the kernel b200_latent_attention runs for these sizes: "latent_mma_kernel" or "latent_generic_kernel". */
+B200_API const char* b200_latent_attention_kernel(const b200_latent_args* args);
 
 #ifdef __cplusplus
 }
