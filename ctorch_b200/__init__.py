@@ -260,7 +260,7 @@ class Tensor:
 
     @staticmethod
     def from_numpy(array: np.ndarray, device: Device | None = None, dtype: int | None = None) -> "Tensor":
-        array = np.ascontiguousarray(array)
+        array = np.asarray(array, order="C")   # (ascontiguousarray would make a scalar a vector)
         code = dtype if dtype is not None else _CODE_OF[array.dtype]
         shape, keep = _shape(array.shape)
         out = C.c_void_p()
@@ -564,7 +564,7 @@ class LanguageModel:
             state = {}
             for name, tensor in self.module.state().items():
                 if name in weights:
-                    array = np.ascontiguousarray(weights[name])
+                    array = np.asarray(weights[name], order="C")
                     state[name] = Tensor.from_numpy(array, dtype=BF16 if array.dtype == np.uint16 else None)
                     if state[name].dtype != tensor.dtype:
                         state[name] = state[name].astype(tensor.dtype)
