@@ -8,7 +8,8 @@ d 2048, 16 layers, 32/8 heads, SwiGLU 8192, bf16 weights, 256 independent sequen
 and prompts are seeded synthetic data.  With N > 1 (one process per GPU under torch.distributed.run) the 256 sequences
 are divided over the GPUs (256 / N each), weights replicated, no collective on the data path: strong scaling.
 `--workload c5` is the 8B shape with adapters, KV-head tensor parallel over the GPUs; `c2` the small decoder (replicas);
-`c3` the decode-attention microbenchmark; `linear` one projection in isolation.
+`c3` the decode-attention microbenchmark; `linear` one projection in isolation; `hybrid` prefill and decode of the hybrid
+decoder beside the grouped-query decoder of equal size (`--size`).
 
 The printed JSON line carries the device-resident throughput (`value`: median of 5 timed rounds of K steps), the
 host-in-the-loop throughput through the C ABI (`e2e`), the roofline of the kernel class that dominates the step
@@ -630,13 +631,78 @@ def run_linear(args) -> dict:
     return line if rank == 0 else {}
 
 
+def measure_model(config: dict, args, local: int, prompt_len: int, prefill_batch: int, batches: list[int]) -> dict:
+    """Prefill and decode throughput of a model made from a configuration, through the same loop for every design."""
+    import ctorch_b200 as B
+    shapes = {n: t.shape for n, t in B.LanguageModel(config, None, device=None).module.state().items() if "rotary." not in n}
+    model = B.LanguageModel(config, W.random_state(shapes), device=local)
+    if args.activations == "bf16" and config["architecture"] == "Ripitar":
+        model.set_activation_dtype("bf16")
+    rng = np.random.default_rng(5)
+    steps = args.steps + args.warmup + 8
+    result = {"parameters": int(sum(np.prod(s, dtype=np.int64) for s in shapes.values())), "decode": {}}
+
+    def prefill(gen, batch):
+        B.timer_start(local)
+        gen.prefill(rng.integers(0, config["vocab"], (batch, prompt_len)))
+        return B.timer_stop(local)
+
+    for batch in sorted({*batches, prefill_batch}, reverse=True):
+        model.new_cache(batch, prompt_len + steps + 1)
+        gen = B.Generation(model, batch, steps + 1)
+        first = prefill(gen, batch)
+        if batch == prefill_batch:   # the first pass packs weights and allocates: the median of three warm ones counts
+            times = []
+            for _ in range(3):
+                model.cache.clear()
+                gen = B.Generation(model, batch, steps + 1)
+                times.append(prefill(gen, batch))
+            ms = sorted(times)[1]
+            result["prefill"] = {"batch": batch, "prompt": prompt_len, "ms": ms, "tokens_per_s": batch * prompt_len / ms * 1e3, "first_ms": first}
+        if batch not in batches:
+            continue
+        gen.step(args.warmup)
+        B.synchronize(local)
+        B.timer_start(local)
+        gen.step(args.steps)
+        ms = B.timer_stop(local) / args.steps
+        result["decode"][str(batch)] = {"ms_per_step": ms, "tokens_per_s": batch / ms * 1e3, "launches": gen.launches_per_step(),
+                                        "profile": gen.profile_step()}
+        del gen
+    return result
+
+
+def run_hybrid(args) -> dict:
+    """The hybrid decoder beside the grouped-query decoder of equal width, feed-forward and number of layer runs (one GPU)."""
+    rank, world, local, dist = distributed()
+    if world > 1:
+        raise SystemExit("the hybrid workload runs on one GPU")
+    prompt, prefill_batch = args.prompt, 8
+    hybrid, grouped = W.HYBRID_SIZES[args.size]
+    batches = [args.batch] if args.batch > 0 else [1, 16, 64, 256]
+    sampler = ClockSampler(local)
+    sampler.start()
+    sampler.mark()
+    ours = measure_model(W.hybrid_config(**hybrid), args, local, prompt, prefill_batch, batches)
+    other = None
+    if not args.no_secondary:
+        other = measure_model(W.transformer_config(**grouped, context=prompt + args.steps + args.warmup + 16), args, local, prompt, prefill_batch, batches)
+    clocks = sampler.stop()
+    top = ours["decode"][str(max(batches))]
+    return {"metric": METRIC, "value": top["tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+            "ms_per_step": top["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"model": f"hybrid {args.size}", "global_batch": max(batches), "seq_len": prompt, "parallelism": "dp1",
+                       "l2": "every step streams more than L2 (weights, states, latents)"},
+            "clocks": clocks, "gpu_launches": top["launches"] * args.steps, "hybrid": ours, "grouped_query": other}
+
+
 def main():
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
     parser.add_argument("--steps", type=int, default=64)
     parser.add_argument("--warmup", type=int, default=8)
     parser.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    parser.add_argument("--workload", default="c4", choices=["c1", "c2", "c3", "c4", "c5", "linear"])
+    parser.add_argument("--workload", default="c4", choices=["c1", "c2", "c3", "c4", "c5", "linear", "hybrid"])
     parser.add_argument("--activations", default="f32", choices=["f32", "bf16"],
                         help="bf16 decoders: precision of the activations between kernels in passes over more than 16 rows")
     parser.add_argument("--batch", type=int, default=0, help="decoder workloads: override the configuration's batch (e.g. c4 with 32 = one GPU's share of the 8-GPU run)")
@@ -647,12 +713,14 @@ def main():
     parser.add_argument("--cpu-steps", type=int, default=4, help="timed CPU-baseline steps of the default run")
     parser.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     parser.add_argument("--no-secondary", action="store_true", help="c4 on one GPU: skip the c3 and c2 companions of the record")
+    parser.add_argument("--size", default="2k", choices=sorted(W.HYBRID_SIZES), help="hybrid only: layer sizes")
+    parser.add_argument("--prompt", type=int, default=1024, help="hybrid only: prompt length")
     parser.add_argument("--small", action="store_true", help="c3 only: batch 16, contexts up to 8192 (profiler captures)")
     args = parser.parse_args()
     if args.warmup < 3:
         args.warmup = 3
-    if args.workload in ("c3", "linear"):
-        line = run_c3(args) if args.workload == "c3" else run_linear(args)
+    if args.workload in ("c3", "linear", "hybrid"):
+        line = {"c3": run_c3, "linear": run_linear, "hybrid": run_hybrid}[args.workload](args)
         if line:
             print(json.dumps(line))
         return

@@ -127,3 +127,49 @@ def kv_bytes_per_token(spec: dict, kv_dtype: str) -> int:
     """Bytes of K and V one cached position holds across all layers, per sequence."""
     hd = spec["d_model"] // spec["heads"]
     return 2 * spec["layers"] * spec["kv_heads"] * hd * (2 if kv_dtype == "bf16" else 4)
+
+
+def hybrid_config(width: int, layers: int, ff: int, heads: int, ssm_heads: int, loop: tuple[int, int, int] | None = None,
+                  vocab: int = 32000) -> dict:
+    """Hybrid decoder of a real model's layer sizes: state-space and latent-attention layers in turn, each with a feed-forward."""
+    ssm = {"type": "mamba2", "mixer": {"heads": ssm_heads, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8},
+           "mlp": {"kind": "dense", "ff": ff}}
+    latent = {"type": "latent_attention",
+              "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 768, "scale": 192 ** -0.5,
+                        "rot": {"dims": 64, "base": 10000.0}},
+              "mlp": {"kind": "dense", "ff": ff}}
+    config = {"architecture": "Ripitar", "vocab": vocab, "width": width, "layers": [(ssm, latent)[i % 2] for i in range(layers)],
+              "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "logit_scale": 1.0}
+    if loop:
+        config["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return config
+
+
+def transformer_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, context: int, vocab: int = 32000) -> dict:
+    return {"architecture": "TransformerDecoder", "vocab": vocab, "layers": layers, "width": width, "heads": heads, "kv_heads": kv_heads,
+            "ff": ff, "context": context, "tied": 1}
+
+
+# (hybrid, grouped-query) arguments of equal width, feed-forward width and number of layer runs
+HYBRID_SIZES = {
+    "1k": (dict(width=1024, layers=12, ff=4096, heads=8, ssm_heads=32), dict(width=1024, layers=12, ff=4096, heads=16, kv_heads=4)),
+    "2k": (dict(width=2048, layers=12, ff=8192, heads=16, ssm_heads=64, loop=(4, 8, 2)), dict(width=2048, layers=16, ff=8192, heads=32, kv_heads=8)),
+    "4k": (dict(width=4096, layers=8, ff=14336, heads=32, ssm_heads=128), dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8)),
+}
+
+
+def random_state(shapes: dict[str, tuple[int, ...]], seed: int = 7) -> dict[str, np.ndarray]:
+    """bf16 bit patterns for every named shape, cut from one seeded block (norm-like vectors around 1)."""
+    block = np.random.default_rng(seed).standard_normal(1 << 22, dtype=np.float32)
+    out = {}
+    for i, (name, shape) in enumerate(shapes.items()):
+        count = int(np.prod(shape)) if shape else 1
+        values = np.resize(block[i * 9973 % 65536:], count).reshape(shape)
+        if len(shape) == 2:
+            values = values * np.float32(shape[1] ** -0.5)
+        elif not name.endswith((".b", "A_log", "dt_bias")):
+            values = 1.0 + 0.05 * values
+        else:
+            values = 0.2 * values
+        out[name] = bf16_bits(values).reshape(shape)
+    return out
