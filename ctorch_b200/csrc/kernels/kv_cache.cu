@@ -63,7 +63,8 @@ __global__ void append_kernel(KvView kv, const float* key, const float* value, i
 
 int make_maps(b200_kv_cache* c) {
     c->has_maps = false;
-    if (c->dtype != B200_BF16 || c->page_size != kFastPageSize || c->head_dim % 64 != 0) return B200_OK;
+    const bool latent = !c->pool[1];   // one pool: boxes may reach past the width (zero-filled), rows only need 16-byte strides
+    if (c->dtype != B200_BF16 || c->page_size != kFastPageSize || c->head_dim % (latent ? 8 : 64) != 0) return B200_OK;
     encode_tiled_fn encode = tensor_map_encoder();
     if (!encode) { set_error("cuTensorMapEncodeTiled is not available from this driver"); return B200_NO_DEVICE; }
     // 2-D view [token rows][head_dim] of a pool; one box = 64 tokens x 64 features (128-byte rows, 128B swizzle).
@@ -72,7 +73,7 @@ int make_maps(b200_kv_cache* c) {
     const cuuint64_t strides[1] = {static_cast<cuuint64_t>(c->head_dim) * 2};
     const cuuint32_t box[2] = {64, static_cast<cuuint32_t>(kFastPageSize)};
     const cuuint32_t element_strides[2] = {1, 1};
-    for (int which = 0; which < 2; ++which) {
+    for (int which = 0; which < (latent ? 1 : 2); ++which) {
         const CUresult result = encode(&c->map[which], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c->pool[which], dims, strides,
                                        box, element_strides, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                                        CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
@@ -135,7 +136,7 @@ static int create_cache(int32_t device, int32_t dtype, int32_t sequences, int32_
         if (e != cudaSuccess) return fail(cuda_status(e, "cudaMemset(lengths)"));
     }
     c->even_lengths = true;
-    const int status = pools == 2 ? make_maps(c) : B200_OK;
+    const int status = make_maps(c);
     if (status != B200_OK) return fail(status);
     *out = c;
     return B200_OK;

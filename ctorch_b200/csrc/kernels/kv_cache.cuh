@@ -48,7 +48,7 @@ __device__ __forceinline__ float kv_load(const KvView& kv, int which, int64_t at
 }
 
 KvView kv_view(const b200_kv_cache* cache);
-// Tensor maps (bf16 pools with head_dim % 64 == 0 and 64-token pages only); nullptr otherwise.
+// Tensor maps (bf16 pools with 64-token pages and head_dim % 64 == 0, latent pools with width % 8 == 0); nullptr otherwise.
 const CUtensorMap* kv_tensor_map(const b200_kv_cache* cache, int which);
 
 }  // namespace b200

@@ -3,11 +3,11 @@
 // (b200_latent_query), attends to the latents themselves, and the weighted latent goes through the value up-projection
 // (b200_latent_value).  Every cached byte serves all heads as key and as value.
 //
-//   * latent_mma_kernel: bf16 caches.  A producer warp copies pages row by row (bulk copies into padded rows, mbarrier ring);
-//     eight consumer warps hold the queries as tensor-core fragments in registers, the query-key product split 4 ways over the
-//     width and 2 ways over the keys of a page; the partial scores meet in shared memory, a warp finishes whole rows of the
+//   * latent_mma_kernel: bf16 caches.  Pages arrive through a TMA ring as boxes of 64 tokens x 64 values (128-byte swizzle, values
+//     past the width zero-filled, mbarrier completion); the consumer warps hold the queries as tensor-core fragments in registers, the query-key product split 4 ways over the
+//     width and 4 or 2 ways over the keys of a page; the partial scores meet in shared memory, a warp finishes whole rows of the
 //     online softmax in f32; then every warp multiplies the weights (as hi + lo planes) with its columns of the same page.
-//     Decode: 16 rows (heads of one token), the queries as hi + lo planes.  Longer passes and wide head counts: 32 rows.
+//     Decode: 16 rows (heads of one token), 16 warps.  Longer passes and wide head counts: 32 rows, 8 warps.
 //   * latent_generic_kernel: f32 caches and odd sizes, f32 FMAs, one (row, head) per CTA.
 #include "kv_cache.cuh"
 #include "mma.cuh"
@@ -115,6 +115,24 @@ __device__ __forceinline__ void head_result(const HeadLinear& h, int row, int he
         const float g = h.gate[row * h.gate_stride + column];
         store_forms(v * (1.0f / (1.0f + expf(-g))), row * static_cast<int64_t>(h.latent.heads) * h.out + column, h.y, h.out_hi, h.out_lo);
     }
+}
+// Two adjacent results (o even) of the tensor-core form.
+__device__ __forceinline__ void head_pair(const HeadLinear& h, int row, int head, int o, float a, float b) {
+    if (h.query && (h.latent.width & 1) == 0 && o + 1 < h.out) {
+        *reinterpret_cast<float2*>(h.y + (static_cast<int64_t>(row) * h.latent.heads + head) * h.latent.width + o) = make_float2(a, b);
+        return;
+    }
+    if (!h.query && !h.y && o + 1 < h.out && (h.out & 1) == 0 && h.out_lo) {
+        const int64_t column = static_cast<int64_t>(head) * h.out + o, at = row * static_cast<int64_t>(h.latent.heads) * h.out + column;
+        const float* gate = h.gate + row * h.gate_stride + column;
+        uint32_t hi, lo;
+        pack_planes(a * (1.0f / (1.0f + expf(-gate[0]))), b * (1.0f / (1.0f + expf(-gate[1]))), hi, lo);
+        *reinterpret_cast<uint32_t*>(h.out_hi + at) = hi;
+        *reinterpret_cast<uint32_t*>(h.out_lo + at) = lo;
+        return;
+    }
+    head_result(h, row, head, o, a);
+    if (o + 1 < h.out) head_result(h, row, head, o + 1, b);
 }
 __device__ __forceinline__ void head_rotated(const HeadLinear& h, int row, int head, int i) {
     const LatentParams& p = h.latent;
@@ -226,9 +244,9 @@ template <int WM> __global__ void __launch_bounds__(kHeadThreads) head_linear_mm
 #pragma unroll
     for (int n = 0; n < kTiles; ++n)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int row = m + (i >> 1) * 8, o = c + n * 8 + (i & 1);
-            if (row < h.row_count && o < h.out) head_result(h, row, head, o, acc[n][i]);
+        for (int i = 0; i < 2; ++i) {
+            const int row = m + i * 8, o = c + n * 8;
+            if (row < h.row_count && o < h.out) head_pair(h, row, head, o, acc[n][2 * i], acc[n][2 * i + 1]);
         }
     if (h.query && blockIdx.x == 0)
         for (int i = threadIdx.x; i < M * h.latent.rot_dim; i += kHeadThreads) {
@@ -271,25 +289,47 @@ struct LatentAttention {
     int32_t* status;
 };
 
-constexpr int kPage = 64, kConsumerWarps = 8, kConsumerThreads = kConsumerWarps * 32, kLatentThreads = kConsumerThreads + 32;
+constexpr int kPage = 64;
 constexpr int kScorePitch = 68, kWeightPitch = 72;
 constexpr float kLog2e = 1.4426950408889634f;
 
-int latent_row_bytes(int width) { return (((width + 15) & ~15) + 8) * 2; }   // odd multiple of 16 bytes: conflict-free ldmatrix
+constexpr int kBoxBytes = kPage * 64 * 2;   // one box of a page: 64 tokens x 64 values
 int latent_fixed_bytes(int m) { return 4 * m * kScorePitch * 4 + 2 * m * kWeightPitch * 2 + 4 * m * 4 + 256; }
 
-__device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kConsumerThreads) : "memory"); }
+// KS: 16-wide steps of the width per quarter; VT: 8-column tiles of the latent per warp; MT: 16-row tiles.
+// MT = 1 (decode steps): 16 consumer warps and a producer warp, so that four warps per scheduler hide the products' latency and the
+// copies run ahead on their own.  MT = 2 (longer passes, whose pages come from L2): 8 warps, which leaves 255 registers for the
+// queries' and the result's fragments; warp 0 issues the copies as pages are finished with.
+template <int MT> struct LatentShape {
+    static constexpr int kWarps = MT == 1 ? 16 : 8, kConsumers = kWarps * 32;
+    static constexpr bool kProducer = MT == 1;
+    static constexpr int kThreads = kConsumers + (kProducer ? 32 : 0);
+};
+template <int THREADS> __device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
-// KS: 16-wide steps of the width per quarter; VT: 8-column tiles of the latent per warp; MT: 16-row tiles.  MT = 1 multiplies the
-// queries as hi + lo planes.
+// Called by a whole warp.
+__device__ __forceinline__ void latent_copy_page(const CUtensorMap* map, const int32_t* table, int page, uint8_t* stage, int boxes, uint64_t* full) {
+    const int row = __ldg(table + page) * kPage;
+    if (elect_one()) {
+        mbar_expect_tx(full, static_cast<uint32_t>(boxes * kBoxBytes));
+        for (int b = 0; b < boxes; ++b) tma_load_2d(stage + b * kBoxBytes, map, b * 64, row, full);
+    }
+    __syncwarp();
+}
+// Byte offset of 16-byte chunk `chunk` (8 values) of a row inside a staged page: boxes side by side, the chunk swizzled by its row.
+__device__ __forceinline__ uint32_t page_offset(int row, int chunk) {
+    return static_cast<uint32_t>((chunk >> 3) * kBoxBytes + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
+}
+
 template <int KS, int VT, int MT>
-__global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __grid_constant__ LatentAttention a) {
-    constexpr int M = 16 * MT, kPlanes = 2;   // fragments per step: planes (MT = 1) or row tiles (MT = 2)
+__global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kernel(const __grid_constant__ LatentAttention a, const __grid_constant__ CUtensorMap map) {
+    using Shape = LatentShape<MT>;
+    constexpr int M = 16 * MT, kWarps = Shape::kWarps, kGroups = kWarps / 4, kKeyTiles = kPage / 8 / kGroups;   // key tiles per warp
     extern __shared__ __align__(16) uint8_t smem[];
     const LatentParams& p = a.latent;
-    const int row_elements = ((p.width + 15) & ~15) + 8, stage_elements = kPage * row_elements;
-    __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem);
-    float* scores = reinterpret_cast<float*>(ring + a.stages * stage_elements);      // [4][M][kScorePitch]
+    const int boxes = (p.width + 63) >> 6, stage_bytes = boxes * kBoxBytes;
+    uint8_t* ring = smem + ((1024u - (smem_u32(smem) & 1023u)) & 1023u);             // swizzled boxes start on 1024-byte boundaries
+    float* scores = reinterpret_cast<float*>(ring + a.stages * stage_bytes);         // [4][M][kScorePitch]
     __nv_bfloat16* weights = reinterpret_cast<__nv_bfloat16*>(scores + 4 * M * kScorePitch);   // [2 planes][M][kWeightPitch]
     float* shrink = reinterpret_cast<float*>(weights + 2 * M * kWeightPitch);       // [M] factor of the accumulators
     float* row_m = shrink + M;
@@ -301,11 +341,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int split = blockIdx.z % a.splits, chunk = blockIdx.z / a.splits, sequence = blockIdx.y;
-    // columns past the width are read by the products (times zero): they must be finite
-    for (int i = threadIdx.x; i < a.stages * kPage; i += kLatentThreads)
-        for (int c = p.width; c < row_elements; ++c) ring[i * row_elements + c] = __float2bfloat16_rn(0.0f);
     if (threadIdx.x == 0) {
-        for (int s = 0; s < a.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], kConsumerWarps); }
+        tma_prefetch_descriptor(&map);
+        for (int s = 0; s < a.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], kWarps); }
         mbar_fence_init();
         *gave_up = 0;
     }
@@ -328,27 +366,25 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
     }
     __syncthreads();
 
-    if (warp == kConsumerWarps) {   // producer
-        const int32_t* table = p.kv.page_table + static_cast<int64_t>(slot) * p.kv.pages_per_seq;
-        const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(p.kv.pool[0]);
-        const uint32_t bytes = static_cast<uint32_t>(p.width) * 2;
+    const int32_t* table = p.kv.page_table + static_cast<int64_t>(slot) * p.kv.pages_per_seq;
+    if (Shape::kProducer && warp == kWarps) {
         for (int t = page0; t < page1; ++t) {
             const int i = t - page0, s = i % a.stages;
             if (i >= a.stages && !mbar_wait(&empty[s], ((i / a.stages) - 1) & 1)) {
                 if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
                 break;
             }
-            if (lane == 0) mbar_expect_tx(&full[s], bytes * kPage);
-            __syncwarp();
-            const __nv_bfloat16* page = pool + static_cast<int64_t>(__ldg(table + t)) * kPage * p.width;
-            for (int r = lane; r < kPage; r += 32) bulk_load(ring + s * stage_elements + r * row_elements, page + r * p.width, bytes, &full[s]);
+            latent_copy_page(&map, table, t, ring + s * stage_bytes, boxes, &full[s]);
         }
         return;
     }
+    if (!Shape::kProducer && warp == 0)   // all stages but one; the last is kept for the page that follows the one in work
+        for (int t = page0; t < min(page1, page0 + a.stages - 1); ++t)
+            latent_copy_page(&map, table, t, ring + (t - page0) * stage_bytes, boxes, &full[t - page0]);
 
     // queries as A fragments: quarter `quarter` of the width
-    const int quarter = warp & 3, half = warp >> 2, steps = (p.width + 15) >> 4;
-    uint32_t q[KS][kPlanes][4];
+    const int quarter = warp & 3, group = warp >> 2, steps = (p.width + 15) >> 4;
+    uint32_t q[KS][MT][4];
     {
         const float* source[2 * MT];
 #pragma unroll
@@ -368,8 +404,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
                     const int at = k + (part >> 1) * 8;
                     float2 v = make_float2(0.0f, 0.0f);
                     if (from && at < p.width) v = *reinterpret_cast<const float2*>(from + at);
-                    if constexpr (MT == 1) pack_planes(v.x, v.y, q[i][0][part], q[i][1][part]);
-                    else q[i][mt][part] = pack_bf16(v.x, v.y);
+                    q[i][mt][part] = pack_bf16(v.x, v.y);
                 }
         }
     }
@@ -380,13 +415,13 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
         for (int v = 0; v < VT; ++v)
 #pragma unroll
             for (int i = 0; i < 4; ++i) o[mt][v][i] = 0.0f;
-    constexpr int kOwn = M / kConsumerWarps;   // rows whose softmax this warp keeps
+    constexpr int kOwn = M / kWarps;   // rows whose softmax this warp keeps; l_own is each lane's share of the sum
     float m_own[kOwn], l_own[kOwn];
 #pragma unroll
     for (int r = 0; r < kOwn; ++r) { m_own[r] = -INFINITY; l_own[r] = 0.0f; }
     const float scale2 = p.scale * kLog2e;
-    const uint32_t key_lane = static_cast<uint32_t>(((half * 32 + (lane >> 4) * 8 + (lane & 7)) * row_elements + ((lane >> 3) & 1) * 8) * 2);
-    const int value_columns = ((p.width + 15) & ~15);
+    const int key_row = group * kKeyTiles * 8 + (lane >> 4) * 8 + (lane & 7), key_chunk = (lane >> 3) & 1, value_chunks = boxes * 8;
+    constexpr int kSpan = VT >= 4 ? 4 : 2;   // value tiles worked at a time
     bool alive = true;
 
     for (int t = page0; t < page1; ++t) {
@@ -395,12 +430,12 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
             if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
             *static_cast<volatile int*>(gave_up) = 1;
         }
-        const uint32_t page = smem_u32(ring + s * stage_elements);
-        float sc[MT][4][4];
+        const uint32_t page = smem_u32(ring + s * stage_bytes);
+        float sc[MT][kKeyTiles][4];
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-            for (int n = 0; n < 4; ++n)
+            for (int n = 0; n < kKeyTiles; ++n)
 #pragma unroll
                 for (int j = 0; j < 4; ++j) sc[mt][n][j] = 0.0f;
 #pragma unroll
@@ -408,20 +443,13 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
             const int step = quarter * KS + k;
             if (step < steps) {
 #pragma unroll
-                for (int n = 0; n < 4; n += 2) {
+                for (int n = 0; n < kKeyTiles; n += 2) {
                     uint32_t b[4];
-                    ldsm_x4(b, page + key_lane + static_cast<uint32_t>(n * 8 * row_elements * 2 + step * 32));
-                    if constexpr (MT == 1) {
-                        mma_16816(sc[0][n], q[k][0], b[0], b[1]);
-                        mma_16816(sc[0][n + 1], q[k][0], b[2], b[3]);
-                        mma_16816(sc[0][n], q[k][1], b[0], b[1]);
-                        mma_16816(sc[0][n + 1], q[k][1], b[2], b[3]);
-                    } else {
+                    ldsm_x4(b, page + page_offset(key_row + n * 8, step * 2 + key_chunk));
 #pragma unroll
-                        for (int mt = 0; mt < MT; ++mt) {
-                            mma_16816(sc[mt][n], q[k][mt], b[0], b[1]);
-                            mma_16816(sc[mt][n + 1], q[k][mt], b[2], b[3]);
-                        }
+                    for (int mt = 0; mt < MT; ++mt) {
+                        mma_16816(sc[mt][n], q[k][mt], b[0], b[1]);
+                        mma_16816(sc[mt][n + 1], q[k][mt], b[2], b[3]);
                     }
                 }
             }
@@ -429,13 +457,18 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-            for (int n = 0; n < 4; ++n) {
-                float* at = scores + (quarter * M + mt * 16 + (lane >> 2)) * kScorePitch + half * 32 + n * 8 + (lane & 3) * 2;
+            for (int n = 0; n < kKeyTiles; ++n) {
+                float* at = scores + (quarter * M + mt * 16 + (lane >> 2)) * kScorePitch + (group * kKeyTiles + n) * 8 + (lane & 3) * 2;
                 *reinterpret_cast<float2*>(at) = make_float2(sc[mt][n][0], sc[mt][n][1]);
                 *reinterpret_cast<float2*>(at + 8 * kScorePitch) = make_float2(sc[mt][n][2], sc[mt][n][3]);
             }
-        consumers_sync();
+        consumers_sync<Shape::kConsumers>();
         if (*static_cast<volatile int*>(gave_up)) { alive = false; break; }   // a page never arrived: every consumer leaves here
+        if (!Shape::kProducer && warp == 0 && t + a.stages - 1 < page1) {
+            // every warp is past the products of page t - 1: its stage takes the next page
+            const int next = t + a.stages - 1, into = (next - page0) % a.stages;
+            latent_copy_page(&map, table, next, ring + into * stage_bytes, boxes, &full[into]);
+        }
 #pragma unroll
         for (int r = 0; r < kOwn; ++r) {
             const int m = warp * kOwn + r, sees = visible[m] - t * kPage;
@@ -450,7 +483,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
             const float top = fmaxf(m_own[r], warp_max(fmaxf(v0, v1)));
             const float base = top == -INFINITY ? 0.0f : top;
             const float p0 = exp2f(v0 - base), p1 = exp2f(v1 - base), factor = exp2f(m_own[r] - base);
-            l_own[r] = l_own[r] * factor + warp_sum(p0 + p1);
+            l_own[r] = l_own[r] * factor + (p0 + p1);
             m_own[r] = top;
             if (lane == 0) shrink[m] = factor;
             __nv_bfloat16 hi, lo;
@@ -461,7 +494,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
             weights[m * kWeightPitch + lane + 32] = hi;
             weights[(M + m) * kWeightPitch + lane + 32] = lo;
         }
-        consumers_sync();
+        consumers_sync<Shape::kConsumers>();
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
             const float f0 = shrink[mt * 16 + (lane >> 2)], f1 = shrink[mt * 16 + (lane >> 2) + 8];
@@ -477,29 +510,39 @@ __global__ void __launch_bounds__(kLatentThreads, 1) latent_mma_kernel(const __g
                 for (int plane = 0; plane < 2; ++plane)
                     ldsm_x4(w[mt][plane], smem_u32(weights + (plane * M + mt * 16 + (lane & 15)) * kWeightPitch + k * 16 + (lane >> 4) * 8));
 #pragma unroll
-            for (int v = 0; v < VT; v += 2) {
-                // tiles past the latent's columns are never stored; their reads stay inside the row
-                const int column = min((warp * VT + v) * 8, value_columns - 16);
-                uint32_t b[4];
-                ldsm_x4_trans(b, page + static_cast<uint32_t>(((k * 16 + (lane & 15)) * row_elements + column + (lane >> 4) * 8) * 2));
+            for (int v = 0; v < VT; v += kSpan) {
+                uint32_t b[kSpan / 2][4];
 #pragma unroll
-                for (int mt = 0; mt < MT; ++mt) {
-                    mma_16816(o[mt][v], w[mt][0], b[0], b[1]);
-                    mma_16816(o[mt][v + 1], w[mt][0], b[2], b[3]);
-                    mma_16816(o[mt][v], w[mt][1], b[0], b[1]);
-                    mma_16816(o[mt][v + 1], w[mt][1], b[2], b[3]);
+                for (int i = 0; i < kSpan / 2; ++i) {
+                    // tiles past the latent's columns are never stored; their reads stay inside the row
+                    const int chunk_of = min(warp * VT + v + 2 * i, value_chunks - 2);
+                    ldsm_x4_trans(b[i], page + page_offset(k * 16 + (lane & 15), chunk_of + (lane >> 4)));
                 }
+                // all tiles of one plane before the other: products that follow each other do not depend on each other
+#pragma unroll
+                for (int plane = 0; plane < 2; ++plane)
+#pragma unroll
+                    for (int i = 0; i < kSpan / 2; ++i)
+#pragma unroll
+                        for (int mt = 0; mt < MT; ++mt) {
+                            mma_16816(o[mt][v + 2 * i], w[mt][plane], b[i][0], b[i][1]);
+                            mma_16816(o[mt][v + 2 * i + 1], w[mt][plane], b[i][2], b[i][3]);
+                        }
             }
         }
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&empty[s]);
+        if constexpr (Shape::kProducer) {
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&empty[s]);
+        }
     }
     if (!alive) return;
+#pragma unroll
+    for (int r = 0; r < kOwn; ++r) l_own[r] = warp_sum(l_own[r]);
     if (lane == 0) {
 #pragma unroll
         for (int r = 0; r < kOwn; ++r) { row_m[warp * kOwn + r] = m_own[r]; row_l[warp * kOwn + r] = l_own[r]; }
     }
-    consumers_sync();
+    consumers_sync<Shape::kConsumers>();
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -593,7 +636,7 @@ __global__ void __launch_bounds__(kGenericThreads) latent_generic_kernel(const _
 }
 
 bool latent_takes_mma(const LatentParams& p) {
-    return p.kv.dtype == B200_BF16 && p.kv.page_size == kPage && p.width % 8 == 0 && p.rank % 8 == 0 && p.rank <= 512 && p.width <= 576;
+    return p.kv.dtype == B200_BF16 && p.kv.page_size == kPage && p.kv.head_dim % 8 == 0 && p.rank % 8 == 0 && p.rank <= 512 && p.width <= 576;
 }
 // Rows of an item: 16 for decode steps of up to 16 heads, 32 otherwise.
 int latent_tile(const LatentParams& p, int max_count) { return max_count == 1 && p.heads <= 16 ? 16 : 32; }
@@ -616,10 +659,10 @@ int latent_splits(const LatentParams& p, int sequences, int max_count, int max_l
     return best;
 }
 
-template <int KS, int VT, int MT> int launch_latent_mma(LatentAttention& a, int sequences, int max_count, cudaStream_t stream) {
+template <int KS, int VT, int MT> int launch_latent_mma(LatentAttention& a, const CUtensorMap& map, int sequences, int max_count, cudaStream_t stream) {
     constexpr int M = 16 * MT;
     const LatentParams& p = a.latent;
-    const int stage = kPage * latent_row_bytes(p.width), fixed = latent_fixed_bytes(M);
+    const int stage = (p.width + 63) / 64 * kBoxBytes, fixed = latent_fixed_bytes(M) + 1024;
     a.stages = std::min(6, (227 * 1024 - fixed) / stage);
     if (a.stages < 2) { set_error("latent attention: two pages of width %d do not fit shared memory", p.width); return B200_UNSUPPORTED; }
     const int smem = fixed + a.stages * stage;
@@ -630,13 +673,14 @@ template <int KS, int VT, int MT> int launch_latent_mma(LatentAttention& a, int 
     B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     const dim3 grid(static_cast<unsigned>((max_count + a.positions_per_item - 1) / a.positions_per_item), static_cast<unsigned>(sequences),
                     static_cast<unsigned>(a.head_chunks * a.splits));
-    return cuda_status(launch_dependent(kernel, grid, dim3(kLatentThreads), smem, stream, a), "latent_mma_kernel launch");
+    return cuda_status(launch_dependent(kernel, grid, dim3(LatentShape<MT>::kThreads), smem, stream, a, map), "latent_mma_kernel launch");
 }
-template <int MT> int pick_latent_mma(LatentAttention& a, int sequences, int max_count, cudaStream_t stream) {
+template <int MT> int pick_latent_mma(LatentAttention& a, const CUtensorMap& map, int sequences, int max_count, cudaStream_t stream) {
     const LatentParams& p = a.latent;
-    if (p.rank <= 128 && p.width <= 192) return launch_latent_mma<3, 2, MT>(a, sequences, max_count, stream);
-    if (p.rank <= 256 && p.width <= 320) return launch_latent_mma<5, 4, MT>(a, sequences, max_count, stream);
-    return launch_latent_mma<9, 8, MT>(a, sequences, max_count, stream);
+    constexpr int kPer = 8 * LatentShape<MT>::kWarps;   // latent columns of one tile per warp
+    if (p.rank <= 128 && p.width <= 192) return launch_latent_mma<3, 2, MT>(a, map, sequences, max_count, stream);
+    if (p.rank <= 256 && p.width <= 320) return launch_latent_mma<5, 256 / kPer, MT>(a, map, sequences, max_count, stream);
+    return launch_latent_mma<9, 512 / kPer, MT>(a, map, sequences, max_count, stream);
 }
 
 }  // namespace
@@ -721,8 +765,10 @@ int b200_latent_attention(const b200_latent_args* args, const b200_rows* pass, c
         a.partial_ml = a.partial + pairs * p.rank;
     }
     const int sequences = a.rows.sequences, max_count = a.rows.max_count;
-    const int status = latent_tile(p, max_count) == 16 ? pick_latent_mma<1>(a, sequences, max_count, as_stream(stream))
-                                                       : pick_latent_mma<2>(a, sequences, max_count, as_stream(stream));
+    const CUtensorMap* map = kv_tensor_map(args->cache, 0);
+    if (!map) { set_error("latent attention: the cache has no tensor map"); return B200_UNSUPPORTED; }
+    const int status = latent_tile(p, max_count) == 16 ? pick_latent_mma<1>(a, *map, sequences, max_count, as_stream(stream))
+                                                       : pick_latent_mma<2>(a, *map, sequences, max_count, as_stream(stream));
     if (status != B200_OK || a.splits == 1) return status;
     return cuda_status(launch_dependent(latent_combine_kernel, dim3(static_cast<unsigned>(a.rows.rows * p.heads)), dim3(128), 0, as_stream(stream),
                                         static_cast<const float*>(a.partial), static_cast<const float*>(a.partial_ml), a.splits, p.rank, a.out),

@@ -11,6 +11,7 @@
 //     time through the packed f32 pipe.
 // The ring has `taps` entries although a token needs only taps - 1 old inputs: the entry a step writes is never one that the
 // same step reads, so the CTAs of a head group need no ordering among themselves.
+#include "mma.cuh"
 #include "rows.cuh"
 
 #include <cmath>
@@ -66,7 +67,7 @@ template <int V> __device__ __forceinline__ void store_lanes(float* p, const Lan
 
 // grid (heads, sequences); one row per sequence.  V = 4 when vdim is a multiple of 4.
 template <int V>
-__global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams p, const RowsView rows) {
+__global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmParams p, const RowsView rows) {
     extern __shared__ __align__(16) float sm[];   // [vdim + 2 state] convolved channels, then [threads * V] partial outputs
     const int P = p.vdim, N = p.state, head = blockIdx.x, row = blockIdx.y;
     const int group = head / (p.heads / p.groups), inner = p.heads * P;
@@ -74,7 +75,8 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams 
     float* partial = sm + ((P + 2 * N + 3) & ~3);
     grid_dependency_wait();
     grid_launch_dependents();
-    const RowPlace place = row_place(rows, row);
+    const int slot = __ldg(rows.slot + row);   // one row per sequence: row and sequence are the same number
+    const RowPlace place{row, slot, rows.lengths[slot]};
     const float* in = p.projected + static_cast<int64_t>(row) * p.stride;
     const bool fresh = place.position == 0;
     float* state = p.ssm_state + (static_cast<int64_t>(place.slot) * p.heads + head) * N * P;
@@ -83,6 +85,19 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams 
     // the convolution so that its latency is covered
     const int columns = P / V, slices = kStepThreads / columns > 0 ? kStepThreads / columns : 1;
     constexpr int kAhead = 8;
+    const int my_slice = columns <= kStepThreads ? static_cast<int>(threadIdx.x) / columns : 0;
+    const int my_column = columns <= kStepThreads ? static_cast<int>(threadIdx.x) % columns : static_cast<int>(threadIdx.x);
+    auto fetch = [&](Lanes<V>(&s)[kAhead], int n0, int column, bool active) {
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i) {
+            const int n = n0 + i * slices;
+#pragma unroll
+            for (int k = 0; k < V; ++k) s[i].v[k] = 0.0f;
+            if (active && !fresh && n < N) s[i] = load_lanes<V>(state + static_cast<int64_t>(n) * P + column * V);
+        }
+    };
+    Lanes<V> s[kAhead];
+    fetch(s, my_slice, my_column, my_column < columns && my_slice < slices);
 
     const bool shared_writer = head % (p.heads / p.groups) == 0;
     for (int i = threadIdx.x; i < P + 2 * N; i += kStepThreads) {
@@ -102,8 +117,7 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams 
     const float *x = mixed, *B = mixed + P, *C = mixed + P + N;
 
     for (int base = 0; base < columns; base += kStepThreads) {
-        const int column = base + (columns <= kStepThreads ? static_cast<int>(threadIdx.x) % columns : static_cast<int>(threadIdx.x));
-        const int slice = columns <= kStepThreads ? static_cast<int>(threadIdx.x) / columns : 0;
+        const int column = base + my_column, slice = my_slice;
         const bool active = column < columns && slice < slices;
         Lanes<V> sum;
 #pragma unroll
@@ -113,14 +127,7 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams 
 #pragma unroll
             for (int k = 0; k < V; ++k) xd.v[k] = x[column * V + k] * dt;
             for (int n0 = slice; n0 < N; n0 += slices * kAhead) {
-                Lanes<V> s[kAhead];
-#pragma unroll
-                for (int i = 0; i < kAhead; ++i) {
-                    const int n = n0 + i * slices;
-#pragma unroll
-                    for (int k = 0; k < V; ++k) s[i].v[k] = 0.0f;
-                    if (!fresh && n < N) s[i] = load_lanes<V>(state + static_cast<int64_t>(n) * P + column * V);
-                }
+                if (base > 0 || n0 != slice) fetch(s, n0, column, true);
 #pragma unroll
                 for (int i = 0; i < kAhead; ++i) {
                     const int n = n0 + i * slices;
@@ -148,23 +155,73 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(const SsmParams 
     }
 }
 
-// mixed[row, c] = silu(conv(x | B | C)), grid (channel blocks, rows)
-__global__ void __launch_bounds__(256) short_conv_kernel(const SsmParams p, const RowsView rows) {
+// mixed[row, c] = silu(conv(x | B | C)), grid (channel blocks, strips of kConvRows rows).  V channels per thread (4 when rows and
+// channel counts allow 16-byte accesses).  TAPS > 0: the inputs of a strip slide through registers, each read once; TAPS = 0: any
+// number of taps, read from L1 again.
+constexpr int kConvRows = 16;
+template <int V, int TAPS> __global__ void __launch_bounds__(128) short_conv_kernel(const SsmParams p, const RowsView rows) {
     grid_dependency_wait();
     grid_launch_dependents();
-    const int c = blockIdx.x * blockDim.x + threadIdx.x, row = blockIdx.y;
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V, inner = p.heads * p.vdim;
     if (c >= p.channels) return;
-    const RowPlace place = row_place(rows, row);
-    const int offset = row - __ldg(rows.first + place.sequence), inner = p.heads * p.vdim;
-    const float* in = p.projected + static_cast<int64_t>(row) * p.stride + inner + c;
-    const float* weight = p.conv_weight + static_cast<int64_t>(c) * p.taps;
-    float acc = p.conv_bias[c];
-    for (int j = 0; j < p.taps; ++j) {
-        const int back = p.taps - 1 - j;   // how many tokens before this one
-        const float v = back <= offset ? in[-static_cast<int64_t>(back) * p.stride] : ring_input(p, place.slot, place.position - back, c);
-        acc = fmaf(weight[j], v, acc);
+    const int row0 = blockIdx.y * kConvRows, row1 = min(rows.rows, row0 + kConvRows);
+    // input of the token `back` places before `row`
+    auto input = [&](int row, int offset, const RowPlace& place, int back) {
+        if (back <= offset) return load_lanes<V>(p.projected + static_cast<int64_t>(row - back) * p.stride + inner + c);
+        Lanes<V> old;
+#pragma unroll
+        for (int k = 0; k < V; ++k) old.v[k] = ring_input(p, place.slot, place.position - back, c + k);
+        return old;
+    };
+    const Lanes<V> bias = load_lanes<V>(p.conv_bias + c);
+    Lanes<V> weight[TAPS > 0 ? TAPS : 1], window[TAPS > 0 ? TAPS : 1];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int k = 0; k < V; ++k) weight[j].v[k] = p.conv_weight[static_cast<int64_t>(c + k) * TAPS + j];
     }
-    p.mixed[static_cast<int64_t>(row) * p.channels + c] = acc * sigmoid_exact(acc);
+    int sequence = -1;
+    for (int row = row0; row < row1; ++row) {
+        const RowPlace place = row_place(rows, row);
+        const int offset = row - __ldg(rows.first + place.sequence);
+        Lanes<V> acc = bias;
+        if constexpr (TAPS > 0) {
+            if (place.sequence != sequence) {   // the strip enters a sequence: its earlier inputs
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) window[j] = input(row, offset, place, TAPS - 1 - j);
+                sequence = place.sequence;
+            }
+            window[TAPS - 1] = input(row, offset, place, 0);
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+                for (int k = 0; k < V; ++k) acc.v[k] = fmaf(weight[j].v[k], window[j].v[k], acc.v[k]);
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j) window[j] = window[j + 1];
+        } else {
+            for (int j = 0; j < p.taps; ++j) {
+                const Lanes<V> v = input(row, offset, place, p.taps - 1 - j);
+#pragma unroll
+                for (int k = 0; k < V; ++k) acc.v[k] = fmaf(p.conv_weight[static_cast<int64_t>(c + k) * p.taps + j], v.v[k], acc.v[k]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc.v[k] *= sigmoid_exact(acc.v[k]);
+        store_lanes<V>(p.mixed + static_cast<int64_t>(row) * p.channels + c, acc);
+    }
+}
+template <int V, int TAPS> int launch_conv(const SsmParams& p, const RowsView& rows, cudaStream_t stream) {
+    const dim3 grid(static_cast<unsigned>((p.channels / V + 127) / 128), static_cast<unsigned>((rows.rows + kConvRows - 1) / kConvRows));
+    return cuda_status(launch_dependent(short_conv_kernel<V, TAPS>, grid, dim3(128), 0, stream, p, rows), "short_conv_kernel launch");
+}
+template <int V> int pick_conv(const SsmParams& p, const RowsView& rows, cudaStream_t stream) {
+    switch (p.taps) {
+    case 2: return launch_conv<V, 2>(p, rows, stream);
+    case 3: return launch_conv<V, 3>(p, rows, stream);
+    case 4: return launch_conv<V, 4>(p, rows, stream);
+    }
+    return launch_conv<V, 0>(p, rows, stream);
 }
 
 // The last inputs of every sequence into its slot's ring, grid (channel blocks, sequences)
@@ -211,7 +268,7 @@ constexpr int kScanWarps = 4;
 // LN lanes of a warp share the state dimension (4 * Q values each, in quads LN * 4 apart), the other 32 / LN lane groups hold
 // four value columns each.  grid (column tiles, heads, sequences).
 template <int LN, int Q>
-__global__ void __launch_bounds__(kScanWarps * 32) ssm_scan_kernel(const SsmParams p, const RowsView rows) {
+__global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_scan_kernel(const SsmParams p, const RowsView rows) {
     constexpr int kNp = LN * 4 * Q;                      // padded state size
     constexpr int kScanTokens = kNp <= 128 ? 16 : 4;     // tokens staged at a time
     constexpr int kGroups = 32 / LN;
@@ -248,16 +305,24 @@ __global__ void __launch_bounds__(kScanWarps * 32) ssm_scan_kernel(const SsmPara
         }
     const float rate = -expf(p.a_log[head]), dt_bias = p.dt_bias[head], skip = p.d[head];
     const int live_columns = min(kColumns, P - column0);
+    const bool aligned = ((p.channels | P | N | inner) & 3) == 0 && (reinterpret_cast<uintptr_t>(p.mixed) & 15) == 0;
 
     auto stage = [&](int chunk) {
         const int buffer = chunk & 1, t0 = chunk * kScanTokens, tokens = min(kScanTokens, count - t0);
-        const int width = live_columns + 2 * N;
-        for (int i = threadIdx.x; i < tokens * width; i += blockDim.x) {
-            const int t = i / width, c = i - t * width;
-            const float* row = p.mixed + static_cast<int64_t>(first + t0 + t) * p.channels;
-            if (c < live_columns) copy_async_4(&sx[buffer][t][c], row + head * P + column0 + c);
-            else if (c < live_columns + N) copy_async_4(&sB[buffer][t][c - live_columns], row + inner + group * N + (c - live_columns));
-            else copy_async_4(&sC[buffer][t][c - live_columns - N], row + inner + (p.groups + group) * N + (c - live_columns - N));
+        // a warp per token; 16 bytes per copy where every row and slice starts on such a boundary
+        const float* from[3] = {p.mixed + head * P + column0, p.mixed + inner + group * N, p.mixed + inner + (p.groups + group) * N};
+        const int width[3] = {live_columns, N, N};
+        for (int t = warp; t < tokens; t += kScanWarps) {
+            const int64_t row = static_cast<int64_t>(first + t0 + t) * p.channels;
+            float* to[3] = {sx[buffer][t], sB[buffer][t], sC[buffer][t]};
+#pragma unroll
+            for (int part = 0; part < 3; ++part) {
+                if (aligned) {
+                    for (int c = lane * 4; c < width[part]; c += 128) copy_async_16(smem_u32(to[part] + c), from[part] + row + c, true);
+                } else {
+                    for (int c = lane; c < width[part]; c += 32) copy_async_4(to[part] + c, from[part] + row + c);
+                }
+            }
         }
         if (threadIdx.x < tokens)
             copy_async_4(&sdt[buffer][threadIdx.x], p.projected + static_cast<int64_t>(first + t0 + threadIdx.x) * p.stride + inner + p.channels + head);
@@ -277,6 +342,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) ssm_scan_kernel(const SsmPara
             dt_mine = softplus(sdt[buffer][lane] + dt_bias);
             decay_mine = expf(rate * dt_mine);
         }
+#pragma unroll 2
         for (int t = 0; t < tokens; ++t) {
             const float dt = __shfl_sync(0xffffffffu, dt_mine, t), decay = __shfl_sync(0xffffffffu, decay_mine, t);
             const float4 xv = *reinterpret_cast<const float4*>(&sx[buffer][t][local]);
@@ -334,40 +400,64 @@ template <int LN, int Q> int launch_scan(const SsmParams& p, const RowsView& row
     return cuda_status(launch_dependent(ssm_scan_kernel<LN, Q>, grid, dim3(kScanWarps * 32), 0, stream, p, rows), "ssm_scan_kernel launch");
 }
 
-// grid (rows, parts)
-__global__ void __launch_bounds__(256) gated_group_norm_kernel(const float* y, const float* z, int64_t z_stride, const float* weight, int width,
+// grid (rows, parts).  V adjacent values per access (4 when everything allows 16-byte accesses).
+template <int V>
+__global__ void __launch_bounds__(128) gated_group_norm_kernel(const float* y, const float* z, int64_t z_stride, const float* weight, int width,
                                                                int parts, float eps, float* out, __nv_bfloat16* out_hi, __nv_bfloat16* out_lo) {
     __shared__ float scratch[32];
     grid_dependency_wait();
     grid_launch_dependents();
     const int64_t row = blockIdx.x;
     const int size = width / parts, c0 = blockIdx.y * size;
-    constexpr int kKeep = 8;   // values a thread keeps in registers; longer parts are computed again
-    float kept[kKeep];
+    constexpr int kKeep = 4;   // accesses whose values a thread keeps in registers; longer parts are computed again
+    Lanes<V> kept[kKeep];
     float squares = 0.0f;
     auto value = [&](int c) {
-        const float g = z[row * z_stride + c0 + c];
-        return y[row * width + c0 + c] * (g * sigmoid_exact(g));
+        const Lanes<V> g = load_lanes<V>(z + row * z_stride + c0 + c), a = load_lanes<V>(y + row * width + c0 + c);
+        Lanes<V> v;
+#pragma unroll
+        for (int k = 0; k < V; ++k) v.v[k] = a.v[k] * (g.v[k] * sigmoid_exact(g.v[k]));
+        return v;
+    };
+    auto finish = [&](int c, const Lanes<V>& v, float inverse) {
+        const Lanes<V> w = load_lanes<V>(weight + c0 + c);
+        Lanes<V> r;
+#pragma unroll
+        for (int k = 0; k < V; ++k) r.v[k] = v.v[k] * inverse * w.v[k];
+        const int64_t at = row * width + c0 + c;
+        if constexpr (V == 4) {
+            if (out) store_lanes<V>(out + at, r);
+            if (out_hi) {
+                uint2 hi, lo;
+                pack_planes(r.v[0], r.v[1], hi.x, lo.x);
+                pack_planes(r.v[2], r.v[3], hi.y, lo.y);
+                *reinterpret_cast<uint2*>(out_hi + at) = hi;
+                if (out_lo) *reinterpret_cast<uint2*>(out_lo + at) = lo;
+            }
+        } else {
+            store_forms(r.v[0], at, out, out_hi, out_lo);
+        }
     };
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
-        const int c = threadIdx.x + i * 256;
-        kept[i] = c < size ? value(c) : 0.0f;
-        squares = fmaf(kept[i], kept[i], squares);
+        const int c = (threadIdx.x + i * 128) * V;
+        if (c < size) kept[i] = value(c);
+#pragma unroll
+        for (int k = 0; k < V; ++k) squares = c < size ? fmaf(kept[i].v[k], kept[i].v[k], squares) : squares;
     }
-    for (int c = threadIdx.x + kKeep * 256; c < size; c += 256) {
-        const float v = value(c);
-        squares = fmaf(v, v, squares);
+    for (int c = (threadIdx.x + kKeep * 128) * V; c < size; c += 128 * V) {
+        const Lanes<V> v = value(c);
+#pragma unroll
+        for (int k = 0; k < V; ++k) squares = fmaf(v.v[k], v.v[k], squares);
     }
     squares = block_sum(squares, scratch);
     const float inverse = 1.0f / sqrtf(squares / static_cast<float>(size) + eps);
 #pragma unroll
     for (int i = 0; i < kKeep; ++i) {
-        const int c = threadIdx.x + i * 256;
-        if (c < size) store_forms(kept[i] * inverse * weight[c0 + c], row * width + c0 + c, out, out_hi, out_lo);
+        const int c = (threadIdx.x + i * 128) * V;
+        if (c < size) finish(c, kept[i], inverse);
     }
-    for (int c = threadIdx.x + kKeep * 256; c < size; c += 256)
-        store_forms(value(c) * inverse * weight[c0 + c], row * width + c0 + c, out, out_hi, out_lo);
+    for (int c = (threadIdx.x + kKeep * 128) * V; c < size; c += 128 * V) finish(c, value(c), inverse);
 }
 
 __global__ void rows_advance_kernel(const RowsView rows) {
@@ -481,8 +571,9 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
     if (a->state > B200_SSM_MAX_STATE) { set_error("b200_ssm_forward: state sizes above %d are not supported", B200_SSM_MAX_STATE); return B200_UNSUPPORTED; }
     if (rows.sequences > 65535) { set_error("b200_ssm_forward: too many sequences in one pass"); return B200_UNSUPPORTED; }
     const unsigned blocks = static_cast<unsigned>((p.channels + 255) / 256);
-    if (rows.rows > 65535) { set_error("b200_ssm_forward: at most 65535 rows in one pass"); return B200_UNSUPPORTED; }
-    int status = cuda_status(launch_dependent(short_conv_kernel, dim3(blocks, static_cast<unsigned>(rows.rows)), dim3(256), 0, s, p, rows), "short_conv_kernel launch");
+    const bool conv_quads = p.channels % 4 == 0 && p.stride % 4 == 0 && (p.heads * p.vdim) % 4 == 0
+        && ((reinterpret_cast<uintptr_t>(p.projected) | reinterpret_cast<uintptr_t>(p.mixed) | reinterpret_cast<uintptr_t>(p.conv_bias)) & 15) == 0;
+    int status = conv_quads ? pick_conv<4>(p, rows, s) : pick_conv<1>(p, rows, s);
     if (status != B200_OK) return status;
     status = cuda_status(launch_dependent(conv_ring_kernel, dim3(blocks, static_cast<unsigned>(rows.sequences)), dim3(256), 0, s, p, rows), "conv_ring_kernel launch");
     if (status != B200_OK) return status;
@@ -501,9 +592,13 @@ int b200_gated_group_norm(const float* y, const float* z, int64_t z_stride, cons
         return B200_BAD_ARGUMENT;
     }
     if (rows == 0) return B200_OK;
-    return cuda_status(launch_dependent(gated_group_norm_kernel, dim3(static_cast<unsigned>(rows), static_cast<unsigned>(parts)), dim3(256), 0,
-                                        as_stream(stream), y, z, z_stride, weight, static_cast<int>(width), static_cast<int>(parts),
-                                        static_cast<float>(eps), out, static_cast<__nv_bfloat16*>(out_hi), static_cast<__nv_bfloat16*>(out_lo)),
+    const bool quads = (width / parts) % 4 == 0 && z_stride % 4 == 0
+        && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(out)
+             | (reinterpret_cast<uintptr_t>(out_hi) << 1) | (reinterpret_cast<uintptr_t>(out_lo) << 1)) & 15) == 0;
+    return cuda_status(launch_dependent(quads ? gated_group_norm_kernel<4> : gated_group_norm_kernel<1>,
+                                        dim3(static_cast<unsigned>(rows), static_cast<unsigned>(parts)), dim3(128), 0, as_stream(stream), y, z, z_stride,
+                                        weight, static_cast<int>(width), static_cast<int>(parts), static_cast<float>(eps), out,
+                                        static_cast<__nv_bfloat16*>(out_hi), static_cast<__nv_bfloat16*>(out_lo)),
                        "gated_group_norm_kernel launch");
 }
 
