@@ -73,7 +73,23 @@ int make_maps(b200_kv_cache* c) {
     const cuuint64_t strides[1] = {static_cast<cuuint64_t>(c->head_dim) * 2};
     const cuuint32_t box[2] = {64, static_cast<cuuint32_t>(kFastPageSize)};
     const cuuint32_t element_strides[2] = {1, 1};
-    for (int which = 0; which < (latent ? 1 : 2); ++which) {
+    if (latent) {
+        // 3-D view [64-value blocks][token rows][64 values]: one copy brings all blocks of a group of tokens.  The last block of a
+        // width that is no multiple of 64 reaches into the next row (the pool has slack behind its last one); readers ignore it.
+        const cuuint64_t blocks = static_cast<cuuint64_t>((c->head_dim + 63) / 64);
+        const cuuint64_t latent_dims[3] = {64, dims[1], blocks};
+        const cuuint64_t latent_strides[2] = {strides[0], 128};
+        const cuuint32_t latent_box[3] = {64, static_cast<cuuint32_t>(kLatentBoxRows), static_cast<cuuint32_t>(blocks)};
+        const cuuint32_t ones[3] = {1, 1, 1};
+        if (blocks > 16) return B200_OK;   // wider than the tensor-core attention takes
+        const CUresult result = encode(&c->map[0], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, c->pool[0], latent_dims, latent_strides, latent_box, ones,
+                                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                                       CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+        if (result != CUDA_SUCCESS) { set_error("cuTensorMapEncodeTiled failed with %d", static_cast<int>(result)); return B200_BAD_ARGUMENT; }
+        c->has_maps = true;
+        return B200_OK;
+    }
+    for (int which = 0; which < 2; ++which) {
         const CUresult result = encode(&c->map[which], CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, c->pool[which], dims, strides,
                                        box, element_strides, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                                        CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
@@ -108,12 +124,13 @@ static int create_cache(int32_t device, int32_t dtype, int32_t sequences, int32_
     c->pages_per_seq = (capacity + page_size - 1) / page_size;
     c->num_pages = c->pages_per_seq * sequences;
     c->pool_bytes = static_cast<size_t>(c->num_pages) * kv_heads * page_size * head_dim * (dtype == B200_BF16 ? 2 : 4);
+    const size_t slack = pools == 1 ? 128 : 0;   // see make_maps
     auto fail = [&](int status) { b200_kv_cache_release(c); return status; };
     for (int which = 0; which < pools; ++which) {
-        cudaError_t e = cudaMalloc(&c->pool[which], c->pool_bytes);
+        cudaError_t e = cudaMalloc(&c->pool[which], c->pool_bytes + slack);
         if (e != cudaSuccess) return fail(cuda_status(e, "cudaMalloc(KV pool)"));
         // Pages start as zeros so that masked positions of a partly filled page are finite.
-        e = cudaMemset(c->pool[which], 0, c->pool_bytes);
+        e = cudaMemset(c->pool[which], 0, c->pool_bytes + slack);
         if (e != cudaSuccess) return fail(cuda_status(e, "cudaMemset(KV pool)"));
     }
     cudaError_t e = cudaMalloc(reinterpret_cast<void**>(&c->page_table), sizeof(int32_t) * c->num_pages);

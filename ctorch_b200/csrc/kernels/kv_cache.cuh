@@ -5,6 +5,7 @@
 
 namespace b200 {
 
+constexpr int kLatentBoxRows = 32; // tokens of one TMA box of a latent pool
 constexpr int kFastPageSize = 64;  // page size the TMA/tensor-core attention path is built for
 
 // What kernels see.  Pools are [page][kv_head][page_size][head_dim]; page_table is [sequences][pages_per_seq].

@@ -3,8 +3,8 @@
 // (b200_latent_query), attends to the latents themselves, and the weighted latent goes through the value up-projection
 // (b200_latent_value).  Every cached byte serves all heads as key and as value.
 //
-//   * latent_mma_kernel: bf16 caches.  Pages arrive through a TMA ring as boxes of 64 tokens x 64 values (128-byte swizzle, values
-//     past the width zero-filled, mbarrier completion); the consumer warps hold the queries as tensor-core fragments in registers, the query-key product split 4 ways over the
+//   * latent_mma_kernel: bf16 caches.  Half pages arrive through a TMA ring as boxes of 32 tokens x 64 values (128-byte swizzle,
+//     one copy for all of them, mbarrier completion); the consumer warps hold the queries as tensor-core fragments in registers, the query-key product split 4 ways over the
 //     width and 4 or 2 ways over the keys of a page; the partial scores meet in shared memory, a warp finishes whole rows of the
 //     online softmax in f32; then every warp multiplies the weights (as hi + lo planes) with its columns of the same page.
 //     Decode: 16 rows (heads of one token), 16 warps.  Longer passes and wide head counts: 32 rows, 8 warps.
@@ -134,10 +134,10 @@ __device__ __forceinline__ void head_pair(const HeadLinear& h, int row, int head
     head_result(h, row, head, o, a);
     if (o + 1 < h.out) head_result(h, row, head, o + 1, b);
 }
-__device__ __forceinline__ void head_rotated(const HeadLinear& h, int row, int head, int i) {
+__device__ __forceinline__ void head_rotated(const HeadLinear& h, int row, int head, int i, int position) {
     const LatentParams& p = h.latent;
     const float* part = h.x + row * h.x_row + head * h.x_head + p.dim;
-    h.y[(static_cast<int64_t>(row) * p.heads + head) * p.width + p.rank + i] = rotated(p, part, i, row_place(h.rows, row).position);
+    h.y[(static_cast<int64_t>(row) * p.heads + head) * p.width + p.rank + i] = rotated(p, part, i, position);
 }
 
 // One warp per output; grid (output blocks, rows, heads).
@@ -154,7 +154,7 @@ template <class W> __global__ void __launch_bounds__(256) head_linear_generic_ke
         if (lane == 0) head_result(h, row, head, o, acc);
     }
     if (h.query && blockIdx.x == 0)
-        for (int i = threadIdx.x; i < h.latent.rot_dim; i += blockDim.x) head_rotated(h, row, head, i);
+        for (int i = threadIdx.x; i < h.latent.rot_dim; i += blockDim.x) head_rotated(h, row, head, i, row_place(h.rows, row).position);
 }
 
 // bf16 weights on the tensor cores; the f32 inputs are split into planes while they are staged.  16 * WM rows x 64 outputs per CTA,
@@ -248,10 +248,10 @@ template <int WM> __global__ void __launch_bounds__(kHeadThreads) head_linear_mm
             const int row = m + i * 8, o = c + n * 8;
             if (row < h.row_count && o < h.out) head_pair(h, row, head, o, acc[n][2 * i], acc[n][2 * i + 1]);
         }
-    if (h.query && blockIdx.x == 0)
-        for (int i = threadIdx.x; i < M * h.latent.rot_dim; i += kHeadThreads) {
-            const int r = i / h.latent.rot_dim;
-            if (row0 + r < h.row_count) head_rotated(h, row0 + r, head, i - r * h.latent.rot_dim);
+    if (h.query)   // the output tiles of a head share the rows' rotated parts
+        for (int r = blockIdx.x + warp * gridDim.x; r < M && row0 + r < h.row_count; r += gridDim.x * (kHeadThreads / 32)) {
+            const int position = row_place(h.rows, row0 + r).position;
+            for (int i = lane; i < h.latent.rot_dim; i += 32) head_rotated(h, row0 + r, head, i, position);
         }
 }
 
@@ -293,7 +293,9 @@ constexpr int kPage = 64;
 constexpr int kScorePitch = 68, kWeightPitch = 72;
 constexpr float kLog2e = 1.4426950408889634f;
 
-constexpr int kBoxBytes = kPage * 64 * 2;   // one box of a page: 64 tokens x 64 values
+constexpr int kHalf = kLatentBoxRows;         // tokens of one ring stage: half a page
+constexpr int kBoxBytes = kHalf * 64 * 2;    // one box: 32 tokens x 64 values
+static_assert(2 * kHalf == kPage);
 int latent_fixed_bytes(int m) { return 4 * m * kScorePitch * 4 + 2 * m * kWeightPitch * 2 + 4 * m * 4 + 256; }
 
 // KS: 16-wide steps of the width per quarter; VT: 8-column tiles of the latent per warp; MT: 16-row tiles.
@@ -308,16 +310,16 @@ template <int MT> struct LatentShape {
 template <int THREADS> __device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
 // Called by a whole warp.
-__device__ __forceinline__ void latent_copy_page(const CUtensorMap* map, const int32_t* table, int page, uint8_t* stage, int boxes, uint64_t* full) {
-    const int row = __ldg(table + page) * kPage;
+__device__ __forceinline__ void latent_copy_half(const CUtensorMap* map, const int32_t* table, int half, uint8_t* stage, int boxes, uint64_t* full) {
+    const int row = __ldg(table + (half >> 1)) * kPage + (half & 1) * kHalf;
     if (elect_one()) {
         mbar_expect_tx(full, static_cast<uint32_t>(boxes * kBoxBytes));
-        for (int b = 0; b < boxes; ++b) tma_load_2d(stage + b * kBoxBytes, map, b * 64, row, full);
+        tma_load_3d(stage, map, 0, row, 0, full);
     }
     __syncwarp();
 }
-// Byte offset of 16-byte chunk `chunk` (8 values) of a row inside a staged page: boxes side by side, the chunk swizzled by its row.
-__device__ __forceinline__ uint32_t page_offset(int row, int chunk) {
+// Byte offset of 16-byte chunk `chunk` (8 values) of a row inside a stage: boxes side by side, the chunk swizzled by its row.
+__device__ __forceinline__ uint32_t stage_offset(int row, int chunk) {
     return static_cast<uint32_t>((chunk >> 3) * kBoxBytes + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
 }
 
@@ -368,19 +370,22 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
 
     const int32_t* table = p.kv.page_table + static_cast<int64_t>(slot) * p.kv.pages_per_seq;
     if (Shape::kProducer && warp == kWarps) {
-        for (int t = page0; t < page1; ++t) {
-            const int i = t - page0, s = i % a.stages;
+        for (int i = 0; i < 2 * (page1 - page0); ++i) {
+            const int s = i % a.stages;
             if (i >= a.stages && !mbar_wait(&empty[s], ((i / a.stages) - 1) & 1)) {
                 if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
                 break;
             }
-            latent_copy_page(&map, table, t, ring + s * stage_bytes, boxes, &full[s]);
+            latent_copy_half(&map, table, 2 * page0 + i, ring + s * stage_bytes, boxes, &full[s]);
         }
         return;
     }
-    if (!Shape::kProducer && warp == 0)   // all stages but one; the last is kept for the page that follows the one in work
-        for (int t = page0; t < min(page1, page0 + a.stages - 1); ++t)
-            latent_copy_page(&map, table, t, ring + (t - page0) * stage_bytes, boxes, &full[t - page0]);
+    int issued = 0;   // halves asked for by warp 0 (without a producer warp)
+    auto issue_until = [&](int end) {
+        for (; issued < min(end, 2 * (page1 - page0)); ++issued)
+            latent_copy_half(&map, table, 2 * page0 + issued, ring + issued % a.stages * stage_bytes, boxes, &full[issued % a.stages]);
+    };
+    if (!Shape::kProducer && warp == 0) issue_until(a.stages);
 
     // queries as A fragments: quarter `quarter` of the width
     const int quarter = warp & 3, group = warp >> 2, steps = (p.width + 15) >> 4;
@@ -420,17 +425,18 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
 #pragma unroll
     for (int r = 0; r < kOwn; ++r) { m_own[r] = -INFINITY; l_own[r] = 0.0f; }
     const float scale2 = p.scale * kLog2e;
-    const int key_row = group * kKeyTiles * 8 + (lane >> 4) * 8 + (lane & 7), key_chunk = (lane >> 3) & 1, value_chunks = boxes * 8;
+    const int key_row = (group * kKeyTiles * 8) % kHalf + (lane >> 4) * 8 + (lane & 7), key_chunk = (lane >> 3) & 1, value_chunks = boxes * 8;
     constexpr int kSpan = VT >= 4 ? 4 : 2;   // value tiles worked at a time
     bool alive = true;
 
     for (int t = page0; t < page1; ++t) {
-        const int i = t - page0, s = i % a.stages;
-        if (!mbar_wait(&full[s], (i / a.stages) & 1)) {
+        const int i = 2 * (t - page0), s0 = i % a.stages, s1 = (i + 1) % a.stages;
+        if (!mbar_wait(&full[s0], (i / a.stages) & 1) || !mbar_wait(&full[s1], ((i + 1) / a.stages) & 1)) {
             if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
             *static_cast<volatile int*>(gave_up) = 1;
         }
-        const uint32_t page = smem_u32(ring + s * stage_bytes);
+        const uint32_t half_at[2] = {smem_u32(ring + s0 * stage_bytes), smem_u32(ring + s1 * stage_bytes)};
+        const uint32_t keys_at = group * kKeyTiles * 8 < kHalf ? half_at[0] : half_at[1];   // a warp's keys lie in one half
         float sc[MT][kKeyTiles][4];
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
@@ -445,7 +451,7 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
 #pragma unroll
                 for (int n = 0; n < kKeyTiles; n += 2) {
                     uint32_t b[4];
-                    ldsm_x4(b, page + page_offset(key_row + n * 8, step * 2 + key_chunk));
+                    ldsm_x4(b, keys_at + stage_offset(key_row + n * 8, step * 2 + key_chunk));
 #pragma unroll
                     for (int mt = 0; mt < MT; ++mt) {
                         mma_16816(sc[mt][n], q[k][mt], b[0], b[1]);
@@ -464,11 +470,7 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
             }
         consumers_sync<Shape::kConsumers>();
         if (*static_cast<volatile int*>(gave_up)) { alive = false; break; }   // a page never arrived: every consumer leaves here
-        if (!Shape::kProducer && warp == 0 && t + a.stages - 1 < page1) {
-            // every warp is past the products of page t - 1: its stage takes the next page
-            const int next = t + a.stages - 1, into = (next - page0) % a.stages;
-            latent_copy_page(&map, table, next, ring + into * stage_bytes, boxes, &full[into]);
-        }
+        if (!Shape::kProducer && warp == 0) issue_until(i + a.stages);   // every warp is past the products of the page before: its stages are free
 #pragma unroll
         for (int r = 0; r < kOwn; ++r) {
             const int m = warp * kOwn + r, sees = visible[m] - t * kPage;
@@ -503,6 +505,12 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
         }
 #pragma unroll
         for (int k = 0; k < kPage / 16; ++k) {
+            if constexpr (Shape::kProducer) {
+                if (k == 2) {   // the first half has been read to its end
+                    __syncwarp();
+                    if (lane == 0) mbar_arrive(&empty[s0]);
+                }
+            }
             uint32_t w[MT][2][4];
 #pragma unroll
             for (int mt = 0; mt < MT; ++mt)
@@ -516,7 +524,7 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
                 for (int i = 0; i < kSpan / 2; ++i) {
                     // tiles past the latent's columns are never stored; their reads stay inside the row
                     const int chunk_of = min(warp * VT + v + 2 * i, value_chunks - 2);
-                    ldsm_x4_trans(b[i], page + page_offset(k * 16 + (lane & 15), chunk_of + (lane >> 4)));
+                    ldsm_x4_trans(b[i], half_at[k >> 1] + stage_offset((k & 1) * 16 + (lane & 15), chunk_of + (lane >> 4)));
                 }
                 // all tiles of one plane before the other: products that follow each other do not depend on each other
 #pragma unroll
@@ -532,7 +540,7 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
         }
         if constexpr (Shape::kProducer) {
             __syncwarp();
-            if (lane == 0) mbar_arrive(&empty[s]);
+            if (lane == 0) mbar_arrive(&empty[s1]);
         }
     }
     if (!alive) return;
@@ -663,8 +671,8 @@ template <int KS, int VT, int MT> int launch_latent_mma(LatentAttention& a, cons
     constexpr int M = 16 * MT;
     const LatentParams& p = a.latent;
     const int stage = (p.width + 63) / 64 * kBoxBytes, fixed = latent_fixed_bytes(M) + 1024;
-    a.stages = std::min(6, (227 * 1024 - fixed) / stage);
-    if (a.stages < 2) { set_error("latent attention: two pages of width %d do not fit shared memory", p.width); return B200_UNSUPPORTED; }
+    a.stages = std::min(8, (227 * 1024 - fixed) / stage);
+    if (a.stages < 4) { set_error("latent attention: two pages of width %d do not fit shared memory", p.width); return B200_UNSUPPORTED; }
     const int smem = fixed + a.stages * stage;
     a.head_chunk = std::min(p.heads, M);
     a.head_chunks = (p.heads + M - 1) / M;
