@@ -309,6 +309,12 @@ template <int MT> struct LatentShape {
 };
 template <int THREADS> __device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
+// 2^v by the hardware unit (relative error about 2^-22; 2^-inf = 0): the weights of the softmax.
+__device__ __forceinline__ float exp2_fast(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
 // Called by a whole warp.
 __device__ __forceinline__ void latent_copy_half(const CUtensorMap* map, const int32_t* table, int half, uint8_t* stage, int boxes, uint64_t* full) {
     const int row = __ldg(table + (half >> 1)) * kPage + (half & 1) * kHalf;
@@ -370,13 +376,15 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
 
     const int32_t* table = p.kv.page_table + static_cast<int64_t>(slot) * p.kv.pages_per_seq;
     if (Shape::kProducer && warp == kWarps) {
+        int s = 0;
+        uint32_t parity = 1;   // of the wait for a free stage; the first round does not wait
         for (int i = 0; i < 2 * (page1 - page0); ++i) {
-            const int s = i % a.stages;
-            if (i >= a.stages && !mbar_wait(&empty[s], ((i / a.stages) - 1) & 1)) {
+            if (i >= a.stages && !mbar_wait(&empty[s], parity)) {
                 if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
                 break;
             }
             latent_copy_half(&map, table, 2 * page0 + i, ring + s * stage_bytes, boxes, &full[s]);
+            if (++s == a.stages) { s = 0; parity ^= 1; }
         }
         return;
     }
@@ -388,7 +396,8 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
     if (!Shape::kProducer && warp == 0) issue_until(a.stages);
 
     // queries as A fragments: quarter `quarter` of the width
-    const int quarter = warp & 3, group = warp >> 2, steps = (p.width + 15) >> 4;
+    // quarter: 16 of the 64 values of every box, so that a warp's fragments lie at constant distances
+    const int quarter = warp & 3, group = warp >> 2;
     uint32_t q[KS][MT][4];
     {
         const float* source[2 * MT];
@@ -400,7 +409,7 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
         }
 #pragma unroll
         for (int i = 0; i < KS; ++i) {
-            const int k = (quarter * KS + i) * 16 + (lane & 3) * 2;
+            const int k = i * 64 + quarter * 16 + (lane & 3) * 2;
 #pragma unroll
             for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -425,13 +434,27 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
 #pragma unroll
     for (int r = 0; r < kOwn; ++r) { m_own[r] = -INFINITY; l_own[r] = 0.0f; }
     const float scale2 = p.scale * kLog2e;
-    const int key_row = (group * kKeyTiles * 8) % kHalf + (lane >> 4) * 8 + (lane & 7), key_chunk = (lane >> 3) & 1, value_chunks = boxes * 8;
+    // Offsets inside a stage (rows of a fragment differ by multiples of 8, so the swizzle is the lane's own)
+    const uint32_t key_offset = stage_offset((group * kKeyTiles * 8) % kHalf + (lane >> 4) * 8 + (lane & 7), quarter * 2 + ((lane >> 3) & 1));
+    uint32_t value_offset[VT / 2];   // tiles past the latent's columns are never stored; their reads stay inside the row
+#pragma unroll
+    for (int v = 0; v < VT / 2; ++v) value_offset[v] = stage_offset(lane & 15, min(warp * VT + 2 * v, boxes * 8 - 2) + (lane >> 4));
+    const uint32_t weight_at = smem_u32(weights + (lane & 15) * kWeightPitch + (lane >> 4) * 8);
+    float* const score_at = scores + (quarter * M + (lane >> 2)) * kScorePitch + group * kKeyTiles * 8 + (lane & 3) * 2;
     constexpr int kSpan = VT >= 4 ? 4 : 2;   // value tiles worked at a time
     bool alive = true;
 
+    int stage = 0;
+    uint32_t phase = 0;
+    auto step_stage = [&] { if (++stage == a.stages) { stage = 0; phase ^= 1; } };
     for (int t = page0; t < page1; ++t) {
-        const int i = 2 * (t - page0), s0 = i % a.stages, s1 = (i + 1) % a.stages;
-        if (!mbar_wait(&full[s0], (i / a.stages) & 1) || !mbar_wait(&full[s1], ((i + 1) / a.stages) & 1)) {
+        const int s0 = stage;
+        const uint32_t phase0 = phase;
+        step_stage();
+        const int s1 = stage;
+        const uint32_t phase1 = phase;
+        step_stage();
+        if (!mbar_wait(&full[s0], phase0) || !mbar_wait(&full[s1], phase1)) {
             if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
             *static_cast<volatile int*>(gave_up) = 1;
         }
@@ -446,12 +469,11 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
                 for (int j = 0; j < 4; ++j) sc[mt][n][j] = 0.0f;
 #pragma unroll
         for (int k = 0; k < KS; ++k) {
-            const int step = quarter * KS + k;
-            if (step < steps) {
+            if (k < boxes) {
 #pragma unroll
                 for (int n = 0; n < kKeyTiles; n += 2) {
                     uint32_t b[4];
-                    ldsm_x4(b, keys_at + stage_offset(key_row + n * 8, step * 2 + key_chunk));
+                    ldsm_x4(b, keys_at + key_offset + static_cast<uint32_t>(k * kBoxBytes + n * 8 * 128));
 #pragma unroll
                     for (int mt = 0; mt < MT; ++mt) {
                         mma_16816(sc[mt][n], q[k][mt], b[0], b[1]);
@@ -464,37 +486,35 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
         for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
             for (int n = 0; n < kKeyTiles; ++n) {
-                float* at = scores + (quarter * M + mt * 16 + (lane >> 2)) * kScorePitch + (group * kKeyTiles + n) * 8 + (lane & 3) * 2;
+                float* at = score_at + mt * 16 * kScorePitch + n * 8;
                 *reinterpret_cast<float2*>(at) = make_float2(sc[mt][n][0], sc[mt][n][1]);
                 *reinterpret_cast<float2*>(at + 8 * kScorePitch) = make_float2(sc[mt][n][2], sc[mt][n][3]);
             }
         consumers_sync<Shape::kConsumers>();
         if (*static_cast<volatile int*>(gave_up)) { alive = false; break; }   // a page never arrived: every consumer leaves here
-        if (!Shape::kProducer && warp == 0) issue_until(i + a.stages);   // every warp is past the products of the page before: its stages are free
+        if (!Shape::kProducer && warp == 0) issue_until(2 * (t - page0) + a.stages);   // every warp is past the products of the page before: its stages are free
 #pragma unroll
         for (int r = 0; r < kOwn; ++r) {
             const int m = warp * kOwn + r, sees = visible[m] - t * kPage;
             float v0 = 0.0f, v1 = 0.0f;
 #pragma unroll
             for (int w = 0; w < 4; ++w) {
-                v0 += scores[(w * M + m) * kScorePitch + lane];
-                v1 += scores[(w * M + m) * kScorePitch + lane + 32];
+                const float2 part = *reinterpret_cast<const float2*>(scores + (w * M + m) * kScorePitch + lane * 2);
+                v0 += part.x;
+                v1 += part.y;
             }
-            v0 = lane < sees ? v0 * scale2 : -INFINITY;
-            v1 = lane + 32 < sees ? v1 * scale2 : -INFINITY;
+            v0 = lane * 2 < sees ? v0 * scale2 : -INFINITY;
+            v1 = lane * 2 + 1 < sees ? v1 * scale2 : -INFINITY;
             const float top = fmaxf(m_own[r], warp_max(fmaxf(v0, v1)));
             const float base = top == -INFINITY ? 0.0f : top;
-            const float p0 = exp2f(v0 - base), p1 = exp2f(v1 - base), factor = exp2f(m_own[r] - base);
+            const float p0 = exp2_fast(v0 - base), p1 = exp2_fast(v1 - base), factor = exp2_fast(m_own[r] - base);
             l_own[r] = l_own[r] * factor + (p0 + p1);
             m_own[r] = top;
             if (lane == 0) shrink[m] = factor;
-            __nv_bfloat16 hi, lo;
-            split_planes(p0, hi, lo);
-            weights[m * kWeightPitch + lane] = hi;
-            weights[(M + m) * kWeightPitch + lane] = lo;
-            split_planes(p1, hi, lo);
-            weights[m * kWeightPitch + lane + 32] = hi;
-            weights[(M + m) * kWeightPitch + lane + 32] = lo;
+            uint32_t hi, lo;
+            pack_planes(p0, p1, hi, lo);
+            *reinterpret_cast<uint32_t*>(weights + m * kWeightPitch + lane * 2) = hi;
+            *reinterpret_cast<uint32_t*>(weights + (M + m) * kWeightPitch + lane * 2) = lo;
         }
         consumers_sync<Shape::kConsumers>();
 #pragma unroll
@@ -516,16 +536,13 @@ __global__ void __launch_bounds__(LatentShape<MT>::kThreads, 1) latent_mma_kerne
             for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
                 for (int plane = 0; plane < 2; ++plane)
-                    ldsm_x4(w[mt][plane], smem_u32(weights + (plane * M + mt * 16 + (lane & 15)) * kWeightPitch + k * 16 + (lane >> 4) * 8));
+                    ldsm_x4(w[mt][plane], weight_at + static_cast<uint32_t>(((plane * M + mt * 16) * kWeightPitch + k * 16) * 2));
 #pragma unroll
             for (int v = 0; v < VT; v += kSpan) {
                 uint32_t b[kSpan / 2][4];
 #pragma unroll
-                for (int i = 0; i < kSpan / 2; ++i) {
-                    // tiles past the latent's columns are never stored; their reads stay inside the row
-                    const int chunk_of = min(warp * VT + v + 2 * i, value_chunks - 2);
-                    ldsm_x4_trans(b[i], half_at[k >> 1] + stage_offset((k & 1) * 16 + (lane & 15), chunk_of + (lane >> 4)));
-                }
+                for (int i = 0; i < kSpan / 2; ++i)
+                    ldsm_x4_trans(b[i], half_at[k >> 1] + value_offset[v / 2 + i] + (k & 1) * 16 * 128);
                 // all tiles of one plane before the other: products that follow each other do not depend on each other
 #pragma unroll
                 for (int plane = 0; plane < 2; ++plane)
