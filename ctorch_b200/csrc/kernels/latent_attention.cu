@@ -116,24 +116,6 @@ __device__ __forceinline__ void head_result(const HeadLinear& h, int row, int he
         store_forms(v * (1.0f / (1.0f + expf(-g))), row * static_cast<int64_t>(h.latent.heads) * h.out + column, h.y, h.out_hi, h.out_lo);
     }
 }
-// Two adjacent results (o even) of the tensor-core form.
-__device__ __forceinline__ void head_pair(const HeadLinear& h, int row, int head, int o, float a, float b) {
-    if (h.query && (h.latent.width & 1) == 0 && o + 1 < h.out) {
-        *reinterpret_cast<float2*>(h.y + (static_cast<int64_t>(row) * h.latent.heads + head) * h.latent.width + o) = make_float2(a, b);
-        return;
-    }
-    if (!h.query && !h.y && o + 1 < h.out && (h.out & 1) == 0 && h.out_lo) {
-        const int64_t column = static_cast<int64_t>(head) * h.out + o, at = row * static_cast<int64_t>(h.latent.heads) * h.out + column;
-        const float* gate = h.gate + row * h.gate_stride + column;
-        uint32_t hi, lo;
-        pack_planes(a * (1.0f / (1.0f + expf(-gate[0]))), b * (1.0f / (1.0f + expf(-gate[1]))), hi, lo);
-        *reinterpret_cast<uint32_t*>(h.out_hi + at) = hi;
-        *reinterpret_cast<uint32_t*>(h.out_lo + at) = lo;
-        return;
-    }
-    head_result(h, row, head, o, a);
-    if (o + 1 < h.out) head_result(h, row, head, o + 1, b);
-}
 __device__ __forceinline__ void head_rotated(const HeadLinear& h, int row, int head, int i, int position) {
     const LatentParams& p = h.latent;
     const float* part = h.x + row * h.x_row + head * h.x_head + p.dim;
@@ -157,124 +139,178 @@ template <class W> __global__ void __launch_bounds__(256) head_linear_generic_ke
         for (int i = threadIdx.x; i < h.latent.rot_dim; i += blockDim.x) head_rotated(h, row, head, i, row_place(h.rows, row).position);
 }
 
-// bf16 weights on the tensor cores; the f32 inputs are split into planes while they are staged.  16 * WM rows x 64 outputs per CTA,
-// 64 input columns at a time.  WM = 4: a warp per 16 rows; WM = 1: the four warps share the 16 rows and split the outputs.
-constexpr int kHeadThreads = 128, kHeadTile = 64, kHeadPitch = 72;
-template <int WM> constexpr int head_linear_smem() { return 2 * (2 * 16 * WM + kHeadTile) * kHeadPitch * 2; }
+// bf16 weights on the tensor cores; the f32 inputs are split into planes while they are staged.  WM x WN warps, each MI x 16 rows by
+// NI x 8 outputs; KC input columns at a time, double-buffered, the next chunk's rows fetched into registers under the products.
+template <int WM, int WN, int MI, int NI, int KC> struct HeadTile {
+    static constexpr int kThreads = WM * WN * 32, kM = WM * MI * 16, kN = WN * NI * 8, kPitch = KC + 8;
+    static constexpr int kSmem = 2 * (2 * kM + kN) * kPitch * 2;
+    static constexpr int kQuads = kM * KC / 4 / kThreads;
+};
 
-template <int WM> __global__ void __launch_bounds__(kHeadThreads) head_linear_mma_kernel(const __grid_constant__ HeadLinear h) {
-    constexpr int M = 16 * WM, kTiles = WM == 4 ? 8 : 2, kQuads = M * kHeadTile / 4 / kHeadThreads;
+template <int WM, int WN, int MI, int NI, int KC, bool QUERY>
+__global__ void __launch_bounds__(WM * WN * 32, WM * WN == 8 ? 2 : 1) head_linear_mma_kernel(const __grid_constant__ HeadLinear h) {
+    using Tile = HeadTile<WM, WN, MI, NI, KC>;
+    constexpr int kPitch = Tile::kPitch;
     extern __shared__ __align__(16) uint8_t smem[];
-    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem);            // [2 buffers][2 planes][M][pitch]
-    __nv_bfloat16* ws = xs + 4 * M * kHeadPitch;                           // [2 buffers][64][pitch]
+    __shared__ int positions[Tile::kM];
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smem);            // [2 buffers][2 planes][kM][pitch]
+    __nv_bfloat16* ws = xs + 4 * Tile::kM * kPitch;                        // [2 buffers][kN][pitch]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int o0 = blockIdx.x * kHeadTile, row0 = blockIdx.y * M, head = blockIdx.z;
+    const int o0 = blockIdx.x * Tile::kN, row0 = blockIdx.y * Tile::kM, head = blockIdx.z;
     const __nv_bfloat16* weight = static_cast<const __nv_bfloat16*>(h.w) + static_cast<int64_t>(head) * h.out * h.in;
     auto stage_weights = [&](int chunk) {
-        __nv_bfloat16* dst = ws + (chunk & 1) * kHeadTile * kHeadPitch;
-        for (int i = threadIdx.x; i < kHeadTile * 8; i += kHeadThreads) {
-            const int o = i >> 3, k = chunk * kHeadTile + (i & 7) * 8;
+        __nv_bfloat16* dst = ws + (chunk & 1) * Tile::kN * kPitch;
+        for (int i = threadIdx.x; i < Tile::kN * (KC / 8); i += Tile::kThreads) {
+            const int o = i / (KC / 8), c = (i % (KC / 8)) * 8, k = chunk * KC + c;
             const bool live = o0 + o < h.out && k < h.in;
-            copy_async_16(smem_u32(dst + o * kHeadPitch + (i & 7) * 8), live ? weight + static_cast<int64_t>(o0 + o) * h.in + k : weight, live);
+            copy_async_16(smem_u32(dst + o * kPitch + c), live ? weight + static_cast<int64_t>(o0 + o) * h.in + k : weight, live);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    float4 ahead[kQuads];
+    float4 ahead[Tile::kQuads];
     auto fetch_rows = [&](int chunk) {
 #pragma unroll
-        for (int j = 0; j < kQuads; ++j) {
-            const int i = threadIdx.x + j * kHeadThreads, r = i >> 4, k = chunk * kHeadTile + (i & 15) * 4;
+        for (int j = 0; j < Tile::kQuads; ++j) {
+            const int i = threadIdx.x + j * Tile::kThreads, r = i / (KC / 4), k = chunk * KC + (i % (KC / 4)) * 4;
             ahead[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (row0 + r < h.row_count && k < h.in)
                 ahead[j] = *reinterpret_cast<const float4*>(h.x + (row0 + r) * h.x_row + head * h.x_head + k);
         }
     };
     auto put_rows = [&](int chunk) {
-        __nv_bfloat16* hi = xs + (chunk & 1) * 2 * M * kHeadPitch;
-        __nv_bfloat16* lo = hi + M * kHeadPitch;
+        __nv_bfloat16* hi = xs + (chunk & 1) * 2 * Tile::kM * kPitch;
+        __nv_bfloat16* lo = hi + Tile::kM * kPitch;
 #pragma unroll
-        for (int j = 0; j < kQuads; ++j) {
-            const int i = threadIdx.x + j * kHeadThreads, r = i >> 4, c = (i & 15) * 4;
+        for (int j = 0; j < Tile::kQuads; ++j) {
+            const int i = threadIdx.x + j * Tile::kThreads, r = i / (KC / 4), c = (i % (KC / 4)) * 4;
             uint32_t h0, l0, h1, l1;
             pack_planes(ahead[j].x, ahead[j].y, h0, l0);
             pack_planes(ahead[j].z, ahead[j].w, h1, l1);
-            *reinterpret_cast<uint2*>(hi + r * kHeadPitch + c) = make_uint2(h0, h1);
-            *reinterpret_cast<uint2*>(lo + r * kHeadPitch + c) = make_uint2(l0, l1);
+            *reinterpret_cast<uint2*>(hi + r * kPitch + c) = make_uint2(h0, h1);
+            *reinterpret_cast<uint2*>(lo + r * kPitch + c) = make_uint2(l0, l1);
         }
     };
-    float acc[kTiles][4];
+    float acc[MI][NI][4];
 #pragma unroll
-    for (int n = 0; n < kTiles; ++n)
+    for (int m = 0; m < MI; ++m)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) acc[n][i] = 0.0f;
+        for (int n = 0; n < NI; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.0f;
 
-    const int chunks = (h.in + kHeadTile - 1) / kHeadTile;
+    const int chunks = (h.in + KC - 1) / KC;
+    const int m0 = (warp / WN) * MI * 16, n0 = (warp % WN) * NI * 8;
     stage_weights(0);          // weights are constants: requested before the producer of x is waited for
     grid_dependency_wait();
     grid_launch_dependents();
     fetch_rows(0);
+    if constexpr (QUERY) {
+        if (threadIdx.x < Tile::kM && row0 + static_cast<int>(threadIdx.x) < h.row_count)
+            positions[threadIdx.x] = row_place(h.rows, row0 + threadIdx.x).position;
+    }
     put_rows(0);
     for (int chunk = 0; chunk < chunks; ++chunk) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         if (chunk + 1 < chunks) { stage_weights(chunk + 1); fetch_rows(chunk + 1); }
-        const __nv_bfloat16* hi = xs + (chunk & 1) * 2 * M * kHeadPitch;
-        const int m0 = WM == 4 ? warp * 16 : 0, n0 = WM == 4 ? 0 : warp * 16;
-        const uint32_t a_hi = smem_u32(hi + (m0 + (lane & 15)) * kHeadPitch + (lane >> 4) * 8);
-        const uint32_t a_lo = a_hi + M * kHeadPitch * 2;
-        const uint32_t b = smem_u32(ws + (chunk & 1) * kHeadTile * kHeadPitch + (n0 + (lane >> 4) * 8 + (lane & 7)) * kHeadPitch + ((lane >> 3) & 1) * 8);
+        const __nv_bfloat16* hi = xs + (chunk & 1) * 2 * Tile::kM * kPitch;
+        const uint32_t a_hi = smem_u32(hi + (m0 + (lane & 15)) * kPitch + (lane >> 4) * 8);
+        const uint32_t a_lo = a_hi + Tile::kM * kPitch * 2;
+        const uint32_t b = smem_u32(ws + (chunk & 1) * Tile::kN * kPitch + (n0 + (lane >> 4) * 8 + (lane & 7)) * kPitch + ((lane >> 3) & 1) * 8);
 #pragma unroll
-        for (int k = 0; k < kHeadTile / 16; ++k) {
-            uint32_t ah[4], al[4];
-            ldsm_x4(ah, a_hi + k * 32);
-            ldsm_x4(al, a_lo + k * 32);
+        for (int k = 0; k < KC / 16; ++k) {
+            uint32_t a[2][MI][4], w[NI / 2][4];
 #pragma unroll
-            for (int n = 0; n < kTiles; n += 2) {
-                uint32_t w[4];
-                ldsm_x4(w, b + n * 8 * kHeadPitch * 2 + k * 32);
-                mma_16816(acc[n], ah, w[0], w[1]);
-                mma_16816(acc[n], al, w[0], w[1]);
-                mma_16816(acc[n + 1], ah, w[2], w[3]);
-                mma_16816(acc[n + 1], al, w[2], w[3]);
+            for (int m = 0; m < MI; ++m) {
+                ldsm_x4(a[0][m], a_hi + m * 16 * kPitch * 2 + k * 32);
+                ldsm_x4(a[1][m], a_lo + m * 16 * kPitch * 2 + k * 32);
             }
+#pragma unroll
+            for (int n = 0; n < NI / 2; ++n) ldsm_x4(w[n], b + n * 16 * kPitch * 2 + k * 32);
+#pragma unroll
+            for (int plane = 0; plane < 2; ++plane)
+#pragma unroll
+                for (int m = 0; m < MI; ++m)
+#pragma unroll
+                    for (int n = 0; n < NI; ++n) mma_16816(acc[m][n], a[plane][m], w[n >> 1][(n & 1) * 2], w[n >> 1][(n & 1) * 2 + 1]);
         }
         if (chunk + 1 < chunks) put_rows(chunk + 1);
     }
-    const int m = row0 + (WM == 4 ? warp * 16 : 0) + (lane >> 2), c = o0 + (WM == 4 ? 0 : warp * 16) + (lane & 3) * 2;
+    const LatentParams& p = h.latent;
 #pragma unroll
-    for (int n = 0; n < kTiles; ++n)
+    for (int m = 0; m < MI; ++m)
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-            const int row = m + i * 8, o = c + n * 8;
-            if (row < h.row_count && o < h.out) head_pair(h, row, head, o, acc[n][2 * i], acc[n][2 * i + 1]);
+            const int row = row0 + m0 + m * 16 + (lane >> 2) + i * 8, o = o0 + n0 + (lane & 3) * 2;
+            if (row >= h.row_count) continue;
+            if constexpr (QUERY) {
+                float* to = h.y + (static_cast<int64_t>(row) * p.heads + head) * p.width + o;
+#pragma unroll
+                for (int n = 0; n < NI; ++n)
+                    if (o + n * 8 < h.out) *reinterpret_cast<float2*>(to + n * 8) = make_float2(acc[m][n][2 * i], acc[m][n][2 * i + 1]);
+            } else {
+                const int64_t column = static_cast<int64_t>(head) * h.out + o, at = static_cast<int64_t>(row) * p.heads * h.out + column;
+                const float* gate = h.gate + row * h.gate_stride + column;
+                float2 g[NI];   // all gates of the row before the first store
+#pragma unroll
+                for (int n = 0; n < NI; ++n) {
+                    g[n] = make_float2(0.0f, 0.0f);
+                    if (o + n * 8 < h.out) g[n] = make_float2(__ldg(gate + n * 8), __ldg(gate + n * 8 + 1));
+                }
+#pragma unroll
+                for (int n = 0; n < NI; ++n) {
+                    if (o + n * 8 >= h.out) continue;
+                    const float v0 = acc[m][n][2 * i] * (1.0f / (1.0f + expf(-g[n].x))), v1 = acc[m][n][2 * i + 1] * (1.0f / (1.0f + expf(-g[n].y)));
+                    if (h.y) *reinterpret_cast<float2*>(h.y + at + n * 8) = make_float2(v0, v1);
+                    if (h.out_hi) {
+                        uint32_t hi, lo;
+                        pack_planes(v0, v1, hi, lo);
+                        *reinterpret_cast<uint32_t*>(h.out_hi + at + n * 8) = hi;
+                        if (h.out_lo) *reinterpret_cast<uint32_t*>(h.out_lo + at + n * 8) = lo;
+                    }
+                }
+            }
         }
-    if (h.query)   // the output tiles of a head share the rows' rotated parts
-        for (int r = blockIdx.x + warp * gridDim.x; r < M && row0 + r < h.row_count; r += gridDim.x * (kHeadThreads / 32)) {
-            const int position = row_place(h.rows, row0 + r).position;
-            for (int i = lane; i < h.latent.rot_dim; i += 32) head_rotated(h, row0 + r, head, i, position);
+    if constexpr (QUERY) {   // the output tiles of a head share the rows' rotated parts, a pair of values at a time
+        const int pairs = p.rot_dim >> 1, live = min(Tile::kM, h.row_count - row0);
+#pragma unroll 4
+        for (int e = threadIdx.x + blockIdx.x * Tile::kThreads; e < live * pairs; e += gridDim.x * Tile::kThreads) {
+            const int r = e / pairs, i = (e - r * pairs) * 2, position = positions[r];
+            const float2 v = *reinterpret_cast<const float2*>(h.x + (row0 + r) * h.x_row + head * h.x_head + p.dim + i);
+            float2 turned = v;
+            if (i < p.rot_dims && static_cast<unsigned>(position) < static_cast<unsigned>(p.positions)) {
+                const int64_t at = static_cast<int64_t>(position) * (p.rot_dims >> 1) + (i >> 1);
+                const float c = __ldg(p.cosine + at), s = __ldg(p.sine + at);
+                turned = make_float2(__fsub_rn(__fmul_rn(v.x, c), __fmul_rn(v.y, s)), __fadd_rn(__fmul_rn(v.y, c), __fmul_rn(v.x, s)));
+            }
+            *reinterpret_cast<float2*>(h.y + (static_cast<int64_t>(row0 + r) * p.heads + head) * p.width + p.rank + i) = turned;
         }
+    }
+}
+
+template <int WM, int WN, int MI, int NI, int KC> int launch_head_mma(const HeadLinear& h, cudaStream_t stream) {
+    using Tile = HeadTile<WM, WN, MI, NI, KC>;
+    auto kernel = h.query ? head_linear_mma_kernel<WM, WN, MI, NI, KC, true> : head_linear_mma_kernel<WM, WN, MI, NI, KC, false>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile::kSmem));
+    const dim3 grid(static_cast<unsigned>((h.out + Tile::kN - 1) / Tile::kN), static_cast<unsigned>((h.row_count + Tile::kM - 1) / Tile::kM),
+                    static_cast<unsigned>(h.latent.heads));
+    return cuda_status(launch_dependent(kernel, grid, dim3(Tile::kThreads), Tile::kSmem, stream, h), "head_linear_mma_kernel launch");
 }
 
 int launch_head_linear(const HeadLinear& h, cudaStream_t stream) {
     const LatentParams& p = h.latent;
     if (h.row_count > 65535 || p.heads > 65535) { set_error("latent attention: at most 65535 rows and heads in one pass"); return B200_UNSUPPORTED; }
-    const unsigned tiles = static_cast<unsigned>((h.out + kHeadTile - 1) / kHeadTile);
-    const bool mma = p.weight_dtype == B200_BF16 && h.in % 8 == 0 && h.x_row % 4 == 0 && h.x_head % 4 == 0
-        && ((reinterpret_cast<uintptr_t>(h.x) | reinterpret_cast<uintptr_t>(h.w)) & 15) == 0;
+    const bool mma = p.weight_dtype == B200_BF16 && h.in % 8 == 0 && h.x_row % 4 == 0 && h.x_head % 4 == 0 && h.out % 2 == 0 && p.width % 2 == 0
+        && p.rot_dim % 2 == 0
+        && ((reinterpret_cast<uintptr_t>(h.x) | reinterpret_cast<uintptr_t>(h.w)) & 15) == 0 && (reinterpret_cast<uintptr_t>(h.y) & 7) == 0;
     if (!mma) {
-        const dim3 grid(tiles, static_cast<unsigned>(h.row_count), static_cast<unsigned>(p.heads));
+        const dim3 grid(static_cast<unsigned>((h.out + 63) / 64), static_cast<unsigned>(h.row_count), static_cast<unsigned>(p.heads));
         return cuda_status(p.weight_dtype == B200_BF16 ? launch_dependent(head_linear_generic_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, h)
                                                        : launch_dependent(head_linear_generic_kernel<float>, grid, dim3(256), 0, stream, h),
                            "head_linear_generic_kernel launch");
     }
-    if (h.row_count <= 16) {
-        B200_CUDA(cudaFuncSetAttribute(head_linear_mma_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, head_linear_smem<1>()));
-        return cuda_status(launch_dependent(head_linear_mma_kernel<1>, dim3(tiles, 1, static_cast<unsigned>(p.heads)), dim3(kHeadThreads),
-                                            head_linear_smem<1>(), stream, h), "head_linear_mma_kernel launch");
-    }
-    B200_CUDA(cudaFuncSetAttribute(head_linear_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, head_linear_smem<4>()));
-    return cuda_status(launch_dependent(head_linear_mma_kernel<4>, dim3(tiles, static_cast<unsigned>((h.row_count + 63) / 64), static_cast<unsigned>(p.heads)),
-                                        dim3(kHeadThreads), head_linear_smem<4>(), stream, h), "head_linear_mma_kernel launch");
+    if (h.row_count <= 256) return launch_head_mma<1, 4, 1, 2, 128>(h, stream);   // 16 rows x 64 outputs: CTAs for every SM
+    return launch_head_mma<4, 2, 2, 8, 64>(h, stream);                            // 128 x 128: least traffic from L2
 }
 
 // ---- attention ----------------------------------------------------------------------------------------------------

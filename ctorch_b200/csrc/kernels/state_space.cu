@@ -330,6 +330,10 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
     };
 
     const int chunks = (count + kScanTokens - 1) / kScanTokens;
+    // after the exchanges below a lane holds column `mine` of its four, summed; lanes ln < 4 write
+    const bool odd = lane & 1, second = lane & 2;
+    const int mine = (odd ? 2 : 0) + (second ? 1 : 0);
+    const bool writes = ln < 4 && column + mine < P;
     stage(0);
     for (int chunk = 0; chunk < chunks; ++chunk) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -342,15 +346,15 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
             dt_mine = softplus(sdt[buffer][lane] + dt_bias);
             decay_mine = expf(rate * dt_mine);
         }
-#pragma unroll 2
-        for (int t = 0; t < tokens; ++t) {
+        float* const y_chunk = p.y + static_cast<int64_t>(first + t0) * inner + head * P + column + mine;
+        auto token = [&](int t) {
             const float dt = __shfl_sync(0xffffffffu, dt_mine, t), decay = __shfl_sync(0xffffffffu, decay_mine, t);
             const float4 xv = *reinterpret_cast<const float4*>(&sx[buffer][t][local]);
             const float x[4] = {xv.x, xv.y, xv.z, xv.w};
             const uint64_t decay2 = pack2(decay, decay);
             uint64_t xd[4], acc[4];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) { xd[k] = pack2(x[k] * dt, x[k] * dt); acc[k] = pack2(0.0f, 0.0f); }
+            for (int k = 0; k < 4; ++k) xd[k] = pack2(x[k] * dt, x[k] * dt);
 #pragma unroll
             for (int q = 0; q < Q; ++q) {
                 const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(&sB[buffer][t][q * LN * 4 + ln * 4]);
@@ -358,7 +362,7 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
                     S[k][2 * q] = fma2(S[k][2 * q], decay2, mul2(xd[k], b.x));
-                    acc[k] = fma2(S[k][2 * q], c.x, acc[k]);
+                    acc[k] = q == 0 ? mul2(S[k][0], c.x) : fma2(S[k][2 * q], c.x, acc[k]);
                     S[k][2 * q + 1] = fma2(S[k][2 * q + 1], decay2, mul2(xd[k], b.y));
                     acc[k] = fma2(S[k][2 * q + 1], c.y, acc[k]);
                 }
@@ -367,18 +371,19 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
 #pragma unroll
             for (int k = 0; k < 4; ++k) { const float2 v = unpack2(acc[k]); part[k] = v.x + v.y; }
             // sum over the LN lanes: two exchanges halve the four columns, the rest are plain butterflies
-            const bool odd = lane & 1, second = lane & 2;
             const float keep0 = odd ? part[2] : part[0], give0 = odd ? part[0] : part[2];
             const float keep1 = odd ? part[3] : part[1], give1 = odd ? part[1] : part[3];
             const float two0 = keep0 + __shfl_xor_sync(0xffffffffu, give0, 1), two1 = keep1 + __shfl_xor_sync(0xffffffffu, give1, 1);
             float one = (second ? two1 : two0) + __shfl_xor_sync(0xffffffffu, second ? two0 : two1, 2);
 #pragma unroll
             for (int o = 4; o < LN; o <<= 1) one += __shfl_xor_sync(0xffffffffu, one, o);
-            const int k = (odd ? 2 : 0) + (second ? 1 : 0);
-            if (ln < 4 && column + k < P) {
-                const float mine = k == 0 ? x[0] : k == 1 ? x[1] : k == 2 ? x[2] : x[3];
-                p.y[static_cast<int64_t>(first + t0 + t) * inner + head * P + column + k] = fmaf(skip, mine, one);
-            }
+            if (writes) y_chunk[static_cast<int64_t>(t) * inner] = fmaf(skip, sx[buffer][t][local + mine], one);
+        };
+        if (tokens == kScanTokens) {
+#pragma unroll 4
+            for (int t = 0; t < kScanTokens; ++t) token(t);
+        } else {
+            for (int t = 0; t < tokens; ++t) token(t);
         }
     }
 #pragma unroll
