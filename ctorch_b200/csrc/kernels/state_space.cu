@@ -1,10 +1,10 @@
 // State-space layers (Mamba-2): short causal convolution, selective recurrence, gated group norm; and the small kernels of
 // packed passes.  Everything here is f32: decays, step sizes, states and norms.
 //
-//   * Decode (one row per sequence): ssm_step_kernel, one CTA per (head, sequence).  It convolves the channels its head needs
-//     from the slot's ring of recent inputs, then streams the head's [state][vdim] matrix through registers once: load,
-//     decay, add dt B x^T, store, and the partial sums of S^T C on the way.  The layer is bound by that traffic
-//     (8 bytes per state value and token).
+//   * Decode (one row per sequence): per (sequence, head) the channels the head needs are convolved from the slot's ring of recent
+//     inputs, then its [state][vdim] matrix is read once - decay, add dt B x^T, partial sums of S^T C - and written back.  The layer
+//     is bound by that traffic (8 bytes per state value and token): ssm_step_stream_kernel has persistent CTAs through which the
+//     states stream by bulk copies; ssm_step_kernel, one CTA per pair, serves the sizes that do not fit it.
 //   * Longer passes: short_conv_kernel over all rows, conv_ring_kernel (the last inputs into the slot's ring), and
 //     ssm_scan_kernel: the state lives in registers across the whole pass, spread over a warp as state-dimension slices
 //     x 4 value columns per lane; tokens are staged through a double-buffered shared-memory chunk; products go two at a
@@ -14,6 +14,7 @@
 #include "mma.cuh"
 #include "rows.cuh"
 
+#include <algorithm>
 #include <cmath>
 
 namespace b200 {
@@ -65,12 +66,179 @@ template <int V> __device__ __forceinline__ void store_lanes(float* p, const Lan
     else p[0] = r.v[0];
 }
 
+// Convolved channels of one head for one token: [x: vdim | B: state | C: state] into `mixed`, and the token's inputs into the
+// slot's ring (B and C are shared by the heads of a group: its first head writes them).
+__device__ __forceinline__ void convolve_head(const SsmParams& p, const float* in, int slot, int position, int head, float* mixed) {
+    const int P = p.vdim, N = p.state, inner = p.heads * P, per_group = p.heads / p.groups, group = head / per_group;
+    const bool shared_writer = head == group * per_group;
+    // the ring entry of the current token; entry of the token `back` places before: ring_at - back, wrapped
+    const int ring_at = position % p.taps;
+    float* const ring = p.conv_state + static_cast<int64_t>(slot) * p.taps * p.channels;
+    for (int i = threadIdx.x; i < P + 2 * N; i += kStepThreads) {
+        const int c = i < P ? head * P + i : i < P + N ? inner + group * N + (i - P) : inner + (p.groups + group) * N + (i - P - N);
+        const float now = in[inner + c];
+        const float* weight = p.conv_weight + c * p.taps;
+        float acc = p.conv_bias[c];
+#pragma unroll 4
+        for (int j = 0; j < p.taps - 1; ++j) {
+            const int back = p.taps - 1 - j, at = ring_at < back ? ring_at - back + p.taps : ring_at - back;
+            const float old = position < back ? 0.0f : ring[at * p.channels + c];
+            acc = fmaf(weight[j], old, acc);
+        }
+        acc = fmaf(weight[p.taps - 1], now, acc);
+        mixed[i] = acc * sigmoid_exact(acc);
+        if (i < P || shared_writer) ring[ring_at * p.channels + c] = now;
+    }
+}
+
+// Streamed step, first half: mixed[row, c] = silu(conv(x | B | C)) of one row per sequence, and the row's inputs into the ring.
+// grid (channel blocks, rows), V channels per thread.
+template <int V> __global__ void __launch_bounds__(128) conv_step_kernel(const SsmParams p, const RowsView rows) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V, row = blockIdx.y, inner = p.heads * p.vdim;
+    if (c >= p.channels) return;
+    const int slot = __ldg(rows.slot + row), position = rows.lengths[slot], ring_at = position % p.taps;
+    float* const ring = p.conv_state + static_cast<int64_t>(slot) * p.taps * p.channels + c;
+    const Lanes<V> now = load_lanes<V>(p.projected + static_cast<int64_t>(row) * p.stride + inner + c);
+    Lanes<V> acc = load_lanes<V>(p.conv_bias + c);
+#pragma unroll 4
+    for (int j = 0; j < p.taps - 1; ++j) {
+        const int back = p.taps - 1 - j, at = ring_at < back ? ring_at - back + p.taps : ring_at - back;
+        const Lanes<V> old = load_lanes<V>(ring + at * p.channels);   // (an unused entry before the sequence's start)
+#pragma unroll
+        for (int k = 0; k < V; ++k)
+            acc.v[k] = fmaf(p.conv_weight[(c + k) * p.taps + j], position < back ? 0.0f : old.v[k], acc.v[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        acc.v[k] = fmaf(p.conv_weight[(c + k) * p.taps + p.taps - 1], now.v[k], acc.v[k]);
+        acc.v[k] *= sigmoid_exact(acc.v[k]);
+    }
+    store_lanes<V>(ring + ring_at * p.channels, now);
+    store_lanes<V>(p.mixed + static_cast<int64_t>(row) * p.channels + c, acc);
+}
+
+// Streamed step, second half: persistent CTAs walk the (sequence, head) pairs.  A producer warp brings a pair's state (one contiguous
+// [state][vdim] block) and its x, B and C by bulk copies into one of two stages while the pair before it is worked on; eight warps
+// update the state in place and leave the partial outputs; the producer sends the stage's state back and refills it.  vdim and state
+// multiples of 4, vdim at most 1024.
+__device__ __forceinline__ void bulk_store(void* dst, const void* src, uint32_t bytes) {
+    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst), "r"(smem_u32(src)), "r"(bytes) : "memory");
+    asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+}
+constexpr int kStreamThreads = kStepThreads + 32;
+struct StreamMeta { float dt, decay, fresh; };
+inline size_t ssm_stream_bytes(int state, int vdim) {
+    return sizeof(float) * (2 * (static_cast<size_t>(state) * vdim + vdim + 2 * state) + 2 * kStepThreads * 4);
+}
+
+__global__ void __launch_bounds__(kStreamThreads) ssm_step_stream_kernel(const SsmParams p, const RowsView rows, int32_t* status) {
+    extern __shared__ __align__(16) float sm[];   // 2 x [state * vdim | x: vdim | B: state | C: state], 2 x [threads * 4] partial outputs
+    __shared__ uint64_t full[2], done[2];
+    __shared__ StreamMeta meta[2];
+    __shared__ int gave_up;
+    const int P = p.vdim, N = p.state, inner = p.heads * P, block = N * P, stage_floats = block + P + 2 * N, columns = P >> 2,
+              slices = kStepThreads / columns;
+    const int units = rows.rows * p.heads;
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < 2; ++s) { mbar_init(&full[s], 1); mbar_init(&done[s], kStepThreads); }
+        mbar_fence_init();
+        gave_up = 0;
+    }
+    grid_dependency_wait();
+    grid_launch_dependents();
+    __syncthreads();
+
+    if (threadIdx.x >= kStepThreads) {   // producer warp; one lane issues, all lanes stay with it
+        if ((threadIdx.x & 31) != 0) return;
+        float* pending[2] = {nullptr, nullptr};
+        int turn = 0;
+        for (int unit = blockIdx.x; unit < units + 2 * static_cast<int>(gridDim.x); unit += gridDim.x, ++turn) {
+            const int stage = turn & 1, row = unit / p.heads, head = unit - row * p.heads;
+            const bool live = unit < units;
+            float dt = 0.0f;
+            float* state = nullptr;
+            bool fresh = true;
+            if (live) {   // operands of this pair, while the stage may still be in use
+                const int slot = __ldg(rows.slot + row);
+                fresh = rows.lengths[slot] == 0;
+                state = p.ssm_state + (static_cast<int64_t>(slot) * p.heads + head) * block;
+                dt = softplus(p.projected[static_cast<int64_t>(row) * p.stride + inner + p.channels + head] + p.dt_bias[head]);
+            }
+            if (turn >= 2 && pending[stage]) {   // the pair two turns ago has been worked on: its state goes back
+                if (!mbar_wait(&done[stage], ((turn >> 1) - 1) & 1)) {
+                    atomicExch(status, B200_DEVICE_TIMEOUT);
+                    break;
+                }
+                bulk_store(pending[stage], sm + stage * stage_floats, static_cast<uint32_t>(block) * 4);
+                asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
+            }
+            pending[stage] = state;
+            if (!live) continue;
+            float* at = sm + stage * stage_floats;
+            meta[stage] = StreamMeta{dt, expf(-expf(p.a_log[head]) * dt), fresh ? 1.0f : 0.0f};
+            mbar_expect_tx(&full[stage], static_cast<uint32_t>((fresh ? 0 : block) + P + 2 * N) * 4);
+            if (!fresh) bulk_load(at, state, static_cast<uint32_t>(block) * 4, &full[stage]);
+            const float* mixed = p.mixed + static_cast<int64_t>(row) * p.channels;
+            const int group = head / (p.heads / p.groups);
+            bulk_load(at + block, mixed + head * P, static_cast<uint32_t>(P) * 4, &full[stage]);
+            bulk_load(at + block + P, mixed + inner + group * N, static_cast<uint32_t>(N) * 4, &full[stage]);
+            bulk_load(at + block + P + N, mixed + inner + (p.groups + group) * N, static_cast<uint32_t>(N) * 4, &full[stage]);
+        }
+        asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+        return;
+    }
+
+    const int slice = static_cast<int>(threadIdx.x) / columns, column = static_cast<int>(threadIdx.x) - slice * columns;
+    const bool active = slice < slices;
+    int turn = 0;
+    for (int unit = blockIdx.x; unit < units; unit += gridDim.x, ++turn) {
+        const int stage = turn & 1, row = unit / p.heads, head = unit - row * p.heads;
+        const bool arrived = mbar_wait(&full[stage], (turn >> 1) & 1);
+        if (!arrived) {
+            if ((threadIdx.x & 31) == 0) atomicExch(status, B200_DEVICE_TIMEOUT);
+            *static_cast<volatile int*>(&gave_up) = 1;
+        }
+        const StreamMeta m = meta[stage];
+        float* at = sm + stage * stage_floats;
+        const float *x = at + block, *B = x + P, *C = B + N;
+        float* partial = sm + 2 * stage_floats + stage * kStepThreads * 4;
+        float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (active && arrived) {
+            float4 xd = *reinterpret_cast<const float4*>(x + column * 4);
+            xd = make_float4(xd.x * m.dt, xd.y * m.dt, xd.z * m.dt, xd.w * m.dt);
+            float4* s = reinterpret_cast<float4*>(at) + column;
+            const bool fresh = m.fresh != 0.0f;
+#pragma unroll 4
+            for (int n = slice; n < N; n += slices) {
+                const float b = B[n], c = C[n];
+                float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                if (!fresh) v = s[n * columns];
+                v = make_float4(fmaf(v.x, m.decay, xd.x * b), fmaf(v.y, m.decay, xd.y * b), fmaf(v.z, m.decay, xd.z * b), fmaf(v.w, m.decay, xd.w * b));
+                sum = make_float4(fmaf(v.x, c, sum.x), fmaf(v.y, c, sum.y), fmaf(v.z, c, sum.z), fmaf(v.w, c, sum.w));
+                s[n * columns] = v;
+            }
+        }
+        reinterpret_cast<float4*>(partial)[threadIdx.x] = sum;
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the updated state is read by the copy engine
+        asm volatile("bar.sync 1, %0;" ::"n"(kStepThreads) : "memory");
+        if (*static_cast<volatile int*>(&gave_up)) return;   // a state never arrived: the eight warps leave together
+        for (int i = threadIdx.x; i < P; i += kStepThreads) {
+            float total = 0.0f;
+            for (int k = 0; k < slices; ++k) total += partial[k * P + i];
+            p.y[static_cast<int64_t>(row) * inner + head * P + i] = fmaf(p.d[head], x[i], total);
+        }
+        mbar_arrive(&done[stage]);
+    }
+}
+
 // grid (heads, sequences); one row per sequence.  V = 4 when vdim is a multiple of 4.
 template <int V>
 __global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmParams p, const RowsView rows) {
     extern __shared__ __align__(16) float sm[];   // [vdim + 2 state] convolved channels, then [threads * V] partial outputs
     const int P = p.vdim, N = p.state, head = blockIdx.x, row = blockIdx.y;
-    const int group = head / (p.heads / p.groups), inner = p.heads * P;
+    const int inner = p.heads * P;
     float* mixed = sm;
     float* partial = sm + ((P + 2 * N + 3) & ~3);
     grid_dependency_wait();
@@ -86,7 +254,7 @@ __global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmPara
     const int columns = P / V, slices = kStepThreads / columns > 0 ? kStepThreads / columns : 1;
     constexpr int kAhead = 8;
     const int my_slice = columns <= kStepThreads ? static_cast<int>(threadIdx.x) / columns : 0;
-    const int my_column = columns <= kStepThreads ? static_cast<int>(threadIdx.x) % columns : static_cast<int>(threadIdx.x);
+    const int my_column = static_cast<int>(threadIdx.x) - my_slice * columns;
     auto fetch = [&](Lanes<V>(&s)[kAhead], int n0, int column, bool active) {
 #pragma unroll
         for (int i = 0; i < kAhead; ++i) {
@@ -99,18 +267,7 @@ __global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmPara
     Lanes<V> s[kAhead];
     fetch(s, my_slice, my_column, my_column < columns && my_slice < slices);
 
-    const bool shared_writer = head % (p.heads / p.groups) == 0;
-    for (int i = threadIdx.x; i < P + 2 * N; i += kStepThreads) {
-        const int c = i < P ? head * P + i : i < P + N ? inner + group * N + (i - P) : inner + (p.groups + group) * N + (i - P - N);
-        const float now = in[inner + c];
-        float acc = p.conv_bias[c];
-        for (int j = 0; j < p.taps - 1; ++j)
-            acc = fmaf(p.conv_weight[static_cast<int64_t>(c) * p.taps + j], ring_input(p, place.slot, place.position - (p.taps - 1 - j), c), acc);
-        acc = fmaf(p.conv_weight[static_cast<int64_t>(c) * p.taps + p.taps - 1], now, acc);
-        mixed[i] = acc * sigmoid_exact(acc);
-        if (i < P || shared_writer)
-            p.conv_state[(static_cast<int64_t>(place.slot) * p.taps + place.position % p.taps) * p.channels + c] = now;
-    }
+    convolve_head(p, in, place.slot, place.position, head, mixed);
     const float dt = softplus(in[inner + p.channels + head] + p.dt_bias[head]);
     const float decay = expf(-expf(p.a_log[head]) * dt);
     __syncthreads();
@@ -565,6 +722,27 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
     cudaStream_t s = as_stream(stream);
     if (rows.max_count == 1) {
         const bool quads = a->vdim % 4 == 0 && (reinterpret_cast<uintptr_t>(a->ssm_state) & 15) == 0;
+        const size_t streamed = ssm_stream_bytes(a->state, a->vdim);
+        const bool aligned = ((reinterpret_cast<uintptr_t>(p.projected) | reinterpret_cast<uintptr_t>(p.mixed) | reinterpret_cast<uintptr_t>(p.conv_bias)
+                               | reinterpret_cast<uintptr_t>(p.conv_state)) & 15) == 0;
+        int device = 0;
+        B200_CUDA(cudaGetDevice(&device));
+        const int64_t units = static_cast<int64_t>(rows.rows) * a->heads;
+        const int64_t per_sm = std::min<int64_t>(7, (228 * 1024) / (streamed + 1024 + 128)), resident = sm_count(device) * per_sm;
+        // streaming pays from a few pairs per CTA on; below that its extra launch and ramp cost more
+        if (quads && a->mixed && aligned && a->state % 4 == 0 && a->vdim <= 4 * kStepThreads && streamed <= 110 * 1024 && units >= 4 * resident) {
+            int32_t* status = device_status_word(device);
+            if (!status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
+            // (rows of `projected` start on 16-byte boundaries only when their stride is a multiple of 4)
+            const unsigned quads_per_row = static_cast<unsigned>(p.stride % 4 == 0 ? 4 : 1);
+            const dim3 grid((static_cast<unsigned>(p.channels) / quads_per_row + 127) / 128, static_cast<unsigned>(rows.rows));
+            const int conv = cuda_status(launch_dependent(quads_per_row == 4 ? conv_step_kernel<4> : conv_step_kernel<1>, grid, dim3(128), 0, s, p, rows),
+                                         "conv_step_kernel launch");
+            if (conv != B200_OK) return conv;
+            B200_CUDA(cudaFuncSetAttribute(ssm_step_stream_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(streamed)));
+            return cuda_status(launch_dependent(ssm_step_stream_kernel, dim3(static_cast<unsigned>(std::min(units, resident))), dim3(kStreamThreads), streamed, s, p, rows, status),
+                               "ssm_step_stream_kernel launch");
+        }
         const size_t smem = sizeof(float) * (((a->vdim + 2 * a->state + 3) & ~3) + kStepThreads * (quads ? 4 : 1));
         if (smem > 200 * 1024) { set_error("b200_ssm_forward: a head of %d x %d values does not fit shared memory", a->state, a->vdim); return B200_UNSUPPORTED; }
         auto kernel = quads ? ssm_step_kernel<4> : ssm_step_kernel<1>;

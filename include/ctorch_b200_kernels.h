@@ -359,7 +359,7 @@ typedef struct b200_ssm_args {
     float* conv_state;
     float* ssm_state;
     const float* projected;        /* [rows, 2*heads*vdim + 2*groups*state + heads] */
-    float* mixed;                  /* workspace [rows, heads*vdim + 2*groups*state], unused by passes of one row per sequence */
+    float* mixed;                  /* workspace [rows, heads*vdim + 2*groups*state]; may be NULL for passes of one row per sequence */
     float* y;                      /* [rows, heads*vdim] */
 } b200_ssm_args;
 /* Convolution, step sizes, recurrence and its output for every row; the slots' states move on.  Passes with one row per

@@ -159,6 +159,44 @@ def test_state_space_recurrence(spec):
     assert float(ssm_state[1].min()) == 5.0 == float(ssm_state[1].max())   # the slot nobody used
 
 
+def test_streamed_state_space_step():
+    """Many sequences: the persistent streaming form of a step, some sequences at their first token, slots in another order than rows."""
+    heads, P, N, G, taps, count = 16, 64, 36, 2, 4, 520
+    channels, inner = heads * P + 2 * G * N, heads * P
+    rng = np.random.default_rng(0)
+    conv_w, conv_b = rng.normal(0, 0.5, (channels, taps)), rng.normal(0, 0.3, channels)
+    dt_bias, a_log, d = rng.uniform(-2, 1, heads), rng.uniform(-1, 1.5, heads), rng.uniform(0.5, 1.5, heads)
+    params = [dev(v) for v in (conv_w, conv_b, dt_bias, a_log, d)]
+    slots = rng.permutation(count)
+    lengths = np.where(np.arange(count) % 3 == 0, 0, 5)   # every third slot starts afresh
+    conv_state, ssm_state = dev(rng.normal(size=(count, taps, channels))), dev(rng.normal(size=(count, heads, N, P)))
+    old_conv, old_state = conv_state.cpu().numpy().astype(np.float64), ssm_state.cpu().numpy().astype(np.float64)
+    x = rng.normal(size=(count, inner + channels + heads))
+    p = Pass([1] * count, slots.tolist(), lengths.tolist())
+    tx, mixed, y = dev(x), torch.empty(count, channels, device="cuda"), torch.empty(count, inner, device="cuda")
+    a = B.SsmArgs(heads, P, N, G, taps, *[t.data_ptr() for t in params], conv_state.data_ptr(), ssm_state.data_ptr(), tx.data_ptr(), mixed.data_ptr(),
+                  y.data_ptr())
+    torch.cuda.synchronize()
+    B.kcheck(B.lib().b200_ssm_forward(C.byref(a), C.byref(p.c), None))
+    torch.cuda.synchronize()
+    got, state = y.cpu().numpy(), ssm_state.cpu().numpy()
+    for r in range(0, count, 7):
+        slot = slots[r]
+        length = lengths[slot]
+        past = np.stack([old_conv[slot, (length - b) % taps] if length - b >= 0 else np.zeros(channels) for b in (3, 2, 1)])
+        if length == 0:
+            past[:] = 0.0
+        m = O.silu((np.concatenate([past, x[r:r + 1, inner:inner + channels]]) * conv_w.T).sum(0) + conv_b)
+        dt = O.softplus(x[r, inner + channels:] + dt_bias)
+        for h in range(heads):
+            g = h // (heads // G)
+            xs, Bm, Cm = m[h * P:(h + 1) * P], m[inner + g * N:inner + (g + 1) * N], m[inner + (G + g) * N:inner + (G + g + 1) * N]
+            S = np.exp(-np.exp(a_log[h]) * dt[h]) * (old_state[slot, h] if length else 0.0) + dt[h] * np.outer(Bm, xs)
+            assert ratio(state[slot, h], S) < 1e-5
+            assert np.abs(got[r, h * P:(h + 1) * P] - (S.T @ Cm + d[h] * xs)).max() < 1e-4
+        assert np.allclose(conv_state[slot, length % taps].cpu().numpy(), x[r, inner:inner + channels], atol=1e-5)
+
+
 @pytest.mark.parametrize("rows, width, parts", [(3, 64, 1), (2, 96, 4), (1, 30, 3), (5, 6000, 2), (4, 16, 16)])
 def test_gated_group_norm(rows, width, parts):
     rng = np.random.default_rng(width)
