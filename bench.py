@@ -729,6 +729,11 @@ def main():
         spec["batch"] = args.batch
     if args.impl == "reference" and int(os.environ.get("RANK", "0")) != 0:
         return   # the CPU arm runs on rank 0 alone
+    if args.impl == "reference":
+        import oracle
+        if not oracle.have_ref():
+            print(json.dumps({"impl": "reference", "unavailable": "the reference's CPU build (oracle/_ref) is not present on this machine"}))
+            return
     weights = W.make_weights(spec)
     line = run_reference(args, spec, weights) if args.impl == "reference" else run_b200(args, spec, weights)
     if line:

@@ -37,7 +37,7 @@ def build(ref: bool = True) -> None:
     """Compile the port and, when the reference tree is present, the reference harness."""
     subprocess.run(["make", "-s", "port"], cwd=HERE, check=True)
     reference = os.environ.get("CTORCH_REFERENCE", "/root/reference")
-    if ref and os.path.isdir(reference):
+    if ref and os.path.isdir(os.path.join(reference, "src", "core")):   # an empty mount counts as absent
         subprocess.run(["make", "-s", "-j8", "ref", "REF=" + reference], cwd=HERE, check=True)
 
 
