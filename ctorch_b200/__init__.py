@@ -54,7 +54,7 @@ class ShadowLinearArgs(C.Structure):
                 ("residual", C.c_void_p), ("qkv", C.POINTER(QkvArgs)), ("y", C.c_void_p), ("out_hi", C.c_void_p),
                 ("out_lo", C.c_void_p), ("out_norm_weight", C.c_void_p), ("out_norm_dtype", C.c_int32), ("sumsq_out", C.c_void_p),
                 ("best_value", C.c_void_p), ("best_index", C.c_void_p), ("y_copies", C.POINTER(C.c_void_p)), ("copies", C.c_int32),
-                ("out_norm", C.POINTER(ElementwiseNorm))]
+                ("out_norm", C.POINTER(ElementwiseNorm)), ("out_stride", C.c_int64)]
 
 
 class Rows(C.Structure):
@@ -74,6 +74,29 @@ class LatentArgs(C.Structure):
                 ("q_rank", C.c_int32), ("rot_dims", C.c_int32), ("scale", C.c_float), ("eps", C.c_double), ("cosine", C.c_void_p),
                 ("sine", C.c_void_p), ("positions", C.c_int32), ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("cache", C.c_void_p),
                 ("weight_dtype", C.c_int32), ("w_key", C.c_void_p), ("w_value", C.c_void_p)]
+
+
+class ChunkArgs(C.Structure):
+    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("rot_dims", C.c_int32), ("chunk", C.c_int32),
+                ("entries", C.c_int32), ("scale", C.c_float), ("eps", C.c_double), ("cosine", C.c_void_p), ("sine", C.c_void_p), ("positions", C.c_int32),
+                ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("dtype", C.c_int32), ("key_cache", C.c_void_p), ("value_cache", C.c_void_p),
+                ("projected", C.c_void_p), ("stride", C.c_int64), ("query", C.c_void_p), ("key", C.c_void_p), ("value", C.c_void_p)]
+
+
+class Units(C.Structure):
+    _fields_ = [("kind", C.c_int32), ("column", C.c_int64), ("count", C.c_int64), ("out", C.c_void_p), ("out_hi", C.c_void_p), ("out_lo", C.c_void_p),
+                ("out_stride", C.c_int64)]
+
+
+class Route(C.Structure):
+    _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("column", C.c_int64), ("chosen", C.c_void_p), ("weight", C.c_void_p), ("rank", C.c_void_p),
+                ("counts", C.c_void_p)]
+
+
+class Experts(C.Structure):
+    _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("rows", C.c_int64), ("inner", C.c_int64), ("ff", C.c_int64), ("weight_dtype", C.c_int32),
+                ("up", C.c_void_p), ("down", C.c_void_p), ("chosen", C.c_void_p), ("weight", C.c_void_p), ("x", C.c_void_p), ("x_hi", C.c_void_p),
+                ("x_lo", C.c_void_p), ("sumsq_in", C.c_void_p), ("parts_in", C.c_int32), ("eps", C.c_double), ("residual", C.c_void_p), ("y", C.c_void_p)]
 
 
 class PassEntry(C.Structure):
@@ -213,6 +236,14 @@ def _declare(l: C.CDLL) -> None:
         "b200_latent_scratch_bytes": (sz, [C.POINTER(LatentArgs), i64, i32, i32, i32]),
         "b200_latent_attention": (C.c_int, [C.POINTER(LatentArgs), C.POINTER(Rows), vp, i32, vp, sz, vp, vp]),
         "b200_latent_value": (C.c_int, [C.POINTER(LatentArgs), i64, vp, vp, i64, vp, vp, vp, vp]),
+        "b200_chunk_prepare": (C.c_int, [C.POINTER(ChunkArgs), C.POINTER(Rows), C.POINTER(Units), C.POINTER(Route), vp]),
+        "b200_chunk_scratch_bytes": (sz, [C.POINTER(ChunkArgs), i64, i32, i32, i32]),
+        "b200_chunk_attention": (C.c_int, [C.POINTER(ChunkArgs), C.POINTER(Rows), i32, vp, sz, vp, vp, vp, i64, vp]),
+        "b200_chunk_attention_kernel": (C.c_char_p, [C.POINTER(ChunkArgs), i64]),
+        "b200_experts_streamed": (C.c_int, [C.POINTER(Experts), vp, vp]),
+        "b200_experts_grouped_bytes": (sz, [C.POINTER(Experts)]),
+        "b200_experts_grouped": (C.c_int, [C.POINTER(Experts), vp, vp, vp, sz, vp]),
+        "b200_experts_takes_grouped": (i32, [C.POINTER(Experts)]),
         "b200_latent_attention_kernel": (C.c_char_p, [C.POINTER(LatentArgs)]),
         "b200_take_device_status": (C.c_int, [i32, vp, C.POINTER(i32)]),
     }

@@ -1,9 +1,5 @@
-// Modules, cache, execution plan and generation of the hybrid decoder (see hybrid.h).
-#include "dl/hybrid.h"
-#include "dl/internal.h"
-#include "dl/plan.h"
-
-#include <cuda_runtime.h>
+// Modules, cache, execution plan and generation of the configured decoders (see hybrid.h, hybrid_plan.h; parallel layers: parallel.cpp).
+#include "dl/hybrid_plan.h"
 
 #include <algorithm>
 #include <atomic>
@@ -13,16 +9,8 @@
 namespace dl::nn {
 
 namespace {
-
 constexpr Index kPassRows = 8192;          // rows of one pass over the layers; longer passes are cut
 constexpr Index kPageSize = 64;
-
-int code_of(DType dtype) { return dtype == DType::bf16 ? B200_BF16 : B200_F32; }
-cudaStream_t cuda_stream(int device) { return static_cast<cudaStream_t>(runtime::stream(device)); }
-float* f32(const Tensor& t) { return static_cast<float*>(t.mutable_data()); }
-
-Tensor host_zeros(Shape shape, TensorOptions options) { return zeros(std::move(shape), options); }
-
 }  // namespace
 
 // ---- modules ------------------------------------------------------------------------------------------------
@@ -53,10 +41,11 @@ LatentAttentionMixer::LatentAttentionMixer(Index width, const LatentAttentionCon
     out = &register_parameter("o", host_zeros({width, c.heads * c.vdim}, options));
 }
 
-HybridLayer::HybridLayer(Index width, const Json& spec, TensorOptions options) {
+HybridLayer::HybridLayer(Index width, const Json& spec, const DecoderDesign& design, TensorOptions options) {
     auto norm = [&](const std::string& name) {
-        DynamicTanh n;
+        RowNorm n;
         n.weight = &register_parameter(name, ones({width}, options));
+        if (design.norm == NormKind::rms) return n;
         n.bias = &register_parameter(name + ".b", host_zeros({width}, options));
         n.alpha = &register_parameter(name + ".alpha", ones({}, options));
         return n;
@@ -74,14 +63,32 @@ HybridLayer::HybridLayer(Index width, const Json& spec, TensorOptions options) {
                                       m.at("kv_rank").positive(), m.at("q_rank").positive(), rot.at("dims").positive(), rot.at("base").number(),
                                       m.at("scale").number()};
         latent = add_module<LatentAttentionMixer>("mix", width, c, options);
+    } else if (type == "attention") {
+        ChunkedAttentionConfig c{m.at("heads").positive(), m.at("kv_heads").positive(), m.at("dim").positive(), m.at("vdim").positive(), 0, 0, 1.0,
+                                 m.at("scale").number()};
+        if (m.has("mask")) c.chunk = m.at("mask").at("size").positive();
+        if (m.has("rot")) {
+            c.rot_dims = m.at("rot").at("dims").positive();
+            c.rot_base = m.at("rot").at("base").number();
+        }
+        chunked = add_module<ChunkedAttentionMixer>("mix", width, c, options);
     } else {
         throw std::invalid_argument("configuration: unknown layer type '" + type + "'");
     }
+    if (design.parallel != (chunked != nullptr))
+        throw std::invalid_argument("configuration: layers of type '" + type + (design.parallel ? "' cannot stand beside a feed-forward" : "' belong to designs with parallel layers"));
     if (spec.has("mlp")) {
         const Json& mlp = spec.at("mlp");
-        if (mlp.at("kind").text() != "dense") throw std::invalid_argument("configuration: unknown feed-forward kind '" + mlp.at("kind").text() + "'");
+        const std::string& kind = mlp.at("kind").text();
+        if (design.parallel && kind == "moe") {
+            const MixtureConfig c{mlp.at("router").at("experts").positive(), mlp.at("router").at("top").positive(), mlp.at("expert").at("ff").positive(),
+                                  mlp.has("shared") ? mlp.at("shared").at("ff").positive() : 0};
+            mixture = add_module<MixtureOfExperts>("mlp", width, c, options);
+            return;
+        }
+        if (kind != "dense") throw std::invalid_argument("configuration: unknown feed-forward kind '" + kind + "'");
         const Index ff = mlp.at("ff").positive();
-        norm2 = norm("norm2");
+        if (!design.parallel) norm2 = norm("norm2");
         gate = &register_parameter("mlp.gate", host_zeros({ff, width}, options));
         up = &register_parameter("mlp.up", host_zeros({ff, width}, options));
         down = &register_parameter("mlp.down", host_zeros({width, ff}, options));
@@ -123,6 +130,10 @@ HybridCache::HybridCache(const HybridDecoder& model, Index slots, Index capacity
     const Device where = Device::cuda(device_);
     lengths_host_.assign(static_cast<std::size_t>(slots), 0);
     lengths_ = zeros({slots}, {DType::f32, where});   // all-zero bits: int32 zeros
+    auto rotary = [&](Index dims, double base) {
+        auto& table = tables_[{dims, base}];
+        if (!table.cosine.defined()) table = rotary_table(dims, base, capacity, where);
+    };
     try {
         for (const auto& r : model.runs()) {
             const HybridLayer& layer = *model.layers()[static_cast<std::size_t>(r.layer)];
@@ -133,8 +144,13 @@ HybridCache::HybridCache(const HybridDecoder& model, Index slots, Index capacity
                 runtime::check(b200_latent_cache_create(device_, code_of(model.dtype()), static_cast<int32_t>(slots),
                                                         static_cast<int32_t>(c.kv_rank + c.rot_dim), static_cast<int32_t>(capacity), kPageSize,
                                                         lengths(), &run.latent), "latent cache allocation");
-                auto& table = tables_[{c.rot_dims, c.rot_base}];
-                if (!table.cosine.defined()) table = rotary_table(c.rot_dims, c.rot_base, capacity, where);
+                rotary(c.rot_dims, c.rot_base);
+            } else if (layer.chunked) {
+                const auto& c = layer.chunked->config();
+                run.entries = c.chunk > 0 ? std::min(c.chunk, capacity) : capacity;
+                run.key = empty({slots, c.kv_heads, run.entries, c.dim}, {model.dtype(), where});
+                run.value = empty({slots, c.kv_heads, run.entries, c.vdim}, {model.dtype(), where});
+                if (c.rot_dims > 0) rotary(c.rot_dims, c.rot_base);
             } else {
                 const auto& c = layer.state_space->config();
                 run.conv = empty({slots, c.taps, layer.state_space->channels()}, {DType::f32, where});
@@ -165,97 +181,38 @@ void HybridCache::release(Index slot) {
 }
 void HybridCache::clear() { for (Index s = 0; s < slots(); ++s) set_length(s, 0); }
 
-// ---- plan ---------------------------------------------------------------------------------------------------
-// Fixed execution plan: packed weights, persistent workspaces, and per layer run
-//     state space:       in-projection -> convolution + recurrence -> gated group norm -> out-projection + residual + next norm
-//     latent attention:  [dq | dkv | g] projection -> norms, rotation, append -> query up-projection -> absorbed query
-//                        -> attention -> value up-projection + gate -> out-projection + residual + next norm
-//     feed-forward:      gate/up + SiLU * up -> down-projection + residual + next norm
-// bf16 models run the projections on the shadow protocol (activations as bf16 hi + lo planes); the Dynamic Tanh norms need no row
-// statistic, so the projection that finishes the residual stream writes the next norm's result itself.  f32 models and sizes the
-// shadow kernels do not take run the same kernels with f32 activations and stand-alone norms.
-class HybridPlan {
-public:
-    explicit HybridPlan(HybridDecoder& owner) : owner_(owner) {}
-
-    void refresh();
-    void reserve(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass);
-    bool shadows_for(Index rows) const;
-    // ids on the device; `pass` describes the rows.  Leaves the residual stream in hidden() and (shadow form) its final norm in the planes.
-    void run(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail = nullptr);
-    // Logits of the last run's rows.
-    void logits(Index rows, float* out, void* stream);
-    // Logits of `count` rows of the last run, picked by device indices.
-    void logits_of(const std::int32_t* index, Index count, float* out, void* stream);
-    bool prepare_choice(Index rows);
-    void choose(Index rows, const TokenFeedback& feedback, void* stream);
-    std::uint64_t buffer_epoch() const { return epoch_; }
-    void set_user(const void* user) { user_ = user; }
-    const void* user() const { return user_; }
-    int device() const { return owner_.embed().device().index; }
-
-    // Pass descriptions: host arrays -> one device block.
-    struct PassMaps {
-        Tensor block;
-        std::shared_ptr<runtime::Storage> staging;
-        b200_rows describe(std::span<const Index> slots, std::span<const Index> counts, HybridCache& cache, int device);
-    };
-    PassMaps maps;
-
-private:
-    struct Norm { Tensor weight, bias; float alpha = 1.0f; };
-    struct Layer {
-        Norm norm1, norm2;
-        const void *in, *out, *down;                // bound to the modules' tensors
-        Tensor wide, gate_up, w_key;                // latent [dq | dkv | g], interleaved feed-forward, per-head transposed keys
-        const void *uq, *w_value;
-        Tensor conv, conv_bias, dt_bias, a_log, d, gated_norm, q_norm, kv_norm;   // f32
-        Index wide_out, inner, mixed_out;           // rows of the first projection; input width of the out-projection
-    };
-    Norm pack_norm(const DynamicTanh& n, double scale = 1.0) const;
-    void linear(const float* x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y, void* stream, const char* what);
-    void shadow(const Tensor& hi, const Tensor& lo, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual,
-                float* y, const Norm* next, Tensor* out_hi, Tensor* out_lo, void* stream, const char* what);
-    b200_latent_args latent_args(const Layer& layer, const LatentAttentionMixer& mixer, const HybridCache& cache, std::size_t run) const;
-    void grow(Tensor& t, Shape shape, DType dtype);
-
-    HybridDecoder& owner_;
-    std::vector<Layer> layers_;
-    Norm final_norm_;
-    Tensor loop_step_;
-    std::uint64_t packed_version_ = ~0ull, epoch_ = 0;
-    const void* user_ = nullptr;
-    Tensor first_, h_, projected_, mixed_, y_, query_, absorbed_, latent_out_, plain_, plain_inner_, scratch_;
-    Tensor n_hi_, n_lo_, i_hi_, i_lo_;        // normed rows [rows, width]; inner rows (gated, attended, activated, query latent)
-    Tensor picked_, p_hi_, p_lo_, best_value_, best_index_;
-};
-
-HybridDecoder::HybridDecoder(const Json& config, TensorOptions options)
-    : width_(config.at("width").positive()), vocab_(config.at("vocab").positive()), dtype_(options.dtype), eps_(config.at("norm").at("eps").number()),
-      embedding_scale_(config.at("embedding").at("scale").number()), logit_scale_(config.at("logit_scale").number()) {
+// ---- decoder ------------------------------------------------------------------------------------------------
+HybridDecoder::HybridDecoder(const Json& config, const DecoderDesign& design, TensorOptions options)
+    : width_(config.at("width").positive()), vocab_(config.at("vocab").positive()), dtype_(options.dtype), design_(design),
+      eps_(config.at("norm").at("eps").number()), embedding_scale_(design.scaled ? config.at("embedding").at("scale").number() : 1.0),
+      logit_scale_(design.scaled ? config.at("logit_scale").number() : 1.0) {
     if (dtype_ != DType::f32 && dtype_ != DType::bf16) throw std::invalid_argument("the B200 decoder path stores weights in f32 or bf16");
     embed_ = &register_parameter("embed", host_zeros({vocab_, width_}, options));
     const auto& specs = config.at("layers").items();
     const auto count = static_cast<Index>(specs.size());
     if (count == 0) throw std::invalid_argument("decoder requires at least one layer");
     for (Index i = 0; i < count; ++i)
-        layers_.push_back(add_module<HybridLayer>("l" + std::to_string(i), width_, specs[static_cast<std::size_t>(i)], options));
-    Index start = 0, stop = 0, times = 1;
+        layers_.push_back(add_module<HybridLayer>("l" + std::to_string(i), width_, specs[static_cast<std::size_t>(i)], design_, options));
+    Index start = 0, stop = 0, times = 0;
     if (config.has("loop")) {
         start = config.at("loop").at("start").integer();
         stop = config.at("loop").at("stop").integer();
         times = config.at("loop").at("times").positive();
         if (start < 0 || stop < start || stop > count) throw std::invalid_argument("configuration: 'loop' must name a range of layers");
-        loop_step_ = &register_parameter("loop.step", host_zeros({times, width_}, options));
+        if ((design_.loop == LoopEntry::joined) != (design_.norm == NormKind::rms))
+            throw std::invalid_argument("this entry of a looped range is not combined with these norms");
+        if (design_.loop == LoopEntry::step) loop_step_ = &register_parameter("loop.step", host_zeros({times, width_}, options));
+        else loop_in_ = &register_parameter("loop.in", host_zeros({width_, 2 * width_}, options));
     }
     for (Index i = 0; i < start; ++i) runs_.push_back({i, -1, false});
-    if (loop_step_)
-        for (Index t = 0; t < times; ++t)
-            for (Index i = start; i < stop; ++i) runs_.push_back({i, t, i == start});
+    for (Index t = 0; t < times; ++t)
+        for (Index i = start; i < stop; ++i) runs_.push_back({i, t, i == start});
     for (Index i = stop; i < count; ++i) runs_.push_back({i, -1, false});
     final_norm_.weight = &register_parameter("final.norm", ones({width_}, options));
-    final_norm_.bias = &register_parameter("final.norm.b", host_zeros({width_}, options));
-    final_norm_.alpha = &register_parameter("final.norm.alpha", ones({}, options));
+    if (design_.norm == NormKind::dynamic_tanh) {
+        final_norm_.bias = &register_parameter("final.norm.b", host_zeros({width_}, options));
+        final_norm_.alpha = &register_parameter("final.norm.alpha", ones({}, options));
+    }
     head_ = &register_parameter("head", host_zeros({vocab_, width_}, options));
 }
 
@@ -265,9 +222,9 @@ HybridPlan& HybridDecoder::plan() {
     return *plan_;
 }
 
-namespace {
 Tensor to_f32(const Tensor& t) { return t.to(Device::cpu()).astype(DType::f32).to(t.device()); }
 
+namespace {
 // [heads * dim, rank] -> per head [rank, dim]
 Tensor transpose_heads(const Tensor& w, Index heads, Index dim, Index rank) {
     const Tensor host = w.to(Device::cpu());
@@ -283,7 +240,7 @@ Tensor transpose_heads(const Tensor& w, Index heads, Index dim, Index rank) {
 }
 }  // namespace
 
-HybridPlan::Norm HybridPlan::pack_norm(const DynamicTanh& n, double scale) const {
+HybridPlan::Norm HybridPlan::pack_norm(const RowNorm& n, double scale) const {
     Norm packed;
     auto scaled = [&](const Tensor& t) {
         Tensor host = t.to(Device::cpu()).astype(DType::f32).clone();
@@ -291,6 +248,8 @@ HybridPlan::Norm HybridPlan::pack_norm(const DynamicTanh& n, double scale) const
         return host.to(t.device());
     };
     packed.weight = scaled(*n.weight);
+    packed.rms = n.rms();
+    if (packed.rms) return packed;
     packed.bias = scaled(*n.bias);
     packed.alpha = n.alpha->to(Device::cpu()).astype(DType::f32).data<float>()[0];
     return packed;
@@ -307,6 +266,11 @@ void HybridPlan::refresh() {
     for (const auto& module : owner_.layers()) {
         Layer l{};
         l.norm1 = pack_norm(module->norm1);
+        if (module->chunked) {
+            pack_parallel(*module, l);
+            layers_.push_back(std::move(l));
+            continue;
+        }
         if (module->state_space) {
             const StateSpaceMixer& m = *module->state_space;
             l.in = m.in->raw_data(); l.out = m.out->raw_data();
@@ -335,6 +299,10 @@ void HybridPlan::refresh() {
     }
     final_norm_ = pack_norm(owner_.final_norm(), owner_.logit_scale());   // logits = head (norm(x) * logit_scale)
     if (owner_.loop_step()) loop_step_ = to_f32(*owner_.loop_step());
+    if (owner_.loop_in()) {   // "loop.in" [x; first] = loop_x_ x + loop_first_ first
+        loop_x_ = owner_.loop_in()->narrow(1, 0, owner_.width());
+        loop_first_ = owner_.loop_in()->narrow(1, owner_.width(), owner_.width());
+    }
     synchronize(Device::cuda(device()));
     packed_version_ = version;
 }
@@ -346,9 +314,10 @@ bool HybridPlan::shadows_for(Index rows) const {
     if (D % 8 || !takes(D, owner_.vocabulary())) return false;
     for (std::size_t i = 0; i < layers_.size(); ++i) {
         const HybridLayer& module = *owner_.layers()[i];
+        if (module.chunked && !takes(D, layers_[i].attention_columns)) return false;
         if (!takes(D, layers_[i].wide_out) || !takes(layers_[i].inner, D)) return false;
         if (module.latent && !takes(module.latent->config().q_rank, module.latent->uq->size(0))) return false;
-        if (module.has_mlp() && (!takes(D, 2 * module.gate->size(0)) || !takes(module.gate->size(0), D))) return false;
+        if (module.has_mlp() && (!takes(D, 2 * module.gate->size(0)) || (!module.chunked && !takes(module.gate->size(0), D)))) return false;
     }
     return true;
 }
@@ -369,7 +338,7 @@ b200_latent_args HybridPlan::latent_args(const Layer& layer, const LatentAttenti
     a.vdim = static_cast<int32_t>(c.vdim); a.kv_rank = static_cast<int32_t>(c.kv_rank); a.q_rank = static_cast<int32_t>(c.q_rank);
     a.rot_dims = static_cast<int32_t>(c.rot_dims);
     a.scale = static_cast<float>(c.scale); a.eps = owner_.eps();
-    const auto& table = cache.rotary(c);
+    const auto& table = cache.rotary(c.rot_dims, c.rot_base);
     a.cosine = table.cosine.data<float>(); a.sine = table.sine.data<float>(); a.positions = static_cast<int32_t>(table.cosine.size(0));
     a.q_norm = layer.q_norm.data<float>(); a.kv_norm = layer.kv_norm.data<float>();
     a.cache = cache.run(run).latent;
@@ -388,7 +357,8 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
         const HybridLayer& module = *owner_.layers()[index];
         wide = std::max(wide, layers_[index].wide_out);
         inner = std::max(inner, layers_[index].inner);
-        if (module.has_mlp()) inner = std::max(inner, module.gate->size(0));
+        if (module.has_mlp() && !module.chunked) inner = std::max(inner, module.gate->size(0));
+        if (module.chunked) continue;   // reserve_parallel
         if (module.state_space) {
             channels = std::max(channels, module.state_space->channels());
             y = std::max(y, module.state_space->inner());
@@ -408,13 +378,22 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
     if (channels) { grow(mixed_, {rows, channels}, DType::f32); grow(y_, {rows, y}, DType::f32); }
     if (query) { grow(query_, {rows, query}, DType::f32); grow(absorbed_, {rows, absorbed}, DType::f32); grow(latent_out_, {rows, latent}, DType::f32); }
     if (bf16 && shadows_for(rows)) {
-        grow(n_hi_, {rows, D}, DType::bf16); grow(n_lo_, {rows, D}, DType::bf16);
-        grow(i_hi_, {rows, inner}, DType::bf16); grow(i_lo_, {rows, inner}, DType::bf16);
+        grow(n_, rows, D);
+        grow(i_, rows, inner);
+        if (owner_.design().norm == NormKind::rms) {
+            Index parts = 1;
+            for (const auto& layer : layers_) parts = std::max<Index>(parts, b200_linear_shadow_parts(rows, layer.inner, D));
+            if (owner_.loop_in()) parts = std::max<Index>(parts, b200_linear_shadow_parts(rows, D, D));
+            grow(squares_, {parts, rows}, DType::f32);
+        }
+        if (owner_.loop_in()) grow(x_, rows, D);
     } else {
         grow(plain_, {rows, D}, DType::f32);
         grow(plain_inner_, {rows, inner}, DType::f32);
     }
     grow(scratch_, {static_cast<Index>(scratch / 4 + 1)}, DType::f32);
+    if (owner_.loop_in()) { grow(joined_first_, {rows, D}, DType::f32); grow(entered_, {rows, D}, DType::f32); }
+    reserve_parallel(rows, max_length, cache, pass);
 }
 
 void HybridPlan::linear(const float* x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y,
@@ -423,67 +402,134 @@ void HybridPlan::linear(const float* x, Index rows, Index in, const void* w, Ind
     probe(0);
 }
 
-void HybridPlan::shadow(const Tensor& hi, const Tensor& lo, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue,
-                        const float* residual, float* y, const Norm* next, Tensor* out_hi, Tensor* out_lo, void* stream, const char* what) {
+void HybridPlan::shadow(const Planes& x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y,
+                        const Norm* next, Planes* to, void* stream, const char* what, Index to_column, Index to_stride) {
     b200_shadow_linear_args args{};
-    args.x_hi = hi.raw_data();
-    args.x_lo = owner_.activation_dtype() == DType::bf16 && rows >= 17 ? nullptr : lo.raw_data();
+    args.x_hi = x.hi.raw_data();
+    args.x_lo = owner_.activation_dtype() == DType::bf16 && rows >= 17 ? nullptr : x.lo.raw_data();
     args.rows = rows; args.in = in; args.weight = w; args.out = out;
     args.epilogue = epilogue; args.residual = residual; args.y = y;
+    if (x.parts > 0) { args.sumsq_in = squares_.data<float>(); args.parts_in = static_cast<int32_t>(x.parts); args.eps = owner_.eps(); }
     b200_elementwise_norm norm{};
-    if (next) {
+    if (to) {
+        args.out_hi = static_cast<std::uint16_t*>(to->hi.mutable_data()) + to_column;
+        args.out_lo = static_cast<std::uint16_t*>(to->lo.mutable_data()) + to_column;
+        args.out_stride = to_stride;
+        to->parts = 0;
+    }
+    if (next && next->rms) {
+        args.out_norm_weight = next->weight.raw_data(); args.out_norm_dtype = B200_F32;
+        args.sumsq_out = f32(squares_);
+        to->parts = b200_linear_shadow_parts(rows, in, out);
+    } else if (next) {
         norm = {next->alpha, next->weight.data<float>(), next->bias.data<float>()};
         args.out_norm = &norm;
     }
-    if (out_hi) { args.out_hi = out_hi->mutable_data(); args.out_lo = out_lo->mutable_data(); }
     runtime::check(b200_linear_shadow(&args, stream), what);
     probe(0);
+}
+
+// Planes of the rows under an RMS norm, whose factor the consumer applies.
+void HybridPlan::planes_of(const float* x, Index rows, const Norm& norm, Planes& to, void* stream) {
+    runtime::check(b200_shadow_from_rows(x, rows, owner_.width(), norm.weight.raw_data(), B200_F32, to.hi.mutable_data(), to.lo.mutable_data(),
+                                         f32(squares_), stream), "norm");
+    to.parts = 1;
+    probe(2);
 }
 
 void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail) {
     const Index rows = pass.rows, D = owner_.width();
     const bool planes = shadows_for(rows);
     float *first = f32(first_), *h = f32(h_);
-    runtime::check(b200_embedding_scaled(owner_.embed().raw_data(), code_of(owner_.dtype()), ids, rows, owner_.vocabulary(), D,
-                                         static_cast<float>(owner_.embedding_scale()), first, stream), "embedding");
-    probe(2);
-    const float* in = first;
-    bool normed = false;   // the previous projection has written this run's norm1
-    auto stand_alone_norm = [&](const float* x, const float* add_rows, const float* add_vector, float* sum, const Norm& n) {
-        const b200_elementwise_norm norm{n.alpha, n.weight.data<float>(), n.bias.data<float>()};
-        runtime::check(b200_dynamic_tanh(x, add_rows, add_vector, rows, D, &norm, sum, planes ? nullptr : f32(plain_),
-                                         planes ? n_hi_.mutable_data() : nullptr, planes ? n_lo_.mutable_data() : nullptr, stream), "norm");
+    const bool rms = owner_.design().norm == NormKind::rms;
+    const auto& runs = owner_.runs();
+    bool normed = false;   // the previous kernel has written this run's norm1
+    auto embed = [&](const Norm* norm, Planes& to) {
+        runtime::check(b200_embedding_shadow(owner_.embed().raw_data(), code_of(owner_.dtype()), ids, rows, owner_.vocabulary(), D,
+                                             norm ? norm->weight.raw_data() : nullptr, B200_F32, first, to.hi.mutable_data(), to.lo.mutable_data(),
+                                             f32(squares_), stream), "embedding");
+        to.parts = norm ? 1 : 0;
         probe(2);
     };
-    // residual projection of inner rows; `next` is the norm that follows it directly (nullptr: something is added first)
-    auto residual_projection = [&](Index inner, const void* w, const Norm* next, const char* what) {
-        if (planes) {
-            shadow(i_hi_, i_lo_, rows, inner, w, D, B200_EPI_RESIDUAL, in, h, next, next ? &n_hi_ : nullptr, next ? &n_lo_ : nullptr, stream, what);
+    if (rms && planes) {
+        if (owner_.loop_in()) embed(nullptr, x_);
+        if (!owner_.loop_in() || !runs.front().begins_pass) {
+            embed(&layers_[static_cast<std::size_t>(runs.front().layer)].norm1, n_);
+            normed = true;
+        }
+    } else {
+        runtime::check(b200_embedding_scaled(owner_.embed().raw_data(), code_of(owner_.dtype()), ids, rows, owner_.vocabulary(), D,
+                                             static_cast<float>(owner_.embedding_scale()), first, stream), "embedding");
+        probe(2);
+    }
+    if (owner_.loop_in()) {   // the embedding output's share of every pass's entry
+        if (planes) shadow(x_, rows, D, loop_first_.raw_data(), D, B200_EPI_STORE, nullptr, f32(joined_first_), nullptr, nullptr, stream, "loop projection");
+        else linear(first, rows, D, loop_first_.raw_data(), D, B200_EPI_STORE, nullptr, f32(joined_first_), stream, "loop projection");
+    }
+    if (grouped_) runtime::check_cuda(cudaMemsetAsync(counts_.mutable_data(), 0, counts_.nbytes(), static_cast<cudaStream_t>(stream)), "cudaMemsetAsync");
+    const float* in = first;
+    auto stand_alone_norm = [&](const float* x, const float* add_rows, const float* add_vector, float* sum, const Norm& n) {
+        if (n.rms && planes) return planes_of(x, rows, n, n_, stream);
+        if (n.rms) {
+            runtime::check(b200_rms_norm(x, n.weight.raw_data(), B200_F32, rows, D, owner_.eps(), f32(plain_), stream), "norm");
         } else {
-            linear(f32(plain_inner_), rows, inner, w, D, B200_EPI_RESIDUAL, in, h, stream, what);
-            if (next) stand_alone_norm(h, nullptr, nullptr, nullptr, *next);
+            const b200_elementwise_norm norm{n.alpha, n.weight.data<float>(), n.bias.data<float>()};
+            runtime::check(b200_dynamic_tanh(x, add_rows, add_vector, rows, D, &norm, sum, planes ? nullptr : f32(plain_),
+                                             planes ? n_.hi.mutable_data() : nullptr, planes ? n_.lo.mutable_data() : nullptr, stream), "norm");
+        }
+        probe(2);
+    };
+    // residual projection of inner rows
+    auto residual_projection = [&](Index inner, const void* w, const float* residual, const After& after, const char* what) {
+        if (planes) {
+            shadow(i_, rows, inner, w, D, B200_EPI_RESIDUAL, residual, h, after.norm, after.norm ? &n_ : after.raw ? &x_ : nullptr, stream, what);
+        } else {
+            linear(f32(plain_inner_), rows, inner, w, D, B200_EPI_RESIDUAL, residual, h, stream, what);
+            if (after.norm) stand_alone_norm(h, nullptr, nullptr, nullptr, *after.norm);
         }
         in = h;
     };
-    const auto& runs = owner_.runs();
+    auto keep = [&](std::vector<float>& rows_after) {
+        const std::size_t at = rows_after.size();
+        rows_after.resize(at + static_cast<std::size_t>(rows * D));
+        runtime::copy_bytes(rows_after.data() + at, Device::cpu(), h, Device::cuda(device()), static_cast<std::size_t>(rows * D) * sizeof(float));
+    };
     for (std::size_t i = 0; i < runs.size(); ++i) {
         const LayerRun& r = runs[i];
         const HybridLayer& module = *owner_.layers()[static_cast<std::size_t>(r.layer)];
         const Layer& layer = layers_[static_cast<std::size_t>(r.layer)];
-        if (r.begins_pass) {
+        if (r.begins_pass && owner_.loop_in()) {
+            float* entered = f32(entered_);
+            if (planes) {
+                shadow(x_, rows, D, loop_x_.raw_data(), D, B200_EPI_RESIDUAL, f32(joined_first_), entered, &layer.norm1, &n_, stream, "loop projection");
+            } else {
+                linear(in, rows, D, loop_x_.raw_data(), D, B200_EPI_RESIDUAL, f32(joined_first_), entered, stream, "loop projection");
+                stand_alone_norm(entered, nullptr, nullptr, nullptr, layer.norm1);
+            }
+            in = entered;
+        } else if (r.begins_pass) {
             stand_alone_norm(in, r.pass > 0 ? first : nullptr, loop_step_.data<float>() + r.pass * D, h, layer.norm1);
             in = h;
         } else if (!normed) {
             stand_alone_norm(in, nullptr, nullptr, nullptr, layer.norm1);
         }
         const bool last = i + 1 == runs.size();
-        const Norm* after_layer = last ? &final_norm_ : runs[i + 1].begins_pass ? nullptr : &layers_[static_cast<std::size_t>(runs[i + 1].layer)].norm1;
-        const Norm* after_mixer = module.has_mlp() ? &layer.norm2 : after_layer;
+        // (where a pass begins next, something is added or projected before the norm)
+        const After after_layer = last ? After{&final_norm_, false}
+            : runs[i + 1].begins_pass ? After{nullptr, owner_.loop_in() != nullptr} : After{&layers_[static_cast<std::size_t>(runs[i + 1].layer)].norm1, false};
+        normed = after_layer.norm != nullptr;
+        if (module.chunked) {
+            const float* residual = run_parallel(i, in, pass, cache, max_length, stream);
+            residual_projection(layer.inner, layer.out, residual, after_layer, "output projection");
+            if (trail) keep(*trail);
+            continue;
+        }
+        const After after_mixer = module.has_mlp() ? After{&layer.norm2, false} : after_layer;
         float* projected = f32(projected_);
-        if (planes) shadow(n_hi_, n_lo_, rows, D, layer.in, layer.wide_out, B200_EPI_STORE, nullptr, projected, nullptr, nullptr, nullptr, stream, "mixer projection");
+        if (planes) shadow(n_, rows, D, layer.in, layer.wide_out, B200_EPI_STORE, nullptr, projected, nullptr, nullptr, stream, "mixer projection");
         else linear(f32(plain_), rows, D, layer.in, layer.wide_out, B200_EPI_STORE, nullptr, projected, stream, "mixer projection");
-        void* inner_hi = planes ? i_hi_.mutable_data() : nullptr;
-        void* inner_lo = planes ? i_lo_.mutable_data() : nullptr;
+        void* inner_hi = planes ? i_.hi.mutable_data() : nullptr;
+        void* inner_lo = planes ? i_.lo.mutable_data() : nullptr;
         float* inner_plain = planes ? nullptr : f32(plain_inner_);
         if (module.state_space) {
             const auto& c = module.state_space->config();
@@ -505,7 +551,7 @@ void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache
             runtime::check(b200_latent_prepare(&a, &pass, projected, inner_plain, inner_hi, inner_lo, stream), "latent norms");
             probe(2);
             const Index query_out = c.heads * (c.dim + c.rot_dim);
-            if (planes) shadow(i_hi_, i_lo_, rows, c.q_rank, layer.uq, query_out, B200_EPI_STORE, nullptr, f32(query_), nullptr, nullptr, nullptr, stream, "query up-projection");
+            if (planes) shadow(i_, rows, c.q_rank, layer.uq, query_out, B200_EPI_STORE, nullptr, f32(query_), nullptr, nullptr, stream, "query up-projection");
             else linear(f32(plain_inner_), rows, c.q_rank, layer.uq, query_out, B200_EPI_STORE, nullptr, f32(query_), stream, "query up-projection");
             runtime::check(b200_latent_query(&a, &pass, f32(query_), f32(absorbed_), stream), "absorbed query");
             probe(0);
@@ -516,25 +562,20 @@ void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache
                                              inner_hi, inner_lo, stream), "value up-projection");
             probe(0);
         }
-        residual_projection(layer.inner, layer.out, after_mixer, "output projection");
+        residual_projection(layer.inner, layer.out, in, after_mixer, "output projection");
         if (module.has_mlp()) {
             const Index ff = module.gate->size(0);
-            if (planes) shadow(n_hi_, n_lo_, rows, D, layer.gate_up.raw_data(), 2 * ff, B200_EPI_SWIGLU, nullptr, nullptr, nullptr, &i_hi_, &i_lo_, stream, "gate/up projection");
+            if (planes) shadow(n_, rows, D, layer.gate_up.raw_data(), 2 * ff, B200_EPI_SWIGLU, nullptr, nullptr, nullptr, &i_, stream, "gate/up projection");
             else linear(f32(plain_), rows, D, layer.gate_up.raw_data(), 2 * ff, B200_EPI_SWIGLU, nullptr, f32(plain_inner_), stream, "gate/up projection");
-            residual_projection(ff, layer.down, after_layer, "down projection");
+            residual_projection(ff, layer.down, in, after_layer, "down projection");
         }
-        normed = after_layer != nullptr;
-        if (trail) {
-            const std::size_t at = trail->size();
-            trail->resize(at + static_cast<std::size_t>(rows * D));
-            runtime::copy_bytes(trail->data() + at, Device::cpu(), h, Device::cuda(device()), static_cast<std::size_t>(rows * D) * sizeof(float));
-        }
+        if (trail) keep(*trail);
     }
 }
 
 void HybridPlan::logits(Index rows, float* out, void* stream) {
     const Index D = owner_.width(), V = owner_.vocabulary();
-    if (shadows_for(rows)) shadow(n_hi_, n_lo_, rows, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, nullptr, nullptr, nullptr, stream, "logits");
+    if (shadows_for(rows)) shadow(n_, rows, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, nullptr, nullptr, stream, "logits");
     else linear(f32(plain_), rows, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, stream, "logits");
 }
 
@@ -542,12 +583,19 @@ void HybridPlan::logits_of(const std::int32_t* index, Index count, float* out, v
     const Index D = owner_.width(), V = owner_.vocabulary();
     const bool planes = shadows_for(count);
     grow(picked_, {count, D}, DType::f32);
-    if (planes) { grow(p_hi_, {count, D}, DType::bf16); grow(p_lo_, {count, D}, DType::bf16); }
+    if (planes) grow(p_, count, D);
     runtime::check(b200_gather_rows(f32(h_), index, count, D, f32(picked_), stream), "gather rows");
-    const b200_elementwise_norm norm{final_norm_.alpha, final_norm_.weight.data<float>(), final_norm_.bias.data<float>()};
-    runtime::check(b200_dynamic_tanh(f32(picked_), nullptr, nullptr, count, D, &norm, nullptr, planes ? nullptr : f32(picked_),
-                                     planes ? p_hi_.mutable_data() : nullptr, planes ? p_lo_.mutable_data() : nullptr, stream), "final norm");
-    if (planes) shadow(p_hi_, p_lo_, count, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, nullptr, nullptr, nullptr, stream, "logits");
+    if (final_norm_.rms && planes) {
+        grow(squares_, {1, count}, DType::f32);
+        planes_of(f32(picked_), count, final_norm_, p_, stream);
+    } else if (final_norm_.rms) {
+        runtime::check(b200_rms_norm(f32(picked_), final_norm_.weight.raw_data(), B200_F32, count, D, owner_.eps(), f32(picked_), stream), "final norm");
+    } else {
+        const b200_elementwise_norm norm{final_norm_.alpha, final_norm_.weight.data<float>(), final_norm_.bias.data<float>()};
+        runtime::check(b200_dynamic_tanh(f32(picked_), nullptr, nullptr, count, D, &norm, nullptr, planes ? nullptr : f32(picked_),
+                                         planes ? p_.hi.mutable_data() : nullptr, planes ? p_.lo.mutable_data() : nullptr, stream), "final norm");
+    }
+    if (planes) shadow(p_, count, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, nullptr, nullptr, stream, "logits");
     else linear(f32(picked_), count, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, stream, "logits");
 }
 
@@ -563,8 +611,9 @@ bool HybridPlan::prepare_choice(Index rows) {
 void HybridPlan::choose(Index rows, const TokenFeedback& f, void* stream) {
     const Index D = owner_.width(), V = owner_.vocabulary();
     b200_shadow_linear_args args{};
-    args.x_hi = n_hi_.raw_data();
-    args.x_lo = owner_.activation_dtype() == DType::bf16 && rows >= 17 ? nullptr : n_lo_.raw_data();
+    args.x_hi = n_.hi.raw_data();
+    args.x_lo = owner_.activation_dtype() == DType::bf16 && rows >= 17 ? nullptr : n_.lo.raw_data();
+    if (n_.parts > 0) { args.sumsq_in = squares_.data<float>(); args.parts_in = static_cast<int32_t>(n_.parts); args.eps = owner_.eps(); }
     args.rows = rows; args.in = D; args.weight = owner_.head().raw_data(); args.out = V;
     args.epilogue = B200_EPI_ARGMAX;
     args.best_value = f32(best_value_);

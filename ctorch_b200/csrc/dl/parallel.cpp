@@ -1,0 +1,239 @@
+// Parallel layers of the configured decoders: chunked attention and a feed-forward or a mixture of experts on one norm (see hybrid.h).
+#include "dl/hybrid_plan.h"
+
+#include <algorithm>
+#include <stdexcept>
+
+namespace dl::nn {
+
+namespace {
+// Up to this many rows the units of a dense feed-forward are projected together with q, k, v and g and activated beside the norms of
+// the heads (a launch less); longer passes project them on their own, where the epilogue activates them without a round trip.
+constexpr Index kRowsBeside = 128;
+
+Index round_up_8(Index n) { return (n + 7) & ~static_cast<Index>(7); }
+}  // namespace
+
+// ---- modules ------------------------------------------------------------------------------------------------
+ChunkedAttentionMixer::ChunkedAttentionMixer(Index width, const ChunkedAttentionConfig& c, TensorOptions options) : config_(c) {
+    if (c.heads % c.kv_heads) throw std::invalid_argument("chunked attention: heads must be a multiple of kv_heads");
+    if (c.rot_dims % 2 || c.rot_dims > c.dim) throw std::invalid_argument("chunked attention: rotated dimensions must be even and at most dim");
+    q = &register_parameter("q", host_zeros({c.heads * c.dim, width}, options));
+    k = &register_parameter("k", host_zeros({c.kv_heads * c.dim, width}, options));
+    v = &register_parameter("v", host_zeros({c.kv_heads * c.vdim, width}, options));
+    q_norm = &register_parameter("q.norm", ones({c.heads * c.dim}, options));
+    k_norm = &register_parameter("k.norm", ones({c.kv_heads * c.dim}, options));
+    gate = &register_parameter("g", host_zeros({c.heads, width}, options));
+    out = &register_parameter("o", host_zeros({width, c.heads * c.vdim}, options));
+}
+Index ChunkedAttentionMixer::columns() const { return config_.heads * (config_.dim + 1) + config_.kv_heads * (config_.dim + config_.vdim); }
+
+MixtureOfExperts::MixtureOfExperts(Index width, const MixtureConfig& c, TensorOptions options) : config_(c) {
+    if (c.top > c.experts) throw std::invalid_argument("mixture of experts: 'top' exceeds the number of experts");
+    if (c.experts > B200_MAX_EXPERTS) throw std::invalid_argument("mixture of experts: more than " + std::to_string(B200_MAX_EXPERTS) + " experts");
+    for (Index e = 0; e < c.experts; ++e) {
+        const std::string name = "e" + std::to_string(e);
+        up.push_back(&register_parameter(name + ".up", host_zeros({c.ff, width}, options)));
+        down.push_back(&register_parameter(name + ".down", host_zeros({width, c.ff}, options)));
+    }
+    router = &register_parameter("router", host_zeros({c.experts, width}, options));
+    if (c.shared_ff > 0) {
+        shared_up = &register_parameter("shared.up", host_zeros({c.shared_ff, width}, options));
+        shared_down = &register_parameter("shared.down", host_zeros({width, c.shared_ff}, options));
+    }
+}
+
+// ---- plan ---------------------------------------------------------------------------------------------------
+void HybridPlan::pack_parallel(const HybridLayer& module, Layer& l) const {
+    const ChunkedAttentionMixer& m = *module.chunked;
+    const Index D = owner_.width();
+    const TensorOptions options{owner_.dtype(), m.q->device()};
+    std::vector<Tensor> rows{*m.q, *m.k, *m.v, *m.gate}, columns{*m.out};
+    Index count = m.columns();
+    auto pad = [&] {   // sections of a projected row start at multiples of eight
+        if (count % 8) rows.push_back(zeros({round_up_8(count) - count, D}, options));
+        count = round_up_8(count);
+    };
+    pad();
+    l.attention_columns = count;
+    if (module.has_mlp()) {
+        l.unit_column = count;
+        l.units = module.gate->size(0);
+        rows.push_back(interleave_rows(*module.gate, *module.up));
+        columns.push_back(*module.down);
+        count += 2 * l.units;
+        pad();
+    } else if (module.mixture) {
+        const MixtureOfExperts& e = *module.mixture;
+        l.router_column = count;
+        rows.push_back(*e.router);
+        count += e.config().experts;
+        pad();
+        if (e.shared_up) {
+            l.unit_column = count;
+            l.units = e.config().shared_ff;
+            rows.push_back(*e.shared_up);
+            columns.push_back(*e.shared_down);
+            count += l.units;
+            pad();
+        }
+        std::vector<Tensor> ups, downs;
+        for (const Tensor* t : e.up) ups.push_back(*t);
+        for (const Tensor* t : e.down) downs.push_back(*t);
+        l.experts_up = concat_rows(ups);
+        l.experts_down = concat_rows(downs);
+    }
+    l.wide = concat_rows(rows);
+    l.in = l.wide.raw_data();
+    l.wide_out = count;
+    l.attended = m.out->size(1);
+    l.joint = columns.size() == 1 ? columns.front() : concat_columns(columns);
+    l.out = l.joint.raw_data();
+    l.inner = l.attended + l.units;
+    l.q_norm = to_f32(*m.q_norm);
+    l.kv_norm = to_f32(*m.k_norm);
+}
+
+bool HybridPlan::units_beside(const HybridLayer& module, Index rows, bool planes) const { return !module.has_mlp() || !planes || rows <= kRowsBeside; }
+
+b200_chunk_args HybridPlan::chunk_args(const Layer& layer, const ChunkedAttentionMixer& mixer, const HybridCache& cache, std::size_t run, Index stride) const {
+    const auto& c = mixer.config();
+    const HybridCache::Run& r = cache.run(run);
+    b200_chunk_args a{};
+    a.heads = static_cast<int32_t>(c.heads); a.kv_heads = static_cast<int32_t>(c.kv_heads); a.dim = static_cast<int32_t>(c.dim);
+    a.vdim = static_cast<int32_t>(c.vdim); a.rot_dims = static_cast<int32_t>(c.rot_dims);
+    // (no position reaches a chunk that is longer than the cache)
+    a.chunk = static_cast<int32_t>(c.chunk > cache.capacity() ? 0 : c.chunk); a.entries = static_cast<int32_t>(r.entries);
+    a.scale = static_cast<float>(c.scale); a.eps = owner_.eps();
+    if (c.rot_dims > 0) {
+        const auto& table = cache.rotary(c.rot_dims, c.rot_base);
+        a.cosine = table.cosine.data<float>(); a.sine = table.sine.data<float>(); a.positions = static_cast<int32_t>(table.cosine.size(0));
+    }
+    a.q_norm = layer.q_norm.data<float>(); a.k_norm = layer.kv_norm.data<float>();
+    a.dtype = code_of(owner_.dtype());
+    a.key_cache = r.key.mutable_data(); a.value_cache = r.value.mutable_data();
+    a.projected = projected_.data<float>(); a.stride = stride;
+    a.query = chunk_query_.mutable_data(); a.key = chunk_key_.mutable_data(); a.value = chunk_value_.mutable_data();
+    return a;
+}
+
+b200_experts HybridPlan::expert_args(const Layer& layer, const MixtureOfExperts& mixture, Index rows) const {
+    const auto& c = mixture.config();
+    b200_experts a{};
+    a.experts = static_cast<int32_t>(c.experts); a.top = static_cast<int32_t>(c.top);
+    a.rows = rows; a.in = owner_.width(); a.ff = c.ff;
+    a.weight_dtype = code_of(owner_.dtype());
+    a.up = layer.experts_up.raw_data(); a.down = layer.experts_down.raw_data();
+    a.chosen = static_cast<const std::int32_t*>(chosen_.raw_data()); a.weight = score_.data<float>();
+    if (shadows_for(rows)) {
+        a.x_hi = n_.hi.raw_data(); a.x_lo = n_.lo.raw_data();
+        a.sumsq_in = squares_.data<float>(); a.parts_in = static_cast<int32_t>(n_.parts);
+    } else {
+        a.x = f32(plain_);
+    }
+    a.eps = owner_.eps();
+    a.residual = f32(h_); a.y = f32(h_);
+    return a;
+}
+
+void HybridPlan::reserve_parallel(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass) {
+    grouped_ = false;
+    Index query = 0, key = 0, value = 0, slots = 0, act = 0, most_experts = 0;
+    for (const auto& module : owner_.layers()) {
+        if (module->chunked) {
+            const auto& c = module->chunked->config();
+            query = std::max(query, c.heads * c.dim);
+            key = std::max(key, c.kv_heads * c.dim);
+            value = std::max(value, c.kv_heads * c.vdim);
+        }
+        if (module->mixture) {
+            const auto& c = module->mixture->config();
+            slots = std::max(slots, c.top);
+            act = std::max(act, c.top * c.ff);
+            most_experts = std::max(most_experts, c.experts);
+        }
+    }
+    if (query == 0) return;
+    grow(chunk_query_, {rows, query}, owner_.dtype());
+    grow(chunk_key_, {rows, key}, owner_.dtype());
+    grow(chunk_value_, {rows, value}, owner_.dtype());
+    if (slots) {
+        grow(chosen_, {rows, slots}, DType::f32);   // int32 payload
+        grow(rank_, {rows, slots}, DType::f32);
+        grow(score_, {rows, slots}, DType::f32);
+        grow(counts_, {static_cast<Index>(owner_.runs().size()), most_experts}, DType::f32);
+    }
+    std::size_t scratch = 0, grouped = 0;
+    bool streamed = false;
+    for (std::size_t i = 0; i < owner_.runs().size(); ++i) {
+        const auto index = static_cast<std::size_t>(owner_.runs()[i].layer);
+        const HybridLayer& module = *owner_.layers()[index];
+        if (module.chunked) {
+            const b200_chunk_args a = chunk_args(layers_[index], *module.chunked, cache, i, layers_[index].wide_out);
+            scratch = std::max(scratch, b200_chunk_scratch_bytes(&a, rows, pass.sequences, pass.max_count, static_cast<int32_t>(max_length)));
+        }
+        if (module.mixture) {
+            const b200_experts a = expert_args(layers_[index], *module.mixture, rows);
+            if (b200_experts_takes_grouped(&a)) grouped = std::max(grouped, b200_experts_grouped_bytes(&a));
+            else streamed = true;
+        }
+    }
+    grow(scratch_, {static_cast<Index>(scratch / 4 + 1)}, DType::f32);
+    if (grouped) grow(expert_scratch_, {static_cast<Index>(grouped / 4)}, DType::f32);
+    if (streamed) grow(expert_act_, {rows, act}, DType::f32);
+    grouped_ = grouped > 0;
+}
+
+const float* HybridPlan::run_parallel(std::size_t run, const float* in, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream) {
+    const LayerRun& r = owner_.runs()[run];
+    const HybridLayer& module = *owner_.layers()[static_cast<std::size_t>(r.layer)];
+    const Layer& layer = layers_[static_cast<std::size_t>(r.layer)];
+    const Index rows = pass.rows, D = owner_.width();
+    const bool planes = shadows_for(rows), beside = units_beside(module, rows, planes);
+    const Index stride = beside ? layer.wide_out : layer.attention_columns;
+    float* projected = f32(projected_);
+    if (planes) shadow(n_, rows, D, layer.in, stride, B200_EPI_STORE, nullptr, projected, nullptr, nullptr, stream, "mixer projection");
+    else linear(f32(plain_), rows, D, layer.in, stride, B200_EPI_STORE, nullptr, projected, stream, "mixer projection");
+    if (!beside) {
+        const auto* gate_up = static_cast<const std::uint16_t*>(layer.in) + layer.unit_column * D;
+        shadow(n_, rows, D, gate_up, 2 * layer.units, B200_EPI_SWIGLU, nullptr, nullptr, nullptr, &i_, stream, "gate/up projection", layer.attended, layer.inner);
+    }
+
+    const b200_chunk_args a = chunk_args(layer, *module.chunked, cache, run, stride);
+    float* inner_plain = planes ? nullptr : f32(plain_inner_);
+    auto* inner_hi = planes ? static_cast<std::uint16_t*>(i_.hi.mutable_data()) : nullptr;
+    auto* inner_lo = planes ? static_cast<std::uint16_t*>(i_.lo.mutable_data()) : nullptr;
+    b200_units units{};
+    if (beside && layer.units > 0) {
+        units.kind = module.has_mlp() ? 1 : 2;
+        units.column = layer.unit_column; units.count = layer.units; units.out_stride = layer.inner;
+        if (planes) { units.out_hi = inner_hi + layer.attended; units.out_lo = inner_lo + layer.attended; }
+        else units.out = inner_plain + layer.attended;
+    }
+    b200_route route{};
+    b200_experts experts{};
+    bool grouped = false;
+    if (module.mixture) {
+        experts = expert_args(layer, *module.mixture, rows);
+        experts.residual = in;
+        grouped = b200_experts_takes_grouped(&experts) != 0;
+        route.experts = experts.experts; route.top = experts.top; route.column = layer.router_column;
+        route.chosen = static_cast<std::int32_t*>(chosen_.mutable_data()); route.weight = f32(score_);
+        if (grouped) {
+            route.rank = static_cast<std::int32_t*>(rank_.mutable_data());
+            route.counts = static_cast<std::int32_t*>(counts_.mutable_data()) + static_cast<Index>(run) * (counts_.numel() / static_cast<Index>(owner_.runs().size()));
+        }
+    }
+    runtime::check(b200_chunk_prepare(&a, &pass, &units, &route, stream), "attention norms");
+    probe(2);
+    runtime::check(b200_chunk_attention(&a, &pass, static_cast<int32_t>(max_length), scratch_.mutable_data(), scratch_.nbytes(), inner_plain, inner_hi, inner_lo,
+                                        layer.inner, stream), "chunked attention");
+    probe(1);
+    if (!module.mixture) return in;
+    if (grouped) runtime::check(b200_experts_grouped(&experts, route.rank, route.counts, expert_scratch_.mutable_data(), expert_scratch_.nbytes(), stream), "experts");
+    else runtime::check(b200_experts_streamed(&experts, f32(expert_act_), stream), "experts");
+    probe(0);
+    return f32(h_);
+}
+
+}  // namespace dl::nn

@@ -79,6 +79,26 @@ Tensor concat_rows(std::span<const Tensor> parts) {
     return result;
 }
 
+Tensor concat_columns(std::span<const Tensor> parts) {
+    Index columns = 0;
+    for (const auto& part : parts) {
+        require_cuda(part, "concat_columns");
+        if (part.ndim() != 2 || part.size(0) != parts.front().size(0) || part.dtype() != parts.front().dtype())
+            throw std::invalid_argument("concat_columns: matrices must share height and dtype");
+        columns += part.size(1);
+    }
+    const int device = parts.front().device().index;
+    runtime::set_device(device);
+    Tensor result = empty({parts.front().size(0), columns}, {parts.front().dtype(), parts.front().device()});
+    const std::size_t pitch = static_cast<std::size_t>(columns) * element_size(result.dtype());
+    std::size_t offset = 0;
+    for (const auto& part : parts) {
+        copy_rows(static_cast<char*>(result.mutable_data()) + offset, pitch, part, device);
+        offset += static_cast<std::size_t>(part.size(1)) * element_size(part.dtype());
+    }
+    return result;
+}
+
 Tensor add(const Tensor& a, const Tensor& b) {
     require_cuda(a, "add");
     if (a.shape() != b.shape() || a.device() != b.device()) throw std::invalid_argument("add: shapes and devices must match");

@@ -12,7 +12,12 @@ namespace {
 
 using Factory = std::shared_ptr<nn::UnaryModule> (*)(const Json&, TensorOptions);
 
-std::shared_ptr<nn::UnaryModule> hybrid(const Json& config, TensorOptions options) { return std::make_shared<nn::HybridDecoder>(config, options); }
+std::shared_ptr<nn::UnaryModule> hybrid(const Json& config, TensorOptions options) {
+    return std::make_shared<nn::HybridDecoder>(config, nn::DecoderDesign{nn::NormKind::dynamic_tanh, nn::LoopEntry::step, false, true}, options);
+}
+std::shared_ptr<nn::UnaryModule> parallel(const Json& config, TensorOptions options) {
+    return std::make_shared<nn::HybridDecoder>(config, nn::DecoderDesign{nn::NormKind::rms, nn::LoopEntry::joined, true, false}, options);
+}
 
 // Grouped-query decoder with its embedding and output layers, under the names of the reference's example model.
 std::shared_ptr<nn::UnaryModule> transformer(const Json& c, TensorOptions options) {
@@ -25,6 +30,7 @@ std::shared_ptr<nn::UnaryModule> transformer(const Json& c, TensorOptions option
 struct Entry { const char* name; Factory make; };
 constexpr Entry kRegistry[] = {
     {"Ripitar", hybrid},
+    {"Sinezen", parallel},
     {"TransformerDecoder", transformer},
 };
 

@@ -1,0 +1,705 @@
+// Chunked grouped-query attention: a position sees its own chunk of positions up to itself, so a slot keeps one chunk of keys and
+// values ([slot][kv_head][entry][dim], position p in entry p mod chunk) however long the sequence grows, and what a step reads is one
+// contiguous block per (sequence, kv head).  Keys and values may have different widths.
+//
+//   * chunk_prepare_kernel, one CTA per row (and one per slice of its feed-forward units): RMS norms over all query and all key heads, rotation of halves, append (or the
+//     workspaces of a longer pass), the activation of feed-forward units and the router's choice for the same row.
+//   * chunk_mma_kernel: bf16, tiles of keys and values through a cp.async ring with swizzled rows, mma.sync products, online softmax
+//     in f32 registers, weights as hi + lo planes, the heads of a group side by side so that a key is fetched once for all of them.
+//       steps (one row per sequence): 16 rows = heads of one token; the warps divide the keys of a tile and merge at the end; keys are
+//         split over CTAs, with a merge kernel, where the (sequence, kv head) pairs do not fill the SMs;
+//       longer passes: 64 rows = positions x heads of a group, 16 per warp; keys before the pass come from the slot, the pass's own
+//         keys from its workspaces.
+//   * chunk_generic_kernel: f32 and odd sizes, f32 FMAs, one (row, head) per CTA.
+//   * chunk_append_kernel: after a longer pass, the rows of every sequence's last chunk go into its slot.
+#include "mma.cuh"
+#include "rows.cuh"
+
+#include <algorithm>
+
+namespace b200 {
+namespace {
+
+struct ChunkParams {
+    int heads, kv_heads, group, dim, vdim, rot_dims, chunk, entries;
+    float scale, eps;
+    const float *cosine, *sine;
+    int positions;
+    const float *q_norm, *k_norm;
+    void *key_cache, *value_cache, *query, *key, *value;
+    const float* projected;
+    int64_t stride;
+    __device__ __forceinline__ int chunk_start(int position) const { return chunk > 0 ? position - position % chunk : 0; }
+    // where (slot, kv head)'s entry of a position begins, in units of one entry
+    __device__ __forceinline__ int64_t entry(int slot, int head, int position) const {
+        return (static_cast<int64_t>(slot) * kv_heads + head) * entries + (position - chunk_start(position));
+    }
+    __device__ __forceinline__ bool fits(int position) const { return position - chunk_start(position) < entries; }
+};
+
+bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
+    if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)
+        || a->rot_dims > a->dim || a->chunk < 0 || a->entries <= 0 || (a->rot_dims > 0 && (!a->cosine || !a->sine)) || !a->q_norm || !a->k_norm
+        || (a->dtype != B200_F32 && a->dtype != B200_BF16) || !a->key_cache || !a->value_cache || !a->projected || !a->query || a->stride <= 0) {
+        set_error("chunked attention: bad pointer or size");
+        return false;
+    }
+    p = ChunkParams{a->heads, a->kv_heads, a->heads / a->kv_heads, a->dim, a->vdim, a->rot_dims, a->chunk, a->entries, a->scale, static_cast<float>(a->eps),
+                    a->cosine, a->sine, a->positions, a->q_norm, a->k_norm, a->key_cache, a->value_cache, a->query, a->key, a->value, a->projected, a->stride};
+    return true;
+}
+
+// ---- between the projection and the attention -----------------------------------------------------------------------
+struct Units { int kind; int64_t column; int count; float* out; __nv_bfloat16 *out_hi, *out_lo; int64_t stride; };
+struct Route { int experts, top; int64_t column; int32_t* chosen; float* weight; int32_t *rank, *counts; };
+
+template <int V> struct Span { float v[V]; };
+template <int V> __device__ __forceinline__ Span<V> load_span(const float* p) {
+    Span<V> r;
+    if constexpr (V == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(p);
+        r.v[0] = q.x; r.v[1] = q.y; r.v[2] = q.z; r.v[3] = q.w;
+    } else {
+        r.v[0] = *p;
+    }
+    return r;
+}
+template <int V> __device__ __forceinline__ void store_span(float* p, const Span<V>& s) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(s.v[0], s.v[1], s.v[2], s.v[3]);
+    else *p = s.v[0];
+}
+template <int V> __device__ __forceinline__ void store_span(__nv_bfloat16* p, const Span<V>& s) {
+    if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(s.v[0], s.v[1]), pack_bf16(s.v[2], s.v[3]));
+    else *p = __float2bfloat16_rn(s.v[0]);
+}
+template <int V> __device__ __forceinline__ float squares_of(const float* x, int count) {
+    float total = 0.0f;
+    for (int c = threadIdx.x * V; c < count; c += blockDim.x * V) {
+        const Span<V> s = load_span<V>(x + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) total = fmaf(s.v[i], s.v[i], total);
+    }
+    return total;
+}
+// V entries of a head from entry d on: normed, weighted, and turned by the row's angles (entry i with entry i + rot_dims / 2).
+template <int V>
+__device__ __forceinline__ Span<V> turned_span(const ChunkParams& p, const float* head, const float* weight, int d, float inverse, const float* cosine,
+                                               const float* sine) {
+    auto normed = [&](int at) {
+        Span<V> s = load_span<V>(head + at);
+        const Span<V> w = load_span<V>(weight + at);
+#pragma unroll
+        for (int i = 0; i < V; ++i) s.v[i] = s.v[i] * inverse * w.v[i];
+        return s;
+    };
+    Span<V> own = normed(d);
+    if (d >= p.rot_dims || !cosine) return own;
+    const int half = p.rot_dims >> 1;
+    const bool upper = d >= half;
+    const Span<V> other = normed(upper ? d - half : d + half);
+    const Span<V> c = load_span<V>(cosine + (upper ? d - half : d)), s = load_span<V>(sine + (upper ? d - half : d));
+#pragma unroll
+    for (int i = 0; i < V; ++i)
+        own.v[i] = upper ? __fadd_rn(__fmul_rn(own.v[i], c.v[i]), __fmul_rn(other.v[i], s.v[i]))
+                         : __fsub_rn(__fmul_rn(own.v[i], c.v[i]), __fmul_rn(other.v[i], s.v[i]));
+    return own;
+}
+
+// The `top` experts with the largest logits (the scores grow with them), the lower index among equals, by one warp.
+__device__ __forceinline__ void choose_experts(const Route& r, int row, const float* logits, float* copy, int lane) {
+    for (int e = lane; e < r.experts; e += 32) copy[e] = logits[e];
+    __syncwarp();
+    for (int k = 0; k < r.top; ++k) {
+        float best = -INFINITY;
+        int at = INT32_MAX;
+        for (int e = lane; e < r.experts; e += 32)
+            if (copy[e] > best || at == INT32_MAX) { best = copy[e]; at = e; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float other = __shfl_xor_sync(0xffffffffu, best, o);
+            const int other_at = __shfl_xor_sync(0xffffffffu, at, o);
+            if (other_at != INT32_MAX && (at == INT32_MAX || other > best || (other == best && other_at < at))) { best = other; at = other_at; }
+        }
+        if (lane == 0) {
+            const int64_t slot = static_cast<int64_t>(row) * r.top + k;
+            r.chosen[slot] = at;
+            r.weight[slot] = 1.0f / (1.0f + expf(-logits[at]));
+            if (r.rank) r.rank[slot] = atomicAdd(r.counts + at, 1);
+            copy[at] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
+constexpr int kPrepareThreads = 256, kUnitSlice = 1024;
+// grid (rows, 1 + slices of the units)
+
+template <class T, int V>
+__global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __grid_constant__ ChunkParams p, const RowsView rows, const bool step,
+                                                                        const __grid_constant__ Units units, const __grid_constant__ Route route) {
+    extern __shared__ float logits_copy[];
+    __shared__ float scratch[32];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row = blockIdx.x;
+    const float* source = p.projected + row * p.stride;
+    if (blockIdx.y > 0) {   // a slice of the row's feed-forward units
+        const float* from = source + units.column;
+        const int begin = (blockIdx.y - 1) * kUnitSlice, end = min(units.count, begin + kUnitSlice);
+        for (int j = begin + threadIdx.x; j < end; j += kPrepareThreads) {
+            const float v = units.kind == 1 ? silu_reference(from[2 * j]) * from[2 * j + 1] : gelu_exact(from[j]);
+            store_forms(v, row * units.stride + j, units.out, units.out_hi, units.out_lo);
+        }
+        return;
+    }
+    if (route.experts > 0 && threadIdx.x >= kPrepareThreads - 32)
+        choose_experts(route, row, source + route.column, logits_copy, threadIdx.x & 31);
+    const RowPlace place = row_place(rows, row);
+    const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
+    const float *k_source = source + q_count, *v_source = k_source + k_count;
+    const float qs = block_sum(squares_of<V>(source, q_count), scratch), ks = block_sum(squares_of<V>(k_source, k_count), scratch);
+    const float q_inverse = 1.0f / sqrtf(qs / static_cast<float>(q_count) + p.eps);
+    const float k_inverse = 1.0f / sqrtf(ks / static_cast<float>(k_count) + p.eps);
+    const int half = p.rot_dims >> 1;
+    const bool turns = half > 0 && place.position < p.positions;
+    const float* cosine = turns ? p.cosine + static_cast<int64_t>(place.position) * half : nullptr;
+    const float* sine = turns ? p.sine + static_cast<int64_t>(place.position) * half : nullptr;
+    for (int c = threadIdx.x * V; c < q_count; c += kPrepareThreads * V) {
+        const int head = c / p.dim, d = c - head * p.dim;
+        store_span<V>(static_cast<T*>(p.query) + static_cast<int64_t>(row) * q_count + c,
+                      turned_span<V>(p, source + head * p.dim, p.q_norm + head * p.dim, d, q_inverse, cosine, sine));
+    }
+    if (!step || p.fits(place.position)) {   // (the host refuses passes that do not fit)
+        for (int c = threadIdx.x * V; c < k_count; c += kPrepareThreads * V) {
+            const int head = c / p.dim, d = c - head * p.dim;
+            T* to = step ? static_cast<T*>(p.key_cache) + p.entry(place.slot, head, place.position) * p.dim + d
+                         : static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + c;
+            store_span<V>(to, turned_span<V>(p, k_source + head * p.dim, p.k_norm + head * p.dim, d, k_inverse, cosine, sine));
+        }
+        for (int c = threadIdx.x * V; c < v_count; c += kPrepareThreads * V) {
+            const int head = c / p.vdim, d = c - head * p.vdim;
+            T* to = step ? static_cast<T*>(p.value_cache) + p.entry(place.slot, head, place.position) * p.vdim + d
+                         : static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + c;
+            store_span<V>(to, load_span<V>(v_source + c));
+        }
+    }
+}
+
+// grid (rows): a row of its sequence's last chunk goes into the slot
+template <class T> __global__ void __launch_bounds__(128) chunk_append_kernel(const __grid_constant__ ChunkParams p, const RowsView rows) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row = blockIdx.x;
+    const RowPlace place = row_place(rows, row);
+    const int last = rows.lengths[place.slot] + __ldg(rows.first + place.sequence + 1) - __ldg(rows.first + place.sequence) - 1;
+    if (p.chunk_start(place.position) != p.chunk_start(last) || !p.fits(place.position)) return;
+    const int k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
+    for (int c = threadIdx.x; c < k_count; c += blockDim.x)
+        static_cast<T*>(p.key_cache)[p.entry(place.slot, c / p.dim, place.position) * p.dim + c % p.dim] =
+            static_cast<const T*>(p.key)[static_cast<int64_t>(row) * k_count + c];
+    for (int c = threadIdx.x; c < v_count; c += blockDim.x)
+        static_cast<T*>(p.value_cache)[p.entry(place.slot, c / p.vdim, place.position) * p.vdim + c % p.vdim] =
+            static_cast<const T*>(p.value)[static_cast<int64_t>(row) * v_count + c];
+}
+
+// ---- attention ------------------------------------------------------------------------------------------------------
+struct ChunkAttention {
+    ChunkParams p;
+    RowsView rows;
+    bool step;                      // every key, the row's own included, is in the slots
+    int positions_per_tile, heads_per_tile, head_tiles, splits;
+    float *partial, *partial_ml;    // splits > 1: [rows, heads, splits, vdim], [rows, heads, splits, 2]
+    float* out;
+    __nv_bfloat16 *out_hi, *out_lo;
+    int64_t out_stride;
+};
+
+__device__ __forceinline__ float head_gate(const ChunkParams& p, int row, int head) {
+    const float g = __ldg(p.projected + row * p.stride + p.heads * p.dim + p.kv_heads * (p.dim + p.vdim) + head);
+    return 1.0f / (1.0f + expf(-g));
+}
+
+// 16-byte piece `chunk` of a tile row of COLUMNS values, swizzled by the row.
+template <int COLUMNS> __device__ __forceinline__ uint32_t tile_offset(int row, int chunk) {
+    return static_cast<uint32_t>(row * COLUMNS * 2 + ((chunk ^ (row & 7)) << 4));
+}
+
+template <int DK, int DV, bool STEP> struct ChunkShape {
+    static constexpr int kWarps = 4, kThreads = kWarps * 32;
+    static constexpr int kRows = STEP ? 16 : 64;
+    static constexpr int kKeys = STEP || DK + DV <= 256 ? 64 : 32;            // keys of a tile
+    static constexpr int kOwnKeys = STEP ? kKeys / kWarps : kKeys;            // keys a warp multiplies
+    static constexpr int kStageBytes = kKeys * (DK + DV) * 2;
+    static constexpr int kStages = STEP ? (DK + DV <= 128 ? 4 : DK + DV <= 320 ? 3 : 2) : 2;
+    static constexpr int kQueryBytes = kRows * DK * 2;
+    static constexpr int kMergeBytes = STEP ? kWarps * kRows * (DV + 2) * 4 : 0;
+    static constexpr int kBody = kStages * kStageBytes > kMergeBytes ? kStages * kStageBytes : kMergeBytes;
+    static constexpr int kSmem = kQueryBytes + kBody;
+};
+
+template <int DK, int DV, bool STEP>
+__global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ ChunkAttention a) {
+    using S = ChunkShape<DK, DV, STEP>;
+    extern __shared__ __align__(128) uint8_t smem[];
+    const ChunkParams& p = a.p;
+    uint8_t* ring = smem + S::kQueryBytes;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int sequence = blockIdx.y, split = blockIdx.z % a.splits, z = blockIdx.z / a.splits;
+    const int head_tile = z % a.head_tiles, kv_head = z / a.head_tiles;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int first = __ldg(a.rows.first + sequence), count = __ldg(a.rows.first + sequence + 1) - first;
+    const int slot = __ldg(a.rows.slot + sequence), length = a.rows.lengths[slot];
+    // the tiles with the most keys start first
+    const int offset = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * a.positions_per_tile;
+    if (offset >= count) return;
+    const int last = min(offset + a.positions_per_tile, count);
+    const int key_begin = p.chunk_start(length + offset), key_end = length + last;   // absolute positions of the tile's keys
+    const int stored_end = STEP ? key_end : length;                                  // keys before it are in the slot
+    const int slot_start = STEP ? key_begin : p.chunk_start(length);                 // position of the slot's entry 0
+    const int tiles = (key_end - key_begin + S::kKeys - 1) / S::kKeys, per_split = (tiles + a.splits - 1) / a.splits;
+    const int tile0 = split * per_split, tile1 = min(tiles, tile0 + per_split);
+
+    // rows of the tile: (position, head of the group)
+    auto row_of = [&](int m, int& position, int& head) {
+        position = offset + m / a.heads_per_tile;
+        const int in_group = head_tile * a.heads_per_tile + m % a.heads_per_tile;
+        head = kv_head * p.group + in_group;
+        return m < a.positions_per_tile * a.heads_per_tile && position < last && in_group < p.group;
+    };
+    {
+        const auto* query = static_cast<const __nv_bfloat16*>(p.query);
+        for (int c = threadIdx.x; c < S::kRows * (DK / 8); c += S::kThreads) {
+            const int m = c / (DK / 8), piece = c % (DK / 8);
+            int position, head;
+            const bool live = row_of(m, position, head) && piece * 8 < p.dim;
+            copy_async_16(smem_u32(smem) + tile_offset<DK>(m, piece),
+                          live ? query + (static_cast<int64_t>(first + position) * p.heads + head) * p.dim + piece * 8 : query, live);
+        }
+    }
+    const auto* key_slot = static_cast<const __nv_bfloat16*>(p.key_cache) + (static_cast<int64_t>(slot) * p.kv_heads + kv_head) * p.entries * p.dim;
+    const auto* value_slot = static_cast<const __nv_bfloat16*>(p.value_cache) + (static_cast<int64_t>(slot) * p.kv_heads + kv_head) * p.entries * p.vdim;
+    const auto* key_rows = static_cast<const __nv_bfloat16*>(p.key);
+    const auto* value_rows = static_cast<const __nv_bfloat16*>(p.value);
+    auto fetch = [&](int tile, int stage) {
+        const int t0 = key_begin + tile * S::kKeys;
+        const uint32_t keys = smem_u32(ring + stage * S::kStageBytes), values = keys + S::kKeys * DK * 2;
+#pragma unroll 4
+        for (int c = threadIdx.x; c < S::kKeys * (DK / 8); c += S::kThreads) {
+            const int n = c / (DK / 8), piece = c % (DK / 8), j = t0 + n;
+            const bool live = j < key_end && piece * 8 < p.dim;
+            const __nv_bfloat16* from = key_slot;
+            if (live) {
+                if (STEP || j < stored_end) from = key_slot + static_cast<int64_t>(j - slot_start) * p.dim + piece * 8;
+                else from = key_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim + piece * 8;
+            }
+            copy_async_16(keys + tile_offset<DK>(n, piece), from, live);
+        }
+#pragma unroll 4
+        for (int c = threadIdx.x; c < S::kKeys * (DV / 8); c += S::kThreads) {
+            const int n = c / (DV / 8), piece = c % (DV / 8), j = t0 + n;
+            const bool live = j < key_end && piece * 8 < p.vdim;
+            const __nv_bfloat16* from = value_slot;
+            if (live) {
+                if (STEP || j < stored_end) from = value_slot + static_cast<int64_t>(j - slot_start) * p.vdim + piece * 8;
+                else from = value_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.vdim + piece * 8;
+            }
+            copy_async_16(values + tile_offset<DV>(n, piece), from, live);
+        }
+    };
+#pragma unroll
+    for (int s = 0; s < S::kStages - 1; ++s) {
+        if (tile0 + s < tile1) fetch(tile0 + s, s);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+
+    const int row_base = STEP ? 0 : warp * 16, key_base = STEP ? warp * S::kOwnKeys : 0;
+    // the two rows of this thread's fragments: which keys they see, [see_from, see_to)
+    int see_from[2], see_to[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        int position, head;
+        const bool live = row_of(row_base + (lane >> 2) + i * 8, position, head);
+        see_from[i] = live ? p.chunk_start(length + position) : 0;
+        see_to[i] = live ? length + position + 1 : 0;
+    }
+    // keys that every live row of this warp sees need no mask
+    const int all_from = warp_max_int(max(see_to[0] ? see_from[0] : 0, see_to[1] ? see_from[1] : 0));
+    const int all_to = -warp_max_int(-min(see_to[0] ? see_to[0] : INT32_MAX, see_to[1] ? see_to[1] : INT32_MAX));
+
+    constexpr int NT = S::kOwnKeys / 8, VT = DV / 8;
+    constexpr bool kHold = DK <= 128;      // query fragments stay in registers
+    uint32_t q[kHold ? DK / 16 : 1][4];
+    float o[VT][4];
+#pragma unroll
+    for (int v = 0; v < VT; ++v)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[v][i] = 0.0f;
+    float top[2] = {-INFINITY, -INFINITY}, total[2] = {0.0f, 0.0f};
+    const float scale2 = p.scale * kLog2e;
+    const uint32_t query_at = smem_u32(smem);
+    const int query_row = row_base + (lane & 15);
+    auto load_query = [&](uint32_t (&f)[4], int k) { ldsm_x4(f, query_at + tile_offset<DK>(query_row, k * 2 + (lane >> 4))); };
+
+    for (int t = tile0; t < tile1; ++t) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(S::kStages - 2) : "memory");
+        __syncthreads();   // the tile is here, and everyone is done with the stage that is filled next
+        if (t + S::kStages - 1 < tile1) fetch(t + S::kStages - 1, (t - tile0 + S::kStages - 1) % S::kStages);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if constexpr (kHold) {
+            if (t == tile0) {
+#pragma unroll
+                for (int k = 0; k < DK / 16; ++k) load_query(q[k], k);
+            }
+        }
+        const uint32_t keys = smem_u32(ring + (t - tile0) % S::kStages * S::kStageBytes), values = keys + S::kKeys * DK * 2;
+        float s[NT][4];
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s[n][i] = 0.0f;
+#pragma unroll
+        for (int k = 0; k < DK / 16; ++k) {
+            if constexpr (!kHold) load_query(q[0], k);
+            const uint32_t (&f)[4] = q[kHold ? k : 0];
+#pragma unroll
+            for (int n = 0; n < NT; n += 2) {
+                uint32_t b[4];
+                ldsm_x4(b, keys + tile_offset<DK>(key_base + n * 8 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)));
+                mma_16816(s[n], f, b[0], b[1]);
+                mma_16816(s[n + 1], f, b[2], b[3]);
+            }
+        }
+        const int t0 = key_begin + t * S::kKeys + key_base;
+        const bool mask = t0 < all_from || t0 + S::kOwnKeys > all_to;
+        float high[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                s[n][i] *= scale2;
+                if (mask) {
+                    const int j = t0 + n * 8 + (lane & 3) * 2 + (i & 1);
+                    if (j < see_from[i >> 1] || j >= see_to[i >> 1]) s[n][i] = -INFINITY;
+                }
+                high[i >> 1] = fmaxf(high[i >> 1], s[n][i]);
+            }
+        float base[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            high[i] = fmaxf(high[i], __shfl_xor_sync(0xffffffffu, high[i], 1));
+            high[i] = fmaxf(high[i], __shfl_xor_sync(0xffffffffu, high[i], 2));
+            const float next = fmaxf(top[i], high[i]);
+            base[i] = next == -INFINITY ? 0.0f : next;
+            const float factor = exp2_fast(top[i] - base[i]);
+            top[i] = next;
+            total[i] *= factor;
+#pragma unroll
+            for (int v = 0; v < VT; ++v) { o[v][2 * i] *= factor; o[v][2 * i + 1] *= factor; }
+        }
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                s[n][i] = exp2_fast(s[n][i] - base[i >> 1]);
+                total[i >> 1] += s[n][i];
+            }
+#pragma unroll
+        for (int k = 0; k < NT / 2; ++k) {
+            uint32_t hi[4], lo[4];
+            pack_planes(s[2 * k][0], s[2 * k][1], hi[0], lo[0]);
+            pack_planes(s[2 * k][2], s[2 * k][3], hi[1], lo[1]);
+            pack_planes(s[2 * k + 1][0], s[2 * k + 1][1], hi[2], lo[2]);
+            pack_planes(s[2 * k + 1][2], s[2 * k + 1][3], hi[3], lo[3]);
+#pragma unroll
+            for (int v = 0; v < VT; v += 2) {
+                uint32_t b[4];
+                ldsm_x4_trans(b, values + tile_offset<DV>(key_base + k * 16 + (lane & 15), v + (lane >> 4)));
+                mma_16816(o[v], hi, b[0], b[1]);
+                mma_16816(o[v + 1], hi, b[2], b[3]);
+                mma_16816(o[v], lo, b[0], b[1]);
+                mma_16816(o[v + 1], lo, b[2], b[3]);
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        total[i] += __shfl_xor_sync(0xffffffffu, total[i], 1);
+        total[i] += __shfl_xor_sync(0xffffffffu, total[i], 2);
+    }
+    auto store = [&](int row, int head, int column, float x, float y) {
+        const int64_t at = row * a.out_stride + head * p.vdim + column;
+        if (a.out) *reinterpret_cast<float2*>(a.out + at) = make_float2(x, y);
+        if (a.out_hi) {
+            uint32_t hi, lo;
+            pack_planes(x, y, hi, lo);
+            *reinterpret_cast<uint32_t*>(a.out_hi + at) = hi;
+            if (a.out_lo) *reinterpret_cast<uint32_t*>(a.out_lo + at) = lo;
+        }
+    };
+    if constexpr (!STEP) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            int position, head;
+            if (!row_of(row_base + (lane >> 2) + i * 8, position, head)) continue;
+            const int row = first + position;
+            const float factor = head_gate(p, row, head) / total[i];
+#pragma unroll
+            for (int v = 0; v < VT; ++v) {
+                const int column = v * 8 + (lane & 3) * 2;
+                if (column < p.vdim) store(row, head, column, o[v][2 * i] * factor, o[v][2 * i + 1] * factor);
+            }
+        }
+    } else {
+        // the warps' shares of the keys meet in shared memory
+        float* merge = reinterpret_cast<float*>(ring);                  // [warps][16][DV]
+        float* merge_ml = merge + S::kWarps * 16 * DV;                  // [warps][16][2]
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int m = (lane >> 2) + i * 8;
+#pragma unroll
+            for (int v = 0; v < VT; ++v)
+                *reinterpret_cast<float2*>(merge + (warp * 16 + m) * DV + v * 8 + (lane & 3) * 2) = make_float2(o[v][2 * i], o[v][2 * i + 1]);
+            if ((lane & 3) == 0) { merge_ml[(warp * 16 + m) * 2] = top[i]; merge_ml[(warp * 16 + m) * 2 + 1] = total[i]; }
+        }
+        __syncthreads();
+        for (int c = threadIdx.x; c < a.heads_per_tile * (DV / 2); c += S::kThreads) {
+            const int m = c / (DV / 2), column = (c % (DV / 2)) * 2;
+            int position, head;
+            if (!row_of(m, position, head) || column >= p.vdim) continue;
+            float best = -INFINITY;
+#pragma unroll
+            for (int w = 0; w < S::kWarps; ++w) best = fmaxf(best, merge_ml[(w * 16 + m) * 2]);
+            const float at = best == -INFINITY ? 0.0f : best;
+            float x = 0.0f, y = 0.0f, sum = 0.0f;
+#pragma unroll
+            for (int w = 0; w < S::kWarps; ++w) {
+                const float factor = exp2_fast(merge_ml[(w * 16 + m) * 2] - at);
+                const float2 v = *reinterpret_cast<const float2*>(merge + (w * 16 + m) * DV + column);
+                x = fmaf(v.x, factor, x);
+                y = fmaf(v.y, factor, y);
+                sum = fmaf(merge_ml[(w * 16 + m) * 2 + 1], factor, sum);
+            }
+            const int row = first + position;
+            if (a.splits == 1) {
+                const float factor = head_gate(p, row, head) / sum;
+                store(row, head, column, x * factor, y * factor);
+            } else {
+                const int64_t part = (static_cast<int64_t>(row) * p.heads + head) * a.splits + split;
+                *reinterpret_cast<float2*>(a.partial + part * p.vdim + column) = make_float2(x, y);
+                if (column == 0) { a.partial_ml[part * 2] = best; a.partial_ml[part * 2 + 1] = sum; }
+            }
+        }
+    }
+}
+
+// One CTA per (head, row): the splits' (max, sum, unscaled accumulator), and the gate.
+__global__ void __launch_bounds__(64) chunk_combine_kernel(const __grid_constant__ ChunkAttention a) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int head = blockIdx.x, row = blockIdx.y;
+    const int64_t at = (static_cast<int64_t>(row) * a.p.heads + head) * a.splits;
+    float best = -INFINITY, total = 0.0f;
+    for (int s = 0; s < a.splits; ++s) best = fmaxf(best, a.partial_ml[(at + s) * 2]);
+    for (int s = 0; s < a.splits; ++s) total = fmaf(a.partial_ml[(at + s) * 2 + 1], exp2_fast(a.partial_ml[(at + s) * 2] - best), total);
+    const float factor = head_gate(a.p, row, head) / total;
+    for (int c = threadIdx.x; c < a.p.vdim; c += blockDim.x) {
+        float v = 0.0f;
+        for (int s = 0; s < a.splits; ++s) v = fmaf(a.partial[(at + s) * a.p.vdim + c], exp2_fast(a.partial_ml[(at + s) * 2] - best), v);
+        store_forms(v * factor, row * a.out_stride + head * a.p.vdim + c, a.out, a.out_hi, a.out_lo);
+    }
+}
+
+constexpr int kGenericThreads = 128, kGenericKeys = 128;
+
+// grid (heads, rows): f32 FMAs over keys of either dtype
+template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_generic_kernel(const __grid_constant__ ChunkAttention a) {
+    extern __shared__ __align__(16) float sm[];   // query [dim], accumulator [vdim], weights [keys], scratch [32]
+    const ChunkParams& p = a.p;
+    float* query = sm;
+    float* acc = query + p.dim;
+    float* w = acc + p.vdim;
+    float* scratch = w + kGenericKeys;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int head = blockIdx.x, row = blockIdx.y, kv_head = head / p.group, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const RowPlace place = row_place(a.rows, row);
+    const int length = a.rows.lengths[place.slot], first = __ldg(a.rows.first + place.sequence);
+    const int begin = p.chunk_start(place.position), end = place.position + 1, stored_end = a.step ? end : length;
+    auto key_at = [&](int j) {
+        return j < stored_end ? static_cast<const T*>(p.key_cache) + p.entry(place.slot, kv_head, j) * p.dim
+                              : static_cast<const T*>(p.key) + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim;
+    };
+    auto value_at = [&](int j) {
+        return j < stored_end ? static_cast<const T*>(p.value_cache) + p.entry(place.slot, kv_head, j) * p.vdim
+                              : static_cast<const T*>(p.value) + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.vdim;
+    };
+    for (int c = threadIdx.x; c < p.dim; c += kGenericThreads)
+        query[c] = load_as_f32(static_cast<const T*>(p.query), (static_cast<int64_t>(row) * p.heads + head) * p.dim + c);
+    for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads) acc[c] = 0.0f;
+    float top = -INFINITY, total = 0.0f;
+    for (int k0 = begin; k0 < end; k0 += kGenericKeys) {
+        const int n = min(kGenericKeys, end - k0);
+        __syncthreads();
+        for (int j = warp; j < n; j += kGenericThreads / 32) {
+            const T* key = key_at(k0 + j);
+            float dot = 0.0f;
+            for (int c = lane; c < p.dim; c += 32) dot = fmaf(query[c], load_as_f32(key, c), dot);
+            dot = warp_sum(dot);
+            if (lane == 0) w[j] = dot * p.scale;
+        }
+        __syncthreads();
+        float high = -INFINITY;
+        for (int j = 0; j < n; ++j) high = fmaxf(high, w[j]);
+        const float next = fmaxf(top, high), factor = expf(top - next);
+        __syncthreads();
+        if (threadIdx.x < n) w[threadIdx.x] = expf(w[threadIdx.x] - next);
+        const float sum = block_sum(threadIdx.x < n ? w[threadIdx.x] : 0.0f, scratch);
+        total = total * factor + sum;
+        top = next;
+        for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads) {
+            float v = acc[c] * factor;
+            for (int j = 0; j < n; ++j) v = fmaf(w[j], load_as_f32(value_at(k0 + j), c), v);
+            acc[c] = v;
+        }
+    }
+    const float scale = head_gate(p, row, head) / total;
+    for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads)
+        store_forms(acc[c] * scale, row * a.out_stride + head * p.vdim + c, a.out, a.out_hi, a.out_lo);
+}
+
+bool chunk_takes_mma(const ChunkParams& p, int dtype, int64_t out_stride) {
+    return dtype == B200_BF16 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.dim <= 256 && p.vdim <= 256 && (out_stride & 1) == 0;
+}
+
+// Splits of a step's keys over CTAs: enough for two CTAs per SM, at least two tiles each.
+int chunk_splits(const ChunkParams& p, int sequences, int max_length, int sms) {
+    const int heads_per_tile = std::min(p.group, 16), items = sequences * p.kv_heads * ((p.group + heads_per_tile - 1) / heads_per_tile);
+    const int keys = std::min(p.entries, max_length), tiles = (keys + 63) / 64;
+    return std::max(1, std::min({(2 * sms + items - 1) / items, tiles / 2, 32}));
+}
+
+template <int DK, int DV, bool STEP> int launch_chunk_mma(const ChunkAttention& a, dim3 grid, cudaStream_t stream) {
+    auto kernel = chunk_mma_kernel<DK, DV, STEP>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkShape<DK, DV, STEP>::kSmem));
+    return cuda_status(launch_dependent(kernel, grid, dim3(128), ChunkShape<DK, DV, STEP>::kSmem, stream, a), "chunk_mma_kernel launch");
+}
+template <bool STEP> int pick_chunk_mma(const ChunkAttention& a, dim3 grid, cudaStream_t stream) {
+    const int d = a.p.dim, e = a.p.vdim;
+    if (d <= 64 && e <= 64) return launch_chunk_mma<64, 64, STEP>(a, grid, stream);
+    if (d <= 64 && e <= 128) return launch_chunk_mma<64, 128, STEP>(a, grid, stream);
+    if (d <= 128 && e <= 64) return launch_chunk_mma<128, 64, STEP>(a, grid, stream);
+    if (d <= 128 && e <= 128) return launch_chunk_mma<128, 128, STEP>(a, grid, stream);
+    if (d <= 192 && e <= 128) return launch_chunk_mma<192, 128, STEP>(a, grid, stream);
+    return launch_chunk_mma<256, 256, STEP>(a, grid, stream);
+}
+
+}  // namespace
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* pass, const b200_units* units, const b200_route* route, void* stream) {
+    ChunkParams p;
+    RowsView rows;
+    if (!chunk_params(args, p) || !rows_view(pass, rows)) return B200_BAD_ARGUMENT;
+    const bool step = rows.max_count == 1;
+    if (!step && (!p.key || !p.value)) { set_error("b200_chunk_prepare: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
+    Units u{};
+    if (units && units->kind) {
+        if (units->kind < 0 || units->kind > 2 || units->column < 0 || units->count < 0 || units->count > INT32_MAX || units->out_stride < units->count
+            || units->column + units->count * (units->kind == 1 ? 2 : 1) > p.stride || (!units->out && !units->out_hi) || (units->out_hi && !units->out_lo)) {
+            set_error("b200_chunk_prepare: inconsistent units");
+            return B200_BAD_ARGUMENT;
+        }
+        u = Units{units->kind, units->column, static_cast<int>(units->count), units->out, static_cast<__nv_bfloat16*>(units->out_hi),
+                  static_cast<__nv_bfloat16*>(units->out_lo), units->out_stride};
+    }
+    Route r{};
+    if (route && route->experts) {
+        if (route->experts < 0 || route->experts > B200_MAX_EXPERTS || route->top <= 0 || route->top > route->experts || route->column < 0
+            || route->column + route->experts > p.stride || !route->chosen || !route->weight || (route->rank && !route->counts)) {
+            set_error("b200_chunk_prepare: inconsistent router");
+            return B200_BAD_ARGUMENT;
+        }
+        r = Route{route->experts, route->top, route->column, route->chosen, route->weight, route->rank, route->counts};
+    }
+    const int q = p.heads * p.dim, k = p.kv_heads * p.dim;
+    auto aligned = [](const void* at) { return (reinterpret_cast<uintptr_t>(at) & 15) == 0; };
+    const bool vector = p.dim % 4 == 0 && p.vdim % 4 == 0 && (p.rot_dims >> 1) % 4 == 0 && p.stride % 4 == 0 && aligned(p.projected) && aligned(p.q_norm)
+        && aligned(p.k_norm) && aligned(p.query) && aligned(p.key) && aligned(p.value) && aligned(p.key_cache) && aligned(p.value_cache)
+        && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0;
+    auto kernel = args->dtype == B200_BF16 ? (vector ? chunk_prepare_kernel<__nv_bfloat16, 4> : chunk_prepare_kernel<__nv_bfloat16, 1>)
+                                           : (vector ? chunk_prepare_kernel<float, 4> : chunk_prepare_kernel<float, 1>);
+    const dim3 grid(static_cast<unsigned>(rows.rows), static_cast<unsigned>(1 + (u.count + kUnitSlice - 1) / kUnitSlice));
+    return cuda_status(launch_dependent(kernel, grid, dim3(kPrepareThreads), static_cast<size_t>(r.experts) * 4,
+                                        as_stream(stream), p, rows, step, u, r), "chunk_prepare_kernel launch");
+}
+
+extern "C" size_t b200_chunk_scratch_bytes(const b200_chunk_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length) {
+    ChunkParams p;
+    if (!chunk_params(args, p) || rows <= 0 || sequences <= 0 || max_count != 1) return 0;
+    int device = 0;
+    if (cudaGetDevice(&device) != cudaSuccess) { cudaGetLastError(); device = -1; }
+    const int splits = chunk_splits(p, sequences, max_length, sm_count(device));
+    return splits > 1 ? static_cast<size_t>(rows) * p.heads * splits * (p.vdim + 2) * sizeof(float) : 0;
+}
+
+extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows* pass, int32_t max_length, void* scratch, size_t scratch_bytes,
+                                    float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream) {
+    ChunkAttention a{};
+    if (!chunk_params(args, a.p) || !rows_view(pass, a.rows)) return B200_BAD_ARGUMENT;
+    const ChunkParams& p = a.p;
+    if ((!out && !out_hi) || (out_hi && !out_lo) || out_stride < static_cast<int64_t>(p.heads) * p.vdim || max_length <= 0) {
+        set_error("b200_chunk_attention: bad pointer or size");
+        return B200_BAD_ARGUMENT;
+    }
+    cudaStream_t s = as_stream(stream);
+    a.step = a.rows.max_count == 1;
+    a.out = out; a.out_hi = static_cast<__nv_bfloat16*>(out_hi); a.out_lo = static_cast<__nv_bfloat16*>(out_lo); a.out_stride = out_stride;
+    a.splits = 1;
+    if (!a.step && (!p.key || !p.value)) { set_error("b200_chunk_attention: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
+    int status = B200_OK;
+    if (chunk_takes_mma(p, args->dtype, out_stride)) {
+        int device = 0;
+        B200_CUDA(cudaGetDevice(&device));
+        const int most = a.step ? 16 : 64;
+        a.heads_per_tile = std::min(p.group, most);
+        a.head_tiles = (p.group + a.heads_per_tile - 1) / a.heads_per_tile;
+        a.positions_per_tile = a.step ? 1 : most / a.heads_per_tile;
+        if (a.step) {
+            a.splits = chunk_splits(p, a.rows.sequences, max_length, sm_count(device));
+            const size_t need = a.splits > 1 ? static_cast<size_t>(a.rows.rows) * p.heads * a.splits * (p.vdim + 2) * sizeof(float) : 0;
+            if (scratch_bytes < need || (need && !scratch)) { set_error("b200_chunk_attention: scratch of %zu bytes, %zu needed", scratch_bytes, need); return B200_BAD_ARGUMENT; }
+            a.partial = static_cast<float*>(scratch);
+            a.partial_ml = a.partial + static_cast<int64_t>(a.rows.rows) * p.heads * a.splits * p.vdim;
+        }
+        const int z = p.kv_heads * a.head_tiles * a.splits;
+        if (a.rows.sequences > 65535 || z > 65535) { set_error("chunked attention: at most 65535 sequences and head tiles in one pass"); return B200_UNSUPPORTED; }
+        const dim3 grid(static_cast<unsigned>((a.rows.max_count + a.positions_per_tile - 1) / a.positions_per_tile), static_cast<unsigned>(a.rows.sequences),
+                        static_cast<unsigned>(z));
+        status = a.step ? pick_chunk_mma<true>(a, grid, s) : pick_chunk_mma<false>(a, grid, s);
+        if (status == B200_OK && a.splits > 1)
+            status = cuda_status(launch_dependent(chunk_combine_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(64), 0, s, a),
+                                 "chunk_combine_kernel launch");
+    } else {
+        if (a.rows.rows > 65535) { set_error("chunked attention: at most 65535 rows in one pass"); return B200_UNSUPPORTED; }
+        const size_t smem = (static_cast<size_t>(p.dim) + p.vdim + kGenericKeys + 32) * sizeof(float);
+        auto kernel = args->dtype == B200_BF16 ? chunk_generic_kernel<__nv_bfloat16> : chunk_generic_kernel<float>;
+        if (smem > 200 * 1024) { set_error("chunked attention: head sizes %d and %d are too large", p.dim, p.vdim); return B200_UNSUPPORTED; }
+        B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+        status = cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(kGenericThreads), smem, s, a),
+                             "chunk_generic_kernel launch");
+    }
+    if (status != B200_OK || a.step) return status;
+    auto append = args->dtype == B200_BF16 ? chunk_append_kernel<__nv_bfloat16> : chunk_append_kernel<float>;
+    return cuda_status(launch_dependent(append, dim3(static_cast<unsigned>(a.rows.rows)), dim3(128), 0, s, p, a.rows), "chunk_append_kernel launch");
+}
+
+extern "C" const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int64_t out_stride) {
+    ChunkParams p;
+    if (!chunk_params(args, p)) return "";
+    return chunk_takes_mma(p, args->dtype, out_stride) ? "chunk_mma_kernel" : "chunk_generic_kernel";
+}

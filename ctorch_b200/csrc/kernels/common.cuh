@@ -60,6 +60,7 @@ __device__ __forceinline__ float warp_max(float v) {
     for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
     return v;
 }
+__device__ __forceinline__ int warp_max_int(int v) { return __reduce_max_sync(0xffffffffu, v); }
 
 // SiLU exactly as the reference states it: v * sigmoid(v), sigmoid through exp(-|v|) in two branches
 // (src/kernels/cpu/pointwise.cpp:31-34,57 of the reference).
@@ -73,6 +74,9 @@ __device__ __forceinline__ float silu_reference(float v) {
 // approximate division (relative error around 1e-6) instead of the IEEE sequence above, a fifth of the instructions.  A row
 // of a SwiGLU epilogue is a dependent chain per lane, so this is what bounds that epilogue's time.
 __device__ __forceinline__ float silu_fast(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
+
+// gelu in its exact form: v * Phi(v)
+__device__ __forceinline__ float gelu_exact(float v) { return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f)); }
 
 // Asks for the 128-byte line at `address` to be brought into L2; nothing waits for it.
 __device__ __forceinline__ void prefetch_l2(const void* address) { asm volatile("prefetch.global.L2 [%0];" ::"l"(address)); }

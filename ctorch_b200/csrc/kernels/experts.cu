@@ -1,0 +1,524 @@
+// Mixture of experts: every slot (row, choice) adds expert(weight * row), expert(x) = down gelu(up x).  The weight multiplies the
+// expert's input, so it joins the row's norm factor in front of the activation.
+//
+//   * streamed: few slots, f32 weights, odd sizes.  expert_up_kernel and expert_down_kernel let every slot stream its expert's rows with
+//     f32 FMAs; the down form adds the choices of a row and the residual itself.
+//   * grouped: the slots are sorted by expert (expert_gather_kernel: planes of the rows copied into order, the list of row tiles
+//     written), then expert_gemm_kernel multiplies tiles of up to 128 slots of ONE expert with its weights on the tensor cores
+//     (persistent CTAs over the list, TMA operand ring, tcgen05, double-buffered accumulator, the row epilogues of the dense kernels);
+//     only the 32-row boxes that hold slots are fetched, so a batch that gives every expert a few rows costs the weight stream.
+//     expert_combine_kernel adds every row's results in the order of its choices: the sum does not depend on the sorting.
+#include "linear_rows.cuh"
+#include "rows.cuh"
+#include "tcgen05.cuh"
+
+#include <algorithm>
+
+namespace b200 {
+namespace {
+
+struct ExpertParams {
+    int experts, top, rows, in, ff;
+    const void *up, *down;
+    const int32_t* chosen;
+    const float* weight;
+    const float* x;
+    const __nv_bfloat16 *x_hi, *x_lo;
+    const float* sumsq_in;
+    int parts_in;
+    float eps;
+    const float* residual;
+    float* y;
+};
+
+bool expert_params(const b200_experts* a, ExpertParams& p) {
+    if (!a || a->experts <= 0 || a->experts > B200_MAX_EXPERTS || a->top <= 0 || a->top > a->experts || a->rows <= 0 || a->in <= 0 || a->ff <= 0
+        || a->rows * a->top > INT32_MAX || a->in > INT32_MAX || a->ff > INT32_MAX || a->experts * std::max(a->in, a->ff) > INT32_MAX
+        || (a->weight_dtype != B200_F32 && a->weight_dtype != B200_BF16) || !a->up || !a->down || !a->chosen || !a->weight
+        || (!a->x && (!a->x_hi || !a->x_lo)) || (a->parts_in > 0 && !a->sumsq_in) || a->parts_in < 0 || !a->residual || !a->y) {
+        set_error("mixture of experts: bad pointer or size");
+        return false;
+    }
+    p = ExpertParams{a->experts, a->top, static_cast<int>(a->rows), static_cast<int>(a->in), static_cast<int>(a->ff), a->up, a->down, a->chosen, a->weight,
+                     a->x, static_cast<const __nv_bfloat16*>(a->x_hi), static_cast<const __nv_bfloat16*>(a->x_lo), a->sumsq_in, a->parts_in,
+                     static_cast<float>(a->eps), a->residual, a->y};
+    return true;
+}
+
+// Factor of a slot's row: the split norm's scale (1 without one) times the router's weight.
+__device__ __forceinline__ float slot_scale(const ExpertParams& p, int slot) {
+    const int row = slot / p.top;
+    float scale = 1.0f;
+    if (p.parts_in > 0) {
+        float total = 0.0f;
+        for (int i = 0; i < p.parts_in; ++i) total += __ldg(p.sumsq_in + static_cast<int64_t>(i) * p.rows + row);
+        scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(total, static_cast<float>(p.in)), p.eps)));
+    }
+    return scale * __ldg(p.weight + slot);
+}
+
+// ---- streamed -------------------------------------------------------------------------------------------------------
+constexpr int kStreamThreads = 256, kFeaturesPerWarp = 4, kFeaturesPerCta = kStreamThreads / 32 * kFeaturesPerWarp;
+
+// Dot products of kFeaturesPerWarp weight rows with a vector in shared memory, by one warp; every lane gets the sums.
+template <class W, bool VECTOR>
+__device__ __forceinline__ void dot_rows(const W* const (&w)[kFeaturesPerWarp], const float* x, int n, int lane, float (&acc)[kFeaturesPerWarp]) {
+    if constexpr (VECTOR) {
+        constexpr int kPer = 16 / sizeof(W);
+#pragma unroll 2
+        for (int k = lane * kPer; k < n; k += 32 * kPer) {
+            float v[kPer];
+#pragma unroll
+            for (int i = 0; i < kPer; i += 4) {
+                const float4 q = *reinterpret_cast<const float4*>(x + k + i);
+                v[i] = q.x; v[i + 1] = q.y; v[i + 2] = q.z; v[i + 3] = q.w;
+            }
+            uint4 raw[kFeaturesPerWarp];
+#pragma unroll
+            for (int f = 0; f < kFeaturesPerWarp; ++f) raw[f] = load_stream_16(w[f] + k);
+#pragma unroll
+            for (int f = 0; f < kFeaturesPerWarp; ++f) {
+                const uint32_t r[4] = {raw[f].x, raw[f].y, raw[f].z, raw[f].w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    if constexpr (sizeof(W) == 2) acc[f] = fmaf(v[2 * i], bf16_lo(r[i]), fmaf(v[2 * i + 1], bf16_hi(r[i]), acc[f]));
+                    else acc[f] = fmaf(v[i], __uint_as_float(r[i]), acc[f]);
+                }
+            }
+        }
+    } else {
+        for (int k = lane; k < n; k += 32)
+#pragma unroll
+            for (int f = 0; f < kFeaturesPerWarp; ++f) acc[f] = fmaf(x[k], load_as_f32(w[f], k), acc[f]);
+    }
+}
+
+// grid (slots, feature blocks): act[slot, f] = gelu(up_f . (scale * row))
+template <class W, bool VECTOR> __global__ void __launch_bounds__(kStreamThreads) expert_up_kernel(const __grid_constant__ ExpertParams p, float* act) {
+    extern __shared__ __align__(16) float x[];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int slot = blockIdx.x, row = slot / p.top, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float scale = slot_scale(p, slot);
+    const int64_t base = static_cast<int64_t>(row) * p.in;
+    for (int c = threadIdx.x; c < p.in; c += kStreamThreads)
+        x[c] = (p.x ? p.x[base + c] : __bfloat162float(p.x_hi[base + c]) + __bfloat162float(p.x_lo[base + c])) * scale;
+    __syncthreads();
+    const int f0 = blockIdx.y * kFeaturesPerCta + warp * kFeaturesPerWarp;
+    if (f0 >= p.ff) return;
+    const int expert = __ldg(p.chosen + slot);
+    const W* w[kFeaturesPerWarp];
+    float acc[kFeaturesPerWarp];
+#pragma unroll
+    for (int f = 0; f < kFeaturesPerWarp; ++f) {
+        w[f] = static_cast<const W*>(p.up) + (static_cast<int64_t>(expert) * p.ff + min(f0 + f, p.ff - 1)) * p.in;
+        acc[f] = 0.0f;
+    }
+    dot_rows<W, VECTOR>(w, x, p.in, lane, acc);
+#pragma unroll
+    for (int f = 0; f < kFeaturesPerWarp; ++f) {
+        const float v = warp_sum(acc[f]);
+        if (lane == f && f0 + f < p.ff) act[static_cast<int64_t>(slot) * p.ff + f0 + f] = gelu_exact(v);
+    }
+}
+
+// grid (rows, feature blocks): y = residual + sum over the choices of down . act
+template <class W, bool VECTOR> __global__ void __launch_bounds__(kStreamThreads) expert_down_kernel(const __grid_constant__ ExpertParams p, const float* act) {
+    extern __shared__ __align__(16) float x[];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int f0 = blockIdx.y * kFeaturesPerCta + warp * kFeaturesPerWarp;
+    float sum[kFeaturesPerWarp];
+#pragma unroll
+    for (int f = 0; f < kFeaturesPerWarp; ++f) sum[f] = 0.0f;
+    for (int k = 0; k < p.top; ++k) {
+        const int slot = row * p.top + k;
+        __syncthreads();
+        for (int c = threadIdx.x; c < p.ff; c += kStreamThreads) x[c] = act[static_cast<int64_t>(slot) * p.ff + c];
+        __syncthreads();
+        const int expert = __ldg(p.chosen + slot);
+        const W* w[kFeaturesPerWarp];
+#pragma unroll
+        for (int f = 0; f < kFeaturesPerWarp; ++f) w[f] = static_cast<const W*>(p.down) + (static_cast<int64_t>(expert) * p.in + min(f0 + f, p.in - 1)) * p.ff;
+        if (f0 < p.in) dot_rows<W, VECTOR>(w, x, p.ff, lane, sum);
+    }
+#pragma unroll
+    for (int f = 0; f < kFeaturesPerWarp; ++f) {
+        const float v = warp_sum(sum[f]);
+        if (lane == f && f0 + f < p.in) {
+            const int64_t at = static_cast<int64_t>(row) * p.in + f0 + f;
+            p.y[at] = p.residual[at] + v;
+        }
+    }
+}
+
+// ---- grouped --------------------------------------------------------------------------------------------------------
+constexpr int kTile = 128;        // slots per row tile; features per weight tile
+constexpr int kBlockK = 64;
+constexpr int kBox = 32;          // slots per activation box
+constexpr int kBoxBytes = kBox * kBlockK * 2;
+constexpr int kPlaneBytes = kTile * kBlockK * 2;
+constexpr int kStages = 3, kStageBytes = 3 * kPlaneBytes;   // x_hi, x_lo, W of one K block
+constexpr int kTileStride = kTile + 4;
+constexpr int kTileBytes = kTile * kTileStride * 4;
+constexpr int kGroupedSmem = kStages * kStageBytes + kTileBytes + 1024 + 2048;
+constexpr int kGroupedThreads = 192;
+
+struct Grouped {
+    __nv_bfloat16 *x_hi, *x_lo;        // [slots, in] in order of their experts
+    __nv_bfloat16 *act_hi, *act_lo;    // [slots, ff]
+    float* y;                          // [slots, in]; shares the memory of x_hi and x_lo, which are read before it is written
+    float* scale;                      // [slots]
+    int32_t* place;                    // [slots] sorted place of slot (row, choice)
+    int4* tiles;                       // (expert, first sorted slot, slots, -)
+    int32_t* tile_count;
+};
+
+size_t round_up_256(size_t n) { return (n + 255) & ~static_cast<size_t>(255); }
+int most_tiles(const ExpertParams& p) {
+    const int slots = p.rows * p.top;
+    return slots / kTile + std::min(p.experts, slots);   // every expert has at most one tile that is not full
+}
+size_t grouped_layout(const ExpertParams& p, uint8_t* base, Grouped& g) {
+    const size_t slots = static_cast<size_t>(p.rows) * p.top;
+    size_t at = 0;
+    auto take = [&](size_t bytes) { uint8_t* here = base + at; at += round_up_256(bytes); return here; };
+    uint8_t* x = take(slots * p.in * 4);
+    g.x_hi = reinterpret_cast<__nv_bfloat16*>(x);
+    g.x_lo = g.x_hi + slots * p.in;
+    g.y = reinterpret_cast<float*>(x);
+    g.act_hi = reinterpret_cast<__nv_bfloat16*>(take(slots * p.ff * 2));
+    g.act_lo = reinterpret_cast<__nv_bfloat16*>(take(slots * p.ff * 2));
+    g.scale = reinterpret_cast<float*>(take(slots * 4));
+    g.place = reinterpret_cast<int32_t*>(take(slots * 4));
+    g.tiles = reinterpret_cast<int4*>(take(static_cast<size_t>(most_tiles(p)) * sizeof(int4)));
+    g.tile_count = reinterpret_cast<int32_t*>(take(4));
+    return at;
+}
+
+// One CTA per slot; CTA 0 also writes the list of row tiles.
+__global__ void __launch_bounds__(256) expert_gather_kernel(const __grid_constant__ ExpertParams p, const __grid_constant__ Grouped g, const int32_t* rank,
+                                                            const int32_t* counts) {
+    extern __shared__ int32_t copy[];   // [experts]
+    __shared__ int32_t before;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int slot = blockIdx.x, expert = __ldg(p.chosen + slot);
+    if (threadIdx.x < 32) {
+        int total = 0;
+        for (int e = threadIdx.x; e < expert; e += 32) total += counts[e];
+        total = __reduce_add_sync(0xffffffffu, total);
+        if (threadIdx.x == 0) before = total;
+    }
+    if (slot == 0)
+        for (int e = threadIdx.x; e < p.experts; e += blockDim.x) copy[e] = counts[e];
+    __syncthreads();
+    const int to = before + rank[slot];
+    const int64_t from_at = static_cast<int64_t>(slot / p.top) * p.in, to_at = static_cast<int64_t>(to) * p.in;
+    for (int c = threadIdx.x * 8; c < p.in; c += blockDim.x * 8) {
+        *reinterpret_cast<uint4*>(g.x_hi + to_at + c) = *reinterpret_cast<const uint4*>(p.x_hi + from_at + c);
+        *reinterpret_cast<uint4*>(g.x_lo + to_at + c) = *reinterpret_cast<const uint4*>(p.x_lo + from_at + c);
+    }
+    if (threadIdx.x == 0) {
+        g.scale[to] = slot_scale(p, slot);
+        g.place[slot] = to;
+    }
+    if (slot == 0) {
+        for (int e = threadIdx.x; e < p.experts; e += blockDim.x) {
+            int tile = 0, row = 0;
+            for (int i = 0; i < e; ++i) { tile += (copy[i] + kTile - 1) / kTile; row += copy[i]; }
+            for (int left = copy[e]; left > 0; left -= kTile, row += kTile) g.tiles[tile++] = make_int4(e, row, min(left, kTile), 0);
+            if (e == p.experts - 1) *g.tile_count = tile;
+        }
+    }
+}
+
+struct ExpertGemm {
+    LinearParams base;          // rows = slots, in, out (features of one expert), results
+    const int4* tiles;
+    const int32_t* tile_count;
+    const float* scale;         // [slots] or NULL
+    int32_t* status;
+};
+
+template <int EPI>
+__global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_constant__ CUtensorMap map_lo,
+                                                                         const __grid_constant__ CUtensorMap map_w, const __grid_constant__ ExpertGemm gp) {
+    const LinearParams& p = gp.base;
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+    float* tile = reinterpret_cast<float*>(smem + kStages * kStageBytes);
+    uint8_t* control = smem + kStages * kStageBytes + kTileBytes;
+    uint64_t* full = reinterpret_cast<uint64_t*>(control);
+    uint64_t* empty = full + kStages;
+    uint64_t* acc_full = empty + kStages;    // [2]
+    uint64_t* acc_empty = acc_full + 2;      // [2]
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
+    volatile int* alive_flag = reinterpret_cast<volatile int*>(control + 256);
+    float* row_scale = reinterpret_cast<float*>(control + 512);
+    constexpr uint32_t kInstruction = mma_instruction_bf16(kTile, kTile);
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int k_blocks = (p.in + kBlockK - 1) / kBlockK;
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < kStages; ++s) {
+            mbar_init(&full[s], 1);
+            mbar_init(&empty[s], 1);
+        }
+        for (int b = 0; b < 2; ++b) {
+            mbar_init(&acc_full[b], 1);
+            mbar_init(&acc_empty[b], 4);
+        }
+        *alive_flag = 1;
+        mbar_fence_init();
+        tma_prefetch_descriptor(&map_hi);
+        tma_prefetch_descriptor(&map_lo);
+        tma_prefetch_descriptor(&map_w);
+    }
+    if (warp == 1) {
+        tmem_alloc(tmem_slot, 2 * kTile);
+        tmem_relinquish();
+    }
+    tc_fence_before_sync();
+    __syncthreads();
+    tc_fence_after_sync();
+    const uint32_t tmem_base = *tmem_slot;
+
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row_tiles = *gp.tile_count, feature_tiles = (p.out + kTile - 1) / kTile, tiles = row_tiles * feature_tiles;
+    const int my_tiles = (tiles - static_cast<int>(blockIdx.x) + static_cast<int>(gridDim.x) - 1) / static_cast<int>(gridDim.x);
+
+    if (warp == 0) {
+        int it = 0;   // K blocks issued so far: the ring does not restart between tiles
+        bool alive = true;
+        for (int j = 0; j < my_tiles && alive; ++j) {
+            const int t = blockIdx.x + j * gridDim.x;
+            const int4 group = __ldg(gp.tiles + t % row_tiles);
+            const int boxes = (group.z + kBox - 1) / kBox, weight_row = group.x * p.out + t / row_tiles * kTile;
+            for (int i = 0; i < k_blocks; ++i, ++it) {
+                const int s = it % kStages;
+                if (!mbar_wait(&empty[s], ((it / kStages) & 1) ^ 1)) {
+                    if (lane == 0) atomicExch(gp.status, B200_DEVICE_TIMEOUT);
+                    alive = false;
+                    break;
+                }
+                if (elect_one()) {
+                    uint8_t* stage = smem + s * kStageBytes;
+                    mbar_expect_tx(&full[s], static_cast<uint32_t>(kPlaneBytes + 2 * boxes * kBoxBytes));
+                    tma_load_2d(stage + 2 * kPlaneBytes, &map_w, i * kBlockK, weight_row, &full[s]);
+                    for (int b = 0; b < boxes; ++b) {
+                        tma_load_2d(stage + b * kBoxBytes, &map_hi, i * kBlockK, group.y + b * kBox, &full[s]);
+                        tma_load_2d(stage + kPlaneBytes + b * kBoxBytes, &map_lo, i * kBlockK, group.y + b * kBox, &full[s]);
+                    }
+                }
+                __syncwarp();
+            }
+        }
+    } else if (warp == 1) {
+        int it = 0;
+        bool alive = true;
+        for (int j = 0; j < my_tiles && alive; ++j) {
+            const int buffer = j & 1;
+            // the epilogue of the tile that used this buffer two tiles ago must have read it (passes at once for j < 2)
+            if (!mbar_wait(&acc_empty[buffer], ((j >> 1) & 1) ^ 1)) {
+                if (lane == 0) atomicExch(gp.status, B200_DEVICE_TIMEOUT);
+                break;
+            }
+            tc_fence_after_sync();
+            const uint32_t accumulator = tmem_base + static_cast<uint32_t>(buffer * kTile);
+            for (int i = 0; i < k_blocks; ++i, ++it) {
+                const int s = it % kStages;
+                if (!mbar_wait(&full[s], (it / kStages) & 1)) {
+                    if (lane == 0) atomicExch(gp.status, B200_DEVICE_TIMEOUT);
+                    alive = false;
+                    break;
+                }
+                tc_fence_after_sync();
+                if (elect_one()) {
+                    const uint32_t stage = smem_u32(smem + s * kStageBytes);
+                    const uint64_t hi = operand_descriptor(stage), lo = operand_descriptor(stage + kPlaneBytes);
+                    const uint64_t w = operand_descriptor(stage + 2 * kPlaneBytes);
+#pragma unroll
+                    for (int k = 0; k < kBlockK / 16; ++k) {
+                        tc_mma_bf16(accumulator, hi + 2 * k, w + 2 * k, kInstruction, (i | k) != 0);
+                        tc_mma_bf16(accumulator, lo + 2 * k, w + 2 * k, kInstruction, 1);
+                    }
+                    tc_commit(&empty[s]);
+                    if (i == k_blocks - 1) tc_commit(&acc_full[buffer]);
+                }
+                __syncwarp();
+            }
+        }
+    } else {
+        // ---- epilogue warps 2-5: TMEM lanes 32 * (warp % 4) .. + 31; named barrier 2 joins the four warps ----
+        const int quarter = warp & 3;
+        const int tile_row = quarter * 32 + lane;
+        const uint32_t own_tile[8] = {smem_u32(tile), 0u, 0u, 0u, 0u, 0u, 0u, 0u};
+        for (int j = 0; j < my_tiles; ++j) {
+            const int t = blockIdx.x + j * gridDim.x;
+            const int4 group = __ldg(gp.tiles + t % row_tiles);
+            const int n0 = t / row_tiles * kTile, buffer = j & 1;
+            row_scale[tile_row] = gp.scale && tile_row < group.z ? __ldg(gp.scale + group.y + tile_row) : 1.0f;
+            const bool ready = mbar_wait_relaxed(&acc_full[buffer], (j >> 1) & 1);
+            if (!ready && lane == 0) { atomicExch(gp.status, B200_DEVICE_TIMEOUT); *alive_flag = 0; }
+            tc_fence_after_sync();
+            if (ready && quarter * 32 < group.z) {   // lanes past the group's slots hold no results
+#pragma unroll 1
+                for (int c = 0; c < kTile / 32; ++c) {
+                    uint32_t r[32];
+                    tmem_load_32(tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + static_cast<uint32_t>(buffer * kTile + c * 32), r);
+                    float4* out4 = reinterpret_cast<float4*>(tile + tile_row * kTileStride + c * 32);
+#pragma unroll
+                    for (int q = 0; q < 8; ++q)
+                        out4[q] = make_float4(__uint_as_float(r[4 * q]), __uint_as_float(r[4 * q + 1]), __uint_as_float(r[4 * q + 2]),
+                                              __uint_as_float(r[4 * q + 3]));
+                }
+            }
+            tc_fence_before_sync();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&acc_empty[buffer]);
+            asm volatile("bar.sync 2, 128;" ::: "memory");    // the tile and the row scales are in shared memory
+            if (*alive_flag == 0) break;                       // same decision in all four warps
+            finish_rows<EPI, kTile>(p, tile, own_tile, 1, row_scale, group.y, n0, t / row_tiles, 0, group.z, quarter, 4, lane, true);
+            asm volatile("bar.sync 2, 128;" ::: "memory");    // the next tile may overwrite the shared-memory tile
+        }
+    }
+    tc_fence_before_sync();
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after_sync();
+        tmem_dealloc(tmem_base, 2 * kTile);
+    }
+}
+
+// One CTA per row: y = residual + the row's results in the order of its choices.
+__global__ void __launch_bounds__(256) expert_combine_kernel(const __grid_constant__ ExpertParams p, const float* results, const int32_t* place) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row = blockIdx.x;
+    const int64_t at = static_cast<int64_t>(row) * p.in;
+    for (int c = threadIdx.x * 4; c < p.in; c += blockDim.x * 4) {
+        float4 sum = *reinterpret_cast<const float4*>(p.residual + at + c);
+        for (int k = 0; k < p.top; ++k) {
+            const float4 v = __ldcs(reinterpret_cast<const float4*>(results + static_cast<int64_t>(__ldg(place + row * p.top + k)) * p.in + c));
+            sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
+        }
+        *reinterpret_cast<float4*>(p.y + at + c) = sum;
+    }
+}
+
+int encode_plane(CUtensorMap* map, const void* base, int64_t rows, int columns, int box_rows) {
+    encode_tiled_fn encode = tensor_map_encoder();
+    if (!encode) { set_error("cuTensorMapEncodeTiled is not available from this driver"); return B200_NO_DEVICE; }
+    const cuuint64_t dims[2] = {static_cast<cuuint64_t>(columns), static_cast<cuuint64_t>(rows)};
+    const cuuint64_t strides[1] = {static_cast<cuuint64_t>(columns) * 2};
+    const cuuint32_t box[2] = {kBlockK, static_cast<cuuint32_t>(box_rows)};
+    const cuuint32_t element_strides[2] = {1, 1};
+    const CUresult result = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, element_strides,
+                                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (result != CUDA_SUCCESS) { set_error("cuTensorMapEncodeTiled(experts) failed with %d", static_cast<int>(result)); return B200_BAD_ARGUMENT; }
+    return B200_OK;
+}
+
+template <int EPI>
+int launch_expert_gemm(const ExpertParams& e, const Grouped& g, const __nv_bfloat16* hi, const __nv_bfloat16* lo, const void* weight, int in, int out,
+                       ExpertGemm gp, int sms, cudaStream_t stream) {
+    alignas(64) CUtensorMap map_hi, map_lo, map_w;
+    const int slots = e.rows * e.top;
+    int status = encode_plane(&map_hi, hi, slots, in, kBox);
+    if (status == B200_OK) status = encode_plane(&map_lo, lo, slots, in, kBox);
+    if (status == B200_OK) status = encode_plane(&map_w, weight, static_cast<int64_t>(e.experts) * out, in, kTile);
+    if (status != B200_OK) return status;
+    gp.base.rows = slots; gp.base.in = in; gp.base.out = out;
+    gp.tiles = g.tiles; gp.tile_count = g.tile_count;
+    auto kernel = expert_gemm_kernel<EPI>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kGroupedSmem));
+    const int64_t bound = static_cast<int64_t>(most_tiles(e)) * ((out + kTile - 1) / kTile);
+    return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(std::min<int64_t>(bound, sms))), dim3(kGroupedThreads), kGroupedSmem, stream, map_hi,
+                                        map_lo, map_w, gp), "expert_gemm_kernel launch");
+}
+
+// Slots up to which every slot streams its expert on its own.
+constexpr int kStreamedSlots = 24;
+
+bool takes_grouped(const b200_experts* a, const ExpertParams& p) {
+    return a->weight_dtype == B200_BF16 && p.x_hi && p.x_lo && p.in % 8 == 0 && p.ff % 8 == 0
+        && ((reinterpret_cast<uintptr_t>(p.x_hi) | reinterpret_cast<uintptr_t>(p.x_lo) | reinterpret_cast<uintptr_t>(p.up) | reinterpret_cast<uintptr_t>(p.down)
+             | reinterpret_cast<uintptr_t>(p.residual) | reinterpret_cast<uintptr_t>(p.y)) & 15) == 0;
+}
+
+}  // namespace
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int32_t b200_experts_takes_grouped(const b200_experts* args) {
+    ExpertParams p;
+    return expert_params(args, p) && takes_grouped(args, p) && p.rows * p.top > kStreamedSlots;
+}
+
+extern "C" size_t b200_experts_grouped_bytes(const b200_experts* args) {
+    ExpertParams p;
+    Grouped g;
+    return expert_params(args, p) ? grouped_layout(p, nullptr, g) : 0;
+}
+
+extern "C" int b200_experts_grouped(const b200_experts* args, const int32_t* rank, const int32_t* counts, void* scratch, size_t scratch_bytes, void* stream) {
+    ExpertParams p;
+    Grouped g;
+    if (!expert_params(args, p)) return B200_BAD_ARGUMENT;
+    if (!rank || !counts || !scratch || (reinterpret_cast<uintptr_t>(scratch) & 255) || scratch_bytes < grouped_layout(p, static_cast<uint8_t*>(scratch), g)) {
+        set_error("b200_experts_grouped: bad workspace");
+        return B200_BAD_ARGUMENT;
+    }
+    if (!takes_grouped(args, p)) { set_error("b200_experts_grouped: needs bf16 planes and widths that are multiples of 8"); return B200_UNSUPPORTED; }
+    int device = 0;
+    B200_CUDA(cudaGetDevice(&device));
+    ExpertGemm gp{};
+    gp.status = device_status_word(device);
+    if (!gp.status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
+    const int sms = sm_count(device), slots = p.rows * p.top;
+    cudaStream_t s = as_stream(stream);
+    int status = cuda_status(launch_dependent(expert_gather_kernel, dim3(static_cast<unsigned>(slots)), dim3(256), static_cast<size_t>(p.experts) * 4, s, p, g, rank,
+                                              counts), "expert_gather_kernel launch");
+    if (status != B200_OK) return status;
+    ExpertGemm up = gp, down = gp;
+    up.scale = g.scale;
+    up.base.out_hi = g.act_hi; up.base.out_lo = g.act_lo;
+    status = launch_expert_gemm<B200_EPI_GELU>(p, g, g.x_hi, g.x_lo, p.up, p.in, p.ff, up, sms, s);
+    if (status != B200_OK) return status;
+    down.base.y = g.y;
+    status = launch_expert_gemm<B200_EPI_STORE>(p, g, g.act_hi, g.act_lo, p.down, p.ff, p.in, down, sms, s);
+    if (status != B200_OK) return status;
+    return cuda_status(launch_dependent(expert_combine_kernel, dim3(static_cast<unsigned>(p.rows)), dim3(256), 0, s, p, static_cast<const float*>(g.y),
+                                        static_cast<const int32_t*>(g.place)), "expert_combine_kernel launch");
+}
+
+extern "C" int b200_experts_streamed(const b200_experts* args, float* act, void* stream) {
+    ExpertParams p;
+    if (!expert_params(args, p) || !act) { if (!act) set_error("b200_experts_streamed: no workspace"); return B200_BAD_ARGUMENT; }
+    const size_t up_smem = (static_cast<size_t>(p.in) * 4 + 15) & ~15ull, down_smem = (static_cast<size_t>(p.ff) * 4 + 15) & ~15ull;
+    const int up_blocks = (p.ff + kFeaturesPerCta - 1) / kFeaturesPerCta, down_blocks = (p.in + kFeaturesPerCta - 1) / kFeaturesPerCta;
+    if (up_smem > 220 * 1024 || down_smem > 220 * 1024 || up_blocks > 65535 || down_blocks > 65535) {
+        set_error("b200_experts_streamed: widths %d and %d are too large", p.in, p.ff);
+        return B200_UNSUPPORTED;
+    }
+    const bool bf16 = args->weight_dtype == B200_BF16;
+    const int per = bf16 ? 8 : 4;
+    const bool vector = p.in % per == 0 && p.ff % per == 0 && ((reinterpret_cast<uintptr_t>(p.up) | reinterpret_cast<uintptr_t>(p.down)) & 15) == 0;
+    auto up = bf16 ? (vector ? expert_up_kernel<__nv_bfloat16, true> : expert_up_kernel<__nv_bfloat16, false>)
+                   : (vector ? expert_up_kernel<float, true> : expert_up_kernel<float, false>);
+    auto down = bf16 ? (vector ? expert_down_kernel<__nv_bfloat16, true> : expert_down_kernel<__nv_bfloat16, false>)
+                     : (vector ? expert_down_kernel<float, true> : expert_down_kernel<float, false>);
+    B200_CUDA(cudaFuncSetAttribute(up, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(up_smem)));
+    B200_CUDA(cudaFuncSetAttribute(down, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(down_smem)));
+    cudaStream_t s = as_stream(stream);
+    const int status = cuda_status(launch_dependent(up, dim3(static_cast<unsigned>(p.rows * p.top), static_cast<unsigned>(up_blocks)), dim3(kStreamThreads), up_smem, s,
+                                                    p, act), "expert_up_kernel launch");
+    if (status != B200_OK) return status;
+    return cuda_status(launch_dependent(down, dim3(static_cast<unsigned>(p.rows), static_cast<unsigned>(down_blocks)), dim3(kStreamThreads), down_smem, s, p,
+                                        static_cast<const float*>(act)), "expert_down_kernel launch");
+}

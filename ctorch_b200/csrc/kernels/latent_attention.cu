@@ -327,7 +327,6 @@ struct LatentAttention {
 
 constexpr int kPage = 64;
 constexpr int kScorePitch = 68, kWeightPitch = 72;
-constexpr float kLog2e = 1.4426950408889634f;
 
 constexpr int kHalf = kLatentBoxRows;         // tokens of one ring stage: half a page
 constexpr int kBoxBytes = kHalf * 64 * 2;    // one box: 32 tokens x 64 values
@@ -345,12 +344,6 @@ template <int MT> struct LatentShape {
 };
 template <int THREADS> __device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
-// 2^v by the hardware unit (relative error about 2^-22; 2^-inf = 0): the weights of the softmax.
-__device__ __forceinline__ float exp2_fast(float v) {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
-    return r;
-}
 // Called by a whole warp.
 __device__ __forceinline__ void latent_copy_half(const CUtensorMap* map, const int32_t* table, int half, uint8_t* stage, int boxes, uint64_t* full) {
     const int row = __ldg(table + (half >> 1)) * kPage + (half & 1) * kHalf;

@@ -35,6 +35,7 @@ struct LinearParams {
     int out_norm_dtype;
     const float* out_norm_bias;        // set: the norm that follows is Dynamic Tanh (f32 weight and bias), which needs no row
     float out_norm_alpha;              //   statistic; the output shadow holds tanh(alpha * row) * weight + bias
+    int64_t out_stride;                // elements between rows of the SwiGLU output shadow
     float* sumsq_out;                  // [tiles][rows] per-tile sums of squares of the (un-weighted) result rows
     // B200_EPI_ARGMAX: per feature tile and row, the preferred value and its feature index
     float* best_value;                 // [tiles][rows]

@@ -65,7 +65,7 @@ __device__ __forceinline__ void finish_pair(const LinearParams& p, int row, int 
     if constexpr (EPI == B200_EPI_SWIGLU) {
         if (p.out_hi) {
             const __nv_bfloat16 hi = __float2bfloat16_rn(a);
-            const int64_t at = static_cast<int64_t>(row) * (p.out >> 1) + (feature0 >> 1);
+            const int64_t at = row * p.out_stride + (feature0 >> 1);
             p.out_hi[at] = hi;
             p.out_lo[at] = __float2bfloat16_rn(a - __bfloat162float(hi));
         }
@@ -95,7 +95,9 @@ __host__ __device__ __forceinline__ bool rows_take_quads(const LinearParams& p) 
               | (p.out_norm_dtype == B200_BF16 ? reinterpret_cast<uintptr_t>(p.out_norm_weight) << 1 : reinterpret_cast<uintptr_t>(p.out_norm_weight));
     }
     if constexpr (EPI == B200_EPI_SWIGLU)
-        bits |= (reinterpret_cast<uintptr_t>(p.y) << 1) | (reinterpret_cast<uintptr_t>(p.out_hi) << 2) | (reinterpret_cast<uintptr_t>(p.out_lo) << 2);
+        bits |= (reinterpret_cast<uintptr_t>(p.y) << 1) | (reinterpret_cast<uintptr_t>(p.out_hi) << 2) | (reinterpret_cast<uintptr_t>(p.out_lo) << 2)
+              | (static_cast<uintptr_t>(p.out_stride) << 3);
+    if constexpr (EPI == B200_EPI_GELU) bits |= (reinterpret_cast<uintptr_t>(p.out_hi) << 1) | (reinterpret_cast<uintptr_t>(p.out_lo) << 1);
     if constexpr (EPI == B200_EPI_QKV) {
         if (p.head_dim & 3) return false;   // a quad never straddles q | k | v or two heads
         bits |= reinterpret_cast<uintptr_t>(p.q_out) | reinterpret_cast<uintptr_t>(p.cosine) << 1 | reinterpret_cast<uintptr_t>(p.sine) << 1
@@ -313,12 +315,29 @@ __device__ __forceinline__ void finish_rows_quads(const LinearParams& p, const f
 #pragma unroll
                 for (int pass = 0; pass < kPasses; ++pass) {
                     if (!live[pass]) continue;
-                    const int64_t at = static_cast<int64_t>(m0 + rows[r]) * (p.out >> 1) + ((n0 + pass * 128 + lane * 4) >> 1);
-                    if (p.y) *reinterpret_cast<float2*>(p.y + at) = result[r][pass];
+                    const int j = (n0 + pass * 128 + lane * 4) >> 1;
+                    if (p.y) *reinterpret_cast<float2*>(p.y + static_cast<int64_t>(m0 + rows[r]) * (p.out >> 1) + j) = result[r][pass];
                     if (p.out_hi) {
+                        const int64_t at = (m0 + rows[r]) * p.out_stride + j;
                         *reinterpret_cast<uint32_t*>(p.out_hi + at) = hi[r][pass];
                         *reinterpret_cast<uint32_t*>(p.out_lo + at) = lo[r][pass];
                     }
+                }
+            }
+        } else if constexpr (EPI == B200_EPI_GELU) {
+#pragma unroll
+            for (int r = 0; r < kBatch; ++r) {
+#pragma unroll
+                for (int pass = 0; pass < kPasses; ++pass) {
+                    if (!live[pass]) continue;
+                    const float4 v = value[r][pass];
+                    const float a = gelu_exact(v.x * scale[r]), b = gelu_exact(v.y * scale[r]), c = gelu_exact(v.z * scale[r]), d = gelu_exact(v.w * scale[r]);
+                    const __nv_bfloat162 hi0 = __floats2bfloat162_rn(a, b), hi1 = __floats2bfloat162_rn(c, d);
+                    const __nv_bfloat162 lo0 = __floats2bfloat162_rn(a - __low2float(hi0), b - __high2float(hi0));
+                    const __nv_bfloat162 lo1 = __floats2bfloat162_rn(c - __low2float(hi1), d - __high2float(hi1));
+                    const int64_t at = static_cast<int64_t>(m0 + rows[r]) * p.out + n0 + pass * 128 + lane * 4;
+                    *reinterpret_cast<uint2*>(p.out_hi + at) = make_uint2(*reinterpret_cast<const uint32_t*>(&hi0), *reinterpret_cast<const uint32_t*>(&hi1));
+                    *reinterpret_cast<uint2*>(p.out_lo + at) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo0), *reinterpret_cast<const uint32_t*>(&lo1));
                 }
             }
         } else if constexpr (EPI == B200_EPI_STORE) {
@@ -505,7 +524,16 @@ __device__ __forceinline__ void finish_rows_pairs(const LinearParams& p, const f
                 const int feature0 = n0 + pass * 64 + lane * 2;
                 if (!ready || feature0 >= p.out) continue;
                 const float a = value[r][pass].x * scale, b = value[r][pass].y * scale;
-                if constexpr (EPI == B200_EPI_ARGMAX) {
+                if constexpr (EPI == B200_EPI_GELU) {
+                    const int64_t at = static_cast<int64_t>(row) * p.out + feature0;
+                    const float ga = gelu_exact(a), gb = gelu_exact(b);
+                    p.out_hi[at] = __float2bfloat16_rn(ga);
+                    p.out_lo[at] = __float2bfloat16_rn(ga - __bfloat162float(__float2bfloat16_rn(ga)));
+                    if (feature0 + 1 < p.out) {
+                        p.out_hi[at + 1] = __float2bfloat16_rn(gb);
+                        p.out_lo[at + 1] = __float2bfloat16_rn(gb - __bfloat162float(__float2bfloat16_rn(gb)));
+                    }
+                } else if constexpr (EPI == B200_EPI_ARGMAX) {
                     const Candidate pair = pair_candidate(feature0, a, b, p.out);
                     if (preferred(pair, best)) best = pair;
                 } else {

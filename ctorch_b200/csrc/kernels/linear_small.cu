@@ -288,6 +288,8 @@ extern "C" int b200_linear_shadow(const b200_shadow_linear_args* args, void* str
     p.sumsq_in = args->sumsq_in; p.parts_in = args->parts_in;
     p.out_hi = static_cast<__nv_bfloat16*>(args->out_hi); p.out_lo = static_cast<__nv_bfloat16*>(args->out_lo);
     p.out_norm_weight = args->out_norm_weight; p.out_norm_dtype = args->out_norm_dtype; p.sumsq_out = args->sumsq_out;
+    p.out_stride = args->out_stride ? args->out_stride : args->out >> 1;
+    if (epilogue == B200_EPI_SWIGLU && p.out_stride < args->out >> 1) { set_error("b200_linear_shadow: rows of the output shadow overlap"); return B200_BAD_ARGUMENT; }
     if (args->out_norm) {
         if (epilogue != B200_EPI_RESIDUAL || !args->out_hi || !args->out_norm->weight || !args->out_norm->bias) {
             set_error("b200_linear_shadow: an elementwise norm needs the residual epilogue, output planes, weight and bias");

@@ -421,7 +421,7 @@ __global__ void __launch_bounds__(kThreads, 2) linear_stream_kernel(const Stream
             if constexpr (SHADOW && EPI == B200_EPI_SWIGLU) {
                 if (p.out_hi && live) {
                     const __nv_bfloat16 hi = __float2bfloat16_rn(a);
-                    const int64_t at = static_cast<int64_t>(row) * (p.out >> 1) + (feature0 >> 1);
+                    const int64_t at = row * p.out_stride + (feature0 >> 1);
                     p.out_hi[at] = hi;
                     p.out_lo[at] = __float2bfloat16_rn(a - __bfloat162float(hi));
                 }

@@ -38,4 +38,13 @@ __device__ __forceinline__ void pack_planes(float a, float b, uint32_t& hi, uint
     lo = pack_bf16(a - __low2float(h), b - __high2float(h));
 }
 
+
+constexpr float kLog2e = 1.4426950408889634f;
+// 2^v by the hardware unit (relative error about 2^-22; 2^-inf = 0): the weights of the softmax.
+__device__ __forceinline__ float exp2_fast(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
+
 }  // namespace b200

@@ -86,11 +86,12 @@ typedef enum b200_epilogue {
     B200_EPI_SWIGLU = 2,    /* weight rows interleaved gate_j, up_j: y[r,j] = silu(gate) * up   (src/nn/decoder.cpp:16) */
     B200_EPI_QKV = 3,       /* fused q|k|v rows: RoPE on q and k, q stored, k and v appended to the KV cache
                                (src/nn/decoder.cpp:80-86) */
-    B200_EPI_ARGMAX = 4     /* shadow linears only: nothing is stored; every feature tile leaves, per row, its best value
+    B200_EPI_ARGMAX = 4,    /* shadow linears only: nothing is stored; every feature tile leaves, per row, its best value
                                and the index of it under the reference's rule (first maximum, first NaN wins:
                                src/kernels/cpu/reduction.cpp:128-151).  b200_argmax_finish merges the tiles.  This is
                                logits + greedy choice without materialising the logits
                                (examples/decoder_generate.cpp:27-30). */
+    B200_EPI_GELU = 5      /* grouped linears only: planes of gelu(acc), the exact (erf) form */
 } b200_epilogue;
 
 /* Extra operands of B200_EPI_QKV. */
@@ -160,6 +161,7 @@ typedef struct b200_shadow_linear_args {
     int32_t copies;                /*   same rows as y - a tensor-parallel rank's slot in each peer's memory (plain peer stores) */
     const b200_elementwise_norm* out_norm; /* residual epilogue: the norm that follows needs no row statistic; the output shadow holds the
                                       normed rows themselves (out_norm_weight and sumsq_out are then unused) */
+    int64_t out_stride;            /* SwiGLU epilogue: elements between rows of the output shadow; 0: out/2 (rows follow each other) */
 } b200_shadow_linear_args;
 /* Up to 16 rows with in <= 2048: streaming kernel (bulk-TMA weight ring, mma.sync).  More rows or a wider input:
  * dense tcgen05 kernel (TMA operand tiles, accumulator in tensor memory; K split over a thread-block cluster when the
@@ -410,6 +412,100 @@ B200_API int b200_latent_value(const b200_latent_args* args, int64_t rows, const
                                float* out, void* out_hi, void* out_lo, void* stream);
 /* Name of the kernel b200_latent_attention runs for these sizes: "latent_mma_kernel" or "latent_generic_kernel". */
 B200_API const char* b200_latent_attention_kernel(const b200_latent_args* args);
+
+/* ---- parallel decoders: chunked attention, mixture of experts ---------------------------------------------------------
+ * (no counterpart in the reference)
+ *
+ * Chunked grouped-query attention: positions, counted from the start of the sequence, fall into chunks of `chunk`; a position
+ * sees its own chunk up to itself.  A slot therefore only keeps the keys and values of the chunk that its next token continues:
+ * key_cache [slots][kv_heads][entries][dim], value_cache [slots][kv_heads][entries][vdim], position p in entry p mod chunk.  A
+ * pass with one row per sequence appends before it attends; longer passes attend to the slot and to their own rows (key and
+ * value workspaces) and leave the sequence's last chunk in the slot afterwards. */
+typedef struct b200_chunk_args {
+    int32_t heads, kv_heads, dim, vdim, rot_dims;
+    int32_t chunk;                 /* positions per chunk; 0: no chunks, every earlier position is seen */
+    int32_t entries;               /* positions a slot holds: chunk, or the capacity where that is smaller or there are no chunks */
+    float scale;
+    double eps;
+    const float* cosine;           /* [positions, rot_dims / 2] */
+    const float* sine;
+    int32_t positions;
+    const float* q_norm;           /* [heads*dim] f32: RMS norm over all query heads at once */
+    const float* k_norm;           /* [kv_heads*dim] f32 */
+    int32_t dtype;                 /* of the caches and workspaces */
+    void* key_cache;
+    void* value_cache;
+    const float* projected;        /* rows [q: heads*dim | k: kv_heads*dim | v: kv_heads*vdim | g: heads | ...], stride floats apart */
+    int64_t stride;
+    void* query;                   /* workspace [rows, heads, dim] */
+    void* key;                     /* workspace [rows, kv_heads, dim]; not used by passes of one row per sequence */
+    void* value;                   /* workspace [rows, kv_heads, vdim] */
+} b200_chunk_args;
+
+/* Activation of feed-forward units that were projected beside the attention's inputs: `kind` 1: silu(gate) * up of `count` interleaved
+ * pairs, 2: exact (erf) gelu of `count` values, starting at column `column` of the projected row.  Result as f32 (out) or planes, out_stride
+ * elements between rows. */
+typedef struct b200_units {
+    int32_t kind;
+    int64_t column, count;
+    float* out;
+    void* out_hi;
+    void* out_lo;
+    int64_t out_stride;
+} b200_units;
+
+/* Router of a mixture of experts: scores sigmoid(logit), the `top` largest are chosen, their scores are the weights.  logits start at
+ * column `column` of the projected row. */
+#define B200_MAX_EXPERTS 1024
+typedef struct b200_route {
+    int32_t experts, top;
+    int64_t column;
+    int32_t* chosen;               /* [rows, top] expert of each slot (row, choice) */
+    float* weight;                 /* [rows, top] */
+    int32_t* rank;                 /* [rows, top] the slot's place among the slots of its expert; NULL: not wanted */
+    int32_t* counts;               /* [experts] slots per expert, zero before the call (with rank) */
+} b200_route;
+
+/* Everything that stands between the projection of a parallel layer and its attention: norms and rotation of queries and keys, append
+ * (or workspaces), the activation of the feed-forward units (units may be NULL) and the router's choice (route may be NULL). */
+B200_API int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* pass, const b200_units* units, const b200_route* route, void* stream);
+/* softmax(scale q.k) v over the visible keys, times sigmoid(g) of the head; out f32 or planes, out_stride elements between rows.
+ * max_length bounds lengths[slot] + rows of any sequence. */
+B200_API size_t b200_chunk_scratch_bytes(const b200_chunk_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length);
+B200_API int b200_chunk_attention(const b200_chunk_args* args, const b200_rows* pass, int32_t max_length, void* scratch, size_t scratch_bytes,
+                                  float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream);
+/* Name of the kernel b200_chunk_attention runs for these sizes: "chunk_mma_kernel" or "chunk_generic_kernel". */
+B200_API const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int64_t out_stride);
+
+/* Experts of one layer: up [experts][ff][in], down [experts][in][ff] (weight dtype), expert(x) = down gelu(up x); slot (row, choice) adds
+ * expert_chosen(weight * row). */
+typedef struct b200_experts {
+    int32_t experts, top;
+    int64_t rows, in, ff;
+    int32_t weight_dtype;
+    const void* up;
+    const void* down;
+    const int32_t* chosen;         /* [rows, top] */
+    const float* weight;           /* [rows, top] */
+    /* the rows: f32, or planes with the partial sums of squares of a split RMS norm (parts_in 0: none) */
+    const float* x;                /* [rows, in] or NULL */
+    const void* x_hi;
+    const void* x_lo;
+    const float* sumsq_in;         /* [parts_in][rows] */
+    int32_t parts_in;
+    double eps;
+    const float* residual;         /* [rows, in] */
+    float* y;                      /* [rows, in] = residual + sum over the choices; may equal residual */
+} b200_experts;
+/* Few slots, f32 weights, odd sizes: every slot streams its expert.  act: workspace f32 [rows, top, ff]. */
+B200_API int b200_experts_streamed(const b200_experts* args, float* act, void* stream);
+/* Many slots (bf16, in and ff multiples of 8, planes): the slots are sorted by expert and multiplied on the tensor cores in tiles of
+ * one expert.  rank and counts come from the router; workspaces of b200_experts_grouped_bytes(...). */
+B200_API size_t b200_experts_grouped_bytes(const b200_experts* args);
+B200_API int b200_experts_grouped(const b200_experts* args, const int32_t* rank, const int32_t* counts, void* scratch, size_t scratch_bytes,
+                                  void* stream);
+/* Whether b200_experts_grouped takes these sizes, and whether it is the faster form. */
+B200_API int32_t b200_experts_takes_grouped(const b200_experts* args);
 
 #ifdef __cplusplus
 }
