@@ -145,6 +145,23 @@ def hybrid_config(width: int, layers: int, ff: int, heads: int, ssm_heads: int, 
     return config
 
 
+def parallel_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, experts: int, top: int = 2, chunk: int = 2048,
+                    loop: tuple[int, int, int] | None = None, vocab: int = 32000) -> dict:
+    """Parallel decoder of a real model's layer sizes: dense and mixture layers in turn; `top` experts and the shared one have the dense
+    feed-forward's active weights (two matrices of width * ff_expert each against three of width * ff)."""
+    expert = 3 * ff // (2 * (top + 1))
+    dim = width // heads
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": chunk}, "rot": {"dims": dim, "base": 500000.0},
+             "scale": dim ** -0.5}
+    mlps = ({"kind": "dense", "ff": ff},
+            {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert}, "shared": {"ff": expert}})
+    config = {"architecture": "Sinezen", "vocab": vocab, "width": width,
+              "layers": [{"type": "attention", "mixer": mixer, "mlp": mlps[i % 2]} for i in range(layers)], "norm": {"eps": 1e-5}}
+    if loop:
+        config["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return config
+
+
 def transformer_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, context: int, vocab: int = 32000) -> dict:
     return {"architecture": "TransformerDecoder", "vocab": vocab, "layers": layers, "width": width, "heads": heads, "kv_heads": kv_heads,
             "ff": ff, "context": context, "tied": 1}
@@ -155,6 +172,13 @@ HYBRID_SIZES = {
     "1k": (dict(width=1024, layers=12, ff=4096, heads=8, ssm_heads=32), dict(width=1024, layers=12, ff=4096, heads=16, kv_heads=4)),
     "2k": (dict(width=2048, layers=12, ff=8192, heads=16, ssm_heads=64, loop=(4, 8, 2)), dict(width=2048, layers=16, ff=8192, heads=32, kv_heads=8)),
     "4k": (dict(width=4096, layers=8, ff=14336, heads=32, ssm_heads=128), dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8)),
+}
+
+# (parallel, grouped-query) arguments, likewise
+PARALLEL_SIZES = {
+    "1k": (dict(width=1024, layers=12, ff=4096, heads=16, kv_heads=4, experts=16), HYBRID_SIZES["1k"][1]),
+    "2k": (dict(width=2048, layers=12, ff=8192, heads=32, kv_heads=8, experts=16, loop=(4, 8, 2)), HYBRID_SIZES["2k"][1]),
+    "4k": (dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8, experts=8), HYBRID_SIZES["4k"][1]),
 }
 
 
