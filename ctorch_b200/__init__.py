@@ -77,7 +77,7 @@ class LatentArgs(C.Structure):
 
 
 class ChunkArgs(C.Structure):
-    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("rot_dims", C.c_int32), ("chunk", C.c_int32),
+    _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("rot_dims", C.c_int32), ("slots", C.c_int32), ("chunk", C.c_int32),
                 ("entries", C.c_int32), ("scale", C.c_float), ("eps", C.c_double), ("cosine", C.c_void_p), ("sine", C.c_void_p), ("positions", C.c_int32),
                 ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("dtype", C.c_int32), ("key_cache", C.c_void_p), ("value_cache", C.c_void_p),
                 ("projected", C.c_void_p), ("stride", C.c_int64), ("query", C.c_void_p), ("key", C.c_void_p), ("value", C.c_void_p)]
@@ -239,7 +239,7 @@ def _declare(l: C.CDLL) -> None:
         "b200_chunk_prepare": (C.c_int, [C.POINTER(ChunkArgs), C.POINTER(Rows), C.POINTER(Units), C.POINTER(Route), vp]),
         "b200_chunk_scratch_bytes": (sz, [C.POINTER(ChunkArgs), i64, i32, i32, i32]),
         "b200_chunk_attention": (C.c_int, [C.POINTER(ChunkArgs), C.POINTER(Rows), i32, vp, sz, vp, vp, vp, i64, vp]),
-        "b200_chunk_attention_kernel": (C.c_char_p, [C.POINTER(ChunkArgs), i64]),
+        "b200_chunk_attention_kernel": (C.c_char_p, [C.POINTER(ChunkArgs), i32, i64]),
         "b200_experts_streamed": (C.c_int, [C.POINTER(Experts), vp, vp]),
         "b200_experts_grouped_bytes": (sz, [C.POINTER(Experts)]),
         "b200_experts_grouped": (C.c_int, [C.POINTER(Experts), vp, vp, vp, sz, vp]),

@@ -102,6 +102,7 @@ b200_chunk_args HybridPlan::chunk_args(const Layer& layer, const ChunkedAttentio
     b200_chunk_args a{};
     a.heads = static_cast<int32_t>(c.heads); a.kv_heads = static_cast<int32_t>(c.kv_heads); a.dim = static_cast<int32_t>(c.dim);
     a.vdim = static_cast<int32_t>(c.vdim); a.rot_dims = static_cast<int32_t>(c.rot_dims);
+    a.slots = static_cast<int32_t>(cache.slots());
     // (no position reaches a chunk that is longer than the cache)
     a.chunk = static_cast<int32_t>(c.chunk > cache.capacity() ? 0 : c.chunk); a.entries = static_cast<int32_t>(r.entries);
     a.scale = static_cast<float>(c.scale); a.eps = owner_.eps();

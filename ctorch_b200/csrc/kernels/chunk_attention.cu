@@ -4,24 +4,28 @@
 //
 //   * chunk_prepare_kernel, one CTA per row (and one per slice of its feed-forward units): RMS norms over all query and all key heads, rotation of halves, append (or the
 //     workspaces of a longer pass), the activation of feed-forward units and the router's choice for the same row.
-//   * chunk_mma_kernel: bf16, tiles of keys and values through a cp.async ring with swizzled rows, mma.sync products, online softmax
-//     in f32 registers, weights as hi + lo planes, the heads of a group side by side so that a key is fetched once for all of them.
-//       steps (one row per sequence): 16 rows = heads of one token; the warps divide the keys of a tile and merge at the end; keys are
-//         split over CTAs, with a merge kernel, where the (sequence, kv head) pairs do not fill the SMs;
-//       longer passes: 64 rows = positions x heads of a group, 16 per warp; keys before the pass come from the slot, the pass's own
-//         keys from its workspaces.
+//   * chunk_step_kernel, chunk_mma_kernel: bf16, mma.sync products, online softmax in f32 registers, weights as hi + lo planes, the heads
+//     of a group side by side so that a key is fetched once for all of them.
+//       steps (one row per sequence): bound by the keys' bytes.  Persistent CTAs walk (sequence, kv head, split) items; a producer warp
+//         streams tiles of 64 keys and values through a TMA ring (boxes of 64 x 64, 128-byte swizzle, mbarrier completion) and runs
+//         into the next item while four consumer warps, which divide the keys of a tile, merge the current one.  Keys are split over
+//         CTAs, with a merge kernel, where the items do not fill the SMs;
+//       longer passes: 64 rows = positions x heads of a group, 16 per warp, a cp.async double buffer; keys before the pass come from the
+//         slot, the pass's own keys from its workspaces.
 //   * chunk_generic_kernel: f32 and odd sizes, f32 FMAs, one (row, head) per CTA.
-//   * chunk_append_kernel: after a longer pass, the rows of every sequence's last chunk go into its slot.
+//   * chunk_append_kernel: a longer pass that begins inside a chunk and ends in another one reads the old chunk from the slot; its last
+//     rows go there afterwards.
 #include "mma.cuh"
 #include "rows.cuh"
 
 #include <algorithm>
+#include <type_traits>
 
 namespace b200 {
 namespace {
 
 struct ChunkParams {
-    int heads, kv_heads, group, dim, vdim, rot_dims, chunk, entries;
+    int heads, kv_heads, group, dim, vdim, rot_dims, slots, chunk, entries;
     float scale, eps;
     const float *cosine, *sine;
     int positions;
@@ -34,17 +38,19 @@ struct ChunkParams {
     __device__ __forceinline__ int64_t entry(int slot, int head, int position) const {
         return (static_cast<int64_t>(slot) * kv_heads + head) * entries + (position - chunk_start(position));
     }
+    // Whether storing the chunk of position `last` overwrites keys that positions from `length` on still see.
+    __device__ __forceinline__ bool overwrites(int length, int last) const { return chunk > 0 && length % chunk != 0 && chunk_start(length) != chunk_start(last); }
     __device__ __forceinline__ bool fits(int position) const { return position - chunk_start(position) < entries; }
 };
 
 bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
     if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)
-        || a->rot_dims > a->dim || a->chunk < 0 || a->entries <= 0 || (a->rot_dims > 0 && (!a->cosine || !a->sine)) || !a->q_norm || !a->k_norm
+        || a->rot_dims > a->dim || a->slots <= 0 || a->chunk < 0 || a->entries <= 0 || (a->rot_dims > 0 && (!a->cosine || !a->sine)) || !a->q_norm || !a->k_norm
         || (a->dtype != B200_F32 && a->dtype != B200_BF16) || !a->key_cache || !a->value_cache || !a->projected || !a->query || a->stride <= 0) {
         set_error("chunked attention: bad pointer or size");
         return false;
     }
-    p = ChunkParams{a->heads, a->kv_heads, a->heads / a->kv_heads, a->dim, a->vdim, a->rot_dims, a->chunk, a->entries, a->scale, static_cast<float>(a->eps),
+    p = ChunkParams{a->heads, a->kv_heads, a->heads / a->kv_heads, a->dim, a->vdim, a->rot_dims, a->slots, a->chunk, a->entries, a->scale, static_cast<float>(a->eps),
                     a->cosine, a->sine, a->positions, a->q_norm, a->k_norm, a->key_cache, a->value_cache, a->query, a->key, a->value, a->projected, a->stride};
     return true;
 }
@@ -146,67 +152,109 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
     if (blockIdx.y > 0) {   // a slice of the row's feed-forward units
         const float* from = source + units.column;
         const int begin = (blockIdx.y - 1) * kUnitSlice, end = min(units.count, begin + kUnitSlice);
-        for (int j = begin + threadIdx.x; j < end; j += kPrepareThreads) {
-            const float v = units.kind == 1 ? silu_reference(from[2 * j]) * from[2 * j + 1] : gelu_exact(from[j]);
-            store_forms(v, row * units.stride + j, units.out, units.out_hi, units.out_lo);
+        auto store = [&](int j, const Span<V>& v) {
+            const int64_t at = row * units.stride + j;
+            if (units.out) store_span<V>(units.out + at, v);
+            if (units.out_hi) {
+                Span<V> rest;
+#pragma unroll
+                for (int i = 0; i < V; ++i) rest.v[i] = v.v[i] - __bfloat162float(__float2bfloat16_rn(v.v[i]));
+                store_span<V>(units.out_hi + at, v);
+                store_span<V>(units.out_lo + at, rest);
+            }
+        };
+        for (int j = begin + threadIdx.x * V; j < end; j += kPrepareThreads * V) {
+            Span<V> v;
+            if (units.kind == 1) {
+                float pairs[2 * V];
+#pragma unroll
+                for (int i = 0; i < 2 * V; i += V) {
+                    const Span<V> part = load_span<V>(from + 2 * j + i);
+#pragma unroll
+                    for (int e = 0; e < V; ++e) pairs[i + e] = part.v[e];
+                }
+#pragma unroll
+                for (int i = 0; i < V; ++i) v.v[i] = silu_reference(pairs[2 * i]) * pairs[2 * i + 1];
+            } else {
+                v = load_span<V>(from + j);
+#pragma unroll
+                for (int i = 0; i < V; ++i) v.v[i] = gelu_exact(v.v[i]);
+            }
+            store(j, v);
         }
         return;
     }
     if (route.experts > 0 && threadIdx.x >= kPrepareThreads - 32)
         choose_experts(route, row, source + route.column, logits_copy, threadIdx.x & 31);
-    const RowPlace place = row_place(rows, row);
+    // where the row belongs: a chain of dependent loads, spread between the sums
+    const int sequence = __ldg(rows.sequence + row);
     const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
     const float *k_source = source + q_count, *v_source = k_source + k_count;
-    const float qs = block_sum(squares_of<V>(source, q_count), scratch), ks = block_sum(squares_of<V>(k_source, k_count), scratch);
+    float qs = squares_of<V>(source, q_count), ks = squares_of<V>(k_source, k_count);
+    const int slot = __ldg(rows.slot + sequence), first = __ldg(rows.first + sequence), end = __ldg(rows.first + sequence + 1);
+    qs = warp_sum(qs);
+    ks = warp_sum(ks);
+    const int length = rows.lengths[slot];
+    if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = qs; scratch[kPrepareThreads / 32 + (threadIdx.x >> 5)] = ks; }
+    __syncthreads();
+    qs = ks = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kPrepareThreads / 32; ++w) { qs += scratch[w]; ks += scratch[kPrepareThreads / 32 + w]; }
+    const int position = length + row - first, last = length + end - first - 1;
+    // The slot takes the row at once where it ends up there and nothing that this pass still reads is overwritten.
+    const bool stored = step || (p.chunk_start(position) == p.chunk_start(last) && !p.overwrites(length, last));
     const float q_inverse = 1.0f / sqrtf(qs / static_cast<float>(q_count) + p.eps);
     const float k_inverse = 1.0f / sqrtf(ks / static_cast<float>(k_count) + p.eps);
     const int half = p.rot_dims >> 1;
-    const bool turns = half > 0 && place.position < p.positions;
-    const float* cosine = turns ? p.cosine + static_cast<int64_t>(place.position) * half : nullptr;
-    const float* sine = turns ? p.sine + static_cast<int64_t>(place.position) * half : nullptr;
+    const bool turns = half > 0 && position < p.positions;
+    const float* cosine = turns ? p.cosine + static_cast<int64_t>(position) * half : nullptr;
+    const float* sine = turns ? p.sine + static_cast<int64_t>(position) * half : nullptr;
     for (int c = threadIdx.x * V; c < q_count; c += kPrepareThreads * V) {
         const int head = c / p.dim, d = c - head * p.dim;
         store_span<V>(static_cast<T*>(p.query) + static_cast<int64_t>(row) * q_count + c,
                       turned_span<V>(p, source + head * p.dim, p.q_norm + head * p.dim, d, q_inverse, cosine, sine));
     }
-    if (!step || p.fits(place.position)) {   // (the host refuses passes that do not fit)
-        for (int c = threadIdx.x * V; c < k_count; c += kPrepareThreads * V) {
-            const int head = c / p.dim, d = c - head * p.dim;
-            T* to = step ? static_cast<T*>(p.key_cache) + p.entry(place.slot, head, place.position) * p.dim + d
-                         : static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + c;
-            store_span<V>(to, turned_span<V>(p, k_source + head * p.dim, p.k_norm + head * p.dim, d, k_inverse, cosine, sine));
-        }
-        for (int c = threadIdx.x * V; c < v_count; c += kPrepareThreads * V) {
-            const int head = c / p.vdim, d = c - head * p.vdim;
-            T* to = step ? static_cast<T*>(p.value_cache) + p.entry(place.slot, head, place.position) * p.vdim + d
-                         : static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + c;
-            store_span<V>(to, load_span<V>(v_source + c));
-        }
+    const bool to_slot = stored && p.fits(position);   // (the host refuses passes that do not fit)
+    for (int c = threadIdx.x * V; c < k_count; c += kPrepareThreads * V) {
+        const int head = c / p.dim, d = c - head * p.dim;
+        const Span<V> v = turned_span<V>(p, k_source + head * p.dim, p.k_norm + head * p.dim, d, k_inverse, cosine, sine);
+        if (to_slot) store_span<V>(static_cast<T*>(p.key_cache) + p.entry(slot, head, position) * p.dim + d, v);
+        if (!step) store_span<V>(static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + c, v);
+    }
+    for (int c = threadIdx.x * V; c < v_count; c += kPrepareThreads * V) {
+        const int head = c / p.vdim, d = c - head * p.vdim;
+        const Span<V> v = load_span<V>(v_source + c);
+        if (to_slot) store_span<V>(static_cast<T*>(p.value_cache) + p.entry(slot, head, position) * p.vdim + d, v);
+        if (!step) store_span<V>(static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + c, v);
     }
 }
 
-// grid (rows): a row of its sequence's last chunk goes into the slot
+// After a longer pass: the rows of a sequence's last chunk go into its slot, where they could not before (see chunk_prepare_kernel).
 template <class T> __global__ void __launch_bounds__(128) chunk_append_kernel(const __grid_constant__ ChunkParams p, const RowsView rows) {
     grid_dependency_wait();
     grid_launch_dependents();
-    const int row = blockIdx.x;
-    const RowPlace place = row_place(rows, row);
-    const int last = rows.lengths[place.slot] + __ldg(rows.first + place.sequence + 1) - __ldg(rows.first + place.sequence) - 1;
-    if (p.chunk_start(place.position) != p.chunk_start(last) || !p.fits(place.position)) return;
-    const int k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
-    for (int c = threadIdx.x; c < k_count; c += blockDim.x)
-        static_cast<T*>(p.key_cache)[p.entry(place.slot, c / p.dim, place.position) * p.dim + c % p.dim] =
-            static_cast<const T*>(p.key)[static_cast<int64_t>(row) * k_count + c];
-    for (int c = threadIdx.x; c < v_count; c += blockDim.x)
-        static_cast<T*>(p.value_cache)[p.entry(place.slot, c / p.vdim, place.position) * p.vdim + c % p.vdim] =
-            static_cast<const T*>(p.value)[static_cast<int64_t>(row) * v_count + c];
+    for (int row = blockIdx.x; row < rows.rows; row += gridDim.x) {
+        const RowPlace place = row_place(rows, row);
+        const int length = rows.lengths[place.slot];
+        const int last = length + __ldg(rows.first + place.sequence + 1) - __ldg(rows.first + place.sequence) - 1;
+        if (!p.overwrites(length, last) || p.chunk_start(place.position) != p.chunk_start(last) || !p.fits(place.position)) continue;
+        const int k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
+        for (int c = threadIdx.x; c < k_count; c += blockDim.x)
+            static_cast<T*>(p.key_cache)[p.entry(place.slot, c / p.dim, place.position) * p.dim + c % p.dim] =
+                static_cast<const T*>(p.key)[static_cast<int64_t>(row) * k_count + c];
+        for (int c = threadIdx.x; c < v_count; c += blockDim.x)
+            static_cast<T*>(p.value_cache)[p.entry(place.slot, c / p.vdim, place.position) * p.vdim + c % p.vdim] =
+                static_cast<const T*>(p.value)[static_cast<int64_t>(row) * v_count + c];
+    }
 }
 
 // ---- attention ------------------------------------------------------------------------------------------------------
 struct ChunkAttention {
     ChunkParams p;
     RowsView rows;
-    bool step;                      // every key, the row's own included, is in the slots
+    bool step;                      // one row per sequence: every key, the row's own included, is in the slots
+    int stages;
+    int32_t* status;
     int positions_per_tile, heads_per_tile, head_tiles, splits;
     float *partial, *partial_ml;    // splits > 1: [rows, heads, splits, vdim], [rows, heads, splits, 2]
     float* out;
@@ -219,33 +267,39 @@ __device__ __forceinline__ float head_gate(const ChunkParams& p, int row, int he
     return 1.0f / (1.0f + expf(-g));
 }
 
+__device__ __forceinline__ void store_pair(const ChunkAttention& a, int row, int head, int column, float x, float y) {
+    const int64_t at = row * a.out_stride + head * a.p.vdim + column;
+    if (a.out) *reinterpret_cast<float2*>(a.out + at) = make_float2(x, y);
+    if (a.out_hi) {
+        uint32_t hi, lo;
+        pack_planes(x, y, hi, lo);
+        *reinterpret_cast<uint32_t*>(a.out_hi + at) = hi;
+        if (a.out_lo) *reinterpret_cast<uint32_t*>(a.out_lo + at) = lo;
+    }
+}
+
 // 16-byte piece `chunk` of a tile row of COLUMNS values, swizzled by the row.
 template <int COLUMNS> __device__ __forceinline__ uint32_t tile_offset(int row, int chunk) {
     return static_cast<uint32_t>(row * COLUMNS * 2 + ((chunk ^ (row & 7)) << 4));
 }
 
-template <int DK, int DV, bool STEP> struct ChunkShape {
+template <int DK, int DV> struct ChunkShape {
     static constexpr int kWarps = 4, kThreads = kWarps * 32;
-    static constexpr int kRows = STEP ? 16 : 64;
-    static constexpr int kKeys = STEP || DK + DV <= 256 ? 64 : 32;            // keys of a tile
-    static constexpr int kOwnKeys = STEP ? kKeys / kWarps : kKeys;            // keys a warp multiplies
+    static constexpr int kRows = 64;
+    static constexpr int kKeys = DK + DV <= 256 ? 64 : 32;   // keys of a tile
     static constexpr int kStageBytes = kKeys * (DK + DV) * 2;
-    static constexpr int kStages = STEP ? (DK + DV <= 128 ? 4 : DK + DV <= 320 ? 3 : 2) : 2;
     static constexpr int kQueryBytes = kRows * DK * 2;
-    static constexpr int kMergeBytes = STEP ? kWarps * kRows * (DV + 2) * 4 : 0;
-    static constexpr int kBody = kStages * kStageBytes > kMergeBytes ? kStages * kStageBytes : kMergeBytes;
-    static constexpr int kSmem = kQueryBytes + kBody;
+    static constexpr int kSmem = kQueryBytes + 2 * kStageBytes;
 };
 
-template <int DK, int DV, bool STEP>
+template <int DK, int DV>
 __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ ChunkAttention a) {
-    using S = ChunkShape<DK, DV, STEP>;
+    using S = ChunkShape<DK, DV>;
     extern __shared__ __align__(128) uint8_t smem[];
     const ChunkParams& p = a.p;
     uint8_t* ring = smem + S::kQueryBytes;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int sequence = blockIdx.y, split = blockIdx.z % a.splits, z = blockIdx.z / a.splits;
-    const int head_tile = z % a.head_tiles, kv_head = z / a.head_tiles;
+    const int sequence = blockIdx.y, head_tile = blockIdx.z % a.head_tiles, kv_head = blockIdx.z / a.head_tiles;
     grid_dependency_wait();
     grid_launch_dependents();
     const int first = __ldg(a.rows.first + sequence), count = __ldg(a.rows.first + sequence + 1) - first;
@@ -255,10 +309,8 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     if (offset >= count) return;
     const int last = min(offset + a.positions_per_tile, count);
     const int key_begin = p.chunk_start(length + offset), key_end = length + last;   // absolute positions of the tile's keys
-    const int stored_end = STEP ? key_end : length;                                  // keys before it are in the slot
-    const int slot_start = STEP ? key_begin : p.chunk_start(length);                 // position of the slot's entry 0
-    const int tiles = (key_end - key_begin + S::kKeys - 1) / S::kKeys, per_split = (tiles + a.splits - 1) / a.splits;
-    const int tile0 = split * per_split, tile1 = min(tiles, tile0 + per_split);
+    const int slot_start = p.chunk_start(length);                                    // position of the slot's entry 0
+    const int tiles = (key_end - key_begin + S::kKeys - 1) / S::kKeys;
 
     // rows of the tile: (position, head of the group)
     auto row_of = [&](int m, int& position, int& head) {
@@ -290,7 +342,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
             const bool live = j < key_end && piece * 8 < p.dim;
             const __nv_bfloat16* from = key_slot;
             if (live) {
-                if (STEP || j < stored_end) from = key_slot + static_cast<int64_t>(j - slot_start) * p.dim + piece * 8;
+                if (j < length) from = key_slot + static_cast<int64_t>(j - slot_start) * p.dim + piece * 8;
                 else from = key_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim + piece * 8;
             }
             copy_async_16(keys + tile_offset<DK>(n, piece), from, live);
@@ -301,19 +353,16 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
             const bool live = j < key_end && piece * 8 < p.vdim;
             const __nv_bfloat16* from = value_slot;
             if (live) {
-                if (STEP || j < stored_end) from = value_slot + static_cast<int64_t>(j - slot_start) * p.vdim + piece * 8;
+                if (j < length) from = value_slot + static_cast<int64_t>(j - slot_start) * p.vdim + piece * 8;
                 else from = value_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.vdim + piece * 8;
             }
             copy_async_16(values + tile_offset<DV>(n, piece), from, live);
         }
     };
-#pragma unroll
-    for (int s = 0; s < S::kStages - 1; ++s) {
-        if (tile0 + s < tile1) fetch(tile0 + s, s);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    }
+    fetch(0, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
 
-    const int row_base = STEP ? 0 : warp * 16, key_base = STEP ? warp * S::kOwnKeys : 0;
+    const int row_base = warp * 16;
     // the two rows of this thread's fragments: which keys they see, [see_from, see_to)
     int see_from[2], see_to[2];
 #pragma unroll
@@ -327,7 +376,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     const int all_from = warp_max_int(max(see_to[0] ? see_from[0] : 0, see_to[1] ? see_from[1] : 0));
     const int all_to = -warp_max_int(-min(see_to[0] ? see_to[0] : INT32_MAX, see_to[1] ? see_to[1] : INT32_MAX));
 
-    constexpr int NT = S::kOwnKeys / 8, VT = DV / 8;
+    constexpr int NT = S::kKeys / 8, VT = DV / 8;
     constexpr bool kHold = DK <= 128;      // query fragments stay in registers
     uint32_t q[kHold ? DK / 16 : 1][4];
     float o[VT][4];
@@ -341,18 +390,18 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     const int query_row = row_base + (lane & 15);
     auto load_query = [&](uint32_t (&f)[4], int k) { ldsm_x4(f, query_at + tile_offset<DK>(query_row, k * 2 + (lane >> 4))); };
 
-    for (int t = tile0; t < tile1; ++t) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(S::kStages - 2) : "memory");
+    for (int t = 0; t < tiles; ++t) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();   // the tile is here, and everyone is done with the stage that is filled next
-        if (t + S::kStages - 1 < tile1) fetch(t + S::kStages - 1, (t - tile0 + S::kStages - 1) % S::kStages);
+        if (t + 1 < tiles) fetch(t + 1, (t + 1) & 1);
         asm volatile("cp.async.commit_group;" ::: "memory");
         if constexpr (kHold) {
-            if (t == tile0) {
+            if (t == 0) {
 #pragma unroll
                 for (int k = 0; k < DK / 16; ++k) load_query(q[k], k);
             }
         }
-        const uint32_t keys = smem_u32(ring + (t - tile0) % S::kStages * S::kStageBytes), values = keys + S::kKeys * DK * 2;
+        const uint32_t keys = smem_u32(ring + (t & 1) * S::kStageBytes), values = keys + S::kKeys * DK * 2;
         float s[NT][4];
 #pragma unroll
         for (int n = 0; n < NT; ++n)
@@ -365,13 +414,13 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 #pragma unroll
             for (int n = 0; n < NT; n += 2) {
                 uint32_t b[4];
-                ldsm_x4(b, keys + tile_offset<DK>(key_base + n * 8 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)));
+                ldsm_x4(b, keys + tile_offset<DK>(n * 8 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)));
                 mma_16816(s[n], f, b[0], b[1]);
                 mma_16816(s[n + 1], f, b[2], b[3]);
             }
         }
-        const int t0 = key_begin + t * S::kKeys + key_base;
-        const bool mask = t0 < all_from || t0 + S::kOwnKeys > all_to;
+        const int t0 = key_begin + t * S::kKeys;
+        const bool mask = t0 < all_from || t0 + S::kKeys > all_to;
         float high[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < NT; ++n)
@@ -414,7 +463,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 #pragma unroll
             for (int v = 0; v < VT; v += 2) {
                 uint32_t b[4];
-                ldsm_x4_trans(b, values + tile_offset<DV>(key_base + k * 16 + (lane & 15), v + (lane >> 4)));
+                ldsm_x4_trans(b, values + tile_offset<DV>(k * 16 + (lane & 15), v + (lane >> 4)));
                 mma_16816(o[v], hi, b[0], b[1]);
                 mma_16816(o[v + 1], hi, b[2], b[3]);
                 mma_16816(o[v], lo, b[0], b[1]);
@@ -428,70 +477,264 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
         total[i] += __shfl_xor_sync(0xffffffffu, total[i], 1);
         total[i] += __shfl_xor_sync(0xffffffffu, total[i], 2);
     }
-    auto store = [&](int row, int head, int column, float x, float y) {
-        const int64_t at = row * a.out_stride + head * p.vdim + column;
-        if (a.out) *reinterpret_cast<float2*>(a.out + at) = make_float2(x, y);
-        if (a.out_hi) {
-            uint32_t hi, lo;
-            pack_planes(x, y, hi, lo);
-            *reinterpret_cast<uint32_t*>(a.out_hi + at) = hi;
-            if (a.out_lo) *reinterpret_cast<uint32_t*>(a.out_lo + at) = lo;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        int position, head;
+        if (!row_of(row_base + (lane >> 2) + i * 8, position, head)) continue;
+        const int row = first + position;
+        const float factor = head_gate(p, row, head) / total[i];
+#pragma unroll
+        for (int v = 0; v < VT; ++v) {
+            const int column = v * 8 + (lane & 3) * 2;
+            if (column < p.vdim) store_pair(a, row, head, column, o[v][2 * i] * factor, o[v][2 * i + 1] * factor);
         }
+    }
+}
+
+// ---- steps ----------------------------------------------------------------------------------------------------------
+constexpr int kStepKeys = 64, kStepBoxBytes = kStepKeys * 64 * 2;
+constexpr int kStepConsumers = 128, kStepThreads = kStepConsumers + 32;
+constexpr int kMaxStages = 6, kStepControlBytes = 256;
+constexpr int kHalfSmem = 113 * 1024;   // two CTAs of this size share an SM
+
+struct StepItem { int sequence, slot, length, kv_head, head_tile, split; };
+
+// Byte offset of 16-byte piece `piece` of a row inside boxes of 64 keys x 64 values, the piece swizzled by its row.
+__device__ __forceinline__ uint32_t box_offset(int row, int piece) {
+    return static_cast<uint32_t>((piece >> 3) * kStepBoxBytes + row * 128 + (((piece & 7) ^ (row & 7)) << 4));
+}
+__device__ __forceinline__ void step_consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kStepConsumers) : "memory"); }
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(kStepThreads) chunk_step_kernel(const __grid_constant__ ChunkAttention a, const __grid_constant__ CUtensorMap key_map,
+                                                                 const __grid_constant__ CUtensorMap value_map) {
+    constexpr int kKeyBoxes = DK / 64, kValueBoxes = DV / 64, kStageBytes = (kKeyBoxes + kValueBoxes) * kStepBoxBytes;
+    extern __shared__ __align__(128) uint8_t smem[];
+    const ChunkParams& p = a.p;
+    uint8_t* ring = smem + ((1024u - (smem_u32(smem) & 1023u)) & 1023u);   // swizzled boxes start on 1024-byte boundaries
+    uint64_t* full = reinterpret_cast<uint64_t*>(ring + a.stages * kStageBytes);
+    uint64_t* empty = full + kMaxStages;
+    int* gave_up = reinterpret_cast<int*>(empty + kMaxStages);
+    float* gates = reinterpret_cast<float*>(gave_up + 2);                                                     // [heads_per_tile]
+    float* merge = reinterpret_cast<float*>(ring + a.stages * kStageBytes + kStepControlBytes);               // [warps][heads_per_tile][DV]
+    float* merge_ml = merge + 4 * a.heads_per_tile * DV;                                                      // [warps][heads_per_tile][2]
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < a.stages; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], kStepConsumers / 32); }
+        mbar_fence_init();
+        *gave_up = 0;
+        tma_prefetch_descriptor(&key_map);
+        tma_prefetch_descriptor(&value_map);
+    }
+    __syncthreads();
+    grid_dependency_wait();
+    grid_launch_dependents();
+
+    const int per_sequence = p.kv_heads * a.head_tiles * a.splits, items = a.rows.sequences * per_sequence;
+    auto load_item = [&](int item) {
+        StepItem it{};
+        if (item < items) {
+            it.sequence = item / per_sequence;
+            const int rest = item - it.sequence * per_sequence, z = rest / a.splits;
+            it.split = rest - z * a.splits;
+            it.kv_head = z / a.head_tiles;
+            it.head_tile = z - it.kv_head * a.head_tiles;
+            it.slot = __ldg(a.rows.slot + it.sequence);
+            it.length = a.rows.lengths[it.slot];
+        }
+        return it;
     };
-    if constexpr (!STEP) {
+    // tiles of an item: the slot holds the keys of the row's chunk, the row's own included, from entry 0 on
+    auto keys_of = [&](const StepItem& it) { return it.length - p.chunk_start(it.length) + 1; };
+    auto range_of = [&](const StepItem& it, int& tile0, int& tile1) {
+        const int tiles = (keys_of(it) + kStepKeys - 1) / kStepKeys, per_split = (tiles + a.splits - 1) / a.splits;
+        tile0 = it.split * per_split;
+        tile1 = min(tiles, tile0 + per_split);
+    };
+    int stage = 0;
+    uint32_t phase = 0;
+    auto next_stage = [&] { if (++stage == a.stages) { stage = 0; phase ^= 1; } };
+    StepItem now = load_item(blockIdx.x);
+
+    if (warp == kStepConsumers / 32) {
+        bool alive = true;
+        for (int item = blockIdx.x; item < items && alive; item += gridDim.x) {
+            const StepItem next = load_item(item + gridDim.x);
+            int tile0, tile1;
+            range_of(now, tile0, tile1);
+            const int row0 = (now.slot * p.kv_heads + now.kv_head) * p.entries;
+            for (int t = tile0; t < tile1; ++t) {
+                if (!mbar_wait(&empty[stage], phase ^ 1)) {   // (passes at once in the first round)
+                    if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
+                    alive = false;
+                    break;
+                }
+                if (elect_one()) {
+                    uint8_t* at = ring + stage * kStageBytes;
+                    mbar_expect_tx(&full[stage], kStageBytes);
+#pragma unroll
+                    for (int b = 0; b < kKeyBoxes; ++b) tma_load_2d(at + b * kStepBoxBytes, &key_map, b * 64, row0 + t * kStepKeys, &full[stage]);
+#pragma unroll
+                    for (int b = 0; b < kValueBoxes; ++b)
+                        tma_load_2d(at + (kKeyBoxes + b) * kStepBoxBytes, &value_map, b * 64, row0 + t * kStepKeys, &full[stage]);
+                }
+                __syncwarp();
+                next_stage();
+            }
+            now = next;
+        }
+        return;
+    }
+
+    constexpr int VT = DV / 8;
+    const float scale2 = p.scale * kLog2e;
+    const int own = warp * 16;   // this warp's keys of a tile
+    for (int item = blockIdx.x; item < items; item += gridDim.x) {
+        const int heads_here = min(a.heads_per_tile, p.group - now.head_tile * a.heads_per_tile);
+        const int head0 = now.kv_head * p.group + now.head_tile * a.heads_per_tile;
+        // queries as fragments: rows are the heads of the token
+        uint32_t q[DK / 16][4];
+        {
+            const auto* query = static_cast<const __nv_bfloat16*>(p.query) + (static_cast<int64_t>(now.sequence) * p.heads + head0) * p.dim;
+#pragma unroll
+            for (int k = 0; k < DK / 16; ++k)
+#pragma unroll
+                for (int part = 0; part < 4; ++part) {
+                    const int m = (lane >> 2) + (part & 1) * 8, column = k * 16 + (lane & 3) * 2 + (part >> 1) * 8;
+                    q[k][part] = m < heads_here && column < p.dim ? *reinterpret_cast<const uint32_t*>(query + m * p.dim + column) : 0u;
+                }
+        }
+        const float gate = threadIdx.x < heads_here ? head_gate(p, now.sequence, head0 + threadIdx.x) : 0.0f;
+        const StepItem next = load_item(item + gridDim.x);
+        int tile0, tile1;
+        range_of(now, tile0, tile1);
+        const int keys = keys_of(now);
+        float o[VT][4];
+#pragma unroll
+        for (int v = 0; v < VT; ++v)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) o[v][i] = 0.0f;
+        float top[2] = {-INFINITY, -INFINITY}, total[2] = {0.0f, 0.0f};
+        for (int t = tile0; t < tile1; ++t) {
+            if (!mbar_wait(&full[stage], phase)) {
+                if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
+                *static_cast<volatile int*>(gave_up) = 1;
+                break;
+            }
+            const uint32_t key_at = smem_u32(ring + stage * kStageBytes), value_at = key_at + kKeyBoxes * kStepBoxBytes;
+            const int seen = keys - t * kStepKeys - own;   // keys of this warp's sixteen that exist
+            if (seen > 0) {
+                float s[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+#pragma unroll
+                for (int k = 0; k < DK / 16; ++k) {
+                    uint32_t b[4];
+                    ldsm_x4(b, key_at + box_offset(own + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)));
+                    mma_16816(s[0], q[k], b[0], b[1]);
+                    mma_16816(s[1], q[k], b[2], b[3]);
+                }
+                float high[2] = {-INFINITY, -INFINITY}, base[2];
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        s[n][i] = n * 8 + (lane & 3) * 2 + (i & 1) < seen ? s[n][i] * scale2 : -INFINITY;
+                        high[i >> 1] = fmaxf(high[i >> 1], s[n][i]);
+                    }
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    high[i] = fmaxf(high[i], __shfl_xor_sync(0xffffffffu, high[i], 1));
+                    high[i] = fmaxf(high[i], __shfl_xor_sync(0xffffffffu, high[i], 2));
+                    base[i] = fmaxf(top[i], high[i]);
+                    const float factor = exp2_fast(top[i] - base[i]);
+                    top[i] = base[i];
+                    total[i] *= factor;
+#pragma unroll
+                    for (int v = 0; v < VT; ++v) { o[v][2 * i] *= factor; o[v][2 * i + 1] *= factor; }
+                }
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        s[n][i] = exp2_fast(s[n][i] - base[i >> 1]);
+                        total[i >> 1] += s[n][i];
+                    }
+                uint32_t hi[4], lo[4];
+                pack_planes(s[0][0], s[0][1], hi[0], lo[0]);
+                pack_planes(s[0][2], s[0][3], hi[1], lo[1]);
+                pack_planes(s[1][0], s[1][1], hi[2], lo[2]);
+                pack_planes(s[1][2], s[1][3], hi[3], lo[3]);
+                // rows past the last key hold what the memory held: they must not reach the products, not even times zero
+                uint32_t live[2] = {0xffffffffu, 0xffffffffu};
+                if (seen < 16) {
+#pragma unroll
+                    for (int h = 0; h < 2; ++h) {
+                        const int left = seen - h * 8 - (lane & 3) * 2;
+                        live[h] = left >= 2 ? 0xffffffffu : left == 1 ? 0x0000ffffu : 0u;
+                    }
+                }
+#pragma unroll
+                for (int v = 0; v < VT; v += 2) {
+                    uint32_t b[4];
+                    ldsm_x4_trans(b, value_at + box_offset(own + (lane & 15), v + (lane >> 4)));
+                    b[0] &= live[0]; b[1] &= live[1]; b[2] &= live[0]; b[3] &= live[1];
+                    mma_16816(o[v], hi, b[0], b[1]);
+                    mma_16816(o[v + 1], hi, b[2], b[3]);
+                    mma_16816(o[v], lo, b[0], b[1]);
+                    mma_16816(o[v + 1], lo, b[2], b[3]);
+                }
+            }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&empty[stage]);
+            next_stage();
+        }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-            int position, head;
-            if (!row_of(row_base + (lane >> 2) + i * 8, position, head)) continue;
-            const int row = first + position;
-            const float factor = head_gate(p, row, head) / total[i];
-#pragma unroll
-            for (int v = 0; v < VT; ++v) {
-                const int column = v * 8 + (lane & 3) * 2;
-                if (column < p.vdim) store(row, head, column, o[v][2 * i] * factor, o[v][2 * i + 1] * factor);
-            }
+            total[i] += __shfl_xor_sync(0xffffffffu, total[i], 1);
+            total[i] += __shfl_xor_sync(0xffffffffu, total[i], 2);
         }
-    } else {
         // the warps' shares of the keys meet in shared memory
-        float* merge = reinterpret_cast<float*>(ring);                  // [warps][16][DV]
-        float* merge_ml = merge + S::kWarps * 16 * DV;                  // [warps][16][2]
-        __syncthreads();
+        step_consumers_sync();   // the item before has been read
+        if (threadIdx.x < heads_here) gates[threadIdx.x] = gate;
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int m = (lane >> 2) + i * 8;
+            if (m >= heads_here) continue;
+            const int at = warp * a.heads_per_tile + m;
 #pragma unroll
             for (int v = 0; v < VT; ++v)
-                *reinterpret_cast<float2*>(merge + (warp * 16 + m) * DV + v * 8 + (lane & 3) * 2) = make_float2(o[v][2 * i], o[v][2 * i + 1]);
-            if ((lane & 3) == 0) { merge_ml[(warp * 16 + m) * 2] = top[i]; merge_ml[(warp * 16 + m) * 2 + 1] = total[i]; }
+                *reinterpret_cast<float2*>(merge + at * DV + v * 8 + (lane & 3) * 2) = make_float2(o[v][2 * i], o[v][2 * i + 1]);
+            if ((lane & 3) == 0) { merge_ml[at * 2] = top[i]; merge_ml[at * 2 + 1] = total[i]; }
         }
-        __syncthreads();
-        for (int c = threadIdx.x; c < a.heads_per_tile * (DV / 2); c += S::kThreads) {
+        step_consumers_sync();
+        if (*static_cast<volatile int*>(gave_up)) return;   // a tile never arrived: every consumer leaves here
+        for (int c = threadIdx.x; c < heads_here * (DV / 2); c += kStepConsumers) {
             const int m = c / (DV / 2), column = (c % (DV / 2)) * 2;
-            int position, head;
-            if (!row_of(m, position, head) || column >= p.vdim) continue;
+            if (column >= p.vdim) continue;
             float best = -INFINITY;
 #pragma unroll
-            for (int w = 0; w < S::kWarps; ++w) best = fmaxf(best, merge_ml[(w * 16 + m) * 2]);
-            const float at = best == -INFINITY ? 0.0f : best;
+            for (int w = 0; w < 4; ++w) best = fmaxf(best, merge_ml[(w * a.heads_per_tile + m) * 2]);
+            const float from = best == -INFINITY ? 0.0f : best;
             float x = 0.0f, y = 0.0f, sum = 0.0f;
 #pragma unroll
-            for (int w = 0; w < S::kWarps; ++w) {
-                const float factor = exp2_fast(merge_ml[(w * 16 + m) * 2] - at);
-                const float2 v = *reinterpret_cast<const float2*>(merge + (w * 16 + m) * DV + column);
+            for (int w = 0; w < 4; ++w) {
+                const int at = w * a.heads_per_tile + m;
+                const float factor = exp2_fast(merge_ml[at * 2] - from);
+                const float2 v = *reinterpret_cast<const float2*>(merge + at * DV + column);
                 x = fmaf(v.x, factor, x);
                 y = fmaf(v.y, factor, y);
-                sum = fmaf(merge_ml[(w * 16 + m) * 2 + 1], factor, sum);
+                sum = fmaf(merge_ml[at * 2 + 1], factor, sum);
             }
-            const int row = first + position;
+            const int head = head0 + m;
             if (a.splits == 1) {
-                const float factor = head_gate(p, row, head) / sum;
-                store(row, head, column, x * factor, y * factor);
+                const float factor = gates[m] / sum;
+                store_pair(a, now.sequence, head, column, x * factor, y * factor);
             } else {
-                const int64_t part = (static_cast<int64_t>(row) * p.heads + head) * a.splits + split;
+                const int64_t part = (static_cast<int64_t>(now.sequence) * p.heads + head) * a.splits + now.split;
                 *reinterpret_cast<float2*>(a.partial + part * p.vdim + column) = make_float2(x, y);
                 if (column == 0) { a.partial_ml[part * 2] = best; a.partial_ml[part * 2 + 1] = sum; }
             }
         }
+        now = next;
     }
 }
 
@@ -571,7 +814,8 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
 }
 
 bool chunk_takes_mma(const ChunkParams& p, int dtype, int64_t out_stride) {
-    return dtype == B200_BF16 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.dim <= 256 && p.vdim <= 256 && (out_stride & 1) == 0;
+    return dtype == B200_BF16 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.dim <= 256 && p.vdim <= 256 && (out_stride & 1) == 0
+        && ((reinterpret_cast<uintptr_t>(p.key_cache) | reinterpret_cast<uintptr_t>(p.value_cache)) & 15) == 0;
 }
 
 // Splits of a step's keys over CTAs: enough for two CTAs per SM, at least two tiles each.
@@ -581,19 +825,59 @@ int chunk_splits(const ChunkParams& p, int sequences, int max_length, int sms) {
     return std::max(1, std::min({(2 * sms + items - 1) / items, tiles / 2, 32}));
 }
 
-template <int DK, int DV, bool STEP> int launch_chunk_mma(const ChunkAttention& a, dim3 grid, cudaStream_t stream) {
-    auto kernel = chunk_mma_kernel<DK, DV, STEP>;
-    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkShape<DK, DV, STEP>::kSmem));
-    return cuda_status(launch_dependent(kernel, grid, dim3(128), ChunkShape<DK, DV, STEP>::kSmem, stream, a), "chunk_mma_kernel launch");
+template <int DK, int DV> int launch_chunk_mma(const ChunkAttention& a, cudaStream_t stream) {
+    auto kernel = chunk_mma_kernel<DK, DV>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkShape<DK, DV>::kSmem));
+    const dim3 grid(static_cast<unsigned>((a.rows.max_count + a.positions_per_tile - 1) / a.positions_per_tile), static_cast<unsigned>(a.rows.sequences),
+                    static_cast<unsigned>(a.p.kv_heads * a.head_tiles));
+    return cuda_status(launch_dependent(kernel, grid, dim3(128), ChunkShape<DK, DV>::kSmem, stream, a), "chunk_mma_kernel launch");
 }
-template <bool STEP> int pick_chunk_mma(const ChunkAttention& a, dim3 grid, cudaStream_t stream) {
-    const int d = a.p.dim, e = a.p.vdim;
-    if (d <= 64 && e <= 64) return launch_chunk_mma<64, 64, STEP>(a, grid, stream);
-    if (d <= 64 && e <= 128) return launch_chunk_mma<64, 128, STEP>(a, grid, stream);
-    if (d <= 128 && e <= 64) return launch_chunk_mma<128, 64, STEP>(a, grid, stream);
-    if (d <= 128 && e <= 128) return launch_chunk_mma<128, 128, STEP>(a, grid, stream);
-    if (d <= 192 && e <= 128) return launch_chunk_mma<192, 128, STEP>(a, grid, stream);
-    return launch_chunk_mma<256, 256, STEP>(a, grid, stream);
+
+int encode_slots(CUtensorMap* map, const void* base, int64_t rows, int columns) {
+    encode_tiled_fn encode = tensor_map_encoder();
+    if (!encode) { set_error("cuTensorMapEncodeTiled is not available from this driver"); return B200_NO_DEVICE; }
+    const cuuint64_t dims[2] = {static_cast<cuuint64_t>(columns), static_cast<cuuint64_t>(rows)};
+    const cuuint64_t strides[1] = {static_cast<cuuint64_t>(columns) * 2};
+    const cuuint32_t box[2] = {64, kStepKeys};
+    const cuuint32_t element_strides[2] = {1, 1};
+    const CUresult result = encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, element_strides,
+                                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (result != CUDA_SUCCESS) { set_error("cuTensorMapEncodeTiled(slots) failed with %d", static_cast<int>(result)); return B200_BAD_ARGUMENT; }
+    return B200_OK;
+}
+
+template <int DK, int DV> int launch_chunk_step(ChunkAttention a, int sms, cudaStream_t stream) {
+    const ChunkParams& p = a.p;
+    alignas(64) CUtensorMap keys, values;
+    const int64_t rows = static_cast<int64_t>(p.slots) * p.kv_heads * p.entries;
+    if (rows > INT32_MAX) { set_error("chunked attention: the slots hold more than 2^31 rows"); return B200_UNSUPPORTED; }
+    int status = encode_slots(&keys, p.key_cache, rows, p.dim);
+    if (status == B200_OK) status = encode_slots(&values, p.value_cache, rows, p.vdim);
+    if (status != B200_OK) return status;
+    const int stage_bytes = (DK + DV) / 64 * kStepBoxBytes, merge_bytes = 4 * a.heads_per_tile * (DV + 2) * 4, fixed = 1024 + kStepControlBytes + merge_bytes;
+    int resident = 2;
+    a.stages = (kHalfSmem - fixed) / stage_bytes;
+    if (a.stages < 2) { resident = 1; a.stages = (2 * kHalfSmem - fixed) / stage_bytes; }
+    a.stages = std::min(a.stages, kMaxStages);
+    const int smem = fixed + a.stages * stage_bytes;
+    auto kernel = chunk_step_kernel<DK, DV>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    const int64_t items = static_cast<int64_t>(a.rows.sequences) * p.kv_heads * a.head_tiles * a.splits;
+    if (items > INT32_MAX) { set_error("chunked attention: too many sequences and heads in one pass"); return B200_UNSUPPORTED; }
+    return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(std::min<int64_t>(items, resident * sms))), dim3(kStepThreads), smem, stream, a, keys,
+                                        values), "chunk_step_kernel launch");
+}
+
+// The smallest pair of compiled head sizes that holds both.
+template <class Launch> int pick_chunk_sizes(const ChunkParams& p, Launch&& launch) {
+    using std::integral_constant;
+    if (p.dim <= 64 && p.vdim <= 64) return launch(integral_constant<int, 64>{}, integral_constant<int, 64>{});
+    if (p.dim <= 64 && p.vdim <= 128) return launch(integral_constant<int, 64>{}, integral_constant<int, 128>{});
+    if (p.dim <= 128 && p.vdim <= 64) return launch(integral_constant<int, 128>{}, integral_constant<int, 64>{});
+    if (p.dim <= 128 && p.vdim <= 128) return launch(integral_constant<int, 128>{}, integral_constant<int, 128>{});
+    if (p.dim <= 192 && p.vdim <= 128) return launch(integral_constant<int, 192>{}, integral_constant<int, 128>{});
+    return launch(integral_constant<int, 256>{}, integral_constant<int, 256>{});
 }
 
 }  // namespace
@@ -628,9 +912,11 @@ extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* 
     }
     const int q = p.heads * p.dim, k = p.kv_heads * p.dim;
     auto aligned = [](const void* at) { return (reinterpret_cast<uintptr_t>(at) & 15) == 0; };
+    auto aligned8 = [](const void* at) { return (reinterpret_cast<uintptr_t>(at) & 7) == 0; };
     const bool vector = p.dim % 4 == 0 && p.vdim % 4 == 0 && (p.rot_dims >> 1) % 4 == 0 && p.stride % 4 == 0 && aligned(p.projected) && aligned(p.q_norm)
         && aligned(p.k_norm) && aligned(p.query) && aligned(p.key) && aligned(p.value) && aligned(p.key_cache) && aligned(p.value_cache)
-        && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0;
+        && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0
+        && (u.kind == 0 || (u.column % 4 == 0 && u.count % 4 == 0 && u.stride % 4 == 0 && aligned(u.out) && aligned8(u.out_hi) && aligned8(u.out_lo)));
     auto kernel = args->dtype == B200_BF16 ? (vector ? chunk_prepare_kernel<__nv_bfloat16, 4> : chunk_prepare_kernel<__nv_bfloat16, 1>)
                                            : (vector ? chunk_prepare_kernel<float, 4> : chunk_prepare_kernel<float, 1>);
     const dim3 grid(static_cast<unsigned>(rows.rows), static_cast<unsigned>(1 + (u.count + kUnitSlice - 1) / kUnitSlice));
@@ -676,11 +962,16 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
             a.partial = static_cast<float*>(scratch);
             a.partial_ml = a.partial + static_cast<int64_t>(a.rows.rows) * p.heads * a.splits * p.vdim;
         }
-        const int z = p.kv_heads * a.head_tiles * a.splits;
-        if (a.rows.sequences > 65535 || z > 65535) { set_error("chunked attention: at most 65535 sequences and head tiles in one pass"); return B200_UNSUPPORTED; }
-        const dim3 grid(static_cast<unsigned>((a.rows.max_count + a.positions_per_tile - 1) / a.positions_per_tile), static_cast<unsigned>(a.rows.sequences),
-                        static_cast<unsigned>(z));
-        status = a.step ? pick_chunk_mma<true>(a, grid, s) : pick_chunk_mma<false>(a, grid, s);
+        if (a.rows.sequences > 65535 || p.kv_heads * a.head_tiles > 65535) {
+            set_error("chunked attention: at most 65535 sequences and head tiles in one pass");
+            return B200_UNSUPPORTED;
+        }
+        a.status = device_status_word(device);
+        if (!a.status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
+        const int sms = sm_count(device);
+        status = pick_chunk_sizes(p, [&](auto dk, auto dv) {
+            return a.step ? launch_chunk_step<decltype(dk)::value, decltype(dv)::value>(a, sms, s) : launch_chunk_mma<decltype(dk)::value, decltype(dv)::value>(a, s);
+        });
         if (status == B200_OK && a.splits > 1)
             status = cuda_status(launch_dependent(chunk_combine_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(64), 0, s, a),
                                  "chunk_combine_kernel launch");
@@ -695,11 +986,12 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
     }
     if (status != B200_OK || a.step) return status;
     auto append = args->dtype == B200_BF16 ? chunk_append_kernel<__nv_bfloat16> : chunk_append_kernel<float>;
-    return cuda_status(launch_dependent(append, dim3(static_cast<unsigned>(a.rows.rows)), dim3(128), 0, s, p, a.rows), "chunk_append_kernel launch");
+    return cuda_status(launch_dependent(append, dim3(static_cast<unsigned>(std::min(a.rows.rows, 1184))), dim3(128), 0, s, p, a.rows), "chunk_append_kernel launch");
 }
 
-extern "C" const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int64_t out_stride) {
+extern "C" const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int32_t max_count, int64_t out_stride) {
     ChunkParams p;
     if (!chunk_params(args, p)) return "";
-    return chunk_takes_mma(p, args->dtype, out_stride) ? "chunk_mma_kernel" : "chunk_generic_kernel";
+    if (!chunk_takes_mma(p, args->dtype, out_stride)) return "chunk_generic_kernel";
+    return max_count == 1 ? "chunk_step_kernel" : "chunk_mma_kernel";
 }

@@ -242,6 +242,15 @@ struct ExpertGemm {
     int32_t* status;
 };
 
+// Order of the tiles: bands of kBand row tiles, inside a band feature tile after feature tile.  What the CTAs work on at a time - a
+// band's rows and its few experts' weights - then stays in L2 until it is finished with.
+constexpr int kBand = 16;
+__device__ __forceinline__ void tile_place(int t, int row_tiles, int feature_tiles, int& row_tile, int& feature_tile) {
+    const int band = t / (kBand * feature_tiles), inside = t - band * kBand * feature_tiles, height = min(kBand, row_tiles - band * kBand);
+    feature_tile = inside / height;
+    row_tile = band * kBand + inside - feature_tile * height;
+}
+
 template <int EPI>
 __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_constant__ CUtensorMap map_lo,
                                                                          const __grid_constant__ CUtensorMap map_w, const __grid_constant__ ExpertGemm gp) {
@@ -295,8 +304,10 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
         bool alive = true;
         for (int j = 0; j < my_tiles && alive; ++j) {
             const int t = blockIdx.x + j * gridDim.x;
-            const int4 group = __ldg(gp.tiles + t % row_tiles);
-            const int boxes = (group.z + kBox - 1) / kBox, weight_row = group.x * p.out + t / row_tiles * kTile;
+            int row_tile, feature_tile;
+            tile_place(t, row_tiles, feature_tiles, row_tile, feature_tile);
+            const int4 group = __ldg(gp.tiles + row_tile);
+            const int boxes = (group.z + kBox - 1) / kBox, weight_row = group.x * p.out + feature_tile * kTile;
             for (int i = 0; i < k_blocks; ++i, ++it) {
                 const int s = it % kStages;
                 if (!mbar_wait(&empty[s], ((it / kStages) & 1) ^ 1)) {
@@ -358,8 +369,10 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
         const uint32_t own_tile[8] = {smem_u32(tile), 0u, 0u, 0u, 0u, 0u, 0u, 0u};
         for (int j = 0; j < my_tiles; ++j) {
             const int t = blockIdx.x + j * gridDim.x;
-            const int4 group = __ldg(gp.tiles + t % row_tiles);
-            const int n0 = t / row_tiles * kTile, buffer = j & 1;
+            int row_tile, feature_tile;
+            tile_place(t, row_tiles, feature_tiles, row_tile, feature_tile);
+            const int4 group = __ldg(gp.tiles + row_tile);
+            const int n0 = feature_tile * kTile, buffer = j & 1;
             row_scale[tile_row] = gp.scale && tile_row < group.z ? __ldg(gp.scale + group.y + tile_row) : 1.0f;
             const bool ready = mbar_wait_relaxed(&acc_full[buffer], (j >> 1) & 1);
             if (!ready && lane == 0) { atomicExch(gp.status, B200_DEVICE_TIMEOUT); *alive_flag = 0; }
@@ -381,7 +394,7 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
             if (lane == 0) mbar_arrive(&acc_empty[buffer]);
             asm volatile("bar.sync 2, 128;" ::: "memory");    // the tile and the row scales are in shared memory
             if (*alive_flag == 0) break;                       // same decision in all four warps
-            finish_rows<EPI, kTile>(p, tile, own_tile, 1, row_scale, group.y, n0, t / row_tiles, 0, group.z, quarter, 4, lane, true);
+            finish_rows<EPI, kTile>(p, tile, own_tile, 1, row_scale, group.y, n0, feature_tile, 0, group.z, quarter, 4, lane, true);
             asm volatile("bar.sync 2, 128;" ::: "memory");    // the next tile may overwrite the shared-memory tile
         }
     }

@@ -423,6 +423,7 @@ B200_API const char* b200_latent_attention_kernel(const b200_latent_args* args);
  * value workspaces) and leave the sequence's last chunk in the slot afterwards. */
 typedef struct b200_chunk_args {
     int32_t heads, kv_heads, dim, vdim, rot_dims;
+    int32_t slots;                 /* of the caches */
     int32_t chunk;                 /* positions per chunk; 0: no chunks, every earlier position is seen */
     int32_t entries;               /* positions a slot holds: chunk, or the capacity where that is smaller or there are no chunks */
     float scale;
@@ -474,8 +475,9 @@ B200_API int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* pa
 B200_API size_t b200_chunk_scratch_bytes(const b200_chunk_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length);
 B200_API int b200_chunk_attention(const b200_chunk_args* args, const b200_rows* pass, int32_t max_length, void* scratch, size_t scratch_bytes,
                                   float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream);
-/* Name of the kernel b200_chunk_attention runs for these sizes: "chunk_mma_kernel" or "chunk_generic_kernel". */
-B200_API const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int64_t out_stride);
+/* Name of the kernel b200_chunk_attention runs for these sizes: "chunk_step_kernel" (passes of one row per sequence), "chunk_mma_kernel"
+ * or "chunk_generic_kernel". */
+B200_API const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int32_t max_count, int64_t out_stride);
 
 /* Experts of one layer: up [experts][ff][in], down [experts][in][ff] (weight dtype), expert(x) = down gelu(up x); slot (row, choice) adds
  * expert_chosen(weight * row). */

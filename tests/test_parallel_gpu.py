@@ -54,12 +54,12 @@ class Chunked:
         self.keep = [dev(np.cos(angle)), dev(np.sin(angle)), dev(self.q_norm), dev(self.k_norm)]
         k = self.keep
         self.kind = kind
-        self.a = B.ChunkArgs(heads, kv_heads, dim, vdim, self.n["dims"], chunk, entries, scale, eps, k[0].data_ptr(), k[1].data_ptr(), capacity,
+        self.a = B.ChunkArgs(heads, kv_heads, dim, vdim, self.n["dims"], slots, chunk, entries, scale, eps, k[0].data_ptr(), k[1].data_ptr(), capacity,
                              k[2].data_ptr(), k[3].data_ptr(), B.BF16 if self.bf16 else B.F32, self.keys.data_ptr(), self.values.data_ptr())
 
-    def kernel(self):
+    def kernels(self):
         self.a.projected, self.a.stride, self.a.query = 16, self.stride, 16
-        return B.lib().b200_chunk_attention_kernel(C.byref(self.a), self.n["heads"] * self.n["vdim"]).decode()
+        return [B.lib().b200_chunk_attention_kernel(C.byref(self.a), count, self.n["heads"] * self.n["vdim"]).decode() for count in (1, 2)]
 
     def attend(self, p, rows, max_length, units=None, route=None, out_stride=None):
         n, count = self.n, rows.shape[0]
@@ -110,7 +110,7 @@ def test_chunked_attention_layer(spec, dtype):
     """Norms over all heads, rotation of halves, append and attention: a prompt of unequal sequences, single rows, portions of two and
     more, in shuffled slots."""
     k = Chunked(**spec, dtype=dtype, seed=spec["dim"])
-    assert k.kernel() == ("chunk_mma_kernel" if dtype == "bf16" and spec["dim"] % 8 == 0 else "chunk_generic_kernel")
+    assert k.kernels() == (["chunk_step_kernel", "chunk_mma_kernel"] if dtype == "bf16" and spec["dim"] % 8 == 0 else ["chunk_generic_kernel"] * 2)
     tol = 5e-6 if dtype == "f32" else 1.5e-2
     rng = np.random.default_rng(9)
     slots, totals = [2, 0, 3], [209, 76, 14]
