@@ -495,7 +495,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 constexpr int kStepKeys = 64, kStepBoxBytes = kStepKeys * 64 * 2;
 constexpr int kStepConsumers = 128, kStepThreads = kStepConsumers + 32;
 constexpr int kMaxStages = 6, kStepControlBytes = 256;
-constexpr int kHalfSmem = 113 * 1024;   // two CTAs of this size share an SM
+constexpr int kSmSmem = 227 * 1024;
 
 struct StepItem { int sequence, slot, length, kv_head, head_tile, split; };
 
@@ -505,8 +505,11 @@ __device__ __forceinline__ uint32_t box_offset(int row, int piece) {
 }
 __device__ __forceinline__ void step_consumers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kStepConsumers) : "memory"); }
 
+// CTAs that share an SM.
+constexpr int step_residents(int columns) { return columns <= 128 ? 3 : columns <= 256 ? 2 : 1; }
+
 template <int DK, int DV>
-__global__ void __launch_bounds__(kStepThreads) chunk_step_kernel(const __grid_constant__ ChunkAttention a, const __grid_constant__ CUtensorMap key_map,
+__global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_step_kernel(const __grid_constant__ ChunkAttention a, const __grid_constant__ CUtensorMap key_map,
                                                                  const __grid_constant__ CUtensorMap value_map) {
     constexpr int kKeyBoxes = DK / 64, kValueBoxes = DV / 64, kStageBytes = (kKeyBoxes + kValueBoxes) * kStepBoxBytes;
     extern __shared__ __align__(128) uint8_t smem[];
@@ -856,10 +859,9 @@ template <int DK, int DV> int launch_chunk_step(ChunkAttention a, int sms, cudaS
     if (status == B200_OK) status = encode_slots(&values, p.value_cache, rows, p.vdim);
     if (status != B200_OK) return status;
     const int stage_bytes = (DK + DV) / 64 * kStepBoxBytes, merge_bytes = 4 * a.heads_per_tile * (DV + 2) * 4, fixed = 1024 + kStepControlBytes + merge_bytes;
-    int resident = 2;
-    a.stages = (kHalfSmem - fixed) / stage_bytes;
-    if (a.stages < 2) { resident = 1; a.stages = (2 * kHalfSmem - fixed) / stage_bytes; }
-    a.stages = std::min(a.stages, kMaxStages);
+    int resident = step_residents(DK + DV) + 1;
+    do a.stages = std::min((kSmSmem / --resident - 1024 - fixed) / stage_bytes, kMaxStages);
+    while (a.stages < 2 && resident > 1);
     const int smem = fixed + a.stages * stage_bytes;
     auto kernel = chunk_step_kernel<DK, DV>;
     B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));

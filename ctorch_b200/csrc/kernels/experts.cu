@@ -154,16 +154,26 @@ template <class W, bool VECTOR> __global__ void __launch_bounds__(kStreamThreads
 }
 
 // ---- grouped --------------------------------------------------------------------------------------------------------
-constexpr int kTile = 128;        // slots per row tile; features per weight tile
+constexpr int kTile = 128;        // features per weight tile, rows of the products
 constexpr int kBlockK = 64;
 constexpr int kBox = 32;          // slots per activation box
 constexpr int kBoxBytes = kBox * kBlockK * 2;
-constexpr int kPlaneBytes = kTile * kBlockK * 2;
-constexpr int kStages = 3, kStageBytes = 3 * kPlaneBytes;   // x_hi, x_lo, W of one K block
+constexpr int kWeightBytes = kTile * kBlockK * 2;
 constexpr int kTileStride = kTile + 4;
-constexpr int kTileBytes = kTile * kTileStride * 4;
-constexpr int kGroupedSmem = kStages * kStageBytes + kTileBytes + 1024 + 2048;
 constexpr int kGroupedThreads = 192;
+// SLOTS: slots of a row tile.  The products always have 128 rows; what a smaller tile leaves out of the stage goes to further stages,
+// that is to more weights in flight, and the rows past its slots multiply whatever lies behind them in shared memory: results that
+// nobody reads.
+template <int SLOTS> struct GroupedShape {
+    static constexpr int kPlaneBytes = SLOTS * kBlockK * 2;
+    static constexpr int kStageBytes = 2 * kPlaneBytes + kWeightBytes;   // W, x_hi, x_lo of one K block
+    static constexpr int kStages = SLOTS == 128 ? 3 : SLOTS == 64 ? 5 : 8;
+    static constexpr int kTileBytes = SLOTS * kTileStride * 4;
+    static constexpr int kTileAt = kStages * kStageBytes;
+    static constexpr int kControlAt = kTileAt + kTileBytes;
+    static constexpr int kSmem = kControlAt + 1024 + 2048;
+    static_assert((kStages - 1) * kStageBytes + kWeightBytes + kPlaneBytes + kTile * kBlockK * 2 <= kControlAt + 2048, "rows past the slots must lie in shared memory");
+};
 
 struct Grouped {
     __nv_bfloat16 *x_hi, *x_lo;        // [slots, in] in order of their experts
@@ -175,10 +185,15 @@ struct Grouped {
     int32_t* tile_count;
 };
 
+// Slots of a row tile: the smallest height that takes an average expert's slots.
+int tile_slots(const ExpertParams& p) {
+    const int average = p.rows * p.top / p.experts;
+    return average <= 24 ? 32 : average <= 48 ? 64 : 128;
+}
 size_t round_up_256(size_t n) { return (n + 255) & ~static_cast<size_t>(255); }
 int most_tiles(const ExpertParams& p) {
     const int slots = p.rows * p.top;
-    return slots / kTile + std::min(p.experts, slots);   // every expert has at most one tile that is not full
+    return slots / tile_slots(p) + std::min(p.experts, slots);   // every expert has at most one tile that is not full
 }
 size_t grouped_layout(const ExpertParams& p, uint8_t* base, Grouped& g) {
     const size_t slots = static_cast<size_t>(p.rows) * p.top;
@@ -199,7 +214,7 @@ size_t grouped_layout(const ExpertParams& p, uint8_t* base, Grouped& g) {
 
 // One CTA per slot; CTA 0 also writes the list of row tiles.
 __global__ void __launch_bounds__(256) expert_gather_kernel(const __grid_constant__ ExpertParams p, const __grid_constant__ Grouped g, const int32_t* rank,
-                                                            const int32_t* counts) {
+                                                            const int32_t* counts, const int height) {
     extern __shared__ int32_t copy[];   // [experts]
     __shared__ int32_t before;
     grid_dependency_wait();
@@ -227,8 +242,8 @@ __global__ void __launch_bounds__(256) expert_gather_kernel(const __grid_constan
     if (slot == 0) {
         for (int e = threadIdx.x; e < p.experts; e += blockDim.x) {
             int tile = 0, row = 0;
-            for (int i = 0; i < e; ++i) { tile += (copy[i] + kTile - 1) / kTile; row += copy[i]; }
-            for (int left = copy[e]; left > 0; left -= kTile, row += kTile) g.tiles[tile++] = make_int4(e, row, min(left, kTile), 0);
+            for (int i = 0; i < e; ++i) { tile += (copy[i] + height - 1) / height; row += copy[i]; }
+            for (int left = copy[e]; left > 0; left -= height, row += height) g.tiles[tile++] = make_int4(e, row, min(left, height), 0);
             if (e == p.experts - 1) *g.tile_count = tile;
         }
     }
@@ -251,14 +266,16 @@ __device__ __forceinline__ void tile_place(int t, int row_tiles, int feature_til
     row_tile = band * kBand + inside - feature_tile * height;
 }
 
-template <int EPI>
+template <int EPI, int SLOTS>
 __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_constant__ CUtensorMap map_lo,
                                                                          const __grid_constant__ CUtensorMap map_w, const __grid_constant__ ExpertGemm gp) {
+    using S = GroupedShape<SLOTS>;
+    constexpr int kStages = S::kStages, kStageBytes = S::kStageBytes;
     const LinearParams& p = gp.base;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-    float* tile = reinterpret_cast<float*>(smem + kStages * kStageBytes);
-    uint8_t* control = smem + kStages * kStageBytes + kTileBytes;
+    float* tile = reinterpret_cast<float*>(smem + S::kTileAt);
+    uint8_t* control = smem + S::kControlAt;
     uint64_t* full = reinterpret_cast<uint64_t*>(control);
     uint64_t* empty = full + kStages;
     uint64_t* acc_full = empty + kStages;    // [2]
@@ -317,11 +334,11 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
                 }
                 if (elect_one()) {
                     uint8_t* stage = smem + s * kStageBytes;
-                    mbar_expect_tx(&full[s], static_cast<uint32_t>(kPlaneBytes + 2 * boxes * kBoxBytes));
-                    tma_load_2d(stage + 2 * kPlaneBytes, &map_w, i * kBlockK, weight_row, &full[s]);
+                    mbar_expect_tx(&full[s], static_cast<uint32_t>(kWeightBytes + 2 * boxes * kBoxBytes));
+                    tma_load_2d(stage, &map_w, i * kBlockK, weight_row, &full[s]);
                     for (int b = 0; b < boxes; ++b) {
-                        tma_load_2d(stage + b * kBoxBytes, &map_hi, i * kBlockK, group.y + b * kBox, &full[s]);
-                        tma_load_2d(stage + kPlaneBytes + b * kBoxBytes, &map_lo, i * kBlockK, group.y + b * kBox, &full[s]);
+                        tma_load_2d(stage + kWeightBytes + b * kBoxBytes, &map_hi, i * kBlockK, group.y + b * kBox, &full[s]);
+                        tma_load_2d(stage + kWeightBytes + S::kPlaneBytes + b * kBoxBytes, &map_lo, i * kBlockK, group.y + b * kBox, &full[s]);
                     }
                 }
                 __syncwarp();
@@ -349,8 +366,8 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
                 tc_fence_after_sync();
                 if (elect_one()) {
                     const uint32_t stage = smem_u32(smem + s * kStageBytes);
-                    const uint64_t hi = operand_descriptor(stage), lo = operand_descriptor(stage + kPlaneBytes);
-                    const uint64_t w = operand_descriptor(stage + 2 * kPlaneBytes);
+                    const uint64_t w = operand_descriptor(stage), hi = operand_descriptor(stage + kWeightBytes);
+                    const uint64_t lo = operand_descriptor(stage + kWeightBytes + S::kPlaneBytes);
 #pragma unroll
                     for (int k = 0; k < kBlockK / 16; ++k) {
                         tc_mma_bf16(accumulator, hi + 2 * k, w + 2 * k, kInstruction, (i | k) != 0);
@@ -377,7 +394,7 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
             const bool ready = mbar_wait_relaxed(&acc_full[buffer], (j >> 1) & 1);
             if (!ready && lane == 0) { atomicExch(gp.status, B200_DEVICE_TIMEOUT); *alive_flag = 0; }
             tc_fence_after_sync();
-            if (ready && quarter * 32 < group.z) {   // lanes past the group's slots hold no results
+            if (ready && quarter * 32 < group.z) {   // (so tile_row < SLOTS) lanes past the group's slots hold no results
 #pragma unroll 1
                 for (int c = 0; c < kTile / 32; ++c) {
                     uint32_t r[32];
@@ -436,6 +453,14 @@ int encode_plane(CUtensorMap* map, const void* base, int64_t rows, int columns, 
     return B200_OK;
 }
 
+template <int EPI, int SLOTS>
+int launch_expert_tiles(const CUtensorMap& hi, const CUtensorMap& lo, const CUtensorMap& w, const ExpertGemm& gp, int ctas, cudaStream_t stream) {
+    auto kernel = expert_gemm_kernel<EPI, SLOTS>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, GroupedShape<SLOTS>::kSmem));
+    return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(ctas)), dim3(kGroupedThreads), GroupedShape<SLOTS>::kSmem, stream, hi, lo, w, gp),
+                       "expert_gemm_kernel launch");
+}
+
 template <int EPI>
 int launch_expert_gemm(const ExpertParams& e, const Grouped& g, const __nv_bfloat16* hi, const __nv_bfloat16* lo, const void* weight, int in, int out,
                        ExpertGemm gp, int sms, cudaStream_t stream) {
@@ -447,11 +472,12 @@ int launch_expert_gemm(const ExpertParams& e, const Grouped& g, const __nv_bfloa
     if (status != B200_OK) return status;
     gp.base.rows = slots; gp.base.in = in; gp.base.out = out;
     gp.tiles = g.tiles; gp.tile_count = g.tile_count;
-    auto kernel = expert_gemm_kernel<EPI>;
-    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kGroupedSmem));
-    const int64_t bound = static_cast<int64_t>(most_tiles(e)) * ((out + kTile - 1) / kTile);
-    return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(std::min<int64_t>(bound, sms))), dim3(kGroupedThreads), kGroupedSmem, stream, map_hi,
-                                        map_lo, map_w, gp), "expert_gemm_kernel launch");
+    const int ctas = static_cast<int>(std::min<int64_t>(static_cast<int64_t>(most_tiles(e)) * ((out + kTile - 1) / kTile), sms));
+    switch (tile_slots(e)) {
+    case 32: return launch_expert_tiles<EPI, 32>(map_hi, map_lo, map_w, gp, ctas, stream);
+    case 64: return launch_expert_tiles<EPI, 64>(map_hi, map_lo, map_w, gp, ctas, stream);
+    default: return launch_expert_tiles<EPI, 128>(map_hi, map_lo, map_w, gp, ctas, stream);
+    }
 }
 
 // Slots up to which every slot streams its expert on its own.
@@ -496,7 +522,7 @@ extern "C" int b200_experts_grouped(const b200_experts* args, const int32_t* ran
     const int sms = sm_count(device), slots = p.rows * p.top;
     cudaStream_t s = as_stream(stream);
     int status = cuda_status(launch_dependent(expert_gather_kernel, dim3(static_cast<unsigned>(slots)), dim3(256), static_cast<size_t>(p.experts) * 4, s, p, g, rank,
-                                              counts), "expert_gather_kernel launch");
+                                              counts, tile_slots(p)), "expert_gather_kernel launch");
     if (status != B200_OK) return status;
     ExpertGemm up = gp, down = gp;
     up.scale = g.scale;

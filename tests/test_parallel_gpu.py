@@ -297,7 +297,7 @@ def test_streamed_experts(rows, experts, top, width, ff, dtype, form):
     assert run_experts(rows, experts, top, width, ff, dtype, form, "some") < (3e-6 if form == "f32" else 3e-5)
 
 
-@pytest.mark.parametrize("rows, experts, top, width, ff", [(1, 2, 1, 8, 8), (25, 8, 1, 64, 72), (60, 70, 5, 200, 136), (700, 5, 2, 136, 264), (300, 300, 3, 64, 32)])
+@pytest.mark.parametrize("rows, experts, top, width, ff", [(1, 2, 1, 8, 8), (25, 8, 1, 64, 72), (60, 70, 5, 200, 136), (90, 6, 2, 136, 200), (700, 5, 2, 136, 264), (300, 300, 3, 64, 32)])
 @pytest.mark.parametrize("load", ["some", "one"])
 def test_grouped_experts(rows, experts, top, width, ff, load):
     assert run_experts(rows, experts, top, width, ff, "bf16", "grouped", load) < 5e-5
