@@ -58,26 +58,26 @@ __device__ __forceinline__ float slot_scale(const ExpertParams& p, int slot) {
 }
 
 // ---- streamed -------------------------------------------------------------------------------------------------------
-constexpr int kStreamThreads = 256, kFeaturesPerWarp = 4, kFeaturesPerCta = kStreamThreads / 32 * kFeaturesPerWarp;
+constexpr int kStreamThreads = 256, kStreamWarps = kStreamThreads / 32;
 
-// Dot products of kFeaturesPerWarp weight rows with a vector in shared memory, by one warp; every lane gets the sums.
-template <class W, bool VECTOR>
-__device__ __forceinline__ void dot_rows(const W* const (&w)[kFeaturesPerWarp], const float* x, int n, int lane, float (&acc)[kFeaturesPerWarp]) {
+// Dot products of F weight rows with a vector in shared memory, by one warp; every lane gets its share of the sums.
+template <class W, bool VECTOR, int F>
+__device__ __forceinline__ void dot_rows(const W* const (&w)[F], const float* x, int n, int lane, float (&acc)[F]) {
     if constexpr (VECTOR) {
         constexpr int kPer = 16 / sizeof(W);
-#pragma unroll 2
+#pragma unroll (8 / F)
         for (int k = lane * kPer; k < n; k += 32 * kPer) {
+            uint4 raw[F];
+#pragma unroll
+            for (int f = 0; f < F; ++f) raw[f] = load_stream_16(w[f] + k);
             float v[kPer];
 #pragma unroll
             for (int i = 0; i < kPer; i += 4) {
                 const float4 q = *reinterpret_cast<const float4*>(x + k + i);
                 v[i] = q.x; v[i + 1] = q.y; v[i + 2] = q.z; v[i + 3] = q.w;
             }
-            uint4 raw[kFeaturesPerWarp];
 #pragma unroll
-            for (int f = 0; f < kFeaturesPerWarp; ++f) raw[f] = load_stream_16(w[f] + k);
-#pragma unroll
-            for (int f = 0; f < kFeaturesPerWarp; ++f) {
+            for (int f = 0; f < F; ++f) {
                 const uint32_t r[4] = {raw[f].x, raw[f].y, raw[f].z, raw[f].w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -89,68 +89,102 @@ __device__ __forceinline__ void dot_rows(const W* const (&w)[kFeaturesPerWarp], 
     } else {
         for (int k = lane; k < n; k += 32)
 #pragma unroll
-            for (int f = 0; f < kFeaturesPerWarp; ++f) acc[f] = fmaf(x[k], load_as_f32(w[f], k), acc[f]);
+            for (int f = 0; f < F; ++f) acc[f] = fmaf(x[k], load_as_f32(w[f], k), acc[f]);
     }
 }
 
-// grid (slots, feature blocks): act[slot, f] = gelu(up_f . (scale * row))
-template <class W, bool VECTOR> __global__ void __launch_bounds__(kStreamThreads) expert_up_kernel(const __grid_constant__ ExpertParams p, float* act) {
+// Asks for the CTA's weight rows [first, last) of an expert while the kernel before is still running.  The router's choice is older than
+// that kernel in every plan; where it is not, a stale number (kept in range) only fetches rows in vain.  Worth it while the grid is about
+// one CTA per SM (F = 1); later waves would only ask for what they are about to load.
+template <class W> __device__ __forceinline__ void prefetch_rows(const W* matrix, int expert, int experts, int out, int in, int first, int last) {
+    const int known = min(max(expert, 0), experts - 1);
+    const auto* at = reinterpret_cast<const uint8_t*>(matrix + (static_cast<int64_t>(known) * out + first) * in);
+    const int64_t bytes = static_cast<int64_t>(last - first) * in * static_cast<int>(sizeof(W));
+    for (int64_t o = static_cast<int64_t>(threadIdx.x) * 128; o < bytes; o += kStreamThreads * 128) prefetch_l2(at + o);
+}
+
+// grid (slots, feature blocks): act[slot, f] = gelu(up_f . (scale * row)), F features per warp
+template <class W, bool VECTOR, int F> __global__ void __launch_bounds__(kStreamThreads) expert_up_kernel(const __grid_constant__ ExpertParams p, float* act) {
     extern __shared__ __align__(16) float x[];
+    const int slot = blockIdx.x, row = slot / p.top, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int block0 = blockIdx.y * kStreamWarps * F, f0 = block0 + warp * F;
+    if constexpr (F == 1) prefetch_rows(static_cast<const W*>(p.up), *static_cast<const volatile int32_t*>(p.chosen + slot), p.experts, p.ff, p.in, block0, min(block0 + kStreamWarps * F, p.ff));
     grid_dependency_wait();
     grid_launch_dependents();
-    const int slot = blockIdx.x, row = slot / p.top, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float scale = slot_scale(p, slot);
     const int64_t base = static_cast<int64_t>(row) * p.in;
     for (int c = threadIdx.x; c < p.in; c += kStreamThreads)
         x[c] = (p.x ? p.x[base + c] : __bfloat162float(p.x_hi[base + c]) + __bfloat162float(p.x_lo[base + c])) * scale;
+    const int expert = *static_cast<const volatile int32_t*>(p.chosen + slot);
     __syncthreads();
-    const int f0 = blockIdx.y * kFeaturesPerCta + warp * kFeaturesPerWarp;
     if (f0 >= p.ff) return;
-    const int expert = __ldg(p.chosen + slot);
-    const W* w[kFeaturesPerWarp];
-    float acc[kFeaturesPerWarp];
+    const W* w[F];
+    float acc[F];
 #pragma unroll
-    for (int f = 0; f < kFeaturesPerWarp; ++f) {
+    for (int f = 0; f < F; ++f) {
         w[f] = static_cast<const W*>(p.up) + (static_cast<int64_t>(expert) * p.ff + min(f0 + f, p.ff - 1)) * p.in;
         acc[f] = 0.0f;
     }
-    dot_rows<W, VECTOR>(w, x, p.in, lane, acc);
+    dot_rows<W, VECTOR, F>(w, x, p.in, lane, acc);
 #pragma unroll
-    for (int f = 0; f < kFeaturesPerWarp; ++f) {
+    for (int f = 0; f < F; ++f) {
         const float v = warp_sum(acc[f]);
         if (lane == f && f0 + f < p.ff) act[static_cast<int64_t>(slot) * p.ff + f0 + f] = gelu_exact(v);
     }
 }
 
 // grid (rows, feature blocks): y = residual + sum over the choices of down . act
-template <class W, bool VECTOR> __global__ void __launch_bounds__(kStreamThreads) expert_down_kernel(const __grid_constant__ ExpertParams p, const float* act) {
+template <class W, bool VECTOR, int F> __global__ void __launch_bounds__(kStreamThreads) expert_down_kernel(const __grid_constant__ ExpertParams p, const float* act) {
     extern __shared__ __align__(16) float x[];
+    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int block0 = blockIdx.y * kStreamWarps * F, f0 = block0 + warp * F;
+    for (int k = 0; F == 1 && k < p.top; ++k)
+        prefetch_rows(static_cast<const W*>(p.down), *static_cast<const volatile int32_t*>(p.chosen + row * p.top + k), p.experts, p.in, p.ff, block0,
+                      min(block0 + kStreamWarps * F, p.in));
     grid_dependency_wait();
     grid_launch_dependents();
-    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int f0 = blockIdx.y * kFeaturesPerCta + warp * kFeaturesPerWarp;
-    float sum[kFeaturesPerWarp];
+    float sum[F];
 #pragma unroll
-    for (int f = 0; f < kFeaturesPerWarp; ++f) sum[f] = 0.0f;
+    for (int f = 0; f < F; ++f) sum[f] = 0.0f;
     for (int k = 0; k < p.top; ++k) {
         const int slot = row * p.top + k;
         __syncthreads();
         for (int c = threadIdx.x; c < p.ff; c += kStreamThreads) x[c] = act[static_cast<int64_t>(slot) * p.ff + c];
+        const int expert = *static_cast<const volatile int32_t*>(p.chosen + slot);
         __syncthreads();
-        const int expert = __ldg(p.chosen + slot);
-        const W* w[kFeaturesPerWarp];
+        const W* w[F];
 #pragma unroll
-        for (int f = 0; f < kFeaturesPerWarp; ++f) w[f] = static_cast<const W*>(p.down) + (static_cast<int64_t>(expert) * p.in + min(f0 + f, p.in - 1)) * p.ff;
-        if (f0 < p.in) dot_rows<W, VECTOR>(w, x, p.ff, lane, sum);
+        for (int f = 0; f < F; ++f) w[f] = static_cast<const W*>(p.down) + (static_cast<int64_t>(expert) * p.in + min(f0 + f, p.in - 1)) * p.ff;
+        if (f0 < p.in) dot_rows<W, VECTOR, F>(w, x, p.ff, lane, sum);
     }
 #pragma unroll
-    for (int f = 0; f < kFeaturesPerWarp; ++f) {
+    for (int f = 0; f < F; ++f) {
         const float v = warp_sum(sum[f]);
         if (lane == f && f0 + f < p.in) {
             const int64_t at = static_cast<int64_t>(row) * p.in + f0 + f;
             p.y[at] = p.residual[at] + v;
         }
     }
+}
+
+template <class W, bool VECTOR, int F> int launch_expert_up(const ExpertParams& p, float* act, size_t smem, cudaStream_t stream) {
+    auto kernel = expert_up_kernel<W, VECTOR, F>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    const dim3 grid(static_cast<unsigned>(p.rows * p.top), static_cast<unsigned>((p.ff + kStreamWarps * F - 1) / (kStreamWarps * F)));
+    return cuda_status(launch_dependent(kernel, grid, dim3(kStreamThreads), smem, stream, p, act), "expert_up_kernel launch");
+}
+template <class W, bool VECTOR, int F> int launch_expert_down(const ExpertParams& p, const float* act, size_t smem, cudaStream_t stream) {
+    auto kernel = expert_down_kernel<W, VECTOR, F>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    const dim3 grid(static_cast<unsigned>(p.rows), static_cast<unsigned>((p.in + kStreamWarps * F - 1) / (kStreamWarps * F)));
+    return cuda_status(launch_dependent(kernel, grid, dim3(kStreamThreads), smem, stream, p, act), "expert_down_kernel launch");
+}
+// Four features per warp, or one where that would leave SMs without a CTA.
+template <class W, bool VECTOR> int launch_streamed(const ExpertParams& p, float* act, size_t up_smem, size_t down_smem, int sms, cudaStream_t stream) {
+    const int64_t up = static_cast<int64_t>(p.rows) * p.top * ((p.ff + 31) / 32), down = static_cast<int64_t>(p.rows) * ((p.in + 31) / 32);
+    const int status = up < 2 * sms ? launch_expert_up<W, VECTOR, 1>(p, act, up_smem, stream) : launch_expert_up<W, VECTOR, 4>(p, act, up_smem, stream);
+    if (status != B200_OK) return status;
+    return down < 2 * sms ? launch_expert_down<W, VECTOR, 1>(p, act, down_smem, stream) : launch_expert_down<W, VECTOR, 4>(p, act, down_smem, stream);
 }
 
 // ---- grouped --------------------------------------------------------------------------------------------------------
@@ -255,6 +289,7 @@ struct ExpertGemm {
     const int32_t* tile_count;
     const float* scale;         // [slots] or NULL
     int32_t* status;
+    bool listed;                // the list is older than the kernel before: the first weights may be asked for while that one runs
 };
 
 // Order of the tiles: bands of kBand row tiles, inside a band feature tile after feature tile.  What the CTAs work on at a time - a
@@ -311,6 +346,23 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
     tc_fence_after_sync();
     const uint32_t tmem_base = *tmem_slot;
 
+    const int k_blocks_ahead = gp.listed && warp == 0 ? min(k_blocks, kStages) : 0;   // K blocks of the first tile whose weights are on their way
+    if (k_blocks_ahead > 0) {
+        const int count = *static_cast<const volatile int32_t*>(gp.tile_count), width = (p.out + kTile - 1) / kTile;
+        if (static_cast<int>(blockIdx.x) < count * width) {
+            int row_tile, feature_tile;
+            tile_place(blockIdx.x, count, width, row_tile, feature_tile);
+            const int4 group = *reinterpret_cast<const int4*>(gp.tiles + row_tile);
+            const int boxes = (group.z + kBox - 1) / kBox;
+            if (elect_one()) {
+                for (int i = 0; i < k_blocks_ahead; ++i) {
+                    mbar_expect_tx(&full[i], static_cast<uint32_t>(kWeightBytes + 2 * boxes * kBoxBytes));
+                    tma_load_2d(smem + i * kStageBytes, &map_w, i * kBlockK, group.x * p.out + feature_tile * kTile, &full[i]);
+                }
+            }
+            __syncwarp();
+        }
+    }
     grid_dependency_wait();
     grid_launch_dependents();
     const int row_tiles = *gp.tile_count, feature_tiles = (p.out + kTile - 1) / kTile, tiles = row_tiles * feature_tiles;
@@ -334,8 +386,10 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
                 }
                 if (elect_one()) {
                     uint8_t* stage = smem + s * kStageBytes;
-                    mbar_expect_tx(&full[s], static_cast<uint32_t>(kWeightBytes + 2 * boxes * kBoxBytes));
-                    tma_load_2d(stage, &map_w, i * kBlockK, weight_row, &full[s]);
+                    if (it >= k_blocks_ahead) {
+                        mbar_expect_tx(&full[s], static_cast<uint32_t>(kWeightBytes + 2 * boxes * kBoxBytes));
+                        tma_load_2d(stage, &map_w, i * kBlockK, weight_row, &full[s]);
+                    }
                     for (int b = 0; b < boxes; ++b) {
                         tma_load_2d(stage + kWeightBytes + b * kBoxBytes, &map_hi, i * kBlockK, group.y + b * kBox, &full[s]);
                         tma_load_2d(stage + kWeightBytes + S::kPlaneBytes + b * kBoxBytes, &map_lo, i * kBlockK, group.y + b * kBox, &full[s]);
@@ -481,7 +535,7 @@ int launch_expert_gemm(const ExpertParams& e, const Grouped& g, const __nv_bfloa
 }
 
 // Slots up to which every slot streams its expert on its own.
-constexpr int kStreamedSlots = 24;
+constexpr int kStreamedSlots = 16;
 
 bool takes_grouped(const b200_experts* a, const ExpertParams& p) {
     return a->weight_dtype == B200_BF16 && p.x_hi && p.x_lo && p.in % 8 == 0 && p.ff % 8 == 0
@@ -530,6 +584,7 @@ extern "C" int b200_experts_grouped(const b200_experts* args, const int32_t* ran
     status = launch_expert_gemm<B200_EPI_GELU>(p, g, g.x_hi, g.x_lo, p.up, p.in, p.ff, up, sms, s);
     if (status != B200_OK) return status;
     down.base.y = g.y;
+    down.listed = true;
     status = launch_expert_gemm<B200_EPI_STORE>(p, g, g.act_hi, g.act_lo, p.down, p.ff, p.in, down, sms, s);
     if (status != B200_OK) return status;
     return cuda_status(launch_dependent(expert_combine_kernel, dim3(static_cast<unsigned>(p.rows)), dim3(256), 0, s, p, static_cast<const float*>(g.y),
@@ -540,24 +595,17 @@ extern "C" int b200_experts_streamed(const b200_experts* args, float* act, void*
     ExpertParams p;
     if (!expert_params(args, p) || !act) { if (!act) set_error("b200_experts_streamed: no workspace"); return B200_BAD_ARGUMENT; }
     const size_t up_smem = (static_cast<size_t>(p.in) * 4 + 15) & ~15ull, down_smem = (static_cast<size_t>(p.ff) * 4 + 15) & ~15ull;
-    const int up_blocks = (p.ff + kFeaturesPerCta - 1) / kFeaturesPerCta, down_blocks = (p.in + kFeaturesPerCta - 1) / kFeaturesPerCta;
-    if (up_smem > 220 * 1024 || down_smem > 220 * 1024 || up_blocks > 65535 || down_blocks > 65535) {
+    if (up_smem > 220 * 1024 || down_smem > 220 * 1024 || p.ff > 65535 * kStreamWarps || p.in > 65535 * kStreamWarps) {
         set_error("b200_experts_streamed: widths %d and %d are too large", p.in, p.ff);
         return B200_UNSUPPORTED;
     }
     const bool bf16 = args->weight_dtype == B200_BF16;
     const int per = bf16 ? 8 : 4;
     const bool vector = p.in % per == 0 && p.ff % per == 0 && ((reinterpret_cast<uintptr_t>(p.up) | reinterpret_cast<uintptr_t>(p.down)) & 15) == 0;
-    auto up = bf16 ? (vector ? expert_up_kernel<__nv_bfloat16, true> : expert_up_kernel<__nv_bfloat16, false>)
-                   : (vector ? expert_up_kernel<float, true> : expert_up_kernel<float, false>);
-    auto down = bf16 ? (vector ? expert_down_kernel<__nv_bfloat16, true> : expert_down_kernel<__nv_bfloat16, false>)
-                     : (vector ? expert_down_kernel<float, true> : expert_down_kernel<float, false>);
-    B200_CUDA(cudaFuncSetAttribute(up, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(up_smem)));
-    B200_CUDA(cudaFuncSetAttribute(down, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(down_smem)));
+    int device = 0;
+    B200_CUDA(cudaGetDevice(&device));
+    const int sms = sm_count(device);
     cudaStream_t s = as_stream(stream);
-    const int status = cuda_status(launch_dependent(up, dim3(static_cast<unsigned>(p.rows * p.top), static_cast<unsigned>(up_blocks)), dim3(kStreamThreads), up_smem, s,
-                                                    p, act), "expert_up_kernel launch");
-    if (status != B200_OK) return status;
-    return cuda_status(launch_dependent(down, dim3(static_cast<unsigned>(p.rows), static_cast<unsigned>(down_blocks)), dim3(kStreamThreads), down_smem, s, p,
-                                        static_cast<const float*>(act)), "expert_down_kernel launch");
+    if (bf16) return vector ? launch_streamed<__nv_bfloat16, true>(p, act, up_smem, down_smem, sms, s) : launch_streamed<__nv_bfloat16, false>(p, act, up_smem, down_smem, sms, s);
+    return vector ? launch_streamed<float, true>(p, act, up_smem, down_smem, sms, s) : launch_streamed<float, false>(p, act, up_smem, down_smem, sms, s);
 }

@@ -43,7 +43,10 @@ CASES = {
                          layer(2, 2, 128, 64, 130, moe(24, 6, 32, 8))], loop=(2, 3, 2), vocab=304),
     # the larger head sizes of the tensor-core attention
     "deep": config(96, [layer(2, 1, 192, 128, 48, dense(64), dims=32), layer(2, 2, 256, 200, 100, moe(8, 1, 48, 16)), layer(3, 1, 72, 96, 31, dense(40))],
-                   vocab=128),
+                   vocab=131),
+    # planes between the kernels, but head sizes and experts without vector loads; an odd vocabulary
+    "uneven": config(64, [layer(3, 1, 12, 8, 9, moe(5, 2, 21, 16), dims=6), layer(4, 2, 20, 18, 14, dense(24)), layer(2, 2, 16, 12, 6, moe(3, 1, 9, 8))],
+                     loop=(0, 1, 2), vocab=97),
 }
 
 
