@@ -4,6 +4,7 @@ from __future__ import annotations
 import numpy as np
 
 from ctorch_b200.workloads import bf16_bits, bf16_to_f32
+import parallel_oracle
 from hybrid_cases import tokens, write_folder  # noqa: F401
 
 
@@ -86,3 +87,17 @@ def make_weights(c, seed=0):
             w = rng.normal(0, {"router": 2.5, "g": 1.5, "down": 1.5, "up": 1.5}.get(leaf, 1.0) / np.sqrt(shape[-1]), shape)
         out[name] = bf16_to_f32(bf16_bits(np.asarray(w, dtype=np.float32))).reshape(shape)
     return out
+
+
+def decided_tokens(c, weights, count, seed=1, margin=0.008):
+    """Random tokens on which no router's choice is a close call, which rounding could turn either way: the first of a few draws."""
+    best, at = None, -1.0
+    for draw in range(30):
+        ids = tokens(c, count, seed=seed + 1000 * draw)
+        calls = [np.inf]
+        parallel_oracle.forward(c, weights, ids, calls=calls)
+        if min(calls) > at:
+            best, at = ids, min(calls)
+        if at > margin:
+            break
+    return best

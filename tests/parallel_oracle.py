@@ -85,8 +85,16 @@ def route(h, w, prefix, top):
     return chosen, np.take_along_axis(scores, chosen, axis=1)
 
 
-def mixture(h, w, prefix, spec):
+def closest_call(h, w, prefix, top):
+    """Smallest distance, over the tokens, between the logits of the last expert chosen and the first one not chosen."""
+    z = np.sort(h @ w[prefix + "router"].T, axis=1)[:, ::-1]
+    return float((z[:, top - 1] - z[:, top]).min()) if z.shape[1] > top else np.inf
+
+
+def mixture(h, w, prefix, spec, calls=None):
     chosen, score = route(h, w, prefix, spec["router"]["top"])
+    if calls is not None:
+        calls.append(closest_call(h, w, prefix, spec["router"]["top"]))
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e, s in zip(chosen[t], score[t]):
@@ -94,11 +102,11 @@ def mixture(h, w, prefix, spec):
     return out + expert(h, w, prefix + "shared.") if spec.get("shared") else out
 
 
-def layer(x, w, i, spec, eps):
+def layer(x, w, i, spec, eps, calls=None):
     h = rms_norm(x, w[f"l{i}.norm1"], eps)
     total = attention(h, w, f"l{i}.mix.", spec["mixer"], eps)
     if spec.get("mlp"):
-        total = total + (dense_ff(h, w, f"l{i}.mlp.") if spec["mlp"]["kind"] == "dense" else mixture(h, w, f"l{i}.mlp.", spec["mlp"]))
+        total = total + (dense_ff(h, w, f"l{i}.mlp.") if spec["mlp"]["kind"] == "dense" else mixture(h, w, f"l{i}.mlp.", spec["mlp"], calls))
     return x + total
 
 
@@ -106,15 +114,15 @@ def enter_pass(x, first, w):
     return np.concatenate([x, first], axis=-1) @ w["loop.in"].T
 
 
-def forward(config, weights, tokens, trail=None):
-    """Logits [T, vocab] of one sequence; `trail` collects the residual stream after every layer run."""
+def forward(config, weights, tokens, trail=None, calls=None):
+    """Logits [T, vocab] of one sequence; `trail` collects the residual stream after every layer run, `calls` the routers' closest calls."""
     w = {n: np.asarray(a, dtype=F) for n, a in weights.items()}
     eps = config["norm"]["eps"]
     x = first = w["embed"][np.asarray(tokens)]
     for i, _, begins in run_order(config):
         if begins:
             x = enter_pass(x, first, w)
-        x = layer(x, w, i, config["layers"][i], eps)
+        x = layer(x, w, i, config["layers"][i], eps, calls)
         if trail is not None:
             trail.append(x.copy())
     return rms_norm(x, w["final.norm"], eps) @ w["head"].T

@@ -333,7 +333,7 @@ def test_prompt_matches_the_statement_layer_by_layer(name, dtype):
     model, w = model_of(name, dtype)
     c = P.CASES[name]
     for count in (71, 9):    # tiles of one expert; slots that stream their experts
-        ids = P.tokens(c, count)
+        ids = P.decided_tokens(c, w, count)
         trail = []
         want = O.forward(c, w, ids, trail)
         model.new_cache(2, 80)
@@ -347,9 +347,9 @@ def test_prompt_matches_the_statement_layer_by_layer(name, dtype):
 @pytest.mark.parametrize("name", P.CASES)
 def test_decoding_and_portions_equal_the_whole_prompt(name, dtype):
     """Token by token, portions of two, unequal portions: the logits of every position equal those of one pass."""
-    model, _ = model_of(name, dtype)
+    model, w = model_of(name, dtype)
     c = P.CASES[name]
-    ids = P.tokens(c, 70, seed=3)
+    ids = P.decided_tokens(c, w, 70, seed=3)
     model.new_cache(1, 70)
     whole = model.run([(0, ids, all_places(70))])
     tol = 1e-5 if dtype == "f32" else 1e-2
@@ -365,11 +365,11 @@ def test_decoding_and_portions_equal_the_whole_prompt(name, dtype):
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
 @pytest.mark.parametrize("name", ["mixed", "wide", "odd", "ones"])
 def test_unequal_batches_equal_each_alone_and_slots_are_reused(name, dtype):
-    model, _ = model_of(name, dtype)
+    model, w = model_of(name, dtype)
     c = P.CASES[name]
-    prompts = [P.tokens(c, n, seed=n) for n in (1, 67, 20, 3, 130)]
-    tails = [4, 6, 1, 9, 5]
-    full = [np.concatenate([p, P.tokens(c, t, seed=100 + t)]) for p, t in zip(prompts, tails)]
+    counts, tails = [1, 67, 20, 3, 130], [4, 6, 1, 9, 5]
+    full = [P.decided_tokens(c, w, n + t, seed=n) for n, t in zip(counts, tails)]
+    prompts = [ids[:n] for ids, n in zip(full, counts)]
     model.new_cache(1, 140)
     alone = []
     for ids in full:
@@ -400,9 +400,9 @@ def test_unequal_batches_equal_each_alone_and_slots_are_reused(name, dtype):
 def test_prompts_and_single_tokens_in_one_pass():
     """A pass in which one request brings a prompt, one goes on by a token and one by three."""
     for dtype in ("f32", "bf16"):
-        model, _ = model_of("mixed", dtype)
+        model, w = model_of("mixed", dtype)
         c = P.CASES["mixed"]
-        full = [P.tokens(c, n, seed=n) for n in (40, 33, 50)]
+        full = [P.decided_tokens(c, w, n, seed=n) for n in (40, 33, 50)]
         model.new_cache(3, 60)
         alone = [model.run([(i, ids, all_places(len(ids)))]) for i, ids in enumerate(full)]
         model.cache.clear()
@@ -431,10 +431,10 @@ def test_long_pass_is_cut_and_joined():
         at += len(wanted)
 
 
-@pytest.mark.parametrize("dtype", ["f32", "bf16"])
-def test_long_decoding_stays_with_the_statement(dtype):
-    model, w = model_of("mixed", dtype)
-    c = P.CASES["mixed"]
+@pytest.mark.parametrize("name, dtype", [("mixed", "f32"), ("plain", "bf16")])   # (plain: every expert is chosen, no call is close)
+def test_long_decoding_stays_with_the_statement(name, dtype):
+    model, w = model_of(name, dtype)
+    c = P.CASES[name]
     ids = P.tokens(c, 300, seed=8)
     want = O.forward(c, w, ids)
     model.new_cache(1, 300)
@@ -519,7 +519,7 @@ def test_single_plane_activations():
     weights = P.make_weights(P.CASES["mixed"], 0)
     model = B.LanguageModel(P.CASES["mixed"], weights)
     model.set_activation_dtype("bf16")
-    ids = P.tokens(P.CASES["mixed"], 60)
+    ids = P.decided_tokens(P.CASES["mixed"], weights, 60, margin=0.05)
     model.new_cache(1, 60)
     assert ratio(model.run([(0, ids, all_places(60))]), O.forward(P.CASES["mixed"], weights, ids)) < 4e-2
 
@@ -550,7 +550,7 @@ def test_command_lines(tmp_path):
                           *[",".join(map(str, p)) for p in prompts]], cwd=ROOT, capture_output=True, text=True, timeout=300)
     assert run.returncode == 0, run.stderr
     assert [[int(t) for t in line.split(",")] for line in run.stdout.split()] == [O.greedy(c, w, p, 4)[0] for p in prompts]
-    a, b = P.tokens(c, 22, seed=5).tolist(), P.tokens(c, 4, seed=6).tolist()
+    a, b = P.decided_tokens(c, w, 22, seed=5).tolist(), P.decided_tokens(c, w, 4, seed=6).tolist()
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": b[:3], "want": []}, {"id": "y", "tokens": a[:20], "want": [0, 15, 16, 19]}], "end": []},
              {"step": 1, "entries": [{"id": "y", "tokens": a[20:21], "want": []}, {"id": "x", "tokens": b[3:], "want": []}], "end": ["x"]},
              {"step": 2, "entries": [{"id": "y", "tokens": a[21:], "want": [0]}], "end": ["y"]},
