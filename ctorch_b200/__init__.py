@@ -48,13 +48,17 @@ class ElementwiseNorm(C.Structure):
     _fields_ = [("alpha", C.c_float), ("weight", C.c_void_p), ("bias", C.c_void_p)]
 
 
+class ClampedUnit(C.Structure):
+    _fields_ = [("slope", C.c_float), ("limit", C.c_float)]
+
+
 class ShadowLinearArgs(C.Structure):
     _fields_ = [("x_hi", C.c_void_p), ("x_lo", C.c_void_p), ("rows", C.c_int64), ("inner", C.c_int64), ("weight", C.c_void_p),
                 ("out", C.c_int64), ("sumsq_in", C.c_void_p), ("parts_in", C.c_int32), ("eps", C.c_double), ("epilogue", C.c_int),
                 ("residual", C.c_void_p), ("qkv", C.POINTER(QkvArgs)), ("y", C.c_void_p), ("out_hi", C.c_void_p),
                 ("out_lo", C.c_void_p), ("out_norm_weight", C.c_void_p), ("out_norm_dtype", C.c_int32), ("sumsq_out", C.c_void_p),
                 ("best_value", C.c_void_p), ("best_index", C.c_void_p), ("y_copies", C.POINTER(C.c_void_p)), ("copies", C.c_int32),
-                ("out_norm", C.POINTER(ElementwiseNorm)), ("out_stride", C.c_int64)]
+                ("out_norm", C.POINTER(ElementwiseNorm)), ("out_stride", C.c_int64), ("unit", C.POINTER(ClampedUnit))]
 
 
 class Rows(C.Structure):
@@ -66,7 +70,8 @@ class Rows(C.Structure):
 class SsmArgs(C.Structure):
     _fields_ = [("heads", C.c_int32), ("vdim", C.c_int32), ("state", C.c_int32), ("groups", C.c_int32), ("taps", C.c_int32),
                 ("conv_weight", C.c_void_p), ("conv_bias", C.c_void_p), ("dt_bias", C.c_void_p), ("a_log", C.c_void_p), ("d", C.c_void_p),
-                ("conv_state", C.c_void_p), ("ssm_state", C.c_void_p), ("projected", C.c_void_p), ("mixed", C.c_void_p), ("y", C.c_void_p)]
+                ("conv_state", C.c_void_p), ("ssm_state", C.c_void_p), ("projected", C.c_void_p), ("mixed", C.c_void_p), ("y", C.c_void_p),
+                ("decay", C.c_void_p), ("stride", C.c_int64)]
 
 
 class LatentArgs(C.Structure):
@@ -76,11 +81,16 @@ class LatentArgs(C.Structure):
                 ("weight_dtype", C.c_int32), ("w_key", C.c_void_p), ("w_value", C.c_void_p)]
 
 
+HEAD_NORM_PROJECTION, HEAD_NORM_NONE, HEAD_NORM_HEAD = 0, 1, 2
+
+
 class ChunkArgs(C.Structure):
     _fields_ = [("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("rot_dims", C.c_int32), ("slots", C.c_int32), ("chunk", C.c_int32),
                 ("entries", C.c_int32), ("scale", C.c_float), ("eps", C.c_double), ("cosine", C.c_void_p), ("sine", C.c_void_p), ("positions", C.c_int32),
                 ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("dtype", C.c_int32), ("key_cache", C.c_void_p), ("value_cache", C.c_void_p),
-                ("projected", C.c_void_p), ("stride", C.c_int64), ("query", C.c_void_p), ("key", C.c_void_p), ("value", C.c_void_p)]
+                ("projected", C.c_void_p), ("stride", C.c_int64), ("query", C.c_void_p), ("key", C.c_void_p), ("value", C.c_void_p),
+                ("q_bias", C.c_void_p), ("k_bias", C.c_void_p), ("norm", C.c_int32), ("rotate_pairs", C.c_int32), ("keys_as_values", C.c_int32),
+                ("keys_elsewhere", C.c_int32), ("no_gate", C.c_int32), ("softcap", C.c_float), ("sink", C.c_void_p), ("scaled", C.c_int32), ("out_scale", C.c_float)]
 
 
 class Units(C.Structure):
@@ -90,13 +100,26 @@ class Units(C.Structure):
 
 class Route(C.Structure):
     _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("column", C.c_int64), ("chosen", C.c_void_p), ("weight", C.c_void_p), ("rank", C.c_void_p),
-                ("counts", C.c_void_p)]
+                ("counts", C.c_void_p), ("softmax", C.c_int32), ("correction", C.c_void_p), ("identity", C.c_int32)]
+
+
+class Sandwich(C.Structure):
+    """The end of a sublayer with a norm behind it: b200_sandwich."""
+    _fields_ = [("after", C.c_void_p), ("next", C.c_void_p), ("eps", C.c_double), ("residual", C.c_void_p), ("x", C.c_void_p), ("normed", C.c_void_p),
+                ("normed_hi", C.c_void_p), ("normed_lo", C.c_void_p)]
+
+
+class PairEmbedding(C.Structure):
+    _fields_ = [("table", C.c_void_p), ("pairs", C.c_void_p), ("dtype", C.c_int32), ("vocab", C.c_int64), ("width", C.c_int64), ("buckets", C.c_int64),
+                ("mul_prev", C.c_int64), ("mul_cur", C.c_int64), ("last", C.c_void_p), ("next", C.c_void_p), ("eps", C.c_double), ("x", C.c_void_p),
+                ("normed", C.c_void_p), ("normed_hi", C.c_void_p), ("normed_lo", C.c_void_p)]
 
 
 class Experts(C.Structure):
     _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("rows", C.c_int64), ("inner", C.c_int64), ("ff", C.c_int64), ("weight_dtype", C.c_int32),
                 ("up", C.c_void_p), ("down", C.c_void_p), ("chosen", C.c_void_p), ("weight", C.c_void_p), ("x", C.c_void_p), ("x_hi", C.c_void_p),
-                ("x_lo", C.c_void_p), ("sumsq_in", C.c_void_p), ("parts_in", C.c_int32), ("eps", C.c_double), ("residual", C.c_void_p), ("y", C.c_void_p)]
+                ("x_lo", C.c_void_p), ("sumsq_in", C.c_void_p), ("parts_in", C.c_int32), ("eps", C.c_double), ("residual", C.c_void_p), ("y", C.c_void_p),
+                ("gated", C.c_int32), ("weigh_results", C.c_int32), ("identity", C.c_int32), ("after", C.POINTER(Sandwich))]
 
 
 class PassEntry(C.Structure):
@@ -226,6 +249,13 @@ def _declare(l: C.CDLL) -> None:
         "b200_scaled_add": (C.c_int, [vp, vp, C.c_float, i64, vp]),
         "b200_gather_rows": (C.c_int, [vp, vp, i64, i64, vp, vp]),
         "b200_rows_advance": (C.c_int, [C.POINTER(Rows), vp]),
+        "b200_rows_advance_tokens": (C.c_int, [C.POINTER(Rows), vp, vp, vp]),
+        "b200_embed_pairs": (C.c_int, [C.POINTER(PairEmbedding), vp, C.POINTER(Rows), vp]),
+        "b200_sandwich_rows": (C.c_int, [vp, i64, i64, C.POINTER(Sandwich), vp]),
+        "b200_soft_cap": (C.c_int, [vp, i64, C.c_float, vp]),
+        "b200_linear_units": (C.c_int, [vp, i64, i64, vp, i32, i64, C.POINTER(ClampedUnit), vp, vp]),
+        "b200_route_rows": (C.c_int, [vp, i64, i64, C.POINTER(Route), vp]),
+        "b200_norm_gated": (C.c_int, [vp, vp, i64, vp, i64, i64, i32, C.c_double, C.c_float, vp, vp, vp, i64, vp]),
         "b200_embedding_scaled": (C.c_int, [vp, i32, vp, i64, i64, i64, C.c_float, vp, vp]),
         "b200_dynamic_tanh": (C.c_int, [vp, vp, vp, i64, i64, C.POINTER(ElementwiseNorm), vp, vp, vp, vp, vp]),
         "b200_ssm_forward": (C.c_int, [C.POINTER(SsmArgs), C.POINTER(Rows), vp]),

@@ -1,4 +1,5 @@
-// Modules, cache, execution plan and generation of the configured decoders (see hybrid.h, hybrid_plan.h; parallel layers: parallel.cpp).
+// Modules, cache, execution plan and generation of the configured decoders (see hybrid.h, hybrid_plan.h; parallel layers: parallel.cpp,
+// sandwich layers: sandwich.cpp).
 #include "dl/hybrid_plan.h"
 
 #include <algorithm>
@@ -41,58 +42,100 @@ LatentAttentionMixer::LatentAttentionMixer(Index width, const LatentAttentionCon
     out = &register_parameter("o", host_zeros({width, c.heads * c.vdim}, options));
 }
 
+namespace {
+GroupedAttentionConfig attention_config(const Json& m, const AttentionKind& kind) {
+    GroupedAttentionConfig c{m.at("heads").positive(), m.at("kv_heads").positive(), m.at("dim").positive(), m.at("vdim").positive(), 0, 0, 1.0,
+                             m.at("scale").number()};
+    c.kind = kind;
+    if (m.has("mask")) c.chunk = m.at("mask").at("size").positive();
+    if (m.has("rot")) {
+        c.rot_dims = m.at("rot").at("dims").positive();
+        c.rot_base = m.at("rot").at("base").number();
+    }
+    if (m.has("softcap")) {
+        c.softcap = m.at("softcap").number();
+        if (!(c.softcap > 0.0)) throw std::invalid_argument("configuration: 'softcap' must be positive");
+    }
+    if (m.has("kv_from")) {
+        c.keys_from = m.at("kv_from").integer();
+        if (c.keys_from < 0) throw std::invalid_argument("configuration: 'kv_from' must be the number of a layer");
+    }
+    return c;
+}
+LightningConfig lightning_config(const Json& m) {
+    LightningConfig c{m.at("heads").positive(), m.at("dim").positive(), m.at("vdim").positive(), {}};
+    for (const Json& d : m.at("decay").items()) c.decay.push_back(d.number());
+    return c;
+}
+}  // namespace
+
 HybridLayer::HybridLayer(Index width, const Json& spec, const DecoderDesign& design, TensorOptions options) {
     auto norm = [&](const std::string& name) {
         RowNorm n;
         n.weight = &register_parameter(name, ones({width}, options));
-        if (design.norm == NormKind::rms) return n;
+        if (design.norm != NormKind::dynamic_tanh) return n;
         n.bias = &register_parameter(name + ".b", host_zeros({width}, options));
         n.alpha = &register_parameter(name + ".alpha", ones({}, options));
         return n;
     };
+    const bool sandwich = design.form == LayerForm::sandwich;
     norm1 = norm("norm1");
+    if (sandwich) after1 = norm("norm1b");
     const std::string& type = spec.at("type").text();
+    const auto mixer = std::find_if(design.mixers.begin(), design.mixers.end(), [&](const MixerDesign& d) { return type == d.type; });
+    if (mixer == design.mixers.end()) throw std::invalid_argument("configuration: unknown layer type '" + type + "' of this architecture");
     const Json& m = spec.at("mixer");
-    if (type == "mamba2") {
+    switch (mixer->kind) {
+    case MixerKind::state_space: {
         const StateSpaceConfig c{m.at("heads").positive(), m.at("vdim").positive(), m.at("state").positive(), m.at("groups").positive(),
                                  m.at("conv").positive(), m.at("norm_groups").positive()};
         state_space = add_module<StateSpaceMixer>("mix", width, c, options);
-    } else if (type == "latent_attention") {
+        break;
+    }
+    case MixerKind::latent: {
         const Json& rot = m.at("rot");
         const LatentAttentionConfig c{m.at("heads").positive(), m.at("dim").positive(), m.at("rot_dim").positive(), m.at("vdim").positive(),
                                       m.at("kv_rank").positive(), m.at("q_rank").positive(), rot.at("dims").positive(), rot.at("base").number(),
                                       m.at("scale").number()};
         latent = add_module<LatentAttentionMixer>("mix", width, c, options);
-    } else if (type == "attention") {
-        ChunkedAttentionConfig c{m.at("heads").positive(), m.at("kv_heads").positive(), m.at("dim").positive(), m.at("vdim").positive(), 0, 0, 1.0,
-                                 m.at("scale").number()};
-        if (m.has("mask")) c.chunk = m.at("mask").at("size").positive();
-        if (m.has("rot")) {
-            c.rot_dims = m.at("rot").at("dims").positive();
-            c.rot_base = m.at("rot").at("base").number();
-        }
-        chunked = add_module<ChunkedAttentionMixer>("mix", width, c, options);
-    } else {
-        throw std::invalid_argument("configuration: unknown layer type '" + type + "'");
+        break;
     }
-    if (design.parallel != (chunked != nullptr))
-        throw std::invalid_argument("configuration: layers of type '" + type + (design.parallel ? "' cannot stand beside a feed-forward" : "' belong to designs with parallel layers"));
-    if (spec.has("mlp")) {
-        const Json& mlp = spec.at("mlp");
-        const std::string& kind = mlp.at("kind").text();
-        if (design.parallel && kind == "moe") {
-            const MixtureConfig c{mlp.at("router").at("experts").positive(), mlp.at("router").at("top").positive(), mlp.at("expert").at("ff").positive(),
-                                  mlp.has("shared") ? mlp.at("shared").at("ff").positive() : 0};
-            mixture = add_module<MixtureOfExperts>("mlp", width, c, options);
-            return;
-        }
-        if (kind != "dense") throw std::invalid_argument("configuration: unknown feed-forward kind '" + kind + "'");
-        const Index ff = mlp.at("ff").positive();
-        if (!design.parallel) norm2 = norm("norm2");
-        gate = &register_parameter("mlp.gate", host_zeros({ff, width}, options));
-        up = &register_parameter("mlp.up", host_zeros({ff, width}, options));
-        down = &register_parameter("mlp.down", host_zeros({width, ff}, options));
+    case MixerKind::attention:
+        attention = add_module<GroupedAttentionMixer>("mix", width, attention_config(m, mixer->attention), options);
+        break;
+    case MixerKind::side_by_side: {
+        const auto pair = add_module<SideBySideMixer>("mix", width, attention_config(m.at("left"), mixer->attention), lightning_config(m.at("right")),
+                                                      m.at("left_scale").number(), m.at("right_scale").number(), options);
+        attention = pair->left;
+        lightning = pair->right;
+        attention_scale = pair->left_scale;
+        lightning_scale = pair->right_scale;
+        break;
     }
+    }
+    if (!spec.has("mlp")) return;
+    const Json& mlp = spec.at("mlp");
+    const std::string& kind = mlp.at("kind").text();
+    if (design.form != LayerForm::parallel) norm2 = norm("norm2");
+    if (sandwich) after2 = norm("norm2b");
+    if (design.mixture && kind == "moe") {
+        const Json& router = mlp.at("router");
+        MixtureConfig c{router.at("experts").positive(), router.at("top").positive(), mlp.at("expert").at("ff").positive(),
+                        mlp.has("shared") ? mlp.at("shared").at("ff").positive() : 0};
+        c.kind = *design.mixture;
+        if (router.has("identity")) c.identity = router.at("identity").integer();
+        mixture = add_module<MixtureOfExperts>("mlp", width, c, options);
+        return;
+    }
+    if (kind != "dense") throw std::invalid_argument("configuration: unknown feed-forward kind '" + kind + "'");
+    const Index ff = mlp.at("ff").positive();
+    if (design.unit_slope > 0.0) {
+        unit_limit = mlp.at("limit").number();
+        if (!(unit_limit > 0.0)) throw std::invalid_argument("configuration: 'limit' must be positive");
+    }
+    gate = &register_parameter("mlp.gate", host_zeros({ff, width}, options));
+    up = &register_parameter("mlp.up", host_zeros({ff, width}, options));
+    down = &register_parameter("mlp.down", host_zeros({width, ff}, options));
 }
 
 void HybridDecoder::set_activation_dtype(DType dtype) {
@@ -130,6 +173,7 @@ HybridCache::HybridCache(const HybridDecoder& model, Index slots, Index capacity
     const Device where = Device::cuda(device_);
     lengths_host_.assign(static_cast<std::size_t>(slots), 0);
     lengths_ = zeros({slots}, {DType::f32, where});   // all-zero bits: int32 zeros
+    if (model.pairs()) last_ = zeros({slots}, {DType::f32, where});
     auto rotary = [&](Index dims, double base) {
         auto& table = tables_[{dims, base}];
         if (!table.cosine.defined()) table = rotary_table(dims, base, capacity, where);
@@ -145,12 +189,18 @@ HybridCache::HybridCache(const HybridDecoder& model, Index slots, Index capacity
                                                         static_cast<int32_t>(c.kv_rank + c.rot_dim), static_cast<int32_t>(capacity), kPageSize,
                                                         lengths(), &run.latent), "latent cache allocation");
                 rotary(c.rot_dims, c.rot_base);
-            } else if (layer.chunked) {
-                const auto& c = layer.chunked->config();
+            } else if (layer.attention) {
+                const auto& c = layer.attention->config();
                 run.entries = c.chunk > 0 ? std::min(c.chunk, capacity) : capacity;
-                run.key = empty({slots, c.kv_heads, run.entries, c.dim}, {model.dtype(), where});
-                run.value = empty({slots, c.kv_heads, run.entries, c.vdim}, {model.dtype(), where});
+                if (layer.attention->own_keys()) {
+                    run.key = empty({slots, c.kv_heads, run.entries, c.dim}, {model.dtype(), where});
+                    run.value = empty({slots, c.kv_heads, run.entries, c.vdim}, {model.dtype(), where});
+                }
                 if (c.rot_dims > 0) rotary(c.rot_dims, c.rot_base);
+                if (layer.lightning) {
+                    const auto& r = layer.lightning->config();
+                    run.state = empty({slots, r.heads, r.dim, r.vdim}, {DType::f32, where});
+                }
             } else {
                 const auto& c = layer.state_space->config();
                 run.conv = empty({slots, c.taps, layer.state_space->channels()}, {DType::f32, where});
@@ -187,7 +237,17 @@ HybridDecoder::HybridDecoder(const Json& config, const DecoderDesign& design, Te
       eps_(config.at("norm").at("eps").number()), embedding_scale_(design.scaled ? config.at("embedding").at("scale").number() : 1.0),
       logit_scale_(design.scaled ? config.at("logit_scale").number() : 1.0) {
     if (dtype_ != DType::f32 && dtype_ != DType::bf16) throw std::invalid_argument("the B200 decoder path stores weights in f32 or bf16");
+    if (config.has("logit_softcap")) {
+        logit_softcap_ = config.at("logit_softcap").number();
+        if (!(logit_softcap_ > 0.0)) throw std::invalid_argument("configuration: 'logit_softcap' must be positive");
+    }
     embed_ = &register_parameter("embed", host_zeros({vocab_, width_}, options));
+    if (design_.form == LayerForm::sandwich) {
+        const Json& pair = config.at("embedding").at("bigram");
+        pair_hash_ = {pair.at("buckets").positive(), pair.at("mul_prev").integer(), pair.at("mul_cur").integer()};
+        pairs_ = &register_parameter("bigram", host_zeros({pair_hash_.buckets + 1, width_}, options));
+        if (config.has("loop")) throw std::invalid_argument("configuration: looped layers are not combined with norms behind the sublayers");
+    }
     const auto& specs = config.at("layers").items();
     const auto count = static_cast<Index>(specs.size());
     if (count == 0) throw std::invalid_argument("decoder requires at least one layer");
@@ -199,15 +259,29 @@ HybridDecoder::HybridDecoder(const Json& config, const DecoderDesign& design, Te
         stop = config.at("loop").at("stop").integer();
         times = config.at("loop").at("times").positive();
         if (start < 0 || stop < start || stop > count) throw std::invalid_argument("configuration: 'loop' must name a range of layers");
-        if ((design_.loop == LoopEntry::joined) != (design_.norm == NormKind::rms))
+        if ((design_.loop == LoopEntry::joined) != (design_.norm != NormKind::dynamic_tanh))
             throw std::invalid_argument("this entry of a looped range is not combined with these norms");
         if (design_.loop == LoopEntry::step) loop_step_ = &register_parameter("loop.step", host_zeros({times, width_}, options));
         else loop_in_ = &register_parameter("loop.in", host_zeros({width_, 2 * width_}, options));
     }
-    for (Index i = 0; i < start; ++i) runs_.push_back({i, -1, false});
+    auto add_run = [&](Index layer, Index pass, bool begins) {
+        const auto own = static_cast<Index>(runs_.size());
+        const auto& mixer = layers_[static_cast<std::size_t>(layer)]->attention;
+        if (!mixer || mixer->own_keys()) return runs_.push_back({layer, pass, begins, own});
+        // the latest run of the layer it names
+        Index from = own - 1;
+        while (from >= 0 && runs_[static_cast<std::size_t>(from)].layer != mixer->config().keys_from) --from;
+        const auto& source = from >= 0 ? layers_[static_cast<std::size_t>(mixer->config().keys_from)]->attention : nullptr;
+        const auto &c = mixer->config();
+        if (!source || !source->own_keys() || source->config().kv_heads != c.kv_heads || source->config().dim != c.dim || source->config().vdim != c.vdim
+            || source->config().chunk != c.chunk)
+            throw std::invalid_argument("configuration: 'kv_from' must name an earlier attention layer with keys of its own and of the same sizes");
+        runs_.push_back({layer, pass, begins, from});
+    };
+    for (Index i = 0; i < start; ++i) add_run(i, -1, false);
     for (Index t = 0; t < times; ++t)
-        for (Index i = start; i < stop; ++i) runs_.push_back({i, t, i == start});
-    for (Index i = stop; i < count; ++i) runs_.push_back({i, -1, false});
+        for (Index i = start; i < stop; ++i) add_run(i, t, i == start);
+    for (Index i = stop; i < count; ++i) add_run(i, -1, false);
     final_norm_.weight = &register_parameter("final.norm", ones({width_}, options));
     if (design_.norm == NormKind::dynamic_tanh) {
         final_norm_.bias = &register_parameter("final.norm.b", host_zeros({width_}, options));
@@ -244,7 +318,8 @@ HybridPlan::Norm HybridPlan::pack_norm(const RowNorm& n, double scale) const {
     Norm packed;
     auto scaled = [&](const Tensor& t) {
         Tensor host = t.to(Device::cpu()).astype(DType::f32).clone();
-        for (Index i = 0; i < host.numel(); ++i) f32(host)[i] = static_cast<float>(static_cast<double>(f32(host)[i]) * scale);
+        const double from = &t == n.weight && owner_.design().norm == NormKind::rms_from_one ? 1.0 : 0.0;
+        for (Index i = 0; i < host.numel(); ++i) f32(host)[i] = static_cast<float>((static_cast<double>(f32(host)[i]) + from) * scale);
         return host.to(t.device());
     };
     packed.weight = scaled(*n.weight);
@@ -266,8 +341,9 @@ void HybridPlan::refresh() {
     for (const auto& module : owner_.layers()) {
         Layer l{};
         l.norm1 = pack_norm(module->norm1);
-        if (module->chunked) {
-            pack_parallel(*module, l);
+        if (module->attention) {
+            if (owner_.design().form == LayerForm::sandwich) pack_sandwich(*module, l);
+            else pack_parallel(*module, l);
             layers_.push_back(std::move(l));
             continue;
         }
@@ -314,10 +390,12 @@ bool HybridPlan::shadows_for(Index rows) const {
     if (D % 8 || !takes(D, owner_.vocabulary())) return false;
     for (std::size_t i = 0; i < layers_.size(); ++i) {
         const HybridLayer& module = *owner_.layers()[i];
-        if (module.chunked && !takes(D, layers_[i].attention_columns)) return false;
+        if (module.attention && !takes(D, layers_[i].attention_columns)) return false;
         if (!takes(D, layers_[i].wide_out) || !takes(layers_[i].inner, D)) return false;
         if (module.latent && !takes(module.latent->config().q_rank, module.latent->uq->size(0))) return false;
-        if (module.has_mlp() && (!takes(D, 2 * module.gate->size(0)) || (!module.chunked && !takes(module.gate->size(0), D)))) return false;
+        if (module.has_mlp() && (!takes(D, 2 * module.gate->size(0)) || (owner_.design().form != LayerForm::parallel && !takes(module.gate->size(0), D))))
+            return false;
+        if (layers_[i].router.defined() && !takes(D, layers_[i].router.size(0))) return false;
     }
     return true;
 }
@@ -357,8 +435,12 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
         const HybridLayer& module = *owner_.layers()[index];
         wide = std::max(wide, layers_[index].wide_out);
         inner = std::max(inner, layers_[index].inner);
-        if (module.has_mlp() && !module.chunked) inner = std::max(inner, module.gate->size(0));
-        if (module.chunked) continue;   // reserve_parallel
+        if (module.has_mlp() && owner_.design().form != LayerForm::parallel) inner = std::max(inner, module.gate->size(0));
+        if (module.lightning) {
+            channels = std::max(channels, module.lightning->channels());
+            y = std::max(y, module.lightning->inner());
+        }
+        if (module.attention) continue;   // reserve_attention
         if (module.state_space) {
             channels = std::max(channels, module.state_space->channels());
             y = std::max(y, module.state_space->inner());
@@ -380,7 +462,7 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
     if (bf16 && shadows_for(rows)) {
         grow(n_, rows, D);
         grow(i_, rows, inner);
-        if (owner_.design().norm == NormKind::rms) {
+        if (owner_.design().norm != NormKind::dynamic_tanh) {
             Index parts = 1;
             for (const auto& layer : layers_) parts = std::max<Index>(parts, b200_linear_shadow_parts(rows, layer.inner, D));
             if (owner_.loop_in()) parts = std::max<Index>(parts, b200_linear_shadow_parts(rows, D, D));
@@ -393,7 +475,14 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
     }
     grow(scratch_, {static_cast<Index>(scratch / 4 + 1)}, DType::f32);
     if (owner_.loop_in()) { grow(joined_first_, {rows, D}, DType::f32); grow(entered_, {rows, D}, DType::f32); }
-    reserve_parallel(rows, max_length, cache, pass);
+    if (owner_.design().form == LayerForm::sandwich) {
+        grow(branch_, {rows, D}, DType::f32);
+        Index outputs = 0;
+        for (const auto& layer : layers_)
+            if (layer.router.defined()) outputs = std::max(outputs, layer.router.size(0));
+        if (outputs) grow(route_logits_, {rows, outputs}, DType::f32);
+    }
+    reserve_attention(rows, max_length, cache, pass);
 }
 
 void HybridPlan::linear(const float* x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y,
@@ -403,12 +492,12 @@ void HybridPlan::linear(const float* x, Index rows, Index in, const void* w, Ind
 }
 
 void HybridPlan::shadow(const Planes& x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y,
-                        const Norm* next, Planes* to, void* stream, const char* what, Index to_column, Index to_stride) {
+                        const Norm* next, Planes* to, void* stream, const char* what, Index to_column, Index to_stride, const b200_clamped_unit* unit) {
     b200_shadow_linear_args args{};
     args.x_hi = x.hi.raw_data();
     args.x_lo = owner_.activation_dtype() == DType::bf16 && rows >= 17 ? nullptr : x.lo.raw_data();
     args.rows = rows; args.in = in; args.weight = w; args.out = out;
-    args.epilogue = epilogue; args.residual = residual; args.y = y;
+    args.epilogue = epilogue; args.residual = residual; args.y = y; args.unit = unit;
     if (x.parts > 0) { args.sumsq_in = squares_.data<float>(); args.parts_in = static_cast<int32_t>(x.parts); args.eps = owner_.eps(); }
     b200_elementwise_norm norm{};
     if (to) {
@@ -438,10 +527,12 @@ void HybridPlan::planes_of(const float* x, Index rows, const Norm& norm, Planes&
 }
 
 void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail) {
+    ids_ = ids;
+    if (owner_.design().form == LayerForm::sandwich) return run_sandwich(ids, pass, cache, max_length, stream, trail);
     const Index rows = pass.rows, D = owner_.width();
     const bool planes = shadows_for(rows);
     float *first = f32(first_), *h = f32(h_);
-    const bool rms = owner_.design().norm == NormKind::rms;
+    const bool rms = owner_.design().norm != NormKind::dynamic_tanh;
     const auto& runs = owner_.runs();
     bool normed = false;   // the previous kernel has written this run's norm1
     auto embed = [&](const Norm* norm, Planes& to) {
@@ -489,11 +580,6 @@ void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache
         }
         in = h;
     };
-    auto keep = [&](std::vector<float>& rows_after) {
-        const std::size_t at = rows_after.size();
-        rows_after.resize(at + static_cast<std::size_t>(rows * D));
-        runtime::copy_bytes(rows_after.data() + at, Device::cpu(), h, Device::cuda(device()), static_cast<std::size_t>(rows * D) * sizeof(float));
-    };
     for (std::size_t i = 0; i < runs.size(); ++i) {
         const LayerRun& r = runs[i];
         const HybridLayer& module = *owner_.layers()[static_cast<std::size_t>(r.layer)];
@@ -518,10 +604,10 @@ void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache
         const After after_layer = last ? After{&final_norm_, false}
             : runs[i + 1].begins_pass ? After{nullptr, owner_.loop_in() != nullptr} : After{&layers_[static_cast<std::size_t>(runs[i + 1].layer)].norm1, false};
         normed = after_layer.norm != nullptr;
-        if (module.chunked) {
+        if (module.attention) {
             const float* residual = run_parallel(i, in, pass, cache, max_length, stream);
             residual_projection(layer.inner, layer.out, residual, after_layer, "output projection");
-            if (trail) keep(*trail);
+            if (trail) keep_rows(rows, *trail);
             continue;
         }
         const After after_mixer = module.has_mlp() ? After{&layer.norm2, false} : after_layer;
@@ -569,7 +655,7 @@ void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache
             else linear(f32(plain_), rows, D, layer.gate_up.raw_data(), 2 * ff, B200_EPI_SWIGLU, nullptr, f32(plain_inner_), stream, "gate/up projection");
             residual_projection(ff, layer.down, in, after_layer, "down projection");
         }
-        if (trail) keep(*trail);
+        if (trail) keep_rows(rows, *trail);
     }
 }
 
@@ -577,6 +663,7 @@ void HybridPlan::logits(Index rows, float* out, void* stream) {
     const Index D = owner_.width(), V = owner_.vocabulary();
     if (shadows_for(rows)) shadow(n_, rows, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, nullptr, nullptr, stream, "logits");
     else linear(f32(plain_), rows, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, stream, "logits");
+    if (owner_.logit_softcap() > 0.0) runtime::check(b200_soft_cap(out, rows * V, static_cast<float>(owner_.logit_softcap()), stream), "logit cap");
 }
 
 void HybridPlan::logits_of(const std::int32_t* index, Index count, float* out, void* stream) {
@@ -597,7 +684,20 @@ void HybridPlan::logits_of(const std::int32_t* index, Index count, float* out, v
     }
     if (planes) shadow(p_, count, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, nullptr, nullptr, stream, "logits");
     else linear(f32(picked_), count, D, owner_.head().raw_data(), V, B200_EPI_STORE, nullptr, out, stream, "logits");
+    if (owner_.logit_softcap() > 0.0) runtime::check(b200_soft_cap(out, count * V, static_cast<float>(owner_.logit_softcap()), stream), "logit cap");
 }
+
+void HybridPlan::keep_rows(Index rows, std::vector<float>& trail) const {
+    const auto count = static_cast<std::size_t>(rows * owner_.width()), at = trail.size();
+    trail.resize(at + count);
+    runtime::copy_bytes(trail.data() + at, Device::cpu(), f32(h_), Device::cuda(device()), count * sizeof(float));
+}
+
+void HybridPlan::advance(const b200_rows& pass, HybridCache& cache, void* stream) {
+    if (owner_.pairs()) runtime::check(b200_rows_advance_tokens(&pass, ids_, cache.last_tokens(), stream), "advance");
+    else runtime::check(b200_rows_advance(&pass, stream), "advance");
+}
+
 
 bool HybridPlan::prepare_choice(Index rows) {
     if (!shadows_for(rows)) return false;
@@ -608,6 +708,7 @@ bool HybridPlan::prepare_choice(Index rows) {
     return true;
 }
 
+// (a cap on the logits keeps their order: the choice is made from the logits before it)
 void HybridPlan::choose(Index rows, const TokenFeedback& f, void* stream) {
     const Index D = owner_.width(), V = owner_.vocabulary();
     b200_shadow_linear_args args{};
@@ -715,7 +816,7 @@ void HybridDecoder::pass(HybridCache& cache, std::span<const PassEntry> entries,
         const b200_rows description = p.maps.describe(slots, counts, cache, device);
         p.reserve(rows, max_length, cache, description);
         p.run(device_ids.data<Index>(), description, cache, max_length, stream, trail);
-        runtime::check(b200_rows_advance(&description, stream), "advance");
+        p.advance(description, cache, stream);
         for (std::size_t m = 0; m < members.size(); ++m) { cache.commit(slots[m], counts[m]); done[members[m]] += counts[m]; }
         while (next < entries.size() && done[next] == static_cast<Index>(entries[next].tokens.size())) ++next;
         if (!picked.empty()) {
@@ -800,7 +901,7 @@ public:
     }
     void step(const Index* ids, Index, void* stream) override { model_->plan().run(ids, pass_, *cache_, cache_->capacity(), stream); }
     void advance(Index, void* stream) override {
-        runtime::check(b200_rows_advance(&pass_, stream), "advance");
+        model_->plan().advance(pass_, *cache_, stream);
         probe(2);
     }
     void logits(Index batch, float* out, void* stream) override { model_->plan().logits(batch, out, stream); }

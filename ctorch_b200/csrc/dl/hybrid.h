@@ -1,10 +1,12 @@
 // Configured decoders: a list of layers with their own mixers and feed-forwards, and a range of layers that may run several times in a
-// row with the same weights.  Two designs are arranged from the pieces here (DecoderDesign):
+// row with the same weights.  Three designs are arranged from the pieces here (DecoderDesign; the registry holds them):
 //   "Ripitar"  state-space (Mamba-2) and latent-attention layers, Dynamic Tanh norms, mixer and SwiGLU feed-forward one after the other;
-//   "Sinezen"  chunked grouped-query attention beside a SwiGLU feed-forward or a mixture of experts that reads the same RMS norm.
+//   "Sinezen"  chunked grouped-query attention beside a SwiGLU feed-forward or a mixture of experts that reads the same RMS norm;
+//   "Lozepel"  a norm before and after every sublayer, three mixers (two kinds of grouped-query attention, and attention side by side with
+//              lightning attention), clamped gated units or a mixture of gated experts, pair embedding, capped logits.
 //
 // The pieces (norms, mixers, feed-forwards, looped range) are separate modules with their constants as parameters; HybridDecoder only
-// arranges them.  Parameter names are the names of the weight files: "embed", "head", "loop.step" or "loop.in",
+// arranges them.  Parameter names are the names of the weight files: "embed", "bigram", "head", "loop.step" or "loop.in",
 // "final.norm{,.alpha,.b}", "l<i>.norm1{,.alpha,.b}", "l<i>.mix.*", "l<i>.mlp.*".
 #pragma once
 
@@ -14,27 +16,60 @@
 
 #include <map>
 #include <memory>
+#include <optional>
 #include <span>
 #include <string>
 #include <vector>
 
 namespace dl::nn {
 
-enum class NormKind { dynamic_tanh, rms };
+// (rms_from_one: the weight is stored as its distance from one)
+enum class NormKind { dynamic_tanh, rms, rms_from_one };
 // How a looped range is entered, before its first layer.
 enum class LoopEntry {
     step,      // x + (embedding output, from the second pass on) + the pass's vector "loop.step"
     joined,    // "loop.in" [x; embedding output], in every pass
 };
+enum class LayerForm {
+    sequential,   // mixer, then feed-forward, each behind its own norm
+    parallel,     // mixer and feed-forward read one norm and are added together
+    sandwich,     // sequential, with a norm behind each sublayer as well, before it is added
+};
+enum class MixerKind { state_space, latent, attention, side_by_side };
+enum class Sink { none, zero, learned };   // a term of the softmax's denominator without a key
+// What kinds of grouped-query attention differ in, beside the sizes and constants of the configuration.
+struct AttentionKind {
+    b200_head_norm norm = B200_HEAD_NORM_PROJECTION;
+    bool rotate_pairs = false;     // entry 2i with entry 2i + 1; otherwise halves
+    bool bias = false;             // on queries and keys
+    bool keys_as_values = false;   // the values are the keys before their rotation
+    bool gate = false;             // one output gate per head
+    Sink sink = Sink::none;
+};
+struct MixtureKind {
+    bool softmax = false;         // scores over all outputs together; otherwise sigmoid
+    bool correction = false;      // a vector added to the scores for the choice alone
+    bool gated = false;           // silu(gate x) * (up x); otherwise gelu(up x)
+    bool weigh_results = false;   // the score multiplies the expert's result; otherwise its input
+};
+// A layer type of a design's configurations and the mixer it stands for (`attention`: with that mixer, or the left one side by side).
+struct MixerDesign {
+    const char* type;
+    MixerKind kind;
+    AttentionKind attention = {};
+};
 // What the layers of a design have in common.
 struct DecoderDesign {
     NormKind norm;
     LoopEntry loop;
-    bool parallel;   // mixer and feed-forward read one norm and are added together
-    bool scaled;     // the configuration gives factors of the embedding and of the logits
+    LayerForm form;
+    bool scaled;                           // the configuration gives factors of the embedding and of the logits
+    std::span<const MixerDesign> mixers;
+    std::optional<MixtureKind> mixture;    // feed-forward kind "moe"
+    double unit_slope = 0.0;               // dense feed-forward: clamped units with this slope, the limit from the configuration; 0: SwiGLU
 };
 
-// Dynamic Tanh: tanh(alpha * x) * w + b; RMS norm: x / sqrt(mean(x^2) + eps) * w, without alpha and bias.  The weight is the module's own
+// Dynamic Tanh: tanh(alpha * x) * w + b; RMS norms: x / sqrt(mean(x^2) + eps) * w (or 1 + w), without alpha and bias.  The weight is the module's own
 // name, alpha and bias beside it, so the names live in the parent.
 struct RowNorm {
     Tensor *weight = nullptr, *alpha = nullptr, *bias = nullptr;
@@ -67,31 +102,65 @@ private:
     LatentAttentionConfig config_;
 };
 
-// Grouped-query attention inside chunks of positions (0: none), RMS norms over all query heads and over all key heads, rotation of
-// halves, one output gate per head; keys and values may differ in size.
-struct ChunkedAttentionConfig {
+// Grouped-query attention, over all earlier positions or inside chunks of them (0: none); keys and values may differ in size.  With
+// keys_from >= 0 the layer has no keys and values of its own and reads those of that layer.
+struct GroupedAttentionConfig {
     Index heads, kv_heads, dim, vdim, chunk, rot_dims;
     double rot_base, scale;
+    double softcap = 0.0;   // score <- softcap tanh(score / softcap); 0: as it is
+    Index keys_from = -1;
+    AttentionKind kind = {};
 };
-class ChunkedAttentionMixer : public Module {
+class GroupedAttentionMixer : public Module {
 public:
-    ChunkedAttentionMixer(Index width, const ChunkedAttentionConfig& config, TensorOptions options);
-    const ChunkedAttentionConfig& config() const { return config_; }
-    Index columns() const;   // rows of q, k, v and g together
-    Tensor *q, *k, *v, *q_norm, *k_norm, *gate, *out;
+    GroupedAttentionMixer(Index width, const GroupedAttentionConfig& config, TensorOptions options);
+    const GroupedAttentionConfig& config() const { return config_; }
+    bool own_keys() const { return config_.keys_from < 0; }
+    Index columns() const;   // rows of q, k, v and g together, as far as there are any
+    Tensor *q, *k = nullptr, *v = nullptr, *q_norm = nullptr, *k_norm = nullptr, *q_bias = nullptr, *k_bias = nullptr, *sink = nullptr, *gate = nullptr, *out;
 private:
-    ChunkedAttentionConfig config_;
+    GroupedAttentionConfig config_;
 };
 
-// Experts down gelu(up x) of which every token takes the `top` with the largest sigmoid scores; the score multiplies the expert's
-// input.  shared_ff: units of an expert of the same form that runs for every token (0: none).
-struct MixtureConfig { Index experts, top, ff, shared_ff; };
+// Lightning attention: SiLU on queries, keys and values, S <- decay S + k v^T per head, o = S^T q; an RMS norm over all heads, a gate per value.
+struct LightningConfig {
+    Index heads, dim, vdim;
+    std::vector<double> decay;   // [heads]
+};
+class LightningMixer : public Module {
+public:
+    LightningMixer(Index width, const LightningConfig& config, TensorOptions options);
+    const LightningConfig& config() const { return config_; }
+    Index inner() const { return config_.heads * config_.vdim; }
+    Index channels() const { return inner() + 2 * config_.heads * config_.dim; }
+    Tensor *q, *k, *v, *gate, *norm, *out;
+private:
+    LightningConfig config_;
+};
+
+// Two mixers on one input; the results are added, each with its factor.
+class SideBySideMixer : public Module {
+public:
+    SideBySideMixer(Index width, const GroupedAttentionConfig& left, const LightningConfig& right, double left_scale, double right_scale, TensorOptions options);
+    std::shared_ptr<GroupedAttentionMixer> left;
+    std::shared_ptr<LightningMixer> right;
+    double left_scale, right_scale;
+};
+
+// Experts of which every token takes the `top` with the largest scores.  identity: further outputs of the router whose expert hands its
+// input through.  shared_ff: units of an expert that runs for every token (0: none; gelu experts only).
+struct MixtureConfig {
+    Index experts, top, ff, shared_ff;
+    Index identity = 0;
+    MixtureKind kind = {};
+    Index outputs() const { return experts + identity; }
+};
 class MixtureOfExperts : public Module {
 public:
     MixtureOfExperts(Index width, const MixtureConfig& config, TensorOptions options);
     const MixtureConfig& config() const { return config_; }
-    std::vector<Tensor*> up, down;
-    Tensor *router, *shared_up = nullptr, *shared_down = nullptr;
+    std::vector<Tensor*> gate, up, down;
+    Tensor *router, *correction = nullptr, *shared_up = nullptr, *shared_down = nullptr;
 private:
     MixtureConfig config_;
 };
@@ -100,9 +169,13 @@ class HybridLayer : public Module {
 public:
     HybridLayer(Index width, const Json& spec, const DecoderDesign& design, TensorOptions options);
     RowNorm norm1, norm2;                           // norm2 only with a feed-forward after the mixer
-    std::shared_ptr<StateSpaceMixer> state_space;   // exactly one of the mixers
+    RowNorm after1, after2;                         // behind the sublayers (sandwich)
+    std::shared_ptr<StateSpaceMixer> state_space;   // exactly one of the mixers, or attention and lightning
     std::shared_ptr<LatentAttentionMixer> latent;
-    std::shared_ptr<ChunkedAttentionMixer> chunked;
+    std::shared_ptr<GroupedAttentionMixer> attention;
+    std::shared_ptr<LightningMixer> lightning;      // beside the attention, with their factors
+    double attention_scale = 1.0, lightning_scale = 1.0;
+    double unit_limit = 0.0;                        // clamped units of the dense feed-forward
     Tensor *gate = nullptr, *up = nullptr, *down = nullptr;   // dense feed-forward
     std::shared_ptr<MixtureOfExperts> mixture;
     bool has_mlp() const { return gate != nullptr; }
@@ -113,10 +186,12 @@ struct LayerRun {
     Index layer;
     Index pass;          // pass of the looped range, -1 outside
     bool begins_pass;    // first layer of a pass: the pass is entered before it (LoopEntry)
+    Index keys_run;      // the run whose keys and values it reads (attention: its own, or one before it)
 };
 
 // What the decoder keeps per sequence: slots of equal capacity, each with its length; per layer run a paged latent cache, a
-// convolution ring and a recurrent state, or the keys and values of one chunk.  A slot is given back by release(); its next sequence starts at position 0, where the
+// convolution ring and a recurrent state, or the keys and values of one chunk (of the whole sequence without chunks); and the last token,
+// where the embedding reads it.  A slot is given back by release(); its next sequence starts at position 0, where the
 // kernels read nothing old.
 class HybridDecoder;
 class HybridCache {
@@ -138,11 +213,12 @@ public:
     struct Run {
         b200_kv_cache* latent = nullptr;
         Tensor conv, state;      // [slots, taps, channels], [slots, heads, state, vdim]
-        Tensor key, value;       // [slots, kv_heads, entries, dim | vdim]
+        Tensor key, value;       // [slots, kv_heads, entries, dim | vdim]; none where another run's are read
         Index entries = 0;
     };
     const Run& run(std::size_t i) const { return runs_[i]; }
     std::int32_t* lengths() const { return static_cast<std::int32_t*>(lengths_.mutable_data()); }
+    std::int32_t* last_tokens() const { return static_cast<std::int32_t*>(last_.mutable_data()); }
     void commit(Index slot, Index count) { lengths_host_[static_cast<std::size_t>(slot)] += count; }
     struct Rotary { Tensor cosine, sine; };
     const Rotary& rotary(Index dims, double base) const { return tables_.at({dims, base}); }
@@ -152,7 +228,7 @@ private:
     Index capacity_;
     int device_;
     std::uint64_t id_;
-    Tensor lengths_;    // int32 payload [slots]
+    Tensor lengths_, last_;    // int32 payload [slots]
     std::vector<Index> lengths_host_;
     std::vector<Run> runs_;
     std::map<std::pair<Index, double>, Rotary> tables_;
@@ -184,6 +260,11 @@ public:
     double eps() const { return eps_; }
     double embedding_scale() const { return embedding_scale_; }
     double logit_scale() const { return logit_scale_; }
+    double logit_softcap() const { return logit_softcap_; }   // 0: none
+    // Table of token pairs (NULL: none), [buckets + 1, width]; the pair's row is (previous * mul_prev + token * mul_cur) mod buckets.
+    const Tensor* pairs() const { return pairs_; }
+    struct PairHash { Index buckets, mul_prev, mul_cur; };
+    const PairHash& pair_hash() const { return pair_hash_; }
     const std::vector<std::shared_ptr<HybridLayer>>& layers() const { return layers_; }
     const std::vector<LayerRun>& runs() const { return runs_; }
     const Tensor& embed() const { return *embed_; }
@@ -201,8 +282,9 @@ private:
     Index width_, vocab_;
     DType dtype_, activation_dtype_ = DType::f32;
     DecoderDesign design_;
-    double eps_, embedding_scale_, logit_scale_;
-    Tensor *embed_, *head_, *loop_step_ = nullptr, *loop_in_ = nullptr;
+    double eps_, embedding_scale_, logit_scale_, logit_softcap_ = 0.0;
+    PairHash pair_hash_{};
+    Tensor *embed_, *head_, *pairs_ = nullptr, *loop_step_ = nullptr, *loop_in_ = nullptr;
     RowNorm final_norm_;
     std::vector<std::shared_ptr<HybridLayer>> layers_;
     std::vector<LayerRun> runs_;

@@ -26,6 +26,10 @@ Tensor to_f32(const Tensor& t);
 //     feed-forward:      gate/up + SiLU * up -> down-projection + residual + next norm
 //     parallel layer:    [q | k | v | g | gate/up or router, shared up] projection -> norms, rotation, append, activation, router
 //                        -> attention + gate -> (experts + residual) -> [o | down] projection of both sublayers + residual + next norm
+//     sandwich layer:    [q | k | v | g | right g, v, k, q] projection -> norms, rotation, append -> attention + gate
+//                        -> (recurrence -> norm + gate) -> [o | right o] projection -> norm, residual, next norm
+//                        -> gate/up + clamped units -> down-projection -> norm, residual, next norm
+//                           or router -> experts, norm, residual, next norm
 // bf16 models run the projections on the shadow protocol (activations as bf16 hi + lo planes).  The projection that finishes the
 // residual stream also writes the next norm: a Dynamic Tanh norm as its result, an RMS norm as weighted rows and partial sums of
 // squares, from which the consumer takes the row's factor.  f32 models and sizes the shadow kernels do not take run the same kernels
@@ -39,6 +43,8 @@ public:
     bool shadows_for(Index rows) const;
     // ids on the device; `pass` describes the rows.  Leaves the residual stream in h_ and (shadow form) its final norm in the planes.
     void run(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail = nullptr);
+    // The rows of the last run become part of the cache.
+    void advance(const b200_rows& pass, HybridCache& cache, void* stream);
     // Logits of the last run's rows.
     void logits(Index rows, float* out, void* stream);
     // Logits of `count` rows of the last run, picked by device indices.
@@ -69,6 +75,13 @@ private:
         const void *uq, *w_value;
         Tensor conv, conv_bias, dt_bias, a_log, d, gated_norm, q_norm, kv_norm;   // f32
         Index wide_out, inner, mixed_out;           // rows of the first projection; input width of the out-projection
+        // grouped-query attention
+        Tensor q_bias, k_bias, sink;                // f32
+        // norms behind the sublayers, router and recurrence beside the attention (sandwich layers)
+        Norm after1, after2;
+        Tensor router, correction, decay, right_norm;
+        Index lightning_column = 0;                 // where its [g | v | k | q] start in a projected row
+        b200_clamped_unit unit{};
         // parallel layers
         Tensor joint, experts_up, experts_down;     // [o | down] columns side by side; the experts' matrices one below the other
         Index attention_columns = 0;                // rows of `wide` before the feed-forward's (q | k | v | g, padded)
@@ -78,22 +91,28 @@ private:
     // What a projection that finishes the residual stream leaves for its successor: a norm's planes, the rows' own planes, or nothing.
     struct After { const Norm* norm; bool raw; };
     Norm pack_norm(const RowNorm& n, double scale = 1.0) const;
+    void pack_attention(const GroupedAttentionMixer& mixer, Layer& layer) const;
+    void pack_experts(const MixtureOfExperts& mixture, Layer& layer) const;
     void pack_parallel(const HybridLayer& module, Layer& layer) const;
-    void reserve_parallel(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass);
+    void pack_sandwich(const HybridLayer& module, Layer& layer) const;
+    void reserve_attention(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass);
+    void run_sandwich(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail);
     // Everything of a parallel layer up to its out-projection; returns the residual that the out-projection adds to.
     const float* run_parallel(std::size_t run, const float* in, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream);
-    b200_chunk_args chunk_args(const Layer& layer, const ChunkedAttentionMixer& mixer, const HybridCache& cache, std::size_t run, Index stride) const;
+    b200_chunk_args chunk_args(const Layer& layer, const HybridLayer& module, const HybridCache& cache, std::size_t run, Index stride) const;
     b200_experts expert_args(const Layer& layer, const MixtureOfExperts& mixture, Index rows) const;
     // Dense feed-forwards of parallel layers: whether their units are projected together with the attention's inputs.
     bool units_beside(const HybridLayer& module, Index rows, bool planes) const;
 
     void linear(const float* x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y, void* stream, const char* what);
-    // `to` receives the planes of the result: of the `next` norm, of the result itself without one, of the SwiGLU units.
+    // `to` receives the planes of the result: of the `next` norm, of the result itself without one, of the gated units.
     void shadow(const Planes& x, Index rows, Index in, const void* w, Index out, b200_epilogue epilogue, const float* residual, float* y, const Norm* next,
-                Planes* to, void* stream, const char* what, Index to_column = 0, Index to_stride = 0);
+                Planes* to, void* stream, const char* what, Index to_column = 0, Index to_stride = 0, const b200_clamped_unit* unit = nullptr);
     void planes_of(const float* x, Index rows, const Norm& norm, Planes& to, void* stream);
     b200_latent_args latent_args(const Layer& layer, const LatentAttentionMixer& mixer, const HybridCache& cache, std::size_t run) const;
     void grow(Tensor& t, Shape shape, DType dtype);
+    // The rows of the stream as f32, for the trail.
+    void keep_rows(Index rows, std::vector<float>& trail) const;
     void grow(Planes& p, Index rows, Index width) { grow(p.hi, {rows, width}, DType::bf16); grow(p.lo, {rows, width}, DType::bf16); }
 
     HybridDecoder& owner_;
@@ -103,6 +122,8 @@ private:
     std::uint64_t packed_version_ = ~0ull, epoch_ = 0;
     const void* user_ = nullptr;
     Tensor first_, h_, projected_, mixed_, y_, query_, absorbed_, latent_out_, plain_, plain_inner_, scratch_;
+    Tensor branch_, route_logits_;            // a sublayer's result before the norm behind it; the router's outputs
+    const Index* ids_ = nullptr;              // of the last run
     Planes n_, i_, x_;                        // normed rows [rows, width]; inner rows (gated, attended, activated, query latent); the stream itself
     Tensor squares_;                          // [parts][rows]
     Tensor joined_first_, entered_;           // loop_first_ of the embedding output; the stream at the start of a pass

@@ -1,4 +1,5 @@
-// Parallel layers of the configured decoders: chunked attention and a feed-forward or a mixture of experts on one norm (see hybrid.h).
+// Grouped-query attention and mixtures of experts of the configured decoders, and their parallel layers: attention and a feed-forward or a
+// mixture on one norm (see hybrid.h).
 #include "dl/hybrid_plan.h"
 
 #include <algorithm>
@@ -15,37 +16,74 @@ Index round_up_8(Index n) { return (n + 7) & ~static_cast<Index>(7); }
 }  // namespace
 
 // ---- modules ------------------------------------------------------------------------------------------------
-ChunkedAttentionMixer::ChunkedAttentionMixer(Index width, const ChunkedAttentionConfig& c, TensorOptions options) : config_(c) {
-    if (c.heads % c.kv_heads) throw std::invalid_argument("chunked attention: heads must be a multiple of kv_heads");
-    if (c.rot_dims % 2 || c.rot_dims > c.dim) throw std::invalid_argument("chunked attention: rotated dimensions must be even and at most dim");
+GroupedAttentionMixer::GroupedAttentionMixer(Index width, const GroupedAttentionConfig& c, TensorOptions options) : config_(c) {
+    const AttentionKind& kind = c.kind;
+    if (c.heads % c.kv_heads) throw std::invalid_argument("grouped attention: heads must be a multiple of kv_heads");
+    if (c.rot_dims % 2 || c.rot_dims > c.dim) throw std::invalid_argument("grouped attention: rotated dimensions must be even and at most dim");
+    if (kind.keys_as_values && c.vdim != c.dim) throw std::invalid_argument("grouped attention: values that are the keys must have their size");
+    if (c.chunk > 0 && !own_keys()) throw std::invalid_argument("grouped attention: chunks need keys of the layer itself");
     q = &register_parameter("q", host_zeros({c.heads * c.dim, width}, options));
-    k = &register_parameter("k", host_zeros({c.kv_heads * c.dim, width}, options));
-    v = &register_parameter("v", host_zeros({c.kv_heads * c.vdim, width}, options));
-    q_norm = &register_parameter("q.norm", ones({c.heads * c.dim}, options));
-    k_norm = &register_parameter("k.norm", ones({c.kv_heads * c.dim}, options));
-    gate = &register_parameter("g", host_zeros({c.heads, width}, options));
+    if (kind.bias) q_bias = &register_parameter("q.b", host_zeros({c.heads * c.dim}, options));
+    if (own_keys()) {
+        k = &register_parameter("k", host_zeros({c.kv_heads * c.dim, width}, options));
+        if (kind.bias) k_bias = &register_parameter("k.b", host_zeros({c.kv_heads * c.dim}, options));
+        if (!kind.keys_as_values) v = &register_parameter("v", host_zeros({c.kv_heads * c.vdim, width}, options));
+    }
+    if (kind.norm == B200_HEAD_NORM_PROJECTION) {
+        q_norm = &register_parameter("q.norm", ones({c.heads * c.dim}, options));
+        if (own_keys()) k_norm = &register_parameter("k.norm", ones({c.kv_heads * c.dim}, options));
+    }
+    if (kind.sink == Sink::learned) sink = &register_parameter("sink", host_zeros({c.heads}, options));
+    if (kind.gate) gate = &register_parameter("g", host_zeros({c.heads, width}, options));
     out = &register_parameter("o", host_zeros({width, c.heads * c.vdim}, options));
 }
-Index ChunkedAttentionMixer::columns() const { return config_.heads * (config_.dim + 1) + config_.kv_heads * (config_.dim + config_.vdim); }
+Index GroupedAttentionMixer::columns() const {
+    Index count = 0;
+    for (const Tensor* t : {q, k, v, gate})
+        if (t) count += t->size(0);
+    return count;
+}
 
 MixtureOfExperts::MixtureOfExperts(Index width, const MixtureConfig& c, TensorOptions options) : config_(c) {
-    if (c.top > c.experts) throw std::invalid_argument("mixture of experts: 'top' exceeds the number of experts");
-    if (c.experts > B200_MAX_EXPERTS) throw std::invalid_argument("mixture of experts: more than " + std::to_string(B200_MAX_EXPERTS) + " experts");
+    if (c.identity < 0) throw std::invalid_argument("mixture of experts: a negative number of identity experts");
+    if (c.top > c.outputs()) throw std::invalid_argument("mixture of experts: 'top' exceeds the number of experts");
+    if (c.outputs() > B200_MAX_EXPERTS) throw std::invalid_argument("mixture of experts: more than " + std::to_string(B200_MAX_EXPERTS) + " experts");
     for (Index e = 0; e < c.experts; ++e) {
         const std::string name = "e" + std::to_string(e);
+        if (c.kind.gated) gate.push_back(&register_parameter(name + ".gate", host_zeros({c.ff, width}, options)));
         up.push_back(&register_parameter(name + ".up", host_zeros({c.ff, width}, options)));
         down.push_back(&register_parameter(name + ".down", host_zeros({width, c.ff}, options)));
     }
-    router = &register_parameter("router", host_zeros({c.experts, width}, options));
+    router = &register_parameter("router", host_zeros({c.outputs(), width}, options));
+    if (c.kind.correction) correction = &register_parameter("correction", host_zeros({c.outputs()}, options));
     if (c.shared_ff > 0) {
+        if (c.kind.gated) throw std::invalid_argument("mixture of experts: a shared expert is not combined with gated experts");
         shared_up = &register_parameter("shared.up", host_zeros({c.shared_ff, width}, options));
         shared_down = &register_parameter("shared.down", host_zeros({width, c.shared_ff}, options));
     }
 }
 
 // ---- plan ---------------------------------------------------------------------------------------------------
+void HybridPlan::pack_attention(const GroupedAttentionMixer& m, Layer& l) const {
+    if (m.q_norm) l.q_norm = to_f32(*m.q_norm);
+    if (m.k_norm) l.kv_norm = to_f32(*m.k_norm);
+    if (m.q_bias) l.q_bias = to_f32(*m.q_bias);
+    if (m.k_bias) l.k_bias = to_f32(*m.k_bias);
+    if (m.sink) l.sink = to_f32(*m.sink);
+    else if (m.config().kind.sink == Sink::zero) l.sink = zeros({m.config().heads}, {DType::f32, m.q->device()});
+}
+
+void HybridPlan::pack_experts(const MixtureOfExperts& e, Layer& l) const {
+    std::vector<Tensor> ups, downs;
+    for (std::size_t i = 0; i < e.up.size(); ++i) ups.push_back(e.gate.empty() ? *e.up[i] : interleave_rows(*e.gate[i], *e.up[i]));
+    for (const Tensor* t : e.down) downs.push_back(*t);
+    l.experts_up = concat_rows(ups);
+    l.experts_down = concat_rows(downs);
+    if (e.correction) l.correction = to_f32(*e.correction);
+}
+
 void HybridPlan::pack_parallel(const HybridLayer& module, Layer& l) const {
-    const ChunkedAttentionMixer& m = *module.chunked;
+    const GroupedAttentionMixer& m = *module.attention;
     const Index D = owner_.width();
     const TensorOptions options{owner_.dtype(), m.q->device()};
     std::vector<Tensor> rows{*m.q, *m.k, *m.v, *m.gate}, columns{*m.out};
@@ -77,11 +115,7 @@ void HybridPlan::pack_parallel(const HybridLayer& module, Layer& l) const {
             count += l.units;
             pad();
         }
-        std::vector<Tensor> ups, downs;
-        for (const Tensor* t : e.up) ups.push_back(*t);
-        for (const Tensor* t : e.down) downs.push_back(*t);
-        l.experts_up = concat_rows(ups);
-        l.experts_down = concat_rows(downs);
+        pack_experts(e, l);
     }
     l.wide = concat_rows(rows);
     l.in = l.wide.raw_data();
@@ -90,15 +124,16 @@ void HybridPlan::pack_parallel(const HybridLayer& module, Layer& l) const {
     l.joint = columns.size() == 1 ? columns.front() : concat_columns(columns);
     l.out = l.joint.raw_data();
     l.inner = l.attended + l.units;
-    l.q_norm = to_f32(*m.q_norm);
-    l.kv_norm = to_f32(*m.k_norm);
+    pack_attention(m, l);
 }
 
 bool HybridPlan::units_beside(const HybridLayer& module, Index rows, bool planes) const { return !module.has_mlp() || !planes || rows <= kRowsBeside; }
 
-b200_chunk_args HybridPlan::chunk_args(const Layer& layer, const ChunkedAttentionMixer& mixer, const HybridCache& cache, std::size_t run, Index stride) const {
-    const auto& c = mixer.config();
-    const HybridCache::Run& r = cache.run(run);
+b200_chunk_args HybridPlan::chunk_args(const Layer& layer, const HybridLayer& module, const HybridCache& cache, std::size_t run, Index stride) const {
+    const auto& c = module.attention->config();
+    const HybridCache::Run& r = cache.run(static_cast<std::size_t>(owner_.runs()[run].keys_run));
+    auto vector = [](const Tensor& t) { return t.defined() ? t.data<float>() : nullptr; };
+    auto workspace = [](const Tensor& t) { return t.defined() ? t.mutable_data() : nullptr; };
     b200_chunk_args a{};
     a.heads = static_cast<int32_t>(c.heads); a.kv_heads = static_cast<int32_t>(c.kv_heads); a.dim = static_cast<int32_t>(c.dim);
     a.vdim = static_cast<int32_t>(c.vdim); a.rot_dims = static_cast<int32_t>(c.rot_dims);
@@ -110,11 +145,15 @@ b200_chunk_args HybridPlan::chunk_args(const Layer& layer, const ChunkedAttentio
         const auto& table = cache.rotary(c.rot_dims, c.rot_base);
         a.cosine = table.cosine.data<float>(); a.sine = table.sine.data<float>(); a.positions = static_cast<int32_t>(table.cosine.size(0));
     }
-    a.q_norm = layer.q_norm.data<float>(); a.k_norm = layer.kv_norm.data<float>();
+    a.q_norm = vector(layer.q_norm); a.k_norm = vector(layer.kv_norm); a.q_bias = vector(layer.q_bias); a.k_bias = vector(layer.k_bias);
+    a.sink = vector(layer.sink);
+    a.norm = c.kind.norm; a.rotate_pairs = c.kind.rotate_pairs; a.keys_as_values = c.kind.keys_as_values; a.keys_elsewhere = !module.attention->own_keys();
+    a.no_gate = !c.kind.gate; a.softcap = static_cast<float>(c.softcap);
+    a.scaled = 1; a.out_scale = static_cast<float>(module.attention_scale);
     a.dtype = code_of(owner_.dtype());
     a.key_cache = r.key.mutable_data(); a.value_cache = r.value.mutable_data();
     a.projected = projected_.data<float>(); a.stride = stride;
-    a.query = chunk_query_.mutable_data(); a.key = chunk_key_.mutable_data(); a.value = chunk_value_.mutable_data();
+    a.query = chunk_query_.mutable_data(); a.key = workspace(chunk_key_); a.value = workspace(chunk_value_);
     return a;
 }
 
@@ -133,19 +172,22 @@ b200_experts HybridPlan::expert_args(const Layer& layer, const MixtureOfExperts&
         a.x = f32(plain_);
     }
     a.eps = owner_.eps();
+    a.gated = c.kind.gated; a.weigh_results = c.kind.weigh_results; a.identity = static_cast<int32_t>(c.identity);
     a.residual = f32(h_); a.y = f32(h_);
     return a;
 }
 
-void HybridPlan::reserve_parallel(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass) {
+void HybridPlan::reserve_attention(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass) {
     grouped_ = false;
     Index query = 0, key = 0, value = 0, slots = 0, act = 0, most_experts = 0;
     for (const auto& module : owner_.layers()) {
-        if (module->chunked) {
-            const auto& c = module->chunked->config();
+        if (module->attention) {
+            const auto& c = module->attention->config();
             query = std::max(query, c.heads * c.dim);
-            key = std::max(key, c.kv_heads * c.dim);
-            value = std::max(value, c.kv_heads * c.vdim);
+            if (c.chunk > 0) {   // without chunks the rows go into the slots at once
+                key = std::max(key, c.kv_heads * c.dim);
+                value = std::max(value, c.kv_heads * c.vdim);
+            }
         }
         if (module->mixture) {
             const auto& c = module->mixture->config();
@@ -156,8 +198,7 @@ void HybridPlan::reserve_parallel(Index rows, Index max_length, const HybridCach
     }
     if (query == 0) return;
     grow(chunk_query_, {rows, query}, owner_.dtype());
-    grow(chunk_key_, {rows, key}, owner_.dtype());
-    grow(chunk_value_, {rows, value}, owner_.dtype());
+    if (key) { grow(chunk_key_, {rows, key}, owner_.dtype()); grow(chunk_value_, {rows, value}, owner_.dtype()); }
     if (slots) {
         grow(chosen_, {rows, slots}, DType::f32);   // int32 payload
         grow(rank_, {rows, slots}, DType::f32);
@@ -169,8 +210,8 @@ void HybridPlan::reserve_parallel(Index rows, Index max_length, const HybridCach
     for (std::size_t i = 0; i < owner_.runs().size(); ++i) {
         const auto index = static_cast<std::size_t>(owner_.runs()[i].layer);
         const HybridLayer& module = *owner_.layers()[index];
-        if (module.chunked) {
-            const b200_chunk_args a = chunk_args(layers_[index], *module.chunked, cache, i, layers_[index].wide_out);
+        if (module.attention) {
+            const b200_chunk_args a = chunk_args(layers_[index], module, cache, i, layers_[index].wide_out);
             scratch = std::max(scratch, b200_chunk_scratch_bytes(&a, rows, pass.sequences, pass.max_count, static_cast<int32_t>(max_length)));
         }
         if (module.mixture) {
@@ -200,7 +241,7 @@ const float* HybridPlan::run_parallel(std::size_t run, const float* in, const b2
         shadow(n_, rows, D, gate_up, 2 * layer.units, B200_EPI_SWIGLU, nullptr, nullptr, nullptr, &i_, stream, "gate/up projection", layer.attended, layer.inner);
     }
 
-    const b200_chunk_args a = chunk_args(layer, *module.chunked, cache, run, stride);
+    const b200_chunk_args a = chunk_args(layer, module, cache, run, stride);
     float* inner_plain = planes ? nullptr : f32(plain_inner_);
     auto* inner_hi = planes ? static_cast<std::uint16_t*>(i_.hi.mutable_data()) : nullptr;
     auto* inner_lo = planes ? static_cast<std::uint16_t*>(i_.lo.mutable_data()) : nullptr;
@@ -228,7 +269,7 @@ const float* HybridPlan::run_parallel(std::size_t run, const float* in, const b2
     runtime::check(b200_chunk_prepare(&a, &pass, &units, &route, stream), "attention norms");
     probe(2);
     runtime::check(b200_chunk_attention(&a, &pass, static_cast<int32_t>(max_length), scratch_.mutable_data(), scratch_.nbytes(), inner_plain, inner_hi, inner_lo,
-                                        layer.inner, stream), "chunked attention");
+                                        layer.inner, stream), "grouped attention");
     probe(1);
     if (!module.mixture) return in;
     if (grouped) runtime::check(b200_experts_grouped(&experts, route.rank, route.counts, expert_scratch_.mutable_data(), expert_scratch_.nbytes(), stream), "experts");

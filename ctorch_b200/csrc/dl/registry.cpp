@@ -12,11 +12,28 @@ namespace {
 
 using Factory = std::shared_ptr<nn::UnaryModule> (*)(const Json&, TensorOptions);
 
+using nn::MixerKind;
+
+constexpr nn::MixerDesign kHybridMixers[] = {{"mamba2", MixerKind::state_space}, {"latent_attention", MixerKind::latent}};
+constexpr nn::MixerDesign kParallelMixers[] = {{"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_PROJECTION, .gate = true}}};
+constexpr nn::MixerDesign kSandwichMixers[] = {
+    {"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_NONE, .rotate_pairs = true, .bias = true, .keys_as_values = true, .gate = true, .sink = nn::Sink::zero}},
+    {"attention_2", MixerKind::attention, {.norm = B200_HEAD_NORM_HEAD, .rotate_pairs = true, .sink = nn::Sink::learned}},
+    {"parallel", MixerKind::side_by_side, {.norm = B200_HEAD_NORM_PROJECTION, .gate = true, .sink = nn::Sink::learned}},
+};
+
 std::shared_ptr<nn::UnaryModule> hybrid(const Json& config, TensorOptions options) {
-    return std::make_shared<nn::HybridDecoder>(config, nn::DecoderDesign{nn::NormKind::dynamic_tanh, nn::LoopEntry::step, false, true}, options);
+    return std::make_shared<nn::HybridDecoder>(
+        config, nn::DecoderDesign{nn::NormKind::dynamic_tanh, nn::LoopEntry::step, nn::LayerForm::sequential, true, kHybridMixers, std::nullopt}, options);
 }
 std::shared_ptr<nn::UnaryModule> parallel(const Json& config, TensorOptions options) {
-    return std::make_shared<nn::HybridDecoder>(config, nn::DecoderDesign{nn::NormKind::rms, nn::LoopEntry::joined, true, false}, options);
+    return std::make_shared<nn::HybridDecoder>(
+        config, nn::DecoderDesign{nn::NormKind::rms, nn::LoopEntry::joined, nn::LayerForm::parallel, false, kParallelMixers, nn::MixtureKind{}}, options);
+}
+std::shared_ptr<nn::UnaryModule> sandwich(const Json& config, TensorOptions options) {
+    return std::make_shared<nn::HybridDecoder>(
+        config, nn::DecoderDesign{nn::NormKind::rms_from_one, nn::LoopEntry::joined, nn::LayerForm::sandwich, false, kSandwichMixers,
+                                  nn::MixtureKind{.softmax = true, .correction = true, .gated = true, .weigh_results = true}, 1.702}, options);
 }
 
 // Grouped-query decoder with its embedding and output layers, under the names of the reference's example model.
@@ -29,6 +46,7 @@ std::shared_ptr<nn::UnaryModule> transformer(const Json& c, TensorOptions option
 
 struct Entry { const char* name; Factory make; };
 constexpr Entry kRegistry[] = {
+    {"Lozepel", sandwich},
     {"Ripitar", hybrid},
     {"Sinezen", parallel},
     {"TransformerDecoder", transformer},

@@ -1,21 +1,24 @@
-// Chunked grouped-query attention: a position sees its own chunk of positions up to itself, so a slot keeps one chunk of keys and
-// values ([slot][kv_head][entry][dim], position p in entry p mod chunk) however long the sequence grows, and what a step reads is one
-// contiguous block per (sequence, kv head).  Keys and values may have different widths.
+// Grouped-query attention over slots.  With chunks a position sees its own chunk of positions up to itself, so a slot keeps one chunk of
+// keys and values ([slot][kv_head][entry][dim], position p in entry p mod chunk) however long the sequence grows; without chunks it keeps
+// all of them.  What a step reads is one contiguous block per (sequence, kv head).  Keys and values may have different widths.
 //
-//   * chunk_prepare_kernel, one CTA per row (and one per slice of its feed-forward units): RMS norms over all query and all key heads, rotation of halves, append (or the
-//     workspaces of a longer pass), the activation of feed-forward units and the router's choice for the same row.
+//   * chunk_prepare_kernel, one CTA per row (and one per slice of its feed-forward units): biases, RMS norms (over all heads at once or per
+//     head), rotation of halves or of adjacent pairs, append (or the workspaces of a longer pass), the activation of feed-forward units and
+//     the router's choice for the same row.
 //   * chunk_step_kernel, chunk_mma_kernel: bf16, mma.sync products, online softmax in f32 registers, weights as hi + lo planes, the heads
-//     of a group side by side so that a key is fetched once for all of them.
+//     of a group side by side so that a key is fetched once for all of them.  Scores may be capped (softcap * tanh), and the denominator
+//     may hold a term without a key (sink), which joins the sums when a row is finished.
 //       steps (one row per sequence): bound by the keys' bytes.  Persistent CTAs walk (sequence, kv head, split) items; a producer warp
 //         streams tiles of 64 keys and values through a TMA ring (boxes of 64 x 64, 128-byte swizzle, mbarrier completion) and runs
 //         into the next item while four consumer warps, which divide the keys of a tile, merge the current one.  Keys are split over
 //         CTAs, with a merge kernel, where the items do not fill the SMs;
 //       longer passes: 64 rows = positions x heads of a group, 16 per warp, a cp.async double buffer; keys before the pass come from the
-//         slot, the pass's own keys from its workspaces.
+//         slot, the pass's own keys from its workspaces (from the slot too without chunks, where they are appended first).
 //   * chunk_generic_kernel: f32 and odd sizes, f32 FMAs, one (row, head) per CTA.
 //   * chunk_append_kernel: a longer pass that begins inside a chunk and ends in another one reads the old chunk from the slot; its last
 //     rows go there afterwards.
 #include "mma.cuh"
+#include "router.cuh"
 #include "rows.cuh"
 
 #include <algorithm>
@@ -33,6 +36,14 @@ struct ChunkParams {
     void *key_cache, *value_cache, *query, *key, *value;
     const float* projected;
     int64_t stride;
+    const float *q_bias, *k_bias, *sink;
+    int norm;
+    bool rotate_pairs, keys_as_values, keys_elsewhere, gated;
+    float softcap, out_scale;
+    __host__ __device__ __forceinline__ int key_columns() const { return keys_elsewhere ? 0 : kv_heads * dim; }
+    __host__ __device__ __forceinline__ int value_columns() const { return keys_elsewhere || keys_as_values ? 0 : kv_heads * vdim; }
+    // Keys of the pass itself are in the slots before the attention starts.
+    __host__ __device__ __forceinline__ bool appends_first(bool step) const { return step || chunk == 0; }
     __device__ __forceinline__ int chunk_start(int position) const { return chunk > 0 ? position - position % chunk : 0; }
     // where (slot, kv head)'s entry of a position begins, in units of one entry
     __device__ __forceinline__ int64_t entry(int slot, int head, int position) const {
@@ -45,19 +56,27 @@ struct ChunkParams {
 
 bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
     if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)
-        || a->rot_dims > a->dim || a->slots <= 0 || a->chunk < 0 || a->entries <= 0 || (a->rot_dims > 0 && (!a->cosine || !a->sine)) || !a->q_norm || !a->k_norm
+        || a->rot_dims > a->dim || a->slots <= 0 || a->chunk < 0 || a->entries <= 0 || (a->rot_dims > 0 && (!a->cosine || !a->sine))
+        || (a->norm == B200_HEAD_NORM_PROJECTION && (!a->q_norm || (!a->k_norm && !a->keys_elsewhere)))
+        || a->norm < B200_HEAD_NORM_PROJECTION || a->norm > B200_HEAD_NORM_HEAD || (a->keys_elsewhere && a->chunk > 0)
+        || (a->keys_as_values && (a->vdim != a->dim || a->norm != B200_HEAD_NORM_NONE)) || !(a->softcap >= 0.0f)
         || (a->dtype != B200_F32 && a->dtype != B200_BF16) || !a->key_cache || !a->value_cache || !a->projected || !a->query || a->stride <= 0) {
-        set_error("chunked attention: bad pointer or size");
+        set_error("grouped attention: bad pointer or size");
         return false;
     }
     p = ChunkParams{a->heads, a->kv_heads, a->heads / a->kv_heads, a->dim, a->vdim, a->rot_dims, a->slots, a->chunk, a->entries, a->scale, static_cast<float>(a->eps),
-                    a->cosine, a->sine, a->positions, a->q_norm, a->k_norm, a->key_cache, a->value_cache, a->query, a->key, a->value, a->projected, a->stride};
+                    a->cosine, a->sine, a->positions, a->q_norm, a->k_norm, a->key_cache, a->value_cache, a->query, a->key, a->value, a->projected, a->stride,
+                    a->q_bias, a->k_bias, a->sink, a->norm, a->rotate_pairs != 0, a->keys_as_values != 0, a->keys_elsewhere != 0, a->no_gate == 0, a->softcap,
+                    a->scaled ? a->out_scale : 1.0f};
+    if (p.heads * p.dim + p.key_columns() + p.value_columns() + (p.gated ? p.heads : 0) > p.stride) {
+        set_error("grouped attention: the projected rows are shorter than the heads");
+        return false;
+    }
     return true;
 }
 
 // ---- between the projection and the attention -----------------------------------------------------------------------
 struct Units { int kind; int64_t column; int count; float* out; __nv_bfloat16 *out_hi, *out_lo; int64_t stride; };
-struct Route { int experts, top; int64_t column; int32_t* chosen; float* weight; int32_t *rank, *counts; };
 
 template <int V> struct Span { float v[V]; };
 template <int V> __device__ __forceinline__ Span<V> load_span(const float* p) {
@@ -78,63 +97,69 @@ template <int V> __device__ __forceinline__ void store_span(__nv_bfloat16* p, co
     if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(s.v[0], s.v[1]), pack_bf16(s.v[2], s.v[3]));
     else *p = __float2bfloat16_rn(s.v[0]);
 }
-template <int V> __device__ __forceinline__ float squares_of(const float* x, int count) {
+// Entries [c, c + V) of a projected row's part, with its bias.
+template <int V> __device__ __forceinline__ Span<V> biased_span(const float* x, const float* bias, int c) {
+    Span<V> s = load_span<V>(x + c);
+    if (bias) {
+        const Span<V> b = load_span<V>(bias + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) s.v[i] += b.v[i];
+    }
+    return s;
+}
+// This thread's share of the sum of squares of entries [begin, end), `threads` threads side by side.
+template <int V> __device__ __forceinline__ float squares_of(const float* x, const float* bias, int begin, int end, int thread, int threads) {
     float total = 0.0f;
-    for (int c = threadIdx.x * V; c < count; c += blockDim.x * V) {
-        const Span<V> s = load_span<V>(x + c);
+    for (int c = begin + thread * V; c < end; c += threads * V) {
+        const Span<V> s = biased_span<V>(x, bias, c);
 #pragma unroll
         for (int i = 0; i < V; ++i) total = fmaf(s.v[i], s.v[i], total);
     }
     return total;
 }
-// V entries of a head from entry d on: normed, weighted, and turned by the row's angles (entry i with entry i + rot_dims / 2).
+// V entries from entry c of a part on, which is entry d of its head: with bias, normed, weighted (weight may be NULL), and turned by the
+// row's angles - entry i with entry i + rot_dims / 2, or entry 2i with entry 2i + 1.
 template <int V>
-__device__ __forceinline__ Span<V> turned_span(const ChunkParams& p, const float* head, const float* weight, int d, float inverse, const float* cosine,
-                                               const float* sine) {
+__device__ __forceinline__ Span<V> turned_span(const ChunkParams& p, const float* part, const float* bias, const float* weight, int c, int d, float inverse,
+                                               const float* cosine, const float* sine) {
     auto normed = [&](int at) {
-        Span<V> s = load_span<V>(head + at);
-        const Span<V> w = load_span<V>(weight + at);
+        Span<V> s = biased_span<V>(part, bias, at);
+        if (weight) {
+            const Span<V> w = load_span<V>(weight + at);
 #pragma unroll
-        for (int i = 0; i < V; ++i) s.v[i] = s.v[i] * inverse * w.v[i];
+            for (int i = 0; i < V; ++i) s.v[i] = s.v[i] * inverse * w.v[i];
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; ++i) s.v[i] *= inverse;
+        }
         return s;
     };
-    Span<V> own = normed(d);
+    Span<V> own = normed(c);
     if (d >= p.rot_dims || !cosine) return own;
+    if (p.rotate_pairs) {
+        if constexpr (V == 1) {
+            const float other = normed(d & 1 ? c - 1 : c + 1).v[0], cs = cosine[d >> 1], sn = sine[d >> 1];
+            own.v[0] = d & 1 ? __fadd_rn(__fmul_rn(own.v[0], cs), __fmul_rn(other, sn)) : __fsub_rn(__fmul_rn(own.v[0], cs), __fmul_rn(other, sn));
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; i += 2) {
+                if (d + i >= p.rot_dims) break;
+                const float cs = cosine[(d + i) >> 1], sn = sine[(d + i) >> 1], u = own.v[i], v = own.v[i + 1];
+                own.v[i] = __fsub_rn(__fmul_rn(u, cs), __fmul_rn(v, sn));
+                own.v[i + 1] = __fadd_rn(__fmul_rn(v, cs), __fmul_rn(u, sn));
+            }
+        }
+        return own;
+    }
     const int half = p.rot_dims >> 1;
     const bool upper = d >= half;
-    const Span<V> other = normed(upper ? d - half : d + half);
-    const Span<V> c = load_span<V>(cosine + (upper ? d - half : d)), s = load_span<V>(sine + (upper ? d - half : d));
+    const Span<V> other = normed(upper ? c - half : c + half);
+    const Span<V> cs = load_span<V>(cosine + (upper ? d - half : d)), sn = load_span<V>(sine + (upper ? d - half : d));
 #pragma unroll
     for (int i = 0; i < V; ++i)
-        own.v[i] = upper ? __fadd_rn(__fmul_rn(own.v[i], c.v[i]), __fmul_rn(other.v[i], s.v[i]))
-                         : __fsub_rn(__fmul_rn(own.v[i], c.v[i]), __fmul_rn(other.v[i], s.v[i]));
+        own.v[i] = upper ? __fadd_rn(__fmul_rn(own.v[i], cs.v[i]), __fmul_rn(other.v[i], sn.v[i]))
+                         : __fsub_rn(__fmul_rn(own.v[i], cs.v[i]), __fmul_rn(other.v[i], sn.v[i]));
     return own;
-}
-
-// The `top` experts with the largest logits (the scores grow with them), the lower index among equals, by one warp.
-__device__ __forceinline__ void choose_experts(const Route& r, int row, const float* logits, float* copy, int lane) {
-    for (int e = lane; e < r.experts; e += 32) copy[e] = logits[e];
-    __syncwarp();
-    for (int k = 0; k < r.top; ++k) {
-        float best = -INFINITY;
-        int at = INT32_MAX;
-        for (int e = lane; e < r.experts; e += 32)
-            if (copy[e] > best || at == INT32_MAX) { best = copy[e]; at = e; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float other = __shfl_xor_sync(0xffffffffu, best, o);
-            const int other_at = __shfl_xor_sync(0xffffffffu, at, o);
-            if (other_at != INT32_MAX && (at == INT32_MAX || other > best || (other == best && other_at < at))) { best = other; at = other_at; }
-        }
-        if (lane == 0) {
-            const int64_t slot = static_cast<int64_t>(row) * r.top + k;
-            r.chosen[slot] = at;
-            r.weight[slot] = 1.0f / (1.0f + expf(-logits[at]));
-            if (r.rank) r.rank[slot] = atomicAdd(r.counts + at, 1);
-            copy[at] = -INFINITY;
-        }
-        __syncwarp();
-    }
 }
 
 constexpr int kPrepareThreads = 256, kUnitSlice = 1024;
@@ -143,7 +168,7 @@ constexpr int kPrepareThreads = 256, kUnitSlice = 1024;
 template <class T, int V>
 __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __grid_constant__ ChunkParams p, const RowsView rows, const bool step,
                                                                         const __grid_constant__ Units units, const __grid_constant__ Route route) {
-    extern __shared__ float logits_copy[];
+    extern __shared__ float extra[];   // [experts] for the router, then one factor per query and key head
     __shared__ float scratch[32];
     grid_dependency_wait();
     grid_launch_dependents();
@@ -185,47 +210,64 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
         return;
     }
     if (route.experts > 0 && threadIdx.x >= kPrepareThreads - 32)
-        choose_experts(route, row, source + route.column, logits_copy, threadIdx.x & 31);
-    // where the row belongs: a chain of dependent loads, spread between the sums
+        choose_experts(route, row, source + route.column, extra, threadIdx.x & 31);
     const int sequence = __ldg(rows.sequence + row);
-    const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
-    const float *k_source = source + q_count, *v_source = k_source + k_count;
-    float qs = squares_of<V>(source, q_count), ks = squares_of<V>(k_source, k_count);
+    const int q_count = p.heads * p.dim, k_count = p.key_columns(), v_count = p.keys_elsewhere ? 0 : p.kv_heads * p.vdim;
+    const float *k_source = source + q_count, *v_source = p.keys_as_values ? k_source : k_source + k_count;
+    const float* v_bias = p.keys_as_values ? p.k_bias : nullptr;
     const int slot = __ldg(rows.slot + sequence), first = __ldg(rows.first + sequence), end = __ldg(rows.first + sequence + 1);
-    qs = warp_sum(qs);
-    ks = warp_sum(ks);
     const int length = rows.lengths[slot];
-    if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = qs; scratch[kPrepareThreads / 32 + (threadIdx.x >> 5)] = ks; }
-    __syncthreads();
-    qs = ks = 0.0f;
+    float q_inverse = 1.0f, k_inverse = 1.0f;
+    float* inverses = extra + route.experts;   // (norm per head)
+    if (p.norm == B200_HEAD_NORM_PROJECTION) {
+        const float qs = warp_sum(squares_of<V>(source, p.q_bias, 0, q_count, threadIdx.x, kPrepareThreads));
+        const float ks = warp_sum(squares_of<V>(k_source, p.k_bias, 0, k_count, threadIdx.x, kPrepareThreads));
+        if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = qs; scratch[kPrepareThreads / 32 + (threadIdx.x >> 5)] = ks; }
+        __syncthreads();
+        float q_total = 0.0f, k_total = 0.0f;
 #pragma unroll
-    for (int w = 0; w < kPrepareThreads / 32; ++w) { qs += scratch[w]; ks += scratch[kPrepareThreads / 32 + w]; }
+        for (int w = 0; w < kPrepareThreads / 32; ++w) { q_total += scratch[w]; k_total += scratch[kPrepareThreads / 32 + w]; }
+        q_inverse = 1.0f / sqrtf(q_total / static_cast<float>(q_count) + p.eps);
+        k_inverse = 1.0f / sqrtf(k_total / static_cast<float>(max(k_count, 1)) + p.eps);
+    } else if (p.norm == B200_HEAD_NORM_HEAD) {
+        const int heads = p.heads + (p.keys_elsewhere ? 0 : p.kv_heads);   // the key heads follow the query heads in the row
+        for (int h = threadIdx.x >> 5; h < heads; h += kPrepareThreads / 32) {
+            const bool is_query = h < p.heads;
+            const int begin = (is_query ? h : h - p.heads) * p.dim;
+            const float squares = warp_sum(squares_of<V>(is_query ? source : k_source, is_query ? p.q_bias : p.k_bias, begin, begin + p.dim, threadIdx.x & 31, 32));
+            if ((threadIdx.x & 31) == 0) inverses[h] = 1.0f / sqrtf(squares / static_cast<float>(p.dim) + p.eps);
+        }
+        __syncthreads();
+    }
     const int position = length + row - first, last = length + end - first - 1;
     // The slot takes the row at once where it ends up there and nothing that this pass still reads is overwritten.
-    const bool stored = step || (p.chunk_start(position) == p.chunk_start(last) && !p.overwrites(length, last));
-    const float q_inverse = 1.0f / sqrtf(qs / static_cast<float>(q_count) + p.eps);
-    const float k_inverse = 1.0f / sqrtf(ks / static_cast<float>(k_count) + p.eps);
+    const bool first_appended = p.appends_first(step);
+    const bool stored = first_appended || (p.chunk_start(position) == p.chunk_start(last) && !p.overwrites(length, last));
     const int half = p.rot_dims >> 1;
     const bool turns = half > 0 && position < p.positions;
     const float* cosine = turns ? p.cosine + static_cast<int64_t>(position) * half : nullptr;
     const float* sine = turns ? p.sine + static_cast<int64_t>(position) * half : nullptr;
+    const float* q_weight = p.norm == B200_HEAD_NORM_PROJECTION ? p.q_norm : nullptr;
+    const float* k_weight = p.norm == B200_HEAD_NORM_PROJECTION ? p.k_norm : nullptr;
     for (int c = threadIdx.x * V; c < q_count; c += kPrepareThreads * V) {
         const int head = c / p.dim, d = c - head * p.dim;
+        const float inverse = p.norm == B200_HEAD_NORM_HEAD ? inverses[head] : q_inverse;
         store_span<V>(static_cast<T*>(p.query) + static_cast<int64_t>(row) * q_count + c,
-                      turned_span<V>(p, source + head * p.dim, p.q_norm + head * p.dim, d, q_inverse, cosine, sine));
+                      turned_span<V>(p, source, p.q_bias, q_weight, c, d, inverse, cosine, sine));
     }
     const bool to_slot = stored && p.fits(position);   // (the host refuses passes that do not fit)
     for (int c = threadIdx.x * V; c < k_count; c += kPrepareThreads * V) {
         const int head = c / p.dim, d = c - head * p.dim;
-        const Span<V> v = turned_span<V>(p, k_source + head * p.dim, p.k_norm + head * p.dim, d, k_inverse, cosine, sine);
+        const float inverse = p.norm == B200_HEAD_NORM_HEAD ? inverses[p.heads + head] : k_inverse;
+        const Span<V> v = turned_span<V>(p, k_source, p.k_bias, k_weight, c, d, inverse, cosine, sine);
         if (to_slot) store_span<V>(static_cast<T*>(p.key_cache) + p.entry(slot, head, position) * p.dim + d, v);
-        if (!step) store_span<V>(static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + c, v);
+        if (!first_appended) store_span<V>(static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + c, v);
     }
     for (int c = threadIdx.x * V; c < v_count; c += kPrepareThreads * V) {
         const int head = c / p.vdim, d = c - head * p.vdim;
-        const Span<V> v = load_span<V>(v_source + c);
+        const Span<V> v = biased_span<V>(v_source, v_bias, c);
         if (to_slot) store_span<V>(static_cast<T*>(p.value_cache) + p.entry(slot, head, position) * p.vdim + d, v);
-        if (!step) store_span<V>(static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + c, v);
+        if (!first_appended) store_span<V>(static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + c, v);
     }
 }
 
@@ -262,9 +304,25 @@ struct ChunkAttention {
     int64_t out_stride;
 };
 
+// Factor of a head's result: its gate, and the layer's scale.
 __device__ __forceinline__ float head_gate(const ChunkParams& p, int row, int head) {
-    const float g = __ldg(p.projected + row * p.stride + p.heads * p.dim + p.kv_heads * (p.dim + p.vdim) + head);
-    return 1.0f / (1.0f + expf(-g));
+    if (!p.gated) return p.out_scale;
+    const float g = __ldg(p.projected + row * p.stride + p.heads * p.dim + p.key_columns() + p.value_columns() + head);
+    return p.out_scale / (1.0f + expf(-g));
+}
+// The scores are kept in units of log2: `scale2` times the product, or cap2 * tanh(product * scale / softcap).  The tensor-core kernels take
+// the hardware's exponential and reciprocal (an error near 1e-6 of the cap), the plain one the exact functions.
+__device__ __forceinline__ float capped_score(float product, float scale_by_cap, float cap2) {
+    const float e = exp2_fast(2.0f * kLog2e * product * scale_by_cap);   // (infinite for large scores: then the cap itself)
+    return cap2 - __fdividef(2.0f * cap2, e + 1.0f);
+}
+// What multiplies a finished accumulator (largest score `top`, in units of log2, and sum `total` of the weights under it): the reciprocal of
+// the denominator, a sink included.
+__device__ __forceinline__ float denominator_factor(const ChunkParams& p, int head, float top, float total) {
+    if (!p.sink) return 1.0f / total;
+    const float sink = __ldg(p.sink + head) * kLog2e, high = fmaxf(top, sink);
+    const float factor = exp2f(top - high);
+    return factor / fmaf(total, factor, exp2f(sink - high));
 }
 
 __device__ __forceinline__ void store_pair(const ChunkAttention& a, int row, int head, int column, float x, float y) {
@@ -311,6 +369,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     const int key_begin = p.chunk_start(length + offset), key_end = length + last;   // absolute positions of the tile's keys
     const int slot_start = p.chunk_start(length);                                    // position of the slot's entry 0
     const int tiles = (key_end - key_begin + S::kKeys - 1) / S::kKeys;
+    const int in_slot = p.appends_first(a.step) ? key_end : length;                  // positions whose keys the slot holds
 
     // rows of the tile: (position, head of the group)
     auto row_of = [&](int m, int& position, int& head) {
@@ -342,7 +401,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
             const bool live = j < key_end && piece * 8 < p.dim;
             const __nv_bfloat16* from = key_slot;
             if (live) {
-                if (j < length) from = key_slot + static_cast<int64_t>(j - slot_start) * p.dim + piece * 8;
+                if (j < in_slot) from = key_slot + static_cast<int64_t>(j - slot_start) * p.dim + piece * 8;
                 else from = key_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim + piece * 8;
             }
             copy_async_16(keys + tile_offset<DK>(n, piece), from, live);
@@ -353,7 +412,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
             const bool live = j < key_end && piece * 8 < p.vdim;
             const __nv_bfloat16* from = value_slot;
             if (live) {
-                if (j < length) from = value_slot + static_cast<int64_t>(j - slot_start) * p.vdim + piece * 8;
+                if (j < in_slot) from = value_slot + static_cast<int64_t>(j - slot_start) * p.vdim + piece * 8;
                 else from = value_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.vdim + piece * 8;
             }
             copy_async_16(values + tile_offset<DV>(n, piece), from, live);
@@ -385,7 +444,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[v][i] = 0.0f;
     float top[2] = {-INFINITY, -INFINITY}, total[2] = {0.0f, 0.0f};
-    const float scale2 = p.scale * kLog2e;
+    const float scale2 = p.scale * kLog2e, cap2 = p.softcap * kLog2e, scale_by_cap = p.softcap > 0.0f ? p.scale / p.softcap : 0.0f;
     const uint32_t query_at = smem_u32(smem);
     const int query_row = row_base + (lane & 15);
     auto load_query = [&](uint32_t (&f)[4], int k) { ldsm_x4(f, query_at + tile_offset<DK>(query_row, k * 2 + (lane >> 4))); };
@@ -426,7 +485,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
         for (int n = 0; n < NT; ++n)
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                s[n][i] *= scale2;
+                s[n][i] = p.softcap > 0.0f ? capped_score(s[n][i], scale_by_cap, cap2) : s[n][i] * scale2;
                 if (mask) {
                     const int j = t0 + n * 8 + (lane & 3) * 2 + (i & 1);
                     if (j < see_from[i >> 1] || j >= see_to[i >> 1]) s[n][i] = -INFINITY;
@@ -482,7 +541,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
         int position, head;
         if (!row_of(row_base + (lane >> 2) + i * 8, position, head)) continue;
         const int row = first + position;
-        const float factor = head_gate(p, row, head) / total[i];
+        const float factor = head_gate(p, row, head) * denominator_factor(p, head, top[i], total[i]);
 #pragma unroll
         for (int v = 0; v < VT; ++v) {
             const int column = v * 8 + (lane & 3) * 2;
@@ -590,7 +649,7 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
     }
 
     constexpr int VT = DV / 8;
-    const float scale2 = p.scale * kLog2e;
+    const float scale2 = p.scale * kLog2e, cap2 = p.softcap * kLog2e, scale_by_cap = p.softcap > 0.0f ? p.scale / p.softcap : 0.0f;
     const int own = warp * 16;   // this warp's keys of a tile
     for (int item = blockIdx.x; item < items; item += gridDim.x) {
         const int heads_here = min(a.heads_per_tile, p.group - now.head_tile * a.heads_per_tile);
@@ -640,7 +699,8 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
                 for (int n = 0; n < 2; ++n)
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
-                        s[n][i] = n * 8 + (lane & 3) * 2 + (i & 1) < seen ? s[n][i] * scale2 : -INFINITY;
+                        const float score = p.softcap > 0.0f ? capped_score(s[n][i], scale_by_cap, cap2) : s[n][i] * scale2;
+                        s[n][i] = n * 8 + (lane & 3) * 2 + (i & 1) < seen ? score : -INFINITY;
                         high[i >> 1] = fmaxf(high[i >> 1], s[n][i]);
                     }
 #pragma unroll
@@ -729,7 +789,7 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
             }
             const int head = head0 + m;
             if (a.splits == 1) {
-                const float factor = gates[m] / sum;
+                const float factor = gates[m] * denominator_factor(p, head, from, sum);
                 store_pair(a, now.sequence, head, column, x * factor, y * factor);
             } else {
                 const int64_t part = (static_cast<int64_t>(now.sequence) * p.heads + head) * a.splits + now.split;
@@ -750,7 +810,7 @@ __global__ void __launch_bounds__(64) chunk_combine_kernel(const __grid_constant
     float best = -INFINITY, total = 0.0f;
     for (int s = 0; s < a.splits; ++s) best = fmaxf(best, a.partial_ml[(at + s) * 2]);
     for (int s = 0; s < a.splits; ++s) total = fmaf(a.partial_ml[(at + s) * 2 + 1], exp2_fast(a.partial_ml[(at + s) * 2] - best), total);
-    const float factor = head_gate(a.p, row, head) / total;
+    const float factor = head_gate(a.p, row, head) * denominator_factor(a.p, head, best, total);
     for (int c = threadIdx.x; c < a.p.vdim; c += blockDim.x) {
         float v = 0.0f;
         for (int s = 0; s < a.splits; ++s) v = fmaf(a.partial[(at + s) * a.p.vdim + c], exp2_fast(a.partial_ml[(at + s) * 2] - best), v);
@@ -773,7 +833,7 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
     const int head = blockIdx.x, row = blockIdx.y, kv_head = head / p.group, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const RowPlace place = row_place(a.rows, row);
     const int length = a.rows.lengths[place.slot], first = __ldg(a.rows.first + place.sequence);
-    const int begin = p.chunk_start(place.position), end = place.position + 1, stored_end = a.step ? end : length;
+    const int begin = p.chunk_start(place.position), end = place.position + 1, stored_end = p.appends_first(a.step) ? end : length;
     auto key_at = [&](int j) {
         return j < stored_end ? static_cast<const T*>(p.key_cache) + p.entry(place.slot, kv_head, j) * p.dim
                               : static_cast<const T*>(p.key) + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim;
@@ -794,7 +854,7 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
             float dot = 0.0f;
             for (int c = lane; c < p.dim; c += 32) dot = fmaf(query[c], load_as_f32(key, c), dot);
             dot = warp_sum(dot);
-            if (lane == 0) w[j] = dot * p.scale;
+            if (lane == 0) w[j] = p.softcap > 0.0f ? p.softcap * tanhf(dot * p.scale / p.softcap) : dot * p.scale;
         }
         __syncthreads();
         float high = -INFINITY;
@@ -810,6 +870,11 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
             for (int j = 0; j < n; ++j) v = fmaf(w[j], load_as_f32(value_at(k0 + j), c), v);
             acc[c] = v;
         }
+    }
+    if (p.sink) {
+        const float sink = __ldg(p.sink + head), high = fmaxf(top, sink), factor = expf(top - high);
+        for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads) acc[c] *= factor;
+        total = fmaf(total, factor, expf(sink - high));
     }
     const float scale = head_gate(p, row, head) / total;
     for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads)
@@ -854,7 +919,7 @@ template <int DK, int DV> int launch_chunk_step(ChunkAttention a, int sms, cudaS
     const ChunkParams& p = a.p;
     alignas(64) CUtensorMap keys, values;
     const int64_t rows = static_cast<int64_t>(p.slots) * p.kv_heads * p.entries;
-    if (rows > INT32_MAX) { set_error("chunked attention: the slots hold more than 2^31 rows"); return B200_UNSUPPORTED; }
+    if (rows > INT32_MAX) { set_error("grouped attention: the slots hold more than 2^31 rows"); return B200_UNSUPPORTED; }
     int status = encode_slots(&keys, p.key_cache, rows, p.dim);
     if (status == B200_OK) status = encode_slots(&values, p.value_cache, rows, p.vdim);
     if (status != B200_OK) return status;
@@ -866,7 +931,7 @@ template <int DK, int DV> int launch_chunk_step(ChunkAttention a, int sms, cudaS
     auto kernel = chunk_step_kernel<DK, DV>;
     B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     const int64_t items = static_cast<int64_t>(a.rows.sequences) * p.kv_heads * a.head_tiles * a.splits;
-    if (items > INT32_MAX) { set_error("chunked attention: too many sequences and heads in one pass"); return B200_UNSUPPORTED; }
+    if (items > INT32_MAX) { set_error("grouped attention: too many sequences and heads in one pass"); return B200_UNSUPPORTED; }
     return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(std::min<int64_t>(items, resident * sms))), dim3(kStepThreads), smem, stream, a, keys,
                                         values), "chunk_step_kernel launch");
 }
@@ -892,7 +957,7 @@ extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* 
     RowsView rows;
     if (!chunk_params(args, p) || !rows_view(pass, rows)) return B200_BAD_ARGUMENT;
     const bool step = rows.max_count == 1;
-    if (!step && (!p.key || !p.value)) { set_error("b200_chunk_prepare: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
+    if (!p.appends_first(step) && (!p.key || !p.value)) { set_error("b200_chunk_prepare: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
     Units u{};
     if (units && units->kind) {
         if (units->kind < 0 || units->kind > 2 || units->column < 0 || units->count < 0 || units->count > INT32_MAX || units->out_stride < units->count
@@ -905,24 +970,22 @@ extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* 
     }
     Route r{};
     if (route && route->experts) {
-        if (route->experts < 0 || route->experts > B200_MAX_EXPERTS || route->top <= 0 || route->top > route->experts || route->column < 0
-            || route->column + route->experts > p.stride || !route->chosen || !route->weight || (route->rank && !route->counts)) {
+        if (!route_view(route, r) || route->column + route->experts > p.stride) {
             set_error("b200_chunk_prepare: inconsistent router");
             return B200_BAD_ARGUMENT;
         }
-        r = Route{route->experts, route->top, route->column, route->chosen, route->weight, route->rank, route->counts};
     }
     const int q = p.heads * p.dim, k = p.kv_heads * p.dim;
     auto aligned = [](const void* at) { return (reinterpret_cast<uintptr_t>(at) & 15) == 0; };
     auto aligned8 = [](const void* at) { return (reinterpret_cast<uintptr_t>(at) & 7) == 0; };
-    const bool vector = p.dim % 4 == 0 && p.vdim % 4 == 0 && (p.rot_dims >> 1) % 4 == 0 && p.stride % 4 == 0 && aligned(p.projected) && aligned(p.q_norm)
-        && aligned(p.k_norm) && aligned(p.query) && aligned(p.key) && aligned(p.value) && aligned(p.key_cache) && aligned(p.value_cache)
+    const bool vector = p.dim % 4 == 0 && p.vdim % 4 == 0 && (p.rotate_pairs || (p.rot_dims >> 1) % 4 == 0) && p.stride % 4 == 0 && aligned(p.projected) && aligned(p.q_norm)
+        && aligned(p.k_norm) && aligned(p.q_bias) && aligned(p.k_bias) && aligned(p.query) && aligned(p.key) && aligned(p.value) && aligned(p.key_cache) && aligned(p.value_cache)
         && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0
         && (u.kind == 0 || (u.column % 4 == 0 && u.count % 4 == 0 && u.stride % 4 == 0 && aligned(u.out) && aligned8(u.out_hi) && aligned8(u.out_lo)));
     auto kernel = args->dtype == B200_BF16 ? (vector ? chunk_prepare_kernel<__nv_bfloat16, 4> : chunk_prepare_kernel<__nv_bfloat16, 1>)
                                            : (vector ? chunk_prepare_kernel<float, 4> : chunk_prepare_kernel<float, 1>);
     const dim3 grid(static_cast<unsigned>(rows.rows), static_cast<unsigned>(1 + (u.count + kUnitSlice - 1) / kUnitSlice));
-    return cuda_status(launch_dependent(kernel, grid, dim3(kPrepareThreads), static_cast<size_t>(r.experts) * 4,
+    return cuda_status(launch_dependent(kernel, grid, dim3(kPrepareThreads), (static_cast<size_t>(r.experts) + (p.norm == B200_HEAD_NORM_HEAD ? p.heads + p.kv_heads : 0)) * 4,
                                         as_stream(stream), p, rows, step, u, r), "chunk_prepare_kernel launch");
 }
 
@@ -948,7 +1011,7 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
     a.step = a.rows.max_count == 1;
     a.out = out; a.out_hi = static_cast<__nv_bfloat16*>(out_hi); a.out_lo = static_cast<__nv_bfloat16*>(out_lo); a.out_stride = out_stride;
     a.splits = 1;
-    if (!a.step && (!p.key || !p.value)) { set_error("b200_chunk_attention: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
+    if (!p.appends_first(a.step) && (!p.key || !p.value)) { set_error("b200_chunk_attention: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
     int status = B200_OK;
     if (chunk_takes_mma(p, args->dtype, out_stride)) {
         int device = 0;
@@ -965,7 +1028,7 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
             a.partial_ml = a.partial + static_cast<int64_t>(a.rows.rows) * p.heads * a.splits * p.vdim;
         }
         if (a.rows.sequences > 65535 || p.kv_heads * a.head_tiles > 65535) {
-            set_error("chunked attention: at most 65535 sequences and head tiles in one pass");
+            set_error("grouped attention: at most 65535 sequences and head tiles in one pass");
             return B200_UNSUPPORTED;
         }
         a.status = device_status_word(device);
@@ -978,15 +1041,15 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
             status = cuda_status(launch_dependent(chunk_combine_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(64), 0, s, a),
                                  "chunk_combine_kernel launch");
     } else {
-        if (a.rows.rows > 65535) { set_error("chunked attention: at most 65535 rows in one pass"); return B200_UNSUPPORTED; }
+        if (a.rows.rows > 65535) { set_error("grouped attention: at most 65535 rows in one pass"); return B200_UNSUPPORTED; }
         const size_t smem = (static_cast<size_t>(p.dim) + p.vdim + kGenericKeys + 32) * sizeof(float);
         auto kernel = args->dtype == B200_BF16 ? chunk_generic_kernel<__nv_bfloat16> : chunk_generic_kernel<float>;
-        if (smem > 200 * 1024) { set_error("chunked attention: head sizes %d and %d are too large", p.dim, p.vdim); return B200_UNSUPPORTED; }
+        if (smem > 200 * 1024) { set_error("grouped attention: head sizes %d and %d are too large", p.dim, p.vdim); return B200_UNSUPPORTED; }
         B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
         status = cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(kGenericThreads), smem, s, a),
                              "chunk_generic_kernel launch");
     }
-    if (status != B200_OK || a.step) return status;
+    if (status != B200_OK || p.appends_first(a.step)) return status;
     auto append = args->dtype == B200_BF16 ? chunk_append_kernel<__nv_bfloat16> : chunk_append_kernel<float>;
     return cuda_status(launch_dependent(append, dim3(static_cast<unsigned>(std::min(a.rows.rows, 1184))), dim3(128), 0, s, p, a.rows), "chunk_append_kernel launch");
 }

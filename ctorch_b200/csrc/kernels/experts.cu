@@ -1,5 +1,7 @@
-// Mixture of experts: every slot (row, choice) adds expert(weight * row), expert(x) = down gelu(up x).  The weight multiplies the
-// expert's input, so it joins the row's norm factor in front of the activation.
+// Mixture of experts: every slot (row, choice) adds expert(weight * row) or weight * expert(row), expert(x) = down gelu(up x) or
+// down (silu(gate x) * (up x)) with gate and up rows interleaved.  A weight of the expert's input joins the row's norm factor in front of
+// the activation; a weight of its result is applied where the choices of a row are added up.  Choices past the experts are identity
+// experts: they add the weighted row itself and have no slots to sort.
 //
 //   * streamed: few slots, f32 weights, odd sizes.  expert_up_kernel and expert_down_kernel let every slot stream its expert's rows with
 //     f32 FMAs; the down form adds the choices of a row and the residual itself.
@@ -7,9 +9,12 @@
 //     written), then expert_gemm_kernel multiplies tiles of up to 128 slots of ONE expert with its weights on the tensor cores
 //     (persistent CTAs over the list, TMA operand ring, tcgen05, double-buffered accumulator, the row epilogues of the dense kernels);
 //     only the 32-row boxes that hold slots are fetched, so a batch that gives every expert a few rows costs the weight stream.
-//     expert_combine_kernel adds every row's results in the order of its choices: the sum does not depend on the sorting.
+//     expert_combine_kernel adds every row's results in the order of its choices: the sum does not depend on the sorting.  Where a norm
+//     stands behind the mixture it finishes the row as well (sandwich.cuh).
 #include "linear_rows.cuh"
+#include "router.cuh"
 #include "rows.cuh"
+#include "sandwich.cuh"
 #include "tcgen05.cuh"
 
 #include <algorithm>
@@ -29,32 +34,55 @@ struct ExpertParams {
     float eps;
     const float* residual;
     float* y;
+    bool gated, weigh_results;
+    int identity;
+    SandwichView after;
+    bool finishes;   // `after` is set
 };
 
 bool expert_params(const b200_experts* a, ExpertParams& p) {
-    if (!a || a->experts <= 0 || a->experts > B200_MAX_EXPERTS || a->top <= 0 || a->top > a->experts || a->rows <= 0 || a->in <= 0 || a->ff <= 0
-        || a->rows * a->top > INT32_MAX || a->in > INT32_MAX || a->ff > INT32_MAX || a->experts * std::max(a->in, a->ff) > INT32_MAX
+    if (!a || a->experts <= 0 || a->experts > B200_MAX_EXPERTS || a->top <= 0 || a->rows <= 0 || a->in <= 0 || a->ff <= 0
+        || a->rows * a->top > INT32_MAX || a->in > INT32_MAX || a->ff > INT32_MAX || a->experts * std::max(a->in, 2 * a->ff) > INT32_MAX || a->top > a->experts + a->identity || a->identity < 0
         || (a->weight_dtype != B200_F32 && a->weight_dtype != B200_BF16) || !a->up || !a->down || !a->chosen || !a->weight
-        || (!a->x && (!a->x_hi || !a->x_lo)) || (a->parts_in > 0 && !a->sumsq_in) || a->parts_in < 0 || !a->residual || !a->y) {
+        || (!a->x && (!a->x_hi || !a->x_lo)) || (a->parts_in > 0 && !a->sumsq_in) || a->parts_in < 0
+        || (!a->y && !a->after)) {
         set_error("mixture of experts: bad pointer or size");
         return false;
     }
     p = ExpertParams{a->experts, a->top, static_cast<int>(a->rows), static_cast<int>(a->in), static_cast<int>(a->ff), a->up, a->down, a->chosen, a->weight,
                      a->x, static_cast<const __nv_bfloat16*>(a->x_hi), static_cast<const __nv_bfloat16*>(a->x_lo), a->sumsq_in, a->parts_in,
-                     static_cast<float>(a->eps), a->residual, a->y};
+                     static_cast<float>(a->eps), a->residual, a->y, a->gated != 0, a->weigh_results != 0, a->identity, SandwichView{}, a->after != nullptr};
+    if (a->after && !sandwich_view(a->after, p.after)) {
+        set_error("mixture of experts: inconsistent norm behind the mixture");
+        return false;
+    }
     return true;
 }
 
-// Factor of a slot's row: the split norm's scale (1 without one) times the router's weight.
-__device__ __forceinline__ float slot_scale(const ExpertParams& p, int slot) {
-    const int row = slot / p.top;
+// Factor of a row: the split norm's scale (1 without one).
+__device__ __forceinline__ float row_factor(const ExpertParams& p, int row) {
     float scale = 1.0f;
     if (p.parts_in > 0) {
         float total = 0.0f;
         for (int i = 0; i < p.parts_in; ++i) total += __ldg(p.sumsq_in + static_cast<int64_t>(i) * p.rows + row);
         scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(total, static_cast<float>(p.in)), p.eps)));
     }
-    return scale * __ldg(p.weight + slot);
+    return scale;
+}
+// Factor of a slot's input: its row's, and the router's weight where that multiplies the input.
+__device__ __forceinline__ float slot_scale(const ExpertParams& p, int slot) {
+    return row_factor(p, slot / p.top) * (p.weigh_results ? 1.0f : __ldg(p.weight + slot));
+}
+__device__ __forceinline__ float row_value(const ExpertParams& p, int64_t at) {
+    return p.x ? p.x[at] : __bfloat162float(p.x_hi[at]) + __bfloat162float(p.x_lo[at]);
+}
+// Weights of a row's identity choices together.
+__device__ __forceinline__ float identity_weight(const ExpertParams& p, int row) {
+    float total = 0.0f;
+    if (p.identity > 0)
+        for (int k = 0; k < p.top; ++k)
+            if (__ldg(p.chosen + row * p.top + k) >= p.experts) total += __ldg(p.weight + row * p.top + k);
+    return total;
 }
 
 // ---- streamed -------------------------------------------------------------------------------------------------------
@@ -65,7 +93,7 @@ template <class W, bool VECTOR, int F>
 __device__ __forceinline__ void dot_rows(const W* const (&w)[F], const float* x, int n, int lane, float (&acc)[F]) {
     if constexpr (VECTOR) {
         constexpr int kPer = 16 / sizeof(W);
-#pragma unroll (8 / F)
+#pragma unroll (F < 8 ? 8 / F : 1)
         for (int k = lane * kPer; k < n; k += 32 * kPer) {
             uint4 raw[F];
 #pragma unroll
@@ -103,33 +131,41 @@ template <class W> __device__ __forceinline__ void prefetch_rows(const W* matrix
     for (int64_t o = static_cast<int64_t>(threadIdx.x) * 128; o < bytes; o += kStreamThreads * 128) prefetch_l2(at + o);
 }
 
-// grid (slots, feature blocks): act[slot, f] = gelu(up_f . (scale * row)), F features per warp
-template <class W, bool VECTOR, int F> __global__ void __launch_bounds__(kStreamThreads) expert_up_kernel(const __grid_constant__ ExpertParams p, float* act) {
+// grid (slots, feature blocks): act[slot, f] = gelu(up_f . (scale * row)), or the gated unit of rows 2f and 2f + 1; F features per warp
+template <class W, bool VECTOR, int F, bool GATED>
+__global__ void __launch_bounds__(kStreamThreads) expert_up_kernel(const __grid_constant__ ExpertParams p, float* act) {
+    constexpr int kPer = GATED ? 2 : 1, kRows = F * kPer;   // weight rows per feature, per warp
     extern __shared__ __align__(16) float x[];
     const int slot = blockIdx.x, row = slot / p.top, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int block0 = blockIdx.y * kStreamWarps * F, f0 = block0 + warp * F;
-    if constexpr (F == 1) prefetch_rows(static_cast<const W*>(p.up), *static_cast<const volatile int32_t*>(p.chosen + slot), p.experts, p.ff, p.in, block0, min(block0 + kStreamWarps * F, p.ff));
+    if constexpr (F == 1) prefetch_rows(static_cast<const W*>(p.up), *static_cast<const volatile int32_t*>(p.chosen + slot), p.experts, p.ff * kPer, p.in, block0 * kPer, min(block0 + kStreamWarps * F, p.ff) * kPer);
     grid_dependency_wait();
     grid_launch_dependents();
+    const int expert = *static_cast<const volatile int32_t*>(p.chosen + slot);
+    if (expert >= p.experts) return;   // an identity expert
     const float scale = slot_scale(p, slot);
     const int64_t base = static_cast<int64_t>(row) * p.in;
-    for (int c = threadIdx.x; c < p.in; c += kStreamThreads)
-        x[c] = (p.x ? p.x[base + c] : __bfloat162float(p.x_hi[base + c]) + __bfloat162float(p.x_lo[base + c])) * scale;
-    const int expert = *static_cast<const volatile int32_t*>(p.chosen + slot);
+    for (int c = threadIdx.x; c < p.in; c += kStreamThreads) x[c] = row_value(p, base + c) * scale;
     __syncthreads();
     if (f0 >= p.ff) return;
-    const W* w[F];
-    float acc[F];
+    const W* w[kRows];
+    float acc[kRows];
 #pragma unroll
-    for (int f = 0; f < F; ++f) {
-        w[f] = static_cast<const W*>(p.up) + (static_cast<int64_t>(expert) * p.ff + min(f0 + f, p.ff - 1)) * p.in;
+    for (int f = 0; f < kRows; ++f) {
+        w[f] = static_cast<const W*>(p.up) + (static_cast<int64_t>(expert) * p.ff * kPer + min(f0 * kPer + f, p.ff * kPer - 1)) * p.in;
         acc[f] = 0.0f;
     }
-    dot_rows<W, VECTOR, F>(w, x, p.in, lane, acc);
+    dot_rows<W, VECTOR, kRows>(w, x, p.in, lane, acc);
 #pragma unroll
     for (int f = 0; f < F; ++f) {
-        const float v = warp_sum(acc[f]);
-        if (lane == f && f0 + f < p.ff) act[static_cast<int64_t>(slot) * p.ff + f0 + f] = gelu_exact(v);
+        float v;
+        if constexpr (GATED) {
+            const float gate = warp_sum(acc[2 * f]), up = warp_sum(acc[2 * f + 1]);
+            v = silu_reference(gate) * up;
+        } else {
+            v = gelu_exact(warp_sum(acc[f]));
+        }
+        if (lane == f && f0 + f < p.ff) act[static_cast<int64_t>(slot) * p.ff + f0 + f] = v;
     }
 }
 
@@ -148,27 +184,31 @@ template <class W, bool VECTOR, int F> __global__ void __launch_bounds__(kStream
     for (int f = 0; f < F; ++f) sum[f] = 0.0f;
     for (int k = 0; k < p.top; ++k) {
         const int slot = row * p.top + k;
-        __syncthreads();
-        for (int c = threadIdx.x; c < p.ff; c += kStreamThreads) x[c] = act[static_cast<int64_t>(slot) * p.ff + c];
         const int expert = *static_cast<const volatile int32_t*>(p.chosen + slot);
+        if (expert >= p.experts) continue;   // (the whole CTA: an identity expert)
+        const float weight = p.weigh_results ? __ldg(p.weight + slot) : 1.0f;
+        __syncthreads();
+        for (int c = threadIdx.x; c < p.ff; c += kStreamThreads) x[c] = act[static_cast<int64_t>(slot) * p.ff + c] * weight;
         __syncthreads();
         const W* w[F];
 #pragma unroll
         for (int f = 0; f < F; ++f) w[f] = static_cast<const W*>(p.down) + (static_cast<int64_t>(expert) * p.in + min(f0 + f, p.in - 1)) * p.ff;
         if (f0 < p.in) dot_rows<W, VECTOR, F>(w, x, p.ff, lane, sum);
     }
+    const float through = identity_weight(p, row) * (p.identity > 0 ? row_factor(p, row) : 1.0f);
 #pragma unroll
     for (int f = 0; f < F; ++f) {
-        const float v = warp_sum(sum[f]);
+        float v = warp_sum(sum[f]);
         if (lane == f && f0 + f < p.in) {
             const int64_t at = static_cast<int64_t>(row) * p.in + f0 + f;
-            p.y[at] = p.residual[at] + v;
+            if (through != 0.0f) v = fmaf(through, row_value(p, at), v);
+            p.y[at] = p.residual ? p.residual[at] + v : v;
         }
     }
 }
 
 template <class W, bool VECTOR, int F> int launch_expert_up(const ExpertParams& p, float* act, size_t smem, cudaStream_t stream) {
-    auto kernel = expert_up_kernel<W, VECTOR, F>;
+    auto kernel = p.gated ? expert_up_kernel<W, VECTOR, F, true> : expert_up_kernel<W, VECTOR, F, false>;
     B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     const dim3 grid(static_cast<unsigned>(p.rows * p.top), static_cast<unsigned>((p.ff + kStreamWarps * F - 1) / (kStreamWarps * F)));
     return cuda_status(launch_dependent(kernel, grid, dim3(kStreamThreads), smem, stream, p, act), "expert_up_kernel launch");
@@ -254,7 +294,8 @@ __global__ void __launch_bounds__(256) expert_gather_kernel(const __grid_constan
     grid_dependency_wait();
     grid_launch_dependents();
     const int slot = blockIdx.x, expert = __ldg(p.chosen + slot);
-    if (threadIdx.x < 32) {
+    const bool sorted = expert < p.experts;   // not an identity expert
+    if (sorted && threadIdx.x < 32) {
         int total = 0;
         for (int e = threadIdx.x; e < expert; e += 32) total += counts[e];
         total = __reduce_add_sync(0xffffffffu, total);
@@ -263,15 +304,17 @@ __global__ void __launch_bounds__(256) expert_gather_kernel(const __grid_constan
     if (slot == 0)
         for (int e = threadIdx.x; e < p.experts; e += blockDim.x) copy[e] = counts[e];
     __syncthreads();
-    const int to = before + rank[slot];
-    const int64_t from_at = static_cast<int64_t>(slot / p.top) * p.in, to_at = static_cast<int64_t>(to) * p.in;
-    for (int c = threadIdx.x * 8; c < p.in; c += blockDim.x * 8) {
-        *reinterpret_cast<uint4*>(g.x_hi + to_at + c) = *reinterpret_cast<const uint4*>(p.x_hi + from_at + c);
-        *reinterpret_cast<uint4*>(g.x_lo + to_at + c) = *reinterpret_cast<const uint4*>(p.x_lo + from_at + c);
-    }
-    if (threadIdx.x == 0) {
-        g.scale[to] = slot_scale(p, slot);
-        g.place[slot] = to;
+    if (sorted) {
+        const int to = before + rank[slot];
+        const int64_t from_at = static_cast<int64_t>(slot / p.top) * p.in, to_at = static_cast<int64_t>(to) * p.in;
+        for (int c = threadIdx.x * 8; c < p.in; c += blockDim.x * 8) {
+            *reinterpret_cast<uint4*>(g.x_hi + to_at + c) = *reinterpret_cast<const uint4*>(p.x_hi + from_at + c);
+            *reinterpret_cast<uint4*>(g.x_lo + to_at + c) = *reinterpret_cast<const uint4*>(p.x_lo + from_at + c);
+        }
+        if (threadIdx.x == 0) {
+            g.scale[to] = slot_scale(p, slot);
+            g.place[slot] = to;
+        }
     }
     if (slot == 0) {
         for (int e = threadIdx.x; e < p.experts; e += blockDim.x) {
@@ -477,19 +520,42 @@ __global__ void __launch_bounds__(kGroupedThreads, 1) expert_gemm_kernel(const _
     }
 }
 
-// One CTA per row: y = residual + the row's results in the order of its choices.
+// One CTA per row: y = residual + the row's results in the order of its choices.  FINISH: the sum goes through the norm behind the mixture.
+template <bool FINISH>
 __global__ void __launch_bounds__(256) expert_combine_kernel(const __grid_constant__ ExpertParams p, const float* results, const int32_t* place) {
+    __shared__ float scratch[FINISH ? 32 : 1];
     grid_dependency_wait();
     grid_launch_dependents();
     const int row = blockIdx.x;
     const int64_t at = static_cast<int64_t>(row) * p.in;
-    for (int c = threadIdx.x * 4; c < p.in; c += blockDim.x * 4) {
-        float4 sum = *reinterpret_cast<const float4*>(p.residual + at + c);
+    const float through = p.identity > 0 ? identity_weight(p, row) * row_factor(p, row) : 0.0f;
+    auto total = [&](int c, float4 sum) {
         for (int k = 0; k < p.top; ++k) {
-            const float4 v = __ldcs(reinterpret_cast<const float4*>(results + static_cast<int64_t>(__ldg(place + row * p.top + k)) * p.in + c));
-            sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
+            const int slot = row * p.top + k;
+            if (p.identity > 0 && __ldg(p.chosen + slot) >= p.experts) continue;
+            const float4 v = __ldcs(reinterpret_cast<const float4*>(results + static_cast<int64_t>(__ldg(place + slot)) * p.in + c));
+            const float w = p.weigh_results ? __ldg(p.weight + slot) : 1.0f;
+            sum.x = fmaf(v.x, w, sum.x); sum.y = fmaf(v.y, w, sum.y); sum.z = fmaf(v.z, w, sum.z); sum.w = fmaf(v.w, w, sum.w);
         }
-        *reinterpret_cast<float4*>(p.y + at + c) = sum;
+        if (through != 0.0f) {
+            const uint2 hi = *reinterpret_cast<const uint2*>(p.x_hi + at + c), lo = *reinterpret_cast<const uint2*>(p.x_lo + at + c);
+            sum.x = fmaf(through, bf16_lo(hi.x) + bf16_lo(lo.x), sum.x);
+            sum.y = fmaf(through, bf16_hi(hi.x) + bf16_hi(lo.x), sum.y);
+            sum.z = fmaf(through, bf16_lo(hi.y) + bf16_lo(lo.y), sum.z);
+            sum.w = fmaf(through, bf16_hi(hi.y) + bf16_hi(lo.y), sum.w);
+        }
+        return sum;
+    };
+    if constexpr (FINISH) {
+        finish_sandwich<4, true>(p.after, row, p.in, [&](int c) {
+            const float4 v = total(c, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
+            return Lanes<4>{{v.x, v.y, v.z, v.w}};
+        }, scratch);
+    } else {
+        for (int c = threadIdx.x * 4; c < p.in; c += blockDim.x * 4) {
+            const float4 sum = p.residual ? *reinterpret_cast<const float4*>(p.residual + at + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            *reinterpret_cast<float4*>(p.y + at + c) = total(c, sum);
+        }
     }
 }
 
@@ -540,7 +606,17 @@ constexpr int kStreamedSlots = 16;
 bool takes_grouped(const b200_experts* a, const ExpertParams& p) {
     return a->weight_dtype == B200_BF16 && p.x_hi && p.x_lo && p.in % 8 == 0 && p.ff % 8 == 0
         && ((reinterpret_cast<uintptr_t>(p.x_hi) | reinterpret_cast<uintptr_t>(p.x_lo) | reinterpret_cast<uintptr_t>(p.up) | reinterpret_cast<uintptr_t>(p.down)
-             | reinterpret_cast<uintptr_t>(p.residual) | reinterpret_cast<uintptr_t>(p.y)) & 15) == 0;
+             | reinterpret_cast<uintptr_t>(p.residual) | reinterpret_cast<uintptr_t>(p.y)) & 15) == 0
+        && (!p.finishes || sandwich_takes_quads(p.after, p.in));
+}
+
+constexpr int kRouteWarps = 8;
+__global__ void __launch_bounds__(kRouteWarps * 32) route_rows_kernel(const float* logits, const int rows, const int64_t stride, const __grid_constant__ Route route) {
+    extern __shared__ float copies[];   // [warps][experts]
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int warp = threadIdx.x >> 5, row = blockIdx.x * kRouteWarps + warp;
+    if (row < rows) choose_experts(route, row, logits + row * stride, copies + warp * route.experts, threadIdx.x & 31);
 }
 
 }  // namespace
@@ -581,18 +657,21 @@ extern "C" int b200_experts_grouped(const b200_experts* args, const int32_t* ran
     ExpertGemm up = gp, down = gp;
     up.scale = g.scale;
     up.base.out_hi = g.act_hi; up.base.out_lo = g.act_lo;
-    status = launch_expert_gemm<B200_EPI_GELU>(p, g, g.x_hi, g.x_lo, p.up, p.in, p.ff, up, sms, s);
+    up.base.out_stride = p.ff;
+    status = p.gated ? launch_expert_gemm<B200_EPI_SWIGLU>(p, g, g.x_hi, g.x_lo, p.up, p.in, 2 * p.ff, up, sms, s)
+                     : launch_expert_gemm<B200_EPI_GELU>(p, g, g.x_hi, g.x_lo, p.up, p.in, p.ff, up, sms, s);
     if (status != B200_OK) return status;
     down.base.y = g.y;
     down.listed = true;
     status = launch_expert_gemm<B200_EPI_STORE>(p, g, g.act_hi, g.act_lo, p.down, p.ff, p.in, down, sms, s);
     if (status != B200_OK) return status;
-    return cuda_status(launch_dependent(expert_combine_kernel, dim3(static_cast<unsigned>(p.rows)), dim3(256), 0, s, p, static_cast<const float*>(g.y),
+    return cuda_status(launch_dependent(p.finishes ? expert_combine_kernel<true> : expert_combine_kernel<false>, dim3(static_cast<unsigned>(p.rows)), dim3(256), 0, s, p, static_cast<const float*>(g.y),
                                         static_cast<const int32_t*>(g.place)), "expert_combine_kernel launch");
 }
 
 extern "C" int b200_experts_streamed(const b200_experts* args, float* act, void* stream) {
     ExpertParams p;
+    if (args && args->after) { set_error("b200_experts_streamed: the norm behind the mixture belongs to the grouped form"); return B200_BAD_ARGUMENT; }
     if (!expert_params(args, p) || !act) { if (!act) set_error("b200_experts_streamed: no workspace"); return B200_BAD_ARGUMENT; }
     const size_t up_smem = (static_cast<size_t>(p.in) * 4 + 15) & ~15ull, down_smem = (static_cast<size_t>(p.ff) * 4 + 15) & ~15ull;
     if (up_smem > 220 * 1024 || down_smem > 220 * 1024 || p.ff > 65535 * kStreamWarps || p.in > 65535 * kStreamWarps) {
@@ -608,4 +687,16 @@ extern "C" int b200_experts_streamed(const b200_experts* args, float* act, void*
     cudaStream_t s = as_stream(stream);
     if (bf16) return vector ? launch_streamed<__nv_bfloat16, true>(p, act, up_smem, down_smem, sms, s) : launch_streamed<__nv_bfloat16, false>(p, act, up_smem, down_smem, sms, s);
     return vector ? launch_streamed<float, true>(p, act, up_smem, down_smem, sms, s) : launch_streamed<float, false>(p, act, up_smem, down_smem, sms, s);
+}
+
+extern "C" int b200_route_rows(const float* logits, int64_t rows, int64_t stride, const b200_route* route, void* stream) {
+    Route r;
+    if (!logits || rows < 0 || rows > INT32_MAX || !route || !route_view(route, r) || stride < r.experts || rows * r.top > INT32_MAX) {
+        set_error("b200_route_rows: bad pointer or size");
+        return B200_BAD_ARGUMENT;
+    }
+    if (rows == 0) return B200_OK;
+    return cuda_status(launch_dependent(route_rows_kernel, dim3(static_cast<unsigned>((rows + kRouteWarps - 1) / kRouteWarps)), dim3(kRouteWarps * 32),
+                                        static_cast<size_t>(kRouteWarps) * r.experts * 4, as_stream(stream), logits, static_cast<int>(rows), stride, r),
+                       "route_rows_kernel launch");
 }

@@ -36,6 +36,7 @@ struct LinearParams {
     const float* out_norm_bias;        // set: the norm that follows is Dynamic Tanh (f32 weight and bias), which needs no row
     float out_norm_alpha;              //   statistic; the output shadow holds tanh(alpha * row) * weight + bias
     int64_t out_stride;                // elements between rows of the SwiGLU output shadow
+    float unit_slope, unit_limit;      // SwiGLU epilogue: clamped units (unit_limit > 0), see gated_unit
     float* sumsq_out;                  // [tiles][rows] per-tile sums of squares of the (un-weighted) result rows
     // B200_EPI_ARGMAX: per feature tile and row, the preferred value and its feature index
     float* best_value;                 // [tiles][rows]
@@ -46,6 +47,17 @@ struct LinearParams {
     float* y_copy[7];
     int copies;
 };
+
+// Unit of the SwiGLU epilogue: silu(gate) * up, or clamped, g = min(gate, limit), u = up within +-limit: g * sigmoid(slope * g) * (u + 1).
+// fast: the hardware's exponential and division (see silu_fast).
+__device__ __forceinline__ float gated_unit(const LinearParams& p, float gate, float up, bool fast) {
+    if (p.unit_limit > 0.0f) {
+        const float g = fminf(gate, p.unit_limit), u = fminf(fmaxf(up, -p.unit_limit), p.unit_limit);
+        const float s = fast ? __fdividef(g, 1.0f + __expf(-p.unit_slope * g)) : __fdiv_rn(g, __fadd_rn(1.0f, expf(-p.unit_slope * g)));
+        return s * (u + 1.0f);
+    }
+    return __fmul_rn(fast ? silu_fast(gate) : silu_reference(gate), up);
+}
 
 // What the output shadow of a residual epilogue holds for the new residual value v: v * w (an RMSNorm follows, whose scale the
 // consumer applies) or the finished Dynamic Tanh norm.
@@ -162,7 +174,7 @@ __device__ __forceinline__ void linear_epilogue(const LinearParams& p, int row, 
         store_copies(p, at, a, b, second);
     } else if constexpr (EPI == B200_EPI_SWIGLU) {
         // rows 2j (gate_j) and 2j+1 (up_j) of the interleaved weight
-        a = __fmul_rn(p.x_hi ? silu_fast(a) : silu_reference(a), b);   // shadow input = bf16 model: see silu_fast
+        a = gated_unit(p, a, b, p.x_hi != nullptr);   // shadow input = bf16 model: see silu_fast
         if (p.y) p.y[static_cast<int64_t>(row) * (p.out >> 1) + (feature0 >> 1)] = a;
     } else if constexpr (EPI == B200_EPI_ARGMAX) {
         // nothing is stored: the kernels reduce the pairs of a tile to one candidate per row themselves

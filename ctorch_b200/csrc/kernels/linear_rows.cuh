@@ -301,8 +301,8 @@ __device__ __forceinline__ void finish_rows_quads(const LinearParams& p, const f
                     // (gate_j, up_j, gate_j+1, up_j+1) of the interleaved weight rows; the shadow input makes this a bf16
                     // model, whose SiLU takes the hardware exponential (see silu_fast)
                     const float4 v = value[r][pass];
-                    const float a = __fmul_rn(silu_fast(v.x * scale[r]), v.y * scale[r]);
-                    const float b = __fmul_rn(silu_fast(v.z * scale[r]), v.w * scale[r]);
+                    const float a = gated_unit(p, v.x * scale[r], v.y * scale[r], true);
+                    const float b = gated_unit(p, v.z * scale[r], v.w * scale[r], true);
                     result[r][pass] = make_float2(a, b);
                     const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
                     const __nv_bfloat162 l = __floats2bfloat162_rn(a - __low2float(h), b - __high2float(h));

@@ -223,10 +223,17 @@ int fill_qkv(LinearParams& p, int epilogue, const b200_qkv_args* qkv, int64_t ro
 }  // namespace
 }  // namespace b200
 
-extern "C" int b200_linear(const float* x, int64_t rows, int64_t in, const void* weight, int32_t weight_dtype,
-                           int64_t out, const void* norm_weight, int32_t norm_dtype, double eps,
-                           b200_epilogue epilogue, const float* residual, const b200_qkv_args* qkv, float* y,
-                           void* stream) {
+// Whether the clamped form of the units is consistent, and into the kernels' parameters.
+static bool fill_unit(b200::LinearParams& p, const b200_clamped_unit* unit, int epilogue) {
+    if (!unit) return true;
+    if (epilogue != B200_EPI_SWIGLU || !(unit->limit > 0.0f)) { b200::set_error("clamped units need the SwiGLU epilogue and a positive limit"); return false; }
+    p.unit_slope = unit->slope; p.unit_limit = unit->limit;
+    return true;
+}
+
+static int linear_rows_f32(const float* x, int64_t rows, int64_t in, const void* weight, int32_t weight_dtype, int64_t out, const void* norm_weight,
+                           int32_t norm_dtype, double eps, b200_epilogue epilogue, const float* residual, const b200_qkv_args* qkv,
+                           const b200_clamped_unit* unit, float* y, void* stream) {
     using namespace b200;
     if (!x || !weight || !y || rows < 0 || in <= 0 || out <= 0 || rows > INT32_MAX || in > INT32_MAX || out > INT32_MAX) {
         set_error("b200_linear: bad pointer or size");
@@ -251,6 +258,7 @@ extern "C" int b200_linear(const float* x, int64_t rows, int64_t in, const void*
         const int status = fill_qkv(p, epilogue, qkv, rows, out);
         if (status != B200_OK) return status;
     }
+    if (!fill_unit(p, unit, epilogue)) return B200_BAD_ARGUMENT;
     cudaStream_t s = as_stream(stream);
     {
         // bf16 weights with a moderate inner size go to the tensor-core streaming kernel
@@ -261,6 +269,18 @@ extern "C" int b200_linear(const float* x, int64_t rows, int64_t in, const void*
     const bool vector = (in * element) % 16 == 0 && reinterpret_cast<uintptr_t>(weight) % 16 == 0;
     return weight_dtype == B200_BF16 ? pick_epilogue<__nv_bfloat16>(p, epilogue, vector, s)
                                      : pick_epilogue<float>(p, epilogue, vector, s);
+}
+
+extern "C" int b200_linear(const float* x, int64_t rows, int64_t in, const void* weight, int32_t weight_dtype,
+                           int64_t out, const void* norm_weight, int32_t norm_dtype, double eps,
+                           b200_epilogue epilogue, const float* residual, const b200_qkv_args* qkv, float* y,
+                           void* stream) {
+    return linear_rows_f32(x, rows, in, weight, weight_dtype, out, norm_weight, norm_dtype, eps, epilogue, residual, qkv, nullptr, y, stream);
+}
+
+extern "C" int b200_linear_units(const float* x, int64_t rows, int64_t in, const void* weight, int32_t weight_dtype, int64_t out,
+                                 const b200_clamped_unit* unit, float* y, void* stream) {
+    return linear_rows_f32(x, rows, in, weight, weight_dtype, out, nullptr, 0, 0.0, B200_EPI_SWIGLU, nullptr, nullptr, unit, y, stream);
 }
 
 extern "C" int b200_linear_shadow(const b200_shadow_linear_args* args, void* stream) {
@@ -298,6 +318,7 @@ extern "C" int b200_linear_shadow(const b200_shadow_linear_args* args, void* str
         p.out_norm_weight = args->out_norm->weight; p.out_norm_dtype = B200_F32;
         p.out_norm_bias = args->out_norm->bias; p.out_norm_alpha = args->out_norm->alpha;
     }
+    if (!fill_unit(p, args->unit, epilogue)) return B200_BAD_ARGUMENT;
     p.best_value = args->best_value; p.best_index = args->best_index;
     if (args->copies < 0 || args->copies > 7 || (args->copies > 0 && (!args->y_copies || (epilogue != B200_EPI_STORE && epilogue != B200_EPI_RESIDUAL)))) {
         set_error("b200_linear_shadow: at most 7 result copies, for store and residual epilogues only");

@@ -37,6 +37,23 @@ __device__ __forceinline__ void store_forms(float v, int64_t at, float* out, __n
     }
 }
 
+// V adjacent f32 values, 4 on a 16-byte boundary or 1.
+template <int V> struct Lanes { float v[V]; };
+template <int V> __device__ __forceinline__ Lanes<V> load_lanes(const float* p) {
+    Lanes<V> r;
+    if constexpr (V == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(p);
+        r.v[0] = q.x; r.v[1] = q.y; r.v[2] = q.z; r.v[3] = q.w;
+    } else {
+        r.v[0] = p[0];
+    }
+    return r;
+}
+template <int V> __device__ __forceinline__ void store_lanes(float* p, const Lanes<V>& r) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else p[0] = r.v[0];
+}
+
 // Sum over the CTA (any block size that is a multiple of 32, at most 1024); every thread gets the result.
 __device__ __forceinline__ float block_sum(float v, float* scratch) {
     v = warp_sum(v);

@@ -1,5 +1,6 @@
 // State-space layers (Mamba-2): short causal convolution, selective recurrence, gated group norm; and the small kernels of
-// packed passes.  Everything here is f32: decays, step sizes, states and norms.
+// packed passes.  Everything here is f32: decays, step sizes, states and norms.  Lightning attention is the same recurrence with a fixed
+// decay per head, a step size of one, no skip and no convolution (only its SiLU): keys for B, queries for C, values for x.
 //
 //   * Decode (one row per sequence): per (sequence, head) the channels the head needs are convolved from the slot's ring of recent
 //     inputs, then its [state][vdim] matrix is read once - decay, add dt B x^T, partial sums of S^T C - and written back.  The layer
@@ -37,6 +38,7 @@ struct SsmParams {
     float *conv_state, *ssm_state;
     const float* projected;
     float *mixed, *y;
+    const float* fixed_decay;   // [heads] or NULL: step sizes and decays come from the projection
 };
 
 __device__ __forceinline__ float softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
@@ -48,23 +50,16 @@ __device__ __forceinline__ float ring_input(const SsmParams& p, int slot, int po
     return p.conv_state[(static_cast<int64_t>(slot) * p.taps + position % p.taps) * p.channels + channel];
 }
 
-constexpr int kStepThreads = 256;
+// Step size and decay of a head for one projected row.
+struct StepRate { float dt, decay; };
+__device__ __forceinline__ StepRate step_rate(const SsmParams& p, const float* row, int head) {
+    if (p.fixed_decay) return {1.0f, __ldg(p.fixed_decay + head)};
+    const float dt = softplus(row[p.heads * p.vdim + p.channels + head] + p.dt_bias[head]);
+    return {dt, expf(-expf(p.a_log[head]) * dt)};
+}
+__device__ __forceinline__ float skip_of(const SsmParams& p, int head) { return p.fixed_decay ? 0.0f : p.d[head]; }
 
-template <int V> struct Lanes { float v[V]; };
-template <int V> __device__ __forceinline__ Lanes<V> load_lanes(const float* p) {
-    Lanes<V> r;
-    if constexpr (V == 4) {
-        const float4 q = *reinterpret_cast<const float4*>(p);
-        r.v[0] = q.x; r.v[1] = q.y; r.v[2] = q.z; r.v[3] = q.w;
-    } else {
-        r.v[0] = p[0];
-    }
-    return r;
-}
-template <int V> __device__ __forceinline__ void store_lanes(float* p, const Lanes<V>& r) {
-    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
-    else p[0] = r.v[0];
-}
+constexpr int kStepThreads = 256;
 
 // Convolved channels of one head for one token: [x: vdim | B: state | C: state] into `mixed`, and the token's inputs into the
 // slot's ring (B and C are shared by the heads of a group: its first head writes them).
@@ -77,6 +72,10 @@ __device__ __forceinline__ void convolve_head(const SsmParams& p, const float* i
     for (int i = threadIdx.x; i < P + 2 * N; i += kStepThreads) {
         const int c = i < P ? head * P + i : i < P + N ? inner + group * N + (i - P) : inner + (p.groups + group) * N + (i - P - N);
         const float now = in[inner + c];
+        if (!p.conv_weight) {
+            mixed[i] = now * sigmoid_exact(now);
+            continue;
+        }
         const float* weight = p.conv_weight + c * p.taps;
         float acc = p.conv_bias[c];
 #pragma unroll 4
@@ -89,6 +88,23 @@ __device__ __forceinline__ void convolve_head(const SsmParams& p, const float* i
         mixed[i] = acc * sigmoid_exact(acc);
         if (i < P || shared_writer) ring[ring_at * p.channels + c] = now;
     }
+}
+
+// mixed[row, c] = silu(x | B | C): the inputs of a recurrence without convolution, grid (channel blocks, rows), V channels per thread.
+template <int V> __global__ void __launch_bounds__(128) activate_channels_kernel(const SsmParams p) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    const int64_t row = blockIdx.y;
+    if (c >= p.channels) return;
+    Lanes<V> v = load_lanes<V>(p.projected + row * p.stride + p.heads * p.vdim + c);
+#pragma unroll
+    for (int k = 0; k < V; ++k) v.v[k] *= sigmoid_exact(v.v[k]);
+    store_lanes<V>(p.mixed + row * p.channels + c, v);
+}
+template <int V> int launch_activate(const SsmParams& p, int rows, cudaStream_t stream) {
+    const dim3 grid(static_cast<unsigned>((p.channels / V + 127) / 128), static_cast<unsigned>(rows));
+    return cuda_status(launch_dependent(activate_channels_kernel<V>, grid, dim3(128), 0, stream, p), "activate_channels_kernel launch");
 }
 
 // Streamed step, first half: mixed[row, c] = silu(conv(x | B | C)) of one row per sequence, and the row's inputs into the ring.
@@ -157,14 +173,14 @@ __global__ void __launch_bounds__(kStreamThreads) ssm_step_stream_kernel(const S
         for (int unit = blockIdx.x; unit < units + 2 * static_cast<int>(gridDim.x); unit += gridDim.x, ++turn) {
             const int stage = turn & 1, row = unit / p.heads, head = unit - row * p.heads;
             const bool live = unit < units;
-            float dt = 0.0f;
+            StepRate rate{};
             float* state = nullptr;
             bool fresh = true;
             if (live) {   // operands of this pair, while the stage may still be in use
                 const int slot = __ldg(rows.slot + row);
                 fresh = rows.lengths[slot] == 0;
                 state = p.ssm_state + (static_cast<int64_t>(slot) * p.heads + head) * block;
-                dt = softplus(p.projected[static_cast<int64_t>(row) * p.stride + inner + p.channels + head] + p.dt_bias[head]);
+                rate = step_rate(p, p.projected + static_cast<int64_t>(row) * p.stride, head);
             }
             if (turn >= 2 && pending[stage]) {   // the pair two turns ago has been worked on: its state goes back
                 if (!mbar_wait(&done[stage], ((turn >> 1) - 1) & 1)) {
@@ -177,7 +193,7 @@ __global__ void __launch_bounds__(kStreamThreads) ssm_step_stream_kernel(const S
             pending[stage] = state;
             if (!live) continue;
             float* at = sm + stage * stage_floats;
-            meta[stage] = StreamMeta{dt, expf(-expf(p.a_log[head]) * dt), fresh ? 1.0f : 0.0f};
+            meta[stage] = StreamMeta{rate.dt, rate.decay, fresh ? 1.0f : 0.0f};
             mbar_expect_tx(&full[stage], static_cast<uint32_t>((fresh ? 0 : block) + P + 2 * N) * 4);
             if (!fresh) bulk_load(at, state, static_cast<uint32_t>(block) * 4, &full[stage]);
             const float* mixed = p.mixed + static_cast<int64_t>(row) * p.channels;
@@ -227,7 +243,7 @@ __global__ void __launch_bounds__(kStreamThreads) ssm_step_stream_kernel(const S
         for (int i = threadIdx.x; i < P; i += kStepThreads) {
             float total = 0.0f;
             for (int k = 0; k < slices; ++k) total += partial[k * P + i];
-            p.y[static_cast<int64_t>(row) * inner + head * P + i] = fmaf(p.d[head], x[i], total);
+            p.y[static_cast<int64_t>(row) * inner + head * P + i] = fmaf(skip_of(p, head), x[i], total);
         }
         mbar_arrive(&done[stage]);
     }
@@ -268,8 +284,7 @@ __global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmPara
     fetch(s, my_slice, my_column, my_column < columns && my_slice < slices);
 
     convolve_head(p, in, place.slot, place.position, head, mixed);
-    const float dt = softplus(in[inner + p.channels + head] + p.dt_bias[head]);
-    const float decay = expf(-expf(p.a_log[head]) * dt);
+    const auto [dt, decay] = step_rate(p, in, head);
     __syncthreads();
     const float *x = mixed, *B = mixed + P, *C = mixed + P + N;
 
@@ -307,7 +322,7 @@ __global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmPara
             float total = 0.0f;
             for (int s = 0; s < slices; ++s) total += partial[(s * (columns <= kStepThreads ? columns : 0)) * V + i];
             const int at = base * V + i;
-            p.y[static_cast<int64_t>(row) * inner + head * P + at] = fmaf(p.d[head], x[at], total);
+            p.y[static_cast<int64_t>(row) * inner + head * P + at] = fmaf(skip_of(p, head), x[at], total);
         }
     }
 }
@@ -460,7 +475,8 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
             }
             S[k][q] = pack2(a, b);
         }
-    const float rate = -expf(p.a_log[head]), dt_bias = p.dt_bias[head], skip = p.d[head];
+    const bool fixed = p.fixed_decay != nullptr;
+    const float rate = fixed ? p.fixed_decay[head] : -expf(p.a_log[head]), dt_bias = fixed ? 0.0f : p.dt_bias[head], skip = skip_of(p, head);
     const int live_columns = min(kColumns, P - column0);
     const bool aligned = ((p.channels | P | N | inner) & 3) == 0 && (reinterpret_cast<uintptr_t>(p.mixed) & 15) == 0;
 
@@ -481,7 +497,7 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
                 }
             }
         }
-        if (threadIdx.x < tokens)
+        if (!fixed && threadIdx.x < tokens)
             copy_async_4(&sdt[buffer][threadIdx.x], p.projected + static_cast<int64_t>(first + t0 + threadIdx.x) * p.stride + inner + p.channels + head);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -498,8 +514,8 @@ __global__ void __launch_bounds__(kScanWarps * 32, LN * Q <= 32 ? 4 : 3) ssm_sca
         if (chunk + 1 < chunks) stage(chunk + 1);
         const int buffer = chunk & 1, t0 = chunk * kScanTokens, tokens = min(kScanTokens, count - t0);
         // step size and decay of token `lane` of the chunk, handed round by shuffles
-        float dt_mine = 0.0f, decay_mine = 1.0f;
-        if (lane < tokens) {
+        float dt_mine = 1.0f, decay_mine = rate;
+        if (!fixed && lane < tokens) {
             dt_mine = softplus(sdt[buffer][lane] + dt_bias);
             decay_mine = expf(rate * dt_mine);
         }
@@ -562,10 +578,12 @@ template <int LN, int Q> int launch_scan(const SsmParams& p, const RowsView& row
     return cuda_status(launch_dependent(ssm_scan_kernel<LN, Q>, grid, dim3(kScanWarps * 32), 0, stream, p, rows), "ssm_scan_kernel launch");
 }
 
-// grid (rows, parts).  V adjacent values per access (4 when everything allows 16-byte accesses).
-template <int V>
+// grid (rows, parts).  V adjacent values per access (4 when everything allows 16-byte accesses).  GATE_FIRST: the norm of y * silu(z);
+// otherwise the norm of y, times sigmoid(z) * factor.
+template <int V, bool GATE_FIRST>
 __global__ void __launch_bounds__(128) gated_group_norm_kernel(const float* y, const float* z, int64_t z_stride, const float* weight, int width,
-                                                               int parts, float eps, float* out, __nv_bfloat16* out_hi, __nv_bfloat16* out_lo) {
+                                                               int parts, float eps, float factor, float* out, __nv_bfloat16* out_hi,
+                                                               __nv_bfloat16* out_lo, int64_t out_stride) {
     __shared__ float scratch[32];
     grid_dependency_wait();
     grid_launch_dependents();
@@ -575,10 +593,12 @@ __global__ void __launch_bounds__(128) gated_group_norm_kernel(const float* y, c
     Lanes<V> kept[kKeep];
     float squares = 0.0f;
     auto value = [&](int c) {
-        const Lanes<V> g = load_lanes<V>(z + row * z_stride + c0 + c), a = load_lanes<V>(y + row * width + c0 + c);
-        Lanes<V> v;
+        Lanes<V> v = load_lanes<V>(y + row * width + c0 + c);
+        if constexpr (GATE_FIRST) {
+            const Lanes<V> g = load_lanes<V>(z + row * z_stride + c0 + c);
 #pragma unroll
-        for (int k = 0; k < V; ++k) v.v[k] = a.v[k] * (g.v[k] * sigmoid_exact(g.v[k]));
+            for (int k = 0; k < V; ++k) v.v[k] *= g.v[k] * sigmoid_exact(g.v[k]);
+        }
         return v;
     };
     auto finish = [&](int c, const Lanes<V>& v, float inverse) {
@@ -586,7 +606,12 @@ __global__ void __launch_bounds__(128) gated_group_norm_kernel(const float* y, c
         Lanes<V> r;
 #pragma unroll
         for (int k = 0; k < V; ++k) r.v[k] = v.v[k] * inverse * w.v[k];
-        const int64_t at = row * width + c0 + c;
+        if constexpr (!GATE_FIRST) {
+            const Lanes<V> g = load_lanes<V>(z + row * z_stride + c0 + c);
+#pragma unroll
+            for (int k = 0; k < V; ++k) r.v[k] *= sigmoid_exact(g.v[k]) * factor;
+        }
+        const int64_t at = row * out_stride + c0 + c;
         if constexpr (V == 4) {
             if (out) store_lanes<V>(out + at, r);
             if (out_hi) {
@@ -622,11 +647,32 @@ __global__ void __launch_bounds__(128) gated_group_norm_kernel(const float* y, c
     for (int c = (threadIdx.x + kKeep * 128) * V; c < size; c += 128 * V) finish(c, value(c), inverse);
 }
 
-__global__ void rows_advance_kernel(const RowsView rows) {
+template <bool GATE_FIRST>
+int launch_group_norm(const float* y, const float* z, int64_t z_stride, const float* weight, int64_t rows, int64_t width, int32_t parts, double eps,
+                      float factor, float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream, const char* what) {
+    if (!y || !z || !weight || rows < 0 || width <= 0 || width > INT32_MAX || parts <= 0 || width % parts || parts > 65535 || (!out && !out_hi)
+        || out_stride < width) {
+        set_error("%s: bad pointer or size", what);
+        return B200_BAD_ARGUMENT;
+    }
+    if (rows == 0) return B200_OK;
+    const bool quads = (width / parts) % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0
+        && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(out)
+             | (reinterpret_cast<uintptr_t>(out_hi) << 1) | (reinterpret_cast<uintptr_t>(out_lo) << 1)) & 15) == 0;
+    return cuda_status(launch_dependent(quads ? gated_group_norm_kernel<4, GATE_FIRST> : gated_group_norm_kernel<1, GATE_FIRST>,
+                                        dim3(static_cast<unsigned>(rows), static_cast<unsigned>(parts)), dim3(128), 0, as_stream(stream), y, z, z_stride,
+                                        weight, static_cast<int>(width), static_cast<int>(parts), static_cast<float>(eps), factor, out,
+                                        static_cast<__nv_bfloat16*>(out_hi), static_cast<__nv_bfloat16*>(out_lo), out_stride),
+                       "gated_group_norm_kernel launch");
+}
+
+__global__ void rows_advance_kernel(const RowsView rows, const int64_t* ids, int32_t* last) {
     grid_dependency_wait();
     grid_launch_dependents();
     const int s = blockIdx.x * blockDim.x + threadIdx.x;
-    if (s < rows.sequences) rows.lengths[rows.slot[s]] += rows.first[s + 1] - rows.first[s];
+    if (s >= rows.sequences) return;
+    rows.lengths[rows.slot[s]] += rows.first[s + 1] - rows.first[s];
+    if (last) last[rows.slot[s]] = static_cast<int32_t>(ids[rows.first[s + 1] - 1]);
 }
 
 __global__ void __launch_bounds__(256) dynamic_tanh_kernel(const float* x, const float* add_rows, const float* add_vector, int width,
@@ -669,7 +715,15 @@ extern "C" {
 int b200_rows_advance(const b200_rows* pass, void* stream) {
     RowsView rows;
     if (!rows_view(pass, rows)) return B200_BAD_ARGUMENT;
-    return cuda_status(launch_dependent(rows_advance_kernel, dim3((rows.sequences + 127) / 128), dim3(128), 0, as_stream(stream), rows),
+    return cuda_status(launch_dependent(rows_advance_kernel, dim3((rows.sequences + 127) / 128), dim3(128), 0, as_stream(stream), rows,
+                                        static_cast<const int64_t*>(nullptr), static_cast<int32_t*>(nullptr)), "rows_advance_kernel launch");
+}
+
+int b200_rows_advance_tokens(const b200_rows* pass, const int64_t* ids, int32_t* last, void* stream) {
+    RowsView rows;
+    if (!rows_view(pass, rows)) return B200_BAD_ARGUMENT;
+    if (!ids || !last) { set_error("b200_rows_advance_tokens: bad pointer"); return B200_BAD_ARGUMENT; }
+    return cuda_status(launch_dependent(rows_advance_kernel, dim3((rows.sequences + 127) / 128), dim3(128), 0, as_stream(stream), rows, ids, last),
                        "rows_advance_kernel launch");
 }
 
@@ -708,15 +762,18 @@ int b200_dynamic_tanh(const float* x, const float* add_rows, const float* add_ve
 int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream) {
     RowsView rows;
     if (!rows_view(pass, rows)) return B200_BAD_ARGUMENT;
-    if (!a || a->heads <= 0 || a->vdim <= 0 || a->state <= 0 || a->groups <= 0 || a->heads % a->groups || a->taps <= 0 || !a->conv_weight
-        || !a->conv_bias || !a->dt_bias || !a->a_log || !a->d || !a->conv_state || !a->ssm_state || !a->projected || !a->y) {
+    if (!a || a->heads <= 0 || a->vdim <= 0 || a->state <= 0 || a->groups <= 0 || a->heads % a->groups || a->taps <= 0
+        || (a->conv_weight ? !a->conv_bias || !a->conv_state : a->taps != 1) || (!a->decay && (!a->dt_bias || !a->a_log || !a->d)) || !a->ssm_state
+        || !a->projected || !a->y || (a->stride && a->stride < 2 * int64_t{a->heads} * a->vdim + 2 * int64_t{a->groups} * a->state + (a->decay ? 0 : a->heads))
+        || a->stride > INT32_MAX) {
         set_error("b200_ssm_forward: bad pointer or size");
         return B200_BAD_ARGUMENT;
     }
     SsmParams p{};
     p.heads = a->heads; p.vdim = a->vdim; p.state = a->state; p.groups = a->groups; p.taps = a->taps;
     p.channels = a->heads * a->vdim + 2 * a->groups * a->state;
-    p.stride = a->heads * a->vdim + p.channels + a->heads;
+    p.stride = a->stride ? static_cast<int>(a->stride) : a->heads * a->vdim + p.channels + (a->decay ? 0 : a->heads);
+    p.fixed_decay = a->decay;
     p.conv_weight = a->conv_weight; p.conv_bias = a->conv_bias; p.dt_bias = a->dt_bias; p.a_log = a->a_log; p.d = a->d;
     p.conv_state = a->conv_state; p.ssm_state = a->ssm_state; p.projected = a->projected; p.mixed = a->mixed; p.y = a->y;
     cudaStream_t s = as_stream(stream);
@@ -733,15 +790,22 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
         if (quads && a->mixed && aligned && a->state % 4 == 0 && a->vdim <= 4 * kStepThreads && streamed <= 110 * 1024 && units >= 4 * resident) {
             int32_t* status = device_status_word(device);
             if (!status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
+            auto stream_steps = [&]() -> int {
+                B200_CUDA(cudaFuncSetAttribute(ssm_step_stream_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(streamed)));
+                return cuda_status(launch_dependent(ssm_step_stream_kernel, dim3(static_cast<unsigned>(std::min(units, resident))), dim3(kStreamThreads), streamed, s, p, rows,
+                                                    status), "ssm_step_stream_kernel launch");
+            };
             // (rows of `projected` start on 16-byte boundaries only when their stride is a multiple of 4)
             const unsigned quads_per_row = static_cast<unsigned>(p.stride % 4 == 0 ? 4 : 1);
+            if (!p.conv_weight) {
+                const int activated = quads_per_row == 4 ? launch_activate<4>(p, rows.rows, s) : launch_activate<1>(p, rows.rows, s);
+                if (activated != B200_OK) return activated;
+                return stream_steps();
+            }
             const dim3 grid((static_cast<unsigned>(p.channels) / quads_per_row + 127) / 128, static_cast<unsigned>(rows.rows));
             const int conv = cuda_status(launch_dependent(quads_per_row == 4 ? conv_step_kernel<4> : conv_step_kernel<1>, grid, dim3(128), 0, s, p, rows),
                                          "conv_step_kernel launch");
-            if (conv != B200_OK) return conv;
-            B200_CUDA(cudaFuncSetAttribute(ssm_step_stream_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(streamed)));
-            return cuda_status(launch_dependent(ssm_step_stream_kernel, dim3(static_cast<unsigned>(std::min(units, resident))), dim3(kStreamThreads), streamed, s, p, rows, status),
-                               "ssm_step_stream_kernel launch");
+            return conv != B200_OK ? conv : stream_steps();
         }
         const size_t smem = sizeof(float) * (((a->vdim + 2 * a->state + 3) & ~3) + kStepThreads * (quads ? 4 : 1));
         if (smem > 200 * 1024) { set_error("b200_ssm_forward: a head of %d x %d values does not fit shared memory", a->state, a->vdim); return B200_UNSUPPORTED; }
@@ -756,9 +820,15 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
     const unsigned blocks = static_cast<unsigned>((p.channels + 255) / 256);
     const bool conv_quads = p.channels % 4 == 0 && p.stride % 4 == 0 && (p.heads * p.vdim) % 4 == 0
         && ((reinterpret_cast<uintptr_t>(p.projected) | reinterpret_cast<uintptr_t>(p.mixed) | reinterpret_cast<uintptr_t>(p.conv_bias)) & 15) == 0;
-    int status = conv_quads ? pick_conv<4>(p, rows, s) : pick_conv<1>(p, rows, s);
-    if (status != B200_OK) return status;
-    status = cuda_status(launch_dependent(conv_ring_kernel, dim3(blocks, static_cast<unsigned>(rows.sequences)), dim3(256), 0, s, p, rows), "conv_ring_kernel launch");
+    int status = B200_OK;
+    if (!p.conv_weight) {
+        if (rows.rows > 65535) { set_error("b200_ssm_forward: at most 65535 rows in one pass"); return B200_UNSUPPORTED; }
+        status = conv_quads ? launch_activate<4>(p, rows.rows, s) : launch_activate<1>(p, rows.rows, s);
+    } else {
+        status = conv_quads ? pick_conv<4>(p, rows, s) : pick_conv<1>(p, rows, s);
+        if (status != B200_OK) return status;
+        status = cuda_status(launch_dependent(conv_ring_kernel, dim3(blocks, static_cast<unsigned>(rows.sequences)), dim3(256), 0, s, p, rows), "conv_ring_kernel launch");
+    }
     if (status != B200_OK) return status;
     if (a->state <= 32) return launch_scan<8, 1>(p, rows, s);
     if (a->state <= 64) return launch_scan<8, 2>(p, rows, s);
@@ -770,19 +840,12 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
 
 int b200_gated_group_norm(const float* y, const float* z, int64_t z_stride, const float* weight, int64_t rows, int64_t width, int32_t parts,
                           double eps, float* out, void* out_hi, void* out_lo, void* stream) {
-    if (!y || !z || !weight || rows < 0 || width <= 0 || width > INT32_MAX || parts <= 0 || width % parts || parts > 65535 || (!out && !out_hi)) {
-        set_error("b200_gated_group_norm: bad pointer or size");
-        return B200_BAD_ARGUMENT;
-    }
-    if (rows == 0) return B200_OK;
-    const bool quads = (width / parts) % 4 == 0 && z_stride % 4 == 0
-        && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(out)
-             | (reinterpret_cast<uintptr_t>(out_hi) << 1) | (reinterpret_cast<uintptr_t>(out_lo) << 1)) & 15) == 0;
-    return cuda_status(launch_dependent(quads ? gated_group_norm_kernel<4> : gated_group_norm_kernel<1>,
-                                        dim3(static_cast<unsigned>(rows), static_cast<unsigned>(parts)), dim3(128), 0, as_stream(stream), y, z, z_stride,
-                                        weight, static_cast<int>(width), static_cast<int>(parts), static_cast<float>(eps), out,
-                                        static_cast<__nv_bfloat16*>(out_hi), static_cast<__nv_bfloat16*>(out_lo)),
-                       "gated_group_norm_kernel launch");
+    return launch_group_norm<true>(y, z, z_stride, weight, rows, width, parts, eps, 1.0f, out, out_hi, out_lo, width, stream, "b200_gated_group_norm");
+}
+
+int b200_norm_gated(const float* y, const float* gate, int64_t gate_stride, const float* weight, int64_t rows, int64_t width, int32_t parts, double eps,
+                    float factor, float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream) {
+    return launch_group_norm<false>(y, gate, gate_stride, weight, rows, width, parts, eps, factor, out, out_hi, out_lo, out_stride, stream, "b200_norm_gated");
 }
 
 }  // extern "C"

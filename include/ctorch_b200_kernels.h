@@ -122,6 +122,14 @@ B200_API int b200_linear(const float* x, int64_t rows, int64_t in, const void* w
                          int64_t out, const void* norm_weight, int32_t norm_dtype, double eps,
                          b200_epilogue epilogue, const float* residual, const b200_qkv_args* qkv, float* y, void* stream);
 
+/* Clamped gated units of the SwiGLU epilogue: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(slope * g) * (u + 1). */
+typedef struct b200_clamped_unit {
+    float slope, limit;
+} b200_clamped_unit;
+/* b200_linear with the SwiGLU epilogue and, where unit is not NULL, those units; y [rows, out/2]. */
+B200_API int b200_linear_units(const float* x, int64_t rows, int64_t in, const void* weight, int32_t weight_dtype, int64_t out,
+                               const b200_clamped_unit* unit, float* y, void* stream);
+
 /* ---- activation shadows (no counterpart in the reference) -------------------------------------------------------
  * Between the kernels of a decode step an f32 activation matrix can travel as a "shadow": two bf16 planes hi + lo
  * (hi = bf16(v), lo = bf16(v - hi), about 16 mantissa bits together), the operand form of the tensor cores.  The
@@ -162,6 +170,7 @@ typedef struct b200_shadow_linear_args {
     const b200_elementwise_norm* out_norm; /* residual epilogue: the norm that follows needs no row statistic; the output shadow holds the
                                       normed rows themselves (out_norm_weight and sumsq_out are then unused) */
     int64_t out_stride;            /* SwiGLU epilogue: elements between rows of the output shadow; 0: out/2 (rows follow each other) */
+    const struct b200_clamped_unit* unit; /* SwiGLU epilogue: the clamped form of the units; NULL: silu(gate) * up */
 } b200_shadow_linear_args;
 /* Up to 16 rows with in <= 2048: streaming kernel (bulk-TMA weight ring, mma.sync).  More rows or a wider input:
  * dense tcgen05 kernel (TMA operand tiles, accumulator in tensor memory; K split over a thread-block cluster when the
@@ -363,6 +372,11 @@ typedef struct b200_ssm_args {
     const float* projected;        /* [rows, 2*heads*vdim + 2*groups*state + heads] */
     float* mixed;                  /* workspace [rows, heads*vdim + 2*groups*state]; may be NULL for passes of one row per sequence */
     float* y;                      /* [rows, heads*vdim] */
+    /* Lightning attention is the same recurrence with fixed decays: S = decay S + k v^T, o = S^T q, with v, k and q in the places of x, B
+     * and C (groups = heads), their SiLU and no step size.  With `decay` set, dt_bias, a_log and d are not read (no skip) and a projected
+     * row has no dt columns; without conv_weight there is no convolution either (taps 1, no conv_state). */
+    const float* decay;            /* [heads] or NULL */
+    int64_t stride;                /* floats between projected rows; 0: the width given above */
 } b200_ssm_args;
 /* Convolution, step sizes, recurrence and its output for every row; the slots' states move on.  Passes with one row per
  * sequence run as one kernel bound by the state's traffic, longer ones as convolution + scan. */
@@ -374,6 +388,11 @@ B200_API int b200_ssm_forward(const b200_ssm_args* args, const b200_rows* pass, 
  * between rows.  Result as f32 (out) and / or shadow planes. */
 B200_API int b200_gated_group_norm(const float* y, const float* z, int64_t z_stride, const float* weight, int64_t rows, int64_t width,
                                    int32_t parts, double eps, float* out, void* out_hi, void* out_lo, void* stream);
+
+/* An RMS norm of each of `parts` equal parts of y's rows, times weight [width], times sigmoid(gate) * factor.  gate has gate_stride floats
+ * between rows, the results out_stride elements. */
+B200_API int b200_norm_gated(const float* y, const float* gate, int64_t gate_stride, const float* weight, int64_t rows, int64_t width,
+                             int32_t parts, double eps, float factor, float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream);
 
 /* One-pool cache of a latent-attention layer: per token kv_rank latent values and the shared rotated key part, width values
  * in all, paged like the other caches with one head.  `lengths` [slots] is the caller's. */
@@ -413,14 +432,14 @@ B200_API int b200_latent_value(const b200_latent_args* args, int64_t rows, const
 /* Name of the kernel b200_latent_attention runs for these sizes: "latent_mma_kernel" or "latent_generic_kernel". */
 B200_API const char* b200_latent_attention_kernel(const b200_latent_args* args);
 
-/* ---- parallel decoders: chunked attention, mixture of experts ---------------------------------------------------------
+/* ---- grouped-query attention in slots, mixture of experts --------------------------------------------------------------
  * (no counterpart in the reference)
  *
- * Chunked grouped-query attention: positions, counted from the start of the sequence, fall into chunks of `chunk`; a position
- * sees its own chunk up to itself.  A slot therefore only keeps the keys and values of the chunk that its next token continues:
+ * Grouped-query attention, optionally in chunks: positions, counted from the start of the sequence, fall into chunks of `chunk`; a
+ * position sees its own chunk up to itself.  A slot therefore only keeps the keys and values of the chunk that its next token continues:
  * key_cache [slots][kv_heads][entries][dim], value_cache [slots][kv_heads][entries][vdim], position p in entry p mod chunk.  A
  * pass with one row per sequence appends before it attends; longer passes attend to the slot and to their own rows (key and
- * value workspaces) and leave the sequence's last chunk in the slot afterwards. */
+ * value workspaces) and leave the sequence's last chunk in the slot afterwards.  Without chunks every pass appends before it attends. */
 typedef struct b200_chunk_args {
     int32_t heads, kv_heads, dim, vdim, rot_dims;
     int32_t slots;                 /* of the caches */
@@ -439,9 +458,24 @@ typedef struct b200_chunk_args {
     const float* projected;        /* rows [q: heads*dim | k: kv_heads*dim | v: kv_heads*vdim | g: heads | ...], stride floats apart */
     int64_t stride;
     void* query;                   /* workspace [rows, heads, dim] */
-    void* key;                     /* workspace [rows, kv_heads, dim]; not used by passes of one row per sequence */
+    void* key;                     /* workspace [rows, kv_heads, dim]; not used by passes of one row per sequence, nor without chunks */
     void* value;                   /* workspace [rows, kv_heads, vdim] */
+    /* Variants; zero is what is described above. */
+    const float* q_bias;           /* [heads*dim] or NULL */
+    const float* k_bias;           /* [kv_heads*dim] or NULL */
+    int32_t norm;                  /* b200_head_norm */
+    int32_t rotate_pairs;          /* 0: entry i turns with entry i + rot_dims / 2; 1: entry 2i with entry 2i + 1 */
+    int32_t keys_as_values;        /* no v columns: the values are the keys (with bias) before norm and rotation; vdim = dim, norm none */
+    int32_t keys_elsewhere;        /* no k and v columns: keys and values are in the slots already, up to the pass's own; without chunks */
+    int32_t no_gate;               /* no g columns */
+    float softcap;                 /* > 0: score <- softcap * tanh(score / softcap) */
+    const float* sink;             /* [heads] or NULL: the softmax's denominator also holds exp(sink) */
+    int32_t scaled;                /* 1: the result is multiplied by out_scale */
+    float out_scale;
 } b200_chunk_args;
+/* Norms of queries and keys: RMS over all heads of the row at once with the weights q_norm and k_norm; none; RMS per head without weights
+ * (after the rotation, which does not change it). */
+enum b200_head_norm { B200_HEAD_NORM_PROJECTION = 0, B200_HEAD_NORM_NONE = 1, B200_HEAD_NORM_HEAD = 2 };
 
 /* Activation of feed-forward units that were projected beside the attention's inputs: `kind` 1: silu(gate) * up of `count` interleaved
  * pairs, 2: exact (erf) gelu of `count` values, starting at column `column` of the projected row.  Result as f32 (out) or planes, out_stride
@@ -465,9 +499,15 @@ typedef struct b200_route {
     float* weight;                 /* [rows, top] */
     int32_t* rank;                 /* [rows, top] the slot's place among the slots of its expert; NULL: not wanted */
     int32_t* counts;               /* [experts] slots per expert, zero before the call (with rank) */
+    /* Variants; zero is what is described above. */
+    int32_t softmax;               /* 1: the scores are the softmax over all outputs */
+    const float* correction;       /* [experts] or NULL: added to the scores for the choice; the weights stay without it */
+    int32_t identity;              /* the last outputs that are identity experts: chosen like the others, but neither ranked nor counted */
 } b200_route;
+/* The choice alone, for `rows` rows of logits with `stride` floats between them (route->column is not used). */
+B200_API int b200_route_rows(const float* logits, int64_t rows, int64_t stride, const b200_route* route, void* stream);
 
-/* Everything that stands between the projection of a parallel layer and its attention: norms and rotation of queries and keys, append
+/* Everything that stands between the projection of a layer and its attention: norms and rotation of queries and keys, append
  * (or workspaces), the activation of the feed-forward units (units may be NULL) and the router's choice (route may be NULL). */
 B200_API int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* pass, const b200_units* units, const b200_route* route, void* stream);
 /* softmax(scale q.k) v over the visible keys, times sigmoid(g) of the head; out f32 or planes, out_stride elements between rows.
@@ -498,7 +538,48 @@ typedef struct b200_experts {
     double eps;
     const float* residual;         /* [rows, in] */
     float* y;                      /* [rows, in] = residual + sum over the choices; may equal residual */
+    /* Variants; zero is what is described above. */
+    int32_t gated;                 /* 1: `up` holds gate and up rows interleaved, [experts][2 ff][in], and expert(x) = down (silu(gate x) * (up x)) */
+    int32_t weigh_results;         /* 1: the score multiplies the expert's result instead of its input */
+    int32_t identity;              /* outputs of the router past `experts` whose result is the input itself (chosen ids experts, ...) */
+    const struct b200_sandwich* after; /* grouped form: the sum goes through b200_sandwich_rows instead of being added to residual (which,
+                                      like y, may then be NULL) */
 } b200_experts;
+/* The end of a sublayer that has a norm behind it: x = residual + rms(y) * after, and the norm before the next sublayer, rms(x) * next, as
+ * f32 (normed) and / or planes.  rms(v) = v / sqrt(mean(v^2) + eps). */
+typedef struct b200_sandwich {
+    const float* after;            /* [width] f32 */
+    const float* next;             /* [width] f32, or NULL: no norm follows */
+    double eps;
+    const float* residual;         /* [rows, width] */
+    float* x;                      /* [rows, width]; may equal residual */
+    float* normed;
+    void* normed_hi;
+    void* normed_lo;
+} b200_sandwich;
+B200_API int b200_sandwich_rows(const float* y, int64_t rows, int64_t width, const b200_sandwich* args, void* stream);
+
+/* Embedding of tokens and of pairs of tokens: x = table[id] + pairs[row], row = (previous id * mul_prev + id * mul_cur) mod buckets, or
+ * row `buckets` for a sequence's first token; and rms(x) * next as in b200_sandwich.  The token before a pass's first is in last [slots]. */
+typedef struct b200_pair_embedding {
+    const void* table;             /* [vocab, width] */
+    const void* pairs;             /* [buckets + 1, width] */
+    int32_t dtype;
+    int64_t vocab, width, buckets, mul_prev, mul_cur;
+    const int32_t* last;
+    const float* next;             /* [width] f32 or NULL */
+    double eps;
+    float* x;
+    float* normed;
+    void* normed_hi;
+    void* normed_lo;
+} b200_pair_embedding;
+B200_API int b200_embed_pairs(const b200_pair_embedding* args, const int64_t* ids, const b200_rows* pass, void* stream);
+/* b200_rows_advance that also leaves every sequence's last token in last[slot]. */
+B200_API int b200_rows_advance_tokens(const b200_rows* pass, const int64_t* ids, int32_t* last, void* stream);
+/* x <- cap * tanh(x / cap) */
+B200_API int b200_soft_cap(float* x, int64_t count, float cap, void* stream);
+
 /* Few slots, f32 weights, odd sizes: every slot streams its expert.  act: workspace f32 [rows, top, ff]. */
 B200_API int b200_experts_streamed(const b200_experts* args, float* act, void* stream);
 /* Many slots (bf16, in and ff multiples of 8, planes): the slots are sorted by expert and multiplied on the tensor cores in tiles of

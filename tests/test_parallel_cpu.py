@@ -39,7 +39,7 @@ def broken(change):
     (lambda c: c["layers"][1]["mlp"].pop("expert"), r"mlp\.expert' is missing"),
     (lambda c: c["loop"].update(stop=5), "range of layers"),
     (lambda c: c["norm"].pop("eps"), "eps' is missing"),
-    (lambda c: c.update(architecture="Ripitar", embedding={"scale": 1.0}, logit_scale=1.0), "parallel layers"),
+    (lambda c: c.update(architecture="Ripitar", embedding={"scale": 1.0}, logit_scale=1.0), "unknown layer type 'attention'"),
 ])
 def test_configuration_errors_name_the_key(change, message):
     with pytest.raises(B.B200Error, match=message):
