@@ -162,6 +162,27 @@ def parallel_config(width: int, layers: int, ff: int, heads: int, kv_heads: int,
     return config
 
 
+def sandwich_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, experts: int, lightning_heads: int, top: int = 2, identity: int = 2,
+                    vocab: int = 32000) -> dict:
+    """Sandwich decoder of a real model's layer sizes: its three mixers in turn, the second kind of attention twice (the second time with the
+    first's keys); dense and mixture layers in turn, `top` experts with the dense feed-forward's weights."""
+    dim = width // heads
+    rot = {"dims": dim, "base": 500000.0}
+    sizes = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    mlps = ({"kind": "dense", "ff": ff, "limit": 7.0},
+            {"kind": "moe", "router": {"experts": experts, "top": top, "identity": identity}, "expert": {"ff": ff // top}})
+    decay = [float(1.0 - 2.0 ** -(1 + 8.0 * h / lightning_heads)) for h in range(lightning_heads)]
+    mixers = (("attention", {**sizes, "rot": rot}), ("attention_2", {**sizes, "rot": rot, "softcap": 50.0}),
+              ("parallel", {"left": sizes, "right": {"heads": lightning_heads, "dim": 128, "vdim": 128, "decay": decay}, "left_scale": 0.6, "right_scale": 0.5}),
+              ("attention_2", {**sizes, "rot": rot, "softcap": 50.0}))
+    config = {"architecture": "Lozepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [],
+              "embedding": {"bigram": {"buckets": vocab - 1, "mul_prev": 1021, "mul_cur": 31}}}
+    for i in range(layers):
+        kind, mixer = mixers[i % 4]
+        config["layers"].append({"type": kind, "mixer": {**mixer, "kv_from": i - 2} if i % 4 == 3 else mixer, "mlp": mlps[i % 2]})
+    return config
+
+
 def transformer_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, context: int, vocab: int = 32000) -> dict:
     return {"architecture": "TransformerDecoder", "vocab": vocab, "layers": layers, "width": width, "heads": heads, "kv_heads": kv_heads,
             "ff": ff, "context": context, "tied": 1}
@@ -181,6 +202,13 @@ PARALLEL_SIZES = {
     "4k": (dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8, experts=8), HYBRID_SIZES["4k"][1]),
 }
 
+# (sandwich, grouped-query) arguments, likewise
+SANDWICH_SIZES = {
+    "1k": (dict(width=1024, layers=12, ff=4096, heads=16, kv_heads=4, experts=16, lightning_heads=8), HYBRID_SIZES["1k"][1]),
+    "2k": (dict(width=2048, layers=16, ff=8192, heads=32, kv_heads=8, experts=16, lightning_heads=16), HYBRID_SIZES["2k"][1]),
+    "4k": (dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8, experts=8, lightning_heads=32), HYBRID_SIZES["4k"][1]),
+}
+
 
 def random_state(shapes: dict[str, tuple[int, ...]], seed: int = 7) -> dict[str, np.ndarray]:
     """bf16 bit patterns for every named shape, cut from one seeded block (norm-like vectors around 1)."""
@@ -191,6 +219,8 @@ def random_state(shapes: dict[str, tuple[int, ...]], seed: int = 7) -> dict[str,
         values = np.resize(block[i * 9973 % 65536:], count).reshape(shape)
         if len(shape) == 2:
             values = values * np.float32(shape[1] ** -0.5)
+        elif name.endswith("correction"):   # the scores decide, so that the experts share the rows
+            values = 0.002 * values
         elif not name.endswith((".b", "A_log", "dt_bias")):
             values = 1.0 + 0.05 * values
         else:
