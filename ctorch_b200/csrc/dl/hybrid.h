@@ -42,7 +42,7 @@ struct AttentionKind {
     b200_head_norm norm = B200_HEAD_NORM_PROJECTION;
     bool rotate_pairs = false;     // entry 2i with entry 2i + 1; otherwise halves
     bool bias = false;             // on queries and keys
-    bool keys_as_values = false;   // the values are the keys before their rotation
+    bool keys_as_values = false;   // unrotated, the keys serve as values too
     bool gate = false;             // one output gate per head
     Sink sink = Sink::none;
 };

@@ -165,10 +165,11 @@ __device__ __forceinline__ Span<V> turned_span(const ChunkParams& p, const float
 constexpr int kPrepareThreads = 256, kUnitSlice = 1024;
 // grid (rows, 1 + slices of the units)
 
-template <class T, int V>
+// NORM: b200_head_norm
+template <class T, int V, int NORM>
 __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __grid_constant__ ChunkParams p, const RowsView rows, const bool step,
                                                                         const __grid_constant__ Units units, const __grid_constant__ Route route) {
-    extern __shared__ float extra[];   // [experts] for the router, then one factor per query and key head
+    extern __shared__ float logits_copy[];
     __shared__ float scratch[32];
     grid_dependency_wait();
     grid_launch_dependents();
@@ -210,58 +211,72 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
         return;
     }
     if (route.experts > 0 && threadIdx.x >= kPrepareThreads - 32)
-        choose_experts(route, row, source + route.column, extra, threadIdx.x & 31);
+        choose_experts(route, row, source + route.column, logits_copy, threadIdx.x & 31);
     const int sequence = __ldg(rows.sequence + row);
     const int q_count = p.heads * p.dim, k_count = p.key_columns(), v_count = p.keys_elsewhere ? 0 : p.kv_heads * p.vdim;
     const float *k_source = source + q_count, *v_source = p.keys_as_values ? k_source : k_source + k_count;
     const float* v_bias = p.keys_as_values ? p.k_bias : nullptr;
+    float q_inverse = 1.0f, k_inverse = 1.0f, qs = 0.0f, ks = 0.0f;
+    if constexpr (NORM == B200_HEAD_NORM_PROJECTION) {
+        qs = squares_of<V>(source, p.q_bias, 0, q_count, threadIdx.x, kPrepareThreads);
+        ks = squares_of<V>(k_source, p.k_bias, 0, k_count, threadIdx.x, kPrepareThreads);
+    }
+    // where the row belongs: a chain of dependent loads, spread between the sums
     const int slot = __ldg(rows.slot + sequence), first = __ldg(rows.first + sequence), end = __ldg(rows.first + sequence + 1);
+    if constexpr (NORM == B200_HEAD_NORM_PROJECTION) {
+        qs = warp_sum(qs);
+        ks = warp_sum(ks);
+    }
     const int length = rows.lengths[slot];
-    float q_inverse = 1.0f, k_inverse = 1.0f;
-    float* inverses = extra + route.experts;   // (norm per head)
-    if (p.norm == B200_HEAD_NORM_PROJECTION) {
-        const float qs = warp_sum(squares_of<V>(source, p.q_bias, 0, q_count, threadIdx.x, kPrepareThreads));
-        const float ks = warp_sum(squares_of<V>(k_source, p.k_bias, 0, k_count, threadIdx.x, kPrepareThreads));
+    if constexpr (NORM == B200_HEAD_NORM_PROJECTION) {
         if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = qs; scratch[kPrepareThreads / 32 + (threadIdx.x >> 5)] = ks; }
         __syncthreads();
-        float q_total = 0.0f, k_total = 0.0f;
+        qs = ks = 0.0f;
 #pragma unroll
-        for (int w = 0; w < kPrepareThreads / 32; ++w) { q_total += scratch[w]; k_total += scratch[kPrepareThreads / 32 + w]; }
-        q_inverse = 1.0f / sqrtf(q_total / static_cast<float>(q_count) + p.eps);
-        k_inverse = 1.0f / sqrtf(k_total / static_cast<float>(max(k_count, 1)) + p.eps);
-    } else if (p.norm == B200_HEAD_NORM_HEAD) {
-        const int heads = p.heads + (p.keys_elsewhere ? 0 : p.kv_heads);   // the key heads follow the query heads in the row
-        for (int h = threadIdx.x >> 5; h < heads; h += kPrepareThreads / 32) {
-            const bool is_query = h < p.heads;
-            const int begin = (is_query ? h : h - p.heads) * p.dim;
-            const float squares = warp_sum(squares_of<V>(is_query ? source : k_source, is_query ? p.q_bias : p.k_bias, begin, begin + p.dim, threadIdx.x & 31, 32));
-            if ((threadIdx.x & 31) == 0) inverses[h] = 1.0f / sqrtf(squares / static_cast<float>(p.dim) + p.eps);
-        }
-        __syncthreads();
+        for (int w = 0; w < kPrepareThreads / 32; ++w) { qs += scratch[w]; ks += scratch[kPrepareThreads / 32 + w]; }
+        q_inverse = 1.0f / sqrtf(qs / static_cast<float>(q_count) + p.eps);
+        k_inverse = 1.0f / sqrtf(ks / static_cast<float>(max(k_count, 1)) + p.eps);
     }
     const int position = length + row - first, last = length + end - first - 1;
     // The slot takes the row at once where it ends up there and nothing that this pass still reads is overwritten.
     const bool first_appended = p.appends_first(step);
     const bool stored = first_appended || (p.chunk_start(position) == p.chunk_start(last) && !p.overwrites(length, last));
+    const bool to_slot = stored && p.fits(position);   // (the host refuses passes that do not fit)
     const int half = p.rot_dims >> 1;
     const bool turns = half > 0 && position < p.positions;
     const float* cosine = turns ? p.cosine + static_cast<int64_t>(position) * half : nullptr;
     const float* sine = turns ? p.sine + static_cast<int64_t>(position) * half : nullptr;
-    const float* q_weight = p.norm == B200_HEAD_NORM_PROJECTION ? p.q_norm : nullptr;
-    const float* k_weight = p.norm == B200_HEAD_NORM_PROJECTION ? p.k_norm : nullptr;
-    for (int c = threadIdx.x * V; c < q_count; c += kPrepareThreads * V) {
-        const int head = c / p.dim, d = c - head * p.dim;
-        const float inverse = p.norm == B200_HEAD_NORM_HEAD ? inverses[head] : q_inverse;
-        store_span<V>(static_cast<T*>(p.query) + static_cast<int64_t>(row) * q_count + c,
-                      turned_span<V>(p, source, p.q_bias, q_weight, c, d, inverse, cosine, sine));
-    }
-    const bool to_slot = stored && p.fits(position);   // (the host refuses passes that do not fit)
-    for (int c = threadIdx.x * V; c < k_count; c += kPrepareThreads * V) {
-        const int head = c / p.dim, d = c - head * p.dim;
-        const float inverse = p.norm == B200_HEAD_NORM_HEAD ? inverses[p.heads + head] : k_inverse;
-        const Span<V> v = turned_span<V>(p, k_source, p.k_bias, k_weight, c, d, inverse, cosine, sine);
+    auto store_query = [&](int c, const Span<V>& v) { store_span<V>(static_cast<T*>(p.query) + static_cast<int64_t>(row) * q_count + c, v); };
+    auto store_key = [&](int head, int d, const Span<V>& v) {
         if (to_slot) store_span<V>(static_cast<T*>(p.key_cache) + p.entry(slot, head, position) * p.dim + d, v);
-        if (!first_appended) store_span<V>(static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + c, v);
+        if (!first_appended) store_span<V>(static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + head * p.dim + d, v);
+    };
+    if constexpr (NORM == B200_HEAD_NORM_HEAD) {
+        // a power of two of neighbouring lanes per head, as many as its entries occupy; the key heads follow the query heads
+        const int lanes = p.dim > 16 * V ? 32 : p.dim > 8 * V ? 16 : 8, lane = threadIdx.x & (lanes - 1), at_once = kPrepareThreads / lanes;
+        const int heads = p.heads + (p.keys_elsewhere ? 0 : p.kv_heads);
+        for (int h0 = 0; h0 < heads; h0 += at_once) {
+            const int h = h0 + static_cast<int>(threadIdx.x) / lanes;
+            const bool live = h < heads, is_query = h < p.heads;
+            const float *part = is_query ? source : k_source, *bias = is_query ? p.q_bias : p.k_bias;
+            const int head = is_query ? h : h - p.heads, begin = head * p.dim;
+            float squares = live ? squares_of<V>(part, bias, begin, begin + p.dim, lane, lanes) : 0.0f;
+            for (int o = lanes >> 1; o > 0; o >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, o);
+            const float inverse = 1.0f / sqrtf(squares / static_cast<float>(p.dim) + p.eps);
+            for (int d = lane * V; live && d < p.dim; d += lanes * V) {
+                const Span<V> v = turned_span<V>(p, part, bias, nullptr, begin + d, d, inverse, cosine, sine);
+                if (is_query) store_query(begin + d, v);
+                else store_key(head, d, v);
+            }
+        }
+    } else {
+        constexpr bool kWeighted = NORM == B200_HEAD_NORM_PROJECTION;
+        for (int c = threadIdx.x * V; c < q_count; c += kPrepareThreads * V)
+            store_query(c, turned_span<V>(p, source, p.q_bias, kWeighted ? p.q_norm : nullptr, c, c % p.dim, q_inverse, cosine, sine));
+        for (int c = threadIdx.x * V; c < k_count; c += kPrepareThreads * V) {
+            const int head = c / p.dim, d = c - head * p.dim;
+            store_key(head, d, turned_span<V>(p, k_source, p.k_bias, kWeighted ? p.k_norm : nullptr, c, d, k_inverse, cosine, sine));
+        }
     }
     for (int c = threadIdx.x * V; c < v_count; c += kPrepareThreads * V) {
         const int head = c / p.vdim, d = c - head * p.vdim;
@@ -982,11 +997,19 @@ extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* 
         && aligned(p.k_norm) && aligned(p.q_bias) && aligned(p.k_bias) && aligned(p.query) && aligned(p.key) && aligned(p.value) && aligned(p.key_cache) && aligned(p.value_cache)
         && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0
         && (u.kind == 0 || (u.column % 4 == 0 && u.count % 4 == 0 && u.stride % 4 == 0 && aligned(u.out) && aligned8(u.out_hi) && aligned8(u.out_lo)));
-    auto kernel = args->dtype == B200_BF16 ? (vector ? chunk_prepare_kernel<__nv_bfloat16, 4> : chunk_prepare_kernel<__nv_bfloat16, 1>)
-                                           : (vector ? chunk_prepare_kernel<float, 4> : chunk_prepare_kernel<float, 1>);
     const dim3 grid(static_cast<unsigned>(rows.rows), static_cast<unsigned>(1 + (u.count + kUnitSlice - 1) / kUnitSlice));
-    return cuda_status(launch_dependent(kernel, grid, dim3(kPrepareThreads), (static_cast<size_t>(r.experts) + (p.norm == B200_HEAD_NORM_HEAD ? p.heads + p.kv_heads : 0)) * 4,
-                                        as_stream(stream), p, rows, step, u, r), "chunk_prepare_kernel launch");
+    auto launch = [&](auto norm) {
+        constexpr int kNorm = decltype(norm)::value;
+        auto kernel = args->dtype == B200_BF16 ? (vector ? chunk_prepare_kernel<__nv_bfloat16, 4, kNorm> : chunk_prepare_kernel<__nv_bfloat16, 1, kNorm>)
+                                               : (vector ? chunk_prepare_kernel<float, 4, kNorm> : chunk_prepare_kernel<float, 1, kNorm>);
+        return cuda_status(launch_dependent(kernel, grid, dim3(kPrepareThreads), static_cast<size_t>(r.experts) * 4, as_stream(stream), p, rows, step, u, r),
+                           "chunk_prepare_kernel launch");
+    };
+    switch (p.norm) {
+    case B200_HEAD_NORM_NONE: return launch(std::integral_constant<int, B200_HEAD_NORM_NONE>{});
+    case B200_HEAD_NORM_HEAD: return launch(std::integral_constant<int, B200_HEAD_NORM_HEAD>{});
+    default: return launch(std::integral_constant<int, B200_HEAD_NORM_PROJECTION>{});
+    }
 }
 
 extern "C" size_t b200_chunk_scratch_bytes(const b200_chunk_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length) {

@@ -167,15 +167,15 @@ def sandwich_config(width: int, layers: int, ff: int, heads: int, kv_heads: int,
     """Sandwich decoder of a real model's layer sizes: its three mixers in turn, the second kind of attention twice (the second time with the
     first's keys); dense and mixture layers in turn, `top` experts with the dense feed-forward's weights."""
     dim = width // heads
-    rot = {"dims": dim, "base": 500000.0}
+    rot = {"dims": dim, "base": 100000.0}
     sizes = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
     mlps = ({"kind": "dense", "ff": ff, "limit": 7.0},
             {"kind": "moe", "router": {"experts": experts, "top": top, "identity": identity}, "expert": {"ff": ff // top}})
     decay = [float(1.0 - 2.0 ** -(1 + 8.0 * h / lightning_heads)) for h in range(lightning_heads)]
-    mixers = (("attention", {**sizes, "rot": rot}), ("attention_2", {**sizes, "rot": rot, "softcap": 50.0}),
-              ("parallel", {"left": sizes, "right": {"heads": lightning_heads, "dim": 128, "vdim": 128, "decay": decay}, "left_scale": 0.6, "right_scale": 0.5}),
-              ("attention_2", {**sizes, "rot": rot, "softcap": 50.0}))
-    config = {"architecture": "Lozepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [],
+    mixers = (("attention", {**sizes, "rot": rot}), ("attention_2", {**sizes, "rot": rot, "softcap": 40.0}),
+              ("parallel", {"left": sizes, "right": {"heads": lightning_heads, "dim": 128, "vdim": 128, "decay": decay}, "left_scale": 0.8, "right_scale": 0.4}),
+              ("attention_2", {**sizes, "rot": rot, "softcap": 40.0}))
+    config = {"architecture": "Lozepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 20.0, "layers": [],
               "embedding": {"bigram": {"buckets": vocab - 1, "mul_prev": 1021, "mul_cur": 31}}}
     for i in range(layers):
         kind, mixer = mixers[i % 4]

@@ -215,14 +215,15 @@ DL_API dl_status dl_decoder_generate(dl_module* decoder, dl_module* embedding, d
 /* ---- models from configurations (no counterpart in the reference) -----------------------------------------
  * A model design is chosen by "architecture" of a JSON configuration: "Ripitar" (hybrid decoder: state-space and latent-attention
  * layers, Dynamic Tanh norms, looped layers), "Sinezen" (parallel decoder: chunked attention beside a feed-forward or a mixture of
- * experts, RMS norms, looped layers) or "TransformerDecoder" (the grouped-query decoder above with its embedding and
+ * experts, RMS norms, looped layers), "Lozepel" (sandwich decoder: a norm before and after every sublayer, three mixers, a clamped
+ * feed-forward or a mixture of gated experts, pair embedding, capped logits) or "TransformerDecoder" (the grouped-query decoder above with its embedding and
  * output layers; keys vocab, layers, width, heads, kv_heads, ff, context, tied). */
 DL_API const char* dl_model_architectures(void);   /* comma-separated */
 DL_API dl_status dl_model_create(const char* config_json, dl_tensor_options options, dl_module** output);
 /* config.json and model.safetensors of a folder; weights are converted to options.dtype (DL_BF16 or DL_F32). */
 DL_API dl_status dl_model_load(const char* folder, dl_tensor_options options, dl_module** output);
 DL_API dl_status dl_state_load_safetensors(const char* path, dl_state** output);
-/* Decoders with a slot cache (the first two): `slots` sequences of up to `capacity` tokens.  Grouped-query decoders: their own caches (both numbers unused). */
+/* Decoders with a slot cache (the first three): `slots` sequences of up to `capacity` tokens.  Grouped-query decoders: their own caches (both numbers unused). */
 DL_API dl_status dl_model_cache_create(const dl_module* model, int64_t slots, int64_t capacity, dl_decoder_cache** output);
 DL_API dl_status dl_model_cache_release_slot(dl_decoder_cache* cache, int64_t slot);
 DL_API dl_status dl_model_cache_slot_length(const dl_decoder_cache* cache, int64_t slot, int64_t* length);

@@ -465,7 +465,7 @@ typedef struct b200_chunk_args {
     const float* k_bias;           /* [kv_heads*dim] or NULL */
     int32_t norm;                  /* b200_head_norm */
     int32_t rotate_pairs;          /* 0: entry i turns with entry i + rot_dims / 2; 1: entry 2i with entry 2i + 1 */
-    int32_t keys_as_values;        /* no v columns: the values are the keys (with bias) before norm and rotation; vdim = dim, norm none */
+    int32_t keys_as_values;        /* no v columns: the biased keys, unrotated, serve as values too; vdim = dim, norm none */
     int32_t keys_elsewhere;        /* no k and v columns: keys and values are in the slots already, up to the pass's own; without chunks */
     int32_t no_gate;               /* no g columns */
     float softcap;                 /* > 0: score <- softcap * tanh(score / softcap) */

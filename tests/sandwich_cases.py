@@ -29,7 +29,7 @@ def second(heads, kv_heads, dim, vdim, mlp, softcap=20.0, **more):
     return rotating("attention_2", heads, kv_heads, dim, vdim, mlp, softcap=softcap, **more)
 
 
-def pair(left, right, mlp, scales=(0.6, 1.3), scale=None):
+def pair(left, right, mlp, scales=(0.75, 1.3), scale=None):
     (heads, kv_heads, dim, vdim), (rheads, rdim, rvdim, decay) = left, right
     assert len(decay) == rheads
     return {"type": "parallel", "mlp": mlp,

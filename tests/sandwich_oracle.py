@@ -64,7 +64,7 @@ def heads_of(x, heads):
 
 
 def attention_keys_as_values(h, w, p, m):
-    """Biased queries and keys, rotated; the values are the keys before rotation; a sink of score 0; one gate per head."""
+    """Biased queries and keys, rotated; unrotated, the keys serve as values too; a sink of score 0; one gate per head."""
     H, G, pos = m["heads"], m["kv_heads"], np.arange(h.shape[0])
     q = heads_of(h @ w[p + "q"].T + w[p + "q.b"], H)
     k = heads_of(h @ w[p + "k"].T + w[p + "k.b"], G)

@@ -140,7 +140,7 @@ def test_choice_is_corrected_and_weights_are_not():
     assert np.allclose(got, 0.2 + 0.5 * 2.0 * O.silu(1.0))
 
 
-def test_values_are_the_keys_before_rotation():
+def test_unrotated_keys_serve_as_values():
     h = np.eye(2)
     w = {"q": np.zeros((2, 2)), "q.b": np.zeros(2), "k": 5.0 * np.eye(2), "k.b": np.array([1.0, 2.0]), "g": np.zeros((1, 2)), "o": np.eye(2)}
     m = {"heads": 1, "kv_heads": 1, "rot": {"dims": 2, "base": 10.0}, "scale": 1.0}

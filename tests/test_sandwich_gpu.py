@@ -113,8 +113,8 @@ class Grouped:
 GROUPED = [dict(kind=1, heads=4, kv_heads=2, dim=16, vdim=16), dict(kind=1, heads=3, kv_heads=1, dim=10, vdim=10, dims=6), dict(kind=1, heads=40, kv_heads=1, dim=96, vdim=96, factor=0.5),
            dict(kind=1, heads=2, kv_heads=2, dim=256, vdim=256, dims=20), dict(kind=1, heads=6, kv_heads=2, dim=20, vdim=20, dims=6),
            dict(kind=2, heads=4, kv_heads=2, dim=24, vdim=16, cap=4.0), dict(kind=2, heads=3, kv_heads=3, dim=10, vdim=14, cap=2.0, dims=2),
-           dict(kind=2, heads=1, kv_heads=1, dim=64, vdim=64), dict(kind=2, heads=20, kv_heads=1, dim=128, vdim=64, cap=1.0, scale=1.0), dict(kind=2, heads=2, kv_heads=1, dim=192, vdim=96, cap=50.0),
-           dict(kind=3, heads=8, kv_heads=2, dim=64, vdim=64, factor=0.6), dict(kind=3, heads=3, kv_heads=1, dim=10, vdim=6, factor=-1.5), dict(kind=3, heads=4, kv_heads=4, dim=72, vdim=128)]
+           dict(kind=2, heads=1, kv_heads=1, dim=64, vdim=64), dict(kind=2, heads=20, kv_heads=1, dim=128, vdim=64, cap=1.0, scale=1.0), dict(kind=2, heads=2, kv_heads=1, dim=192, vdim=96, cap=45.0),
+           dict(kind=3, heads=8, kv_heads=2, dim=64, vdim=64, factor=0.7), dict(kind=3, heads=3, kv_heads=1, dim=10, vdim=6, factor=-1.5), dict(kind=3, heads=4, kv_heads=4, dim=72, vdim=128)]
 
 
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
@@ -192,7 +192,7 @@ def test_one_key_stands_out(kind, heads, kv_heads, dtype):
     assert at <= T
 
 
-@pytest.mark.parametrize("kind, group, dim, vdim, cap", [(1, 4, 64, 64, 0.0), (2, 1, 128, 128, 3.0), (3, 20, 64, 48, 0.0), (2, 6, 48, 48, 50.0)])
+@pytest.mark.parametrize("kind, group, dim, vdim, cap", [(1, 4, 64, 64, 0.0), (2, 1, 128, 128, 3.0), (3, 20, 64, 48, 0.0), (2, 6, 40, 56, 45.0)])
 def test_split_keys_of_a_step(kind, group, dim, vdim, cap):
     """Few long sequences: the keys of a step are split over CTAs, the sink joins once."""
     k = Grouped(kind, group, 1, dim, vdim, "bf16", slots=3, capacity=2100, cap=cap, sinks=np.full(group, 6.0), seed=group)
@@ -347,9 +347,9 @@ def test_pair_embedding(dtype, width):
 def test_capped_logits():
     x = np.random.default_rng(0).normal(0, 40, 70001)
     t = dev(x)
-    B.kcheck(B.lib().b200_soft_cap(t.data_ptr(), x.size, 30.0, None))
+    B.kcheck(B.lib().b200_soft_cap(t.data_ptr(), x.size, 35.0, None))
     torch.cuda.synchronize()
-    assert ratio(t.cpu(), O.soft_cap(x, 30.0)) < 1e-6
+    assert ratio(t.cpu(), O.soft_cap(x, 35.0)) < 1e-6
 
 
 # ---- feed-forwards ----------------------------------------------------------------------------------------------
