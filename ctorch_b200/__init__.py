@@ -71,7 +71,7 @@ class SsmArgs(C.Structure):
     _fields_ = [("heads", C.c_int32), ("vdim", C.c_int32), ("state", C.c_int32), ("groups", C.c_int32), ("taps", C.c_int32),
                 ("conv_weight", C.c_void_p), ("conv_bias", C.c_void_p), ("dt_bias", C.c_void_p), ("a_log", C.c_void_p), ("d", C.c_void_p),
                 ("conv_state", C.c_void_p), ("ssm_state", C.c_void_p), ("projected", C.c_void_p), ("mixed", C.c_void_p), ("y", C.c_void_p),
-                ("decay", C.c_void_p), ("stride", C.c_int64)]
+                ("decay", C.c_void_p), ("stride", C.c_int64), ("delta", C.c_int32)]
 
 
 class LatentArgs(C.Structure):
@@ -90,7 +90,9 @@ class ChunkArgs(C.Structure):
                 ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("dtype", C.c_int32), ("key_cache", C.c_void_p), ("value_cache", C.c_void_p),
                 ("projected", C.c_void_p), ("stride", C.c_int64), ("query", C.c_void_p), ("key", C.c_void_p), ("value", C.c_void_p),
                 ("q_bias", C.c_void_p), ("k_bias", C.c_void_p), ("norm", C.c_int32), ("rotate_pairs", C.c_int32), ("keys_as_values", C.c_int32),
-                ("keys_elsewhere", C.c_int32), ("no_gate", C.c_int32), ("softcap", C.c_float), ("sink", C.c_void_p), ("scaled", C.c_int32), ("out_scale", C.c_float)]
+                ("keys_elsewhere", C.c_int32), ("no_gate", C.c_int32), ("softcap", C.c_float), ("sink", C.c_void_p), ("scaled", C.c_int32), ("out_scale", C.c_float),
+                ("window", C.c_int32), ("keep", C.c_int32), ("pool", C.c_int32), ("pool_state", C.c_void_p), ("norm_values", C.c_int32), ("gate_values", C.c_int32),
+                ("talk", C.c_void_p)]
 
 
 class Units(C.Structure):
@@ -100,13 +102,13 @@ class Units(C.Structure):
 
 class Route(C.Structure):
     _fields_ = [("experts", C.c_int32), ("top", C.c_int32), ("column", C.c_int64), ("chosen", C.c_void_p), ("weight", C.c_void_p), ("rank", C.c_void_p),
-                ("counts", C.c_void_p), ("softmax", C.c_int32), ("correction", C.c_void_p), ("identity", C.c_int32)]
+                ("counts", C.c_void_p), ("softmax", C.c_int32), ("correction", C.c_void_p), ("identity", C.c_int32), ("bias", C.c_void_p), ("chosen_softmax", C.c_int32)]
 
 
 class Sandwich(C.Structure):
     """The end of a sublayer with a norm behind it: b200_sandwich."""
     _fields_ = [("after", C.c_void_p), ("next", C.c_void_p), ("eps", C.c_double), ("residual", C.c_void_p), ("x", C.c_void_p), ("normed", C.c_void_p),
-                ("normed_hi", C.c_void_p), ("normed_lo", C.c_void_p)]
+                ("normed_hi", C.c_void_p), ("normed_lo", C.c_void_p), ("plain", C.c_int32)]
 
 
 class PairEmbedding(C.Structure):
@@ -259,6 +261,7 @@ def _declare(l: C.CDLL) -> None:
         "b200_embedding_scaled": (C.c_int, [vp, i32, vp, i64, i64, i64, C.c_float, vp, vp]),
         "b200_dynamic_tanh": (C.c_int, [vp, vp, vp, i64, i64, C.POINTER(ElementwiseNorm), vp, vp, vp, vp, vp]),
         "b200_ssm_forward": (C.c_int, [C.POINTER(SsmArgs), C.POINTER(Rows), vp]),
+        "b200_head_norm_gated": (C.c_int, [vp, vp, i64, vp, i64, i32, i32, C.c_double, vp, vp, vp, i64, vp]),
         "b200_gated_group_norm": (C.c_int, [vp, vp, i64, vp, i64, i64, i32, C.c_double, vp, vp, vp, vp]),
         "b200_latent_cache_create": (C.c_int, [i32, i32, i32, i32, i32, i32, vp, pp]),
         "b200_latent_prepare": (C.c_int, [C.POINTER(LatentArgs), C.POINTER(Rows), vp, vp, vp, vp, vp]),

@@ -1,5 +1,5 @@
 // Modules, cache, execution plan and generation of the configured decoders (see hybrid.h, hybrid_plan.h; parallel layers: parallel.cpp,
-// sandwich layers: sandwich.cpp).
+// layers with norms behind the sublayers: sandwich.cpp, delta.cpp).
 #include "dl/hybrid_plan.h"
 
 #include <algorithm>
@@ -47,10 +47,21 @@ GroupedAttentionConfig attention_config(const Json& m, const AttentionKind& kind
     GroupedAttentionConfig c{m.at("heads").positive(), m.at("kv_heads").positive(), m.at("dim").positive(), m.at("vdim").positive(), 0, 0, 1.0,
                              m.at("scale").number()};
     c.kind = kind;
-    if (m.has("mask")) c.chunk = m.at("mask").at("size").positive();
+    if (m.has("mask")) {
+        const Json& mask = m.at("mask");
+        (kind.mask == AttentionMask::chunks ? c.chunk : c.window) = mask.at("size").positive();
+        if (kind.mask == AttentionMask::window) {
+            if (mask.has("keep_first")) c.keep = mask.at("keep_first").integer();
+            if (mask.has("pool")) c.pool = mask.at("pool").positive();
+            if (c.keep < 0) throw std::invalid_argument("configuration: 'keep_first' must not be negative");
+        }
+    }
     if (m.has("rot")) {
-        c.rot_dims = m.at("rot").at("dims").positive();
-        c.rot_base = m.at("rot").at("base").number();
+        const Json& rot = m.at("rot");
+        c.rot_dims = rot.at("dims").positive();
+        c.rot_base = rot.at("base").number();
+        if (rot.has("scaling")) c.rot_factor = rot.at("scaling").at("factor").number();
+        if (!(c.rot_factor > 0.0)) throw std::invalid_argument("configuration: the scaling 'factor' must be positive");
     }
     if (m.has("softcap")) {
         c.softcap = m.at("softcap").number();
@@ -78,8 +89,8 @@ HybridLayer::HybridLayer(Index width, const Json& spec, const DecoderDesign& des
         n.alpha = &register_parameter(name + ".alpha", ones({}, options));
         return n;
     };
-    const bool sandwich = design.form == LayerForm::sandwich;
-    norm1 = norm("norm1");
+    const bool sandwich = design.form == LayerForm::sandwich, behind = design.form == LayerForm::behind;
+    (behind ? after1 : norm1) = norm("norm1");
     if (sandwich) after1 = norm("norm1b");
     const std::string& type = spec.at("type").text();
     const auto mixer = std::find_if(design.mixers.begin(), design.mixers.end(), [&](const MixerDesign& d) { return type == d.type; });
@@ -112,11 +123,15 @@ HybridLayer::HybridLayer(Index width, const Json& spec, const DecoderDesign& des
         lightning_scale = pair->right_scale;
         break;
     }
+    case MixerKind::delta:
+        delta = add_module<DeltaMixer>("mix", width, DeltaConfig{m.at("heads").positive(), m.at("kv_heads").positive(), m.at("dim").positive(),
+                                                                 m.at("vdim").positive(), m.at("conv").positive()}, options);
+        break;
     }
     if (!spec.has("mlp")) return;
     const Json& mlp = spec.at("mlp");
     const std::string& kind = mlp.at("kind").text();
-    if (design.form != LayerForm::parallel) norm2 = norm("norm2");
+    if (design.form != LayerForm::parallel) (behind ? after2 : norm2) = norm("norm2");
     if (sandwich) after2 = norm("norm2b");
     if (design.mixture && kind == "moe") {
         const Json& router = mlp.at("router");
@@ -148,13 +163,13 @@ void HybridDecoder::set_activation_dtype(DType dtype) {
 namespace {
 std::atomic<std::uint64_t> hybrid_cache_ids{1};
 
-// cos / sin of position * base^(-2i/dims), computed in f64 on the host and rounded once.
-HybridCache::Rotary rotary_table(Index dims, double base, Index positions, Device device) {
+// cos / sin of position * base^(-2i/dims) / factor, computed in f64 on the host and rounded once.
+HybridCache::Rotary rotary_table(Index dims, double base, double factor, Index positions, Device device) {
     if (base <= 0) throw std::invalid_argument("rotary base must be positive");
     const Index half = dims / 2;
     Tensor cosine = empty({positions, half}, {DType::f32, Device::cpu()}), sine = empty({positions, half}, {DType::f32, Device::cpu()});
     for (Index i = 0; i < half; ++i) {
-        const double frequency = std::pow(base, -2.0 * static_cast<double>(i) / static_cast<double>(dims));
+        const double frequency = std::pow(base, -2.0 * static_cast<double>(i) / static_cast<double>(dims)) / factor;
         for (Index p = 0; p < positions; ++p) {
             f32(cosine)[p * half + i] = static_cast<float>(std::cos(static_cast<double>(p) * frequency));
             f32(sine)[p * half + i] = static_cast<float>(std::sin(static_cast<double>(p) * frequency));
@@ -174,9 +189,9 @@ HybridCache::HybridCache(const HybridDecoder& model, Index slots, Index capacity
     lengths_host_.assign(static_cast<std::size_t>(slots), 0);
     lengths_ = zeros({slots}, {DType::f32, where});   // all-zero bits: int32 zeros
     if (model.pairs()) last_ = zeros({slots}, {DType::f32, where});
-    auto rotary = [&](Index dims, double base) {
-        auto& table = tables_[{dims, base}];
-        if (!table.cosine.defined()) table = rotary_table(dims, base, capacity, where);
+    auto rotary = [&](Index dims, double base, double factor = 1.0) {
+        auto& table = tables_[{dims, base, factor}];
+        if (!table.cosine.defined()) table = rotary_table(dims, base, factor, capacity, where);
     };
     try {
         for (const auto& r : model.runs()) {
@@ -192,15 +207,26 @@ HybridCache::HybridCache(const HybridDecoder& model, Index slots, Index capacity
             } else if (layer.attention) {
                 const auto& c = layer.attention->config();
                 run.entries = c.chunk > 0 ? std::min(c.chunk, capacity) : capacity;
+                if (c.window > 0 && c.window < capacity && c.keep + c.window < capacity) {   // (otherwise every position sees all before it)
+                    run.window = c.window;
+                    run.keep = c.keep;
+                    run.pools = c.pool;
+                    run.entries = c.keep + c.window + (c.pool > 0 ? capacity / c.pool : 0);
+                    if (c.pool > 0) run.pool = empty({slots, c.kv_heads, c.dim + c.vdim}, {DType::f32, where});
+                }
                 if (layer.attention->own_keys()) {
                     run.key = empty({slots, c.kv_heads, run.entries, c.dim}, {model.dtype(), where});
                     run.value = empty({slots, c.kv_heads, run.entries, c.vdim}, {model.dtype(), where});
                 }
-                if (c.rot_dims > 0) rotary(c.rot_dims, c.rot_base);
+                if (c.rot_dims > 0) rotary(c.rot_dims, c.rot_base, c.rot_factor);
                 if (layer.lightning) {
                     const auto& r = layer.lightning->config();
                     run.state = empty({slots, r.heads, r.dim, r.vdim}, {DType::f32, where});
                 }
+            } else if (layer.delta) {
+                const auto& c = layer.delta->config();
+                run.conv = empty({slots, c.taps, layer.delta->channels()}, {DType::f32, where});
+                run.state = empty({slots, c.heads, c.dim, c.vdim}, {DType::f32, where});
             } else {
                 const auto& c = layer.state_space->config();
                 run.conv = empty({slots, c.taps, layer.state_space->channels()}, {DType::f32, where});
@@ -241,18 +267,35 @@ HybridDecoder::HybridDecoder(const Json& config, const DecoderDesign& design, Te
         logit_softcap_ = config.at("logit_softcap").number();
         if (!(logit_softcap_ > 0.0)) throw std::invalid_argument("configuration: 'logit_softcap' must be positive");
     }
+    if (design_.residual_factor) residual_factor_ = config.at("residual_mult").number();
     embed_ = &register_parameter("embed", host_zeros({vocab_, width_}, options));
-    if (design_.form == LayerForm::sandwich) {
+    if (design_.pairs) {
         const Json& pair = config.at("embedding").at("bigram");
         pair_hash_ = {pair.at("buckets").positive(), pair.at("mul_prev").integer(), pair.at("mul_cur").integer()};
         pairs_ = &register_parameter("bigram", host_zeros({pair_hash_.buckets + 1, width_}, options));
-        if (config.has("loop")) throw std::invalid_argument("configuration: looped layers are not combined with norms behind the sublayers");
     }
+    if ((design_.form == LayerForm::sandwich || design_.form == LayerForm::behind) && config.has("loop"))
+        throw std::invalid_argument("configuration: looped layers are not combined with norms behind the sublayers");
     const auto& specs = config.at("layers").items();
     const auto count = static_cast<Index>(specs.size());
     if (count == 0) throw std::invalid_argument("decoder requires at least one layer");
-    for (Index i = 0; i < count; ++i)
-        layers_.push_back(add_module<HybridLayer>("l" + std::to_string(i), width_, specs[static_cast<std::size_t>(i)], design_, options));
+    std::vector<Index> module_of(static_cast<std::size_t>(count), -1);   // the module that a layer of the configuration runs
+    for (Index i = 0; i < count; ++i) {
+        const Json& spec = specs[static_cast<std::size_t>(i)];
+        if (spec.has("weights_of")) continue;
+        module_of[static_cast<std::size_t>(i)] = static_cast<Index>(layers_.size());
+        layers_.push_back(add_module<HybridLayer>("l" + std::to_string(i), width_, spec, design_, options));
+    }
+    for (Index i = 0; i < count; ++i) {
+        Index from = i;
+        for (Index hops = 0; specs[static_cast<std::size_t>(from)].has("weights_of"); ++hops) {
+            from = specs[static_cast<std::size_t>(from)].at("weights_of").integer();
+            if (from < 0 || from >= count || hops >= count) throw std::invalid_argument("configuration: 'weights_of' must name a layer with weights");
+        }
+        if (specs[static_cast<std::size_t>(i)].at("type").text() != specs[static_cast<std::size_t>(from)].at("type").text())
+            throw std::invalid_argument("configuration: 'weights_of' must name a layer of the same type");
+        module_of[static_cast<std::size_t>(i)] = module_of[static_cast<std::size_t>(from)];
+    }
     Index start = 0, stop = 0, times = 0;
     if (config.has("loop")) {
         start = config.at("loop").at("start").integer();
@@ -264,15 +307,17 @@ HybridDecoder::HybridDecoder(const Json& config, const DecoderDesign& design, Te
         if (design_.loop == LoopEntry::step) loop_step_ = &register_parameter("loop.step", host_zeros({times, width_}, options));
         else loop_in_ = &register_parameter("loop.in", host_zeros({width_, 2 * width_}, options));
     }
-    auto add_run = [&](Index layer, Index pass, bool begins) {
+    auto add_run = [&](Index number, Index pass, bool begins) {
         const auto own = static_cast<Index>(runs_.size());
+        const Index layer = module_of[static_cast<std::size_t>(number)];
         const auto& mixer = layers_[static_cast<std::size_t>(layer)]->attention;
         if (!mixer || mixer->own_keys()) return runs_.push_back({layer, pass, begins, own});
         // the latest run of the layer it names
+        const auto& c = mixer->config();
+        const Index wanted = c.keys_from < count ? module_of[static_cast<std::size_t>(c.keys_from)] : -1;
         Index from = own - 1;
-        while (from >= 0 && runs_[static_cast<std::size_t>(from)].layer != mixer->config().keys_from) --from;
-        const auto& source = from >= 0 ? layers_[static_cast<std::size_t>(mixer->config().keys_from)]->attention : nullptr;
-        const auto &c = mixer->config();
+        while (from >= 0 && runs_[static_cast<std::size_t>(from)].layer != wanted) --from;
+        const auto& source = from >= 0 ? layers_[static_cast<std::size_t>(wanted)]->attention : nullptr;
         if (!source || !source->own_keys() || source->config().kv_heads != c.kv_heads || source->config().dim != c.dim || source->config().vdim != c.vdim
             || source->config().chunk != c.chunk)
             throw std::invalid_argument("configuration: 'kv_from' must name an earlier attention layer with keys of its own and of the same sizes");
@@ -287,7 +332,7 @@ HybridDecoder::HybridDecoder(const Json& config, const DecoderDesign& design, Te
         final_norm_.bias = &register_parameter("final.norm.b", host_zeros({width_}, options));
         final_norm_.alpha = &register_parameter("final.norm.alpha", ones({}, options));
     }
-    head_ = &register_parameter("head", host_zeros({vocab_, width_}, options));
+    head_ = design_.tied ? embed_ : &register_parameter("head", host_zeros({vocab_, width_}, options));
 }
 
 HybridDecoder::~HybridDecoder() = default;
@@ -340,9 +385,9 @@ void HybridPlan::refresh() {
     layers_.clear();
     for (const auto& module : owner_.layers()) {
         Layer l{};
-        l.norm1 = pack_norm(module->norm1);
-        if (module->attention) {
-            if (owner_.design().form == LayerForm::sandwich) pack_sandwich(*module, l);
+        if (module->norm1.weight) l.norm1 = pack_norm(module->norm1);
+        if (module->after1.weight || module->attention) {
+            if (module->after1.weight) pack_sandwich(*module, l);
             else pack_parallel(*module, l);
             layers_.push_back(std::move(l));
             continue;
@@ -440,6 +485,11 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
             channels = std::max(channels, module.lightning->channels());
             y = std::max(y, module.lightning->inner());
         }
+        if (module.delta) {
+            channels = std::max(channels, module.delta->channels());
+            y = std::max(y, module.delta->inner());
+            continue;
+        }
         if (module.attention) continue;   // reserve_attention
         if (module.state_space) {
             channels = std::max(channels, module.state_space->channels());
@@ -475,7 +525,7 @@ void HybridPlan::reserve(Index rows, Index max_length, const HybridCache& cache,
     }
     grow(scratch_, {static_cast<Index>(scratch / 4 + 1)}, DType::f32);
     if (owner_.loop_in()) { grow(joined_first_, {rows, D}, DType::f32); grow(entered_, {rows, D}, DType::f32); }
-    if (owner_.design().form == LayerForm::sandwich) {
+    if (norms_behind()) {
         grow(branch_, {rows, D}, DType::f32);
         Index outputs = 0;
         for (const auto& layer : layers_)
@@ -528,7 +578,7 @@ void HybridPlan::planes_of(const float* x, Index rows, const Norm& norm, Planes&
 
 void HybridPlan::run(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail) {
     ids_ = ids;
-    if (owner_.design().form == LayerForm::sandwich) return run_sandwich(ids, pass, cache, max_length, stream, trail);
+    if (norms_behind()) return run_sandwich(ids, pass, cache, max_length, stream, trail);
     const Index rows = pass.rows, D = owner_.width();
     const bool planes = shadows_for(rows);
     float *first = f32(first_), *h = f32(h_);

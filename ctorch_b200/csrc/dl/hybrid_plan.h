@@ -30,6 +30,8 @@ Tensor to_f32(const Tensor& t);
 //                        -> (recurrence -> norm + gate) -> [o | right o] projection -> norm, residual, next norm
 //                        -> gate/up + clamped units -> down-projection -> norm, residual, next norm
 //                           or router -> experts, norm, residual, next norm
+//     layer with norms behind it alone: as a sandwich layer, with the stream itself in the place of the norms before the sublayers; a delta
+//                        rule in the place of the attention: [g | v | k | q | a | b] projection -> convolution + recurrence -> norm + gate
 // bf16 models run the projections on the shadow protocol (activations as bf16 hi + lo planes).  The projection that finishes the
 // residual stream also writes the next norm: a Dynamic Tanh norm as its result, an RMS norm as weighted rows and partial sums of
 // squares, from which the consumer takes the row's factor.  f32 models and sizes the shadow kernels do not take run the same kernels
@@ -55,6 +57,7 @@ public:
     void set_user(const void* user) { user_ = user; }
     const void* user() const { return user_; }
     int device() const { return owner_.embed().device().index; }
+    bool norms_behind() const { return owner_.design().form == LayerForm::sandwich || owner_.design().form == LayerForm::behind; }
 
     // Pass descriptions: host arrays -> one device block.
     struct PassMaps {
@@ -79,7 +82,7 @@ private:
         Tensor q_bias, k_bias, sink;                // f32
         // norms behind the sublayers, router and recurrence beside the attention (sandwich layers)
         Norm after1, after2;
-        Tensor router, correction, decay, right_norm;
+        Tensor router, router_bias, correction, decay, right_norm, talk;
         Index lightning_column = 0;                 // where its [g | v | k | q] start in a projected row
         b200_clamped_unit unit{};
         // parallel layers
@@ -95,6 +98,9 @@ private:
     void pack_experts(const MixtureOfExperts& mixture, Layer& layer) const;
     void pack_parallel(const HybridLayer& module, Layer& layer) const;
     void pack_sandwich(const HybridLayer& module, Layer& layer) const;
+    void pack_delta(const DeltaMixer& mixer, Layer& layer) const;
+    // The recurrence of a delta layer from its projected rows to the input of its out-projection.
+    void run_delta(std::size_t run, const b200_rows& pass, HybridCache& cache, void* stream);
     void reserve_attention(Index rows, Index max_length, const HybridCache& cache, const b200_rows& pass);
     void run_sandwich(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail);
     // Everything of a parallel layer up to its out-projection; returns the residual that the out-projection adds to.

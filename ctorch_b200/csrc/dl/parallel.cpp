@@ -21,7 +21,8 @@ GroupedAttentionMixer::GroupedAttentionMixer(Index width, const GroupedAttention
     if (c.heads % c.kv_heads) throw std::invalid_argument("grouped attention: heads must be a multiple of kv_heads");
     if (c.rot_dims % 2 || c.rot_dims > c.dim) throw std::invalid_argument("grouped attention: rotated dimensions must be even and at most dim");
     if (kind.keys_as_values && c.vdim != c.dim) throw std::invalid_argument("grouped attention: values that are the keys must have their size");
-    if (c.chunk > 0 && !own_keys()) throw std::invalid_argument("grouped attention: chunks need keys of the layer itself");
+    if ((c.chunk > 0 || c.window > 0) && !own_keys()) throw std::invalid_argument("grouped attention: chunks and windows need keys of the layer itself");
+    if (c.keep > 0 && c.pool > 0) throw std::invalid_argument("grouped attention: kept first positions are not combined with pooled blocks");
     q = &register_parameter("q", host_zeros({c.heads * c.dim, width}, options));
     if (kind.bias) q_bias = &register_parameter("q.b", host_zeros({c.heads * c.dim}, options));
     if (own_keys()) {
@@ -29,12 +30,14 @@ GroupedAttentionMixer::GroupedAttentionMixer(Index width, const GroupedAttention
         if (kind.bias) k_bias = &register_parameter("k.b", host_zeros({c.kv_heads * c.dim}, options));
         if (!kind.keys_as_values) v = &register_parameter("v", host_zeros({c.kv_heads * c.vdim, width}, options));
     }
-    if (kind.norm == B200_HEAD_NORM_PROJECTION) {
-        q_norm = &register_parameter("q.norm", ones({c.heads * c.dim}, options));
-        if (own_keys()) k_norm = &register_parameter("k.norm", ones({c.kv_heads * c.dim}, options));
+    if (kind.norm == B200_HEAD_NORM_PROJECTION || (kind.norm == B200_HEAD_NORM_HEAD && kind.head_weights)) {
+        const bool per_head = kind.norm == B200_HEAD_NORM_HEAD;
+        q_norm = &register_parameter("q.norm", ones({per_head ? c.dim : c.heads * c.dim}, options));
+        if (own_keys()) k_norm = &register_parameter("k.norm", ones({per_head ? c.dim : c.kv_heads * c.dim}, options));
     }
     if (kind.sink == Sink::learned) sink = &register_parameter("sink", host_zeros({c.heads}, options));
-    if (kind.gate) gate = &register_parameter("g", host_zeros({c.heads, width}, options));
+    if (kind.gate != OutputGate::none) gate = &register_parameter("g", host_zeros({kind.gate == OutputGate::head ? c.heads : c.heads * c.vdim, width}, options));
+    if (kind.talk) talk = &register_parameter("talk", host_zeros({c.heads, c.heads}, options));
     out = &register_parameter("o", host_zeros({width, c.heads * c.vdim}, options));
 }
 Index GroupedAttentionMixer::columns() const {
@@ -55,6 +58,7 @@ MixtureOfExperts::MixtureOfExperts(Index width, const MixtureConfig& c, TensorOp
         down.push_back(&register_parameter(name + ".down", host_zeros({width, c.ff}, options)));
     }
     router = &register_parameter("router", host_zeros({c.outputs(), width}, options));
+    if (c.kind.bias) bias = &register_parameter("router.b", host_zeros({c.outputs()}, options));
     if (c.kind.correction) correction = &register_parameter("correction", host_zeros({c.outputs()}, options));
     if (c.shared_ff > 0) {
         if (c.kind.gated) throw std::invalid_argument("mixture of experts: a shared expert is not combined with gated experts");
@@ -71,6 +75,7 @@ void HybridPlan::pack_attention(const GroupedAttentionMixer& m, Layer& l) const 
     if (m.k_bias) l.k_bias = to_f32(*m.k_bias);
     if (m.sink) l.sink = to_f32(*m.sink);
     else if (m.config().kind.sink == Sink::zero) l.sink = zeros({m.config().heads}, {DType::f32, m.q->device()});
+    if (m.talk) l.talk = to_f32(*m.talk);
 }
 
 void HybridPlan::pack_experts(const MixtureOfExperts& e, Layer& l) const {
@@ -80,6 +85,7 @@ void HybridPlan::pack_experts(const MixtureOfExperts& e, Layer& l) const {
     l.experts_up = concat_rows(ups);
     l.experts_down = concat_rows(downs);
     if (e.correction) l.correction = to_f32(*e.correction);
+    if (e.bias) l.router_bias = to_f32(*e.bias);
 }
 
 void HybridPlan::pack_parallel(const HybridLayer& module, Layer& l) const {
@@ -142,14 +148,17 @@ b200_chunk_args HybridPlan::chunk_args(const Layer& layer, const HybridLayer& mo
     a.chunk = static_cast<int32_t>(c.chunk > cache.capacity() ? 0 : c.chunk); a.entries = static_cast<int32_t>(r.entries);
     a.scale = static_cast<float>(c.scale); a.eps = owner_.eps();
     if (c.rot_dims > 0) {
-        const auto& table = cache.rotary(c.rot_dims, c.rot_base);
+        const auto& table = cache.rotary(c.rot_dims, c.rot_base, c.rot_factor);
         a.cosine = table.cosine.data<float>(); a.sine = table.sine.data<float>(); a.positions = static_cast<int32_t>(table.cosine.size(0));
     }
     a.q_norm = vector(layer.q_norm); a.k_norm = vector(layer.kv_norm); a.q_bias = vector(layer.q_bias); a.k_bias = vector(layer.k_bias);
     a.sink = vector(layer.sink);
     a.norm = c.kind.norm; a.rotate_pairs = c.kind.rotate_pairs; a.keys_as_values = c.kind.keys_as_values; a.keys_elsewhere = !module.attention->own_keys();
-    a.no_gate = !c.kind.gate; a.softcap = static_cast<float>(c.softcap);
+    a.no_gate = c.kind.gate != OutputGate::head; a.gate_values = c.kind.gate == OutputGate::value; a.softcap = static_cast<float>(c.softcap);
     a.scaled = 1; a.out_scale = static_cast<float>(module.attention_scale);
+    a.window = static_cast<int32_t>(r.window); a.keep = static_cast<int32_t>(r.keep); a.pool = static_cast<int32_t>(r.pools);
+    a.pool_state = r.pool.defined() ? f32(r.pool) : nullptr;
+    a.norm_values = c.kind.norm_values; a.talk = vector(layer.talk);
     a.dtype = code_of(owner_.dtype());
     a.key_cache = r.key.mutable_data(); a.value_cache = r.value.mutable_data();
     a.projected = projected_.data<float>(); a.stride = stride;
@@ -184,7 +193,7 @@ void HybridPlan::reserve_attention(Index rows, Index max_length, const HybridCac
         if (module->attention) {
             const auto& c = module->attention->config();
             query = std::max(query, c.heads * c.dim);
-            if (c.chunk > 0) {   // without chunks the rows go into the slots at once
+            if (c.chunk > 0 || c.window > 0) {   // without either the rows go into the slots at once
                 key = std::max(key, c.kv_heads * c.dim);
                 value = std::max(value, c.kv_heads * c.vdim);
             }

@@ -15,11 +15,18 @@ using Factory = std::shared_ptr<nn::UnaryModule> (*)(const Json&, TensorOptions)
 using nn::MixerKind;
 
 constexpr nn::MixerDesign kHybridMixers[] = {{"mamba2", MixerKind::state_space}, {"latent_attention", MixerKind::latent}};
-constexpr nn::MixerDesign kParallelMixers[] = {{"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_PROJECTION, .gate = true}}};
+using nn::OutputGate;
+
+constexpr nn::MixerDesign kParallelMixers[] = {{"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_PROJECTION, .gate = OutputGate::head}}};
 constexpr nn::MixerDesign kSandwichMixers[] = {
-    {"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_NONE, .rotate_pairs = true, .bias = true, .keys_as_values = true, .gate = true, .sink = nn::Sink::zero}},
+    {"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_NONE, .rotate_pairs = true, .bias = true, .keys_as_values = true, .gate = OutputGate::head, .sink = nn::Sink::zero}},
     {"attention_2", MixerKind::attention, {.norm = B200_HEAD_NORM_HEAD, .rotate_pairs = true, .sink = nn::Sink::learned}},
-    {"parallel", MixerKind::side_by_side, {.norm = B200_HEAD_NORM_PROJECTION, .gate = true, .sink = nn::Sink::learned}},
+    {"parallel", MixerKind::side_by_side, {.norm = B200_HEAD_NORM_PROJECTION, .gate = OutputGate::head, .sink = nn::Sink::learned}},
+};
+constexpr nn::MixerDesign kPostNormMixers[] = {
+    {"attention", MixerKind::attention, {.norm = B200_HEAD_NORM_PROJECTION, .gate = OutputGate::value, .mask = nn::AttentionMask::window, .norm_values = true}},
+    {"attention_2", MixerKind::attention, {.norm = B200_HEAD_NORM_HEAD, .mask = nn::AttentionMask::window, .head_weights = true, .talk = true}},
+    {"delta", MixerKind::delta},
 };
 
 std::shared_ptr<nn::UnaryModule> hybrid(const Json& config, TensorOptions options) {
@@ -33,7 +40,12 @@ std::shared_ptr<nn::UnaryModule> parallel(const Json& config, TensorOptions opti
 std::shared_ptr<nn::UnaryModule> sandwich(const Json& config, TensorOptions options) {
     return std::make_shared<nn::HybridDecoder>(
         config, nn::DecoderDesign{nn::NormKind::rms_from_one, nn::LoopEntry::joined, nn::LayerForm::sandwich, false, kSandwichMixers,
-                                  nn::MixtureKind{.softmax = true, .correction = true, .gated = true, .weigh_results = true}, 1.702}, options);
+                                  nn::MixtureKind{.softmax = true, .correction = true, .gated = true, .weigh_results = true}, 1.702, true}, options);
+}
+std::shared_ptr<nn::UnaryModule> post_norm(const Json& config, TensorOptions options) {
+    return std::make_shared<nn::HybridDecoder>(
+        config, nn::DecoderDesign{nn::NormKind::rms, nn::LoopEntry::joined, nn::LayerForm::behind, false, kPostNormMixers,
+                                  nn::MixtureKind{.gated = true, .weigh_results = true, .bias = true, .chosen_softmax = true}, 0.0, false, true, true}, options);
 }
 
 // Grouped-query decoder with its embedding and output layers, under the names of the reference's example model.
@@ -48,6 +60,7 @@ struct Entry { const char* name; Factory make; };
 constexpr Entry kRegistry[] = {
     {"Lozepel", sandwich},
     {"Ripitar", hybrid},
+    {"Rizovik", post_norm},
     {"Sinezen", parallel},
     {"TransformerDecoder", transformer},
 };

@@ -1,5 +1,6 @@
-// Sandwich layers of the configured decoders: a norm before and after every sublayer, attention alone or side by side with lightning
-// attention, clamped gated units or a mixture of gated experts, and the embedding of token pairs (see hybrid.h).
+// Layers of the configured decoders with a norm behind every sublayer, and one before it or none: attention alone or side by side with
+// lightning attention or the delta rule (delta.cpp), clamped gated units or a mixture of gated experts, and the embedding of token pairs
+// (see hybrid.h).
 #include "dl/hybrid_plan.h"
 
 #include <algorithm>
@@ -32,9 +33,28 @@ SideBySideMixer::SideBySideMixer(Index width, const GroupedAttentionConfig& l, c
 
 // ---- plan ---------------------------------------------------------------------------------------------------
 void HybridPlan::pack_sandwich(const HybridLayer& module, Layer& l) const {
-    const GroupedAttentionMixer& m = *module.attention;
     const Index D = owner_.width();
-    const TensorOptions options{owner_.dtype(), m.q->device()};
+    const TensorOptions options{owner_.dtype(), owner_.embed().device()};
+    // (what a sublayer adds is multiplied by the factor of the residual: in the weight of the norm behind it)
+    l.after1 = pack_norm(module.after1, owner_.residual_factor());
+    if (module.after2.weight) l.after2 = pack_norm(module.after2, owner_.residual_factor());
+    if (module.norm2.weight) l.norm2 = pack_norm(module.norm2);
+    if (module.has_mlp()) {
+        l.gate_up = interleave_rows(*module.gate, *module.up);
+        l.down = module.down->raw_data();
+        l.unit = {static_cast<float>(owner_.design().unit_slope), static_cast<float>(module.unit_limit)};
+    } else if (module.mixture) {
+        const Tensor& router = *module.mixture->router;
+        const Index outputs = router.size(0), padded = round_up_8(outputs);
+        l.router = router;
+        if (padded > outputs) {
+            const Tensor parts[2] = {router, zeros({padded - outputs, D}, options)};
+            l.router = concat_rows(parts);
+        }
+        pack_experts(*module.mixture, l);
+    }
+    if (module.delta) return pack_delta(*module.delta, l);
+    const GroupedAttentionMixer& m = *module.attention;
     std::vector<Tensor> rows, columns{*m.out};
     for (const Tensor* t : {m.q, m.k, m.v, m.gate})
         if (t) rows.push_back(*t);
@@ -65,24 +85,6 @@ void HybridPlan::pack_sandwich(const HybridLayer& module, Layer& l) const {
     l.attended = m.out->size(1);
     l.inner = l.joint.size(1);
     pack_attention(m, l);
-    l.after1 = pack_norm(module.after1);
-    if (!module.after2.weight) return;
-    l.norm2 = pack_norm(module.norm2);
-    l.after2 = pack_norm(module.after2);
-    if (module.has_mlp()) {
-        l.gate_up = interleave_rows(*module.gate, *module.up);
-        l.down = module.down->raw_data();
-        l.unit = {static_cast<float>(owner_.design().unit_slope), static_cast<float>(module.unit_limit)};
-    } else {
-        const Tensor& router = *module.mixture->router;
-        const Index outputs = router.size(0), padded = round_up_8(outputs);
-        l.router = router;
-        if (padded > outputs) {
-            const Tensor parts[2] = {router, zeros({padded - outputs, D}, options)};
-            l.router = concat_rows(parts);
-        }
-        pack_experts(*module.mixture, l);
-    }
 }
 
 void HybridPlan::run_sandwich(const Index* ids, const b200_rows& pass, HybridCache& cache, Index max_length, void* stream, std::vector<float>* trail) {
@@ -94,12 +96,22 @@ void HybridPlan::run_sandwich(const Index* ids, const b200_rows& pass, HybridCac
     auto* inner_hi = planes ? static_cast<std::uint16_t*>(i_.hi.mutable_data()) : nullptr;
     auto* inner_lo = planes ? static_cast<std::uint16_t*>(i_.lo.mutable_data()) : nullptr;
     n_.parts = i_.parts = 0;   // the norms are finished where they are written
-    // the stream's next norm, as planes or f32 rows
+    // the stream's next norm, or (in front of a sublayer without a norm before it) the stream, as planes or f32 rows
     auto normed_to = [&](auto& args) {
         if (planes) { args.normed_hi = n_.hi.mutable_data(); args.normed_lo = n_.lo.mutable_data(); }
         else args.normed = f32(plain_);
     };
-    {
+    if (!owner_.pairs()) {
+        if (planes) {
+            runtime::check(b200_embedding_shadow(owner_.embed().raw_data(), code_of(owner_.dtype()), ids, rows, owner_.vocabulary(), D,
+                                                 nullptr, B200_F32, h, n_.hi.mutable_data(), n_.lo.mutable_data(), f32(squares_), stream), "embedding");
+        } else {
+            for (float* to : {h, f32(plain_)}) {
+                runtime::check(b200_embedding_scaled(owner_.embed().raw_data(), code_of(owner_.dtype()), ids, rows, owner_.vocabulary(), D, 1.0f, to, stream), "embedding");
+            }
+        }
+        probe(2);
+    } else {
         const auto& hash = owner_.pair_hash();
         b200_pair_embedding e{};
         e.table = owner_.embed().raw_data(); e.pairs = owner_.pairs()->raw_data(); e.dtype = code_of(owner_.dtype());
@@ -115,7 +127,9 @@ void HybridPlan::run_sandwich(const Index* ids, const b200_rows& pass, HybridCac
     // the end of a sublayer whose result is in `branch`
     auto sandwich_args = [&](const Norm& after, const Norm& next) {
         b200_sandwich a{};
-        a.after = after.weight.data<float>(); a.next = next.weight.data<float>(); a.eps = owner_.eps();
+        a.after = after.weight.data<float>(); a.eps = owner_.eps();
+        if (next.weight.defined()) a.next = next.weight.data<float>();
+        else a.plain = 1;
         a.residual = h; a.x = h;
         normed_to(a);
         return a;
@@ -139,12 +153,16 @@ void HybridPlan::run_sandwich(const Index* ids, const b200_rows& pass, HybridCac
         const Norm& next = i + 1 == runs.size() ? final_norm_ : layers_[static_cast<std::size_t>(runs[i + 1].layer)].norm1;
         // ---- mixer ----
         project(layer.in, layer.wide_out, projected, "mixer projection");
-        const b200_chunk_args a = chunk_args(layer, module, cache, i, layer.wide_out);
-        runtime::check(b200_chunk_prepare(&a, &pass, nullptr, nullptr, stream), "attention norms");
-        probe(2);
-        runtime::check(b200_chunk_attention(&a, &pass, static_cast<int32_t>(max_length), scratch_.mutable_data(), scratch_.nbytes(), inner_plain, inner_hi, inner_lo,
-                                            layer.inner, stream), "grouped attention");
-        probe(1);
+        if (module.delta) {
+            run_delta(i, pass, cache, stream);
+        } else {
+            const b200_chunk_args a = chunk_args(layer, module, cache, i, layer.wide_out);
+            runtime::check(b200_chunk_prepare(&a, &pass, nullptr, nullptr, stream), "attention norms");
+            probe(2);
+            runtime::check(b200_chunk_attention(&a, &pass, static_cast<int32_t>(max_length), scratch_.mutable_data(), scratch_.nbytes(), inner_plain, inner_hi, inner_lo,
+                                                layer.inner, stream), "grouped attention");
+            probe(1);
+        }
         if (module.lightning) {
             const auto& c = module.lightning->config();
             b200_ssm_args r{};
@@ -181,6 +199,8 @@ void HybridPlan::run_sandwich(const Index* ids, const b200_rows& pass, HybridCac
             b200_route route{};
             route.experts = static_cast<int32_t>(module.mixture->config().outputs()); route.top = e.top; route.identity = e.identity;
             route.softmax = module.mixture->config().kind.softmax;
+            route.chosen_softmax = module.mixture->config().kind.chosen_softmax;
+            route.bias = layer.router_bias.defined() ? layer.router_bias.data<float>() : nullptr;
             route.correction = layer.correction.defined() ? layer.correction.data<float>() : nullptr;
             route.chosen = static_cast<std::int32_t*>(chosen_.mutable_data()); route.weight = f32(score_);
             if (sorted) {

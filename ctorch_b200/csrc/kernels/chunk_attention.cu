@@ -40,19 +40,44 @@ struct ChunkParams {
     int norm;
     bool rotate_pairs, keys_as_values, keys_elsewhere, gated;
     float softcap, out_scale;
+    int window, keep, pool;
+    float* pool_state;
+    bool norm_values, gate_values;
+    const float* talk;
     __host__ __device__ __forceinline__ int key_columns() const { return keys_elsewhere ? 0 : kv_heads * dim; }
     __host__ __device__ __forceinline__ int value_columns() const { return keys_elsewhere || keys_as_values ? 0 : kv_heads * vdim; }
     // Keys of the pass itself are in the slots before the attention starts.
-    __host__ __device__ __forceinline__ bool appends_first(bool step) const { return step || chunk == 0; }
+    __host__ __device__ __forceinline__ bool appends_first(bool step) const { return step || (chunk == 0 && window == 0); }
     __device__ __forceinline__ int chunk_start(int position) const { return chunk > 0 ? position - position % chunk : 0; }
-    // where (slot, kv head)'s entry of a position begins, in units of one entry
-    __device__ __forceinline__ int64_t entry(int slot, int head, int position) const {
-        return (static_cast<int64_t>(slot) * kv_heads + head) * entries + (position - chunk_start(position));
+    // The entry that holds a position: of its chunk, of the first positions that stay, or of the window's ring.
+    __device__ __forceinline__ int place(int position) const {
+        if (window > 0) return position < keep ? position : keep + (position - keep) % window;
+        return position - chunk_start(position);
     }
-    // Whether storing the chunk of position `last` overwrites keys that positions from `length` on still see.
-    __device__ __forceinline__ bool overwrites(int length, int last) const { return chunk > 0 && length % chunk != 0 && chunk_start(length) != chunk_start(last); }
-    __device__ __forceinline__ bool fits(int position) const { return position - chunk_start(position) < entries; }
+    // where (slot, kv head)'s entry number `place` begins, in units of one entry
+    __device__ __forceinline__ int64_t entry_at(int slot, int head, int at) const { return (static_cast<int64_t>(slot) * kv_heads + head) * entries + at; }
+    __device__ __forceinline__ int64_t entry(int slot, int head, int position) const { return entry_at(slot, head, place(position)); }
+    // The first position of the run of positions up to itself that `position` sees; and, before it, the kept positions or pooled blocks.
+    __device__ __forceinline__ int first_seen(int position) const { return window > 0 ? max(0, position - window + 1) : chunk_start(position); }
+    __device__ __forceinline__ int blocks_seen(int position) const { return position < window ? 0 : (position - window + 1) / pool; }
+    __device__ __forceinline__ int before_run(int position) const { return pool > 0 ? blocks_seen(position) : min(keep, first_seen(position)); }
+    // Entries that a position sees once it is in its slot: they are the first ones of the slot, in whatever order.
+    __device__ __forceinline__ int entries_seen(int position) const {
+        if (window > 0) return min(position + 1, keep + window) + (pool > 0 ? blocks_seen(position) : 0);
+        return position - chunk_start(position) + 1;
+    }
+    // Whether storing the rows of a pass from position `length` to `last` overwrites keys that the pass itself still reads.
+    __device__ __forceinline__ bool overwrites(int length, int last) const {
+        return window > 0 ? length > 0 : chunk > 0 && length % chunk != 0 && chunk_start(length) != chunk_start(last);
+    }
+    // Whether a position's key is still of use behind position `last`.
+    __device__ __forceinline__ bool outlasts(int position, int last) const {
+        return window > 0 ? position < keep || position > last - window : chunk_start(position) == chunk_start(last);
+    }
+    __device__ __forceinline__ bool fits(int position) const { return place(position) < entries; }
 };
+// Head dimensions from which lanes are handed out to a head: a power of two of neighbouring lanes, as many as its values occupy.
+__device__ __forceinline__ int lanes_per_head(int size, int per_lane) { return size > 16 * per_lane ? 32 : size > 8 * per_lane ? 16 : 8; }
 
 bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
     if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)
@@ -60,6 +85,9 @@ bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
         || (a->norm == B200_HEAD_NORM_PROJECTION && (!a->q_norm || (!a->k_norm && !a->keys_elsewhere)))
         || a->norm < B200_HEAD_NORM_PROJECTION || a->norm > B200_HEAD_NORM_HEAD || (a->keys_elsewhere && a->chunk > 0)
         || (a->keys_as_values && (a->vdim != a->dim || a->norm != B200_HEAD_NORM_NONE)) || !(a->softcap >= 0.0f)
+        || a->window < 0 || a->keep < 0 || a->pool < 0 || (a->window > 0 && (a->chunk > 0 || a->keys_elsewhere || a->entries < a->keep + a->window))
+        || ((a->keep > 0 || a->pool > 0) && a->window == 0) || (a->pool > 0 && (a->keep > 0 || !a->pool_state)) || (a->talk && a->sink)
+        || (a->norm == B200_HEAD_NORM_HEAD && !a->q_norm != !a->k_norm && !a->keys_elsewhere) || (a->gate_values && !a->no_gate)
         || (a->dtype != B200_F32 && a->dtype != B200_BF16) || !a->key_cache || !a->value_cache || !a->projected || !a->query || a->stride <= 0) {
         set_error("grouped attention: bad pointer or size");
         return false;
@@ -67,8 +95,8 @@ bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
     p = ChunkParams{a->heads, a->kv_heads, a->heads / a->kv_heads, a->dim, a->vdim, a->rot_dims, a->slots, a->chunk, a->entries, a->scale, static_cast<float>(a->eps),
                     a->cosine, a->sine, a->positions, a->q_norm, a->k_norm, a->key_cache, a->value_cache, a->query, a->key, a->value, a->projected, a->stride,
                     a->q_bias, a->k_bias, a->sink, a->norm, a->rotate_pairs != 0, a->keys_as_values != 0, a->keys_elsewhere != 0, a->no_gate == 0, a->softcap,
-                    a->scaled ? a->out_scale : 1.0f};
-    if (p.heads * p.dim + p.key_columns() + p.value_columns() + (p.gated ? p.heads : 0) > p.stride) {
+                    a->scaled ? a->out_scale : 1.0f, a->window, a->keep, a->pool, a->pool_state, a->norm_values != 0, a->gate_values != 0, a->talk};
+    if (p.heads * p.dim + p.key_columns() + p.value_columns() + (p.gate_values ? p.heads * p.vdim : p.gated ? p.heads : 0) > p.stride) {
         set_error("grouped attention: the projected rows are shorter than the heads");
         return false;
     }
@@ -97,6 +125,11 @@ template <int V> __device__ __forceinline__ void store_span(__nv_bfloat16* p, co
     if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(s.v[0], s.v[1]), pack_bf16(s.v[2], s.v[3]));
     else *p = __float2bfloat16_rn(s.v[0]);
 }
+// The value that a cache of T holds for v.
+template <class T> __device__ __forceinline__ float rounded_to(float v) {
+    if constexpr (sizeof(T) == 2) return __bfloat162float(__float2bfloat16_rn(v));
+    else return v;
+}
 // Entries [c, c + V) of a projected row's part, with its bias.
 template <int V> __device__ __forceinline__ Span<V> biased_span(const float* x, const float* bias, int c) {
     Span<V> s = load_span<V>(x + c);
@@ -117,15 +150,15 @@ template <int V> __device__ __forceinline__ float squares_of(const float* x, con
     }
     return total;
 }
-// V entries from entry c of a part on, which is entry d of its head: with bias, normed, weighted (weight may be NULL), and turned by the
-// row's angles - entry i with entry i + rot_dims / 2, or entry 2i with entry 2i + 1.
-template <int V>
+// V entries from entry c of a part on, which is entry d of its head: with bias, normed, weighted (weight may be NULL; PER_HEAD: the same for
+// every head), and turned by the row's angles - entry i with entry i + rot_dims / 2, or entry 2i with entry 2i + 1.
+template <int V, bool PER_HEAD = false>
 __device__ __forceinline__ Span<V> turned_span(const ChunkParams& p, const float* part, const float* bias, const float* weight, int c, int d, float inverse,
                                                const float* cosine, const float* sine) {
     auto normed = [&](int at) {
         Span<V> s = biased_span<V>(part, bias, at);
         if (weight) {
-            const Span<V> w = load_span<V>(weight + at);
+            const Span<V> w = load_span<V>(weight + (PER_HEAD ? at - c + d : at));
 #pragma unroll
             for (int i = 0; i < V; ++i) s.v[i] = s.v[i] * inverse * w.v[i];
         } else {
@@ -240,20 +273,40 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
     const int position = length + row - first, last = length + end - first - 1;
     // The slot takes the row at once where it ends up there and nothing that this pass still reads is overwritten.
     const bool first_appended = p.appends_first(step);
-    const bool stored = first_appended || (p.chunk_start(position) == p.chunk_start(last) && !p.overwrites(length, last));
+    const bool stored = first_appended || (p.outlasts(position, last) && !p.overwrites(length, last));
     const bool to_slot = stored && p.fits(position);   // (the host refuses passes that do not fit)
     const int half = p.rot_dims >> 1;
     const bool turns = half > 0 && position < p.positions;
     const float* cosine = turns ? p.cosine + static_cast<int64_t>(position) * half : nullptr;
     const float* sine = turns ? p.sine + static_cast<int64_t>(position) * half : nullptr;
     auto store_query = [&](int c, const Span<V>& v) { store_span<V>(static_cast<T*>(p.query) + static_cast<int64_t>(row) * q_count + c, v); };
+    // A step's share of the block that is being pooled: the sum of what the cache holds, and its mean once the block is complete.
+    const int place = p.place(position);
+    const bool pools = step && p.pool > 0, pool_begins = pools && position % p.pool == 0, pool_ends = pools && (position + 1) % p.pool == 0;
+    auto pool_up = [&](T* cache, int size, int head, int offset, int d, const Span<V>& v) {
+        float* sum = p.pool_state + (static_cast<int64_t>(slot) * p.kv_heads + head) * (p.dim + p.vdim) + offset + d;
+        Span<V> total = pool_begins ? Span<V>{} : load_span<V>(sum);
+#pragma unroll
+        for (int i = 0; i < V; ++i) total.v[i] += rounded_to<T>(v.v[i]);
+        if (!pool_ends) return store_span<V>(sum, total);
+#pragma unroll
+        for (int i = 0; i < V; ++i) total.v[i] /= static_cast<float>(p.pool);
+        const int at = p.window + position / p.pool;
+        if (at < p.entries) store_span<V>(cache + p.entry_at(slot, head, at) * size + d, total);
+    };
     auto store_key = [&](int head, int d, const Span<V>& v) {
-        if (to_slot) store_span<V>(static_cast<T*>(p.key_cache) + p.entry(slot, head, position) * p.dim + d, v);
+        if (to_slot) store_span<V>(static_cast<T*>(p.key_cache) + p.entry_at(slot, head, place) * p.dim + d, v);
         if (!first_appended) store_span<V>(static_cast<T*>(p.key) + static_cast<int64_t>(row) * k_count + head * p.dim + d, v);
+        if (pools) pool_up(static_cast<T*>(p.key_cache), p.dim, head, 0, d, v);
+    };
+    auto store_value = [&](int head, int d, const Span<V>& v) {
+        if (to_slot) store_span<V>(static_cast<T*>(p.value_cache) + p.entry_at(slot, head, place) * p.vdim + d, v);
+        if (!first_appended) store_span<V>(static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + head * p.vdim + d, v);
+        if (pools) pool_up(static_cast<T*>(p.value_cache), p.vdim, head, p.dim, d, v);
     };
     if constexpr (NORM == B200_HEAD_NORM_HEAD) {
-        // a power of two of neighbouring lanes per head, as many as its entries occupy; the key heads follow the query heads
-        const int lanes = p.dim > 16 * V ? 32 : p.dim > 8 * V ? 16 : 8, lane = threadIdx.x & (lanes - 1), at_once = kPrepareThreads / lanes;
+        // the key heads follow the query heads
+        const int lanes = lanes_per_head(p.dim, V), lane = threadIdx.x & (lanes - 1), at_once = kPrepareThreads / lanes;
         const int heads = p.heads + (p.keys_elsewhere ? 0 : p.kv_heads);
         for (int h0 = 0; h0 < heads; h0 += at_once) {
             const int h = h0 + static_cast<int>(threadIdx.x) / lanes;
@@ -264,7 +317,7 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
             for (int o = lanes >> 1; o > 0; o >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, o);
             const float inverse = 1.0f / sqrtf(squares / static_cast<float>(p.dim) + p.eps);
             for (int d = lane * V; live && d < p.dim; d += lanes * V) {
-                const Span<V> v = turned_span<V>(p, part, bias, nullptr, begin + d, d, inverse, cosine, sine);
+                const Span<V> v = turned_span<V, true>(p, part, bias, is_query ? p.q_norm : p.k_norm, begin + d, d, inverse, cosine, sine);
                 if (is_query) store_query(begin + d, v);
                 else store_key(head, d, v);
             }
@@ -278,15 +331,65 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
             store_key(head, d, turned_span<V>(p, k_source, p.k_bias, kWeighted ? p.k_norm : nullptr, c, d, k_inverse, cosine, sine));
         }
     }
+    if (p.norm_values && v_count > 0) {
+        const int lanes = lanes_per_head(p.vdim, V), lane = threadIdx.x & (lanes - 1), at_once = kPrepareThreads / lanes;
+        for (int h0 = 0; h0 < p.kv_heads; h0 += at_once) {
+            const int head = h0 + static_cast<int>(threadIdx.x) / lanes, begin = head * p.vdim;
+            const bool live = head < p.kv_heads;
+            float squares = live ? squares_of<V>(v_source, v_bias, begin, begin + p.vdim, lane, lanes) : 0.0f;
+            for (int o = lanes >> 1; o > 0; o >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, o);
+            const float inverse = 1.0f / sqrtf(squares / static_cast<float>(p.vdim) + p.eps);
+            for (int d = lane * V; live && d < p.vdim; d += lanes * V) {
+                Span<V> v = biased_span<V>(v_source, v_bias, begin + d);
+#pragma unroll
+                for (int i = 0; i < V; ++i) v.v[i] *= inverse;
+                store_value(head, d, v);
+            }
+        }
+        return;
+    }
     for (int c = threadIdx.x * V; c < v_count; c += kPrepareThreads * V) {
-        const int head = c / p.vdim, d = c - head * p.vdim;
-        const Span<V> v = biased_span<V>(v_source, v_bias, c);
-        if (to_slot) store_span<V>(static_cast<T*>(p.value_cache) + p.entry(slot, head, position) * p.vdim + d, v);
-        if (!first_appended) store_span<V>(static_cast<T*>(p.value) + static_cast<int64_t>(row) * v_count + c, v);
+        const int head = c / p.vdim;
+        store_value(head, c - head * p.vdim, biased_span<V>(v_source, v_bias, c));
     }
 }
 
-// After a longer pass: the rows of a sequence's last chunk go into its slot, where they could not before (see chunk_prepare_kernel).
+// Before the attention of a longer pass: the blocks of `pool` positions that the pass completes, and the sum of the one it leaves open.  grid
+// (blocks of a sequence, sequences); CTA 0 takes the first block, which earlier passes may have begun, and the open one.
+template <class T> __global__ void __launch_bounds__(128) chunk_pool_kernel(const __grid_constant__ ChunkParams p, const RowsView rows) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int sequence = blockIdx.y, first = __ldg(rows.first + sequence), count = __ldg(rows.first + sequence + 1) - first;
+    const int slot = __ldg(rows.slot + sequence), length = rows.lengths[slot], end = length + count;
+    const int block0 = length / p.pool, block1 = (end - 1) / p.pool, per_head = p.dim + p.vdim;
+    auto pool_block = [&](int block) {
+        const int from = max(block * p.pool, length), to = min((block + 1) * p.pool, end), at = p.window + block;
+        const bool complete = to == (block + 1) * p.pool;
+        for (int c = threadIdx.x; c < p.kv_heads * per_head; c += blockDim.x) {
+            const int head = c / per_head, d = c - head * per_head;
+            const bool is_key = d < p.dim;
+            const T* source = is_key ? static_cast<const T*>(p.key) + head * p.dim + d : static_cast<const T*>(p.value) + head * p.vdim + d - p.dim;
+            const int64_t stride = p.kv_heads * (is_key ? p.dim : p.vdim);
+            float* sum = p.pool_state + static_cast<int64_t>(slot) * p.kv_heads * per_head + c;
+            float total = from > block * p.pool ? *sum : 0.0f;
+            for (int j = from; j < to; ++j) total += load_as_f32(source, (first + j - length) * stride);
+            if (!complete) *sum = total;
+            else if (at >= p.entries) continue;
+            else if (is_key) store_from_f32(static_cast<T*>(p.key_cache), p.entry_at(slot, head, at) * p.dim + d, total / static_cast<float>(p.pool));
+            else store_from_f32(static_cast<T*>(p.value_cache), p.entry_at(slot, head, at) * p.vdim + d - p.dim, total / static_cast<float>(p.pool));
+        }
+    };
+    const int block = block0 + static_cast<int>(blockIdx.x);
+    if (blockIdx.x == 0) {
+        pool_block(block0);
+        if (block1 > block0) pool_block(block1);   // (the same thread has read what earlier passes left)
+    } else if (block < block1) {
+        pool_block(block);
+    }
+}
+
+// After a longer pass: the rows that later ones see (of a sequence's last chunk or window) go into its slot, where they could not before
+// (see chunk_prepare_kernel).
 template <class T> __global__ void __launch_bounds__(128) chunk_append_kernel(const __grid_constant__ ChunkParams p, const RowsView rows) {
     grid_dependency_wait();
     grid_launch_dependents();
@@ -294,7 +397,7 @@ template <class T> __global__ void __launch_bounds__(128) chunk_append_kernel(co
         const RowPlace place = row_place(rows, row);
         const int length = rows.lengths[place.slot];
         const int last = length + __ldg(rows.first + place.sequence + 1) - __ldg(rows.first + place.sequence) - 1;
-        if (!p.overwrites(length, last) || p.chunk_start(place.position) != p.chunk_start(last) || !p.fits(place.position)) continue;
+        if (!p.overwrites(length, last) || !p.outlasts(place.position, last) || !p.fits(place.position)) continue;
         const int k_count = p.kv_heads * p.dim, v_count = p.kv_heads * p.vdim;
         for (int c = threadIdx.x; c < k_count; c += blockDim.x)
             static_cast<T*>(p.key_cache)[p.entry(place.slot, c / p.dim, place.position) * p.dim + c % p.dim] =
@@ -325,6 +428,11 @@ __device__ __forceinline__ float head_gate(const ChunkParams& p, int row, int he
     const float g = __ldg(p.projected + row * p.stride + p.heads * p.dim + p.key_columns() + p.value_columns() + head);
     return p.out_scale / (1.0f + expf(-g));
 }
+// A value's own gate, where every value of a head has one.
+__device__ __forceinline__ float value_gate(const ChunkParams& p, int row, int head, int column) {
+    const float g = __ldg(p.projected + row * p.stride + p.heads * p.dim + p.key_columns() + p.value_columns() + head * p.vdim + column);
+    return 1.0f / (1.0f + expf(-g));
+}
 // The scores are kept in units of log2: `scale2` times the product, or cap2 * tanh(product * scale / softcap).  The tensor-core kernels take
 // the hardware's exponential and reciprocal (an error near 1e-6 of the cap), the plain one the exact functions.
 __device__ __forceinline__ float capped_score(float product, float scale_by_cap, float cap2) {
@@ -342,6 +450,10 @@ __device__ __forceinline__ float denominator_factor(const ChunkParams& p, int he
 
 __device__ __forceinline__ void store_pair(const ChunkAttention& a, int row, int head, int column, float x, float y) {
     const int64_t at = row * a.out_stride + head * a.p.vdim + column;
+    if (a.p.gate_values) {
+        x *= value_gate(a.p, row, head, column);
+        y *= value_gate(a.p, row, head, column + 1);
+    }
     if (a.out) *reinterpret_cast<float2*>(a.out + at) = make_float2(x, y);
     if (a.out_hi) {
         uint32_t hi, lo;
@@ -381,10 +493,23 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     const int offset = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * a.positions_per_tile;
     if (offset >= count) return;
     const int last = min(offset + a.positions_per_tile, count);
-    const int key_begin = p.chunk_start(length + offset), key_end = length + last;   // absolute positions of the tile's keys
-    const int slot_start = p.chunk_start(length);                                    // position of the slot's entry 0
-    const int tiles = (key_end - key_begin + S::kKeys - 1) / S::kKeys;
+    // The tile's keys: `extra` kept positions or pooled blocks, then the positions from key_begin to key_end.
+    const int key_begin = p.first_seen(length + offset), key_end = length + last;
+    const int extra = p.pool > 0 ? p.blocks_seen(key_end - 1) : min(p.keep, key_begin), keys = extra + key_end - key_begin;
+    const int tiles = (keys + S::kKeys - 1) / S::kKeys;
     const int in_slot = p.appends_first(a.step) ? key_end : length;                  // positions whose keys the slot holds
+    const int slot_start = p.chunk_start(length);                                    // position of the slot's entry 0
+    const int ring_from = max(key_begin, p.keep), ring_at = p.window > 0 ? (ring_from - p.keep) % p.window : 0;
+    // entry of key n in the slot, or -1 - (row of the pass)
+    auto key_place = [&](int n) {
+        if (n < extra) return p.pool > 0 ? p.window + n : n;
+        const int j = key_begin + n - extra;
+        if (j >= in_slot) return -1 - (first + j - length);
+        if (p.window == 0) return j - slot_start;
+        if (j < p.keep) return j;
+        const int at = ring_at + j - ring_from;   // (the slot holds less than a window from ring_from on)
+        return p.keep + (at < p.window ? at : at - p.window);
+    };
 
     // rows of the tile: (position, head of the group)
     auto row_of = [&](int m, int& position, int& head) {
@@ -408,47 +533,50 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     const auto* key_rows = static_cast<const __nv_bfloat16*>(p.key);
     const auto* value_rows = static_cast<const __nv_bfloat16*>(p.value);
     auto fetch = [&](int tile, int stage) {
-        const int t0 = key_begin + tile * S::kKeys;
-        const uint32_t keys = smem_u32(ring + stage * S::kStageBytes), values = keys + S::kKeys * DK * 2;
+        const int t0 = tile * S::kKeys;
+        const uint32_t key_tile = smem_u32(ring + stage * S::kStageBytes), value_tile = key_tile + S::kKeys * DK * 2;
 #pragma unroll 4
         for (int c = threadIdx.x; c < S::kKeys * (DK / 8); c += S::kThreads) {
-            const int n = c / (DK / 8), piece = c % (DK / 8), j = t0 + n;
-            const bool live = j < key_end && piece * 8 < p.dim;
+            const int n = c / (DK / 8), piece = c % (DK / 8);
+            const bool live = t0 + n < keys && piece * 8 < p.dim;
             const __nv_bfloat16* from = key_slot;
             if (live) {
-                if (j < in_slot) from = key_slot + static_cast<int64_t>(j - slot_start) * p.dim + piece * 8;
-                else from = key_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim + piece * 8;
+                const int at = key_place(t0 + n);
+                if (at >= 0) from = key_slot + static_cast<int64_t>(at) * p.dim + piece * 8;
+                else from = key_rows + (static_cast<int64_t>(-1 - at) * p.kv_heads + kv_head) * p.dim + piece * 8;
             }
-            copy_async_16(keys + tile_offset<DK>(n, piece), from, live);
+            copy_async_16(key_tile + tile_offset<DK>(n, piece), from, live);
         }
 #pragma unroll 4
         for (int c = threadIdx.x; c < S::kKeys * (DV / 8); c += S::kThreads) {
-            const int n = c / (DV / 8), piece = c % (DV / 8), j = t0 + n;
-            const bool live = j < key_end && piece * 8 < p.vdim;
+            const int n = c / (DV / 8), piece = c % (DV / 8);
+            const bool live = t0 + n < keys && piece * 8 < p.vdim;
             const __nv_bfloat16* from = value_slot;
             if (live) {
-                if (j < in_slot) from = value_slot + static_cast<int64_t>(j - slot_start) * p.vdim + piece * 8;
-                else from = value_rows + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.vdim + piece * 8;
+                const int at = key_place(t0 + n);
+                if (at >= 0) from = value_slot + static_cast<int64_t>(at) * p.vdim + piece * 8;
+                else from = value_rows + (static_cast<int64_t>(-1 - at) * p.kv_heads + kv_head) * p.vdim + piece * 8;
             }
-            copy_async_16(values + tile_offset<DV>(n, piece), from, live);
+            copy_async_16(value_tile + tile_offset<DV>(n, piece), from, live);
         }
     };
     fetch(0, 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
 
     const int row_base = warp * 16;
-    // the two rows of this thread's fragments: which keys they see, [see_from, see_to)
-    int see_from[2], see_to[2];
+    // the two rows of this thread's fragments: which keys they see, [see_from, see_to) and the first see_extra
+    int see_from[2], see_to[2], see_extra[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         int position, head;
         const bool live = row_of(row_base + (lane >> 2) + i * 8, position, head);
-        see_from[i] = live ? p.chunk_start(length + position) : 0;
-        see_to[i] = live ? length + position + 1 : 0;
+        see_from[i] = live ? extra + p.first_seen(length + position) - key_begin : 0;
+        see_to[i] = live ? extra + length + position + 1 - key_begin : 0;
+        see_extra[i] = !live ? 0 : p.pool > 0 ? p.blocks_seen(length + position) : p.keep;
     }
     // keys that every live row of this warp sees need no mask
-    const int all_from = warp_max_int(max(see_to[0] ? see_from[0] : 0, see_to[1] ? see_from[1] : 0));
-    const int all_to = -warp_max_int(-min(see_to[0] ? see_to[0] : INT32_MAX, see_to[1] ? see_to[1] : INT32_MAX));
+    auto least = [&](const int (&v)[2]) { return -warp_max_int(-min(see_to[0] ? v[0] : INT32_MAX, see_to[1] ? v[1] : INT32_MAX)); };
+    const int all_from = warp_max_int(max(see_to[0] ? see_from[0] : 0, see_to[1] ? see_from[1] : 0)), all_to = least(see_to), all_extra = least(see_extra);
 
     constexpr int NT = S::kKeys / 8, VT = DV / 8;
     constexpr bool kHold = DK <= 128;      // query fragments stay in registers
@@ -475,7 +603,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
                 for (int k = 0; k < DK / 16; ++k) load_query(q[k], k);
             }
         }
-        const uint32_t keys = smem_u32(ring + (t & 1) * S::kStageBytes), values = keys + S::kKeys * DK * 2;
+        const uint32_t key_tile = smem_u32(ring + (t & 1) * S::kStageBytes), value_tile = key_tile + S::kKeys * DK * 2;
         float s[NT][4];
 #pragma unroll
         for (int n = 0; n < NT; ++n)
@@ -488,13 +616,13 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 #pragma unroll
             for (int n = 0; n < NT; n += 2) {
                 uint32_t b[4];
-                ldsm_x4(b, keys + tile_offset<DK>(n * 8 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)));
+                ldsm_x4(b, key_tile + tile_offset<DK>(n * 8 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)));
                 mma_16816(s[n], f, b[0], b[1]);
                 mma_16816(s[n + 1], f, b[2], b[3]);
             }
         }
-        const int t0 = key_begin + t * S::kKeys;
-        const bool mask = t0 < all_from || t0 + S::kKeys > all_to;
+        const int t0 = t * S::kKeys;
+        const bool mask = t0 + S::kKeys > all_to || (t0 < all_from && t0 + S::kKeys > all_extra);
         float high[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int n = 0; n < NT; ++n)
@@ -503,7 +631,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
                 s[n][i] = p.softcap > 0.0f ? capped_score(s[n][i], scale_by_cap, cap2) : s[n][i] * scale2;
                 if (mask) {
                     const int j = t0 + n * 8 + (lane & 3) * 2 + (i & 1);
-                    if (j < see_from[i >> 1] || j >= see_to[i >> 1]) s[n][i] = -INFINITY;
+                    if (j >= see_to[i >> 1] || (j < see_from[i >> 1] && j >= see_extra[i >> 1])) s[n][i] = -INFINITY;
                 }
                 high[i >> 1] = fmaxf(high[i >> 1], s[n][i]);
             }
@@ -537,7 +665,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 #pragma unroll
             for (int v = 0; v < VT; v += 2) {
                 uint32_t b[4];
-                ldsm_x4_trans(b, values + tile_offset<DV>(k * 16 + (lane & 15), v + (lane >> 4)));
+                ldsm_x4_trans(b, value_tile + tile_offset<DV>(k * 16 + (lane & 15), v + (lane >> 4)));
                 mma_16816(o[v], hi, b[0], b[1]);
                 mma_16816(o[v + 1], hi, b[2], b[3]);
                 mma_16816(o[v], lo, b[0], b[1]);
@@ -621,8 +749,8 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
         }
         return it;
     };
-    // tiles of an item: the slot holds the keys of the row's chunk, the row's own included, from entry 0 on
-    auto keys_of = [&](const StepItem& it) { return it.length - p.chunk_start(it.length) + 1; };
+    // tiles of an item: the slot holds the keys that the row sees, its own included, from entry 0 on
+    auto keys_of = [&](const StepItem& it) { return p.entries_seen(it.length); };
     auto range_of = [&](const StepItem& it, int& tile0, int& tile1) {
         const int tiles = (keys_of(it) + kStepKeys - 1) / kStepKeys, per_split = (tiles + a.splits - 1) / a.splits;
         tile0 = it.split * per_split;
@@ -829,11 +957,29 @@ __global__ void __launch_bounds__(64) chunk_combine_kernel(const __grid_constant
     for (int c = threadIdx.x; c < a.p.vdim; c += blockDim.x) {
         float v = 0.0f;
         for (int s = 0; s < a.splits; ++s) v = fmaf(a.partial[(at + s) * a.p.vdim + c], exp2_fast(a.partial_ml[(at + s) * 2] - best), v);
+        if (a.p.gate_values) v *= value_gate(a.p, row, head, c);
         store_forms(v * factor, row * a.out_stride + head * a.p.vdim + c, a.out, a.out_hi, a.out_lo);
     }
 }
 
 constexpr int kGenericThreads = 128, kGenericKeys = 128;
+
+// The keys and values of one row as the plain kernels walk them: kept positions or pooled blocks, then the run up to the row itself.
+template <class T> struct RowKeys {
+    const ChunkParams& p;
+    int slot, first, length, extra, begin, count, stored_end;
+    __device__ __forceinline__ RowKeys(const ChunkAttention& a, const RowPlace& place)
+        : p(a.p), slot(place.slot), first(__ldg(a.rows.first + place.sequence)), length(a.rows.lengths[place.slot]), extra(a.p.before_run(place.position)),
+          begin(a.p.first_seen(place.position)), count(extra + place.position + 1 - begin), stored_end(a.p.appends_first(a.step) ? place.position + 1 : length) {}
+    __device__ __forceinline__ const T* at(const void* cache, const void* rows, int size, int kv_head, int n) const {
+        if (n < extra) return static_cast<const T*>(cache) + p.entry_at(slot, kv_head, p.pool > 0 ? p.window + n : n) * size;
+        const int j = begin + n - extra;
+        return j < stored_end ? static_cast<const T*>(cache) + p.entry(slot, kv_head, j) * size
+                              : static_cast<const T*>(rows) + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * size;
+    }
+    __device__ __forceinline__ const T* key(int kv_head, int n) const { return at(p.key_cache, p.key, p.dim, kv_head, n); }
+    __device__ __forceinline__ const T* value(int kv_head, int n) const { return at(p.value_cache, p.value, p.vdim, kv_head, n); }
+};
 
 // grid (heads, rows): f32 FMAs over keys of either dtype
 template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_generic_kernel(const __grid_constant__ ChunkAttention a) {
@@ -846,26 +992,16 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
     grid_dependency_wait();
     grid_launch_dependents();
     const int head = blockIdx.x, row = blockIdx.y, kv_head = head / p.group, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const RowPlace place = row_place(a.rows, row);
-    const int length = a.rows.lengths[place.slot], first = __ldg(a.rows.first + place.sequence);
-    const int begin = p.chunk_start(place.position), end = place.position + 1, stored_end = p.appends_first(a.step) ? end : length;
-    auto key_at = [&](int j) {
-        return j < stored_end ? static_cast<const T*>(p.key_cache) + p.entry(place.slot, kv_head, j) * p.dim
-                              : static_cast<const T*>(p.key) + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.dim;
-    };
-    auto value_at = [&](int j) {
-        return j < stored_end ? static_cast<const T*>(p.value_cache) + p.entry(place.slot, kv_head, j) * p.vdim
-                              : static_cast<const T*>(p.value) + (static_cast<int64_t>(first + j - length) * p.kv_heads + kv_head) * p.vdim;
-    };
+    const RowKeys<T> keys(a, row_place(a.rows, row));
     for (int c = threadIdx.x; c < p.dim; c += kGenericThreads)
         query[c] = load_as_f32(static_cast<const T*>(p.query), (static_cast<int64_t>(row) * p.heads + head) * p.dim + c);
     for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads) acc[c] = 0.0f;
     float top = -INFINITY, total = 0.0f;
-    for (int k0 = begin; k0 < end; k0 += kGenericKeys) {
-        const int n = min(kGenericKeys, end - k0);
+    for (int k0 = 0; k0 < keys.count; k0 += kGenericKeys) {
+        const int n = min(kGenericKeys, keys.count - k0);
         __syncthreads();
         for (int j = warp; j < n; j += kGenericThreads / 32) {
-            const T* key = key_at(k0 + j);
+            const T* key = keys.key(kv_head, k0 + j);
             float dot = 0.0f;
             for (int c = lane; c < p.dim; c += 32) dot = fmaf(query[c], load_as_f32(key, c), dot);
             dot = warp_sum(dot);
@@ -882,7 +1018,7 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
         top = next;
         for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads) {
             float v = acc[c] * factor;
-            for (int j = 0; j < n; ++j) v = fmaf(w[j], load_as_f32(value_at(k0 + j), c), v);
+            for (int j = 0; j < n; ++j) v = fmaf(w[j], load_as_f32(keys.value(kv_head, k0 + j), c), v);
             acc[c] = v;
         }
     }
@@ -893,7 +1029,94 @@ template <class T> __global__ void __launch_bounds__(kGenericThreads) chunk_gene
     }
     const float scale = head_gate(p, row, head) / total;
     for (int c = threadIdx.x; c < p.vdim; c += kGenericThreads)
-        store_forms(acc[c] * scale, row * a.out_stride + head * p.vdim + c, a.out, a.out_hi, a.out_lo);
+        store_forms(acc[c] * (p.gate_values ? scale * value_gate(p, row, head, c) : scale), row * a.out_stride + head * p.vdim + c, a.out, a.out_hi, a.out_lo);
+}
+
+// Mixed heads, f32 FMAs: one CTA per row, all heads together.  A first sweep over the keys finds every head's largest score and sum, a
+// second one the weights, mixed, and the values under them.
+constexpr int kTalkThreads = 256, kTalkKeys = 64;
+size_t talk_generic_bytes(const ChunkParams& p) {
+    return (static_cast<size_t>(p.heads) * (p.dim + p.vdim + 2 * kTalkKeys + p.heads + 2)) * sizeof(float);
+}
+template <class T> __global__ void __launch_bounds__(kTalkThreads) talk_generic_kernel(const __grid_constant__ ChunkAttention a) {
+    extern __shared__ __align__(16) float sm[];
+    const ChunkParams& p = a.p;
+    const int H = p.heads;
+    float* query = sm;                        // [H][dim]
+    float* acc = query + H * p.dim;           // [H][vdim]
+    float* score = acc + H * p.vdim;          // [H][keys]
+    float* mixed = score + H * kTalkKeys;     // [H][keys]
+    float* talk = mixed + H * kTalkKeys;      // [H][H]
+    float* top = talk + H * H;                // [H]
+    float* total = top + H;                   // [H]
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const RowKeys<T> keys(a, row_place(a.rows, row));
+    for (int c = threadIdx.x; c < H * p.dim; c += kTalkThreads) query[c] = load_as_f32(static_cast<const T*>(p.query), static_cast<int64_t>(row) * H * p.dim + c);
+    for (int c = threadIdx.x; c < H * p.vdim; c += kTalkThreads) acc[c] = 0.0f;
+    for (int c = threadIdx.x; c < H * H; c += kTalkThreads) talk[c] = p.talk[c];
+    for (int h = threadIdx.x; h < H; h += kTalkThreads) { top[h] = -INFINITY; total[h] = 0.0f; }
+    auto scores = [&](int k0, int n) {   // a warp per key and kv head, its heads one after the other
+        for (int u = warp; u < n * p.kv_heads; u += kTalkThreads / 32) {
+            const int j = u / p.kv_heads, kv_head = u - j * p.kv_heads;
+            const T* key = keys.key(kv_head, k0 + j);
+            for (int h = kv_head * p.group; h < (kv_head + 1) * p.group; ++h) {
+                float dot = 0.0f;
+                for (int c = lane; c < p.dim; c += 32) dot = fmaf(query[h * p.dim + c], load_as_f32(key, c), dot);
+                dot = warp_sum(dot);
+                if (lane == 0) score[h * kTalkKeys + j] = p.softcap > 0.0f ? p.softcap * tanhf(dot * p.scale / p.softcap) : dot * p.scale;
+            }
+        }
+    };
+    for (int k0 = 0; k0 < keys.count; k0 += kTalkKeys) {
+        const int n = min(kTalkKeys, keys.count - k0);
+        __syncthreads();
+        scores(k0, n);
+        __syncthreads();
+        for (int h = warp; h < H; h += kTalkThreads / 32) {
+            float high = top[h];
+            for (int j = lane; j < n; j += 32) high = fmaxf(high, score[h * kTalkKeys + j]);
+            high = warp_max(high);
+            float sum = 0.0f;
+            for (int j = lane; j < n; j += 32) sum += expf(score[h * kTalkKeys + j] - high);
+            sum = warp_sum(sum);
+            if (lane == 0) {
+                total[h] = total[h] * expf(top[h] - high) + sum;
+                top[h] = high;
+            }
+        }
+    }
+    for (int k0 = 0; k0 < keys.count; k0 += kTalkKeys) {
+        const int n = min(kTalkKeys, keys.count - k0);
+        __syncthreads();
+        scores(k0, n);
+        __syncthreads();
+        for (int u = threadIdx.x; u < H * n; u += kTalkThreads) {
+            const int h = u / n, at = h * kTalkKeys + u - h * n;
+            score[at] = expf(score[at] - top[h]) / total[h];
+        }
+        __syncthreads();
+        for (int u = threadIdx.x; u < H * n; u += kTalkThreads) {
+            const int h = u / n, j = u - h * n;
+            float sum = 0.0f;
+            for (int g = 0; g < H; ++g) sum = fmaf(talk[h * H + g], score[g * kTalkKeys + j], sum);
+            mixed[h * kTalkKeys + j] = sum;
+        }
+        __syncthreads();
+        for (int c = threadIdx.x; c < H * p.vdim; c += kTalkThreads) {
+            const int h = c / p.vdim, d = c - h * p.vdim;
+            float v = acc[c];
+            for (int j = 0; j < n; ++j) v = fmaf(mixed[h * kTalkKeys + j], load_as_f32(keys.value(h / p.group, k0 + j), d), v);
+            acc[c] = v;
+        }
+    }
+    __syncthreads();
+    for (int c = threadIdx.x; c < H * p.vdim; c += kTalkThreads) {
+        const int h = c / p.vdim, d = c - h * p.vdim;
+        const float factor = p.gate_values ? p.out_scale * value_gate(p, row, h, d) : head_gate(p, row, h);
+        store_forms(acc[c] * factor, row * a.out_stride + c, a.out, a.out_hi, a.out_lo);
+    }
 }
 
 bool chunk_takes_mma(const ChunkParams& p, int dtype, int64_t out_stride) {
@@ -995,7 +1218,7 @@ extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* 
     auto aligned8 = [](const void* at) { return (reinterpret_cast<uintptr_t>(at) & 7) == 0; };
     const bool vector = p.dim % 4 == 0 && p.vdim % 4 == 0 && (p.rotate_pairs || (p.rot_dims >> 1) % 4 == 0) && p.stride % 4 == 0 && aligned(p.projected) && aligned(p.q_norm)
         && aligned(p.k_norm) && aligned(p.q_bias) && aligned(p.k_bias) && aligned(p.query) && aligned(p.key) && aligned(p.value) && aligned(p.key_cache) && aligned(p.value_cache)
-        && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0
+        && aligned(p.pool_state) && (p.rot_dims == 0 || (aligned(p.cosine) && aligned(p.sine))) && q % 4 == 0 && k % 4 == 0
         && (u.kind == 0 || (u.column % 4 == 0 && u.count % 4 == 0 && u.stride % 4 == 0 && aligned(u.out) && aligned8(u.out_hi) && aligned8(u.out_lo)));
     const dim3 grid(static_cast<unsigned>(rows.rows), static_cast<unsigned>(1 + (u.count + kUnitSlice - 1) / kUnitSlice));
     auto launch = [&](auto norm) {
@@ -1036,7 +1259,20 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
     a.splits = 1;
     if (!p.appends_first(a.step) && (!p.key || !p.value)) { set_error("b200_chunk_attention: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
     int status = B200_OK;
-    if (chunk_takes_mma(p, args->dtype, out_stride)) {
+    if (!a.step && p.pool > 0) {
+        auto pool = args->dtype == B200_BF16 ? chunk_pool_kernel<__nv_bfloat16> : chunk_pool_kernel<float>;
+        if (a.rows.sequences > 65535) { set_error("grouped attention: at most 65535 sequences in one pass"); return B200_UNSUPPORTED; }
+        const dim3 grid(static_cast<unsigned>(a.rows.max_count / p.pool + 2), static_cast<unsigned>(a.rows.sequences));
+        status = cuda_status(launch_dependent(pool, grid, dim3(128), 0, s, p, a.rows), "chunk_pool_kernel launch");
+        if (status != B200_OK) return status;
+    }
+    if (p.talk) {
+        const size_t smem = talk_generic_bytes(p);
+        auto kernel = args->dtype == B200_BF16 ? talk_generic_kernel<__nv_bfloat16> : talk_generic_kernel<float>;
+        if (smem > 220 * 1024) { set_error("mixed heads: %d heads of %d and %d are too large", p.heads, p.dim, p.vdim); return B200_UNSUPPORTED; }
+        B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+        status = cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(a.rows.rows)), dim3(kTalkThreads), smem, s, a), "talk_generic_kernel launch");
+    } else if (chunk_takes_mma(p, args->dtype, out_stride)) {
         int device = 0;
         B200_CUDA(cudaGetDevice(&device));
         const int most = a.step ? 16 : 64;

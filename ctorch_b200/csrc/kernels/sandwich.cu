@@ -100,7 +100,7 @@ int b200_embed_pairs(const b200_pair_embedding* e, const int64_t* ids, const b20
     if (!status) { set_error("b200_embed_pairs: the device status word could not be allocated"); return B200_NO_DEVICE; }
     const PairParams p{e->table, e->pairs, e->vocab, e->buckets, e->mul_prev, e->mul_cur, static_cast<int>(e->width), e->last, ids};
     const SandwichView a{nullptr, e->next, static_cast<float>(e->eps), nullptr, e->x, e->normed, static_cast<__nv_bfloat16*>(e->normed_hi),
-                         static_cast<__nv_bfloat16*>(e->normed_lo)};
+                         static_cast<__nv_bfloat16*>(e->normed_lo), false};
     const bool quads = sandwich_takes_quads(a, e->width) && ((reinterpret_cast<uintptr_t>(e->table) | reinterpret_cast<uintptr_t>(e->pairs)) & 15) == 0;
     auto kernel = e->dtype == B200_BF16 ? (quads ? embed_pairs_kernel<__nv_bfloat16, 4> : embed_pairs_kernel<__nv_bfloat16, 1>)
                                         : (quads ? embed_pairs_kernel<float, 4> : embed_pairs_kernel<float, 1>);

@@ -16,6 +16,7 @@ struct SandwichView {
     const float* residual;
     float *x, *normed;
     __nv_bfloat16 *normed_hi, *normed_lo;
+    bool plain;   // no norm follows: the planes take the stream itself
 };
 
 template <int V> __device__ __forceinline__ void store_normed(const SandwichView& a, int64_t at, const Lanes<V>& r) {
@@ -65,6 +66,7 @@ __device__ __forceinline__ void finish_sandwich(const SandwichView& a, int64_t r
             for (int k = 0; k < V; ++k) v.v[k] = fmaf(v.v[k] * factor, w.v[k], r.v[k]);
         }
         store_lanes<V>(a.x + base + c, v);
+        if (a.plain) store_normed<V>(a, base + c, v);
         squares = squares_of(v, squares);
         return v;
     };
@@ -88,9 +90,11 @@ __device__ __forceinline__ void finish_sandwich(const SandwichView& a, int64_t r
 
 // Host: checks and converts the C struct (false: inconsistent), and whether its rows take 16-byte accesses.
 inline bool sandwich_view(const b200_sandwich* a, SandwichView& v) {
-    if (!a || !a->after || !a->residual || !a->x || (a->next && !a->normed && !a->normed_hi) || (a->normed_hi && !a->normed_lo)) return false;
+    if (!a || !a->after || !a->residual || !a->x || (a->next && !a->normed && !a->normed_hi) || (a->normed_hi && !a->normed_lo)
+        || (a->plain && (a->next || (!a->normed && !a->normed_hi))))
+        return false;
     v = SandwichView{a->after, a->next, static_cast<float>(a->eps), a->residual, a->x, a->normed, static_cast<__nv_bfloat16*>(a->normed_hi),
-                     static_cast<__nv_bfloat16*>(a->normed_lo)};
+                     static_cast<__nv_bfloat16*>(a->normed_lo), a->plain != 0};
     return true;
 }
 inline bool sandwich_takes_quads(const SandwichView& v, int64_t width) {

@@ -1,6 +1,7 @@
 // State-space layers (Mamba-2): short causal convolution, selective recurrence, gated group norm; and the small kernels of
 // packed passes.  Everything here is f32: decays, step sizes, states and norms.  Lightning attention is the same recurrence with a fixed
-// decay per head, a step size of one, no skip and no convolution (only its SiLU): keys for B, queries for C, values for x.
+// decay per head, a step size of one, no skip and no convolution (only its SiLU): keys for B, queries for C, values for x.  The gated delta
+// rule shares the convolution and takes its own steps and scan (delta_rule.cu).
 //
 //   * Decode (one row per sequence): per (sequence, head) the channels the head needs are convolved from the slot's ring of recent
 //     inputs, then its [state][vdim] matrix is read once - decay, add dt B x^T, partial sums of S^T C - and written back.  The layer
@@ -12,8 +13,7 @@
 //     time through the packed f32 pipe.
 // The ring has `taps` entries although a token needs only taps - 1 old inputs: the entry a step writes is never one that the
 // same step reads, so the CTAs of a head group need no ordering among themselves.
-#include "mma.cuh"
-#include "rows.cuh"
+#include "state_space.cuh"
 
 #include <algorithm>
 #include <cmath>
@@ -32,63 +32,7 @@ bool rows_view(const b200_rows* pass, RowsView& view) {
 
 namespace {
 
-struct SsmParams {
-    int heads, vdim, state, groups, taps, channels, stride;
-    const float *conv_weight, *conv_bias, *dt_bias, *a_log, *d;
-    float *conv_state, *ssm_state;
-    const float* projected;
-    float *mixed, *y;
-    const float* fixed_decay;   // [heads] or NULL: step sizes and decays come from the projection
-};
-
-__device__ __forceinline__ float softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
-__device__ __forceinline__ float sigmoid_exact(float v) { return 1.0f / (1.0f + expf(-v)); }
-
-// Input of the convolution at `position` of a slot, from the ring of earlier passes (zero before the sequence's start).
-__device__ __forceinline__ float ring_input(const SsmParams& p, int slot, int position, int channel) {
-    if (position < 0) return 0.0f;
-    return p.conv_state[(static_cast<int64_t>(slot) * p.taps + position % p.taps) * p.channels + channel];
-}
-
-// Step size and decay of a head for one projected row.
-struct StepRate { float dt, decay; };
-__device__ __forceinline__ StepRate step_rate(const SsmParams& p, const float* row, int head) {
-    if (p.fixed_decay) return {1.0f, __ldg(p.fixed_decay + head)};
-    const float dt = softplus(row[p.heads * p.vdim + p.channels + head] + p.dt_bias[head]);
-    return {dt, expf(-expf(p.a_log[head]) * dt)};
-}
 __device__ __forceinline__ float skip_of(const SsmParams& p, int head) { return p.fixed_decay ? 0.0f : p.d[head]; }
-
-constexpr int kStepThreads = 256;
-
-// Convolved channels of one head for one token: [x: vdim | B: state | C: state] into `mixed`, and the token's inputs into the
-// slot's ring (B and C are shared by the heads of a group: its first head writes them).
-__device__ __forceinline__ void convolve_head(const SsmParams& p, const float* in, int slot, int position, int head, float* mixed) {
-    const int P = p.vdim, N = p.state, inner = p.heads * P, per_group = p.heads / p.groups, group = head / per_group;
-    const bool shared_writer = head == group * per_group;
-    // the ring entry of the current token; entry of the token `back` places before: ring_at - back, wrapped
-    const int ring_at = position % p.taps;
-    float* const ring = p.conv_state + static_cast<int64_t>(slot) * p.taps * p.channels;
-    for (int i = threadIdx.x; i < P + 2 * N; i += kStepThreads) {
-        const int c = i < P ? head * P + i : i < P + N ? inner + group * N + (i - P) : inner + (p.groups + group) * N + (i - P - N);
-        const float now = in[inner + c];
-        if (!p.conv_weight) {
-            mixed[i] = now * sigmoid_exact(now);
-            continue;
-        }
-        const float* weight = p.conv_weight + c * p.taps;
-        float acc = p.conv_bias[c];
-#pragma unroll 4
-        for (int j = 0; j < p.taps - 1; ++j) {
-            const int back = p.taps - 1 - j, at = ring_at < back ? ring_at - back + p.taps : ring_at - back;
-            const float old = position < back ? 0.0f : ring[at * p.channels + c];
-            acc = fmaf(weight[j], old, acc);
-        }
-        acc = fmaf(weight[p.taps - 1], now, acc);
-        mixed[i] = acc * sigmoid_exact(acc);
-        if (i < P || shared_writer) ring[ring_at * p.channels + c] = now;
-    }
-}
 
 // mixed[row, c] = silu(x | B | C): the inputs of a recurrence without convolution, grid (channel blocks, rows), V channels per thread.
 template <int V> __global__ void __launch_bounds__(128) activate_channels_kernel(const SsmParams p) {
@@ -139,10 +83,6 @@ template <int V> __global__ void __launch_bounds__(128) conv_step_kernel(const S
 // [state][vdim] block) and its x, B and C by bulk copies into one of two stages while the pair before it is worked on; eight warps
 // update the state in place and leave the partial outputs; the producer sends the stage's state back and refills it.  vdim and state
 // multiples of 4, vdim at most 1024.
-__device__ __forceinline__ void bulk_store(void* dst, const void* src, uint32_t bytes) {
-    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst), "r"(smem_u32(src)), "r"(bytes) : "memory");
-    asm volatile("cp.async.bulk.commit_group;" ::: "memory");
-}
 constexpr int kStreamThreads = kStepThreads + 32;
 struct StreamMeta { float dt, decay, fresh; };
 inline size_t ssm_stream_bytes(int state, int vdim) {
@@ -410,31 +350,6 @@ __global__ void __launch_bounds__(256) conv_ring_kernel(const SsmParams p, const
 }
 
 // ---- scan -----------------------------------------------------------------------------------------------------
-// Packed f32 pairs: two independent IEEE operations per instruction.
-__device__ __forceinline__ uint64_t pack2(float a, float b) {
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ float2 unpack2(uint64_t v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-    uint64_t r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
-__device__ __forceinline__ void copy_async_4(float* dst, const float* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-
 constexpr int kScanWarps = 4;
 
 // LN lanes of a warp share the state dimension (4 * Q values each, in quads LN * 4 apart), the other 32 / LN lane groups hold
@@ -666,6 +581,60 @@ int launch_group_norm(const float* y, const float* z, int64_t z_stride, const fl
                        "gated_group_norm_kernel launch");
 }
 
+// An RMS norm per head of `size` values, times weight [size], times silu(z): a warp per (row, head), the head in registers.  V adjacent
+// values per access.
+constexpr int kHeadNormWarps = 8, kHeadNormKeep = 4;
+template <int V>
+__global__ void __launch_bounds__(kHeadNormWarps * 32) head_norm_gated_kernel(const float* y, const float* z, int64_t z_stride, const float* weight, int64_t units,
+                                                                             int heads, int size, float eps, float* out, __nv_bfloat16* out_hi,
+                                                                             __nv_bfloat16* out_lo, int64_t out_stride) {
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int64_t unit = static_cast<int64_t>(blockIdx.x) * kHeadNormWarps + (threadIdx.x >> 5);
+    if (unit >= units) return;
+    const int lane = threadIdx.x & 31;
+    const int64_t row = unit / heads;
+    const int head = static_cast<int>(unit - row * heads);
+    const float *from = y + unit * size, *gate = z + row * z_stride + static_cast<int64_t>(head) * size;
+    const int64_t to = row * out_stride + static_cast<int64_t>(head) * size;
+    Lanes<V> kept[kHeadNormKeep];
+    float squares = 0.0f;
+    auto add = [&](const Lanes<V>& v) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) squares = fmaf(v.v[k], v.v[k], squares);
+    };
+#pragma unroll
+    for (int i = 0; i < kHeadNormKeep; ++i) {
+        const int c = (lane + i * 32) * V;
+        if (c < size) { kept[i] = load_lanes<V>(from + c); add(kept[i]); }
+    }
+    for (int c = (lane + kHeadNormKeep * 32) * V; c < size; c += 32 * V) add(load_lanes<V>(from + c));
+    const float inverse = 1.0f / sqrtf(warp_sum(squares) / static_cast<float>(size) + eps);
+    auto finish = [&](int c, Lanes<V> v) {
+        const Lanes<V> w = load_lanes<V>(weight + c), g = load_lanes<V>(gate + c);
+#pragma unroll
+        for (int k = 0; k < V; ++k) v.v[k] = v.v[k] * inverse * w.v[k] * (g.v[k] * sigmoid_exact(g.v[k]));
+        if constexpr (V == 4) {
+            if (out) store_lanes<V>(out + to + c, v);
+            if (out_hi) {
+                uint2 hi, lo;
+                pack_planes(v.v[0], v.v[1], hi.x, lo.x);
+                pack_planes(v.v[2], v.v[3], hi.y, lo.y);
+                *reinterpret_cast<uint2*>(out_hi + to + c) = hi;
+                if (out_lo) *reinterpret_cast<uint2*>(out_lo + to + c) = lo;
+            }
+        } else {
+            store_forms(v.v[0], to + c, out, out_hi, out_lo);
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kHeadNormKeep; ++i) {
+        const int c = (lane + i * 32) * V;
+        if (c < size) finish(c, kept[i]);
+    }
+    for (int c = (lane + kHeadNormKeep * 32) * V; c < size; c += 32 * V) finish(c, load_lanes<V>(from + c));
+}
+
 __global__ void rows_advance_kernel(const RowsView rows, const int64_t* ids, int32_t* last) {
     grid_dependency_wait();
     grid_launch_dependents();
@@ -762,9 +731,11 @@ int b200_dynamic_tanh(const float* x, const float* add_rows, const float* add_ve
 int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream) {
     RowsView rows;
     if (!rows_view(pass, rows)) return B200_BAD_ARGUMENT;
+    const int rates = !a || a->decay ? 0 : a->delta ? 2 : 1;   // columns per head behind the channels
     if (!a || a->heads <= 0 || a->vdim <= 0 || a->state <= 0 || a->groups <= 0 || a->heads % a->groups || a->taps <= 0
-        || (a->conv_weight ? !a->conv_bias || !a->conv_state : a->taps != 1) || (!a->decay && (!a->dt_bias || !a->a_log || !a->d)) || !a->ssm_state
-        || !a->projected || !a->y || (a->stride && a->stride < 2 * int64_t{a->heads} * a->vdim + 2 * int64_t{a->groups} * a->state + (a->decay ? 0 : a->heads))
+        || (a->conv_weight ? !a->conv_bias || !a->conv_state : a->taps != 1) || (!a->decay && (!a->dt_bias || !a->a_log || (!a->d && !a->delta))) || !a->ssm_state
+        || (a->delta && (a->decay || !a->conv_weight))
+        || !a->projected || !a->y || (a->stride && a->stride < 2 * int64_t{a->heads} * a->vdim + 2 * int64_t{a->groups} * a->state + rates * a->heads)
         || a->stride > INT32_MAX) {
         set_error("b200_ssm_forward: bad pointer or size");
         return B200_BAD_ARGUMENT;
@@ -772,14 +743,14 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
     SsmParams p{};
     p.heads = a->heads; p.vdim = a->vdim; p.state = a->state; p.groups = a->groups; p.taps = a->taps;
     p.channels = a->heads * a->vdim + 2 * a->groups * a->state;
-    p.stride = a->stride ? static_cast<int>(a->stride) : a->heads * a->vdim + p.channels + (a->decay ? 0 : a->heads);
+    p.stride = a->stride ? static_cast<int>(a->stride) : a->heads * a->vdim + p.channels + rates * a->heads;
     p.fixed_decay = a->decay;
     p.conv_weight = a->conv_weight; p.conv_bias = a->conv_bias; p.dt_bias = a->dt_bias; p.a_log = a->a_log; p.d = a->d;
     p.conv_state = a->conv_state; p.ssm_state = a->ssm_state; p.projected = a->projected; p.mixed = a->mixed; p.y = a->y;
     cudaStream_t s = as_stream(stream);
     if (rows.max_count == 1) {
         const bool quads = a->vdim % 4 == 0 && (reinterpret_cast<uintptr_t>(a->ssm_state) & 15) == 0;
-        const size_t streamed = ssm_stream_bytes(a->state, a->vdim);
+        const size_t streamed = a->delta ? 0 : ssm_stream_bytes(a->state, a->vdim);
         const bool aligned = ((reinterpret_cast<uintptr_t>(p.projected) | reinterpret_cast<uintptr_t>(p.mixed) | reinterpret_cast<uintptr_t>(p.conv_bias)
                                | reinterpret_cast<uintptr_t>(p.conv_state)) & 15) == 0;
         int device = 0;
@@ -787,10 +758,14 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
         const int64_t units = static_cast<int64_t>(rows.rows) * a->heads;
         const int64_t per_sm = std::min<int64_t>(7, (228 * 1024) / (streamed + 1024 + 128)), resident = sm_count(device) * per_sm;
         // streaming pays from a few pairs per CTA on; below that its extra launch and ramp cost more
-        if (quads && a->mixed && aligned && a->state % 4 == 0 && a->vdim <= 4 * kStepThreads && streamed <= 110 * 1024 && units >= 4 * resident) {
+        const bool streams = a->mixed && aligned
+            && (a->delta ? delta_step_streams(p, rows, sm_count(device))
+                         : quads && a->state % 4 == 0 && a->vdim <= 4 * kStepThreads && streamed <= 110 * 1024 && units >= 4 * resident);
+        if (streams) {
             int32_t* status = device_status_word(device);
             if (!status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
             auto stream_steps = [&]() -> int {
+                if (a->delta) return launch_delta_step_stream(p, rows, sm_count(device), status, s);
                 B200_CUDA(cudaFuncSetAttribute(ssm_step_stream_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(streamed)));
                 return cuda_status(launch_dependent(ssm_step_stream_kernel, dim3(static_cast<unsigned>(std::min(units, resident))), dim3(kStreamThreads), streamed, s, p, rows,
                                                     status), "ssm_step_stream_kernel launch");
@@ -807,6 +782,7 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
                                          "conv_step_kernel launch");
             return conv != B200_OK ? conv : stream_steps();
         }
+        if (a->delta) return launch_delta_step(p, rows, s);
         const size_t smem = sizeof(float) * (((a->vdim + 2 * a->state + 3) & ~3) + kStepThreads * (quads ? 4 : 1));
         if (smem > 200 * 1024) { set_error("b200_ssm_forward: a head of %d x %d values does not fit shared memory", a->state, a->vdim); return B200_UNSUPPORTED; }
         auto kernel = quads ? ssm_step_kernel<4> : ssm_step_kernel<1>;
@@ -830,6 +806,7 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
         status = cuda_status(launch_dependent(conv_ring_kernel, dim3(blocks, static_cast<unsigned>(rows.sequences)), dim3(256), 0, s, p, rows), "conv_ring_kernel launch");
     }
     if (status != B200_OK) return status;
+    if (a->delta) return launch_delta_scan(p, rows, s);
     if (a->state <= 32) return launch_scan<8, 1>(p, rows, s);
     if (a->state <= 64) return launch_scan<8, 2>(p, rows, s);
     if (a->state <= 96) return launch_scan<8, 3>(p, rows, s);
@@ -846,6 +823,25 @@ int b200_gated_group_norm(const float* y, const float* z, int64_t z_stride, cons
 int b200_norm_gated(const float* y, const float* gate, int64_t gate_stride, const float* weight, int64_t rows, int64_t width, int32_t parts, double eps,
                     float factor, float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream) {
     return launch_group_norm<false>(y, gate, gate_stride, weight, rows, width, parts, eps, factor, out, out_hi, out_lo, out_stride, stream, "b200_norm_gated");
+}
+
+int b200_head_norm_gated(const float* y, const float* gate, int64_t gate_stride, const float* weight, int64_t rows, int32_t heads, int32_t size, double eps,
+                         float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream) {
+    if (!y || !gate || !weight || rows < 0 || heads <= 0 || size <= 0 || (!out && !out_hi) || out_stride < static_cast<int64_t>(heads) * size
+        || rows * heads > int64_t{INT32_MAX} * kHeadNormWarps) {
+        set_error("b200_head_norm_gated: bad pointer or size");
+        return B200_BAD_ARGUMENT;
+    }
+    if (rows == 0) return B200_OK;
+    const bool quads = size % 4 == 0 && gate_stride % 4 == 0 && out_stride % 4 == 0
+        && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(out)
+             | (reinterpret_cast<uintptr_t>(out_hi) << 1) | (reinterpret_cast<uintptr_t>(out_lo) << 1)) & 15) == 0;
+    const int64_t units = rows * heads;
+    return cuda_status(launch_dependent(quads ? head_norm_gated_kernel<4> : head_norm_gated_kernel<1>,
+                                        dim3(static_cast<unsigned>((units + kHeadNormWarps - 1) / kHeadNormWarps)), dim3(kHeadNormWarps * 32), 0, as_stream(stream), y,
+                                        gate, gate_stride, weight, units, static_cast<int>(heads), static_cast<int>(size), static_cast<float>(eps), out,
+                                        static_cast<__nv_bfloat16*>(out_hi), static_cast<__nv_bfloat16*>(out_lo), out_stride),
+                       "head_norm_gated_kernel launch");
 }
 
 }  // extern "C"

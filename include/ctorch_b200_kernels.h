@@ -377,6 +377,10 @@ typedef struct b200_ssm_args {
      * row has no dt columns; without conv_weight there is no convolution either (taps 1, no conv_state). */
     const float* decay;            /* [heads] or NULL */
     int64_t stride;                /* floats between projected rows; 0: the width given above */
+    /* The gated delta rule: with k, q and v in the places of B, C and x, unit vectors k / |k| and q / (|q| sqrt(state)) (lengths with 1e-6
+     * under the root), beta = sigmoid of heads further columns behind the dt columns, and g = exp(-exp(a_log) dt):
+     *   S = g S, u = beta (v - S^T k), S = S + k u^T, y = S^T q.   d is not read (no skip). */
+    int32_t delta;                 /* 1: the delta rule; needs the convolution */
 } b200_ssm_args;
 /* Convolution, step sizes, recurrence and its output for every row; the slots' states move on.  Passes with one row per
  * sequence run as one kernel bound by the state's traffic, longer ones as convolution + scan. */
@@ -393,6 +397,10 @@ B200_API int b200_gated_group_norm(const float* y, const float* z, int64_t z_str
  * between rows, the results out_stride elements. */
 B200_API int b200_norm_gated(const float* y, const float* gate, int64_t gate_stride, const float* weight, int64_t rows, int64_t width,
                              int32_t parts, double eps, float factor, float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream);
+
+/* An RMS norm of every head of `size` values, times weight [size] (the same for all heads), times silu(gate). */
+B200_API int b200_head_norm_gated(const float* y, const float* gate, int64_t gate_stride, const float* weight, int64_t rows, int32_t heads,
+                                  int32_t size, double eps, float* out, void* out_hi, void* out_lo, int64_t out_stride, void* stream);
 
 /* One-pool cache of a latent-attention layer: per token kv_rank latent values and the shared rotated key part, width values
  * in all, paged like the other caches with one head.  `lengths` [slots] is the caller's. */
@@ -472,9 +480,21 @@ typedef struct b200_chunk_args {
     const float* sink;             /* [heads] or NULL: the softmax's denominator also holds exp(sink) */
     int32_t scaled;                /* 1: the result is multiplied by out_scale */
     float out_scale;
+    /* A sliding window instead of chunks: a position sees the last `window` positions up to itself, and beside them either the sequence's
+     * first `keep` positions, or one key and value per block of `pool` positions (counted from 0) that lies wholly before the window - the
+     * means of the block's keys and values as the cache holds them.  The slot holds position p < keep in entry p, later ones in entry
+     * keep + (p - keep) mod window, block b in entry window + b: what a position sees, are the first entries.  entries >= keep + window
+     * (+ blocks).  Longer passes need the key and value workspaces. */
+    int32_t window;                /* 0: none */
+    int32_t keep;
+    int32_t pool;                  /* not with keep */
+    float* pool_state;             /* pool: [slots][kv_heads][dim + vdim], sums of the block that a slot's sequence is in */
+    int32_t norm_values;           /* 1: every head's value is divided by its root mean square */
+    int32_t gate_values;           /* 1 (with no_gate): heads*vdim g columns, sigmoid(g) of every value in place of the head's */
+    const float* talk;             /* [heads][heads] or NULL: softmax weights of head h <- sum over g of talk[h][g] times those of head g (no sink) */
 } b200_chunk_args;
-/* Norms of queries and keys: RMS over all heads of the row at once with the weights q_norm and k_norm; none; RMS per head without weights
- * (after the rotation, which does not change it). */
+/* Norms of queries and keys, before the rotation: RMS over all heads of the row at once with the weights q_norm and k_norm; none; RMS per head,
+ * with weights q_norm and k_norm [dim] for every head, or without (NULL). */
 enum b200_head_norm { B200_HEAD_NORM_PROJECTION = 0, B200_HEAD_NORM_NONE = 1, B200_HEAD_NORM_HEAD = 2 };
 
 /* Activation of feed-forward units that were projected beside the attention's inputs: `kind` 1: silu(gate) * up of `count` interleaved
@@ -503,6 +523,8 @@ typedef struct b200_route {
     int32_t softmax;               /* 1: the scores are the softmax over all outputs */
     const float* correction;       /* [experts] or NULL: added to the scores for the choice; the weights stay without it */
     int32_t identity;              /* the last outputs that are identity experts: chosen like the others, but neither ranked nor counted */
+    const float* bias;             /* [experts] or NULL: added to the logits, for the choice and the weights */
+    int32_t chosen_softmax;        /* 1: the largest logits are chosen, the weights are the softmax over their logits alone */
 } b200_route;
 /* The choice alone, for `rows` rows of logits with `stride` floats between them (route->column is not used). */
 B200_API int b200_route_rows(const float* logits, int64_t rows, int64_t stride, const b200_route* route, void* stream);
@@ -556,6 +578,7 @@ typedef struct b200_sandwich {
     float* normed;
     void* normed_hi;
     void* normed_lo;
+    int32_t plain;                 /* 1 (next NULL): normed and the planes receive x itself */
 } b200_sandwich;
 B200_API int b200_sandwich_rows(const float* y, int64_t rows, int64_t width, const b200_sandwich* args, void* stream);
 

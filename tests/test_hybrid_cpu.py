@@ -17,7 +17,7 @@ def host_model(c, dtype="bf16", weights=None):
 
 
 def test_registry_names_the_designs():
-    assert B.architectures() == ["Lozepel", "Ripitar", "Sinezen", "TransformerDecoder"]
+    assert B.architectures() == ["Lozepel", "Ripitar", "Rizovik", "Sinezen", "TransformerDecoder"]
     with pytest.raises(B.B200Error, match="unknown architecture 'Nothing'"):
         host_model({"architecture": "Nothing", "vocab": 4})
 
