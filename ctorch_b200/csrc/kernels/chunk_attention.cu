@@ -417,6 +417,11 @@ struct ChunkAttention {
     int32_t* status;
     int positions_per_tile, heads_per_tile, head_tiles, splits;
     float *partial, *partial_ml;    // splits > 1: [rows, heads, splits, vdim], [rows, heads, splits, 2]
+    // mixed heads: the tables between the kernels of b200_chunk_attention, for the positions [begin, begin + span) of the sequences from
+    // first_sequence on
+    float *table, *table_ml;        // [sequence, position, heads, pitch] scores, then packed weights; [..., heads, splits, 2] their largest and sum
+    int64_t pitch;
+    int first_sequence, begin, span;
     float* out;
     __nv_bfloat16 *out_hi, *out_lo;
     int64_t out_stride;
@@ -463,45 +468,55 @@ __device__ __forceinline__ void store_pair(const ChunkAttention& a, int row, int
     }
 }
 
+// Row of the tables of mixed heads.
+__device__ __forceinline__ int64_t table_row(const ChunkAttention& a, int sequence, int position) {
+    return static_cast<int64_t>(sequence - a.first_sequence) * a.span + position - a.begin;
+}
+// Two adjacent weights (hi | lo << 16 each) as operand pairs.
+__device__ __forceinline__ void unpack_weights(uint2 w, uint32_t& hi, uint32_t& lo) {
+    hi = __byte_perm(w.x, w.y, 0x5410);
+    lo = __byte_perm(w.x, w.y, 0x7632);
+}
+// What the attention kernels do: everything, or (mixed heads) the scores with their largest and sum, or the values under given weights.
+enum ChunkPart { kWhole = 0, kScores = 1, kValues = 2 };
+
 // 16-byte piece `chunk` of a tile row of COLUMNS values, swizzled by the row.
 template <int COLUMNS> __device__ __forceinline__ uint32_t tile_offset(int row, int chunk) {
     return static_cast<uint32_t>(row * COLUMNS * 2 + ((chunk ^ (row & 7)) << 4));
 }
 
-template <int DK, int DV> struct ChunkShape {
-    static constexpr int kWarps = 4, kThreads = kWarps * 32;
-    static constexpr int kRows = 64;
-    static constexpr int kKeys = DK + DV <= 256 ? 64 : 32;   // keys of a tile
-    static constexpr int kStageBytes = kKeys * (DK + DV) * 2;
-    static constexpr int kQueryBytes = kRows * DK * 2;
-    static constexpr int kSmem = kQueryBytes + 2 * kStageBytes;
-};
-
-template <int DK, int DV>
-__global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ ChunkAttention a) {
-    using S = ChunkShape<DK, DV>;
-    extern __shared__ __align__(128) uint8_t smem[];
-    const ChunkParams& p = a.p;
-    uint8_t* ring = smem + S::kQueryBytes;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int sequence = blockIdx.y, head_tile = blockIdx.z % a.head_tiles, kv_head = blockIdx.z / a.head_tiles;
-    grid_dependency_wait();
-    grid_launch_dependents();
-    const int first = __ldg(a.rows.first + sequence), count = __ldg(a.rows.first + sequence + 1) - first;
-    const int slot = __ldg(a.rows.slot + sequence), length = a.rows.lengths[slot];
-    // the tiles with the most keys start first
-    const int offset = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * a.positions_per_tile;
-    if (offset >= count) return;
-    const int last = min(offset + a.positions_per_tile, count);
-    // The tile's keys: `extra` kept positions or pooled blocks, then the positions from key_begin to key_end.
-    const int key_begin = p.first_seen(length + offset), key_end = length + last;
-    const int extra = p.pool > 0 ? p.blocks_seen(key_end - 1) : min(p.keep, key_begin), keys = extra + key_end - key_begin;
-    const int tiles = (keys + S::kKeys - 1) / S::kKeys;
-    const int in_slot = p.appends_first(a.step) ? key_end : length;                  // positions whose keys the slot holds
-    const int slot_start = p.chunk_start(length);                                    // position of the slot's entry 0
-    const int ring_from = max(key_begin, p.keep), ring_at = p.window > 0 ? (ring_from - p.keep) % p.window : 0;
+// The rows and keys of one CTA of a longer pass: some positions of a sequence x some heads of a group; the keys that they see - `extra` kept
+// positions or pooled blocks, then the positions from key_begin to key_end.
+struct TileRows {
+    const ChunkAttention& a;
+    const ChunkParams& p;
+    int sequence, head_tile, kv_head, first, count, slot, length, offset, last;
+    int key_begin, key_end, extra, keys, in_slot, slot_start, ring_from, ring_at;
+    __device__ __forceinline__ TileRows(const ChunkAttention& attention, int sequence_, int z, int offset_)
+        : a(attention), p(attention.p), sequence(sequence_), head_tile(z % attention.head_tiles), kv_head(z / attention.head_tiles), offset(offset_) {
+        first = __ldg(a.rows.first + sequence);
+        count = __ldg(a.rows.first + sequence + 1) - first;
+        slot = __ldg(a.rows.slot + sequence);
+        length = a.rows.lengths[slot];
+        last = min(offset + a.positions_per_tile, count);
+        key_begin = p.first_seen(length + offset);
+        key_end = length + last;
+        extra = p.pool > 0 ? p.blocks_seen(key_end - 1) : min(p.keep, key_begin);
+        keys = extra + key_end - key_begin;
+        in_slot = p.appends_first(a.step) ? key_end : length;   // positions whose keys the slot holds
+        slot_start = p.chunk_start(length);                     // position of the slot's entry 0
+        ring_from = max(key_begin, p.keep);
+        ring_at = p.window > 0 ? (ring_from - p.keep) % p.window : 0;
+    }
+    // row m of the tile: position inside the pass, and head
+    __device__ __forceinline__ bool row(int m, int& position, int& head) const {
+        position = offset + m / a.heads_per_tile;
+        const int in_group = head_tile * a.heads_per_tile + m % a.heads_per_tile;
+        head = kv_head * p.group + in_group;
+        return m < a.positions_per_tile * a.heads_per_tile && position < last && in_group < p.group;
+    }
     // entry of key n in the slot, or -1 - (row of the pass)
-    auto key_place = [&](int n) {
+    __device__ __forceinline__ int place(int n) const {
         if (n < extra) return p.pool > 0 ? p.window + n : n;
         const int j = key_begin + n - extra;
         if (j >= in_slot) return -1 - (first + j - length);
@@ -509,56 +524,65 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
         if (j < p.keep) return j;
         const int at = ring_at + j - ring_from;   // (the slot holds less than a window from ring_from on)
         return p.keep + (at < p.window ? at : at - p.window);
-    };
-
-    // rows of the tile: (position, head of the group)
-    auto row_of = [&](int m, int& position, int& head) {
-        position = offset + m / a.heads_per_tile;
-        const int in_group = head_tile * a.heads_per_tile + m % a.heads_per_tile;
-        head = kv_head * p.group + in_group;
-        return m < a.positions_per_tile * a.heads_per_tile && position < last && in_group < p.group;
-    };
-    {
-        const auto* query = static_cast<const __nv_bfloat16*>(p.query);
-        for (int c = threadIdx.x; c < S::kRows * (DK / 8); c += S::kThreads) {
-            const int m = c / (DK / 8), piece = c % (DK / 8);
-            int position, head;
-            const bool live = row_of(m, position, head) && piece * 8 < p.dim;
-            copy_async_16(smem_u32(smem) + tile_offset<DK>(m, piece),
-                          live ? query + (static_cast<int64_t>(first + position) * p.heads + head) * p.dim + piece * 8 : query, live);
+    }
+    // COLUMNS values of ROWS keys from key t0 on to shared memory, swizzled, by 128 threads
+    template <int COLUMNS, int ROWS>
+    __device__ __forceinline__ void fetch(uint32_t to, int t0, const void* cache, const void* workspace, int size) const {
+        const auto* stored = static_cast<const __nv_bfloat16*>(cache) + (static_cast<int64_t>(slot) * p.kv_heads + kv_head) * p.entries * size;
+        const auto* fresh = static_cast<const __nv_bfloat16*>(workspace) + kv_head * size;
+#pragma unroll 4
+        for (int c = threadIdx.x; c < ROWS * (COLUMNS / 8); c += 128) {
+            const int n = c / (COLUMNS / 8), piece = c % (COLUMNS / 8);
+            const bool live = t0 + n < keys && piece * 8 < size;
+            const __nv_bfloat16* from = stored;
+            if (live) {
+                const int at = place(t0 + n);
+                from = (at >= 0 ? stored + static_cast<int64_t>(at) * size : fresh + static_cast<int64_t>(-1 - at) * p.kv_heads * size) + piece * 8;
+            }
+            copy_async_16(to + tile_offset<COLUMNS>(n, piece), from, live);
         }
     }
-    const auto* key_slot = static_cast<const __nv_bfloat16*>(p.key_cache) + (static_cast<int64_t>(slot) * p.kv_heads + kv_head) * p.entries * p.dim;
-    const auto* value_slot = static_cast<const __nv_bfloat16*>(p.value_cache) + (static_cast<int64_t>(slot) * p.kv_heads + kv_head) * p.entries * p.vdim;
-    const auto* key_rows = static_cast<const __nv_bfloat16*>(p.key);
-    const auto* value_rows = static_cast<const __nv_bfloat16*>(p.value);
-    auto fetch = [&](int tile, int stage) {
-        const int t0 = tile * S::kKeys;
-        const uint32_t key_tile = smem_u32(ring + stage * S::kStageBytes), value_tile = key_tile + S::kKeys * DK * 2;
-#pragma unroll 4
-        for (int c = threadIdx.x; c < S::kKeys * (DK / 8); c += S::kThreads) {
-            const int n = c / (DK / 8), piece = c % (DK / 8);
-            const bool live = t0 + n < keys && piece * 8 < p.dim;
-            const __nv_bfloat16* from = key_slot;
-            if (live) {
-                const int at = key_place(t0 + n);
-                if (at >= 0) from = key_slot + static_cast<int64_t>(at) * p.dim + piece * 8;
-                else from = key_rows + (static_cast<int64_t>(-1 - at) * p.kv_heads + kv_head) * p.dim + piece * 8;
-            }
-            copy_async_16(key_tile + tile_offset<DK>(n, piece), from, live);
+    // ROWS x COLUMNS queries of the tile
+    template <int COLUMNS, int ROWS> __device__ __forceinline__ void fetch_queries(uint32_t to) const {
+        const auto* query = static_cast<const __nv_bfloat16*>(p.query);
+        for (int c = threadIdx.x; c < ROWS * (COLUMNS / 8); c += 128) {
+            const int m = c / (COLUMNS / 8), piece = c % (COLUMNS / 8);
+            int position, head;
+            const bool live = row(m, position, head) && piece * 8 < p.dim;
+            copy_async_16(to + tile_offset<COLUMNS>(m, piece), live ? query + (static_cast<int64_t>(first + position) * p.heads + head) * p.dim + piece * 8 : query, live);
         }
-#pragma unroll 4
-        for (int c = threadIdx.x; c < S::kKeys * (DV / 8); c += S::kThreads) {
-            const int n = c / (DV / 8), piece = c % (DV / 8);
-            const bool live = t0 + n < keys && piece * 8 < p.vdim;
-            const __nv_bfloat16* from = value_slot;
-            if (live) {
-                const int at = key_place(t0 + n);
-                if (at >= 0) from = value_slot + static_cast<int64_t>(at) * p.vdim + piece * 8;
-                else from = value_rows + (static_cast<int64_t>(-1 - at) * p.kv_heads + kv_head) * p.vdim + piece * 8;
-            }
-            copy_async_16(value_tile + tile_offset<DV>(n, piece), from, live);
-        }
+    }
+};
+// the tiles with the most keys start first
+__device__ __forceinline__ int tile_begin(const ChunkAttention& a) { return a.begin + (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * a.positions_per_tile; }
+
+template <int DK, int DV, int PART = kWhole> struct ChunkShape {
+    static constexpr int kWarps = 4, kThreads = kWarps * 32;
+    static constexpr int kRows = 64;
+    static constexpr int kKeys = PART != kWhole || DK + DV <= 256 ? 64 : 32;   // keys of a tile
+    static constexpr int kKeyBytes = kKeys * DK * 2, kStageBytes = PART == kScores ? kKeyBytes : kKeyBytes + kKeys * DV * 2;
+    static constexpr int kQueryBytes = kRows * DK * 2;
+    static constexpr int kSmem = kQueryBytes + 2 * kStageBytes;
+};
+
+// PART kWhole or kScores
+template <int DK, int DV, int PART>
+__global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ ChunkAttention a) {
+    using S = ChunkShape<DK, DV, PART>;
+    extern __shared__ __align__(128) uint8_t smem[];
+    const ChunkParams& p = a.p;
+    uint8_t* ring = smem + S::kQueryBytes;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const TileRows tile(a, a.first_sequence + blockIdx.y, blockIdx.z, tile_begin(a));
+    if (tile.offset >= tile.count) return;
+    const int tiles = (tile.keys + S::kKeys - 1) / S::kKeys;
+    tile.fetch_queries<DK, S::kRows>(smem_u32(smem));
+    auto fetch = [&](int t, int stage) {
+        const uint32_t at = smem_u32(ring + stage * S::kStageBytes);
+        tile.fetch<DK, S::kKeys>(at, t * S::kKeys, p.key_cache, p.key, p.dim);
+        if constexpr (PART == kWhole) tile.fetch<DV, S::kKeys>(at + S::kKeyBytes, t * S::kKeys, p.value_cache, p.value, p.vdim);
     };
     fetch(0, 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -566,19 +590,22 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
     const int row_base = warp * 16;
     // the two rows of this thread's fragments: which keys they see, [see_from, see_to) and the first see_extra
     int see_from[2], see_to[2], see_extra[2];
+    float* table[2] = {nullptr, nullptr};
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         int position, head;
-        const bool live = row_of(row_base + (lane >> 2) + i * 8, position, head);
-        see_from[i] = live ? extra + p.first_seen(length + position) - key_begin : 0;
-        see_to[i] = live ? extra + length + position + 1 - key_begin : 0;
-        see_extra[i] = !live ? 0 : p.pool > 0 ? p.blocks_seen(length + position) : p.keep;
+        const bool live = tile.row(row_base + (lane >> 2) + i * 8, position, head);
+        const int at = tile.length + position;
+        see_from[i] = live ? tile.extra + p.first_seen(at) - tile.key_begin : 0;
+        see_to[i] = live ? tile.extra + at + 1 - tile.key_begin : 0;
+        see_extra[i] = !live ? 0 : p.pool > 0 ? p.blocks_seen(at) : p.keep;
+        if (PART == kScores && live) table[i] = a.table + (table_row(a, tile.sequence, position) * p.heads + head) * a.pitch + (lane & 3) * 2;
     }
     // keys that every live row of this warp sees need no mask
     auto least = [&](const int (&v)[2]) { return -warp_max_int(-min(see_to[0] ? v[0] : INT32_MAX, see_to[1] ? v[1] : INT32_MAX)); };
     const int all_from = warp_max_int(max(see_to[0] ? see_from[0] : 0, see_to[1] ? see_from[1] : 0)), all_to = least(see_to), all_extra = least(see_extra);
 
-    constexpr int NT = S::kKeys / 8, VT = DV / 8;
+    constexpr int NT = S::kKeys / 8, VT = PART == kWhole ? DV / 8 : 1;
     constexpr bool kHold = DK <= 128;      // query fragments stay in registers
     uint32_t q[kHold ? DK / 16 : 1][4];
     float o[VT][4];
@@ -603,7 +630,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
                 for (int k = 0; k < DK / 16; ++k) load_query(q[k], k);
             }
         }
-        const uint32_t key_tile = smem_u32(ring + (t & 1) * S::kStageBytes), value_tile = key_tile + S::kKeys * DK * 2;
+        const uint32_t key_tile = smem_u32(ring + (t & 1) * S::kStageBytes), value_tile = key_tile + S::kKeyBytes;
         float s[NT][4];
 #pragma unroll
         for (int n = 0; n < NT; ++n)
@@ -635,6 +662,14 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
                 }
                 high[i >> 1] = fmaxf(high[i >> 1], s[n][i]);
             }
+        if constexpr (PART == kScores) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                if (!table[i]) continue;
+#pragma unroll
+                for (int n = 0; n < NT; ++n) *reinterpret_cast<float2*>(table[i] + t0 + n * 8) = make_float2(s[n][2 * i], s[n][2 * i + 1]);
+            }
+        }
         float base[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
@@ -655,6 +690,7 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
                 s[n][i] = exp2_fast(s[n][i] - base[i >> 1]);
                 total[i >> 1] += s[n][i];
             }
+        if constexpr (PART == kScores) continue;
 #pragma unroll
         for (int k = 0; k < NT / 2; ++k) {
             uint32_t hi[4], lo[4];
@@ -682,14 +718,155 @@ __global__ void __launch_bounds__(128) chunk_mma_kernel(const __grid_constant__ 
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         int position, head;
-        if (!row_of(row_base + (lane >> 2) + i * 8, position, head)) continue;
-        const int row = first + position;
+        if (!tile.row(row_base + (lane >> 2) + i * 8, position, head)) continue;
+        if constexpr (PART == kScores) {
+            float* ml = a.table_ml + (table_row(a, tile.sequence, position) * p.heads + head) * 2;
+            if ((lane & 3) == 0) { ml[0] = top[i]; ml[1] = total[i]; }
+            continue;
+        }
+        const int row = tile.first + position;
         const float factor = head_gate(p, row, head) * denominator_factor(p, head, top[i], total[i]);
 #pragma unroll
         for (int v = 0; v < VT; ++v) {
             const int column = v * 8 + (lane & 3) * 2;
             if (column < p.vdim) store_pair(a, row, head, column, o[v][2 * i] * factor, o[v][2 * i + 1] * factor);
         }
+    }
+}
+
+// Longer passes of mixed heads: the values under the packed weights of the table.  The tiles are those of the scores.
+template <int DV> struct ValueShape {
+    static constexpr int kKeys = 64, kWeightBytes = 64 * (kKeys + 4) * 4, kStageBytes = kWeightBytes + kKeys * DV * 2, kSmem = 2 * kStageBytes;
+};
+template <int DV> __global__ void __launch_bounds__(128) talk_values_kernel(const __grid_constant__ ChunkAttention a) {
+    using S = ValueShape<DV>;
+    constexpr int kPitch = S::kKeys + 4;   // words between the rows of a weight tile
+    extern __shared__ __align__(128) uint8_t smem[];
+    const ChunkParams& p = a.p;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const TileRows tile(a, a.first_sequence + blockIdx.y, blockIdx.z, tile_begin(a));
+    if (tile.offset >= tile.count) return;
+    const int tiles = (tile.keys + S::kKeys - 1) / S::kKeys;
+    auto fetch = [&](int t, int stage) {
+        const uint32_t at = smem_u32(smem + stage * S::kStageBytes);
+#pragma unroll 4
+        for (int c = threadIdx.x; c < 64 * (S::kKeys / 4); c += 128) {
+            const int m = c / (S::kKeys / 4), piece = c % (S::kKeys / 4);
+            int position, head;
+            const bool live = tile.row(m, position, head);
+            const float* from = live ? a.table + (table_row(a, tile.sequence, position) * p.heads + head) * a.pitch + t * S::kKeys + piece * 4 : a.table;
+            copy_async_16(at + (m * kPitch + piece * 4) * 4, from, live);
+        }
+        tile.fetch<DV, S::kKeys>(at + S::kWeightBytes, t * S::kKeys, p.value_cache, p.value, p.vdim);
+    };
+    fetch(0, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    constexpr int VT = DV / 8;
+    float o[VT][4];
+#pragma unroll
+    for (int v = 0; v < VT; ++v)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) o[v][i] = 0.0f;
+    for (int t = 0; t < tiles; ++t) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();   // the tile is here, and everyone is done with the stage that is filled next
+        if (t + 1 < tiles) fetch(t + 1, (t + 1) & 1);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        const uint8_t* stage = smem + (t & 1) * S::kStageBytes;
+        const uint32_t value_tile = smem_u32(stage + S::kWeightBytes);
+        const uint32_t* weights = reinterpret_cast<const uint32_t*>(stage) + (warp * 16 + (lane >> 2)) * kPitch + (lane & 3) * 2;
+#pragma unroll
+        for (int k = 0; k < S::kKeys / 16; ++k) {
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int part = 0; part < 4; ++part)
+                unpack_weights(*reinterpret_cast<const uint2*>(weights + (part & 1) * 8 * kPitch + k * 16 + (part >> 1) * 8), hi[part], lo[part]);
+#pragma unroll
+            for (int v = 0; v < VT; v += 2) {
+                uint32_t b[4];
+                ldsm_x4_trans(b, value_tile + tile_offset<DV>(k * 16 + (lane & 15), v + (lane >> 4)));
+                mma_16816(o[v], hi, b[0], b[1]);
+                mma_16816(o[v + 1], hi, b[2], b[3]);
+                mma_16816(o[v], lo, b[0], b[1]);
+                mma_16816(o[v + 1], lo, b[2], b[3]);
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        int position, head;
+        if (!tile.row(warp * 16 + (lane >> 2) + i * 8, position, head)) continue;
+        const int row = tile.first + position;
+        const float factor = head_gate(p, row, head);
+#pragma unroll
+        for (int v = 0; v < VT; ++v) {
+            const int column = v * 8 + (lane & 3) * 2;
+            if (column < p.vdim) store_pair(a, row, head, column, o[v][2 * i] * factor, o[v][2 * i + 1] * factor);
+        }
+    }
+}
+
+// Between the two: scores -> softmax weights, mixed over the heads -> packed bf16 planes, in place.  grid (blocks of keys, positions,
+// sequences); two adjacent keys per thread, HEADS >= heads of them in registers.
+constexpr int kMixThreads = 128;
+template <int HEADS> __global__ void __launch_bounds__(kMixThreads) talk_mix_kernel(const __grid_constant__ ChunkAttention a) {
+    extern __shared__ __align__(16) float talk[];   // [heads][HEADS], columns past the heads zero
+    __shared__ float top[HEADS], inverse[HEADS];
+    const ChunkParams& p = a.p;
+    const int H = p.heads;
+    for (int c = threadIdx.x; c < H * HEADS; c += kMixThreads) talk[c] = c % HEADS < H ? __ldg(p.talk + (c / HEADS) * H + c % HEADS) : 0.0f;
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const int sequence = a.first_sequence + blockIdx.z, position = a.begin + blockIdx.y;
+    const int count = __ldg(a.rows.first + sequence + 1) - __ldg(a.rows.first + sequence);
+    if (position >= count) return;
+    int keys;
+    if (a.step) keys = p.entries_seen(a.rows.lengths[__ldg(a.rows.slot + sequence)]);
+    else keys = TileRows(a, sequence, 0, a.begin + (position - a.begin) / a.positions_per_tile * a.positions_per_tile).keys;
+    keys = (keys + 63) / 64 * 64;   // (the tables are written in whole tiles)
+    if (static_cast<int>(blockIdx.x) * kMixThreads * 2 >= keys) return;
+    const int64_t row = table_row(a, sequence, position) * H;
+    for (int h = threadIdx.x; h < HEADS; h += kMixThreads) {
+        float high = -INFINITY, total = 0.0f;
+        if (h < H) {
+            const float* ml = a.table_ml + (row + h) * a.splits * 2;
+            for (int s = 0; s < a.splits; ++s) high = fmaxf(high, ml[s * 2]);
+            for (int s = 0; s < a.splits; ++s) total = fmaf(ml[s * 2 + 1], exp2_fast(ml[s * 2] - high), total);
+        }
+        top[h] = h < H ? high : 0.0f;
+        inverse[h] = h < H ? 1.0f / total : 0.0f;
+    }
+    __syncthreads();
+    const int n = (blockIdx.x * kMixThreads + threadIdx.x) * 2;
+    if (n >= keys) return;
+    float* at = a.table + row * a.pitch + n;
+    float2 w[HEADS];
+#pragma unroll
+    for (int h = 0; h < HEADS; ++h) {
+        w[h] = h < H ? *reinterpret_cast<const float2*>(at + h * a.pitch) : make_float2(-INFINITY, -INFINITY);
+    }
+#pragma unroll
+    for (int h = 0; h < HEADS; ++h) {
+        const float high = top[h], factor = inverse[h];
+        w[h] = make_float2(exp2_fast(w[h].x - high) * factor, exp2_fast(w[h].y - high) * factor);
+    }
+    for (int h = 0; h < H; ++h) {
+        float2 sum = make_float2(0.0f, 0.0f);
+        const float4* t = reinterpret_cast<const float4*>(talk + h * HEADS);
+#pragma unroll
+        for (int g = 0; g < HEADS / 4; ++g) {
+            const float4 v = t[g];
+            sum.x = fmaf(v.x, w[4 * g].x, sum.x); sum.y = fmaf(v.x, w[4 * g].y, sum.y);
+            sum.x = fmaf(v.y, w[4 * g + 1].x, sum.x); sum.y = fmaf(v.y, w[4 * g + 1].y, sum.y);
+            sum.x = fmaf(v.z, w[4 * g + 2].x, sum.x); sum.y = fmaf(v.z, w[4 * g + 2].y, sum.y);
+            sum.x = fmaf(v.w, w[4 * g + 3].x, sum.x); sum.y = fmaf(v.w, w[4 * g + 3].y, sum.y);
+        }
+        uint32_t hi, lo;
+        pack_planes(sum.x, sum.y, hi, lo);
+        *reinterpret_cast<uint2*>(at + h * a.pitch) = make_uint2(__byte_perm(hi, lo, 0x5410), __byte_perm(hi, lo, 0x7632));
     }
 }
 
@@ -710,10 +887,11 @@ __device__ __forceinline__ void step_consumers_sync() { asm volatile("bar.sync 1
 // CTAs that share an SM.
 constexpr int step_residents(int columns) { return columns <= 128 ? 3 : columns <= 256 ? 2 : 1; }
 
-template <int DK, int DV>
+// PART kScores leaves a tile's scores and their largest and sum in the tables, kValues takes packed weights from there.
+template <int DK, int DV, int PART>
 __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_step_kernel(const __grid_constant__ ChunkAttention a, const __grid_constant__ CUtensorMap key_map,
                                                                  const __grid_constant__ CUtensorMap value_map) {
-    constexpr int kKeyBoxes = DK / 64, kValueBoxes = DV / 64, kStageBytes = (kKeyBoxes + kValueBoxes) * kStepBoxBytes;
+    constexpr int kKeyBoxes = PART == kValues ? 0 : DK / 64, kValueBoxes = PART == kScores ? 0 : DV / 64, kStageBytes = (kKeyBoxes + kValueBoxes) * kStepBoxBytes;
     extern __shared__ __align__(128) uint8_t smem[];
     const ChunkParams& p = a.p;
     uint8_t* ring = smem + ((1024u - (smem_u32(smem) & 1023u)) & 1023u);   // swizzled boxes start on 1024-byte boundaries
@@ -799,7 +977,7 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
         const int head0 = now.kv_head * p.group + now.head_tile * a.heads_per_tile;
         // queries as fragments: rows are the heads of the token
         uint32_t q[DK / 16][4];
-        {
+        if constexpr (PART != kValues) {
             const auto* query = static_cast<const __nv_bfloat16*>(p.query) + (static_cast<int64_t>(now.sequence) * p.heads + head0) * p.dim;
 #pragma unroll
             for (int k = 0; k < DK / 16; ++k)
@@ -820,6 +998,13 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
 #pragma unroll
             for (int i = 0; i < 4; ++i) o[v][i] = 0.0f;
         float top[2] = {-INFINITY, -INFINITY}, total[2] = {0.0f, 0.0f};
+        float* table[2] = {nullptr, nullptr};
+        if constexpr (PART != kWhole) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                if ((lane >> 2) + i * 8 < heads_here)
+                    table[i] = a.table + (static_cast<int64_t>(now.sequence) * p.heads + head0 + (lane >> 2) + i * 8) * a.pitch + own + (lane & 3) * 2;
+        }
         for (int t = tile0; t < tile1; ++t) {
             if (!mbar_wait(&full[stage], phase)) {
                 if (lane == 0) atomicExch(a.status, B200_DEVICE_TIMEOUT);
@@ -828,7 +1013,22 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
             }
             const uint32_t key_at = smem_u32(ring + stage * kStageBytes), value_at = key_at + kKeyBoxes * kStepBoxBytes;
             const int seen = keys - t * kStepKeys - own;   // keys of this warp's sixteen that exist
+            if (PART == kScores && seen <= 0) {
+#pragma unroll
+                for (int i = 0; i < 2; ++i)
+                    if (table[i]) {
+                        *reinterpret_cast<float2*>(table[i] + t * kStepKeys) = make_float2(-INFINITY, -INFINITY);
+                        *reinterpret_cast<float2*>(table[i] + t * kStepKeys + 8) = make_float2(-INFINITY, -INFINITY);
+                    }
+            }
             if (seen > 0) {
+                uint32_t hi[4], lo[4];
+                if constexpr (PART == kValues) {
+#pragma unroll
+                    for (int part = 0; part < 4; ++part)
+                        unpack_weights(table[part & 1] ? __ldcg(reinterpret_cast<const uint2*>(table[part & 1] + t * kStepKeys + (part >> 1) * 8)) : make_uint2(0u, 0u),
+                                       hi[part], lo[part]);
+                } else {
                 float s[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
 #pragma unroll
                 for (int k = 0; k < DK / 16; ++k) {
@@ -846,6 +1046,14 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
                         s[n][i] = n * 8 + (lane & 3) * 2 + (i & 1) < seen ? score : -INFINITY;
                         high[i >> 1] = fmaxf(high[i >> 1], s[n][i]);
                     }
+                if constexpr (PART == kScores) {
+#pragma unroll
+                    for (int i = 0; i < 2; ++i)
+                        if (table[i]) {
+                            *reinterpret_cast<float2*>(table[i] + t * kStepKeys) = make_float2(s[0][2 * i], s[0][2 * i + 1]);
+                            *reinterpret_cast<float2*>(table[i] + t * kStepKeys + 8) = make_float2(s[1][2 * i], s[1][2 * i + 1]);
+                        }
+                }
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
                     high[i] = fmaxf(high[i], __shfl_xor_sync(0xffffffffu, high[i], 1));
@@ -864,11 +1072,11 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
                         s[n][i] = exp2_fast(s[n][i] - base[i >> 1]);
                         total[i >> 1] += s[n][i];
                     }
-                uint32_t hi[4], lo[4];
                 pack_planes(s[0][0], s[0][1], hi[0], lo[0]);
                 pack_planes(s[0][2], s[0][3], hi[1], lo[1]);
                 pack_planes(s[1][0], s[1][1], hi[2], lo[2]);
                 pack_planes(s[1][2], s[1][3], hi[3], lo[3]);
+                }
                 // rows past the last key hold what the memory held: they must not reach the products, not even times zero
                 uint32_t live[2] = {0xffffffffu, 0xffffffffu};
                 if (seen < 16) {
@@ -879,7 +1087,7 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
                     }
                 }
 #pragma unroll
-                for (int v = 0; v < VT; v += 2) {
+                for (int v = 0; PART != kScores && v < VT; v += 2) {
                     uint32_t b[4];
                     ldsm_x4_trans(b, value_at + box_offset(own + (lane & 15), v + (lane >> 4)));
                     b[0] &= live[0]; b[1] &= live[1]; b[2] &= live[0]; b[3] &= live[1];
@@ -907,13 +1115,26 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
             if (m >= heads_here) continue;
             const int at = warp * a.heads_per_tile + m;
 #pragma unroll
-            for (int v = 0; v < VT; ++v)
+            for (int v = 0; PART != kScores && v < VT; ++v)
                 *reinterpret_cast<float2*>(merge + at * DV + v * 8 + (lane & 3) * 2) = make_float2(o[v][2 * i], o[v][2 * i + 1]);
             if ((lane & 3) == 0) { merge_ml[at * 2] = top[i]; merge_ml[at * 2 + 1] = total[i]; }
         }
         step_consumers_sync();
         if (*static_cast<volatile int*>(gave_up)) return;   // a tile never arrived: every consumer leaves here
-        for (int c = threadIdx.x; c < heads_here * (DV / 2); c += kStepConsumers) {
+        if constexpr (PART == kScores) {
+            if (threadIdx.x < heads_here) {
+                float best = -INFINITY, sum = 0.0f;
+                for (int w = 0; w < 4; ++w) best = fmaxf(best, merge_ml[(w * a.heads_per_tile + threadIdx.x) * 2]);
+                for (int w = 0; w < 4; ++w) {
+                    const float* ml = merge_ml + (w * a.heads_per_tile + threadIdx.x) * 2;
+                    sum = fmaf(ml[1], exp2_fast(ml[0] - (best == -INFINITY ? 0.0f : best)), sum);
+                }
+                float* to = a.table_ml + ((static_cast<int64_t>(now.sequence) * p.heads + head0 + threadIdx.x) * a.splits + now.split) * 2;
+                to[0] = best;
+                to[1] = sum;
+            }
+        }
+        for (int c = threadIdx.x; PART != kScores && c < heads_here * (DV / 2); c += kStepConsumers) {
             const int m = c / (DV / 2), column = (c % (DV / 2)) * 2;
             if (column >= p.vdim) continue;
             float best = -INFINITY;
@@ -924,15 +1145,19 @@ __global__ void __launch_bounds__(kStepThreads, step_residents(DK + DV)) chunk_s
 #pragma unroll
             for (int w = 0; w < 4; ++w) {
                 const int at = w * a.heads_per_tile + m;
-                const float factor = exp2_fast(merge_ml[at * 2] - from);
+                const float factor = PART == kValues ? 1.0f : exp2_fast(merge_ml[at * 2] - from);
                 const float2 v = *reinterpret_cast<const float2*>(merge + at * DV + column);
                 x = fmaf(v.x, factor, x);
                 y = fmaf(v.y, factor, y);
                 sum = fmaf(merge_ml[at * 2 + 1], factor, sum);
             }
             const int head = head0 + m;
+            if constexpr (PART == kValues) {   // the weights are finished: a share counts as it is
+                best = 0.0f;
+                sum = now.split == 0 ? 1.0f : 0.0f;
+            }
             if (a.splits == 1) {
-                const float factor = gates[m] * denominator_factor(p, head, from, sum);
+                const float factor = PART == kValues ? gates[m] : gates[m] * denominator_factor(p, head, from, sum);
                 store_pair(a, now.sequence, head, column, x * factor, y * factor);
             } else {
                 const int64_t part = (static_cast<int64_t>(now.sequence) * p.heads + head) * a.splits + now.split;
@@ -1131,12 +1356,31 @@ int chunk_splits(const ChunkParams& p, int sequences, int max_length, int sms) {
     return std::max(1, std::min({(2 * sms + items - 1) / items, tiles / 2, 32}));
 }
 
-template <int DK, int DV> int launch_chunk_mma(const ChunkAttention& a, cudaStream_t stream) {
-    auto kernel = chunk_mma_kernel<DK, DV>;
-    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkShape<DK, DV>::kSmem));
-    const dim3 grid(static_cast<unsigned>((a.rows.max_count + a.positions_per_tile - 1) / a.positions_per_tile), static_cast<unsigned>(a.rows.sequences),
-                    static_cast<unsigned>(a.p.kv_heads * a.head_tiles));
-    return cuda_status(launch_dependent(kernel, grid, dim3(128), ChunkShape<DK, DV>::kSmem, stream, a), "chunk_mma_kernel launch");
+// grid of the tiles of the positions [begin, begin + span) of `sequences` sequences
+dim3 tile_grid(const ChunkAttention& a, int sequences) {
+    return dim3(static_cast<unsigned>((a.span + a.positions_per_tile - 1) / a.positions_per_tile), static_cast<unsigned>(sequences),
+                static_cast<unsigned>(a.p.kv_heads * a.head_tiles));
+}
+template <int DK, int DV, int PART = kWhole> int launch_chunk_mma(const ChunkAttention& a, int sequences, cudaStream_t stream) {
+    constexpr int kSmem = ChunkShape<DK, DV, PART>::kSmem;
+    auto kernel = chunk_mma_kernel<DK, DV, PART>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    return cuda_status(launch_dependent(kernel, tile_grid(a, sequences), dim3(128), kSmem, stream, a), "chunk_mma_kernel launch");
+}
+template <int DV> int launch_talk_values(const ChunkAttention& a, int sequences, cudaStream_t stream) {
+    auto kernel = talk_values_kernel<DV>;
+    B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ValueShape<DV>::kSmem));
+    return cuda_status(launch_dependent(kernel, tile_grid(a, sequences), dim3(128), ValueShape<DV>::kSmem, stream, a), "talk_values_kernel launch");
+}
+int launch_talk_mix(const ChunkAttention& a, int sequences, cudaStream_t stream) {
+    auto launch = [&](auto kernel, int heads) {
+        const dim3 grid(static_cast<unsigned>((a.pitch + 2 * kMixThreads - 1) / (2 * kMixThreads)), static_cast<unsigned>(a.span), static_cast<unsigned>(sequences));
+        return cuda_status(launch_dependent(kernel, grid, dim3(kMixThreads), static_cast<size_t>(a.p.heads) * heads * 4, stream, a), "talk_mix_kernel launch");
+    };
+    if (a.p.heads <= 8) return launch(talk_mix_kernel<8>, 8);
+    if (a.p.heads <= 16) return launch(talk_mix_kernel<16>, 16);
+    if (a.p.heads <= 32) return launch(talk_mix_kernel<32>, 32);
+    return launch(talk_mix_kernel<64>, 64);
 }
 
 int encode_slots(CUtensorMap* map, const void* base, int64_t rows, int columns) {
@@ -1153,7 +1397,7 @@ int encode_slots(CUtensorMap* map, const void* base, int64_t rows, int columns) 
     return B200_OK;
 }
 
-template <int DK, int DV> int launch_chunk_step(ChunkAttention a, int sms, cudaStream_t stream) {
+template <int DK, int DV, int PART = kWhole> int launch_chunk_step(ChunkAttention a, int sms, cudaStream_t stream) {
     const ChunkParams& p = a.p;
     alignas(64) CUtensorMap keys, values;
     const int64_t rows = static_cast<int64_t>(p.slots) * p.kv_heads * p.entries;
@@ -1161,12 +1405,12 @@ template <int DK, int DV> int launch_chunk_step(ChunkAttention a, int sms, cudaS
     int status = encode_slots(&keys, p.key_cache, rows, p.dim);
     if (status == B200_OK) status = encode_slots(&values, p.value_cache, rows, p.vdim);
     if (status != B200_OK) return status;
-    const int stage_bytes = (DK + DV) / 64 * kStepBoxBytes, merge_bytes = 4 * a.heads_per_tile * (DV + 2) * 4, fixed = 1024 + kStepControlBytes + merge_bytes;
+    const int stage_bytes = ((PART == kValues ? 0 : DK) + (PART == kScores ? 0 : DV)) / 64 * kStepBoxBytes, merge_bytes = 4 * a.heads_per_tile * (DV + 2) * 4, fixed = 1024 + kStepControlBytes + merge_bytes;
     int resident = step_residents(DK + DV) + 1;
     do a.stages = std::min((kSmSmem / --resident - 1024 - fixed) / stage_bytes, kMaxStages);
     while (a.stages < 2 && resident > 1);
     const int smem = fixed + a.stages * stage_bytes;
-    auto kernel = chunk_step_kernel<DK, DV>;
+    auto kernel = chunk_step_kernel<DK, DV, PART>;
     B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     const int64_t items = static_cast<int64_t>(a.rows.sequences) * p.kv_heads * a.head_tiles * a.splits;
     if (items > INT32_MAX) { set_error("grouped attention: too many sequences and heads in one pass"); return B200_UNSUPPORTED; }
@@ -1183,6 +1427,80 @@ template <class Launch> int pick_chunk_sizes(const ChunkParams& p, Launch&& laun
     if (p.dim <= 128 && p.vdim <= 128) return launch(integral_constant<int, 128>{}, integral_constant<int, 128>{});
     if (p.dim <= 192 && p.vdim <= 128) return launch(integral_constant<int, 192>{}, integral_constant<int, 128>{});
     return launch(integral_constant<int, 256>{}, integral_constant<int, 256>{});
+}
+
+// The smallest compiled size that holds one.
+template <class Launch> int pick_head_size(int size, Launch&& launch) {
+    using std::integral_constant;
+    if (size <= 64) return launch(integral_constant<int, 64>{});
+    if (size <= 128) return launch(integral_constant<int, 128>{});
+    return launch(integral_constant<int, 256>{});
+}
+
+// Mixed heads: positions and sequences whose tables are filled at a time.  Longer passes go in portions whose tables stay in L2.
+constexpr size_t kTableBytes = size_t{72} << 20;
+constexpr int kMostMixedHeads = 64;
+struct TalkPlan { int64_t pitch; int span, sequences; };
+TalkPlan talk_plan(const ChunkParams& p, int sequences, int max_count, int max_length) {
+    const bool step = max_count == 1;
+    const int tile = step ? 1 : 64 / std::min(p.group, 64);
+    int64_t keys = max_length;
+    if (p.window > 0) keys = std::min<int64_t>(keys, static_cast<int64_t>(p.window) + tile - 1) + (p.pool > 0 ? max_length / p.pool : p.keep);
+    TalkPlan plan;
+    plan.pitch = (keys + 63) / 64 * 64;
+    plan.span = step ? 1 : (max_count + tile - 1) / tile * tile;
+    plan.sequences = sequences;
+    if (step) return plan;
+    const size_t per_tile = static_cast<size_t>(tile) * p.heads * static_cast<size_t>(plan.pitch) * 4, tiles = std::max<size_t>(1, kTableBytes / per_tile);
+    plan.sequences = static_cast<int>(std::min<size_t>(static_cast<size_t>(sequences), tiles));
+    plan.span = static_cast<int>(std::min<size_t>(static_cast<size_t>(plan.span), tiles / static_cast<size_t>(plan.sequences) * static_cast<size_t>(tile)));
+    return plan;
+}
+size_t talk_table_words(const ChunkParams& p, const TalkPlan& plan) { return static_cast<size_t>(plan.sequences) * plan.span * p.heads * static_cast<size_t>(plan.pitch); }
+size_t talk_scratch_bytes(const ChunkParams& p, const TalkPlan& plan, int splits) {
+    const size_t rows = static_cast<size_t>(plan.sequences) * plan.span * p.heads;
+    return (talk_table_words(p, plan) + rows * splits * 2 + (splits > 1 ? rows * splits * (p.vdim + 2) : 0)) * sizeof(float);
+}
+bool talk_takes_mma(const ChunkParams& p, int dtype, int64_t out_stride) {
+    return p.talk && p.heads <= kMostMixedHeads && chunk_takes_mma(p, dtype, out_stride);
+}
+
+// scores -> mixed softmax weights -> values
+int launch_talk(ChunkAttention a, int max_length, void* scratch, size_t scratch_bytes, int sms, cudaStream_t stream) {
+    const ChunkParams& p = a.p;
+    const TalkPlan plan = talk_plan(p, a.rows.sequences, a.rows.max_count, max_length);
+    const size_t need = talk_scratch_bytes(p, plan, a.splits), rows = static_cast<size_t>(plan.sequences) * plan.span * p.heads;
+    if (scratch_bytes < need || !scratch || (reinterpret_cast<uintptr_t>(scratch) & 15)) {
+        set_error("b200_chunk_attention: scratch of %zu bytes, %zu needed", scratch_bytes, need);
+        return B200_BAD_ARGUMENT;
+    }
+    a.pitch = plan.pitch;
+    a.table = static_cast<float*>(scratch);
+    a.table_ml = a.table + talk_table_words(p, plan);
+    a.partial = a.table_ml + rows * a.splits * 2;
+    a.partial_ml = a.partial + (a.splits > 1 ? rows * a.splits * p.vdim : 0);
+    if (a.step) {
+        a.span = 1;
+        int status = pick_head_size(p.dim, [&](auto dk) { return launch_chunk_step<decltype(dk)::value, 64, kScores>(a, sms, stream); });
+        if (status == B200_OK) status = launch_talk_mix(a, a.rows.sequences, stream);
+        if (status == B200_OK) status = pick_head_size(p.vdim, [&](auto dv) { return launch_chunk_step<64, decltype(dv)::value, kValues>(a, sms, stream); });
+        if (status == B200_OK && a.splits > 1)
+            status = cuda_status(launch_dependent(chunk_combine_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(64), 0, stream, a),
+                                 "chunk_combine_kernel launch");
+        return status;
+    }
+    for (int sequence = 0; sequence < a.rows.sequences; sequence += plan.sequences)
+        for (int begin = 0; begin < a.rows.max_count; begin += plan.span) {
+            const int sequences = std::min(plan.sequences, a.rows.sequences - sequence);
+            a.first_sequence = sequence;
+            a.begin = begin;
+            a.span = plan.span;
+            int status = pick_head_size(p.dim, [&](auto dk) { return launch_chunk_mma<decltype(dk)::value, 64, kScores>(a, sequences, stream); });
+            if (status == B200_OK) status = launch_talk_mix(a, sequences, stream);
+            if (status == B200_OK) status = pick_head_size(p.vdim, [&](auto dv) { return launch_talk_values<decltype(dv)::value>(a, sequences, stream); });
+            if (status != B200_OK) return status;
+        }
+    return B200_OK;
 }
 
 }  // namespace
@@ -1237,10 +1555,11 @@ extern "C" int b200_chunk_prepare(const b200_chunk_args* args, const b200_rows* 
 
 extern "C" size_t b200_chunk_scratch_bytes(const b200_chunk_args* args, int64_t rows, int32_t sequences, int32_t max_count, int32_t max_length) {
     ChunkParams p;
-    if (!chunk_params(args, p) || rows <= 0 || sequences <= 0 || max_count != 1) return 0;
+    if (!chunk_params(args, p) || rows <= 0 || sequences <= 0 || (max_count != 1 && !p.talk)) return 0;
     int device = 0;
     if (cudaGetDevice(&device) != cudaSuccess) { cudaGetLastError(); device = -1; }
-    const int splits = chunk_splits(p, sequences, max_length, sm_count(device));
+    const int splits = max_count == 1 ? chunk_splits(p, sequences, max_length, sm_count(device)) : 1;
+    if (p.talk) return p.heads <= kMostMixedHeads ? talk_scratch_bytes(p, talk_plan(p, sequences, max_count, max_length), splits) : 0;
     return splits > 1 ? static_cast<size_t>(rows) * p.heads * splits * (p.vdim + 2) * sizeof(float) : 0;
 }
 
@@ -1266,7 +1585,7 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
         status = cuda_status(launch_dependent(pool, grid, dim3(128), 0, s, p, a.rows), "chunk_pool_kernel launch");
         if (status != B200_OK) return status;
     }
-    if (p.talk) {
+    if (p.talk && !talk_takes_mma(p, args->dtype, out_stride)) {
         const size_t smem = talk_generic_bytes(p);
         auto kernel = args->dtype == B200_BF16 ? talk_generic_kernel<__nv_bfloat16> : talk_generic_kernel<float>;
         if (smem > 220 * 1024) { set_error("mixed heads: %d heads of %d and %d are too large", p.heads, p.dim, p.vdim); return B200_UNSUPPORTED; }
@@ -1281,7 +1600,7 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
         a.positions_per_tile = a.step ? 1 : most / a.heads_per_tile;
         if (a.step) {
             a.splits = chunk_splits(p, a.rows.sequences, max_length, sm_count(device));
-            const size_t need = a.splits > 1 ? static_cast<size_t>(a.rows.rows) * p.heads * a.splits * (p.vdim + 2) * sizeof(float) : 0;
+            const size_t need = a.splits > 1 && !p.talk ? static_cast<size_t>(a.rows.rows) * p.heads * a.splits * (p.vdim + 2) * sizeof(float) : 0;
             if (scratch_bytes < need || (need && !scratch)) { set_error("b200_chunk_attention: scratch of %zu bytes, %zu needed", scratch_bytes, need); return B200_BAD_ARGUMENT; }
             a.partial = static_cast<float*>(scratch);
             a.partial_ml = a.partial + static_cast<int64_t>(a.rows.rows) * p.heads * a.splits * p.vdim;
@@ -1293,10 +1612,12 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
         a.status = device_status_word(device);
         if (!a.status) { set_error("the device status word could not be allocated"); return B200_NO_DEVICE; }
         const int sms = sm_count(device);
-        status = pick_chunk_sizes(p, [&](auto dk, auto dv) {
-            return a.step ? launch_chunk_step<decltype(dk)::value, decltype(dv)::value>(a, sms, s) : launch_chunk_mma<decltype(dk)::value, decltype(dv)::value>(a, s);
+        a.span = a.rows.max_count;
+        status = p.talk ? launch_talk(a, max_length, scratch, scratch_bytes, sms, s) : pick_chunk_sizes(p, [&](auto dk, auto dv) {
+            constexpr int kDim = decltype(dk)::value, kValueDim = decltype(dv)::value;
+            return a.step ? launch_chunk_step<kDim, kValueDim>(a, sms, s) : launch_chunk_mma<kDim, kValueDim>(a, a.rows.sequences, s);
         });
-        if (status == B200_OK && a.splits > 1)
+        if (status == B200_OK && a.splits > 1 && !p.talk)
             status = cuda_status(launch_dependent(chunk_combine_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)), dim3(64), 0, s, a),
                                  "chunk_combine_kernel launch");
     } else {
@@ -1316,6 +1637,7 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
 extern "C" const char* b200_chunk_attention_kernel(const b200_chunk_args* args, int32_t max_count, int64_t out_stride) {
     ChunkParams p;
     if (!chunk_params(args, p)) return "";
+    if (p.talk) return !talk_takes_mma(p, args->dtype, out_stride) ? "talk_generic_kernel" : max_count == 1 ? "chunk_step_kernel" : "talk_values_kernel";
     if (!chunk_takes_mma(p, args->dtype, out_stride)) return "chunk_generic_kernel";
     return max_count == 1 ? "chunk_step_kernel" : "chunk_mma_kernel";
 }
