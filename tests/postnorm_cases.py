@@ -45,13 +45,13 @@ CASES = {
     # sizes equal or one
     "ones": config(16, [delta(1, 1, 16, 16, 1, moe(1, 1, 16)), pooled(1, 1, 16, 16, 1, 1, moe(1, 1, 16)), mixing(1, 1, 16, 16, 1, 1, moe(1, 1, 16))], vocab=16, factor=1.0),
     # nothing a multiple of 8: the kernels without vector loads; blocks longer than the window
-    "odd": config(36, [pooled(3, 1, 10, 14, 7, 11, moe(5, 2, 21), dims=6), delta(6, 3, 9, 7, 5, moe(3, 2, 13)), mixing(3, 3, 14, 6, 5, 9, moe(4, 4, 9), dims=2, factor=3.0),
-                       delta(5, 5, 7, 9, 2, None)], vocab=53, eps=1e-3, factor=1.3),
+    "odd": config(36, [pooled(3, 1, 10, 14, 7, 11, moe(5, 2, 21), dims=6), delta(6, 3, 9, 7, 5, moe(3, 3, 13)), mixing(3, 3, 14, 6, 5, 9, moe(4, 4, 9), dims=2, factor=3.0),
+                       delta(5, 5, 7, 9, 2, None)], vocab=53, eps=0.03, factor=0.9),
     # layers without a feed-forward, every expert chosen, windows longer than most sequences, no kept tokens
     "plain": config(72, [mixing(5, 5, 40, 72, 200, 0, None), pooled(10, 5, 40, 72, 128, 64, moe(4, 4, 56)), delta(2, 1, 40, 8, 4, None), mixing(10, 5, 40, 24, 64, 70, moe(3, 3, 40), factor=8.0)],
                     vocab=200, weights_of=((4, 1),)),
     # heads past a step's tile and past the registers of the mixing kernel, many experts, larger states
-    "wide": config(128, [pooled(40, 2, 16, 16, 65, 16, moe(64, 3, 64)), mixing(72, 2, 8, 8, 40, 5, moe(24, 6, 32)), delta(2, 2, 130, 64, 4, moe(16, 8, 32)), mixing(20, 1, 128, 64, 48, 2, None)],
+    "wide": config(128, [pooled(40, 2, 16, 16, 65, 16, moe(40, 1, 64)), mixing(72, 2, 8, 8, 40, 5, moe(9, 9, 32)), delta(2, 2, 130, 64, 4, moe(12, 2, 32)), mixing(20, 1, 128, 64, 48, 2, None)],
                    vocab=304),
     # the larger head sizes of the tensor-core attention, a state beyond the narrow scan
     "deep": config(96, [mixing(2, 1, 192, 128, 30, 4, moe(8, 1, 48), dims=32), pooled(2, 2, 256, 256, 24, 5, None), delta(3, 1, 264, 128, 4, moe(6, 2, 40)), pooled(3, 1, 72, 96, 63, 2, None, dims=10)],
@@ -91,8 +91,8 @@ def weight_shapes(c):
 
 
 def make_weights(c, seed=0):
-    """bf16-representable f32 weights by name: rows of about unit gain, norm weights away from one, routers with clear choices, queries
-    that tell keys apart, decays that remember."""
+    """bf16-representable f32 weights by name: rows of about unit gain, norm weights away from one, routers with clear choices, decays
+    that remember."""
     rng = np.random.default_rng(seed)
     out = {}
     for name, shape in weight_shapes(c).items():
@@ -108,7 +108,7 @@ def make_weights(c, seed=0):
         elif leaf == "conv":
             w = rng.normal(0, 0.7, shape)
         elif len(shape) == 1:
-            w = rng.uniform(0.6, 1.4, shape) * (2.0 if name.endswith("q.norm") else 1.0)
+            w = rng.uniform(0.6, 1.4, shape)
         elif name == "embed":
             w = rng.normal(0, 1.0, shape)
         else:
@@ -117,10 +117,10 @@ def make_weights(c, seed=0):
     return out
 
 
-def decided_tokens(c, weights, count, seed=1, margin=0.02):
+def decided_tokens(c, weights, count, seed=1, margin=0.06):
     """Random tokens on which no router's choice is a close call, which rounding could turn either way: the first of a few draws."""
     best, at = None, -1.0
-    for draw in range(30):
+    for draw in range(40):
         ids = tokens(c, count, seed=seed + 1000 * draw)
         calls = [np.inf]
         postnorm_oracle.forward(c, weights, ids, calls=calls)

@@ -123,7 +123,7 @@ class Windowed:
 
 
 WINDOWS = [dict(kind=1, heads=4, kv_heads=2, dim=16, vdim=24, size=40, pool=8), dict(kind=1, heads=3, kv_heads=1, dim=10, vdim=14, size=9, pool=13),
-           dict(kind=1, heads=40, kv_heads=1, dim=96, vdim=96, size=65, pool=3), dict(kind=1, heads=2, kv_heads=2, dim=256, vdim=256, size=64, pool=64),
+           dict(kind=1, heads=40, kv_heads=1, dim=96, vdim=96, size=65, pool=3), dict(kind=1, heads=2, kv_heads=2, dim=256, vdim=256, size=64, pool=64, scale=0.1),
            dict(kind=1, heads=6, kv_heads=2, dim=20, vdim=12, size=1, pool=1), dict(kind=1, heads=2, kv_heads=1, dim=64, vdim=64, size=127, pool=5),
            dict(kind=1, heads=2, kv_heads=1, dim=64, vdim=128, size=50, pool=0), dict(kind=1, heads=2, kv_heads=1, dim=64, vdim=64, size=1000, pool=5),
            dict(kind=2, heads=4, kv_heads=2, dim=24, vdim=16, size=40, keep=5, factor=3.0), dict(kind=2, heads=3, kv_heads=3, dim=10, vdim=14, size=6, keep=11),
@@ -187,6 +187,8 @@ def test_one_key_stands_out(size, pool, keep, heads, kv_heads, dtype):
     want = k.want(rows)
     # every key that is answered or not shows: moving the window by one, or leaving out a kept token, changes answers a lot
     for planted in (dict(size=size - 1), dict(size=size + 1), *([dict(keep=keep - 1), dict(keep=keep + 1)] if keep else [])):
+        if pool == 1:
+            break      # a block of one token is that token: the window has no edge
         kept = dict(k.n)
         k.n.update(planted)
         assert np.abs(k.want(rows) - want).max() > 0.3, planted
