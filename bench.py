@@ -9,7 +9,8 @@ and prompts are seeded synthetic data.  With N > 1 (one process per GPU under to
 are divided over the GPUs (256 / N each), weights replicated, no collective on the data path: strong scaling.
 `--workload c5` is the 8B shape with adapters, KV-head tensor parallel over the GPUs; `c2` the small decoder (replicas);
 `c3` the decode-attention microbenchmark; `linear` one projection in isolation; `hybrid`, `parallel` and `sandwich`
-prefill and decode of the hybrid, the parallel and the sandwich decoder beside the grouped-query decoder of equal size (`--size`).
+prefill and decode of the hybrid, the parallel and the sandwich decoder beside the grouped-query decoder of equal size (`--size`);
+`postnorm` the post-norm decoder beside the sandwich decoder.
 
 The printed JSON line carries the device-resident throughput (`value`: median of 5 timed rounds of K steps), the
 host-in-the-loop throughput through the C ABI (`e2e`), the roofline of the kernel class that dominates the step
@@ -673,16 +674,17 @@ def measure_model(config: dict, args, local: int, prompt_len: int, prefill_batch
 
 
 def run_hybrid(args) -> dict:
-    """The hybrid, the parallel or the sandwich decoder beside the grouped-query decoder of equal width, (active) feed-forward and number of layer runs
-    (one GPU)."""
+    """The hybrid, the parallel or the sandwich decoder beside the grouped-query decoder, or the post-norm decoder beside the sandwich decoder, of equal
+    width, (active) feed-forward and number of layer runs (one GPU)."""
     rank, world, local, dist = distributed()
     name = args.workload
     if world > 1:
         raise SystemExit(f"the {name} workload runs on one GPU")
     prompt, prefill_batch = args.prompt, 8
     sizes, make = {"hybrid": (W.HYBRID_SIZES, W.hybrid_config), "parallel": (W.PARALLEL_SIZES, W.parallel_config),
-                   "sandwich": (W.SANDWICH_SIZES, W.sandwich_config)}[name]
-    own, grouped = sizes[args.size]
+                   "sandwich": (W.SANDWICH_SIZES, W.sandwich_config), "postnorm": (W.POSTNORM_SIZES, W.postnorm_config)}[name]
+    own, closest = sizes[args.size]
+    other_name = "sandwich" if name == "postnorm" else "grouped_query"
     config = make(**own)
     batches = [args.batch] if args.batch > 0 else [1, 16, 64, 256]
     sampler = ClockSampler(local)
@@ -691,14 +693,15 @@ def run_hybrid(args) -> dict:
     ours = measure_model(config, args, local, prompt, prefill_batch, batches)
     other = None
     if not args.no_secondary:
-        other = measure_model(W.transformer_config(**grouped, context=prompt + args.steps + args.warmup + 16), args, local, prompt, prefill_batch, batches)
+        beside = W.sandwich_config(**closest) if name == "postnorm" else W.transformer_config(**closest, context=prompt + args.steps + args.warmup + 16)
+        other = measure_model(beside, args, local, prompt, prefill_batch, batches)
     clocks = sampler.stop()
     top = ours["decode"][str(max(batches))]
     return {"metric": METRIC, "value": top["tokens_per_s"], "unit": UNIT, "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
             "ms_per_step": top["ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
             "config": {"model": f"{name} {args.size}", "global_batch": max(batches), "seq_len": prompt, "parallelism": "dp1",
                        "l2": "every step streams more than L2 (weights, states, caches)"},
-            "clocks": clocks, "gpu_launches": top["launches"] * args.steps, name: ours, "grouped_query": other}
+            "clocks": clocks, "gpu_launches": top["launches"] * args.steps, name: ours, other_name: other}
 
 
 def main():
@@ -707,7 +710,7 @@ def main():
     parser.add_argument("--steps", type=int, default=64)
     parser.add_argument("--warmup", type=int, default=8)
     parser.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    parser.add_argument("--workload", default="c4", choices=["c1", "c2", "c3", "c4", "c5", "linear", "hybrid", "parallel", "sandwich"])
+    parser.add_argument("--workload", default="c4", choices=["c1", "c2", "c3", "c4", "c5", "linear", "hybrid", "parallel", "sandwich", "postnorm"])
     parser.add_argument("--activations", default="f32", choices=["f32", "bf16"],
                         help="bf16 decoders: precision of the activations between kernels in passes over more than 16 rows")
     parser.add_argument("--batch", type=int, default=0, help="decoder workloads: override the configuration's batch (e.g. c4 with 32 = one GPU's share of the 8-GPU run)")
@@ -718,13 +721,13 @@ def main():
     parser.add_argument("--cpu-steps", type=int, default=4, help="timed CPU-baseline steps of the default run")
     parser.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     parser.add_argument("--no-secondary", action="store_true", help="c4 on one GPU: skip the c3 and c2 companions of the record")
-    parser.add_argument("--size", default="2k", choices=sorted(W.HYBRID_SIZES), help="hybrid, parallel and sandwich only: layer sizes")
-    parser.add_argument("--prompt", type=int, default=1024, help="hybrid, parallel and sandwich only: prompt length")
+    parser.add_argument("--size", default="2k", choices=sorted(W.HYBRID_SIZES), help="hybrid, parallel, sandwich and postnorm only: layer sizes")
+    parser.add_argument("--prompt", type=int, default=1024, help="hybrid, parallel, sandwich and postnorm only: prompt length")
     parser.add_argument("--small", action="store_true", help="c3 only: batch 16, contexts up to 8192 (profiler captures)")
     args = parser.parse_args()
     if args.warmup < 3:
         args.warmup = 3
-    if args.workload in ("c3", "linear", "hybrid", "parallel", "sandwich"):
+    if args.workload in ("c3", "linear", "hybrid", "parallel", "sandwich", "postnorm"):
         line = {"c3": run_c3, "linear": run_linear}.get(args.workload, run_hybrid)(args)
         if line:
             print(json.dumps(line))

@@ -92,7 +92,7 @@ class ChunkArgs(C.Structure):
                 ("q_bias", C.c_void_p), ("k_bias", C.c_void_p), ("norm", C.c_int32), ("rotate_pairs", C.c_int32), ("keys_as_values", C.c_int32),
                 ("keys_elsewhere", C.c_int32), ("no_gate", C.c_int32), ("softcap", C.c_float), ("sink", C.c_void_p), ("scaled", C.c_int32), ("out_scale", C.c_float),
                 ("window", C.c_int32), ("keep", C.c_int32), ("pool", C.c_int32), ("pool_state", C.c_void_p), ("norm_values", C.c_int32), ("gate_values", C.c_int32),
-                ("talk", C.c_void_p)]
+                ("talk", C.c_void_p), ("table_bytes", C.c_int64)]
 
 
 class Units(C.Structure):

@@ -44,6 +44,7 @@ struct ChunkParams {
     float* pool_state;
     bool norm_values, gate_values;
     const float* talk;
+    size_t table_bytes;
     __host__ __device__ __forceinline__ int key_columns() const { return keys_elsewhere ? 0 : kv_heads * dim; }
     __host__ __device__ __forceinline__ int value_columns() const { return keys_elsewhere || keys_as_values ? 0 : kv_heads * vdim; }
     // Keys of the pass itself are in the slots before the attention starts.
@@ -95,7 +96,7 @@ bool chunk_params(const b200_chunk_args* a, ChunkParams& p) {
     p = ChunkParams{a->heads, a->kv_heads, a->heads / a->kv_heads, a->dim, a->vdim, a->rot_dims, a->slots, a->chunk, a->entries, a->scale, static_cast<float>(a->eps),
                     a->cosine, a->sine, a->positions, a->q_norm, a->k_norm, a->key_cache, a->value_cache, a->query, a->key, a->value, a->projected, a->stride,
                     a->q_bias, a->k_bias, a->sink, a->norm, a->rotate_pairs != 0, a->keys_as_values != 0, a->keys_elsewhere != 0, a->no_gate == 0, a->softcap,
-                    a->scaled ? a->out_scale : 1.0f, a->window, a->keep, a->pool, a->pool_state, a->norm_values != 0, a->gate_values != 0, a->talk};
+                    a->scaled ? a->out_scale : 1.0f, a->window, a->keep, a->pool, a->pool_state, a->norm_values != 0, a->gate_values != 0, a->talk, static_cast<size_t>(std::max<int64_t>(0, a->table_bytes))};
     if (p.heads * p.dim + p.key_columns() + p.value_columns() + (p.gate_values ? p.heads * p.vdim : p.gated ? p.heads : 0) > p.stride) {
         set_error("grouped attention: the projected rows are shorter than the heads");
         return false;
@@ -355,29 +356,42 @@ __global__ void __launch_bounds__(kPrepareThreads) chunk_prepare_kernel(const __
 }
 
 // Before the attention of a longer pass: the blocks of `pool` positions that the pass completes, and the sum of the one it leaves open.  grid
-// (blocks of a sequence, sequences); CTA 0 takes the first block, which earlier passes may have begun, and the open one.
-template <class T> __global__ void __launch_bounds__(128) chunk_pool_kernel(const __grid_constant__ ChunkParams p, const RowsView rows) {
+// (blocks of a sequence, sequences, column blocks), V columns per thread; CTA 0 takes the first block, which earlier passes may have begun,
+// and the open one.
+constexpr int kPoolThreads = 128;
+template <class T, int V> __global__ void __launch_bounds__(kPoolThreads) chunk_pool_kernel(const __grid_constant__ ChunkParams p, const RowsView rows) {
     grid_dependency_wait();
     grid_launch_dependents();
+    const int per_head = p.dim + p.vdim, c = (blockIdx.z * kPoolThreads + threadIdx.x) * V;
+    if (c >= p.kv_heads * per_head) return;
     const int sequence = blockIdx.y, first = __ldg(rows.first + sequence), count = __ldg(rows.first + sequence + 1) - first;
     const int slot = __ldg(rows.slot + sequence), length = rows.lengths[slot], end = length + count;
-    const int block0 = length / p.pool, block1 = (end - 1) / p.pool, per_head = p.dim + p.vdim;
+    const int block0 = length / p.pool, block1 = (end - 1) / p.pool, head = c / per_head, d = c - head * per_head;
+    const bool is_key = d < p.dim;
+    const int size = is_key ? p.dim : p.vdim, at_head = is_key ? d : d - p.dim;
+    const T* source = static_cast<const T*>(is_key ? p.key : p.value) + head * size + at_head;
+    const int64_t stride = static_cast<int64_t>(p.kv_heads) * size;
+    T* cache = static_cast<T*>(is_key ? p.key_cache : p.value_cache);
+    float* sum = p.pool_state + static_cast<int64_t>(slot) * p.kv_heads * per_head + c;
     auto pool_block = [&](int block) {
         const int from = max(block * p.pool, length), to = min((block + 1) * p.pool, end), at = p.window + block;
-        const bool complete = to == (block + 1) * p.pool;
-        for (int c = threadIdx.x; c < p.kv_heads * per_head; c += blockDim.x) {
-            const int head = c / per_head, d = c - head * per_head;
-            const bool is_key = d < p.dim;
-            const T* source = is_key ? static_cast<const T*>(p.key) + head * p.dim + d : static_cast<const T*>(p.value) + head * p.vdim + d - p.dim;
-            const int64_t stride = p.kv_heads * (is_key ? p.dim : p.vdim);
-            float* sum = p.pool_state + static_cast<int64_t>(slot) * p.kv_heads * per_head + c;
-            float total = from > block * p.pool ? *sum : 0.0f;
-            for (int j = from; j < to; ++j) total += load_as_f32(source, (first + j - length) * stride);
-            if (!complete) *sum = total;
-            else if (at >= p.entries) continue;
-            else if (is_key) store_from_f32(static_cast<T*>(p.key_cache), p.entry_at(slot, head, at) * p.dim + d, total / static_cast<float>(p.pool));
-            else store_from_f32(static_cast<T*>(p.value_cache), p.entry_at(slot, head, at) * p.vdim + d - p.dim, total / static_cast<float>(p.pool));
+        Span<V> total{};
+        if (from > block * p.pool) total = load_span<V>(sum);
+#pragma unroll 8
+        for (int j = from; j < to; ++j) {
+            const T* row = source + (first + j - length) * stride;
+            if constexpr (V == 4 && sizeof(T) == 2) {
+                const uint2 q = __ldcg(reinterpret_cast<const uint2*>(row));
+                total.v[0] += bf16_lo(q.x); total.v[1] += bf16_hi(q.x); total.v[2] += bf16_lo(q.y); total.v[3] += bf16_hi(q.y);
+            } else {
+#pragma unroll
+                for (int i = 0; i < V; ++i) total.v[i] += load_as_f32(row, i);
+            }
         }
+        if (to < (block + 1) * p.pool) return store_span<V>(sum, total);
+#pragma unroll
+        for (int i = 0; i < V; ++i) total.v[i] /= static_cast<float>(p.pool);
+        if (at < p.entries) store_span<V>(cache + p.entry_at(slot, head, at) * size + at_head, total);
     };
     const int block = block0 + static_cast<int>(blockIdx.x);
     if (blockIdx.x == 0) {
@@ -455,9 +469,11 @@ __device__ __forceinline__ float denominator_factor(const ChunkParams& p, int he
 
 __device__ __forceinline__ void store_pair(const ChunkAttention& a, int row, int head, int column, float x, float y) {
     const int64_t at = row * a.out_stride + head * a.p.vdim + column;
-    if (a.p.gate_values) {
-        x *= value_gate(a.p, row, head, column);
-        y *= value_gate(a.p, row, head, column + 1);
+    if (a.p.gate_values) {   // (hardware exponential and division: an error near 1e-6, as in the weights)
+        const ChunkParams& p = a.p;
+        const float2 g = __ldg(reinterpret_cast<const float2*>(p.projected + row * p.stride + p.heads * p.dim + p.key_columns() + p.value_columns() + head * p.vdim + column));
+        x = __fdividef(x, 1.0f + exp2_fast(-kLog2e * g.x));
+        y = __fdividef(y, 1.0f + exp2_fast(-kLog2e * g.y));
     }
     if (a.out) *reinterpret_cast<float2*>(a.out + at) = make_float2(x, y);
     if (a.out_hi) {
@@ -810,14 +826,22 @@ template <int DV> __global__ void __launch_bounds__(128) talk_values_kernel(cons
 }
 
 // Between the two: scores -> softmax weights, mixed over the heads -> packed bf16 planes, in place.  grid (blocks of keys, positions,
-// sequences); two adjacent keys per thread, HEADS >= heads of them in registers.
-constexpr int kMixThreads = 128;
-template <int HEADS> __global__ void __launch_bounds__(kMixThreads) talk_mix_kernel(const __grid_constant__ ChunkAttention a) {
-    extern __shared__ __align__(16) float talk[];   // [heads][HEADS], columns past the heads zero
-    __shared__ float top[HEADS], inverse[HEADS];
+// sequences); a warp takes 32 keys of all heads at a time through the tensor cores: the matrix times the weights, both as two planes.
+// Lane l loads the four keys from 4 (l / 4) on, one for each of four products of eight keys; so column c of product j is key 4 c + j,
+// and every lane also ends with runs of four keys.  BLOCKS x 16 >= heads.
+constexpr int kMixThreads = 128, kMixKeys = 512;
+template <int BLOCKS> __global__ void __launch_bounds__(kMixThreads) talk_mix_kernel(const __grid_constant__ ChunkAttention a) {
+    constexpr bool kHold = BLOCKS <= 2;   // the matrix stays in registers
+    __shared__ uint32_t matrix[2][BLOCKS * BLOCKS * 4][32];   // planes of its fragments
+    __shared__ float top[BLOCKS * 16], inverse[BLOCKS * 16];
     const ChunkParams& p = a.p;
-    const int H = p.heads;
-    for (int c = threadIdx.x; c < H * HEADS; c += kMixThreads) talk[c] = c % HEADS < H ? __ldg(p.talk + (c / HEADS) * H + c % HEADS) : 0.0f;
+    const int H = p.heads, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int c = threadIdx.x; c < BLOCKS * BLOCKS * 4 * 32; c += kMixThreads) {
+        const int l = c & 31, part = (c >> 5) & 3, block = c >> 7;
+        const int to = block / BLOCKS * 16 + (l >> 2) + (part & 1) * 8, from = block % BLOCKS * 16 + (l & 3) * 2 + (part >> 1) * 8;
+        auto entry = [&](int g) { return to < H && g < H ? __ldg(p.talk + to * H + g) : 0.0f; };
+        pack_planes(entry(from), entry(from + 1), matrix[0][block * 4 + part][l], matrix[1][block * 4 + part][l]);
+    }
     grid_dependency_wait();
     grid_launch_dependents();
     const int sequence = a.first_sequence + blockIdx.z, position = a.begin + blockIdx.y;
@@ -826,10 +850,11 @@ template <int HEADS> __global__ void __launch_bounds__(kMixThreads) talk_mix_ker
     int keys;
     if (a.step) keys = p.entries_seen(a.rows.lengths[__ldg(a.rows.slot + sequence)]);
     else keys = TileRows(a, sequence, 0, a.begin + (position - a.begin) / a.positions_per_tile * a.positions_per_tile).keys;
-    keys = (keys + 63) / 64 * 64;   // (the tables are written in whole tiles)
-    if (static_cast<int>(blockIdx.x) * kMixThreads * 2 >= keys) return;
+    keys = min((keys + 63) / 64 * 64, (static_cast<int>(blockIdx.x) + 1) * kMixKeys);   // (the tables are written in whole tiles)
+    const int key0 = blockIdx.x * kMixKeys;
+    if (key0 >= keys) return;
     const int64_t row = table_row(a, sequence, position) * H;
-    for (int h = threadIdx.x; h < HEADS; h += kMixThreads) {
+    for (int h = threadIdx.x; h < BLOCKS * 16; h += kMixThreads) {
         float high = -INFINITY, total = 0.0f;
         if (h < H) {
             const float* ml = a.table_ml + (row + h) * a.splits * 2;
@@ -840,33 +865,83 @@ template <int HEADS> __global__ void __launch_bounds__(kMixThreads) talk_mix_ker
         inverse[h] = h < H ? 1.0f / total : 0.0f;
     }
     __syncthreads();
-    const int n = (blockIdx.x * kMixThreads + threadIdx.x) * 2;
-    if (n >= keys) return;
-    float* at = a.table + row * a.pitch + n;
-    float2 w[HEADS];
+    uint32_t held[2][kHold ? BLOCKS * BLOCKS : 1][4];
+    if constexpr (kHold) {
 #pragma unroll
-    for (int h = 0; h < HEADS; ++h) {
-        w[h] = h < H ? *reinterpret_cast<const float2*>(at + h * a.pitch) : make_float2(-INFINITY, -INFINITY);
+        for (int plane = 0; plane < 2; ++plane)
+#pragma unroll
+            for (int m = 0; m < BLOCKS * BLOCKS; ++m)
+#pragma unroll
+                for (int part = 0; part < 4; ++part) held[plane][m][part] = matrix[plane][m * 4 + part][lane];
     }
+    const int head0 = (lane & 3) * 2;
+    for (int n = key0 + warp * 32; n < keys; n += 4 * 32) {
+        float* const at = a.table + row * a.pitch + n;
+        uint32_t hi[BLOCKS][4][2], lo[BLOCKS][4][2];
+        float4 score[BLOCKS][4];
 #pragma unroll
-    for (int h = 0; h < HEADS; ++h) {
-        const float high = top[h], factor = inverse[h];
-        w[h] = make_float2(exp2_fast(w[h].x - high) * factor, exp2_fast(w[h].y - high) * factor);
-    }
-    for (int h = 0; h < H; ++h) {
-        float2 sum = make_float2(0.0f, 0.0f);
-        const float4* t = reinterpret_cast<const float4*>(talk + h * HEADS);
+        for (int k = 0; k < BLOCKS; ++k)
 #pragma unroll
-        for (int g = 0; g < HEADS / 4; ++g) {
-            const float4 v = t[g];
-            sum.x = fmaf(v.x, w[4 * g].x, sum.x); sum.y = fmaf(v.x, w[4 * g].y, sum.y);
-            sum.x = fmaf(v.y, w[4 * g + 1].x, sum.x); sum.y = fmaf(v.y, w[4 * g + 1].y, sum.y);
-            sum.x = fmaf(v.z, w[4 * g + 2].x, sum.x); sum.y = fmaf(v.z, w[4 * g + 2].y, sum.y);
-            sum.x = fmaf(v.w, w[4 * g + 3].x, sum.x); sum.y = fmaf(v.w, w[4 * g + 3].y, sum.y);
+            for (int i = 0; i < 4; ++i) {
+                const int h = k * 16 + head0 + (i & 1) + (i >> 1) * 8;
+                score[k][i] = h < H ? __ldcg(reinterpret_cast<const float4*>(at + h * a.pitch + (lane >> 2) * 4)) : make_float4(-INFINITY, -INFINITY, -INFINITY, -INFINITY);
+            }
+#pragma unroll
+        for (int k = 0; k < BLOCKS; ++k) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int h = k * 16 + head0 + (i & 1) + (i >> 1) * 8;
+                const float high = top[h], factor = inverse[h];
+                float4& w = score[k][i];
+                w = make_float4(exp2_fast(w.x - high) * factor, exp2_fast(w.y - high) * factor, exp2_fast(w.z - high) * factor, exp2_fast(w.w - high) * factor);
+            }
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const float4 u = score[k][2 * i], v = score[k][2 * i + 1];
+                pack_planes(u.x, v.x, hi[k][0][i], lo[k][0][i]);
+                pack_planes(u.y, v.y, hi[k][1][i], lo[k][1][i]);
+                pack_planes(u.z, v.z, hi[k][2][i], lo[k][2][i]);
+                pack_planes(u.w, v.w, hi[k][3][i], lo[k][3][i]);
+            }
         }
-        uint32_t hi, lo;
-        pack_planes(sum.x, sum.y, hi, lo);
-        *reinterpret_cast<uint2*>(at + h * a.pitch) = make_uint2(__byte_perm(hi, lo, 0x5410), __byte_perm(hi, lo, 0x7632));
+#pragma unroll
+        for (int m = 0; m < BLOCKS; ++m) {
+            float c[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) c[j][i] = 0.0f;
+#pragma unroll
+            for (int k = 0; k < BLOCKS; ++k) {
+                uint32_t t_hi[4], t_lo[4];
+#pragma unroll
+                for (int part = 0; part < 4; ++part) {
+                    t_hi[part] = kHold ? held[0][kHold ? m * BLOCKS + k : 0][part] : matrix[0][(m * BLOCKS + k) * 4 + part][lane];
+                    t_lo[part] = kHold ? held[1][kHold ? m * BLOCKS + k : 0][part] : matrix[1][(m * BLOCKS + k) * 4 + part][lane];
+                }
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    mma_16816(c[j], t_hi, hi[k][j][0], hi[k][j][1]);
+                    mma_16816(c[j], t_hi, lo[k][j][0], lo[k][j][1]);
+                    mma_16816(c[j], t_lo, hi[k][j][0], hi[k][j][1]);
+                }
+            }
+            // (every lane's loads of these keys are behind the products)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int h = m * 16 + (lane >> 2) + half * 8;
+                if (h >= H) continue;
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    uint32_t first_hi, first_lo, last_hi, last_lo;
+                    pack_planes(c[0][half * 2 + i], c[1][half * 2 + i], first_hi, first_lo);
+                    pack_planes(c[2][half * 2 + i], c[3][half * 2 + i], last_hi, last_lo);
+                    *reinterpret_cast<uint4*>(at + h * a.pitch + (head0 + i) * 4) =
+                        make_uint4(__byte_perm(first_hi, first_lo, 0x5410), __byte_perm(first_hi, first_lo, 0x7632), __byte_perm(last_hi, last_lo, 0x5410),
+                                   __byte_perm(last_hi, last_lo, 0x7632));
+                }
+            }
+        }
     }
 }
 
@@ -1346,6 +1421,7 @@ template <class T> __global__ void __launch_bounds__(kTalkThreads) talk_generic_
 
 bool chunk_takes_mma(const ChunkParams& p, int dtype, int64_t out_stride) {
     return dtype == B200_BF16 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.dim <= 256 && p.vdim <= 256 && (out_stride & 1) == 0
+        && (!p.gate_values || ((p.stride & 1) == 0 && (reinterpret_cast<uintptr_t>(p.projected) & 7) == 0))
         && ((reinterpret_cast<uintptr_t>(p.key_cache) | reinterpret_cast<uintptr_t>(p.value_cache)) & 15) == 0;
 }
 
@@ -1373,14 +1449,9 @@ template <int DV> int launch_talk_values(const ChunkAttention& a, int sequences,
     return cuda_status(launch_dependent(kernel, tile_grid(a, sequences), dim3(128), ValueShape<DV>::kSmem, stream, a), "talk_values_kernel launch");
 }
 int launch_talk_mix(const ChunkAttention& a, int sequences, cudaStream_t stream) {
-    auto launch = [&](auto kernel, int heads) {
-        const dim3 grid(static_cast<unsigned>((a.pitch + 2 * kMixThreads - 1) / (2 * kMixThreads)), static_cast<unsigned>(a.span), static_cast<unsigned>(sequences));
-        return cuda_status(launch_dependent(kernel, grid, dim3(kMixThreads), static_cast<size_t>(a.p.heads) * heads * 4, stream, a), "talk_mix_kernel launch");
-    };
-    if (a.p.heads <= 8) return launch(talk_mix_kernel<8>, 8);
-    if (a.p.heads <= 16) return launch(talk_mix_kernel<16>, 16);
-    if (a.p.heads <= 32) return launch(talk_mix_kernel<32>, 32);
-    return launch(talk_mix_kernel<64>, 64);
+    auto kernel = a.p.heads <= 16 ? talk_mix_kernel<1> : a.p.heads <= 32 ? talk_mix_kernel<2> : a.p.heads <= 48 ? talk_mix_kernel<3> : talk_mix_kernel<4>;
+    const dim3 grid(static_cast<unsigned>((a.pitch + kMixKeys - 1) / kMixKeys), static_cast<unsigned>(a.span), static_cast<unsigned>(sequences));
+    return cuda_status(launch_dependent(kernel, grid, dim3(kMixThreads), 0, stream, a), "talk_mix_kernel launch");
 }
 
 int encode_slots(CUtensorMap* map, const void* base, int64_t rows, int columns) {
@@ -1437,9 +1508,10 @@ template <class Launch> int pick_head_size(int size, Launch&& launch) {
     return launch(integral_constant<int, 256>{});
 }
 
-// Mixed heads: positions and sequences whose tables are filled at a time.  Longer passes go in portions whose tables stay in L2.
-constexpr size_t kTableBytes = size_t{72} << 20;
-constexpr int kMostMixedHeads = 64;
+// Mixed heads: positions and sequences whose tables are filled at a time; longer passes go in portions.  (Portions whose tables stay in L2
+// leave the SMs half empty and are slower than tables that do not.)
+constexpr size_t kTableBytes = size_t{768} << 20;
+constexpr int kMostMixedHeads = 64;   // (talk_mix_kernel)
 struct TalkPlan { int64_t pitch; int span, sequences; };
 TalkPlan talk_plan(const ChunkParams& p, int sequences, int max_count, int max_length) {
     const bool step = max_count == 1;
@@ -1451,7 +1523,8 @@ TalkPlan talk_plan(const ChunkParams& p, int sequences, int max_count, int max_l
     plan.span = step ? 1 : (max_count + tile - 1) / tile * tile;
     plan.sequences = sequences;
     if (step) return plan;
-    const size_t per_tile = static_cast<size_t>(tile) * p.heads * static_cast<size_t>(plan.pitch) * 4, tiles = std::max<size_t>(1, kTableBytes / per_tile);
+    const size_t per_tile = static_cast<size_t>(tile) * p.heads * static_cast<size_t>(plan.pitch) * 4;
+    const size_t tiles = std::max<size_t>(1, (p.table_bytes ? p.table_bytes : kTableBytes) / per_tile);
     plan.sequences = static_cast<int>(std::min<size_t>(static_cast<size_t>(sequences), tiles));
     plan.span = static_cast<int>(std::min<size_t>(static_cast<size_t>(plan.span), tiles / static_cast<size_t>(plan.sequences) * static_cast<size_t>(tile)));
     return plan;
@@ -1579,10 +1652,15 @@ extern "C" int b200_chunk_attention(const b200_chunk_args* args, const b200_rows
     if (!p.appends_first(a.step) && (!p.key || !p.value)) { set_error("b200_chunk_attention: longer passes need key and value workspaces"); return B200_BAD_ARGUMENT; }
     int status = B200_OK;
     if (!a.step && p.pool > 0) {
-        auto pool = args->dtype == B200_BF16 ? chunk_pool_kernel<__nv_bfloat16> : chunk_pool_kernel<float>;
+        const bool quads = p.dim % 4 == 0 && p.vdim % 4 == 0
+            && ((reinterpret_cast<uintptr_t>(p.key) | reinterpret_cast<uintptr_t>(p.value) | reinterpret_cast<uintptr_t>(p.key_cache)
+                 | reinterpret_cast<uintptr_t>(p.value_cache) | reinterpret_cast<uintptr_t>(p.pool_state)) & 15) == 0;
+        auto pool = args->dtype == B200_BF16 ? (quads ? chunk_pool_kernel<__nv_bfloat16, 4> : chunk_pool_kernel<__nv_bfloat16, 1>)
+                                             : (quads ? chunk_pool_kernel<float, 4> : chunk_pool_kernel<float, 1>);
         if (a.rows.sequences > 65535) { set_error("grouped attention: at most 65535 sequences in one pass"); return B200_UNSUPPORTED; }
-        const dim3 grid(static_cast<unsigned>(a.rows.max_count / p.pool + 2), static_cast<unsigned>(a.rows.sequences));
-        status = cuda_status(launch_dependent(pool, grid, dim3(128), 0, s, p, a.rows), "chunk_pool_kernel launch");
+        const int columns = p.kv_heads * (p.dim + p.vdim), per_block = kPoolThreads * (quads ? 4 : 1);
+        const dim3 grid(static_cast<unsigned>(a.rows.max_count / p.pool + 2), static_cast<unsigned>(a.rows.sequences), static_cast<unsigned>((columns + per_block - 1) / per_block));
+        status = cuda_status(launch_dependent(pool, grid, dim3(kPoolThreads), 0, s, p, a.rows), "chunk_pool_kernel launch");
         if (status != B200_OK) return status;
     }
     if (p.talk && !talk_takes_mma(p, args->dtype, out_stride)) {

@@ -183,6 +183,20 @@ def sandwich_config(width: int, layers: int, ff: int, heads: int, kv_heads: int,
     return config
 
 
+def postnorm_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, experts: int, delta_heads: int, top: int = 2, window: int = 512, pool: int = 16,
+                    keep: int = 8, vocab: int = 32000) -> dict:
+    """Post-norm decoder of a real model's layer sizes: the delta rule, the window with pooled blocks and the window with mixed heads in turn, a
+    mixture behind each of them, `top` experts with a dense feed-forward's weights."""
+    dim = width // heads
+    sizes = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // top}}
+    mixers = (("delta", {"heads": delta_heads, "kv_heads": delta_heads // 2, "dim": 128, "vdim": 128, "conv": 4}),
+              ("attention", {**sizes, "mask": {"size": window, "pool": pool}, "rot": {"base": 500000.0, "dims": dim // 2}}),
+              ("attention_2", {**sizes, "mask": {"size": window, "keep_first": keep}, "rot": {"base": 10000.0, "dims": dim // 2, "scaling": {"factor": 4.0}}}))
+    return {"architecture": "Rizovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+            "layers": [{"type": mixers[i % 3][0], "mixer": mixers[i % 3][1], "mlp": mlp} for i in range(layers)]}
+
+
 def transformer_config(width: int, layers: int, ff: int, heads: int, kv_heads: int, context: int, vocab: int = 32000) -> dict:
     return {"architecture": "TransformerDecoder", "vocab": vocab, "layers": layers, "width": width, "heads": heads, "kv_heads": kv_heads,
             "ff": ff, "context": context, "tied": 1}
@@ -207,6 +221,13 @@ SANDWICH_SIZES = {
     "1k": (dict(width=1024, layers=12, ff=4096, heads=16, kv_heads=4, experts=16, lightning_heads=8), HYBRID_SIZES["1k"][1]),
     "2k": (dict(width=2048, layers=16, ff=8192, heads=32, kv_heads=8, experts=16, lightning_heads=16), HYBRID_SIZES["2k"][1]),
     "4k": (dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8, experts=8, lightning_heads=32), HYBRID_SIZES["4k"][1]),
+}
+
+# (post-norm, sandwich) arguments: the closest design, of equal width, heads, layers and experts
+POSTNORM_SIZES = {
+    "1k": (dict(width=1024, layers=12, ff=4096, heads=16, kv_heads=4, experts=16, delta_heads=8), SANDWICH_SIZES["1k"][0]),
+    "2k": (dict(width=2048, layers=16, ff=8192, heads=32, kv_heads=8, experts=16, delta_heads=16), SANDWICH_SIZES["2k"][0]),
+    "4k": (dict(width=4096, layers=8, ff=14336, heads=32, kv_heads=8, experts=8, delta_heads=32), SANDWICH_SIZES["4k"][0]),
 }
 
 

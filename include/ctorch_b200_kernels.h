@@ -492,6 +492,7 @@ typedef struct b200_chunk_args {
     int32_t norm_values;           /* 1: every head's value is divided by its root mean square */
     int32_t gate_values;           /* 1 (with no_gate): heads*vdim g columns, sigmoid(g) of every value in place of the head's */
     const float* talk;             /* [heads][heads] or NULL: softmax weights of head h <- sum over g of talk[h][g] times those of head g (no sink) */
+    int64_t table_bytes;           /* mixed heads: most bytes of scores that are kept at a time; 0: the default */
 } b200_chunk_args;
 /* Norms of queries and keys, before the rotation: RMS over all heads of the row at once with the weights q_norm and k_norm; none; RMS per head,
  * with weights q_norm and k_norm [dim] for every head, or without (NULL). */

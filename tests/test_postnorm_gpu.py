@@ -226,10 +226,12 @@ def test_mixed_heads_in_portions_of_the_tables():
     """A pass whose tables of scores exceed what is kept at a time: portions of positions, and of sequences."""
     k = Windowed(2, 32, 4, 16, 16, "bf16", 300, 0, 5, slots=40, capacity=800, seed=4)
     rng = np.random.default_rng(5)
+    k.a.table_bytes = 24 << 20
     for totals in ([700, 431, 640], [40] * 36):
         data = [rng.normal(size=(t, k.stride)) for t in totals]
         slots = rng.permutation(40)[:len(totals)].tolist()
         got = k.attend(Pass(totals, slots, [0] * 40), np.concatenate(data), 800)
+        assert k.scratch < 26 << 20
         at = 0
         for i, r in enumerate(data):
             if len(totals) < 9 or i % 7 == 0:
