@@ -205,8 +205,7 @@ void HybridPlan::reserve_attention(Index rows, Index max_length, const HybridCac
             most_experts = std::max(most_experts, c.experts);
         }
     }
-    if (query == 0) return;
-    grow(chunk_query_, {rows, query}, owner_.dtype());
+    if (query) grow(chunk_query_, {rows, query}, owner_.dtype());
     if (key) { grow(chunk_key_, {rows, key}, owner_.dtype()); grow(chunk_value_, {rows, value}, owner_.dtype()); }
     if (slots) {
         grow(chosen_, {rows, slots}, DType::f32);   // int32 payload
@@ -229,7 +228,7 @@ void HybridPlan::reserve_attention(Index rows, Index max_length, const HybridCac
             else streamed = true;
         }
     }
-    grow(scratch_, {static_cast<Index>(scratch / 4 + 1)}, DType::f32);
+    if (scratch) grow(scratch_, {static_cast<Index>(scratch / 4 + 1)}, DType::f32);
     if (grouped) grow(expert_scratch_, {static_cast<Index>(grouped / 4)}, DType::f32);
     if (streamed) grow(expert_act_, {rows, act}, DType::f32);
     grouped_ = grouped > 0;

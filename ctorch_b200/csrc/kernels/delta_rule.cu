@@ -431,7 +431,7 @@ int launch_delta_step(const SsmParams& p, const RowsView& rows, cudaStream_t str
     const size_t smem = sizeof(float) * (((p.vdim + 2 * p.state + 3) & ~3) + 2 * kStepThreads * wide + std::min(p.vdim, kStepThreads * wide));
     if (smem > 200 * 1024) { set_error("delta rule: a head of %d x %d values does not fit shared memory", p.state, p.vdim); return B200_UNSUPPORTED; }
     auto kernel = quads ? delta_step_kernel<4> : delta_step_kernel<1>;
-    if (smem > 48 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    if (smem > 46 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(rows.sequences)), dim3(kStepThreads), smem, stream, p, rows),
                        "delta_step_kernel launch");
 }

@@ -802,7 +802,7 @@ int b200_latent_attention(const b200_latent_args* args, const b200_rows* pass, c
     if (!latent_takes_mma(p)) {
         const size_t smem = sizeof(float) * (p.width + p.rank + kGenericKeys + 32 + 2) + sizeof(int64_t) * kGenericKeys;
         if (smem > 200 * 1024 || a.rows.rows > 65535) { set_error("latent attention: sizes outside the generic kernel"); return B200_UNSUPPORTED; }
-        if (smem > 48 * 1024) B200_CUDA(cudaFuncSetAttribute(latent_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+        if (smem > 46 * 1024) B200_CUDA(cudaFuncSetAttribute(latent_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
         return cuda_status(launch_dependent(latent_generic_kernel, dim3(static_cast<unsigned>(p.heads), static_cast<unsigned>(a.rows.rows)),
                                             dim3(kGenericThreads), smem, as_stream(stream), a), "latent_generic_kernel launch");
     }

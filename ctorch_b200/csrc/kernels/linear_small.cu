@@ -171,7 +171,8 @@ template <class W, int R, int EPI, bool VECTOR> int launch(const LinearParams& p
     const int chunk = p.in < kChunk ? p.in : kChunk;
     const size_t smem = sizeof(float) * R * (((chunk + 7) >> 3) << 3);
     auto kernel = linear_small_kernel<W, R, EPI, VECTOR>;
-    if (smem > 48 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    // (48 KB without the attribute, the kernel's static arrays included)
+    if (smem > 46 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     kernel<<<dim3(row_tiles, feature_blocks), kThreads, smem, stream>>>(p);
     return cuda_status(cudaGetLastError(), "linear_small_kernel launch");
 }

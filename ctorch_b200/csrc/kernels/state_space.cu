@@ -786,7 +786,7 @@ int b200_ssm_forward(const b200_ssm_args* a, const b200_rows* pass, void* stream
         const size_t smem = sizeof(float) * (((a->vdim + 2 * a->state + 3) & ~3) + kStepThreads * (quads ? 4 : 1));
         if (smem > 200 * 1024) { set_error("b200_ssm_forward: a head of %d x %d values does not fit shared memory", a->state, a->vdim); return B200_UNSUPPORTED; }
         auto kernel = quads ? ssm_step_kernel<4> : ssm_step_kernel<1>;
-        if (smem > 48 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+        if (smem > 46 * 1024) B200_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
         return cuda_status(launch_dependent(kernel, dim3(static_cast<unsigned>(a->heads), static_cast<unsigned>(rows.sequences)), dim3(kStepThreads),
                                             smem, s, p, rows), "ssm_step_kernel launch");
     }

@@ -56,6 +56,9 @@ CASES = {
     # the larger head sizes of the tensor-core attention, a state beyond the narrow scan
     "deep": config(96, [mixing(2, 1, 192, 128, 30, 4, moe(8, 1, 48), dims=32), pooled(2, 2, 256, 256, 24, 5, None), delta(3, 1, 264, 128, 4, moe(6, 2, 40)), pooled(3, 1, 72, 96, 63, 2, None, dims=10)],
                    vocab=131),
+    # the recurrence alone, with mixtures; then attention alone, without
+    "recurrent": config(40, [delta(4, 4, 96, 16, 3, moe(2, 2, 64)), delta(9, 3, 40, 32, 4, moe(2, 1, 16))], vocab=64, weights_of=((2, 0),)),
+    "attending": config(48, [pooled(2, 2, 32, 32, 12, 6, None), mixing(4, 1, 16, 16, 9, 2, None)], vocab=70),
     # planes between the kernels, but head sizes and experts without vector loads; an odd vocabulary
     "uneven": config(64, [mixing(4, 2, 20, 12, 25, 6, moe(5, 2, 21), dims=6), delta(4, 4, 10, 6, 3, moe(3, 1, 9)), pooled(4, 1, 12, 18, 31, 6, moe(6, 2, 24), dims=6)], vocab=97, factor=0.5),
 }

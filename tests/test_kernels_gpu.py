@@ -96,7 +96,7 @@ def run_linear(x, w, epilogue=0, norm=None, eps=1e-5, residual=None, qkv=None, o
 
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
 @pytest.mark.parametrize("rows,inner,out", [(1, 256, 256), (2, 768, 1280), (3, 64, 97), (5, 2048, 768), (8, 4096, 130),
-                                            (11, 768, 514), (16, 768, 2048), (4, 12, 8), (1, 6152, 66), (19, 72, 40)])
+                                            (11, 768, 514), (16, 768, 2048), (4, 12, 8), (1, 6152, 66), (19, 72, 40), (9, 1536, 20)])
 def test_linear_store(dtype, rows, inner, out):
     rng = np.random.default_rng(rows * 1000 + inner + out)
     x = rng.standard_normal((rows, inner), dtype=np.float32)

@@ -515,7 +515,7 @@ def test_greedy_generation_equals_the_statement(name):
         assert margin > 1e-4 and list(row) == want
 
 
-@pytest.mark.parametrize("name, batch", [("mixed", 1), ("mixed", 20), ("wide", 40), ("plain", 150), ("uneven", 3), ("deep", 30), ("ones", 2)])
+@pytest.mark.parametrize("name, batch", [("mixed", 1), ("mixed", 20), ("wide", 40), ("plain", 150), ("uneven", 3), ("deep", 30), ("ones", 2), ("recurrent", 9), ("attending", 3)])
 def test_bf16_generation_feeds_back_its_own_choice(name, batch):
     """bf16 loop (fused logits + choice; streaming and dense projections; streamed and grouped experts): replaying its tokens gives
     logits whose best is the token chosen next, and the logits asked for on demand are those."""
