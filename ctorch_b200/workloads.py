@@ -192,8 +192,8 @@ def postnorm_config(width: int, layers: int, ff: int, heads: int, kv_heads: int,
     mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // top}}
     mixers = (("delta", {"heads": delta_heads, "kv_heads": delta_heads // 2, "dim": 128, "vdim": 128, "conv": 4}),
               ("attention", {**sizes, "mask": {"size": window, "pool": pool}, "rot": {"base": 500000.0, "dims": dim // 2}}),
-              ("attention_2", {**sizes, "mask": {"size": window, "keep_first": keep}, "rot": {"base": 10000.0, "dims": dim // 2, "scaling": {"factor": 4.0}}}))
-    return {"architecture": "Rizovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.7,
+              ("attention_2", {**sizes, "mask": {"size": window, "keep_first": keep}, "rot": {"base": 10000.0, "dims": dim // 2, "scaling": {"factor": 8.0}}}))
+    return {"architecture": "Rizovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.8,
             "layers": [{"type": mixers[i % 3][0], "mixer": mixers[i % 3][1], "mlp": mlp} for i in range(layers)]}
 
 
